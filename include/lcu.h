@@ -56,7 +56,20 @@ typedef enum {
     LCU_W_GATE_UP = 5,   /* blk.N.ffn_gate_up   [2*di, d]         gate|up   */
     LCU_W_DOWN = 6,      /* blk.N.ffn_down      [d, di]                     */
     LCU_W_OUT_NORM = 7,  /* output_norm         [d]                         */
-    LCU_W_LM_HEAD = 8    /* output.weight       [vocab, d]                  */
+    LCU_W_LM_HEAD = 8,   /* output.weight       [vocab, d]                  */
+    /* Models described layer by layer (lcu_ctx_create_layers); packed shapes from lcu_layer_weight_shape.  All bf16
+     * except LCU_W_SCALARS; EMBD, OUT_NORM (one f32 gain) and LM_HEAD are shared with the kinds above. */
+    LCU_W_LAT_IN = 16,   /* rows: query latent | latent | head gates        */
+    LCU_W_Q_NORM = 17,   /* norm weight of the query latent                 */
+    LCU_W_KV_NORM = 18,  /* norm weight of the latent                       */
+    LCU_W_UQ = 19,       /* latent -> queries, [heads][dim] rows            */
+    LCU_W_UKT = 20,      /* key map transposed per head: [heads][latent][dim] */
+    LCU_W_UKV = 21,      /* key map rows [heads][dim], then value map rows [heads][v_dim] */
+    LCU_W_LAT_OUT = 22,  /* output projection, [heads][v_dim] columns       */
+    LCU_W_UP = 23,       /* feed-forward up                                 */
+    LCU_W_FF_DOWN = 24,  /* feed-forward down                               */
+    LCU_W_SHIFT = 25,    /* token-shift weights                             */
+    LCU_W_SCALARS = 26   /* f32: mixer norm gain, feed-forward norm gain, activation p, q */
 } lcu_weight_kind;
 
 /* Model description: the fields llama.cu/src/model/mod.rs:61-78 reads from GGUF metadata.
@@ -72,6 +85,25 @@ typedef struct {
     int32_t max_tokens;   /* largest round in tokens; 0 = 1024 (NTOKS, exec/engine.rs:68)  */
     int32_t max_seqs;     /* most requests in one round; 0 = 64                            */
 } lcu_model_desc;
+
+/* Mixers and activations of layered models */
+enum { LCU_MIX_LATENT = 1 };  /* latent attention: per-head keys and values are linear maps of one cached vector per token */
+enum { LCU_ACT_XIELU = 1 };
+
+/* One layer of a model described layer by layer: x += norm(mixer(h)), x += norm(ff(x)), both norms RMS with a single gain
+ * on the sublayer's OUTPUT, h = x or (token_shift) x mixed per coordinate with the previous token's x.  (No counterpart in
+ * the reference, whose models are LLaMA-shaped.) */
+typedef struct {
+    int32_t mixer;       /* LCU_MIX_LATENT                                                      */
+    int32_t heads, dim, v_dim; /* query/key and value size per head                             */
+    int32_t q_rank, kv_rank;   /* query latent, cached latent                                   */
+    int32_t out_gate;    /* 1: head h's output is multiplied by sigmoid(W_g h)_h                 */
+    int32_t token_shift; /* 1: the mixer reads h + (previous h - h) * shift (recurrent state)    */
+    int32_t ff;          /* feed-forward width, 0: the layer has none                            */
+    int32_t ff_act;      /* LCU_ACT_XIELU                                                        */
+    int32_t weights_of;  /* -1, or the layer whose tensors this one uses (own cache and state)   */
+    float scale;         /* of the attention scores                                              */
+} lcu_layer_desc;
 
 /* == `KVPair` (llama.cu/src/op/random_sample/mod.rs:29-36) == cub::KeyValuePair<int,half> */
 typedef struct {
@@ -107,6 +139,15 @@ LCU_API int lcu_version(void);
 LCU_API int lcu_ctx_create(const lcu_model_desc *desc, int device, int tp_rank, int tp_size, void *nccl_comm,
                    lcu_ctx **out);
 LCU_API int lcu_ctx_destroy(lcu_ctx *ctx);
+/* A context for a model described layer by layer: desc gives n_layers, d, vocab, nctx, eps, act_dtype (LCU_BF16, or LCU_F32:
+ * every operation in true 32-bit arithmetic), weight_dtype (LCU_BF16), page_tokens, max_tokens, max_seqs; its other fields are
+ * ignored.  Pages hold page_tokens latents of every layer; sequences of models with token shift also take one of max_seqs
+ * recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
+ * graphs, round builder, sampling).  One GPU.  (No counterpart in the reference.) */
+LCU_API int lcu_ctx_create_layers(const lcu_model_desc *desc, const lcu_layer_desc *layers, int device, lcu_ctx **out);
+/* Packed (zero-padded) shape of one weight of a layered context; layer is ignored for EMBD, OUT_NORM and LM_HEAD.
+ * LCU_ERR_INVALID when the layer has no such weight. */
+LCU_API int lcu_layer_weight_shape(const lcu_ctx *ctx, int layer, int kind, int *rows_out, int *cols_out);
 /* Registers a caller-owned device tensor (weights stay where `load_weight` put them,
  * load/mod.rs:23-67).  `bytes` must equal the per-rank size for that kind.  Q8_0 linear
  * weights are passed in the plane layout produced by lcu_repack_q8_0. */
@@ -144,6 +185,9 @@ LCU_API int lcu_seq_create(lcu_ctx *ctx, int *seq_out);          /* == KVCache::
 LCU_API int lcu_seq_resize(lcu_ctx *ctx, int seq, uint32_t len); /* == KVCache::update: grows or shrinks */
 LCU_API int lcu_seq_len(const lcu_ctx *ctx, int seq);            /* tokens currently backed by pages */
 LCU_API int lcu_seq_free(lcu_ctx *ctx, int seq);
+/* Largest position <= len from which the sequence can be continued: len itself when everything a model keeps is per token,
+ * the position its recurrent state covers (or 0) otherwise.  lcu_step refuses any other position with LCU_ERR_STATE. */
+LCU_API int lcu_seq_resumable(const lcu_ctx *ctx, int seq, uint32_t len);
 
 /* ------------------------------------------------------------------ one round
  * == the body of `Worker::lead`'s loop from `load_inputs` to `output_head.launch`
@@ -163,9 +207,17 @@ LCU_API int lcu_seq_free(lcu_ctx *ctx, int seq);
 LCU_API int lcu_step(lcu_ctx *ctx, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens,
              const lcu_sample_args *args, const float *randoms, const uint32_t *fast_map, int n_fast,
              lcu_kv_pair *out_dev);
+/* One round that samples nothing: every layer as lcu_step, then the logits of the asked token slots (indices into `tokens`,
+ * any number from 0 to max_tokens, any order) as f32 rows of lcu_logits_stride() elements at `logits_dev`.  (No counterpart
+ * in the reference.) */
+LCU_API int lcu_step_logits(lcu_ctx *ctx, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens,
+                            int n_rows, const uint32_t *rows, float *logits_dev);
+/* Elements from one row of logits to the next (the vocabulary, padded for layered models). */
+LCU_API int lcu_logits_stride(const lcu_ctx *ctx);
 /* Device pointer to the logits of the last round, [n_req, vocab] in the activation dtype. */
 LCU_API const void *lcu_logits(const lcu_ctx *ctx);
-/* Device pointer to the hidden state (residual stream) of the last round, [n_tok, d]. */
+/* Device pointer to the hidden state (residual stream) of the last round, [n_tok, d]; layered models: f32, rows padded to
+ * a multiple of 64. */
 LCU_API const void *lcu_hidden(const lcu_ctx *ctx);
 /* Error word written by bounded device-side waits; 0 = none.  Synchronises `stream`.
  * Bits: 4 = a tcgen05 / TMA pipeline wait ran out, 16 = a peer never delivered its part of an all-reduce (or its head
@@ -184,7 +236,8 @@ LCU_API int lcu_set_wait_limit_us(lcu_ctx *ctx, long long us);
  * 4 down->next QKV, 5 last down->LM head; -1 = default), "gemv_ctas_per_sm" (1, 2; read at a shape's first launch),
  * "q8_rows" (1, 2, 4), "tc" (0: no tcgen05 kernel), "tc_block" (64, 128, 256), "tc_cluster" (0..2),
  * "p2p_scatter_ranks", "p2p_scatter_min", "gemv_lean_norm" (0: general RMSNorm prologue in the one-token GEMV),
- * "rms_pdl" (0: the stand-alone RMSNorm of batched rounds is a plain launch).
+ * "rms_pdl" (0: the stand-alone RMSNorm of batched rounds is a plain launch), "expand_min" (latent attention: fewest tokens of
+ * a portion that expands keys and values; 0 = from the operation counts, -1 = never).
  * `ctx` (may be NULL) drops its captured rounds.  A measurement aid without counterpart in the reference. */
 LCU_API int lcu_set_tuning(lcu_ctx *ctx, const char *key, long long value);
 /* Tensor parallelism over peer memory: 1 (default) = arg-max rounds shard the LM head by vocabulary rows — every rank

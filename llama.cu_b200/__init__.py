@@ -17,6 +17,8 @@ LIB_PATH = os.path.join(_HERE, "liblcu.so")
 
 F16, BF16, F32, Q8_0, U32 = 0, 1, 2, 3, 4
 W_EMBD, W_ATTN_NORM, W_QKV, W_O, W_FFN_NORM, W_GATE_UP, W_DOWN, W_OUT_NORM, W_LM_HEAD = range(9)
+(W_LAT_IN, W_Q_NORM, W_KV_NORM, W_UQ, W_UKT, W_UKV, W_LAT_OUT, W_UP, W_FF_DOWN, W_SHIFT, W_SCALARS) = range(16, 27)
+MIX_LATENT, ACT_XIELU = 1, 1
 LINEAR_KINDS = (W_QKV, W_O, W_GATE_UP, W_DOWN)
 NO_OUTPUT = 2**64 - 1  # LCU_ENGINE_NO_OUTPUT: a prefill chunk that samples nothing
 OK, ERR_INVALID, ERR_CUDA, ERR_OVERFLOW, ERR_NO_PAGES, ERR_STATE, ERR_COMM, ERR_TIMEOUT = 0, -1, -2, -3, -4, -5, -6, -7
@@ -32,6 +34,12 @@ class ModelDesc(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "d", "nh", "nkvh", "dh", "di", "vocab", "nctx")] + [
         ("eps", C.c_float), ("theta", C.c_float)] + [
         (n, C.c_int32) for n in ("act_dtype", "weight_dtype", "norm_dtype", "page_tokens", "max_tokens", "max_seqs")]
+
+
+class LayerDesc(C.Structure):
+    """One layer of a model described layer by layer (lcu_layer_desc)."""
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "v_dim", "q_rank", "kv_rank", "out_gate", "token_shift", "ff",
+                                         "ff_act", "weights_of")] + [("scale", C.c_float)]
 
 
 class KVPair(C.Structure):
@@ -77,6 +85,8 @@ _SIGNATURES = {
     "lcu_last_error_string": (C.c_char_p, []),
     "lcu_version": (C.c_int, []),
     "lcu_ctx_create": (C.c_int, [C.POINTER(ModelDesc), C.c_int, C.c_int, C.c_int, C.c_void_p, C.POINTER(C.c_void_p)]),
+    "lcu_ctx_create_layers": (C.c_int, [C.POINTER(ModelDesc), C.POINTER(LayerDesc), C.c_int, C.POINTER(C.c_void_p)]),
+    "lcu_layer_weight_shape": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.POINTER(C.c_int), C.POINTER(C.c_int)]),
     "lcu_ctx_destroy": (C.c_int, [C.c_void_p]),
     "lcu_set_weight": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_size_t]),
     "lcu_weight_bytes": (C.c_size_t, [C.c_void_p, C.c_int]),
@@ -95,6 +105,9 @@ _SIGNATURES = {
     "lcu_seq_resize": (C.c_int, [C.c_void_p, C.c_int, C.c_uint32]),
     "lcu_seq_len": (C.c_int, [C.c_void_p, C.c_int]),
     "lcu_seq_free": (C.c_int, [C.c_void_p, C.c_int]),
+    "lcu_seq_resumable": (C.c_int, [C.c_void_p, C.c_int, C.c_uint32]),
+    "lcu_step_logits": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.POINTER(Req), C.c_void_p, C.c_int, C.c_void_p, C.c_void_p]),
+    "lcu_logits_stride": (C.c_int, [C.c_void_p]),
     "lcu_step": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.POINTER(Req), C.c_void_p, C.POINTER(SampleArgs),
                            C.c_void_p, C.c_void_p, C.c_int, C.c_void_p]),
     "lcu_logits": (C.c_void_p, [C.c_void_p]),
@@ -246,13 +259,19 @@ class Context:
     (llama.cu/src/handle.rs, exec/group.rs, exec/output_head.rs).
     """
 
-    def __init__(self, desc: ModelDesc, device=0, tp_rank=0, tp_size=1, comm=None):
+    def __init__(self, desc: ModelDesc, device=0, tp_rank=0, tp_size=1, comm=None, layers=None):
         self.lib = load_library()
         self.desc = desc
         self.device = device
         self.tp_rank, self.tp_size = tp_rank, tp_size
         h = C.c_void_p()
-        check(self.lib.lcu_ctx_create(C.byref(desc), device, tp_rank, tp_size, comm, C.byref(h)))
+        self.layers = layers  # LayerDesc array of a model described layer by layer, None for the LLaMA family
+        if layers is not None:
+            if tp_size != 1:
+                raise ValueError("models described layer by layer run on one GPU")
+            check(self.lib.lcu_ctx_create_layers(C.byref(desc), layers, device, C.byref(h)))
+        else:
+            check(self.lib.lcu_ctx_create(C.byref(desc), device, tp_rank, tp_size, comm, C.byref(h)))
         self.h = h
         self._keep = []  # tensors registered with the library stay alive here
 
@@ -271,6 +290,11 @@ class Context:
     # ---- weights
     def weight_bytes(self, kind):
         return self.lib.lcu_weight_bytes(self.h, kind)
+
+    def layer_weight_shape(self, layer, kind):
+        r, c = C.c_int(), C.c_int()
+        check(self.lib.lcu_layer_weight_shape(self.h, layer, kind, C.byref(r), C.byref(c)))
+        return r.value, c.value
 
     def set_weight(self, layer, kind, tensor):
         nbytes = tensor.numel() * tensor.element_size()
@@ -322,6 +346,10 @@ class Context:
     def seq_len(self, seq):
         return self.lib.lcu_seq_len(self.h, seq)
 
+    def seq_resumable(self, seq, length):
+        """Largest position <= length the sequence can be continued from (recurrent state cannot be rolled back)."""
+        return self.lib.lcu_seq_resumable(self.h, seq, length)
+
     def seq_free(self, seq):
         check(self.lib.lcu_seq_free(self.h, seq))
 
@@ -340,17 +368,34 @@ class Context:
         check(self.lib.lcu_step(self.h, stream_ptr(stream), n, creqs, tokens.ctypes.data, cargs, ptr(rnd), ptr(fm),
                                 0 if fm is None else len(fm), ptr(out)))
 
+    def step_logits(self, reqs, tokens, rows, stream=None):
+        """One round that samples nothing: the f32 logits [len(rows), vocab] of the asked token slots (a device tensor, not
+        synchronised)."""
+        import torch
+        n = len(reqs)
+        creqs = (Req * n)(*[Req(*r) for r in reqs])
+        tokens = np.ascontiguousarray(tokens, dtype=np.uint32)
+        rows = np.ascontiguousarray(rows, dtype=np.uint32)
+        ld = self.lib.lcu_logits_stride(self.h)
+        out = torch.empty(max(len(rows), 1), ld, dtype=torch.float32, device=f"cuda:{self.device}")
+        check(self.lib.lcu_step_logits(self.h, stream_ptr(stream), n, creqs, tokens.ctypes.data, len(rows), rows.ctypes.data, out.data_ptr()))
+        return out[:len(rows), :self.desc.vocab]
+
     def logits(self, n_req):
         """The last round's logits [n_req, vocab] (a copy, after synchronising)."""
         import torch
         torch.cuda.synchronize(self.device)
-        return _view(self.lib.lcu_logits(self.h), n_req * self.desc.vocab, self.desc.act_dtype,
-                     self.device).view(n_req, self.desc.vocab).clone()
+        ld = self.lib.lcu_logits_stride(self.h)
+        return _view(self.lib.lcu_logits(self.h), n_req * ld, self.desc.act_dtype,
+                     self.device).view(n_req, ld)[:, :self.desc.vocab].clone()
 
     def hidden(self, n_tok):
         """The residual stream after the last layer of the last round, [n_tok, d] (a copy)."""
         import torch
         torch.cuda.synchronize(self.device)
+        if self.layers is not None:
+            ld = (self.desc.d + 63) // 64 * 64
+            return _view(self.lib.lcu_hidden(self.h), n_tok * ld, F32, self.device).view(n_tok, ld)[:, :self.desc.d].clone()
         return _view(self.lib.lcu_hidden(self.h), n_tok * self.desc.d, self.desc.act_dtype,
                      self.device).view(n_tok, self.desc.d).clone()
 
@@ -460,17 +505,18 @@ class GGuf:
 class _RawDevice:
     """Zero-copy view of library-owned device memory through __cuda_array_interface__."""
 
-    def __init__(self, address, n_elems):
-        self.__cuda_array_interface__ = {"shape": (n_elems,), "typestr": "<i2", "data": (address, False),
+    def __init__(self, address, n_elems, typestr):
+        self.__cuda_array_interface__ = {"shape": (n_elems,), "typestr": typestr, "data": (address, False),
                                          "version": 2}
 
 
 def _view(address, n_elems, dt, device):
     import torch
-    t = torch.as_tensor(_RawDevice(address, n_elems), device=f"cuda:{device}")
+    t = torch.as_tensor(_RawDevice(address, n_elems, "<f4" if dt == F32 else "<i2"), device=f"cuda:{device}")
     return t.view(torch_dtype(dt))
 
 
 from .model import (CONFIGS, ModelConfig, iter_synth_weights_torch, load_model, synth_weights_numpy,  # noqa: E402,F401
                     synth_weights_torch, tp_slice_numpy)
+from .layered import LayeredConfig, load_pretrained  # noqa: E402,F401
 from .host import Service, Session, StepRendezvous, generate, generate_continuous  # noqa: E402,F401

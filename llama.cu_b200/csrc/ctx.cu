@@ -12,6 +12,7 @@
 
 #include "attention.cuh"
 #include "common.cuh"
+#include "ctx.cuh"
 #include "gemv.cuh"
 #include "ops.cuh"
 #include "p2p.cuh"
@@ -62,96 +63,20 @@ using namespace lcu;
 
 // ------------------------------------------------------------------ context
 
-struct LayerWeights {
-    const void *attn_norm = nullptr, *qkv = nullptr, *o = nullptr, *ffn_norm = nullptr, *gate_up = nullptr,
-               *down = nullptr;
-};
-
-struct SeqState {
-    bool used = false;
-    uint32_t len = 0;  // tokens backed by pages
-    std::vector<int> pages;
-};
-
-struct StepGraph {
-    cudaGraphExec_t exec = nullptr;
-    int launches = 0;
-};
-
-struct lcu_ctx {
-    lcu_model_desc desc;
-    int device = 0, tp_rank = 0, tp_size = 1;
-    void *comm = nullptr;
-    int dt = LCU_F16;
-    // per-rank shapes
-    int nh_l = 0, nkvh_l = 0, di_l = 0, qd = 0, kvd = 0;
-    int max_tokens = 0, max_seqs = 0;
-
-    std::vector<LayerWeights> layers;
-    const void *embd = nullptr, *out_norm = nullptr, *lm_head = nullptr;
-    const float *sin_t = nullptr, *cos_t = nullptr;
-    float *own_tables = nullptr;
-
-    // KV pages
-    void *pool = nullptr;
-    bool own_pool = false;
-    KvGeom geom{};
-    int n_pages = 0, pt_stride = 0;
-    std::vector<int> free_pages;
-    std::vector<SeqState> seqs;
-
-    // arena (one allocation)
-    void *arena = nullptr;
-    void *x = nullptr, *q = nullptr, *att = nullptr, *act = nullptr, *logits = nullptr, *hbuf = nullptr;
-    void *sk_ws = nullptr;
-    unsigned *sk_tickets = nullptr;
-    size_t sk_ws_bytes = 0;
-    bool batched_ok = false;  // tensor-core path for rounds of more than 4 tokens
-    void *attn_scratch = nullptr, *sample_ws = nullptr;
-    size_t sample_ws_bytes = 0;
-    lcu_kv_pair *pre_pairs = nullptr;  // copy of the last round's output pairs (token feedback)
-    uint32_t *dev_status = nullptr;
-    unsigned char *desc_dev = nullptr;  // per-round descriptor
-    size_t desc_cap = 0;
-    // pinned staging ring for the descriptor
-    static constexpr int RING = 4;
-    unsigned char *desc_host[RING] = {nullptr, nullptr, nullptr, nullptr};
-    cudaEvent_t desc_event[RING] = {nullptr, nullptr, nullptr, nullptr};
-    bool desc_used[RING] = {false, false, false, false};
-    int ring_idx = 0;
-
-    // tensor parallelism over peer memory (set up by lcu_p2p_create / lcu_p2p_attach)
-    P2pState p2p;
-
-    // LM head sharded by vocabulary rows under tensor parallelism (peer-memory transport, arg-max rounds)
-    bool head_shard = true;           // lcu_set_head_sharding
-    lcu_kv_pair *head_local = nullptr;  // this rank's candidates
-    uint32_t sticky_status = 0;       // last value lcu_device_status read
-
-    bool use_graph = true;
-    std::map<std::vector<int>, StepGraph> graphs;
-    int last_launches = 0;
-    double last_bytes = 0;
-    int last_n_tok = 0, last_n_req = 0;
-};
-
-// offsets of the sections of a round descriptor (all 16-byte aligned)
-struct DescLayout {
-    size_t tokens, pos, tok_req, out_idx, fast_map, args, randoms, page_table, groups, total;
-};
-static DescLayout desc_layout(int n_tok, int n_req, int pt_stride) {
+static DescLayout desc_layout(int n_tok, int n_req, int n_out, int pt_stride) {
     DescLayout L;
     size_t o = 0;
     auto take = [&](size_t bytes) { size_t r = o; o += (bytes + 15) & ~(size_t)15; return r; };
     L.tokens = take((size_t)n_tok * 4);
     L.pos = take((size_t)n_tok * 4);
     L.tok_req = take((size_t)n_tok * 4);
-    L.out_idx = take((size_t)n_req * 4);
+    L.out_idx = take((size_t)n_out * 4);
     L.fast_map = take((size_t)n_req * 8);
     L.args = take((size_t)n_req * sizeof(lcu_sample_args));
     L.randoms = take((size_t)n_req * 4);
     L.page_table = take((size_t)n_req * pt_stride * 4);
     L.groups = take((size_t)n_tok * 8);  // token groups of the prefill form of attention (at most one per token)
+    L.stack = take(stack_desc_bytes(n_tok, n_req));
     L.total = o;
     return L;
 }
@@ -238,6 +163,159 @@ static void p2p_release(lcu_ctx *c) {
     st = P2pState();
 }
 
+extern "C" int lcu_ctx_destroy(lcu_ctx *c);
+
+// Allocates a context of either family: `layers` describes the layers of a layered model, nullptr means LLaMA layers.
+static int ctx_create(const lcu_model_desc &d, const lcu_layer_desc *layers, int device, int tp_rank, int tp_size, void *nccl_comm, lcu_ctx **out) {
+    int ndev = 0;
+    LCU_CHECK_CUDA(cudaGetDeviceCount(&ndev));
+    LCU_REQUIRE(device >= 0 && device < ndev, "ctx_create: device %d of %d", device, ndev);
+    LCU_CHECK_CUDA(cudaSetDevice(device));
+    cudaDeviceProp prop;
+    LCU_CHECK_CUDA(cudaGetDeviceProperties(&prop, device));
+    if (prop.major != 10) {
+        set_error("ctx_create: device %d is sm_%d%d; this library is built for sm_100a only", device, prop.major, prop.minor);
+        return LCU_ERR_CUDA;
+    }
+
+    lcu_ctx *c = new lcu_ctx();
+    c->desc = d;
+    c->device = device;
+    c->tp_rank = tp_rank;
+    c->tp_size = tp_size;
+    c->comm = nccl_comm;
+    c->dt = d.act_dtype;
+    c->nh_l = d.nh / tp_size;
+    c->nkvh_l = d.nkvh / tp_size;
+    c->di_l = d.di / tp_size;
+    c->qd = c->nh_l * d.dh;
+    c->kvd = c->nkvh_l * d.dh;
+    c->max_tokens = d.max_tokens > 0 ? d.max_tokens : 1024;
+    c->max_seqs = d.max_seqs > 0 ? d.max_seqs : 64;
+    if (c->max_seqs > c->max_tokens) c->max_seqs = c->max_tokens;
+    c->layers.resize(d.n_layers);
+
+    // page geometry: the reference maps 2 MiB pages (memory.rs:14-19); keep a power of two
+    int pt = d.page_tokens;
+    if (pt <= 0 && layers) pt = 64;  // one page is one tile of the latent attention
+    if (pt <= 0) {
+        size_t per_tok = (size_t)d.n_layers * 2 * c->kvd * 2;
+        pt = 16;
+        while (pt < 64 && (size_t)pt * 2 * per_tok <= ((size_t)2 << 20)) pt *= 2;
+    }
+    if (pt < 8 || pt > 128 || (pt & (pt - 1))) {
+        set_error("ctx_create: page_tokens %d must be a power of two in [8,128]", pt);
+        delete c;
+        return LCU_ERR_INVALID;
+    }
+    c->geom.n_layers = d.n_layers;
+    c->geom.nkvh = c->nkvh_l;
+    c->geom.dh = d.dh;
+    c->geom.page_tokens = pt;
+    c->geom.page_shift = 0;
+    while ((1 << c->geom.page_shift) < pt) ++c->geom.page_shift;
+    c->geom.page_elems = (size_t)d.n_layers * 2 * c->nkvh_l * pt * d.dh;
+    c->pt_stride = (d.nctx + pt - 1) / pt;
+    c->seqs.resize(1024);
+
+    // arena
+    size_t eb = dt_bytes(c->dt);
+    // (layered models: activations live in an arena of their own, see stack_create)
+    size_t sz_x = layers ? 256 : align256((size_t)c->max_tokens * d.d * eb);
+    size_t sz_q = align256((size_t)c->max_tokens * c->qd * eb);
+    size_t sz_act = align256((size_t)c->max_tokens * c->di_l * eb);
+    size_t sz_logits = align256((size_t)c->max_seqs * stack_pad(d.vocab, layers ? 8 : 1) * eb);
+    size_t sz_attn = 0;
+    for (int n = 1; n <= c->max_tokens && !layers; ++n) {
+        int sp = attn_splits(c, n);
+        if (sp > 1) {
+            size_t b = attn_scratch_bytes(n, c->nh_l, c->nkvh_l, d.dh, sp, c->max_tokens);
+            if (b > sz_attn) sz_attn = b;
+        }
+    }
+    sz_attn = align256(sz_attn + 256);
+    c->sample_ws_bytes = align256(sample_workspace_bytes(c->max_seqs, (size_t)d.vocab));
+    size_t sz_pairs = align256((size_t)c->max_tokens * sizeof(lcu_kv_pair));
+    size_t sz_head_local = align256((size_t)c->max_seqs * sizeof(lcu_kv_pair));
+    c->desc_cap = align256(desc_layout(c->max_tokens, c->max_seqs, c->max_tokens > c->max_seqs ? c->max_tokens : c->max_seqs, c->pt_stride).total);
+    const size_t sz_sk_ws = (size_t)16 << 20, sz_sk_tickets = (size_t)16 << 10;
+    size_t total = sz_x + 2 * sz_q + sz_act + sz_logits + sz_attn + c->sample_ws_bytes + sz_pairs + 512 + c->desc_cap +
+                   sz_x + sz_sk_ws + sz_sk_tickets + sz_head_local;
+    cudaError_t e = cudaMalloc(&c->arena, total);
+    if (e != cudaSuccess) {
+        delete c;
+        return cuda_fail(e, "cudaMalloc(arena)");
+    }
+    cudaMemset(c->arena, 0, total);
+    unsigned char *p = reinterpret_cast<unsigned char *>(c->arena);
+    c->x = p; p += sz_x;
+    c->q = p; p += sz_q;
+    c->att = p; p += sz_q;
+    c->act = p; p += sz_act;
+    c->logits = p; p += sz_logits;
+    c->attn_scratch = p; p += sz_attn;
+    c->sample_ws = p; p += c->sample_ws_bytes;
+    c->pre_pairs = reinterpret_cast<lcu_kv_pair *>(p); p += sz_pairs;
+    c->dev_status = reinterpret_cast<uint32_t *>(p);
+    p += 512;
+    c->desc_dev = p; p += c->desc_cap;
+    c->hbuf = p; p += sz_x;
+    c->sk_ws = p; p += sz_sk_ws;
+    c->sk_tickets = reinterpret_cast<unsigned *>(p); p += sz_sk_tickets;
+    c->head_local = reinterpret_cast<lcu_kv_pair *>(p);
+    c->sk_ws_bytes = sz_sk_ws;
+    for (int i = 0; i < lcu_ctx::RING; ++i) {
+        e = cudaMallocHost(reinterpret_cast<void **>(&c->desc_host[i]), c->desc_cap);
+        if (e == cudaSuccess) e = cudaEventCreateWithFlags(&c->desc_event[i], cudaEventDisableTiming);
+        if (e != cudaSuccess) {
+            lcu_ctx_destroy(c);
+            return cuda_fail(e, "descriptor staging");
+        }
+    }
+    if (layers) {
+        int rc = stack_create(c, layers);
+        if (rc) {
+            lcu_ctx_destroy(c);
+            return rc;
+        }
+        *out = c;
+        return LCU_OK;
+    }
+    // prepare every kernel variant now: nothing but launches may happen inside a capture
+    {
+        bool q8 = d.weight_dtype == LCU_Q8_0;
+        int rc = gemv_warm(d.d, c->qd + 2 * c->kvd, q8, c->dt);
+        if (!rc) rc = gemv_warm(c->qd, d.d, q8, c->dt);
+        if (!rc) rc = gemv_warm(c->di_l, d.d, q8, c->dt);
+        if (!rc) rc = gemv_warm(d.d, d.vocab & ~1, false, c->dt);
+        if (!rc) {
+            AttnArgs a{};
+            a.n_tok = 1; a.nh = c->nh_l; a.nkvh = c->nkvh_l; a.dh = d.dh; a.n_splits = 1;
+            rc = attn_launch(a, c->dt, nullptr, false, true);
+            if (!rc) rc = attn_prefill_launch(a, nullptr, 0, c->dt, nullptr, true);
+        }
+        if (rc) {
+            lcu_ctx_destroy(c);
+            return rc;
+        }
+        // the batched (tensor-core) form of the linear layers
+        c->batched_ok = gemm_skinny_supported(d.d, q8) && gemm_skinny_supported(c->qd, q8) && gemm_skinny_supported(c->di_l, q8);
+        if (c->batched_ok) {
+            rc = gemm_skinny_warm(d.d, c->qd + 2 * c->kvd, c->dt, q8);
+            if (!rc) rc = gemm_skinny_warm(c->qd, d.d, c->dt, q8);
+            if (!rc) rc = gemm_skinny_warm(c->di_l, d.d, c->dt, q8);
+            if (!rc) rc = gemm_skinny_warm(d.d, d.vocab & ~1, c->dt);
+            if (!rc && gemm_tc_supported(d.d, q8)) rc = gemm_tc_warm(c->dt);
+            if (rc) {
+                lcu_ctx_destroy(c);
+                return rc;
+            }
+        }
+    }
+    *out = c;
+    return LCU_OK;
+}
+
 extern "C" {
 
 const char *lcu_last_error_string(void) { return g_err; }
@@ -245,6 +323,11 @@ int lcu_version(void) { return 100; }
 
 size_t lcu_weight_bytes(const lcu_ctx *c, int kind) {
     if (!c) return 0;
+    if (c->stack) {  // only the kinds every layer shares
+        int rows, cols, eb;
+        const bool ok = (kind == LCU_W_EMBD || kind == LCU_W_OUT_NORM || kind == LCU_W_LM_HEAD) && stack_weight_shape(c, 0, kind, &rows, &cols, &eb);
+        return ok ? (size_t)rows * cols * eb : 0;
+    }
     size_t n = weight_elems(c, kind);
     if (kind == LCU_W_ATTN_NORM || kind == LCU_W_FFN_NORM || kind == LCU_W_OUT_NORM)
         return n * dt_bytes(c->desc.norm_dtype);
@@ -284,142 +367,18 @@ int lcu_ctx_create(const lcu_model_desc *desc, int device, int tp_rank, int tp_s
     int g = d.nh / d.nkvh;
     LCU_REQUIRE(g == 1 || g == 2 || g == 4 || g == 8, "ctx_create: nh/nkvh = %d (1, 2, 4, 8)", g);
 
-    int ndev = 0;
-    LCU_CHECK_CUDA(cudaGetDeviceCount(&ndev));
-    LCU_REQUIRE(device >= 0 && device < ndev, "ctx_create: device %d of %d", device, ndev);
-    LCU_CHECK_CUDA(cudaSetDevice(device));
-    cudaDeviceProp prop;
-    LCU_CHECK_CUDA(cudaGetDeviceProperties(&prop, device));
-    if (prop.major != 10) {
-        set_error("ctx_create: device %d is sm_%d%d; this library is built for sm_100a only", device, prop.major, prop.minor);
-        return LCU_ERR_CUDA;
-    }
+    return ctx_create(d, nullptr, device, tp_rank, tp_size, nccl_comm, out);
+}
 
-    lcu_ctx *c = new lcu_ctx();
-    c->desc = d;
-    c->device = device;
-    c->tp_rank = tp_rank;
-    c->tp_size = tp_size;
-    c->comm = nccl_comm;
-    c->dt = d.act_dtype;
-    c->nh_l = d.nh / tp_size;
-    c->nkvh_l = d.nkvh / tp_size;
-    c->di_l = d.di / tp_size;
-    c->qd = c->nh_l * d.dh;
-    c->kvd = c->nkvh_l * d.dh;
-    c->max_tokens = d.max_tokens > 0 ? d.max_tokens : 1024;
-    c->max_seqs = d.max_seqs > 0 ? d.max_seqs : 64;
-    if (c->max_seqs > c->max_tokens) c->max_seqs = c->max_tokens;
-    c->layers.resize(d.n_layers);
-
-    // page geometry: the reference maps 2 MiB pages (memory.rs:14-19); keep a power of two
-    int pt = d.page_tokens;
-    if (pt <= 0) {
-        size_t per_tok = (size_t)d.n_layers * 2 * c->kvd * 2;
-        pt = 16;
-        while (pt < 64 && (size_t)pt * 2 * per_tok <= ((size_t)2 << 20)) pt *= 2;
-    }
-    if (pt < 8 || pt > 128 || (pt & (pt - 1))) {
-        set_error("ctx_create: page_tokens %d must be a power of two in [8,128]", pt);
-        delete c;
-        return LCU_ERR_INVALID;
-    }
-    c->geom.n_layers = d.n_layers;
-    c->geom.nkvh = c->nkvh_l;
-    c->geom.dh = d.dh;
-    c->geom.page_tokens = pt;
-    c->geom.page_shift = 0;
-    while ((1 << c->geom.page_shift) < pt) ++c->geom.page_shift;
-    c->geom.page_elems = (size_t)d.n_layers * 2 * c->nkvh_l * pt * d.dh;
-    c->pt_stride = (d.nctx + pt - 1) / pt;
-    c->seqs.resize(1024);
-
-    // arena
-    size_t eb = 2;
-    size_t sz_x = align256((size_t)c->max_tokens * d.d * eb);
-    size_t sz_q = align256((size_t)c->max_tokens * c->qd * eb);
-    size_t sz_act = align256((size_t)c->max_tokens * c->di_l * eb);
-    size_t sz_logits = align256((size_t)c->max_seqs * d.vocab * eb);
-    size_t sz_attn = 0;
-    for (int n = 1; n <= c->max_tokens; ++n) {
-        int sp = attn_splits(c, n);
-        if (sp > 1) {
-            size_t b = attn_scratch_bytes(n, c->nh_l, c->nkvh_l, d.dh, sp, c->max_tokens);
-            if (b > sz_attn) sz_attn = b;
-        }
-    }
-    sz_attn = align256(sz_attn + 256);
-    c->sample_ws_bytes = align256(sample_workspace_bytes(c->max_seqs, (size_t)d.vocab));
-    size_t sz_pairs = align256((size_t)c->max_tokens * sizeof(lcu_kv_pair));
-    size_t sz_head_local = align256((size_t)c->max_seqs * sizeof(lcu_kv_pair));
-    c->desc_cap = align256(desc_layout(c->max_tokens, c->max_seqs, c->pt_stride).total);
-    const size_t sz_sk_ws = (size_t)16 << 20, sz_sk_tickets = (size_t)16 << 10;
-    size_t total = sz_x + 2 * sz_q + sz_act + sz_logits + sz_attn + c->sample_ws_bytes + sz_pairs + 512 + c->desc_cap +
-                   sz_x + sz_sk_ws + sz_sk_tickets + sz_head_local;
-    cudaError_t e = cudaMalloc(&c->arena, total);
-    if (e != cudaSuccess) {
-        delete c;
-        return cuda_fail(e, "cudaMalloc(arena)");
-    }
-    cudaMemset(c->arena, 0, total);
-    unsigned char *p = reinterpret_cast<unsigned char *>(c->arena);
-    c->x = p; p += sz_x;
-    c->q = p; p += sz_q;
-    c->att = p; p += sz_q;
-    c->act = p; p += sz_act;
-    c->logits = p; p += sz_logits;
-    c->attn_scratch = p; p += sz_attn;
-    c->sample_ws = p; p += c->sample_ws_bytes;
-    c->pre_pairs = reinterpret_cast<lcu_kv_pair *>(p); p += sz_pairs;
-    c->dev_status = reinterpret_cast<uint32_t *>(p);
-    p += 512;
-    c->desc_dev = p; p += c->desc_cap;
-    c->hbuf = p; p += sz_x;
-    c->sk_ws = p; p += sz_sk_ws;
-    c->sk_tickets = reinterpret_cast<unsigned *>(p); p += sz_sk_tickets;
-    c->head_local = reinterpret_cast<lcu_kv_pair *>(p);
-    c->sk_ws_bytes = sz_sk_ws;
-    for (int i = 0; i < lcu_ctx::RING; ++i) {
-        e = cudaMallocHost(reinterpret_cast<void **>(&c->desc_host[i]), c->desc_cap);
-        if (e == cudaSuccess) e = cudaEventCreateWithFlags(&c->desc_event[i], cudaEventDisableTiming);
-        if (e != cudaSuccess) {
-            lcu_ctx_destroy(c);
-            return cuda_fail(e, "descriptor staging");
-        }
-    }
-    // prepare every kernel variant now: nothing but launches may happen inside a capture
-    {
-        bool q8 = d.weight_dtype == LCU_Q8_0;
-        int rc = gemv_warm(d.d, c->qd + 2 * c->kvd, q8, c->dt);
-        if (!rc) rc = gemv_warm(c->qd, d.d, q8, c->dt);
-        if (!rc) rc = gemv_warm(c->di_l, d.d, q8, c->dt);
-        if (!rc) rc = gemv_warm(d.d, d.vocab & ~1, false, c->dt);
-        if (!rc) {
-            AttnArgs a{};
-            a.n_tok = 1; a.nh = c->nh_l; a.nkvh = c->nkvh_l; a.dh = d.dh; a.n_splits = 1;
-            rc = attn_launch(a, c->dt, nullptr, false, true);
-            if (!rc) rc = attn_prefill_launch(a, nullptr, 0, c->dt, nullptr, true);
-        }
-        if (rc) {
-            lcu_ctx_destroy(c);
-            return rc;
-        }
-        // the batched (tensor-core) form of the linear layers
-        c->batched_ok = gemm_skinny_supported(d.d, q8) && gemm_skinny_supported(c->qd, q8) && gemm_skinny_supported(c->di_l, q8);
-        if (c->batched_ok) {
-            rc = gemm_skinny_warm(d.d, c->qd + 2 * c->kvd, c->dt, q8);
-            if (!rc) rc = gemm_skinny_warm(c->qd, d.d, c->dt, q8);
-            if (!rc) rc = gemm_skinny_warm(c->di_l, d.d, c->dt, q8);
-            if (!rc) rc = gemm_skinny_warm(d.d, d.vocab & ~1, c->dt);
-            if (!rc && gemm_tc_supported(d.d, q8)) rc = gemm_tc_warm(c->dt);
-            if (rc) {
-                lcu_ctx_destroy(c);
-                return rc;
-            }
-        }
-    }
-    *out = c;
-    return LCU_OK;
+int lcu_ctx_create_layers(const lcu_model_desc *desc, const lcu_layer_desc *layers, int device, lcu_ctx **out) {
+    LCU_REQUIRE(desc && layers && out, "ctx_create_layers: null argument");
+    lcu_model_desc d = *desc;
+    LCU_REQUIRE(d.n_layers > 0 && d.d > 0 && d.vocab > 0 && d.nctx > 0, "ctx_create_layers: non-positive model dimension");
+    LCU_REQUIRE(d.d <= 16384, "ctx_create_layers: width %d (at most 16384)", d.d);
+    LCU_REQUIRE(d.act_dtype == LCU_BF16 || d.act_dtype == LCU_F32, "ctx_create_layers: activation dtype %d (bf16 or f32)", d.act_dtype);
+    LCU_REQUIRE(d.weight_dtype == LCU_BF16, "ctx_create_layers: weight dtype %d (bf16)", d.weight_dtype);
+    d.nh = d.nkvh = d.dh = d.di = 0;
+    return ctx_create(d, layers, device, 0, 1, nullptr, out);
 }
 
 int lcu_ctx_destroy(lcu_ctx *c) {
@@ -435,6 +394,7 @@ int lcu_ctx_destroy(lcu_ctx *c) {
     if (c->own_pool && c->pool) cudaFree(c->pool);
     if (c->own_tables) cudaFree(c->own_tables);
     p2p_release(c);
+    stack_destroy(c);
     if (c->arena) cudaFree(c->arena);
     delete c;
     return LCU_OK;
@@ -442,6 +402,15 @@ int lcu_ctx_destroy(lcu_ctx *c) {
 
 int lcu_set_weight(lcu_ctx *c, int layer, int kind, const void *dev_ptr, size_t bytes) {
     LCU_REQUIRE(c && dev_ptr, "set_weight: null argument");
+    if (c->stack && kind >= LCU_W_LAT_IN) {
+        int rows, cols, eb;
+        LCU_REQUIRE(stack_weight_shape(c, layer, kind, &rows, &cols, &eb), "set_weight: layer %d has no weight of kind %d", layer, kind);
+        LCU_REQUIRE(bytes == (size_t)rows * cols * eb, "set_weight: kind %d of layer %d expects [%d, %d] (%zu bytes), got %zu bytes", kind, layer,
+                    rows, cols, (size_t)rows * cols * eb, bytes);
+        LCU_REQUIRE(((uintptr_t)dev_ptr % 16) == 0, "set_weight: pointer must be 16-byte aligned");
+        drop_graphs(c);
+        return stack_set_weight(c, layer, kind, dev_ptr);
+    }
     size_t want = lcu_weight_bytes(c, kind);
     LCU_REQUIRE(want > 0, "set_weight: unknown kind %d", kind);
     LCU_REQUIRE(bytes == want, "set_weight: kind %d expects %zu bytes on this rank, got %zu", kind, want, bytes);
@@ -463,6 +432,13 @@ int lcu_set_weight(lcu_ctx *c, int layer, int kind, const void *dev_ptr, size_t 
     case LCU_W_DOWN: L.down = dev_ptr; break;
     }
     drop_graphs(c);
+    return LCU_OK;
+}
+
+int lcu_layer_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows_out, int *cols_out) {
+    LCU_REQUIRE(c && c->stack && rows_out && cols_out, "layer_weight_shape: needs a layered context");
+    int eb;
+    LCU_REQUIRE(stack_weight_shape(c, layer, kind, rows_out, cols_out, &eb), "layer_weight_shape: layer %d has no weight of kind %d", layer, kind);
     return LCU_OK;
 }
 
@@ -493,7 +469,7 @@ int lcu_kv_pool_attach(lcu_ctx *c, void *dev_ptr, size_t bytes) {
     LCU_REQUIRE(c && dev_ptr, "kv_pool_attach: null argument");
     LCU_REQUIRE(!c->pool, "kv_pool_attach: a pool is already attached");
     LCU_REQUIRE(((uintptr_t)dev_ptr % 256) == 0, "kv_pool_attach: pool must be 256-byte aligned");
-    size_t page_bytes = c->geom.page_elems * 2;
+    size_t page_bytes = c->geom.page_elems * dt_bytes(c->dt);
     int n = (int)(bytes / page_bytes);
     LCU_REQUIRE(n >= 1, "kv_pool_attach: %zu bytes hold no page of %zu bytes", bytes, page_bytes);
     c->pool = dev_ptr;
@@ -506,7 +482,7 @@ int lcu_kv_pool_attach(lcu_ctx *c, void *dev_ptr, size_t bytes) {
 int lcu_kv_pool_create(lcu_ctx *c, size_t bytes) {
     LCU_REQUIRE(c, "kv_pool_create: null context");
     LCU_REQUIRE(!c->pool, "kv_pool_create: a pool already exists");
-    size_t page_bytes = c->geom.page_elems * 2;
+    size_t page_bytes = c->geom.page_elems * dt_bytes(c->dt);
     size_t n = bytes / page_bytes;
     LCU_REQUIRE(n >= 1, "kv_pool_create: %zu bytes hold no page of %zu bytes", bytes, page_bytes);
     void *p = nullptr;
@@ -522,7 +498,7 @@ int lcu_kv_pool_create(lcu_ctx *c, size_t bytes) {
 }
 
 int lcu_kv_page_tokens(const lcu_ctx *c) { return c ? c->geom.page_tokens : 0; }
-size_t lcu_kv_page_bytes(const lcu_ctx *c) { return c ? c->geom.page_elems * 2 : 0; }
+size_t lcu_kv_page_bytes(const lcu_ctx *c) { return c ? c->geom.page_elems * dt_bytes(c->dt) : 0; }
 int lcu_kv_pages_total(const lcu_ctx *c) { return c ? c->n_pages : 0; }
 int lcu_kv_pages_free(const lcu_ctx *c) { return c ? (int)c->free_pages.size() : 0; }
 
@@ -533,6 +509,8 @@ int lcu_seq_create(lcu_ctx *c, int *seq_out) {
             c->seqs[i].used = true;
             c->seqs[i].len = 0;
             c->seqs[i].pages.clear();
+            c->seqs[i].slot = -1;
+            c->seqs[i].state_len = 0;
             *seq_out = (int)i;
             return LCU_OK;
         }
@@ -580,7 +558,16 @@ int lcu_seq_free(lcu_ctx *c, int seq) {
     s.pages.clear();
     s.len = 0;
     s.used = false;
+    if (s.slot >= 0) c->free_slots.push_back(s.slot);
+    s.slot = -1;
     return LCU_OK;
+}
+
+int lcu_seq_resumable(const lcu_ctx *c, int seq, uint32_t len) {
+    if (!c || seq < 0 || seq >= (int)c->seqs.size() || !c->seqs[seq].used) return -1;
+    if (!c->stack || !c->stack->n_slots) return (int)len;
+    const SeqState &s = c->seqs[seq];
+    return s.slot >= 0 && s.state_len <= len ? (int)s.state_len : 0;
 }
 
 int lcu_set_cuda_graph(lcu_ctx *c, int enabled) {
@@ -600,6 +587,7 @@ int lcu_set_tuning(lcu_ctx *c, const char *key, long long value) {
     else if (k == "tc") t.tc = value != 0;
     else if (k == "tc_block") { LCU_REQUIRE(value == 64 || value == 128 || value == 256, "set_tuning: tc_block = %lld (64, 128, 256)", value); t.tc_block = (int)value; }
     else if (k == "tc_cluster") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: tc_cluster = %lld (0..2)", value); t.tc_cluster = (int)value; }
+    else if (k == "expand_min") t.expand_min = (int)value;
     else if (k == "p2p_scatter_ranks") t.p2p_scatter_ranks = (int)value;
     else if (k == "p2p_scatter_min") t.p2p_scatter_min = (long)value;
     else {
@@ -630,6 +618,7 @@ int lcu_reset_status(lcu_ctx *c) {
 }
 int lcu_last_launch_count(const lcu_ctx *c) { return c ? c->last_launches : 0; }
 double lcu_last_step_bytes(const lcu_ctx *c) { return c ? c->last_bytes : 0.0; }
+int lcu_logits_stride(const lcu_ctx *c) { return !c ? 0 : (c->stack ? c->stack->vocab_p : c->desc.vocab); }
 const void *lcu_logits(const lcu_ctx *c) { return c ? c->logits : nullptr; }
 const void *lcu_hidden(const lcu_ctx *c) { return c ? c->x : nullptr; }
 
@@ -646,14 +635,6 @@ int lcu_device_status(lcu_ctx *c, lcu_stream_t stream, uint32_t *status_out) {
 // ------------------------------------------------------------------ the round
 
 namespace {
-
-struct Round {
-    int n_tok, n_req, n_fast;
-    int n_groups;  // token groups for the prefill form of attention (0: decode form)
-    bool any_sampling;
-    bool decode_only;  // one new token per sequence
-    DescLayout L;
-};
 
 // Enqueues every kernel of one round on `s`; returns the number of launches through *count.
 int enqueue_round(lcu_ctx *c, const Round &r, lcu_kv_pair *out_dev, cudaStream_t s, int *count) {
@@ -695,6 +676,17 @@ int enqueue_round(lcu_ctx *c, const Round &r, lcu_kv_pair *out_dev, cudaStream_t
             if (rc) return rc;
             ++launches;
         }
+    }
+    if (c->stack) {  // layered models: their own layers and head projection, the sampler of every model
+        rc = stack_layers(c, r, s, &launches);
+        if (!rc) rc = stack_head(c, r, out_idx, r.n_out, r.logits_f32, s, &launches);
+        if (!rc && !r.logits_f32) {
+            rc = sample_rows(out_dev, c->pre_pairs, c->logits, r.n_req, (size_t)d.vocab, r.any_sampling ? args : nullptr, randoms, dt, c->sample_ws,
+                             c->sample_ws_bytes, s, false, r.any_sampling, (size_t)c->stack->vocab_p);
+            launches += r.any_sampling ? 3 : 2;
+        }
+        *count = launches;
+        return rc;
     }
     rc = op_embedding(c->x, c->embd, tokens, r.n_tok, (size_t)d.d * 2, s, r.n_fast > 0);
     if (rc) return rc;
@@ -866,6 +858,26 @@ int enqueue_round(lcu_ctx *c, const Round &r, lcu_kv_pair *out_dev, cudaStream_t
         if (rc) return rc;
     }
 
+    if (r.logits_f32) {  // asked rows, as f32, a block of rows at a time through the logits buffer; nothing is sampled
+        for (int r0 = 0; r0 < r.n_out; ) {
+            int nt = gemv_max_tokens(d.d);
+            if (nt > r.n_out - r0) nt = r.n_out - r0;
+            if (nt > c->max_seqs) nt = c->max_seqs;
+            if (nt == 3) nt = 2;
+            GemvArgs a{};
+            a.w = c->lm_head; a.x = c->x; a.stride_x = d.d; a.x_rows = out_idx + r0; a.n_tok = nt; a.in = d.d; a.out = d.vocab;
+            a.prologue = PRO_RMSNORM; a.norm_w = c->out_norm; a.norm_f32 = d.norm_dtype == LCU_F32; a.eps = d.eps;
+            a.epilogue = EPI_STORE; a.y = c->logits; a.stride_y = d.vocab; a.pdl_trigger = 2; a.early_prefetch = 1;
+            rc = gemv_launch(a, dt, s, false);
+            if (!rc) rc = op_rows_to_f32(r.logits_f32 + (size_t)r0 * d.vocab, c->logits, (size_t)nt * d.vocab, dt, s);
+            if (rc) return rc;
+            launches += 2;
+            r0 += nt;
+        }
+        *count = launches;
+        return LCU_OK;
+    }
+
     // --- head (exec/engine.rs:90,201): gather + RMSNorm + LM head + sampling.  The reference runs it on the lead rank
     // alone; with the peer-memory transport an arg-max round shards it by vocabulary rows instead: every rank streams
     // vocab / tp rows, arg-maxes them, the lead rank keeps the best candidate per row (lowest index among equals).
@@ -976,15 +988,17 @@ extern "C" int lcu_p2p_attach(lcu_ctx *c, const void *handles) {
 
 extern "C" int lcu_p2p_enabled(const lcu_ctx *c) { return c && c->p2p.ready ? 1 : 0; }
 
-extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens,
-                        const lcu_sample_args *args, const float *randoms, const uint32_t *fast_map, int n_fast,
-                        lcu_kv_pair *out_dev) {
+// One round.  rows == nullptr: the last token of every request goes through the head and the sampler (lcu_step); otherwise the
+// logits of the asked token slots (lcu_step_logits).
+static int run_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens, const lcu_sample_args *args,
+                    const float *randoms, const uint32_t *fast_map, int n_fast, lcu_kv_pair *out_dev, int n_rows, const uint32_t *rows,
+                    float *logits_dev) {
     LCU_REQUIRE(c && reqs && tokens, "step: null argument");
     LCU_REQUIRE(n_req >= 1 && n_req <= c->max_seqs, "step: %d requests (1..%d)", n_req, c->max_seqs);
-    LCU_REQUIRE(c->tp_rank != 0 || out_dev, "step: the lead rank needs an output buffer");
+    LCU_REQUIRE(c->tp_rank != 0 || out_dev || logits_dev, "step: the lead rank needs an output buffer");
     LCU_REQUIRE(n_fast >= 0 && n_fast <= n_req && (n_fast == 0 || fast_map), "step: bad fast_map");
     const lcu_model_desc &d = c->desc;
-    LCU_REQUIRE(d.vocab % 2 == 0, "step: vocab %d must be even", d.vocab);
+    LCU_REQUIRE(c->stack || d.vocab % 2 == 0, "step: vocab %d must be even", d.vocab);
     if (!c->pool) { set_error("step: no KV pool"); return LCU_ERR_STATE; }
     const bool head_everywhere = c->p2p.ready && c->head_shard && head_rows_per_rank(c) > 0;
     if (!c->embd || ((c->tp_rank == 0 || head_everywhere) && (!c->out_norm || !c->lm_head))) { set_error("step: embedding / output weights missing"); return LCU_ERR_STATE; }
@@ -992,7 +1006,8 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
         set_error("step: a bounded device-side wait ran out earlier (status %u); the group is broken until lcu_reset_status", c->sticky_status);
         return LCU_ERR_TIMEOUT;
     }
-    for (int l = 0; l < d.n_layers; ++l) {
+    if (c->stack && !stack_ready(c)) return LCU_ERR_STATE;
+    for (int l = 0; l < d.n_layers && !c->stack; ++l) {
         const LayerWeights &W = c->layers[l];
         if (!W.attn_norm || !W.qkv || !W.o || !W.ffn_norm || !W.gate_up || !W.down) {
             set_error("step: weights of layer %d missing", l);
@@ -1000,8 +1015,9 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
         }
     }
     LCU_CHECK_CUDA(cudaSetDevice(c->device));
-    int rc = ensure_tables(c);
+    int rc = c->stack ? LCU_OK : ensure_tables(c);
     if (rc) return rc;
+    const bool recurrent = c->stack && c->stack->n_slots > 0;
 
     // validate, then back every sequence with pages (KVCache::update, exec/group.rs:134-144)
     int n_tok = 0;
@@ -1023,6 +1039,21 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
             any_sampling = true;
         }
     }
+    int slots_needed = 0;
+    for (int i = 0; i < n_req && recurrent; ++i) {  // a sequence goes on where its recurrent state ends, or starts again
+        const SeqState &sq = c->seqs[reqs[i].seq];
+        if (sq.slot < 0) ++slots_needed;
+        if (reqs[i].pos != 0 && (sq.slot < 0 || sq.state_len != reqs[i].pos)) {
+            set_error("step: request %d starts at %u, the recurrent state of sequence %d is that after %u tokens", i, reqs[i].pos, reqs[i].seq,
+                      sq.slot < 0 ? 0u : sq.state_len);
+            return LCU_ERR_STATE;
+        }
+    }
+    if (slots_needed > (int)c->free_slots.size()) {
+        set_error("step: %d recurrent-state slots needed, %zu free", slots_needed, c->free_slots.size());
+        return LCU_ERR_NO_PAGES;
+    }
+    for (int i = 0; i < n_rows; ++i) LCU_REQUIRE(rows[i] < (uint32_t)n_tok, "step_logits: row %d names token slot %u of %d", i, rows[i], n_tok);
     LCU_REQUIRE(n_tok <= c->max_tokens, "step: %d tokens exceed max_tokens %d", n_tok, c->max_tokens);
     for (int i = 0; i < n_fast; ++i)
         LCU_REQUIRE(fast_map[2 * i] < (uint32_t)c->max_tokens && fast_map[2 * i + 1] < (uint32_t)n_tok, "step: fast_map entry %d out of range", i);
@@ -1040,11 +1071,21 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
         rc = lcu_seq_resize(c, reqs[i].seq, reqs[i].pos + reqs[i].len);
         if (rc) return rc;
     }
+    for (int i = 0; i < n_req && recurrent; ++i) {
+        SeqState &sq = c->seqs[reqs[i].seq];
+        if (sq.slot < 0) {
+            sq.slot = c->free_slots.back();
+            c->free_slots.pop_back();
+        }
+    }
 
     // stage the round descriptor in the next pinned buffer (BufN, exec/engine.rs:373-429)
     Round r;
     r.n_tok = n_tok; r.n_req = n_req; r.n_fast = n_fast; r.any_sampling = any_sampling; r.decode_only = decode_only;
-    r.L = desc_layout(n_tok, n_req, c->pt_stride);
+    r.n_groups = 0;
+    r.n_out = rows ? n_rows : n_req;
+    r.logits_f32 = logits_dev;
+    r.L = desc_layout(n_tok, n_req, r.n_out, c->pt_stride);
     cudaStream_t s = as_stream(stream);
     int slot = c->ring_idx;
     c->ring_idx = (c->ring_idx + 1) % lcu_ctx::RING;
@@ -1063,13 +1104,17 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
                 hp[t] = reqs[i].pos + j;
                 hr[t] = i;
             }
-            ho[i] = (uint32_t)(t - 1);  // out_idx() with out == 1, exec/engine.rs:360-371
+            if (!rows) ho[i] = (uint32_t)(t - 1);  // out_idx() with out == 1, exec/engine.rs:360-371
             const SeqState &sq = c->seqs[reqs[i].seq];
             for (size_t pg = 0; pg < sq.pages.size(); ++pg) ht[(size_t)i * c->pt_stride + pg] = sq.pages[pg];
         }
+        for (int i = 0; rows && i < n_rows; ++i) ho[i] = rows[i];
+        if (c->stack) {
+            rc = stack_stage(c, r, reqs, H);
+            if (rc) return rc;
+        }
         // prompts in the round: consecutive tokens of a request are grouped for the prefill form of attention
-        r.n_groups = 0;
-        if (!decode_only && attn_prefill_supported(c->pt_stride)) {
+        if (!c->stack && !decode_only && attn_prefill_supported(c->pt_stride)) {
             int32_t *hg = reinterpret_cast<int32_t *>(H + r.L.groups);
             const int gt = attn_prefill_group_tokens(c->nh_l, c->nkvh_l);
             int t0 = 0;
@@ -1093,9 +1138,20 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
     LCU_CHECK_CUDA(cudaMemcpyAsync(c->desc_dev, H, r.L.total, cudaMemcpyHostToDevice, s));
     LCU_CHECK_CUDA(cudaEventRecord(c->desc_event[slot], s));
     c->desc_used[slot] = true;
+    // the round writes the other half of its sequences' state; until it is enqueued no position is resumable
+    for (int i = 0; i < n_req && recurrent; ++i) c->seqs[reqs[i].seq].state_len = ~0u;
+    auto finish = [&](int code) -> int {
+        for (int i = 0; i < n_req && recurrent && code == LCU_OK; ++i) {
+            SeqState &sq = c->seqs[reqs[i].seq];
+            sq.gen ^= 1;
+            sq.state_len = reqs[i].pos + reqs[i].len;
+        }
+        return code;
+    };
 
     // algorithmic bytes of the round: every linear weight once, the LM head, the cached K/V
-    {
+    if (c->stack) c->last_bytes = stack_step_bytes(c, reqs, n_req, r.n_out);
+    else {
         double wb = d.weight_dtype == LCU_Q8_0 ? 34.0 / 32.0 : 2.0;
         double per_layer = ((double)(c->qd + 2 * c->kvd) * d.d + (double)d.d * c->qd + 2.0 * c->di_l * d.d + (double)d.d * c->di_l) * wb;
         const bool sharded = head_everywhere && !any_sampling;
@@ -1111,12 +1167,12 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
 
     // decode rounds replay a captured graph; everything else (and stream 0) runs eagerly.
     // NCCL collectives are captured like any other node (exec/step.rs:82-86).
-    bool graph_ok = c->use_graph && decode_only && s != nullptr;
+    bool graph_ok = c->use_graph && decode_only && s != nullptr && !logits_dev;
     if (!graph_ok) {
         int count = 0;
         rc = enqueue_round(c, r, out_dev, s, &count);
         c->last_launches = count;
-        return rc;
+        return finish(rc);
     }
     std::vector<int> key = {n_req, n_tok, n_fast, any_sampling ? 1 : 0, (int)((uintptr_t)out_dev & 0x7fffffff),
                             (int)((uintptr_t)out_dev >> 31), c->head_shard ? 1 : 0};
@@ -1144,7 +1200,21 @@ extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_re
     }
     LCU_CHECK_CUDA(cudaGraphLaunch(it->second.exec, s));
     c->last_launches = it->second.launches;
-    return LCU_OK;
+    return finish(LCU_OK);
+}
+
+extern "C" int lcu_step(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens,
+                        const lcu_sample_args *args, const float *randoms, const uint32_t *fast_map, int n_fast,
+                        lcu_kv_pair *out_dev) {
+    return run_step(c, stream, n_req, reqs, tokens, args, randoms, fast_map, n_fast, out_dev, 0, nullptr, nullptr);
+}
+
+extern "C" int lcu_step_logits(lcu_ctx *c, lcu_stream_t stream, int n_req, const lcu_req *reqs, const uint32_t *tokens,
+                               int n_rows, const uint32_t *rows, float *logits_dev) {
+    LCU_REQUIRE(c && logits_dev && n_rows >= 0 && n_rows <= c->max_tokens && (rows || n_rows == 0), "step_logits: bad arguments");
+    LCU_REQUIRE(c->tp_size == 1, "step_logits: one GPU only");
+    static const uint32_t none = 0;
+    return run_step(c, stream, n_req, reqs, tokens, nullptr, nullptr, nullptr, 0, nullptr, n_rows, rows ? rows : &none, logits_dev);
 }
 
 namespace lcu {

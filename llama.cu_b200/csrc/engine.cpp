@@ -271,6 +271,8 @@ int lcu_engine_cache_send(lcu_engine *e, const uint32_t *tokens, uint32_t n, con
         const std::vector<uint32_t> &h = kv.second.history;
         uint32_t len = 0;
         while (len < h.size() && len + 1 < n && h[len] == tokens[len]) ++len;
+        // a recurrent state cannot be rolled back: such a cache is reused up to the position its state covers, or not at all
+        if (e->ctx) len = (uint32_t)lcu_seq_resumable(e->ctx, kv.second.seq, len);
         if (!found || len >= best_len) { found = true; best_key = kv.first; best_len = len; }
     }
     int seq;

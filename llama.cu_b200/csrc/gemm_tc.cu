@@ -163,6 +163,17 @@ __device__ __forceinline__ void tc_finish(const GemvArgs &a, int n, int first, f
             dst = reinterpret_cast<T *>(a.kv_pool) + a.geom.block_off(pre.page, a.layer, sect - 1, head) + (size_t)slot * a.dh + e;
         }
     }
+    if (a.epilogue == EPI_STORE_F32) {
+        float4 *f = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.y) + (size_t)n * a.stride_y + first);
+        f[0] = make_float4(v[0], v[1], v[2], v[3]);
+        f[1] = make_float4(v[4], v[5], v[6], v[7]);
+        return;
+    }
+    if (a.epilogue == EPI_XIELU) {
+        const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = xielu_act(v[i], sp, sq);
+    }
     uint4 o;
     o.x = Act<T>::pack(v[0], v[1]); o.y = Act<T>::pack(v[2], v[3]); o.z = Act<T>::pack(v[4], v[5]); o.w = Act<T>::pack(v[6], v[7]);
     if (a.push.n && (a.epilogue == EPI_STORE || a.epilogue == EPI_RESIDUAL)) {
@@ -769,6 +780,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
         vec_ok = vec_ok && a.dh % 8 == 0 && a.qd % 8 == 0 && a.kvd % 8 == 0 && ((uintptr_t)a.kv_pool % 16) == 0 &&
                  ((uintptr_t)a.sin_t % 16) == 0 && ((uintptr_t)a.cos_t % 16) == 0;
     const int vec = vec_ok ? 1 : 0;
+    LCU_REQUIRE(vec || a.epilogue < EPI_STORE_F32, "gemm_tc: epilogue %d needs rows of a multiple of 8 outputs", a.epilogue);
     // ---- weight rows on M (any output shape; row blocks of 128)
     rc = tc_make_map(&mw, a.w, dt, (uint64_t)a.out, (uint64_t)a.in, (uint64_t)a.in, 64);
     if (rc) return rc;
@@ -823,7 +835,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
             GemvArgs b = a;
             b.n_tok = a.n_tok - t0 < 64 ? a.n_tok - t0 : 64;
             b.x = reinterpret_cast<const unsigned char *>(a.x) + (size_t)t0 * a.stride_x * 2;
-            b.y = reinterpret_cast<unsigned char *>(a.y) + (size_t)t0 * a.stride_y * 2;
+            b.y = reinterpret_cast<unsigned char *>(a.y) + (size_t)t0 * a.stride_y * 2;  // 16-bit outputs only (f32 ones have the 16-byte epilogue)
             if (a.res) b.res = reinterpret_cast<const unsigned char *>(a.res) + (size_t)t0 * a.stride_res * 2;
             if (a.pos) { b.pos = a.pos + t0; b.tok_seq = a.tok_seq + t0; }
             int rc2 = tc_launch_t<T>(b, dt, s, pdl, dry);

@@ -52,7 +52,8 @@ __device__ __forceinline__ void vec8_to_f32(const uint4 &v, float f[8]) {
 
 // PRO: 0 = activations staged as they are, 1 = RMSNorm (any token count, f32 or 16-bit norm weights), 2 = RMSNorm of one
 // token from registers
-template <class T, bool Q8, int NT, int KI, int RP, int PRO>
+// STK: the epilogues of layered models instead of the LLaMA ones
+template <class T, bool Q8, int NT, int KI, int RP, int PRO, bool STK>
 __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(const GemvArgs a, int KS, int RS, int n_pairs) {
     constexpr int R = 2 * RP;
     constexpr int VE = Q8 ? 16 : 8;  // weights per 16-byte vector
@@ -64,7 +65,7 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
     const int ks = warp % KS, rs = warp / KS;
     const int nvec = a.in / VE;
     const size_t row_bytes = Q8 ? (size_t)a.in : (size_t)a.in * 2;
-    const bool swiglu = a.epilogue == EPI_SWIGLU;
+    const bool swiglu = !STK && a.epilogue == EPI_SWIGLU;
 
     const int p_begin = (int)((long long)n_pairs * blockIdx.x / gridDim.x);
     const int p_end = (int)((long long)n_pairs * (blockIdx.x + 1) / gridDim.x);
@@ -108,7 +109,7 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
     // descriptor and constant tables, not from the predecessor -- staged in shared memory here, before the dependency
     // wait, so that the epilogues of the row groups (and the kernel's tail) hold no chain of global loads
     __shared__ RopeStage rope_stage;
-    const bool rope_staged = a.epilogue == EPI_ROPE_KV && a.dh <= 128;
+    const bool rope_staged = !STK && a.epilogue == EPI_ROPE_KV && a.dh <= 128;
     if (rope_staged) {
         const int half_dh = a.dh >> 1;
         for (int i = threadIdx.x; i < a.n_tok * half_dh; i += blockDim.x) {
@@ -262,7 +263,7 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
         // the finishing lanes ask for their residual pair now: it arrives while the group is multiplied and reduced
         EpiPre pre;
         if (rope_staged) pre.rope = &rope_stage;
-        if (a.epilogue == EPI_RESIDUAL && ks == 0 && rs < RS && lane < RP * NT) {
+        if (!STK && a.epilogue == EPI_RESIDUAL && ks == 0 && rs < RS && lane < RP * NT) {
             const int rp = lane / NT, t = lane - rp * NT;
             const int p = p_begin + g * group_pairs + rs * RP + rp;
             if (p < p_end && t < a.n_tok) {
@@ -363,7 +364,8 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
                     va += src[(2 * rp) * NT + t];
                     vb += src[(2 * rp + 1) * NT + t];
                 }
-                gemv_epilogue<T>(a, p, t, va, vb, pre);
+                if constexpr (STK) stack_epilogue<T>(a, p, t, va, vb);
+                else gemv_epilogue<T>(a, p, t, va, vb, pre);
             }
         }
     }
@@ -411,9 +413,9 @@ static GemvPlan plan_for(int in, bool q8, int nt) {
     return best;
 }
 
-template <class T, bool Q8, int NT, int KI, int RP, int PRO>
+template <class T, bool Q8, int NT, int KI, int RP, int PRO, bool STK>
 static int launch_inst(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaStream_t s, bool pdl, bool dry) {
-    auto kernel = gemv_kernel<T, Q8, NT, KI, RP, PRO>;
+    auto kernel = gemv_kernel<T, Q8, NT, KI, RP, PRO, STK>;
     // activations + double-buffered per-warp partial sums (also the RMSNorm scratch)
     size_t smem = (size_t)NT * a.in * sizeof(T) + (size_t)2 * 16 * (2 * RP * NT) * sizeof(float);
     int block = pl.nwarps * 32;
@@ -458,15 +460,18 @@ static int launch_inst(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaS
     return LCU_OK;
 }
 
-template <class T, bool Q8, int NT>
+template <class T, bool Q8, int NT, bool STK>
 static int launch_nt(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaStream_t s, bool pdl, bool dry) {
     // prologue variant: the one-token register form needs 16-bit norm weights and at most two vectors per thread
     const int pro = a.prologue != PRO_RMSNORM ? 0 : ((NT == 1 && !a.norm_f32 && a.lean_norm && a.in / 8 <= 2 * pl.nwarps * 32) ? 2 : 1);
 #define LCU_GEMV_CASE(KI_, RP_)                                                                                   \
     if (pl.KI == KI_ && pl.RP == RP_) {                                                                           \
-        if (pro == 0) return launch_inst<T, Q8, NT, KI_, RP_, 0>(a, pl, n_pairs, s, pdl, dry);                    \
-        if (pro == 1) return launch_inst<T, Q8, NT, KI_, RP_, 1>(a, pl, n_pairs, s, pdl, dry);                    \
-        if constexpr (NT == 1) return launch_inst<T, Q8, NT, KI_, RP_, 2>(a, pl, n_pairs, s, pdl, dry);           \
+        if (pro == 0) return launch_inst<T, Q8, NT, KI_, RP_, 0, STK>(a, pl, n_pairs, s, pdl, dry);               \
+        if constexpr (STK) return LCU_ERR_INVALID;                                                                \
+        else {                                                                                                    \
+        if (pro == 1) return launch_inst<T, Q8, NT, KI_, RP_, 1, STK>(a, pl, n_pairs, s, pdl, dry);                    \
+        if constexpr (NT == 1) return launch_inst<T, Q8, NT, KI_, RP_, 2, STK>(a, pl, n_pairs, s, pdl, dry);      \
+        }                                                                                                         \
     }
     if constexpr (Q8) {
         LCU_GEMV_CASE(1, 4) LCU_GEMV_CASE(1, 2) LCU_GEMV_CASE(2, 2) LCU_GEMV_CASE(4, 1) LCU_GEMV_CASE(8, 1)
@@ -482,15 +487,15 @@ static int launch_nt(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaStr
     return LCU_ERR_INVALID;
 }
 
-template <class T, bool Q8>
+template <class T, bool Q8, bool STK>
 static int launch_t(const GemvArgs &a, cudaStream_t s, bool pdl, bool dry) {
     int nt = a.n_tok <= 1 ? 1 : (a.n_tok == 2 ? 2 : 4);
     GemvPlan pl = plan_for(a.in, Q8, nt);
     int n_pairs = a.out / 2;
     switch (nt) {
-    case 1: return launch_nt<T, Q8, 1>(a, pl, n_pairs, s, pdl, dry);
-    case 2: return launch_nt<T, Q8, 2>(a, pl, n_pairs, s, pdl, dry);
-    default: return launch_nt<T, Q8, 4>(a, pl, n_pairs, s, pdl, dry);
+    case 1: return launch_nt<T, Q8, 1, STK>(a, pl, n_pairs, s, pdl, dry);
+    case 2: return launch_nt<T, Q8, 2, STK>(a, pl, n_pairs, s, pdl, dry);
+    default: return launch_nt<T, Q8, 4, STK>(a, pl, n_pairs, s, pdl, dry);
     }
 }
 
@@ -512,10 +517,14 @@ int gemv_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry) {
         LCU_REQUIRE(a.out == a.qd + 2 * a.kvd && a.dh % 2 == 0, "gemv: rope/kv epilogue shape mismatch");
     GemvArgs b = a;
     b.lean_norm = tuning().gemv_lean_norm;
-    if (dt == LCU_F16) return b.w_q8 ? launch_t<__half, true>(b, s, pdl, dry) : launch_t<__half, false>(b, s, pdl, dry);
+    if (b.epilogue >= EPI_STORE_F32) {
+        LCU_REQUIRE(dt == LCU_BF16 && !b.w_q8, "gemv: epilogue %d takes bf16 activations and weights", b.epilogue);
+        return launch_t<__nv_bfloat16, false, true>(b, s, pdl, dry);
+    }
+    if (dt == LCU_F16) return b.w_q8 ? launch_t<__half, true, false>(b, s, pdl, dry) : launch_t<__half, false, false>(b, s, pdl, dry);
     if (dt == LCU_BF16) {
         LCU_REQUIRE(!b.w_q8, "gemv: Q8_0 weights are supported with f16 activations only");
-        return launch_t<__nv_bfloat16, false>(b, s, pdl, dry);
+        return launch_t<__nv_bfloat16, false, false>(b, s, pdl, dry);
     }
     set_error("gemv: activation dtype %d unsupported", dt);
     return LCU_ERR_INVALID;
@@ -527,12 +536,12 @@ namespace lcu {
 // Sets the shared-memory attribute and caches the occupancy of every kernel variant a
 // context with these shapes can launch, so that nothing of the kind happens inside a
 // stream capture.
-int gemv_warm(int in, int out, bool q8, int dt) {
+int gemv_warm(int in, int out, bool q8, int dt, int epilogue) {
     for (int nt = 1; nt <= gemv_max_tokens(in); nt *= 2) {
         GemvArgs a{};
-        a.in = in; a.out = out; a.n_tok = nt; a.w_q8 = q8; a.stride_x = in; a.epilogue = EPI_STORE;
+        a.in = in; a.out = out; a.n_tok = nt; a.w_q8 = q8; a.stride_x = in; a.epilogue = epilogue;
         // every prologue variant: none, RMSNorm with 16-bit and with f32 norm weights
-        for (int v = 0; v < 3; ++v) {
+        for (int v = 0; v < (epilogue >= EPI_STORE_F32 ? 1 : 3); ++v) {
             a.prologue = v == 0 ? PRO_NONE : PRO_RMSNORM;
             a.norm_f32 = v == 2;
             int rc = gemv_launch(a, dt, nullptr, false, true);

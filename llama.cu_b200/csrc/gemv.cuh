@@ -7,7 +7,9 @@
 namespace lcu {
 
 enum GemvPrologue { PRO_NONE = 0, PRO_RMSNORM = 1 };
-enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU = 3 };
+enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU = 3,
+                    EPI_STORE_F32 = 4,  // y is f32
+                    EPI_XIELU = 5 };    // y = xielu(row) with the two numbers at act_pq
 
 struct GemvArgs {
     // weights [out, in] row-major in the activation dtype, or Q8_0 planes
@@ -41,6 +43,7 @@ struct GemvArgs {
     const int32_t *tok_seq;     // [n_tok] sequence slot of each token
     const int32_t *page_table;  // [slots, pt_stride]
     int pt_stride;
+    const float *act_pq;  // EPI_XIELU: p, q
     // EPI_SWIGLU: rows [0,di) gate, [di,2di) up; y gets [n_tok, di]
     int di;
     // tuning: 0 = trigger dependents at kernel start, 1 = after the main loop, 2 = never (implicit at exit)
@@ -55,6 +58,12 @@ struct GemvArgs {
 // ---- fused epilogue of one row pair for one token, shared by the GEMV and the batched kernel
 __device__ __forceinline__ float swiglu_act(float gate, float up) {
     return gate * __fdividef(1.f, 1.f + expf(-gate)) * up;
+}
+
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// xIELU with sp = softplus(p), sq = softplus(q): quadratic above zero, a scaled exp(z) - 1 - z below, both plus z / 2
+__device__ __forceinline__ float xielu_act(float z, float sp, float sq) {
+    return z > 0.f ? fmaf(sp * z, z, 0.5f * z) : fmaf(0.5f + sq, expm1f(z) - z, 0.5f * z);
 }
 
 // Values an epilogue would otherwise fetch from global memory behind the weight stream: the per-token constants of the
@@ -146,12 +155,24 @@ __device__ void gemv_epilogue(const GemvArgs &a, int pair, int t, float va, floa
     }
 }
 
+// Epilogues of layered models (never mixed with the ones above in one kernel instance of the GEMV): f32 rows for a norm
+// that follows in 32-bit, or the activated row.
+template <class T>
+__device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int t, float va, float vb) {
+    const size_t off = (size_t)t * a.stride_y + (size_t)pair * 2;
+    if (a.epilogue == EPI_STORE_F32) {
+        *reinterpret_cast<float2 *>(reinterpret_cast<float *>(a.y) + off) = make_float2(va, vb);
+    } else {
+        const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
+        *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(xielu_act(va, sp, sq), xielu_act(vb, sp, sq));
+    }
+}
 #endif  // __CUDACC__
 
 // Enqueues one GEMV; dt = LCU_F16 / LCU_BF16.  pdl: launch with programmatic serialisation.
 int gemv_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry = false);
 // Prepares (attributes, occupancy) every variant used for this shape without launching.
-int gemv_warm(int in, int out, bool q8, int dt);
+int gemv_warm(int in, int out, bool q8, int dt, int epilogue = EPI_STORE);
 // Batched form for up to 64 tokens per launch (gemm_skinny.cu): same arguments and epilogues, but the
 // activations must be prepared (no RMSNorm prologue, no row gather).
 bool gemm_skinny_supported(int in, int w_q8);

@@ -24,27 +24,32 @@ template <class T> __device__ __forceinline__ float bits_to_f(uint16_t b);
 template <> __device__ __forceinline__ float bits_to_f<__half>(uint16_t b) { return __half2float(__ushort_as_half(b)); }
 template <> __device__ __forceinline__ float bits_to_f<__nv_bfloat16>(uint16_t b) { return __uint_as_float((uint32_t)b << 16); }
 
-struct ArgPair {
-    float v;
-    uint32_t i;
-    uint16_t bits;
-};
+// Rows of f32 logits (T = float): the arg-max compares them in full; the stochastic sampler, whose keys are 16 bits wide,
+// and the value reported in the pair round them to bf16 first.
+template <> __device__ __forceinline__ float bits_to_f<float>(uint16_t b) { return __uint_as_float((uint32_t)b << 16); }
+template <class T> struct LogitRaw { using type = uint16_t; };
+template <> struct LogitRaw<float> { using type = float; };
+template <class T> __device__ __forceinline__ float logit_f(uint16_t v) { return bits_to_f<T>(v); }
+template <class T> __device__ __forceinline__ float logit_f(float v) { return v; }
+__device__ __forceinline__ uint16_t logit_bits(uint16_t v) { return v; }
+__device__ __forceinline__ uint16_t logit_bits(float v) { return __bfloat16_as_ushort(__float2bfloat16_rn(v)); }
+
 __device__ __forceinline__ bool arg_better(float v, uint32_t i, float bv, uint32_t bi) {
     return v > bv || (v == bv && i < bi);
 }
 
 template <class T>
-__global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t *__restrict__ logits, size_t n, int nblk,
+__global__ void __launch_bounds__(256) argmax_partial_kernel(const typename LogitRaw<T>::type *__restrict__ logits, size_t ld, size_t n, int nblk,
                                                              float *__restrict__ pv, uint32_t *__restrict__ pi) {
     grid_dep_launch();
     grid_dep_wait();
     const int row = blockIdx.y, blk = blockIdx.x;
-    const uint16_t *x = logits + (size_t)row * n;
+    const typename LogitRaw<T>::type *x = logits + (size_t)row * ld;
     size_t begin = (size_t)blk * ARGMAX_CHUNK, end = begin + ARGMAX_CHUNK;
     if (end > n) end = n;
     float bv = -INFINITY;
     uint32_t bi = 0xffffffffu;
-    if (((reinterpret_cast<uintptr_t>(x) | (n * 2)) & 15) == 0) {
+    if (sizeof(*x) == 2 && ((reinterpret_cast<uintptr_t>(x) | (n * 2)) & 15) == 0) {
         // rows that start on 16 bytes: eight values per load (the order of the visits does not matter, ties go to the
         // lower index through arg_better)
         for (size_t i = begin + 8 * (size_t)threadIdx.x; i < end; i += 8 * (size_t)blockDim.x) {
@@ -58,7 +63,7 @@ __global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t *__r
         }
     } else {
         for (size_t i = begin + threadIdx.x; i < end; i += blockDim.x) {
-            float v = bits_to_f<T>(x[i]);
+            float v = logit_f<T>(x[i]);
             if (arg_better(v, (uint32_t)i, bv, bi) || bi == 0xffffffffu) { bv = v; bi = (uint32_t)i; }
         }
     }
@@ -82,7 +87,7 @@ __global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t *__r
 }
 
 template <class T>
-__global__ void __launch_bounds__(256) argmax_final_kernel(const uint16_t *__restrict__ logits, size_t n, int nblk,
+__global__ void __launch_bounds__(256) argmax_final_kernel(const typename LogitRaw<T>::type *__restrict__ logits, size_t ld, int nblk,
                                                            const float *__restrict__ pv, const uint32_t *__restrict__ pi,
                                                            const lcu_sample_args *__restrict__ args,
                                                            lcu_kv_pair *__restrict__ out, lcu_kv_pair *__restrict__ out_copy) {
@@ -116,7 +121,7 @@ __global__ void __launch_bounds__(256) argmax_final_kernel(const uint16_t *__res
             if (si[w] != 0xffffffffu && (bi == 0xffffffffu || arg_better(sv[w], si[w], bv, bi))) { bv = sv[w]; bi = si[w]; }
         lcu_kv_pair r;
         r.idx = bi;
-        r.val = logits[(size_t)row * n + bi];
+        r.val = logit_bits(logits[(size_t)row * ld + bi]);
         r.pad = 0;
         out[row] = r;
         if (out_copy) out_copy[row] = r;
@@ -132,7 +137,7 @@ constexpr int SAMPLE_BINS = 65536;
 constexpr int BINS_PER_THREAD = SAMPLE_BINS / SAMPLE_THREADS;
 
 template <class T>
-__global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const uint16_t *__restrict__ logits, size_t n,
+__global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const typename LogitRaw<T>::type *__restrict__ logits, size_t ld, size_t n,
                                                                     const lcu_sample_args *__restrict__ args,
                                                                     const float *__restrict__ randoms,
                                                                     uint32_t *__restrict__ hist_all,
@@ -143,7 +148,7 @@ __global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const uint16
     const int row = blockIdx.x, tid = threadIdx.x;
     const lcu_sample_args sa = args[row];
     if (sa.temperature == 0.f || sa.top_k == 1) return;  // arg-max rows are handled elsewhere
-    const uint16_t *x = logits + (size_t)row * n;
+    const typename LogitRaw<T>::type *x = logits + (size_t)row * ld;
     uint32_t *hist = hist_all + (size_t)row * SAMPLE_BINS;
 
     __shared__ double s_w[SAMPLE_THREADS];
@@ -156,7 +161,7 @@ __global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const uint16
     for (int b = tid; b < SAMPLE_BINS; b += SAMPLE_THREADS) hist[b] = 0;
     if (tid == 0) { s_max = -1; s_bin = -1; s_rank = 1; s_found = 0; s_cumk = -1.0; }
     __syncthreads();
-    for (size_t i = tid; i < n; i += SAMPLE_THREADS) atomicAdd(&hist[key_of(x[i])], 1u);
+    for (size_t i = tid; i < n; i += SAMPLE_THREADS) atomicAdd(&hist[key_of(logit_bits(x[i]))], 1u);
     __syncthreads();
 
     // thread `tid` owns bins hi, hi-1, ..., hi-63 (descending keys); thread 0 holds the largest keys
@@ -271,7 +276,7 @@ __global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const uint16
     uint32_t seen = 0;
     for (size_t base = 0; base < n; base += SAMPLE_THREADS) {
         size_t i = base + tid;
-        bool hit = i < n && key_of(x[i]) == (uint32_t)bin;
+        bool hit = i < n && key_of(logit_bits(x[i])) == (uint32_t)bin;
         unsigned bal = __ballot_sync(0xffffffffu, hit);
         if (lane == 0) s_cnt[warp] = __popc(bal);
         __syncthreads();
@@ -284,7 +289,7 @@ __global__ void __launch_bounds__(SAMPLE_THREADS) sample_row_kernel(const uint16
         if (hit && my == (uint32_t)rank) {
             lcu_kv_pair r;
             r.idx = (uint32_t)i;
-            r.val = x[i];
+            r.val = logit_bits(x[i]);
             r.pad = 0;
             out[row] = r;
             if (out_copy) out_copy[row] = r;
@@ -306,38 +311,39 @@ size_t sample_workspace_bytes(int rows, size_t n) {
     return argmax_workspace_bytes(rows, n) + align256((size_t)rows * SAMPLE_BINS * 4);
 }
 
+template <class T>
+static int sample_rows_t(lcu_kv_pair *out, lcu_kv_pair *out_copy, const void *logits, size_t ld, int rows, size_t n,
+                         const lcu_sample_args *args_dev, const float *randoms_dev, float *pv, uint32_t *pi, uint32_t *hist, cudaStream_t s,
+                         bool pdl, bool any_sampling) {
+    const int nblk = n_blocks(n);
+    const typename LogitRaw<T>::type *lg = reinterpret_cast<const typename LogitRaw<T>::type *>(logits);
+    LCU_CHECK_CUDA(launch_kernel(argmax_partial_kernel<T>, dim3(nblk, rows), dim3(256), 0, s, pdl, lg, ld, n, nblk, pv, pi));
+    LCU_CHECK_CUDA(launch_kernel(argmax_final_kernel<T>, dim3(rows), dim3(256), 0, s, pdl, lg, ld, nblk, (const float *)pv,
+                                 (const uint32_t *)pi, args_dev, out, out_copy));
+    if (any_sampling)
+        LCU_CHECK_CUDA(launch_kernel(sample_row_kernel<T>, dim3(rows), dim3(SAMPLE_THREADS), 0, s, false, lg, ld, n, args_dev, randoms_dev,
+                                     hist, out, out_copy));
+    return LCU_OK;
+}
+
 int sample_rows(lcu_kv_pair *out, lcu_kv_pair *out_copy, const void *logits, int rows, size_t n,
                 const lcu_sample_args *args_dev, const float *randoms_dev, int dt, void *workspace,
-                size_t workspace_len, cudaStream_t s, bool pdl, bool any_sampling) {
+                size_t workspace_len, cudaStream_t s, bool pdl, bool any_sampling, size_t ld) {
     if (rows <= 0) return LCU_OK;
-    LCU_REQUIRE(dt == LCU_F16 || dt == LCU_BF16, "sample: logits dtype %d unsupported", dt);
-    LCU_REQUIRE(n > 0 && n < 0xffffffffull, "sample: n = %zu", n);
+    if (ld == 0) ld = n;
+    LCU_REQUIRE(dt == LCU_F16 || dt == LCU_BF16 || dt == LCU_F32, "sample: logits dtype %d unsupported", dt);
+    LCU_REQUIRE(n > 0 && n < 0xffffffffull && ld >= n, "sample: n = %zu, row stride %zu", n, ld);
     if (!args_dev) any_sampling = false;
     size_t need = any_sampling ? sample_workspace_bytes(rows, n) : argmax_workspace_bytes(rows, n);
     LCU_REQUIRE(workspace && workspace_len >= need, "sample: workspace of %zu bytes, %zu needed", workspace_len, need);
     LCU_REQUIRE(!any_sampling || randoms_dev, "sample: sampling rows need random numbers");
-    int nblk = n_blocks(n);
     unsigned char *p = reinterpret_cast<unsigned char *>(workspace);
     float *pv = reinterpret_cast<float *>(p);
-    uint32_t *pi = reinterpret_cast<uint32_t *>(p + align256((size_t)rows * nblk * 4));
+    uint32_t *pi = reinterpret_cast<uint32_t *>(p + align256((size_t)rows * n_blocks(n) * 4));
     uint32_t *hist = reinterpret_cast<uint32_t *>(p + argmax_workspace_bytes(rows, n));
-    const uint16_t *lg = reinterpret_cast<const uint16_t *>(logits);
-    if (dt == LCU_F16) {
-        LCU_CHECK_CUDA(launch_kernel(argmax_partial_kernel<__half>, dim3(nblk, rows), dim3(256), 0, s, pdl, lg, n, nblk, pv, pi));
-        LCU_CHECK_CUDA(launch_kernel(argmax_final_kernel<__half>, dim3(rows), dim3(256), 0, s, pdl, lg, n, nblk,
-                                     (const float *)pv, (const uint32_t *)pi, args_dev, out, out_copy));
-        if (any_sampling)
-            LCU_CHECK_CUDA(launch_kernel(sample_row_kernel<__half>, dim3(rows), dim3(SAMPLE_THREADS), 0, s, false, lg, n,
-                                         args_dev, randoms_dev, hist, out, out_copy));
-    } else {
-        LCU_CHECK_CUDA(launch_kernel(argmax_partial_kernel<__nv_bfloat16>, dim3(nblk, rows), dim3(256), 0, s, pdl, lg, n, nblk, pv, pi));
-        LCU_CHECK_CUDA(launch_kernel(argmax_final_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, pdl, lg, n, nblk,
-                                     (const float *)pv, (const uint32_t *)pi, args_dev, out, out_copy));
-        if (any_sampling)
-            LCU_CHECK_CUDA(launch_kernel(sample_row_kernel<__nv_bfloat16>, dim3(rows), dim3(SAMPLE_THREADS), 0, s, false, lg,
-                                         n, args_dev, randoms_dev, hist, out, out_copy));
-    }
-    return LCU_OK;
+    if (dt == LCU_F16) return sample_rows_t<__half>(out, out_copy, logits, ld, rows, n, args_dev, randoms_dev, pv, pi, hist, s, pdl, any_sampling);
+    if (dt == LCU_F32) return sample_rows_t<float>(out, out_copy, logits, ld, rows, n, args_dev, randoms_dev, pv, pi, hist, s, pdl, any_sampling);
+    return sample_rows_t<__nv_bfloat16>(out, out_copy, logits, ld, rows, n, args_dev, randoms_dev, pv, pi, hist, s, pdl, any_sampling);
 }
 
 }  // namespace lcu

@@ -1,0 +1,498 @@
+// Rounds of models described layer by layer: shapes and storage, the plan of a round's attention, and the launches of every
+// layer.  Context, pages, descriptor staging, graphs and sampling are those of ctx.cu.
+#include "ctx.cuh"
+#include "gemv.cuh"
+#include "stack.cuh"
+
+namespace lcu {
+
+static size_t align256(size_t v) { return (v + 255) & ~(size_t)255; }
+static size_t act_bytes(const lcu_ctx *c) { return c->dt == LCU_F32 ? 4 : 2; }
+
+// offsets inside the stack section of the round descriptor
+struct StackDesc {
+    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, total;
+};
+constexpr int EXPAND_GROUP = 64;  // query tokens per group of the expanded attention
+static StackDesc stack_desc(int n_tok, int n_req) {
+    StackDesc d;
+    size_t o = 0;
+    auto take = [&](size_t bytes) { size_t r = o; o += (bytes + 15) & ~(size_t)15; return r; };
+    d.req_first = take((size_t)(n_req + 1) * 4);
+    d.req_pos = take((size_t)n_req * 4);
+    d.req_slot = take((size_t)n_req * 4);
+    d.abs_first = take((size_t)(n_req + 1) * 4);
+    d.abs_id = take((size_t)n_req * 4);
+    d.abs_tok = take((size_t)n_tok * 4);
+    d.xreq = take((size_t)n_req * 16);
+    d.xgroups = take((size_t)(n_tok / EXPAND_GROUP + n_req) * 16);
+    d.total = o;
+    return d;
+}
+size_t stack_desc_bytes(int max_tok, int max_req) { return stack_desc(max_tok, max_req).total; }
+
+// Fewest tokens of a portion for which expanding pays: per cached token and head the absorbed form multiplies 2 r_p
+// numbers per query, the expanded one dim + v_dim per query plus r_p (dim + v_dim) for the expansion itself.
+static int layer_expand_min(const StackLayer &L) {
+    const int t = tuning().expand_min;
+    if (t < 0 || !expanded_attn_supported(L.dim_p, L.vdim_p)) return 1 << 30;
+    if (t > 0) return t < 2 ? 2 : t;
+    const long kv = L.dim_p + L.vdim_p, gain = 2l * L.r_p - kv;
+    if (gain <= 0) return 1 << 30;
+    const long n = L.r_p * kv / gain + 1;
+    return n < 16 ? 16 : (int)n;
+}
+static int round_expand_min(const Stack &S) {
+    int m = 2;  // one decision per request and round: the most demanding layer decides
+    for (const StackLayer &L : S.layers) { const int v = layer_expand_min(L); if (v > m) m = v; }
+    return m;
+}
+
+// Split-KV depth of the absorbed attention for a round: enough CTAs to fill the SMs once (a CTA takes most of an SM's shared
+// memory) when every context is full, fixed per round shape so that captured rounds stay valid.
+static int attn_splits_for(const lcu_ctx *c, int blocks) {
+    if (c->dt == LCU_F32) return 1;
+    const int tiles = (c->desc.nctx + 63) / 64;
+    int z = (sm_count() + blocks - 1) / (blocks > 0 ? blocks : 1);
+    if (z > 32) z = 32;
+    if (z > tiles) z = tiles;
+    return z < 1 ? 1 : z;
+}
+
+static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, int i) {
+    const lcu_layer_desc &l = layers[i];
+    LCU_REQUIRE(l.mixer == LCU_MIX_LATENT, "layer %d: unknown mixer %d", i, l.mixer);
+    LCU_REQUIRE(l.heads > 0 && l.dim > 0 && l.v_dim > 0 && l.q_rank > 0 && l.kv_rank > 0 && l.ff >= 0, "layer %d: non-positive size", i);
+    LCU_REQUIRE(l.kv_rank <= 512 && l.dim <= 512, "layer %d: latent of %d, head size %d (at most 512)", i, l.kv_rank, l.dim);
+    LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_XIELU, "layer %d: unknown activation %d", i, l.ff_act);
+    LCU_REQUIRE(l.weights_of >= -1 && l.weights_of < d.n_layers && l.weights_of != i, "layer %d uses the weights of layer %d", i, l.weights_of);
+    return LCU_OK;
+}
+
+int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
+    const lcu_model_desc &d = c->desc;
+    for (int i = 0; i < d.n_layers; ++i) {
+        int rc = check_layer(d, layers, i);
+        if (rc) return rc;
+    }
+    Stack *S = new Stack();
+    c->stack = S;
+    S->d_p = stack_pad(d.d, 64);
+    S->vocab_p = stack_pad(d.vocab, 8);
+    S->layers.resize(d.n_layers);
+    S->w.resize(d.n_layers);
+    size_t off = 0;
+    int max_lat = 0, max_qr = 0, max_q = 0, max_hr = 0, max_hv = 64, max_ff = 64, max_kv = 0;
+    bool any_shift = false, can_expand = c->dt != LCU_F32;
+    for (int i = 0; i < d.n_layers; ++i) {
+        StackLayer &L = S->layers[i];
+        L.d = layers[i];
+        L.src = i;
+        for (int hops = 0; layers[L.src].weights_of >= 0; ++hops) {
+            LCU_REQUIRE(hops < d.n_layers, "layer %d: the shared weights form a circle", i);
+            L.src = layers[L.src].weights_of;
+        }
+        const lcu_layer_desc &o = layers[L.src];
+        LCU_REQUIRE(o.heads == L.d.heads && o.dim == L.d.dim && o.v_dim == L.d.v_dim && o.q_rank == L.d.q_rank && o.kv_rank == L.d.kv_rank &&
+                        o.out_gate == L.d.out_gate && o.ff == L.d.ff && o.token_shift == L.d.token_shift,
+                    "layer %d differs from layer %d whose weights it uses", i, L.src);
+        L.dim_p = stack_pad(L.d.dim, 16);
+        L.vdim_p = stack_pad(L.d.v_dim, 16);
+        L.qr_p = stack_pad(L.d.q_rank, 64);
+        L.r_p = stack_pad(L.d.kv_rank, 64);
+        L.g_p = L.d.out_gate ? stack_pad(L.d.heads, 8) : 0;
+        L.ff_p = stack_pad(L.d.ff, 64);
+        L.hv_p = stack_pad(L.d.heads * L.vdim_p, 64);
+        L.c_off = off;
+        off += (size_t)L.r_p * c->geom.page_tokens;
+        any_shift = any_shift || L.d.token_shift;
+        can_expand = can_expand && expanded_attn_supported(L.dim_p, L.vdim_p);
+        auto up = [](int &m, int v) { if (v > m) m = v; };
+        up(max_lat, L.in_rows()); up(max_qr, L.qr_p); up(max_q, L.d.heads * L.dim_p); up(max_hr, L.d.heads * L.r_p);
+        up(max_hv, L.hv_p); up(max_ff, L.ff_p); up(max_kv, L.kv_cols()); up(S->max_heads, L.d.heads); up(S->max_r, L.r_p);
+    }
+    c->geom.page_elems = off;
+    S->n_slots = any_shift ? c->max_seqs : 0;
+    c->free_slots.clear();
+    for (int i = S->n_slots - 1; i >= 0; --i) c->free_slots.push_back(i);
+
+    const size_t T = (size_t)c->max_tokens, eb = act_bytes(c);
+    S->abs_cap = c->max_tokens;
+    S->expand_cap = can_expand ? stack_pad(d.nctx > c->max_tokens ? d.nctx : c->max_tokens, 64) : 0;
+    // partial rows: a small round is split so that about one CTA per SM runs, a large one is not split
+    size_t rows = 0;
+    for (const StackLayer &L : S->layers)
+        for (int dec = 0; dec < 2; ++dec)
+            for (int n = 1; n <= c->max_tokens; n = n < 64 ? n + 1 : (n == c->max_tokens ? n + 1 : (2 * n < c->max_tokens ? 2 * n : c->max_tokens))) {
+                const int rpb = latent_attn_rows_per_block(L.d.heads, L.r_p, dec != 0, c->dt);
+                const int blocks = dec ? n * ((L.d.heads + rpb - 1) / rpb) : n * L.d.heads / rpb + 1;
+                // between two sampled sizes the split depth does not grow while the rows at most double
+                const size_t r = (size_t)(n < 64 || n == c->max_tokens ? n : 2 * n) * L.d.heads * attn_splits_for(c, blocks);
+                if (r > rows) rows = r;
+            }
+    S->part_rows = rows;
+    size_t total = 0;
+    auto reserve = [&](size_t bytes) { size_t r = total; total += align256(bytes); return r; };
+    const size_t o_x0 = reserve(T * S->d_p * 4), o_x1 = reserve(T * S->d_p * 4), o_y = reserve(T * S->d_p * 4), o_lat = reserve(T * max_lat * 4),
+                 o_state = reserve((size_t)2 * d.n_layers * S->n_slots * S->d_p * 4), o_h = reserve(T * S->d_p * eb), o_cq = reserve(T * max_qr * eb),
+                 o_q = reserve(T * max_q * eb), o_qa = reserve(T * max_hr * eb), o_att = reserve(T * max_hv * eb), o_act = reserve(T * max_ff * eb),
+                 o_xc = reserve((size_t)S->expand_cap * S->max_r * eb), o_xkv = reserve((size_t)S->expand_cap * max_kv * eb),
+                 o_hout = reserve((T > (size_t)c->max_seqs ? T : c->max_seqs) * S->d_p * eb), o_po = reserve(rows * S->max_r * 4),
+                 o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4);
+    LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
+    LCU_CHECK_CUDA(cudaMemset(S->arena, 0, total));  // pads of att (columns past the heads) stay zero from here on
+    unsigned char *p = reinterpret_cast<unsigned char *>(S->arena);
+    S->x[0] = reinterpret_cast<float *>(p + o_x0); S->x[1] = reinterpret_cast<float *>(p + o_x1);
+    S->y = reinterpret_cast<float *>(p + o_y); S->lat = reinterpret_cast<float *>(p + o_lat); S->state = reinterpret_cast<float *>(p + o_state);
+    S->h = p + o_h; S->cq = p + o_cq; S->q = p + o_q; S->qa = p + o_qa; S->att = p + o_att; S->act = p + o_act;
+    S->xc = p + o_xc; S->xkv = p + o_xkv; S->hout = p + o_hout;
+    S->part_o = reinterpret_cast<float *>(p + o_po); S->part_ml = reinterpret_cast<float *>(p + o_pml); S->part_n = reinterpret_cast<int *>(p + o_pn);
+
+    // every kernel variant a round can launch
+    int rc = latent_attn_launch(LatentAttnArgs{}, c->dt, nullptr, false, true);
+    if (rc || c->dt == LCU_F32) return rc;
+    rc = head_linear_launch(HeadLinearArgs{}, nullptr, false, true);
+    if (!rc) rc = gemm_tc_warm(c->dt);
+    for (const StackLayer &L : S->layers) {
+        if (rc) break;
+        if (S->expand_cap) {
+            ExpandedAttnArgs e{};
+            e.dim_p = L.dim_p; e.vdim_p = L.vdim_p;
+            rc = expanded_attn_launch(e, nullptr, true);
+        }
+        if (!rc) rc = gemv_warm(S->d_p, L.in_rows(), false, c->dt, EPI_STORE_F32);
+        if (!rc) rc = gemv_warm(L.qr_p, L.d.heads * L.dim_p, false, c->dt);
+        if (!rc) rc = gemv_warm(L.hv_p, S->d_p, false, c->dt, EPI_STORE_F32);
+        if (!rc && L.d.ff) rc = gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_XIELU);
+        if (!rc && L.d.ff) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
+    }
+    if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt);
+    if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, EPI_STORE_F32);
+    return rc;
+}
+
+void stack_destroy(lcu_ctx *c) {
+    if (!c->stack) return;
+    if (c->stack->arena) cudaFree(c->stack->arena);
+    delete c->stack;
+    c->stack = nullptr;
+}
+
+// ------------------------------------------------------------------ weights
+
+bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *cols, int *elem_bytes) {
+    const Stack &S = *c->stack;
+    *elem_bytes = 2;
+    switch (kind) {
+    case LCU_W_EMBD: *rows = c->desc.vocab; *cols = S.d_p; return true;
+    case LCU_W_LM_HEAD: *rows = S.vocab_p; *cols = S.d_p; return true;
+    case LCU_W_OUT_NORM: *rows = 1; *cols = 1; *elem_bytes = 4; return true;
+    default: break;
+    }
+    if (layer < 0 || layer >= c->desc.n_layers || S.layers[layer].src != layer) return false;
+    const StackLayer &L = S.layers[layer];
+    switch (kind) {
+    case LCU_W_LAT_IN: *rows = L.in_rows(); *cols = S.d_p; return true;
+    case LCU_W_Q_NORM: *rows = 1; *cols = L.qr_p; return true;
+    case LCU_W_KV_NORM: *rows = 1; *cols = L.r_p; return true;
+    case LCU_W_UQ: *rows = L.d.heads * L.dim_p; *cols = L.qr_p; return true;
+    case LCU_W_UKT: *rows = L.d.heads * L.r_p; *cols = L.dim_p; return true;
+    case LCU_W_UKV: *rows = L.kv_cols(); *cols = L.r_p; return true;
+    case LCU_W_LAT_OUT: *rows = S.d_p; *cols = L.hv_p; return true;
+    case LCU_W_UP: *rows = L.ff_p; *cols = S.d_p; return L.d.ff > 0;
+    case LCU_W_FF_DOWN: *rows = S.d_p; *cols = L.ff_p; return L.d.ff > 0;
+    case LCU_W_SHIFT: *rows = 1; *cols = S.d_p; return L.d.token_shift != 0;
+    case LCU_W_SCALARS: *rows = 1; *cols = 4; *elem_bytes = 4; return true;
+    default: return false;
+    }
+}
+
+int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
+    StackWeights &w = c->stack->w[layer];
+    switch (kind) {
+    case LCU_W_LAT_IN: w.in = ptr; break;
+    case LCU_W_Q_NORM: w.q_norm = ptr; break;
+    case LCU_W_KV_NORM: w.kv_norm = ptr; break;
+    case LCU_W_UQ: w.uq = ptr; break;
+    case LCU_W_UKT: w.ukt = ptr; break;
+    case LCU_W_UKV: w.ukv = ptr; break;
+    case LCU_W_LAT_OUT: w.out = ptr; break;
+    case LCU_W_UP: w.up = ptr; break;
+    case LCU_W_FF_DOWN: w.down = ptr; break;
+    case LCU_W_SHIFT: w.shift = ptr; break;
+    case LCU_W_SCALARS: w.scalars = reinterpret_cast<const float *>(ptr); break;
+    default: set_error("set_weight: unknown kind %d", kind); return LCU_ERR_INVALID;
+    }
+    return LCU_OK;
+}
+
+bool stack_ready(const lcu_ctx *c) {
+    const Stack &S = *c->stack;
+    for (size_t i = 0; i < S.layers.size(); ++i) {
+        if (S.layers[i].src != (int)i) continue;
+        const StackWeights &w = S.w[i];
+        const lcu_layer_desc &d = S.layers[i].d;
+        if (!w.in || !w.q_norm || !w.kv_norm || !w.uq || !w.ukt || !w.ukv || !w.out || !w.scalars || (d.ff && (!w.up || !w.down)) ||
+            (d.token_shift && !w.shift)) {
+            set_error("step: weights of layer %zu missing", i);
+            return false;
+        }
+    }
+    return true;
+}
+
+// ------------------------------------------------------------------ the round
+
+int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
+    const Stack &S = *c->stack;
+    StackRound &q = r.sr;
+    q = StackRound();
+    const StackDesc D = stack_desc(r.n_tok, r.n_req);
+    unsigned char *B = H + r.L.stack;
+    int32_t *first = reinterpret_cast<int32_t *>(B + D.req_first), *pos = reinterpret_cast<int32_t *>(B + D.req_pos),
+            *slot = reinterpret_cast<int32_t *>(B + D.req_slot), *afirst = reinterpret_cast<int32_t *>(B + D.abs_first),
+            *aid = reinterpret_cast<int32_t *>(B + D.abs_id), *atok = reinterpret_cast<int32_t *>(B + D.abs_tok);
+    int4 *xreq = reinterpret_cast<int4 *>(B + D.xreq), *xg = reinterpret_cast<int4 *>(B + D.xgroups);
+    const int expand_min = S.expand_cap ? round_expand_min(S) : 1 << 30;
+    int t = 0, nx = 0, ng = 0;
+    StackRound::Batch cur{0, 0, 0, 0, 0};
+    for (int i = 0; i < r.n_req; ++i) {
+        const SeqState &sq = c->seqs[reqs[i].seq];
+        const int len = (int)reqs[i].len, ctx = (int)reqs[i].pos + len;
+        first[i] = t;
+        pos[i] = (int)reqs[i].pos;
+        slot[i] = sq.slot * 2 + sq.gen;
+        if (len < expand_min) {
+            aid[q.n_abs_req] = i;
+            afirst[q.n_abs_req++] = q.n_abs_tok;
+            for (int j = 0; j < len; ++j) atok[q.n_abs_tok++] = t + j;
+        } else {
+            if (cur.n_req && cur.n_rows + ctx > S.expand_cap) {  // the batch is full (one request always fits)
+                q.batches.push_back(cur);
+                cur = StackRound::Batch{0, nx, 0, ng, 0};
+            }
+            xreq[nx++] = make_int4(i, ctx, cur.n_rows, 0);
+            for (int j = 0; j < len; j += EXPAND_GROUP) {
+                xg[ng++] = make_int4(t + j, len - j < EXPAND_GROUP ? len - j : EXPAND_GROUP, pos[i] + j, cur.n_rows);
+                ++cur.n_groups;
+            }
+            cur.n_rows += ctx;
+            ++cur.n_req;
+        }
+        t += len;
+    }
+    first[r.n_req] = t;
+    afirst[q.n_abs_req] = q.n_abs_tok;
+    if (cur.n_req) q.batches.push_back(cur);
+    q.abs_decode = r.decode_only;
+    return LCU_OK;
+}
+
+namespace {
+
+struct Launcher {
+    lcu_ctx *c;
+    cudaStream_t s;
+    int *count;
+
+    // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
+    int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr) {
+        if (c->dt == LCU_F32) {
+            LinearF32Args a{};
+            a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w;
+            a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
+            a.n = n; a.in = in; a.out = out; a.heads = 1;
+            a.epilogue = epilogue == EPI_STORE ? EPI_STORE_F32 : epilogue;
+            a.act_pq = act_pq;
+            ++*count;
+            return linear_f32_launch(a, s);
+        }
+        const size_t yb = epilogue == EPI_STORE_F32 ? 4 : 2;
+        const bool tc = n > 4;
+        for (int t0 = 0; t0 < n;) {
+            const int most = tc ? tuning().tc_block : gemv_max_tokens(in);
+            const int nt = n - t0 < most ? n - t0 : most;
+            GemvArgs a{};
+            a.w = w;
+            a.x = reinterpret_cast<const unsigned char *>(x) + (size_t)t0 * in * 2;
+            a.stride_x = in; a.n_tok = nt; a.in = in; a.out = out;
+            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq;
+            a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
+            a.stride_y = stride_y;
+            a.pdl_trigger = 2;
+            a.early_prefetch = 1;
+            int rc = tc ? gemm_tc_launch(a, c->dt, s, false) : gemv_launch(a, c->dt, s, false);
+            if (rc) return rc;
+            ++*count;
+            t0 += nt;
+        }
+        return LCU_OK;
+    }
+};
+
+}  // namespace
+
+int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
+    Stack &S = *c->stack;
+    const lcu_model_desc &d = c->desc;
+    const int dt = c->dt, n = r.n_tok;
+    const size_t eb = act_bytes(c);
+    Launcher L{c, s, count};
+    unsigned char *D = c->desc_dev, *B = D + r.L.stack;
+    const StackDesc o = stack_desc(r.n_tok, r.n_req);
+    const uint32_t *tokens = reinterpret_cast<const uint32_t *>(D + r.L.tokens), *pos = reinterpret_cast<const uint32_t *>(D + r.L.pos);
+    const int32_t *tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req), *page_table = reinterpret_cast<const int32_t *>(D + r.L.page_table);
+    auto i32 = [&](size_t off) { return reinterpret_cast<const int32_t *>(B + off); };
+    const StackRound &q = r.sr;
+    gemm_tc_set_scratch(c->sk_ws, c->sk_ws_bytes, c->sk_tickets, 4096, c->dev_status);
+    int rc, cur = 0;
+
+    MixInputArgs mi{};
+    mi.n_tok = n; mi.d = d.d; mi.d_p = S.d_p; mi.eps = d.eps;
+    mi.state_gen_stride = (size_t)d.n_layers * S.n_slots * S.d_p;
+    mi.tok_req = tok_req; mi.req_first = i32(o.req_first); mi.req_pos = i32(o.req_pos); mi.req_slot = i32(o.req_slot);
+    mi.h = S.h;
+    // x (and the shifted input of layer `next`, if there is one) after a sublayer's output y; layer -1: the embedding
+    auto residual = [&](const float *gain, int next, bool mixer_input) -> int {
+        MixInputArgs a = mi;
+        if (gain) {
+            a.x_in = S.x[cur]; a.y = S.y; a.gain = gain;
+            cur ^= 1;
+        } else {
+            a.embd = c->embd; a.tokens = tokens;
+        }
+        a.x_out = S.x[cur];
+        if (mixer_input) {
+            if (next >= d.n_layers) a.h = nullptr;  // the head reads x itself
+            else if (S.layers[next].d.token_shift) {
+                a.shift = S.w[S.layers[next].src].shift;
+                a.state = S.state + (size_t)next * S.n_slots * S.d_p;
+            }
+        }
+        ++*count;
+        return op_mix_input(a, dt, s, false);
+    };
+    rc = residual(nullptr, 0, true);
+    if (rc) return rc;
+    for (int l = 0; l < d.n_layers; ++l) {
+        const StackLayer &Y = S.layers[l];
+        const StackWeights &W = S.w[Y.src];
+        const int heads = Y.d.heads, lat_stride = Y.in_rows(), q_stride = heads * Y.dim_p;
+        // --- both latents and the head gates in one projection; norms; append to the cache; queries
+        rc = L.linear(W.in, S.d_p, Y.in_rows(), S.h, n, S.lat, lat_stride, EPI_STORE_F32);
+        if (rc) return rc;
+        LatentNormArgs ln{};
+        ln.lat = S.lat; ln.stride = lat_stride; ln.n_tok = n; ln.q_rank = Y.d.q_rank; ln.qr_p = Y.qr_p; ln.kv_rank = Y.d.kv_rank; ln.r_p = Y.r_p;
+        ln.q_norm = W.q_norm; ln.kv_norm = W.kv_norm; ln.eps = d.eps; ln.cq = S.cq;
+        ln.pool = c->pool; ln.page_elems = c->geom.page_elems; ln.c_off = Y.c_off; ln.page_shift = c->geom.page_shift;
+        ln.tok_req = tok_req; ln.pos = pos; ln.page_table = page_table; ln.pt_stride = c->pt_stride;
+        rc = latent_norm_launch(ln, dt, s, false);
+        if (rc) return rc;
+        ++*count;
+        rc = L.linear(W.uq, Y.qr_p, q_stride, S.cq, n, S.q, q_stride, EPI_STORE);
+        if (rc) return rc;
+        const float *gate = Y.d.out_gate ? S.lat + Y.qr_p + Y.r_p : nullptr;
+        const unsigned char *uv = reinterpret_cast<const unsigned char *>(W.ukv) + (size_t)heads * Y.dim_p * Y.r_p * 2;
+
+        // --- absorbed form: queries into latent space, attention over the cached latents, value map of the merged rows
+        if (q.n_abs_tok) {
+            const int rpb = latent_attn_rows_per_block(heads, Y.r_p, q.abs_decode, dt);
+            const int blocks = q.abs_decode ? q.n_abs_tok * ((heads + rpb - 1) / rpb) : q.n_abs_tok * heads / rpb + 1;
+            const int splits = attn_splits_for(c, blocks);
+            LCU_REQUIRE((size_t)q.n_abs_tok * heads * splits <= S.part_rows, "step: attention partials of %d tokens do not fit", q.n_abs_tok);
+            LatentAttnArgs a{};
+            a.q = S.qa; a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift;
+            a.page_table = page_table; a.pt_stride = c->pt_stride; a.req_first = i32(o.abs_first); a.req_id = i32(o.abs_id); a.req_pos = i32(o.req_pos);
+            a.n_req = q.n_abs_req; a.n_tok = q.n_abs_tok; a.decode = q.abs_decode; a.heads = heads; a.r_p = Y.r_p; a.scale = Y.d.scale;
+            a.part_o = S.part_o; a.part_ml = S.part_ml; a.part_n = S.part_n; a.splits = splits;
+            if (dt == LCU_F32) {
+                LinearF32Args f{};
+                f.x = reinterpret_cast<const float *>(S.q); f.stride_x = q_stride; f.head_x = Y.dim_p; f.x_rows = i32(o.abs_tok);
+                f.w = W.ukt; f.y = reinterpret_cast<float *>(S.qa); f.stride_y = heads * Y.r_p; f.head_y = Y.r_p;
+                f.n = q.n_abs_tok; f.in = Y.dim_p; f.out = Y.r_p; f.heads = heads; f.epilogue = EPI_STORE_F32;
+                rc = linear_f32_launch(f, s);
+                if (!rc) rc = latent_attn_launch(a, dt, s, false);
+                f = LinearF32Args{};
+                f.x = S.part_o; f.stride_x = heads * Y.r_p; f.head_x = Y.r_p; f.w = uv;
+                f.y = reinterpret_cast<float *>(S.att); f.stride_y = Y.hv_p; f.head_y = Y.vdim_p; f.y_rows = i32(o.abs_tok);
+                f.n = q.n_abs_tok; f.in = Y.r_p; f.out = Y.vdim_p; f.heads = heads; f.epilogue = EPI_STORE_F32;
+                f.gate = gate; f.stride_gate = lat_stride;
+                if (!rc) rc = linear_f32_launch(f, s);
+            } else {
+                HeadLinearArgs f{};
+                f.x = S.q; f.stride_x = q_stride; f.head_x = Y.dim_p; f.x_rows = i32(o.abs_tok); f.w = W.ukt;
+                f.y = S.qa; f.stride_y = heads * Y.r_p; f.head_y = Y.r_p; f.n = q.n_abs_tok; f.in = Y.dim_p; f.out = Y.r_p; f.heads = heads;
+                rc = head_linear_launch(f, s, false);
+                if (!rc) rc = latent_attn_launch(a, dt, s, false);
+                f = HeadLinearArgs{};
+                f.w = uv; f.y = S.att; f.stride_y = Y.hv_p; f.head_y = Y.vdim_p; f.y_rows = i32(o.abs_tok);
+                f.n = q.n_abs_tok; f.in = Y.r_p; f.out = Y.vdim_p; f.heads = heads;
+                f.part_o = S.part_o; f.part_ml = S.part_ml; f.part_n = S.part_n; f.splits = splits;
+                f.gate = gate; f.stride_gate = lat_stride;
+                if (!rc) rc = head_linear_launch(f, s, false);
+            }
+            if (rc) return rc;
+            *count += 3;
+        }
+        // --- expanded form, a batch of requests at a time
+        for (const StackRound::Batch &b : q.batches) {
+            const int4 *xreq = reinterpret_cast<const int4 *>(B + o.xreq) + b.req0, *xg = reinterpret_cast<const int4 *>(B + o.xgroups) + b.group0;
+            rc = latent_gather_launch(S.xc, c->pool, c->geom.page_elems, Y.c_off, c->geom.page_shift, page_table, c->pt_stride, xreq, b.n_req,
+                                      b.n_rows, Y.r_p, s);
+            if (!rc) rc = L.linear(W.ukv, Y.r_p, Y.kv_cols(), S.xc, b.n_rows, S.xkv, Y.kv_cols(), EPI_STORE);
+            if (rc) return rc;
+            ExpandedAttnArgs a{};
+            a.q = S.q; a.stride_q = q_stride; a.kv = S.xkv; a.stride_kv = Y.kv_cols(); a.o = S.att; a.stride_o = Y.hv_p;
+            a.groups = xg; a.n_groups = b.n_groups; a.heads = heads; a.dim_p = Y.dim_p; a.vdim_p = Y.vdim_p; a.scale = Y.d.scale;
+            a.gate = gate; a.stride_gate = lat_stride;
+            rc = expanded_attn_launch(a, s);
+            if (rc) return rc;
+            *count += 2;
+        }
+        // --- output projection, norm of its result, residual
+        rc = L.linear(W.out, Y.hv_p, S.d_p, S.att, n, S.y, S.d_p, EPI_STORE_F32);
+        if (!rc) rc = residual(W.scalars, l + 1, Y.d.ff == 0);
+        if (rc || !Y.d.ff) {
+            if (rc) return rc;
+            continue;
+        }
+        // --- feed-forward
+        rc = L.linear(W.up, S.d_p, Y.ff_p, S.h, n, S.act, Y.ff_p, EPI_XIELU, W.scalars + 2);
+        if (!rc) rc = L.linear(W.down, Y.ff_p, S.d_p, S.act, n, S.y, S.d_p, EPI_STORE_F32);
+        if (!rc) rc = residual(W.scalars + 1, l + 1, true);
+        if (rc) return rc;
+    }
+    (void)eb;
+    c->x = S.x[cur];
+    return LCU_OK;
+}
+
+int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, float *out_f32, cudaStream_t s, int *count) {
+    (void)r;
+    if (n_rows <= 0) return LCU_OK;
+    Stack &S = *c->stack;
+    int rc = op_scalar_norm_rows(S.hout, reinterpret_cast<const float *>(c->x), rows, n_rows, c->desc.d, S.d_p,
+                                 reinterpret_cast<const float *>(c->out_norm), 0, c->desc.eps, c->dt, s, false);
+    if (rc) return rc;
+    ++*count;
+    Launcher L{c, s, count};
+    void *y = out_f32 ? reinterpret_cast<void *>(out_f32) : c->logits;
+    return L.linear(c->lm_head, S.d_p, S.vocab_p, S.hout, n_rows, y, S.vocab_p, out_f32 ? EPI_STORE_F32 : EPI_STORE);
+}
+
+// Algorithmic bytes of a round: the weights the round's forms of attention touch, the head, the cached latents read.
+double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_out) {
+    const Stack &S = *c->stack;
+    const double wb = 2.0, eb = (double)act_bytes(c);
+    double bytes = n_out ? (double)S.vocab_p * S.d_p * wb : 0.0;
+    for (const StackLayer &L : S.layers) {
+        const lcu_layer_desc &d = L.d;
+        bytes += wb * ((double)L.in_rows() * S.d_p + (double)d.heads * L.dim_p * L.qr_p + (double)L.kv_cols() * L.r_p + (double)S.d_p * L.hv_p +
+                       2.0 * L.ff_p * S.d_p);
+        for (int i = 0; i < n_req; ++i)
+            for (uint32_t j = 0; j < reqs[i].len; ++j) bytes += (double)(reqs[i].pos + j + 1) * L.r_p * eb;
+    }
+    return bytes;
+}
+
+}  // namespace lcu

@@ -1,0 +1,144 @@
+// Residual, norm and token-shift steps of layered models, and small row operations.
+#include "stack.cuh"
+
+namespace lcu {
+
+// One block per token.  A token's shifted input needs the PREVIOUS token's new residual: the block computes that row as
+// well (it may belong to another block of this launch, so it cannot be read), except at the start of a request, where it
+// comes from the sequence's state.  The state is double-buffered by generation: the block of a request's first token reads
+// one half, the block of its last token writes the other, so their order does not matter.  MAXV float4 values of each row
+// per thread stay in registers between the two passes.
+template <class T, int MAXV>
+__global__ void mix_input_kernel(const MixInputArgs a) {
+    grid_dep_launch();
+    const int t = blockIdx.x;
+    __shared__ float2 part[32];
+    const int r = a.tok_req[t];
+    const int first = a.req_first[r];
+    const bool shifted = a.shift != nullptr;
+    const bool at_start = t == first;
+    const bool prev_row = shifted && !at_start;
+    const int n4 = a.d_p / 4;
+    grid_dep_wait();
+    float4 x0[MAXV], x1[MAXV], y0[MAXV], y1[MAXV];
+    float s0 = 0.f, s1 = 0.f;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const size_t row0 = (size_t)t * a.d_p, row1 = prev_row ? row0 - a.d_p : row0;
+    const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0, e1 = a.embd && prev_row ? (size_t)a.tokens[t - 1] * a.d_p : e0;
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        x0[j] = x1[j] = y0[j] = y1[j] = zero;
+        if (i < n4) {
+            if (a.embd) {
+                x0[j] = ld4_bf16(a.embd, e0 + 4 * i);
+                if (prev_row) x1[j] = ld4_bf16(a.embd, e1 + 4 * i);
+            } else {
+                x0[j] = *reinterpret_cast<const float4 *>(a.x_in + row0 + 4 * i);
+                y0[j] = *reinterpret_cast<const float4 *>(a.y + row0 + 4 * i);
+                s0 += dot4(y0[j]);
+                if (prev_row) {
+                    x1[j] = *reinterpret_cast<const float4 *>(a.x_in + row1 + 4 * i);
+                    y1[j] = *reinterpret_cast<const float4 *>(a.y + row1 + 4 * i);
+                    s1 += dot4(y1[j]);
+                }
+            }
+        }
+    }
+    float r0 = 0.f, r1 = 0.f;
+    if (!a.embd) {
+        const float2 s = block_sum2(s0, s1, part);
+        r0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
+        r1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
+    }
+    const float *st_in = nullptr;
+    float *st_out = nullptr;
+    if (shifted) {
+        const int sg = a.req_slot[r];
+        const size_t off = (size_t)(sg >> 1) * a.d_p;
+        if (at_start && a.req_pos[r] > 0) st_in = a.state + (size_t)(sg & 1) * a.state_gen_stride + off;
+        if (t + 1 == a.req_first[r + 1]) st_out = a.state + (size_t)((sg & 1) ^ 1) * a.state_gen_stride + off;
+    }
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        float4 v = x0[j], p = x1[j];
+        if (!a.embd) {
+            const float4 g = a.gain_stride ? *reinterpret_cast<const float4 *>(a.gain + 4 * i)
+                                           : make_float4(a.gain[0], a.gain[0], a.gain[0], a.gain[0]);
+            v.x += y0[j].x * r0 * g.x; v.y += y0[j].y * r0 * g.y; v.z += y0[j].z * r0 * g.z; v.w += y0[j].w * r0 * g.w;
+            p.x += y1[j].x * r1 * g.x; p.y += y1[j].y * r1 * g.y; p.z += y1[j].z * r1 * g.z; p.w += y1[j].w * r1 * g.w;
+        }
+        if (a.x_out) *reinterpret_cast<float4 *>(a.x_out + row0 + 4 * i) = v;
+        if (st_out) *reinterpret_cast<float4 *>(st_out + 4 * i) = v;
+        if (!a.h) continue;
+        if (shifted) {
+            if (at_start) p = st_in ? *reinterpret_cast<const float4 *>(st_in + 4 * i) : zero;
+            const float4 m = ld4_bf16(a.shift, 4 * i);
+            v.x += (p.x - v.x) * m.x; v.y += (p.y - v.y) * m.y; v.z += (p.z - v.z) * m.z; v.w += (p.w - v.w) * m.w;
+        }
+        st4<T>(reinterpret_cast<T *>(a.h) + row0 + 4 * i, v);
+    }
+}
+
+template <class T>
+static int mix_input_t(const MixInputArgs &a, cudaStream_t s, bool pdl) {
+    const int n4 = a.d_p / 4;
+    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(mix_input_kernel<T, 1>, dim3(a.n_tok), dim3(128), 0, s, pdl, a));
+    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(mix_input_kernel<T, 2>, dim3(a.n_tok), dim3(512), 0, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(mix_input_kernel<T, 4>, dim3(a.n_tok), dim3(1024), 0, s, pdl, a));
+    return LCU_OK;
+}
+
+int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl) {
+    if (a.n_tok <= 0) return LCU_OK;
+    LCU_REQUIRE(a.d_p % 4 == 0 && a.d_p <= 16384, "mix_input: width %d (a multiple of 4, at most 16384)", a.d_p);
+    return dt == LCU_F32 ? mix_input_t<float>(a, s, pdl) : mix_input_t<__nv_bfloat16>(a, s, pdl);
+}
+
+template <class T>
+__global__ void __launch_bounds__(256) scalar_norm_rows_kernel(T *__restrict__ y, const float *__restrict__ x, const uint32_t *__restrict__ rows,
+                                                               int d, int d_p, const float *__restrict__ gain, int gain_stride, float eps) {
+    grid_dep_launch();
+    __shared__ float2 part[32];
+    grid_dep_wait();
+    const float *xr = x + (size_t)rows[blockIdx.x] * d_p;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < d_p / 4; i += blockDim.x) ss += dot4(reinterpret_cast<const float4 *>(xr)[i]);
+    const float r = 1.f / sqrtf(block_sum2(ss, 0.f, part).x / (float)d + eps);
+    for (int i = threadIdx.x; i < d_p / 4; i += blockDim.x) {
+        float4 v = reinterpret_cast<const float4 *>(xr)[i];
+        const float4 g = gain_stride ? reinterpret_cast<const float4 *>(gain)[i] : make_float4(gain[0], gain[0], gain[0], gain[0]);
+        v.x *= r * g.x; v.y *= r * g.y; v.z *= r * g.z; v.w *= r * g.w;
+        st4<T>(y + (size_t)blockIdx.x * d_p + 4 * i, v);
+    }
+}
+
+int op_scalar_norm_rows(void *y, const float *x, const uint32_t *rows, int n, int d, int d_p, const float *gain, int gain_stride, float eps,
+                        int dt, cudaStream_t s, bool pdl) {
+    if (n <= 0) return LCU_OK;
+    if (dt == LCU_F32)
+        LCU_CHECK_CUDA(launch_kernel(scalar_norm_rows_kernel<float>, dim3(n), dim3(256), 0, s, pdl, (float *)y, x, rows, d, d_p, gain, gain_stride, eps));
+    else
+        LCU_CHECK_CUDA(launch_kernel(scalar_norm_rows_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, s, pdl, (__nv_bfloat16 *)y, x, rows, d, d_p,
+                                     gain, gain_stride, eps));
+    return LCU_OK;
+}
+
+template <class T>
+__global__ void rows_to_f32_kernel(float *__restrict__ dst, const T *__restrict__ src, size_t n) {
+    size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) dst[i] = Act<T>::to_f(src[i]);
+}
+
+int op_rows_to_f32(float *dst, const void *src, size_t n, int dt, cudaStream_t s) {
+    if (!n) return LCU_OK;
+    const unsigned grid = (unsigned)((n + 255) / 256);
+    if (dt == LCU_F16) rows_to_f32_kernel<__half><<<grid, 256, 0, s>>>(dst, (const __half *)src, n);
+    else rows_to_f32_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(dst, (const __nv_bfloat16 *)src, n);
+    LCU_CHECK_CUDA(cudaGetLastError());
+    return LCU_OK;
+}
+
+}  // namespace lcu

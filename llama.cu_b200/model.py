@@ -190,7 +190,8 @@ def load_model(cfg, weights, device=0, kv_bytes=None, tp_rank=0, tp_size=1, comm
     creates the KV pool."""
     import torch
     dev = f"cuda:{device}"
-    ctx = Context(cfg.desc(page_tokens, max_tokens, max_seqs, nctx), device, tp_rank, tp_size, comm)
+    layers = cfg.layer_descs() if hasattr(cfg, "layer_descs") else None  # models described layer by layer (layered.py)
+    ctx = Context(cfg.desc(page_tokens, max_tokens, max_seqs, nctx), device, tp_rank, tp_size, comm, layers=layers)
     lib = load_library()
     items = weights.items() if isinstance(weights, dict) else weights
     for (layer, kind), w in items:
@@ -203,7 +204,7 @@ def load_model(cfg, weights, device=0, kv_bytes=None, tp_rank=0, tp_size=1, comm
         elif isinstance(w, np.ndarray):
             t = torch.from_numpy(w.view(np.int16)).to(dev)
         else:
-            t = w
+            t = w.to(dev)
         # linear weights are cut per rank; the LM head stays whole on the lead rank and is cut by vocabulary rows on
         # the others (used when arg-max rounds shard the head, see lcu_set_head_sharding)
         if tp_size > 1 and (kind in LINEAR_KINDS or (kind == W_LM_HEAD and tp_rank != 0)):
