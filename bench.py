@@ -35,6 +35,8 @@ WORKLOADS = {
     "llama8b-q8_0-b16": ("llama8b_q8", 16, (128, 128)),
     "llama70b-f16-b64": ("llama70b", 64, (1024, 1024)),
     "llama70b-tp8shard-f16-b64": ("llama70b_tp8shard", 64, (1024, 1024)),  # one rank's share, for profiling
+    "zefedra8b-bf16-b1": ("zefedra8b", 1, (128, 128)),
+    "zefedra8b-bf16-b32": ("zefedra8b", 32, (128, 1024)),
     "tiny-f16-b1": ("tiny", 1, (16, 16)),
 }
 DEFAULT_WORKLOAD = "llama8b-f16-b1"
@@ -471,6 +473,107 @@ def run_decode(L, env, cfg, batch, prompt_range, steps, warmup, want_e2e=True, w
     return res
 
 
+# --family-bench: sizes at which a layered family runs beside the LLaMA shape of equal width and feed-forward, cut to
+# `layers` layers and a vocabulary of 32000 (name, layered config, LLaMA config, layers)
+FAMILY_SIZES = [("8b", "zefedra8b", "llama8b", 8), ("1b", "zefedra1b", "llama1b", 8)]
+FAMILY_PREFILL = (2048, 8192)                            # prompt lengths
+FAMILY_DECODE = ((1, 1024), (32, 1024), (32, 4096), (4, 8192))  # (sequences, context)
+
+
+def kernel_table(events, steps):
+    """{kernel: [launches per step, us per launch]} of profiled CUDA events, template arguments cut off."""
+    import re
+    import torch
+    table = {}
+    for e in events:
+        if e.device_type != torch.autograd.DeviceType.CUDA:
+            continue
+        name = re.sub(r"<.*", "", e.name.replace("void ", "").replace("lcu::", ""))
+        row = table.setdefault(name, [0, 0.0])
+        row[0] += 1
+        row[1] += e.time_range.end - e.time_range.start
+    return {k: [round(n / steps, 2), round(t / n, 2)] for k, (n, t) in sorted(table.items(), key=lambda kv: -kv[1][1])}
+
+
+def family_bench(L, env, only=None, profile_kernels=False):
+    """Prefill and decode throughput of the layered family and of its LLaMA counterpart; one JSON line per measurement.
+    Prefill: one prompt in one round.  Decode: a captured round, device-side token feedback; weights exceed L2.
+    Device time between CUDA events, after warm-up."""
+    import numpy as np
+    import torch
+    from dataclasses import replace
+    from llama_cu_b200.model import reduced
+    from torch.profiler import ProfilerActivity, profile
+    dev = env.dev
+    for size, lname, gname, layers in FAMILY_SIZES:
+        if only and size not in only:
+            continue
+        for cname in (lname, gname):
+            cfg = replace(reduced(L.CONFIGS[cname], layers, 32000), act_dtype=L.BF16)
+            nctx = 8192 + 128
+            tokens = max(max(b * (c + 128) for b, c in FAMILY_DECODE), nctx)
+            ctx = L.load_model(cfg, L.iter_synth_weights_torch(cfg, 0, dev), device=env.local_rank,
+                               kv_bytes=tokens * cfg.kv_bytes_per_token() + (64 << 20), max_tokens=8192, max_seqs=64, nctx=nctx)
+            torch.cuda.empty_cache()
+            stream = torch.cuda.Stream(device=dev)
+            out = torch.zeros(64, 2, dtype=torch.int32, device=dev)
+            rng = np.random.default_rng(5)
+            line = {"bench": "family", "size": size, "model": cname, "layers": layers, "vocab": cfg.vocab, "dtype": "bf16", "data": "synthetic"}
+
+            def timed(fn, reps, warm):
+                for _ in range(warm):
+                    fn()
+                stream.synchronize()
+                a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                with ClockSampler(env.local_rank) as clocks:
+                    a.record(stream)
+                    for _ in range(reps):
+                        fn()
+                    b.record(stream)
+                    stream.synchronize()
+                table = None
+                if profile_kernels:
+                    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+                        for _ in range(2):
+                            fn()
+                        stream.synchronize()
+                    table = kernel_table(prof.events(), 2)
+                return a.elapsed_time(b) / reps, clocks.summary(), table
+
+            with torch.cuda.stream(stream):
+                for n in FAMILY_PREFILL:
+                    prompt = rng.integers(3, cfg.vocab, n).astype(np.uint32)
+                    seq = ctx.seq_create()
+                    ms, clocks, table = timed(lambda: ctx.step([(seq, 0, n)], prompt, out, stream=stream), 5, 3)
+                    ctx.seq_free(seq)
+                    print(json.dumps(dict(line, phase="prefill", tokens=n, ms=ms, tokens_s=n / ms * 1e3, clocks=clocks,
+                                          kernels=table)), flush=True)
+                for batch, c in FAMILY_DECODE:
+                    seqs = [ctx.seq_create() for _ in range(batch)]
+                    for s in seqs:
+                        for p in range(0, c, 1024):
+                            ctx.step([(s, p, min(1024, c - p))], rng.integers(3, cfg.vocab, min(1024, c - p)).astype(np.uint32), out, stream=stream)
+                    pos = [c]
+                    fm = np.array([[i, i] for i in range(batch)], dtype=np.uint32)
+                    ctx.step([(s, pos[0], 1) for s in seqs], np.full(batch, 7, np.uint32), out, stream=stream)
+                    pos[0] += 1
+
+                    def one():
+                        ctx.step([(s, pos[0], 1) for s in seqs], np.zeros(batch, np.uint32), out, fast_map=fm, stream=stream)
+                        pos[0] += 1
+                    ms, clocks, table = timed(one, 32, 8)
+                    gbs = ctx.last_step_bytes / ms / 1e6
+                    print(json.dumps(dict(line, phase="decode", batch=batch, context=c, ms=ms, tokens_s=batch / ms * 1e3,
+                                          launches=ctx.last_launch_count, step_gb=ctx.last_step_bytes / 1e9, gbs=gbs,
+                                          frac_of_measured=gbs / load_peaks()[0], clocks=clocks, kernels=table)), flush=True)
+                    for s in seqs:
+                        ctx.seq_free(s)
+            assert ctx.device_status() == 0
+            ctx.close()
+            del ctx
+            torch.cuda.empty_cache()
+
+
 def step_roofline(res):
     peak, _ = load_peaks()
     gbs = res["step_bytes"] / (res["ms_per_step"] * 1e-3) / 1e9
@@ -504,6 +607,9 @@ def main():
                     help="run only the small linear-layer case used for profiler captures")
     ap.add_argument("--probe-q8", action="store_true", help="with --probe-linear: Q8_0 weights")
     ap.add_argument("--probe-shape", default="gate_up", choices=["gate_up", "down", "qkv", "o"])
+    ap.add_argument("--family-bench", nargs="*", default=None, metavar="SIZE", choices=[s[0] for s in FAMILY_SIZES],
+                    help="prefill and decode throughput of the layered family beside the LLaMA shape of equal width, instead of the workload")
+    ap.add_argument("--family-kernels", action="store_true", help="with --family-bench: launches and time of every kernel (CUPTI)")
     args = ap.parse_args()
     if args.probe_linear > 0:
         probe_linear(args.probe_linear, q8=args.probe_q8, shape=args.probe_shape)
@@ -518,12 +624,16 @@ def main():
     for kv in args.tune:
         key, value = kv.split("=", 1)
         L.set_tuning(key, int(value))
+    if args.family_bench is not None:
+        family_bench(L, env, args.family_bench, args.family_kernels)
+        return 0
     cname, batch, prange = WORKLOADS[args.workload]
     cfg = L.CONFIGS[cname]
     if args.layers > 0:
         from llama_cu_b200.model import reduced
         cfg = reduced(cfg, min(args.layers, cfg.n_layers))
     dtype_name = {(0, 0): "f16", (1, 1): "bf16", (0, 3): "f16 activations, q8_0 weights"}[(cfg.act_dtype, cfg.wdt)]
+    layered = isinstance(cfg, L.LayeredConfig)  # no GEMV roofline record, CPU port or reference kernels of these
     config = {"workload": args.workload, "shape": cname, "batch": batch, "prompt_tokens": list(prange),
               "parallelism": f"tp{args.gpus}", "l2": "inputs larger than L2 (weights streamed once per step)"}
     if args.layers > 0:
@@ -531,6 +641,9 @@ def main():
     if args.tune:
         config["tuning"] = args.tune
 
+    if args.impl == "reference" and layered:
+        print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this family"}), flush=True)
+        return 0
     if args.impl == "reference":
         # the reference's own CPU implementation does not exist (it is CUDA-only and its Rust
         # host cannot be built here); this arm times the oracle port on the host cores
@@ -571,13 +684,14 @@ def main():
         parity = tp_parity(L, env)
 
     # ---- the headline workload
-    res = run_decode(L, env, cfg, batch, prange, args.steps, args.warmup, want_e2e=not args.no_e2e, timeline=args.timeline)
+    res = run_decode(L, env, cfg, batch, prange, args.steps, args.warmup, want_e2e=not args.no_e2e, timeline=args.timeline,
+                     want_roofline=not layered)
     config["tp_collectives"] = res["tp_collectives"]
     bad_status = any(res["device_status_all_ranks"])
 
     # ---- the reference's own kernels + cuBLAS on the same shapes (single GPU; oracle/_ref, built from the reference tree)
     ref_kernels = None
-    if rank == 0 and world == 1 and not args.no_ref_kernels and args.layers == 0:
+    if rank == 0 and world == 1 and not args.no_ref_kernels and args.layers == 0 and not layered:
         try:
             from oracle import ref_baseline
             ref_kernels = ref_baseline.bench_record(cfg, batch, prange, res["nctx"])
@@ -607,7 +721,7 @@ def main():
             bad_status = bad_status or any(r5["device_status_all_ranks"])
 
     cpu = None
-    if rank == 0 and world == 1 and not args.no_cpu_baseline:
+    if rank == 0 and world == 1 and not args.no_cpu_baseline and not layered:
         cpu = cpu_reference(cfg, 6, 2, budget_s=30.0)
 
     if rank == 0:

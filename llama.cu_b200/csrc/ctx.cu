@@ -587,6 +587,7 @@ int lcu_set_tuning(lcu_ctx *c, const char *key, long long value) {
     else if (k == "tc") t.tc = value != 0;
     else if (k == "tc_block") { LCU_REQUIRE(value == 64 || value == 128 || value == 256, "set_tuning: tc_block = %lld (64, 128, 256)", value); t.tc_block = (int)value; }
     else if (k == "tc_cluster") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: tc_cluster = %lld (0..2)", value); t.tc_cluster = (int)value; }
+    else if (k == "stack_pdl") t.stack_pdl = value != 0;
     else if (k == "expand_min") t.expand_min = (int)value;
     else if (k == "p2p_scatter_ranks") t.p2p_scatter_ranks = (int)value;
     else if (k == "p2p_scatter_min") t.p2p_scatter_min = (long)value;
@@ -682,7 +683,7 @@ int enqueue_round(lcu_ctx *c, const Round &r, lcu_kv_pair *out_dev, cudaStream_t
         if (!rc) rc = stack_head(c, r, out_idx, r.n_out, r.logits_f32, s, &launches);
         if (!rc && !r.logits_f32) {
             rc = sample_rows(out_dev, c->pre_pairs, c->logits, r.n_req, (size_t)d.vocab, r.any_sampling ? args : nullptr, randoms, dt, c->sample_ws,
-                             c->sample_ws_bytes, s, false, r.any_sampling, (size_t)c->stack->vocab_p);
+                             c->sample_ws_bytes, s, stack_pdl(c, r.n_tok), r.any_sampling, (size_t)c->stack->vocab_p);
             launches += r.any_sampling ? 3 : 2;
         }
         *count = launches;
@@ -742,8 +743,10 @@ int enqueue_round(lcu_ctx *c, const Round &r, lcu_kv_pair *out_dev, cudaStream_t
         }
         for (int t0 = 0; t0 < n;) {
             int nt;
-            // token blocks of up to 256 on the tcgen05 path (a weight tile is then streamed once per 256 tokens), 64 otherwise
-            const int blk = (tc_on && gemm_tc_supported(proto.in, proto.w_q8)) ? tuning().tc_block : 64;
+            // token blocks of 256 on the tcgen05 path (a weight tile is then streamed once per 256 tokens), all blocks in one
+            // launch unless the output goes to peers or the tuning value asks for smaller launches; 64 otherwise
+            const int tcb = tuning().tc_block < 256 || push ? tuning().tc_block : GEMM_TC_MAX_TOKENS;
+            const int blk = (tc_on && gemm_tc_supported(proto.in, proto.w_q8)) ? tcb : 64;
             if (batched) nt = n - t0 < blk ? n - t0 : blk;
             else {
                 nt = gemv_max_tokens(proto.in);

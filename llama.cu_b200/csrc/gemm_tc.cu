@@ -518,6 +518,7 @@ __device__ __forceinline__ float4 tc_ld_dsmem4(uint32_t local_saddr, uint32_t ct
 // Token blocks of 128 and 256 (prefill): the MMA takes all N tokens at once (tcgen05 allows N up to 256 columns of
 // TMEM per accumulator), so a weight tile is streamed once per 256 tokens instead of once per 64; the epilogue then
 // walks the accumulator in passes of NS = 64 tokens through the same staging tile and the same two cluster barriers.
+// Rounds of more than 256 tokens put their 256-token blocks on grid.y of ONE launch.
 template <class T>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
@@ -535,6 +536,7 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
     const bool swiglu = a.epilogue == EPI_SWIGLU;
     const int ks = (int)tc_cluster_rank();
     const int rb = (int)blockIdx.x / KS;
+    const int tb = (int)blockIdx.y * N;  // first token of this CTA's block
     const int kb0 = (int)((long)ks * nkb / KS), kb1 = (int)((long)(ks + 1) * nkb / KS);
     const int n_units = kb1 - kb0;
     const int tm_cols = N < 32 ? 32 : N;
@@ -570,7 +572,7 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
                 tc_tma_2d(dst, &map_w, kx, swiglu ? rb * 64 : rb * TC_BM, bar);
                 tc_tma_2d(dst + TC_A_BYTES / 2, &map_w, kx, swiglu ? a.di + rb * 64 : rb * TC_BM + 64, bar);
             }
-            if (acts) tc_tma_2d(dst + TC_A_BYTES, &map_x, kx, 0, bar);
+            if (acts) tc_tma_2d(dst + TC_A_BYTES, &map_x, kx, tb, bar);
         };
         const int first = n_units < n_stages ? n_units : n_stages;
         for (int j = 0; j < first; ++j) issue(j, true, false);
@@ -633,7 +635,7 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
         __syncthreads();
         tc_cluster_sync();  // every CTA of the row block has staged its partial tile
 
-        if (warp >= 2 && t0 < a.n_tok) {
+        if (warp >= 2 && tb + t0 < a.n_tok) {
             // ---------------- this CTA's share of the items: chunk c of 8 rows (8 pairs for SwiGLU) with c % KS == ks
             const int et = tid - 64;
             const int chunks = swiglu ? 8 : 16;
@@ -641,13 +643,13 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
             TcPre pre[8];
             int cnt = 0;
             for (int idx = et; idx < mine * NS; idx += 128, ++cnt) {
-                const int c = ks + (idx % mine) * KS, n = t0 + idx / mine;
+                const int c = ks + (idx % mine) * KS, n = tb + t0 + idx / mine;
                 const int first = swiglu ? rb * 64 + 8 * c : rb * TC_BM + 8 * c;
                 if (n < a.n_tok && first + 8 <= (swiglu ? a.di : a.out)) tc_prefetch<T>(a, n, first, pre[cnt]);
             }
             cnt = 0;
             for (int idx = et; idx < mine * NS; idx += 128, ++cnt) {
-                const int c = ks + (idx % mine) * KS, nl = idx / mine, n = t0 + nl;
+                const int c = ks + (idx % mine) * KS, nl = idx / mine, n = tb + t0 + nl;
                 const int first = swiglu ? rb * 64 + 8 * c : rb * TC_BM + 8 * c;
                 if (!(n < a.n_tok && first + 8 <= (swiglu ? a.di : a.out))) continue;
                 float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
@@ -794,7 +796,8 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
         // blocks the balanced stream-K split wins: 4.75 against 4.95 ms), 2: wherever it applies, 0: never
         const int cluster_mode = tuning().tc_cluster;
         const int n_rb_c = (n_pairs + 63) / 64, nkb_c = a.in / TC_BK;
-        int KS = sms / n_rb_c;
+        const int n_tb = (a.n_tok + N - 1) / N;  // token blocks: more than one only for rounds of more than 256 tokens
+        int KS = sms / (n_rb_c * n_tb);
         if (KS > 8) KS = 8;
         if (KS < 1) KS = 1;
         while (KS > 1 && nkb_c / KS < 4) --KS;
@@ -811,7 +814,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
             if (st > TC_MAX_STAGES) st = TC_MAX_STAGES;
             const uint32_t idesc_c = (1u << 4) | (fmt << 7) | (fmt << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(TC_BM >> 4) << 24);
             cudaLaunchConfig_t cfg = {};
-            cfg.gridDim = dim3(n_rb_c * KS);
+            cfg.gridDim = dim3(n_rb_c * KS, n_tb);
             cfg.blockDim = dim3(TC_THREADS);
             cfg.dynamicSmemBytes = fixed + (size_t)st * stage_bytes;
             cfg.stream = s;
@@ -825,7 +828,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
             cfg.attrs = attr;
             cfg.numAttrs = pdl ? 2 : 1;
             LCU_CHECK_CUDA(cudaLaunchKernelEx(&cfg, gemm_tck_kernel<T>, a, mw, mx, N, st, KS, idesc_c, status));
-            g_linear_last_ctas = n_rb_c * KS;
+            g_linear_last_ctas = n_rb_c * KS * n_tb;
             return LCU_OK;
         }
     }
@@ -868,7 +871,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
 }
 
 int gemm_tc_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry) {
-    LCU_REQUIRE(a.n_tok >= 1 && a.n_tok <= 256, "gemm_tc: n_tok = %d (1..256)", a.n_tok);
+    LCU_REQUIRE(a.n_tok >= 1 && a.n_tok <= GEMM_TC_MAX_TOKENS, "gemm_tc: n_tok = %d (1..%d)", a.n_tok, GEMM_TC_MAX_TOKENS);
     LCU_REQUIRE(dry || gemm_tc_supported(a.in, a.w_q8), "gemm_tc: in = %d unsupported", a.in);
     LCU_REQUIRE(a.out > 0 && a.out % 2 == 0, "gemm_tc: out = %d must be even", a.out);
     LCU_REQUIRE(a.prologue == PRO_NONE && !a.x_rows, "gemm_tc: takes prepared activations only");

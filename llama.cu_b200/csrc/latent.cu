@@ -74,85 +74,85 @@ int latent_norm_launch(const LatentNormArgs &a, int dt, cudaStream_t s, bool pdl
 }
 
 // ------------------------------------------------------------------ per-head linear layers
-// Weight rows on M (16 per warp), tokens on N.  The whole K range of both operands is requested up front in chunks of 128
-// columns and multiplied chunk by chunk as they land.  Without `x` the activations are the merged attention partials:
-// sum over splits of exp(m_s - M) o_s, divided by the merged sum.
+// Weight rows on M (16 per warp), tokens on N.  The whole K range of both operands is requested up front, the weights ahead of the
+// dependency wait.  Without `x` the activations are the merged attention partials:
+// sum over splits of 2^(m_s - M) o_s (running maxima are kept in powers of two), divided by the merged sum.
 constexpr int HL_THREADS = 128;
 constexpr int HL_MAX_SPLITS = 64;
 
 template <int NT>
 __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinearArgs a) {
-    constexpr int NF = NT / 8;
+    constexpr int NF = NT / 8, YLD = 64 + 8;
     extern __shared__ __align__(16) unsigned char smem[];
     const int ld = a.in + 8;
     bf16 *Ws = reinterpret_cast<bf16 *>(smem);   // [64][in + 8]
     bf16 *Xs = Ws + (size_t)64 * ld;             // [NT][in + 8]
+    __shared__ __align__(16) bf16 Ys[NT * YLD];  // output tile, token-major
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, t4 = lane & 3;
     const int o0 = blockIdx.x * 64, h = blockIdx.y, n0 = blockIdx.z * NT;
-    const bf16 *w = reinterpret_cast<const bf16 *>(a.w) + (size_t)h * a.out * a.in;
+    const int nt = min(NT, a.n - n0), no = min(64, a.out - o0);
+    const bf16 *w = reinterpret_cast<const bf16 *>(a.w) + ((size_t)h * a.out + o0) * a.in;
     grid_dep_launch();
-    const int nchunk = (a.in + 127) / 128;
-    for (int c = 0; c < nchunk; ++c) {  // weights do not depend on the previous kernel
-        const int cols = min(128, a.in - c * 128) / 8;
-        for (int i = tid; i < 64 * cols; i += HL_THREADS) {
-            const int r = i / cols, k = c * 128 + (i - r * cols) * 8;
-            la_cp_async_16(Ws + r * ld + k, w + (size_t)(o0 + r < a.out ? o0 + r : 0) * a.in + k, o0 + r < a.out);
-        }
-        la_commit();
-    }
+    const int ch = a.in / 8;
+    // rows are dealt to lane groups of the chunk count's next power of two, so no lane computes a division per chunk
+    const int lpr = ch >= 32 ? 32 : (ch > 16 ? 32 : (ch > 8 ? 16 : (ch > 4 ? 8 : (ch > 2 ? 4 : 2)))), rpw = 32 / lpr;
+    const int lr = warp * rpw + lane / lpr, lc = lane % lpr, rstep = 4 * rpw;
+    for (int r = lr; r < 64; r += rstep)  // weights do not depend on the previous kernel
+        for (int c = lc; c < ch; c += lpr) la_cp_async_16(Ws + (size_t)r * ld + c * 8, w + (r < no ? (size_t)r * a.in + c * 8 : 0), r < no);
+    la_commit();
     grid_dep_wait();
     if (a.x) {
         const bf16 *x = reinterpret_cast<const bf16 *>(a.x) + (size_t)h * a.head_x;
-        const int cols = a.in / 8;
-        for (int i = tid; i < NT * cols; i += HL_THREADS) {
-            const int r = i / cols, k = (i - r * cols) * 8;
-            const bool ok = n0 + r < a.n;
-            const size_t row = ok ? (size_t)(a.x_rows ? a.x_rows[n0 + r] : n0 + r) : 0;
-            la_cp_async_16(Xs + r * ld + k, x + row * a.stride_x + k, ok);
+        for (int r = lr; r < NT; r += rstep) {
+            const size_t row = r < nt ? (size_t)(a.x_rows ? a.x_rows[n0 + r] : n0 + r) * a.stride_x : 0;
+            for (int c = lc; c < ch; c += lpr) la_cp_async_16(Xs + (size_t)r * ld + c * 8, x + row + (r < nt ? c * 8 : 0), r < nt);
         }
         la_commit();
-        la_wait<0>();
-        __syncthreads();
     } else {
-        __shared__ float wt[NT][HL_MAX_SPLITS];
+        // a warp per row: lane s holds split s's weight 2^(m_s - M) / sum (two splits per lane)
         for (int r = warp; r < NT; r += HL_THREADS / 32) {
-            if (n0 + r >= a.n) continue;
             const size_t row = (size_t)(n0 + r) * a.heads + h;
-            const int ns = a.part_n[row];
-            const float2 *ml = reinterpret_cast<const float2 *>(a.part_ml) + row * a.splits;
-            const float2 e0 = lane < ns ? ml[lane] : make_float2(-INFINITY, 0.f);
-            const float2 e1 = lane + 32 < ns ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
-            const float M = warp_max(fmaxf(e0.x, e1.x));
-            const float w0 = e0.x == -INFINITY ? 0.f : expf(e0.x - M), w1 = e1.x == -INFINITY ? 0.f : expf(e1.x - M);
-            const float inv = 1.f / warp_sum(w0 * e0.y + w1 * e1.y);
-            wt[r][lane] = w0 * inv;
-            wt[r][lane + 32] = w1 * inv;
-        }
-        __syncthreads();
-        const int cols = a.in / 4;
-        for (int i = tid; i < NT * cols; i += HL_THREADS) {
-            const int r = i / cols, k = (i - r * cols) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (n0 + r < a.n) {
-                const size_t row = (size_t)(n0 + r) * a.heads + h;
-                const int ns = a.part_n[row];
-                const float *src = a.part_o + row * a.splits * a.in + k;
-#pragma unroll 4
-                for (int s2 = 0; s2 < ns; ++s2) {
-                    const float4 o = *reinterpret_cast<const float4 *>(src + (size_t)s2 * a.in);
-                    const float f = wt[r][s2];
-                    v.x = fmaf(f, o.x, v.x); v.y = fmaf(f, o.y, v.y); v.z = fmaf(f, o.z, v.z); v.w = fmaf(f, o.w, v.w);
-                }
+            const int ns = r < nt ? a.part_n[row] : 0;
+            float w0 = 0.f, w1 = 0.f;
+            if (ns) {
+                const float2 *ml = reinterpret_cast<const float2 *>(a.part_ml) + row * a.splits;
+                const float2 e0 = lane < ns ? ml[lane] : make_float2(-INFINITY, 0.f);
+                const float2 e1 = lane + 32 < ns ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
+                const float M = warp_max(fmaxf(e0.x, e1.x));
+                w0 = e0.x == -INFINITY ? 0.f : exp2f(e0.x - M);
+                w1 = e1.x == -INFINITY ? 0.f : exp2f(e1.x - M);
+                const float inv = 1.f / warp_sum(w0 * e0.y + w1 * e1.y);
+                w0 *= inv;
+                w1 *= inv;
             }
-            st4<bf16>(Xs + r * ld + k, v);
+            const int c = lane * 4;  // up to four 4-column pieces of the row per lane (a row holds at most 512)
+            float4 v[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float *src = a.part_o + row * a.splits * a.in + c;
+#pragma unroll 2
+            for (int s2 = 0; s2 < ns; ++s2, src += a.in) {
+                const float f = __shfl_sync(0xffffffffu, s2 < 32 ? w0 : w1, s2 & 31);
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (c + 128 * k < a.in) {
+                        const float4 o = *reinterpret_cast<const float4 *>(src + 128 * k);
+                        v[k].x = fmaf(f, o.x, v[k].x); v[k].y = fmaf(f, o.y, v[k].y);
+                        v[k].z = fmaf(f, o.z, v[k].z); v[k].w = fmaf(f, o.w, v[k].w);
+                    }
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (c + 128 * k < a.in) st4<bf16>(Xs + (size_t)r * ld + c + 128 * k, v[k]);
         }
-        la_wait<0>();
-        __syncthreads();
     }
+    la_wait<0>();
+    __syncthreads();
     float acc[NF][4];
 #pragma unroll
     for (int i = 0; i < NF; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     const bf16 *wrow = Ws + (size_t)(warp * 16 + (lane & 15)) * ld + (lane >> 4) * 8;
+#pragma unroll 4
     for (int k = 0; k < a.in; k += 16) {
         uint32_t af[4];
         la_ldsm4(af, wrow + k);
@@ -170,19 +170,27 @@ __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinea
             }
         }
     }
-    bf16 *y = reinterpret_cast<bf16 *>(a.y) + (size_t)h * a.head_y;
 #pragma unroll
     for (int f = 0; f < NF; ++f)
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
-            const int n = n0 + f * 8 + 2 * t4 + c;
-            if (n >= a.n) continue;
-            const size_t row = (size_t)(a.y_rows ? a.y_rows[n] : n);
-            const float g = a.gate ? 1.f / (1.f + expf(-a.gate[row * a.stride_gate + h])) : 1.f;
-            const int oa = o0 + warp * 16 + gid, ob = oa + 8;
-            if (oa < a.out) y[row * a.stride_y + oa] = __float2bfloat16_rn(acc[f][c] * g);
-            if (ob < a.out) y[row * a.stride_y + ob] = __float2bfloat16_rn(acc[f][c + 2] * g);
+            bf16 *d = Ys + (f * 8 + 2 * t4 + c) * YLD + warp * 16 + gid;
+            float g = 1.f;
+            if (a.gate && f * 8 + 2 * t4 + c < nt) {
+                const int n = n0 + f * 8 + 2 * t4 + c;
+                g = 1.f / (1.f + expf(-a.gate[(size_t)(a.y_rows ? a.y_rows[n] : n) * a.stride_gate + h]));
+            }
+            d[0] = __float2bfloat16_rn(acc[f][c] * g);
+            d[8] = __float2bfloat16_rn(acc[f][c + 2] * g);
         }
+    __syncthreads();
+    bf16 *y = reinterpret_cast<bf16 *>(a.y) + (size_t)h * a.head_y + o0;
+    for (int i = tid; i < nt * 8; i += HL_THREADS) {
+        const int r = i >> 3, c = (i & 7) * 8;
+        if (c < no)
+            *reinterpret_cast<uint4 *>(y + (size_t)(a.y_rows ? a.y_rows[n0 + r] : n0 + r) * a.stride_y + c) =
+                *reinterpret_cast<const uint4 *>(Ys + r * YLD + c);
+    }
 }
 
 // Shared-memory attribute of a kernel (set when a context is created: nothing but launches may happen inside a capture).
@@ -207,16 +215,26 @@ int head_linear_launch(const HeadLinearArgs &a, cudaStream_t s, bool pdl, bool d
     LCU_REQUIRE(a.x || a.splits <= HL_MAX_SPLITS, "head_linear: %d splits", a.splits);
     if (dry) {
         int rc = head_linear_t<8>(a, s, pdl, true);
+        if (!rc) rc = head_linear_t<16>(a, s, pdl, true);
+        if (!rc) rc = head_linear_t<32>(a, s, pdl, true);
         return rc ? rc : head_linear_t<64>(a, s, pdl, true);
     }
     if (a.n <= 0) return LCU_OK;
-    return a.n <= 8 ? head_linear_t<8>(a, s, pdl, false) : head_linear_t<64>(a, s, pdl, false);
+    LCU_REQUIRE(a.out % 8 == 0 && a.stride_y % 8 == 0 && a.head_y % 8 == 0, "head_linear: outputs must be multiples of 8");
+    // the widest token tile that still gives every SM a CTA (weights are read once per token tile)
+    const long tiles = (long)((a.out + 63) / 64) * a.heads;
+    int nt = 64;
+    while (nt > 8 && (nt >= 2 * a.n || tiles * ((a.n + nt - 1) / nt) < sm_count())) nt /= 2;
+    if (nt == 8) return head_linear_t<8>(a, s, pdl, false);
+    if (nt == 16) return head_linear_t<16>(a, s, pdl, false);
+    return nt == 32 ? head_linear_t<32>(a, s, pdl, false) : head_linear_t<64>(a, s, pdl, false);
 }
 
 // ------------------------------------------------------------------ absorbed attention
 constexpr int LA_THREADS = 256;
 constexpr int LA_TILE = 64;
 constexpr int LA_ROWS_F32 = 8;
+constexpr int LD_WARPS = 8, LD_THREADS = 32 * LD_WARPS, LD_SLICES = LD_WARPS / 2;
 
 // Row block b of this launch: its request, first row (token, head pairs of absorbed tokens, token-major), row count.
 // Called by every thread; the search runs in warp 0.
@@ -265,12 +283,12 @@ __device__ __forceinline__ LaBlock la_find_block(const LatentAttnArgs &a, int b,
     return r;
 }
 
-// One CTA: up to 16 MT rows of one request against the tiles of one split.  Both products run on tensor cores over the SAME
+// Portion form: up to 64 rows of one request against the tiles of one split.  Both products run on tensor cores over the SAME
 // shared-memory tile of latents (keys as stored, values through a transposing ldmatrix); tiles are double-buffered.
-//   scores  [16 MT rows x 64 positions]: warps tile rows x positions;   output [16 MT rows x R]: a warp owns R / 8 columns
-template <int MT, int RB>
+//   scores  [64 rows x 64 positions]: warps tile rows x positions;   output [64 rows x R]: a warp owns R / 8 columns
+template <int RB>
 __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const LatentAttnArgs a) {
-    constexpr int ROWS = 16 * MT;
+    constexpr int MT = 4, ROWS = 16 * MT;
     constexpr int NTW = RB / 64;          // most 8-column output tiles per warp
     constexpr int PG = 8 / MT;            // position groups of the score product
     constexpr int SN = LA_TILE / PG / 8;  // 8-position score tiles per warp
@@ -339,6 +357,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
 #pragma unroll
         for (int i = 0; i < NTW; ++i) acc[m][i][0] = acc[m][i][1] = acc[m][i][2] = acc[m][i][3] = 0.f;
     const int ntw = R / 64;
+    const float scale2 = a.scale * 1.4426950408889634f;  // scores in powers of two
     const int wm = warp % MT, wp = warp / MT;  // score product: row tile, position group
 
     for (int tile = tile0; tile < tile1; ++tile) {
@@ -353,28 +372,17 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
 #pragma unroll
             for (int i = 0; i < SN; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
             const bf16 *qrow = Qs + (size_t)(wm * 16 + (lane & 15)) * ld + (lane >> 4) * 8;
-            if constexpr (SN == 1) {
-                const bf16 *crow = C + (size_t)(wp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;
+            const bf16 *crow = C + (size_t)(wp * SN * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * ld + ((lane >> 3) & 1) * 8;
 #pragma unroll 4
-                for (int k = 0; k < R; k += 16) {
-                    uint32_t af[4], b[2];
-                    la_ldsm4(af, qrow + k);
-                    la_ldsm2(b, crow + k);
-                    mma16816<bf16>(sc[0], af[0], af[1], af[2], af[3], b[0], b[1]);
-                }
-            } else {
-                const bf16 *crow = C + (size_t)(wp * SN * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * ld + ((lane >> 3) & 1) * 8;
-#pragma unroll 4
-                for (int k = 0; k < R; k += 16) {
-                    uint32_t af[4];
-                    la_ldsm4(af, qrow + k);
+            for (int k = 0; k < R; k += 16) {
+                uint32_t af[4];
+                la_ldsm4(af, qrow + k);
 #pragma unroll
-                    for (int np = 0; np < SN / 2; ++np) {
-                        uint32_t b[4];
-                        la_ldsm4(b, crow + (size_t)np * 16 * ld + k);
-                        mma16816<bf16>(sc[2 * np], af[0], af[1], af[2], af[3], b[0], b[1]);
-                        mma16816<bf16>(sc[2 * np + 1], af[0], af[1], af[2], af[3], b[2], b[3]);
-                    }
+                for (int np = 0; np < SN / 2; ++np) {
+                    uint32_t b[4];
+                    la_ldsm4(b, crow + (size_t)np * 16 * ld + k);
+                    mma16816<bf16>(sc[2 * np], af[0], af[1], af[2], af[3], b[0], b[1]);
+                    mma16816<bf16>(sc[2 * np + 1], af[0], af[1], af[2], af[3], b[2], b[3]);
                 }
             }
 #pragma unroll
@@ -391,16 +399,16 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
             const int r = warp + 8 * i;
             const int lim = r < blk.rows ? pos0 + (blk.row0 + r) / a.heads : -1;
             const int p0 = tile * LA_TILE + lane, p1 = p0 + 32;
-            const float s0 = p0 <= lim ? S[r * SROW + lane] * a.scale : -INFINITY;
-            const float s1 = p1 <= lim ? S[r * SROW + lane + 32] * a.scale : -INFINITY;
+            const float s0 = p0 <= lim ? S[r * SROW + lane] * scale2 : -INFINITY;
+            const float s1 = p1 <= lim ? S[r * SROW + lane + 32] * scale2 : -INFINITY;
             const float mo = m_run[r], mn = fmaxf(mo, warp_max(fmaxf(s0, s1)));
-            const bf16 pa = __float2bfloat16_rn(s0 == -INFINITY ? 0.f : expf(s0 - mn));
-            const bf16 pb = __float2bfloat16_rn(s1 == -INFINITY ? 0.f : expf(s1 - mn));
+            const bf16 pa = __float2bfloat16_rn(s0 == -INFINITY ? 0.f : exp2f(s0 - mn));
+            const bf16 pb = __float2bfloat16_rn(s1 == -INFINITY ? 0.f : exp2f(s1 - mn));
             const float sum = warp_sum(__bfloat162float(pa) + __bfloat162float(pb));
             Ps[r * PROW + lane] = pa;
             Ps[r * PROW + lane + 32] = pb;
             if (lane == 0) {
-                const float c = mo == -INFINITY ? 0.f : expf(mo - mn);
+                const float c = mo == -INFINITY ? 0.f : exp2f(mo - mn);
                 corr[r] = c;
                 l_run[r] = l_run[r] * c + sum;
                 m_run[r] = mn;
@@ -446,6 +454,234 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
             const int r = m * 16 + gid + 8 * hf;
             if (r >= blk.rows) continue;
             float *o = a.part_o + ((size_t)(blk.row0 + r) * a.splits + sp) * R + warp * (R / 8) + 2 * t4;
+#pragma unroll
+            for (int i = 0; i < NTW; ++i)
+                if (i < ntw) *reinterpret_cast<float2 *>(o + i * 8) = make_float2(acc[m][i][2 * hf], acc[m][i][2 * hf + 1]);
+        }
+    if (tid < blk.rows) {
+        const size_t row = blk.row0 + tid;
+        reinterpret_cast<float2 *>(a.part_ml)[row * a.splits + sp] = make_float2(m_run[tid], l_run[tid]);
+        if (sp == 0) a.part_n[row] = my_splits;
+    }
+}
+
+// Decode form (up to 32 rows per CTA).  The latent dimension is cut into slices, one per pair of warps; a warp keeps
+// its slice of the query fragments in registers for the whole kernel and computes partial scores of 32 positions, which the
+// softmax sums over the slices: every byte of a tile crosses the shared-memory port once per product.  Slices and output
+// columns are dealt in whole MMA steps, so any latent size that is a multiple of 16 works.  The gather of tile
+// t + 1 is in flight during all of tile t.
+template <int MT, int RB>
+__global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const LatentAttnArgs a) {
+    constexpr int ROWS = 16 * MT, RPW = ROWS / LD_WARPS;  // rows of the CTA, softmax rows per warp
+    constexpr int NTW = RB > 8 * LD_WARPS ? RB / (8 * LD_WARPS) : 1;  // most 8-column output tiles per warp == most k-steps of a slice
+    constexpr int PROW = LA_TILE + 8, SROW = LA_TILE + 4;
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int R = a.r_p, ld = R + 8;
+    bf16 *Cs = reinterpret_cast<bf16 *>(smem);                  // [2][TILE][ld]
+    bf16 *Ps = Cs + (size_t)2 * LA_TILE * ld;                   // [ROWS][PROW]
+    float *S = reinterpret_cast<float *>(Ps + ROWS * PROW);     // [slices][ROWS][SROW]
+    float *corr = S + LD_SLICES * ROWS * SROW, *m_run = corr + ROWS, *l_run = m_run + ROWS;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, t4 = lane & 3;
+    const int sp = blockIdx.y;
+    grid_dep_launch();
+
+    const LaBlock blk = la_find_block(a, blockIdx.x, ROWS);
+    if (blk.req < 0) return;
+    const int rr = a.req_id[blk.req];
+    const int pos0 = a.req_pos[rr] - blk.tok0;
+    const int ctx = pos0 + (blk.row0 + blk.rows - 1) / a.heads + 1;
+    const int n_tiles = (ctx + LA_TILE - 1) / LA_TILE;
+    const int tps = (n_tiles + a.splits - 1) / a.splits;
+    const int my_splits = (n_tiles + tps - 1) / tps;
+    if (sp >= my_splits) return;
+    const int tile0 = sp * tps, tile1 = min(n_tiles, tile0 + tps);
+    const int32_t *pages = a.page_table + (size_t)rr * a.pt_stride;
+    const bf16 *pool = reinterpret_cast<const bf16 *>(a.pool) + a.c_off;
+    const int pmask = (1 << a.page_shift) - 1;
+    const int CH = R / 8, dj = LD_THREADS / CH, dc = LD_THREADS - dj * CH, lj = tid / CH, lc = tid - lj * CH;
+    const bool whole_page = a.page_shift >= 6 && dc == 0;  // a tile lies in one page and a thread keeps its column
+    auto load_tile = [&](int tile, int buf) {
+        bf16 *dst = Cs + (size_t)buf * LA_TILE * ld;
+        const int p0 = tile * LA_TILE;
+        if (whole_page) {
+            const bf16 *src = pool + (size_t)pages[p0 >> a.page_shift] * a.page_elems + (size_t)(p0 & pmask) * R + lc * 8;
+            bf16 *d = dst + lc * 8;
+            const int last = ctx - p0;
+#pragma unroll 4
+            for (int j = lj; j < LA_TILE; j += dj) la_cp_async_16(d + (size_t)j * ld, src + (j < last ? (size_t)j * R : 0), j < last);
+            return;
+        }
+        int j = lj, c = lc;
+        while (j < LA_TILE) {
+            const int pos = p0 + j;
+            const bool ok = pos < ctx;
+            const size_t off = ok ? (size_t)pages[pos >> a.page_shift] * a.page_elems + (size_t)(pos & pmask) * R + c * 8 : 0;
+            la_cp_async_16(dst + (size_t)j * ld + c * 8, pool + off, ok);
+            j += dj;
+            c += dc;
+            if (c >= CH) { c -= CH; ++j; }
+        }
+    };
+    for (int i = tid; i < ROWS; i += LD_THREADS) {
+        m_run[i] = -INFINITY;
+        l_run[i] = 0.f;
+    }
+    const int ksl = warp >> 1, ph = warp & 1;  // latent slice, half of the tile's positions
+    const int k_first = ksl * (R / 16) / LD_SLICES, nk = (ksl + 1) * (R / 16) / LD_SLICES - k_first;      // 16-wide steps of the slice
+    const int c_first = warp * (R / 8) / LD_WARPS, ntw = (warp + 1) * (R / 8) / LD_WARPS - c_first;       // 8-wide output tiles
+    const float scale2 = a.scale * 1.4426950408889634f;  // scores in powers of two
+    grid_dep_wait();
+    load_tile(tile0, 0);
+    la_commit();
+    uint32_t qf[MT][NTW][4];
+    {
+        const bf16 *q = reinterpret_cast<const bf16 *>(a.q) + (size_t)blk.row0 * R + k_first * 16 + 2 * t4;
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const int ra = m * 16 + gid, rb = ra + 8;
+#pragma unroll
+            for (int k = 0; k < NTW; ++k) {
+                const bool in = k < nk;
+                qf[m][k][0] = in && ra < blk.rows ? *reinterpret_cast<const uint32_t *>(q + (size_t)ra * R + k * 16) : 0u;
+                qf[m][k][1] = in && rb < blk.rows ? *reinterpret_cast<const uint32_t *>(q + (size_t)rb * R + k * 16) : 0u;
+                qf[m][k][2] = in && ra < blk.rows ? *reinterpret_cast<const uint32_t *>(q + (size_t)ra * R + k * 16 + 8) : 0u;
+                qf[m][k][3] = in && rb < blk.rows ? *reinterpret_cast<const uint32_t *>(q + (size_t)rb * R + k * 16 + 8) : 0u;
+            }
+        }
+    }
+    float acc[MT][NTW][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < NTW; ++i) acc[m][i][0] = acc[m][i][1] = acc[m][i][2] = acc[m][i][3] = 0.f;
+    int lim[RPW];  // last visible position of the rows whose softmax this warp computes
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) lim[i] = warp + LD_WARPS * i < blk.rows ? pos0 + (blk.row0 + warp + LD_WARPS * i) / a.heads : -1;
+
+    for (int tile = tile0; tile < tile1; ++tile) {
+        const int buf = (tile - tile0) & 1;
+        la_wait<0>();
+        __syncthreads();  // the tile has landed for everyone, and everyone is done with the other buffer
+        if (tile + 1 < tile1) load_tile(tile + 1, buf ^ 1);
+        la_commit();
+        const bf16 *C = Cs + (size_t)buf * LA_TILE * ld;
+        {
+            float sc[MT][4][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[m][i][0] = sc[m][i][1] = sc[m][i][2] = sc[m][i][3] = 0.f;
+            const bf16 *crow = C + (size_t)(ph * 32 + (lane & 7) + ((lane >> 4) & 1) * 8) * ld + k_first * 16 + ((lane >> 3) & 1) * 8;
+#pragma unroll
+            for (int k = 0; k < NTW; ++k) {
+                if (k < nk) {
+#pragma unroll
+                    for (int np = 0; np < 2; ++np) {
+                        uint32_t b[4];
+                        la_ldsm4(b, crow + (size_t)np * 16 * ld + k * 16);
+#pragma unroll
+                        for (int m = 0; m < MT; ++m) {
+                            mma16816<bf16>(sc[m][2 * np], qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3], b[0], b[1]);
+                            mma16816<bf16>(sc[m][2 * np + 1], qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3], b[2], b[3]);
+                        }
+                    }
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    float *d = S + ((size_t)ksl * ROWS + m * 16 + gid) * SROW + ph * 32 + i * 8 + 2 * t4;
+                    *reinterpret_cast<float2 *>(d) = make_float2(sc[m][i][0], sc[m][i][1]);
+                    *reinterpret_cast<float2 *>(d + 8 * SROW) = make_float2(sc[m][i][2], sc[m][i][3]);
+                }
+        }
+        __syncthreads();
+        {
+            float s0[RPW], s1[RPW], mx[RPW], sum[RPW];
+            const int p0 = tile * LA_TILE + lane, p1 = p0 + 32;
+#pragma unroll
+            for (int i = 0; i < RPW; ++i) {
+                const float *sr = S + (warp + LD_WARPS * i) * SROW + lane;
+                s0[i] = s1[i] = 0.f;
+#pragma unroll
+                for (int k = 0; k < LD_SLICES; ++k) {
+                    s0[i] += sr[k * ROWS * SROW];
+                    s1[i] += sr[k * ROWS * SROW + 32];
+                }
+                s0[i] = p0 <= lim[i] ? s0[i] * scale2 : -INFINITY;
+                s1[i] = p1 <= lim[i] ? s1[i] * scale2 : -INFINITY;
+                mx[i] = fmaxf(s0[i], s1[i]);
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < RPW; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], o));
+#pragma unroll
+            for (int i = 0; i < RPW; ++i) {
+                const int r = warp + LD_WARPS * i;
+                mx[i] = fmaxf(m_run[r], mx[i]);
+                const bf16 pa = __float2bfloat16_rn(s0[i] == -INFINITY ? 0.f : exp2f(s0[i] - mx[i]));
+                const bf16 pb = __float2bfloat16_rn(s1[i] == -INFINITY ? 0.f : exp2f(s1[i] - mx[i]));
+                Ps[r * PROW + lane] = pa;
+                Ps[r * PROW + lane + 32] = pb;
+                sum[i] = __bfloat162float(pa) + __bfloat162float(pb);
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < RPW; ++i) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], o);
+            __syncwarp();
+            if (lane == 0) {
+#pragma unroll
+                for (int i = 0; i < RPW; ++i) {
+                    const int r = warp + LD_WARPS * i;
+                    const float c = m_run[r] == -INFINITY ? 0.f : exp2f(m_run[r] - mx[i]);
+                    corr[r] = c;
+                    l_run[r] = l_run[r] * c + sum[i];
+                    m_run[r] = mx[i];
+                }
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const float c0 = corr[m * 16 + gid], c1 = corr[m * 16 + gid + 8];
+            if (!__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) continue;  // no running maximum moved
+#pragma unroll
+            for (int i = 0; i < NTW; ++i) {
+                acc[m][i][0] *= c0; acc[m][i][1] *= c0;
+                acc[m][i][2] *= c1; acc[m][i][3] *= c1;
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < LA_TILE; k += 16) {
+            uint32_t pf[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) la_ldsm4(pf[m], Ps + (m * 16 + (lane & 15)) * PROW + k + (lane >> 4) * 8);
+            const bf16 *vrow = C + (size_t)(k + (lane & 15)) * ld + c_first * 8 + (lane >> 4) * 8;
+#pragma unroll
+            for (int i = 0; i < NTW; i += 2) {
+                if (i < ntw) {  // an odd count reads 8 columns past the warp's own: inside the padded row, not used
+                    uint32_t b[4];
+                    la_ldsm4t(b, vrow + i * 8);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        mma16816<bf16>(acc[m][i], pf[m][0], pf[m][1], pf[m][2], pf[m][3], b[0], b[1]);
+                        if (NTW > 1 && i + 1 < ntw)
+                            mma16816<bf16>(acc[m][i + 1 < NTW ? i + 1 : i], pf[m][0], pf[m][1], pf[m][2], pf[m][3], b[2], b[3]);
+                    }
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            const int r = m * 16 + gid + 8 * hf;
+            if (r >= blk.rows) continue;
+            float *o = a.part_o + ((size_t)(blk.row0 + r) * a.splits + sp) * R + c_first * 8 + 2 * t4;
 #pragma unroll
             for (int i = 0; i < NTW; ++i)
                 if (i < ntw) *reinterpret_cast<float2 *>(o + i * 8) = make_float2(acc[m][i][2 * hf], acc[m][i][2 * hf + 1]);
@@ -516,18 +752,25 @@ __global__ void __launch_bounds__(LA_ROWS_F32 * 32) latent_attn_f32_kernel(const
 int latent_attn_rows_per_block(int heads, int r_p, bool decode, int dt) {
     (void)r_p;
     if (dt == LCU_F32) return LA_ROWS_F32;
-    return !decode || heads > 32 ? 64 : (heads > 16 ? 32 : 16);
+    return !decode ? 64 : (heads > 16 ? 32 : 16);
 }
 
-static size_t la_smem(int mt, int r_p) {
+static size_t ld_smem(int mt, int r_p) {
+    return (size_t)2 * LA_TILE * (r_p + 8) * 2 + (size_t)16 * mt * (LA_TILE + 8) * 2 + (size_t)16 * mt * (LD_SLICES * (LA_TILE + 4) + 3) * 4;
+}
+static size_t lp_smem(int mt, int r_p) {
     return (size_t)(16 * mt + 2 * LA_TILE) * (r_p + 8) * 2 + (size_t)16 * mt * (LA_TILE + 8) * 2 + (size_t)16 * mt * (LA_TILE + 4 + 3) * 4;
 }
 
 template <int MT, int RB>
 static int la_inst(const LatentAttnArgs &a, dim3 grid, cudaStream_t s, bool pdl, bool dry) {
-    const size_t smem = la_smem(MT, a.r_p);
-    if (dry) return raise_smem(latent_attn_kernel<MT, RB>, la_smem(MT, RB));
-    LCU_CHECK_CUDA(launch_kernel(latent_attn_kernel<MT, RB>, grid, dim3(LA_THREADS), smem, s, pdl, a));
+    if constexpr (MT == 4) {
+        if (dry) return raise_smem(latent_attn_kernel<RB>, lp_smem(MT, RB));
+        LCU_CHECK_CUDA(launch_kernel(latent_attn_kernel<RB>, grid, dim3(LA_THREADS), lp_smem(MT, a.r_p), s, pdl, a));
+    } else {
+        if (dry) return raise_smem(latent_decode_kernel<MT, RB>, ld_smem(MT, RB));
+        LCU_CHECK_CUDA(launch_kernel(latent_decode_kernel<MT, RB>, grid, dim3(LD_THREADS), ld_smem(MT, a.r_p), s, pdl, a));
+    }
     return LCU_OK;
 }
 
@@ -644,6 +887,7 @@ __global__ void __launch_bounds__(128) expanded_attn_kernel(const ExpandedAttnAr
     }
     load_tile(0, 0);
     la_commit();
+    const float scale2 = a.scale * 1.4426950408889634f;  // scores in powers of two
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     float o[NTO][4];
 #pragma unroll
@@ -675,10 +919,10 @@ __global__ void __launch_bounds__(128) expanded_attn_kernel(const ExpandedAttnAr
 #pragma unroll
         for (int nt = 0; nt < NTS; ++nt) {
             const int p = tile * LA_TILE + nt * 8 + 2 * t4;
-            sc[nt][0] = p <= lim0 ? sc[nt][0] * a.scale : -INFINITY;
-            sc[nt][1] = p + 1 <= lim0 ? sc[nt][1] * a.scale : -INFINITY;
-            sc[nt][2] = p <= lim1 ? sc[nt][2] * a.scale : -INFINITY;
-            sc[nt][3] = p + 1 <= lim1 ? sc[nt][3] * a.scale : -INFINITY;
+            sc[nt][0] = p <= lim0 ? sc[nt][0] * scale2 : -INFINITY;
+            sc[nt][1] = p + 1 <= lim0 ? sc[nt][1] * scale2 : -INFINITY;
+            sc[nt][2] = p <= lim1 ? sc[nt][2] * scale2 : -INFINITY;
+            sc[nt][3] = p + 1 <= lim1 ? sc[nt][3] * scale2 : -INFINITY;
             mt0 = fmaxf(mt0, fmaxf(sc[nt][0], sc[nt][1]));
             mt1 = fmaxf(mt1, fmaxf(sc[nt][2], sc[nt][3]));
         }
@@ -687,7 +931,7 @@ __global__ void __launch_bounds__(128) expanded_attn_kernel(const ExpandedAttnAr
         mt1 = fmaxf(mt1, __shfl_xor_sync(0xffffffffu, mt1, 1));
         mt1 = fmaxf(mt1, __shfl_xor_sync(0xffffffffu, mt1, 2));
         const float mn0 = fmaxf(m0, mt0), mn1 = fmaxf(m1, mt1);
-        const float c0 = m0 == -INFINITY ? 0.f : expf(m0 - mn0), c1 = m1 == -INFINITY ? 0.f : expf(m1 - mn1);
+        const float c0 = m0 == -INFINITY ? 0.f : exp2f(m0 - mn0), c1 = m1 == -INFINITY ? 0.f : exp2f(m1 - mn1);
         const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
         m0 = mn0;
         m1 = mn1;
@@ -695,8 +939,8 @@ __global__ void __launch_bounds__(128) expanded_attn_kernel(const ExpandedAttnAr
         float s0 = 0.f, s1 = 0.f;
 #pragma unroll
         for (int nt = 0; nt < NTS; ++nt) {
-            pa[nt][0] = Act<bf16>::pack(expf(sc[nt][0] - mu0), expf(sc[nt][1] - mu0));
-            pa[nt][1] = Act<bf16>::pack(expf(sc[nt][2] - mu1), expf(sc[nt][3] - mu1));
+            pa[nt][0] = Act<bf16>::pack(exp2f(sc[nt][0] - mu0), exp2f(sc[nt][1] - mu0));
+            pa[nt][1] = Act<bf16>::pack(exp2f(sc[nt][2] - mu1), exp2f(sc[nt][3] - mu1));
             const float2 f0 = Act<bf16>::to_f2(pa[nt][0]), f1 = Act<bf16>::to_f2(pa[nt][1]);
             s0 += f0.x + f0.y;
             s1 += f1.x + f1.y;

@@ -366,6 +366,7 @@ extern "C" int lcu_argmax_rows_noalloc(lcu_kv_pair *out, const void *logits, int
                                        lcu_stream_t stream) {
     using namespace lcu;
     LCU_REQUIRE(out && logits, "argmax_rows_noalloc: null argument");
+    LCU_REQUIRE(dt == LCU_F16 || dt == LCU_BF16, "argmax_rows_noalloc: logits dtype %d unsupported", dt);
     LCU_REQUIRE(rows >= 1 && n >= 1, "argmax_rows_noalloc: rows = %d, n = %zu", rows, n);
     size_t slots = (size_t)rows * ((n + ARGMAX_CHUNK - 1) / ARGMAX_CHUNK);
     if (slots > NOALLOC_SLOTS || argmax_workspace_bytes(rows, n) > sizeof(g_noalloc_scratch)) {

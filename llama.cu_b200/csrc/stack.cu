@@ -53,7 +53,7 @@ static int round_expand_min(const Stack &S) {
 static int attn_splits_for(const lcu_ctx *c, int blocks) {
     if (c->dt == LCU_F32) return 1;
     const int tiles = (c->desc.nctx + 63) / 64;
-    int z = (sm_count() + blocks - 1) / (blocks > 0 ? blocks : 1);
+    int z = sm_count() / (blocks > 0 ? blocks : 1);
     if (z > 32) z = 32;
     if (z > tiles) z = tiles;
     return z < 1 ? 1 : z;
@@ -288,12 +288,15 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
     return LCU_OK;
 }
 
+bool stack_pdl(const lcu_ctx *c, int n_tok) { return tuning().stack_pdl && c->dt != LCU_F32 && n_tok <= 256; }
+
 namespace {
 
 struct Launcher {
     lcu_ctx *c;
     cudaStream_t s;
     int *count;
+    bool pdl;
 
     // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
     int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr) {
@@ -310,7 +313,7 @@ struct Launcher {
         const size_t yb = epilogue == EPI_STORE_F32 ? 4 : 2;
         const bool tc = n > 4;
         for (int t0 = 0; t0 < n;) {
-            const int most = tc ? tuning().tc_block : gemv_max_tokens(in);
+            const int most = tc ? (tuning().tc_block < 256 ? tuning().tc_block : GEMM_TC_MAX_TOKENS) : gemv_max_tokens(in);
             const int nt = n - t0 < most ? n - t0 : most;
             GemvArgs a{};
             a.w = w;
@@ -319,9 +322,10 @@ struct Launcher {
             a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq;
             a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
             a.stride_y = stride_y;
-            a.pdl_trigger = 2;
-            a.early_prefetch = 1;
-            int rc = tc ? gemm_tc_launch(a, c->dt, s, false) : gemv_launch(a, c->dt, s, false);
+            // a dependent launch requests its first weights ahead of the wait for its predecessor
+            a.pdl_trigger = pdl ? 0 : 2;
+            a.early_prefetch = pdl ? 3 : 1;
+            int rc = tc ? gemm_tc_launch(a, c->dt, s, pdl) : gemv_launch(a, c->dt, s, pdl);
             if (rc) return rc;
             ++*count;
             t0 += nt;
@@ -337,7 +341,8 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
     const lcu_model_desc &d = c->desc;
     const int dt = c->dt, n = r.n_tok;
     const size_t eb = act_bytes(c);
-    Launcher L{c, s, count};
+    const bool pdl = stack_pdl(c, n);
+    Launcher L{c, s, count, pdl};
     unsigned char *D = c->desc_dev, *B = D + r.L.stack;
     const StackDesc o = stack_desc(r.n_tok, r.n_req);
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(D + r.L.tokens), *pos = reinterpret_cast<const uint32_t *>(D + r.L.pos);
@@ -370,7 +375,7 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
             }
         }
         ++*count;
-        return op_mix_input(a, dt, s, false);
+        return op_mix_input(a, dt, s, pdl);
     };
     rc = residual(nullptr, 0, true);
     if (rc) return rc;
@@ -386,7 +391,7 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
         ln.q_norm = W.q_norm; ln.kv_norm = W.kv_norm; ln.eps = d.eps; ln.cq = S.cq;
         ln.pool = c->pool; ln.page_elems = c->geom.page_elems; ln.c_off = Y.c_off; ln.page_shift = c->geom.page_shift;
         ln.tok_req = tok_req; ln.pos = pos; ln.page_table = page_table; ln.pt_stride = c->pt_stride;
-        rc = latent_norm_launch(ln, dt, s, false);
+        rc = latent_norm_launch(ln, dt, s, pdl);
         if (rc) return rc;
         ++*count;
         rc = L.linear(W.uq, Y.qr_p, q_stride, S.cq, n, S.q, q_stride, EPI_STORE);
@@ -404,14 +409,14 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
             a.q = S.qa; a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift;
             a.page_table = page_table; a.pt_stride = c->pt_stride; a.req_first = i32(o.abs_first); a.req_id = i32(o.abs_id); a.req_pos = i32(o.req_pos);
             a.n_req = q.n_abs_req; a.n_tok = q.n_abs_tok; a.decode = q.abs_decode; a.heads = heads; a.r_p = Y.r_p; a.scale = Y.d.scale;
-            a.part_o = S.part_o; a.part_ml = S.part_ml; a.part_n = S.part_n; a.splits = splits;
+            a.part_o = S.part_o; a.part_ml = S.part_ml; a.part_n = S.part_n; a.splits = splits; a.status = c->dev_status;
             if (dt == LCU_F32) {
                 LinearF32Args f{};
                 f.x = reinterpret_cast<const float *>(S.q); f.stride_x = q_stride; f.head_x = Y.dim_p; f.x_rows = i32(o.abs_tok);
                 f.w = W.ukt; f.y = reinterpret_cast<float *>(S.qa); f.stride_y = heads * Y.r_p; f.head_y = Y.r_p;
                 f.n = q.n_abs_tok; f.in = Y.dim_p; f.out = Y.r_p; f.heads = heads; f.epilogue = EPI_STORE_F32;
                 rc = linear_f32_launch(f, s);
-                if (!rc) rc = latent_attn_launch(a, dt, s, false);
+                if (!rc) rc = latent_attn_launch(a, dt, s, pdl);
                 f = LinearF32Args{};
                 f.x = S.part_o; f.stride_x = heads * Y.r_p; f.head_x = Y.r_p; f.w = uv;
                 f.y = reinterpret_cast<float *>(S.att); f.stride_y = Y.hv_p; f.head_y = Y.vdim_p; f.y_rows = i32(o.abs_tok);
@@ -422,14 +427,14 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
                 HeadLinearArgs f{};
                 f.x = S.q; f.stride_x = q_stride; f.head_x = Y.dim_p; f.x_rows = i32(o.abs_tok); f.w = W.ukt;
                 f.y = S.qa; f.stride_y = heads * Y.r_p; f.head_y = Y.r_p; f.n = q.n_abs_tok; f.in = Y.dim_p; f.out = Y.r_p; f.heads = heads;
-                rc = head_linear_launch(f, s, false);
-                if (!rc) rc = latent_attn_launch(a, dt, s, false);
+                rc = head_linear_launch(f, s, pdl);
+                if (!rc) rc = latent_attn_launch(a, dt, s, pdl);
                 f = HeadLinearArgs{};
                 f.w = uv; f.y = S.att; f.stride_y = Y.hv_p; f.head_y = Y.vdim_p; f.y_rows = i32(o.abs_tok);
                 f.n = q.n_abs_tok; f.in = Y.r_p; f.out = Y.vdim_p; f.heads = heads;
                 f.part_o = S.part_o; f.part_ml = S.part_ml; f.part_n = S.part_n; f.splits = splits;
                 f.gate = gate; f.stride_gate = lat_stride;
-                if (!rc) rc = head_linear_launch(f, s, false);
+                if (!rc) rc = head_linear_launch(f, s, pdl);
             }
             if (rc) return rc;
             *count += 3;
@@ -468,14 +473,14 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
 }
 
 int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, float *out_f32, cudaStream_t s, int *count) {
-    (void)r;
     if (n_rows <= 0) return LCU_OK;
     Stack &S = *c->stack;
+    const bool pdl = stack_pdl(c, r.n_tok);
     int rc = op_scalar_norm_rows(S.hout, reinterpret_cast<const float *>(c->x), rows, n_rows, c->desc.d, S.d_p,
-                                 reinterpret_cast<const float *>(c->out_norm), 0, c->desc.eps, c->dt, s, false);
+                                 reinterpret_cast<const float *>(c->out_norm), 0, c->desc.eps, c->dt, s, pdl);
     if (rc) return rc;
     ++*count;
-    Launcher L{c, s, count};
+    Launcher L{c, s, count, pdl};
     void *y = out_f32 ? reinterpret_cast<void *>(out_f32) : c->logits;
     return L.linear(c->lm_head, S.d_p, S.vocab_p, S.hout, n_rows, y, S.vocab_p, out_f32 ? EPI_STORE_F32 : EPI_STORE);
 }

@@ -75,6 +75,8 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H);
 int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count);
 // final norm of the asked rows and the LM head; logits in the activation dtype, or f32 at `out_f32`
 int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, float *out_f32, cudaStream_t s, int *count);
+// rounds short enough for every launch to be a programmatic dependent of its predecessor
+bool stack_pdl(const lcu_ctx *c, int n_tok);
 double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_out);
 
 // ---- stack_ops.cu
@@ -171,6 +173,7 @@ struct LatentAttnArgs {
     float *part_o, *part_ml;    // [row][splits][r_p] unnormalised, [row][splits][2]
     int *part_n;                // [row] splits used
     int splits;                 // grid depth
+    uint32_t *status;           // bit 4: a bounded wait ran out
 };
 int latent_attn_rows_per_block(int heads, int r_p, bool decode, int dt);
 int latent_attn_launch(const LatentAttnArgs &a, int dt, cudaStream_t s, bool pdl, bool dry = false);

@@ -48,6 +48,11 @@ class LayeredConfig:
     eps: float
     act_dtype: int = BF16  # or F32: everything in 32-bit arithmetic
     nctx: int = 2048
+    arch: str = "Zefedra"  # key of `architectures()`
+
+    @property
+    def family(self):
+        return architectures()[self.arch]
 
     @property
     def n_layers(self):

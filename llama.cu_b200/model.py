@@ -11,6 +11,8 @@ import numpy as np
 
 from . import (BF16, F16, F32, LINEAR_KINDS, Q8_0, W_ATTN_NORM, W_DOWN, W_EMBD, W_FFN_NORM, W_GATE_UP, W_LM_HEAD,
                W_O, W_OUT_NORM, W_QKV, Context, ModelDesc, check, load_library, stream_ptr)
+from . import zefedra
+from .layered import LayeredConfig
 
 
 @dataclass(frozen=True)
@@ -69,8 +71,15 @@ CONFIGS = {
 }
 
 
+# layered families at the widths of the LLaMA shapes above (no published checkpoint has these sizes)
+CONFIGS["zefedra8b"] = zefedra.uniform("zefedra8b", 32, 4096, 32, 128, 128, 1536, 512, 14336, 128256)
+CONFIGS["zefedra1b"] = zefedra.uniform("zefedra1b", 16, 2048, 16, 128, 128, 768, 256, 8192, 128256)
+
+
 def reduced(cfg, n_layers, vocab=None, name=None):
     """The same layer shape with fewer layers (and optionally a smaller vocabulary)."""
+    if isinstance(cfg, LayeredConfig):
+        return replace(cfg, layers=cfg.layers[:n_layers], vocab=vocab or cfg.vocab, name=name or f"{cfg.name}-L{n_layers}")
     return replace(cfg, n_layers=n_layers, vocab=vocab or cfg.vocab, name=name or f"{cfg.name}-L{n_layers}")
 
 
@@ -131,6 +140,9 @@ def iter_synth_weights_torch(cfg, seed=0, device="cuda:0"):
     """Generator form of synth_weights_torch: yields ((layer, kind), tensor) one tensor at a time, so a
     tensor-parallel rank can slice each full tensor and drop it before the next one is drawn."""
     import torch
+    if isinstance(cfg, LayeredConfig):
+        yield from cfg.family.synth_weights(cfg, seed, device)
+        return
     g = torch.Generator(device=device)
     g.manual_seed(seed)
     tdt = torch.float16 if cfg.act_dtype == F16 else torch.bfloat16
@@ -190,7 +202,7 @@ def load_model(cfg, weights, device=0, kv_bytes=None, tp_rank=0, tp_size=1, comm
     creates the KV pool."""
     import torch
     dev = f"cuda:{device}"
-    layers = cfg.layer_descs() if hasattr(cfg, "layer_descs") else None  # models described layer by layer (layered.py)
+    layers = cfg.layer_descs() if isinstance(cfg, LayeredConfig) else None
     ctx = Context(cfg.desc(page_tokens, max_tokens, max_seqs, nctx), device, tp_rank, tp_size, comm, layers=layers)
     lib = load_library()
     items = weights.items() if isinstance(weights, dict) else weights

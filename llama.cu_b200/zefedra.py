@@ -21,6 +21,13 @@ def read_config(raw):
     return LayeredConfig("zefedra", raw["width"], raw["vocab"], tuple(layers), raw["norm"]["eps"])
 
 
+def uniform(name, n_layers, d, heads, dim, v_dim, q_rank, kv_rank, ff, vocab, gated=True, eps=1e-6, nctx=2048):
+    """A model of equal layers, gated and plain mixers alternating (`gated`) or all plain."""
+    def layer(i):
+        return LayerConfig(LatentMixer(heads, dim, v_dim, q_rank, kv_rank, dim ** -0.5, gated and i % 2 == 1), ff)
+    return LayeredConfig(name, d, vocab, tuple(layer(i) for i in range(n_layers)), eps, nctx=nctx)
+
+
 def tensor_shapes(cfg):
     """{name: shape} of the model file."""
     out = {"embed": (cfg.vocab, cfg.d), "final.norm": (), "head": (cfg.vocab, cfg.d)}
@@ -56,6 +63,11 @@ def pack(cfg, tensors):
                             g=t(p + "mix.g") if l.mixer.out_gate else None)
         for kind, w in parts + pack_block(cfg.d, l.ff, t(p + "norm1"), shift=t(p + "shift"), **ff):
             yield (i, kind), w
+
+
+def synth_weights(cfg, seed=0, device="cuda:0"):
+    """Seeded random weights in the library's layouts: yields ((layer, kind), tensor)."""
+    return pack(cfg, synth_tensors(cfg, seed, device))
 
 
 def synth_tensors(cfg, seed=0, device="cuda:0"):
