@@ -18,13 +18,12 @@
 //     scratch memory and the last CTA of a row block to arrive adds them in split order.
 // Every mbarrier wait is bounded by a wall-clock limit: on expiry the kernel records a status bit,
 // skips the remaining work, frees its TMEM and returns.
-#include <cuda.h>
-
 #include <cstdlib>
 #include <map>
 #include <mutex>
 
 #include "gemv.cuh"
+#include "tc.cuh"
 
 namespace lcu {
 
@@ -32,62 +31,6 @@ constexpr int TC_THREADS = 192;
 constexpr int TC_BM = 128;         // weight rows per CTA tile
 constexpr int TC_BK = 64;          // K elements per stage (128 bytes: one swizzle row)
 constexpr int TC_A_BYTES = TC_BM * TC_BK * 2;
-constexpr unsigned long long TC_WAIT_NS = 2000000000ull;
-
-// ------------------------------------------------------------------ PTX helpers
-__device__ __forceinline__ unsigned long long tc_ns() {
-    unsigned long long t;
-    asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
-    return t;
-}
-__device__ __forceinline__ uint32_t tc_smem(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void tc_mbar_init(uint32_t bar, uint32_t count) {
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count) : "memory");
-}
-__device__ __forceinline__ void tc_mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ bool tc_mbar_try(uint32_t bar, uint32_t parity) {
-    uint32_t ok;
-    asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}"
-                 : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    return ok != 0;
-}
-__device__ __forceinline__ bool tc_mbar_wait(uint32_t bar, uint32_t parity, volatile int *abort_flag) {
-    if (tc_mbar_try(bar, parity)) return true;
-    unsigned long long t0 = tc_ns();
-    for (unsigned it = 1;; ++it) {
-        if (tc_mbar_try(bar, parity)) return true;
-        if ((it & 255u) == 0 && (*abort_flag || tc_ns() - t0 > TC_WAIT_NS)) return false;
-    }
-}
-__device__ __forceinline__ void tc_tma_2d(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-                 ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
-}
-// shared-memory operand descriptor: K-major tile, 128-byte swizzle, 8-row groups 1024 bytes apart
-__device__ __forceinline__ uint64_t tc_desc(uint32_t saddr) {
-    return (uint64_t)((saddr >> 4) & 0x3FFFu) | (1ull << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
-}
-__device__ __forceinline__ void tc_mma_f16(uint32_t d_tmem, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
-                 ::"r"(d_tmem), "l"(a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void tc_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tc_ld16(uint32_t taddr, uint32_t r[16]) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-                   "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-                 : "r"(taddr) : "memory");
-}
-
-__device__ __forceinline__ void tc_ld8(uint32_t taddr, uint32_t r[8]) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
-                 : "r"(taddr) : "memory");
-}
 
 constexpr int TC_MAX_STAGES = 12;
 
@@ -678,26 +621,6 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
 }
 
 // ------------------------------------------------------------------ host side
-
-typedef CUresult (*TcEncodeFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
-                               const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
-                               CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static TcEncodeFn tc_encode_fn() {
-    static TcEncodeFn fn = nullptr;
-    static bool tried = false;
-    static std::mutex mu;
-    std::lock_guard<std::mutex> lk(mu);
-    if (!tried) {
-        tried = true;
-        void *p = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-            q == cudaDriverEntryPointSuccess)
-            fn = reinterpret_cast<TcEncodeFn>(p);
-    }
-    return fn;
-}
 
 // 2-D map of a row-major [rows, cols] matrix of 16-bit elements; box = 64 columns x box_rows rows, 128-byte swizzle
 static int tc_make_map(CUtensorMap *m, const void *base, int dt, uint64_t rows, uint64_t cols, uint64_t row_stride,

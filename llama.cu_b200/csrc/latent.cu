@@ -465,7 +465,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_kernel(const Latent
     }
 }
 
-// Decode form (up to 32 rows per CTA).  The latent dimension is cut into slices, one per pair of warps; a warp keeps
+// Decode form for pages of fewer than 64 tokens (see latent_tc.cu for the others), up to 32 rows per CTA.  The latent dimension is cut into slices, one per pair of warps; a warp keeps
 // its slice of the query fragments in registers for the whole kernel and computes partial scores of 32 positions, which the
 // softmax sums over the slices: every byte of a tile crosses the shared-memory port once per product.  Slices and output
 // columns are dealt in whole MMA steps, so any latent size that is a multiple of 16 works.  The gather of tile
@@ -749,9 +749,9 @@ __global__ void __launch_bounds__(LA_ROWS_F32 * 32) latent_attn_f32_kernel(const
 }
 
 // rows per CTA: as many 16-row tiles as the heads of one token need (decode), or 64 to share every tile among many queries
-int latent_attn_rows_per_block(int heads, int r_p, bool decode, int dt) {
-    (void)r_p;
+int latent_attn_rows_per_block(int heads, bool decode, int dt, int page_tokens) {
     if (dt == LCU_F32) return LA_ROWS_F32;
+    if (decode && latent_tc_supported(page_tokens)) return latent_tc_rows(heads);
     return !decode ? 64 : (heads > 16 ? 32 : 16);
 }
 
@@ -793,12 +793,13 @@ int latent_attn_launch(const LatentAttnArgs &a, int dt, cudaStream_t s, bool pdl
     const size_t smem_f32 = (size_t)(LA_ROWS_F32 * a.r_p + 32 * (a.r_p + 1)) * 4;
     if (dry) {
         if (dt == LCU_F32) return raise_smem(latent_attn_f32_kernel, (size_t)(LA_ROWS_F32 * 512 + 32 * 513) * 4);
-        int rc = la_rb<1>(a, dim3(1), s, false, true);
+        int rc = latent_tc_launch(a, s, false, true);
+        if (!rc) rc = la_rb<1>(a, dim3(1), s, false, true);
         if (!rc) rc = la_rb<2>(a, dim3(1), s, false, true);
         return rc ? rc : la_rb<4>(a, dim3(1), s, false, true);
     }
     if (a.n_tok <= 0) return LCU_OK;
-    const int rpb = latent_attn_rows_per_block(a.heads, a.r_p, a.decode != 0, dt);
+    const int rpb = latent_attn_rows_per_block(a.heads, a.decode != 0, dt, 1 << a.page_shift);
     // upper bound of row blocks: the exact count of a decode round, one partial block per request otherwise
     const long blocks = a.decode ? (long)a.n_tok * ((a.heads + rpb - 1) / rpb) : (long)a.n_tok * a.heads / rpb + a.n_req;
     LCU_REQUIRE(blocks < (1l << 31) && a.splits >= 1 && a.splits <= HL_MAX_SPLITS, "latent attention: grid out of range");
@@ -808,6 +809,7 @@ int latent_attn_launch(const LatentAttnArgs &a, int dt, cudaStream_t s, bool pdl
         LCU_CHECK_CUDA(launch_kernel(latent_attn_f32_kernel, grid, dim3(LA_ROWS_F32 * 32), smem_f32, s, false, a));
         return LCU_OK;
     }
+    if (a.decode && latent_tc_supported(1 << a.page_shift)) return latent_tc_launch(a, s, pdl);
     return rpb == 16 ? la_rb<1>(a, grid, s, pdl, false) : (rpb == 32 ? la_rb<2>(a, grid, s, pdl, false) : la_rb<4>(a, grid, s, pdl, false));
 }
 

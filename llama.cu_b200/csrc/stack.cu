@@ -124,7 +124,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     for (const StackLayer &L : S->layers)
         for (int dec = 0; dec < 2; ++dec)
             for (int n = 1; n <= c->max_tokens; n = n < 64 ? n + 1 : (n == c->max_tokens ? n + 1 : (2 * n < c->max_tokens ? 2 * n : c->max_tokens))) {
-                const int rpb = latent_attn_rows_per_block(L.d.heads, L.r_p, dec != 0, c->dt);
+                const int rpb = latent_attn_rows_per_block(L.d.heads, dec != 0, c->dt, c->geom.page_tokens);
                 const int blocks = dec ? n * ((L.d.heads + rpb - 1) / rpb) : n * L.d.heads / rpb + 1;
                 // between two sampled sizes the split depth does not grow while the rows at most double
                 const size_t r = (size_t)(n < 64 || n == c->max_tokens ? n : 2 * n) * L.d.heads * attn_splits_for(c, blocks);
@@ -401,12 +401,12 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
 
         // --- absorbed form: queries into latent space, attention over the cached latents, value map of the merged rows
         if (q.n_abs_tok) {
-            const int rpb = latent_attn_rows_per_block(heads, Y.r_p, q.abs_decode, dt);
+            const int rpb = latent_attn_rows_per_block(heads, q.abs_decode, dt, c->geom.page_tokens);
             const int blocks = q.abs_decode ? q.n_abs_tok * ((heads + rpb - 1) / rpb) : q.n_abs_tok * heads / rpb + 1;
             const int splits = attn_splits_for(c, blocks);
             LCU_REQUIRE((size_t)q.n_abs_tok * heads * splits <= S.part_rows, "step: attention partials of %d tokens do not fit", q.n_abs_tok);
             LatentAttnArgs a{};
-            a.q = S.qa; a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift;
+            a.q = S.qa; a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift; a.n_pages = c->n_pages;
             a.page_table = page_table; a.pt_stride = c->pt_stride; a.req_first = i32(o.abs_first); a.req_id = i32(o.abs_id); a.req_pos = i32(o.req_pos);
             a.n_req = q.n_abs_req; a.n_tok = q.n_abs_tok; a.decode = q.abs_decode; a.heads = heads; a.r_p = Y.r_p; a.scale = Y.d.scale;
             a.part_o = S.part_o; a.part_ml = S.part_ml; a.part_n = S.part_n; a.splits = splits; a.status = c->dev_status;

@@ -161,7 +161,7 @@ struct LatentAttnArgs {
     const void *q;              // [rows, r_p]
     const void *pool;
     size_t page_elems, c_off;
-    int page_shift;
+    int page_shift, n_pages;
     const int32_t *page_table;
     int pt_stride;
     const int32_t *req_first;   // [n_req + 1] first absorbed token of each absorbed request
@@ -175,8 +175,12 @@ struct LatentAttnArgs {
     int splits;                 // grid depth
     uint32_t *status;           // bit 4: a bounded wait ran out
 };
-int latent_attn_rows_per_block(int heads, int r_p, bool decode, int dt);
+int latent_attn_rows_per_block(int heads, bool decode, int dt, int page_tokens);
 int latent_attn_launch(const LatentAttnArgs &a, int dt, cudaStream_t s, bool pdl, bool dry = false);
+// ---- latent_tc.cu: the decode form on tcgen05 (pages of at least 64 tokens)
+bool latent_tc_supported(int page_tokens);
+int latent_tc_rows(int heads);
+int latent_tc_launch(const LatentAttnArgs &a, cudaStream_t s, bool pdl, bool dry = false);
 // copies the cached latents of the batch's requests into consecutive rows
 int latent_gather_launch(void *dst, const void *pool, size_t page_elems, size_t c_off, int page_shift, const int32_t *page_table,
                          int pt_stride, const int4 *reqs, int n_req, int max_rows, int r_p, cudaStream_t s);
