@@ -7,11 +7,13 @@
 // S^T and O^T live in TMEM.  Per CTA (one row block of one token, one split of its context):
 //   - warp 0 (one lane): TMA producer; a ring of pieces [128 positions x 128 latents], loaded page by page (two boxes of
 //     64 latents, 128-byte swizzle); pieces return to the ring as the second product finishes with them;
-//   - warp 1 (one lane): MMA issuer;
-//   - warps 2..5: softmax, one position per thread.  Column maxima by a transposing butterfly over the warp, then across
-//     the four warps; the output is rescaled only when some maximum has grown by more than a factor of 2^8 (until then the
-//     weights are taken relative to the older, smaller maximum, which changes nothing but their scale); probabilities go
-//     to shared memory as bf16, the row sums are those of the rounded values.
+//   - warp 1: MMA issuer (the whole warp runs the loop, so operand descriptors stay in uniform registers; one elected lane
+//     issues);
+//   - warps 2..5: softmax, one position per thread.  Weights are taken relative to a reference maximum per head that moves
+//     only when some score exceeds it by more than a factor of 2^8 (which changes nothing but the weights' common scale): the
+//     usual tile needs one vote, no reduction and no rescale.  When the reference moves, column maxima come from a
+//     transposing butterfly over the warp and across the four warps, and O^T is rescaled in TMEM.  Probabilities go to
+//     shared memory as bf16 rows of heads (an MN-major operand); the row sums are those of the rounded values.
 // Rows of a tile past the context are zeroed in shared memory before the products.  Every wait is bounded: when one runs
 // out the CTA records a status bit, waits for its own copies, frees its TMEM and returns.
 #include "stack.cuh"
@@ -33,8 +35,8 @@ struct LtShared {
     unsigned long long full[LT_MAX_SLOTS], empty[LT_MAX_SLOTS], q_full, s_full, z_ready, p_ready, o_done;
     uint32_t tmem_base;
     int abort_flag;
-    float mx[4][N];                // column maxima of each softmax warp
-    float ref[4][N], corr[4][N];   // every warp's own copy of the reference maxima and the rescale factors
+    alignas(16) float mx[4][N];    // column maxima of each softmax warp
+    alignas(16) float ref[4][N], corr[4][N];   // every warp's own copy of the reference maxima and the rescale factors
 };
 
 __device__ __forceinline__ void lt_tma_3d(uint32_t dst, const CUtensorMap *map, int x, int y, int z, uint32_t bar) {
@@ -45,6 +47,35 @@ __device__ __forceinline__ void lt_tma_3d(uint32_t dst, const CUtensorMap *map, 
 // (the K direction) 1024 bytes apart
 __device__ __forceinline__ uint64_t lt_desc_mn(uint32_t saddr) {
     return (uint64_t)((saddr >> 4) & 0x3FFFu) | ((uint64_t)(LT_BOX >> 4) << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
+}
+// probabilities [position][N heads], MN-major with the swizzle of their row size; groups of 8 positions 16 N bytes apart
+template <int N>
+__device__ __forceinline__ uint64_t lt_desc_p(uint32_t saddr) {
+    constexpr uint64_t layout = N == 64 ? 2 : (N == 32 ? 4 : 6);  // 128-, 64-, 32-byte swizzle
+    return (uint64_t)((saddr >> 4) & 0x3FFFu) | (1ull << 16) | ((uint64_t)N << 32) | (1ull << 46) | (layout << 61);
+}
+// byte offset of 16-byte chunk j (8 heads) of position p
+template <int N>
+__device__ __forceinline__ int lt_p_off(int p, int j) {
+    const int x = N == 64 ? (p & 7) : (N == 32 ? ((p >> 1) & 3) : ((p >> 2) & 1));
+    return p * (2 * N) + ((j ^ x) << 4);
+}
+__device__ __forceinline__ bool lt_elect() {
+    uint32_t r;
+    asm volatile("{\n .reg .pred p;\n elect.sync _|p, 0xffffffff;\n selp.u32 %0, 1, 0, p;\n}" : "=r"(r));
+    return r != 0;
+}
+__device__ __forceinline__ float lt_exp2(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+// barrier of the four softmax warps that also ORs a flag
+__device__ __forceinline__ bool lt_sync_or(bool v) {
+    uint32_t r;
+    asm volatile("{\n .reg .pred p, q;\n setp.ne.u32 p, %1, 0;\n bar.red.or.pred q, 4, 128, p;\n selp.u32 %0, 1, 0, q;\n}"
+                 : "=r"(r) : "r"((uint32_t)v) : "memory");
+    return r != 0;
 }
 __device__ __forceinline__ void lt_st16(uint32_t taddr, const uint32_t r[16]) {
     asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
@@ -98,15 +129,19 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
     const int R = a.r_p, nbox = R / 64, npiece = (nbox + 1) / 2;
     unsigned char *ring = smem;                                    // [n_slots][LT_PIECE]
     unsigned char *Qs = ring + (size_t)n_slots * LT_PIECE;         // [nbox][N][128 bytes]
-    unsigned char *Ps = Qs + (size_t)nbox * N * 128;               // [2][N][128 bytes]
+    unsigned char *Ps = Qs + (size_t)nbox * N * 128;               // [128 positions][N], swizzled
     LtShared<N> *sh = reinterpret_cast<LtShared<N> *>(Ps + (size_t)2 * N * 128);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     grid_dep_launch();
+    if (tid == 0) {
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&map_c) : "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&map_q) : "memory");
+    }
 
     // row block: one token, up to N of its heads
     const int bpt = (a.heads + N - 1) / N, req = (int)blockIdx.x / bpt, h0 = ((int)blockIdx.x - req * bpt) * N;
     const int row0 = req * a.heads + h0, rows = min(N, a.heads - h0);
-    const int rr = a.req_id[req];
+    const int rr = req;  // a decode round: every request of it, in order
     const int ctx = a.req_pos[rr] + 1;
     const int sp = blockIdx.y;
     const int n_tiles = (ctx + LT_POS - 1) / LT_POS;
@@ -176,42 +211,58 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
             for (int j = it > n_slots ? it - n_slots : 0; j < it; ++j)
                 tc_mbar_wait(tc_smem(&sh->full[j % n_slots]), (uint32_t)(j / n_slots) & 1u, &never);
         }
-    } else if (warp == 1 && lane == 0) {
+    } else if (warp == 1) {
         // ---------------- MMA issuer
         const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-        const uint32_t id_o = id_s | (1u << 15);  // A is MN-major
-        bool ok = tc_mbar_wait(tc_smem(&sh->q_full), 0u, &sh->abort_flag);
-        int it = 0;
-        for (int tile = tile0; tile < tile1 && ok; ++tile, it += npiece) {
-            if (tail && tile == tile1 - 1) ok = tc_mbar_wait(tc_smem(&sh->z_ready), 0u, &sh->abort_flag);
+        const uint32_t id_o = id_s | (1u << 15) | (1u << 16);  // both operands MN-major
+        const uint64_t ring_k = tc_desc(tc_smem(ring)), ring_mn = lt_desc_mn(tc_smem(ring)), q_k = tc_desc(tc_smem(Qs)), p_mn = lt_desc_p<N>(tc_smem(Ps));
+        bool ok = __all_sync(0xffffffffu, tc_mbar_wait(tc_smem(&sh->q_full), 0u, &sh->abort_flag));
+        int slot = 0;        // ring position of the tile's first piece
+        uint32_t phase = 0;  // its parity
+        for (int tile = tile0; tile < tile1 && ok; ++tile) {
+            if (tail && tile == tile1 - 1) ok = __all_sync(0xffffffffu, tc_mbar_wait(tc_smem(&sh->z_ready), 0u, &sh->abort_flag));
+            int sl = slot;
+            uint32_t ph = phase;
             for (int p = 0; p < npiece && ok; ++p) {
-                const int slot = (it + p) % n_slots;
-                ok = tc_mbar_wait(tc_smem(&sh->full[slot]), (uint32_t)((it + p) / n_slots) & 1u, &sh->abort_flag);
+                ok = __all_sync(0xffffffffu, tc_mbar_wait(tc_smem(&sh->full[sl]), ph, &sh->abort_flag));
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                for (int b = 0; b < min(2, nbox - 2 * p); ++b) {
-                    const uint32_t sa = tc_smem(ring + (size_t)slot * LT_PIECE + b * LT_BOX), sb = tc_smem(Qs + (size_t)(2 * p + b) * N * 128);
+                const uint64_t da = ring_k + (uint64_t)(sl * (LT_PIECE >> 4)), db = q_k + (uint64_t)(p * (2 * N * 128 >> 4));
+                if (lt_elect()) {
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) tc_mma_f16(tmem, tc_desc(sa + k * 32), tc_desc(sb + k * 32), id_s, (p > 0 || b > 0 || k > 0) ? 1u : 0u);
+                    for (int k = 0; k < 4; ++k) tc_mma_f16(tmem, da + 2 * k, db + 2 * k, id_s, (p > 0 || k > 0) ? 1u : 0u);
+                    if (2 * p + 1 < nbox) {
+#pragma unroll
+                        for (int k = 0; k < 4; ++k) tc_mma_f16(tmem, da + (LT_BOX >> 4) + 2 * k, db + (N * 128 >> 4) + 2 * k, id_s, 1u);
+                    }
                 }
+                __syncwarp();
+                if (++sl == n_slots) { sl = 0; ph ^= 1u; }
             }
             if (!ok) break;
-            tc_commit(tc_smem(&sh->s_full));
-            ok = tc_mbar_wait(tc_smem(&sh->p_ready), (uint32_t)(tile - tile0) & 1u, &sh->abort_flag);
+            if (lt_elect()) tc_commit(tc_smem(&sh->s_full));
+            __syncwarp();
+            ok = __all_sync(0xffffffffu, tc_mbar_wait(tc_smem(&sh->p_ready), (uint32_t)(tile - tile0) & 1u, &sh->abort_flag));
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             for (int p = 0; p < npiece; ++p) {
-                const int slot = (it + p) % n_slots;
-                const uint32_t sa = tc_smem(ring + (size_t)slot * LT_PIECE), sb = tc_smem(Ps);
+                const uint64_t da = ring_mn + (uint64_t)(slot * (LT_PIECE >> 4));
+                if (lt_elect()) {
 #pragma unroll
-                for (int k = 0; k < 8; ++k)
-                    tc_mma_f16(tmem_o + p * N, lt_desc_mn(sa + k * 2048), tc_desc(sb + (k >> 2) * (N * 128) + (k & 3) * 32), id_o,
-                               (tile > tile0 || k > 0) ? 1u : 0u);
-                tc_commit(tc_smem(&sh->empty[slot]));
+                    for (int k = 0; k < 8; ++k)  // 16 positions: 2 KB of the tile, 16 rows of probabilities
+                        tc_mma_f16(tmem_o + p * N, da + k * (2048 >> 4), p_mn + k * (32 * N >> 4), id_o, (tile > tile0 || k > 0) ? 1u : 0u);
+                    tc_commit(tc_smem(&sh->empty[slot]));
+                }
+                __syncwarp();
+                if (++slot == n_slots) { slot = 0; phase ^= 1u; }
             }
         }
-        if (!ok) stop();
-        else tc_commit(tc_smem(&sh->o_done));
+        if (!ok) {
+            if (lane == 0) stop();
+        } else if (lt_elect()) {
+            tc_commit(tc_smem(&sh->o_done));
+        }
+        __syncwarp();
     } else if (warp >= 2) {
         // ---------------- softmax and epilogue
         const int q = warp & 3, pt = q * 32 + lane;  // a warp may only touch TMEM lanes [32 q, 32 q + 32)
@@ -222,6 +273,8 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
         for (int c = 0; c < N; ++c) l[c] = 0.f;
 #pragma unroll
         for (int g = 0; g < NG; ++g) ref_c[g] = -INFINITY;
+        for (int c = lane; c < N; c += 32) sh->ref[q][c] = 0.f;
+        __syncwarp();
         bool ok = true;
         for (int tile = tile0; tile < tile1; ++tile) {
             const int p0 = tile * LT_POS;
@@ -246,40 +299,45 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
                 for (int c = 0; c < N; c += 16) tc_ld16(tmem + lanes + c, raw + c);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             }
-            const bool visible = p0 + pt < ctx;
-            float v[N];
-#pragma unroll
-            for (int c = 0; c < N; ++c) v[c] = ok && visible ? __uint_as_float(raw[c]) * scale2 : -INFINITY;
-#pragma unroll
-            for (int g = 0; g < NG; ++g) {
-                float w[GC];
-#pragma unroll
-                for (int c = 0; c < GC; ++c) w[c] = v[g * GC + c];
-                const float m = lt_columns<GC, true>(w);
-                if (lane < GC) sh->mx[q][g * GC + lane] = m;
-            }
             if (!lt_sync_and(ok)) { ok = false; break; }
-            float m_new[NG];
-            bool grew = false;
+            const bool visible = p0 + pt < ctx;
+            // scores relative to the references; the first tile always sets them
+            float v[N], top = -INFINITY;
 #pragma unroll
-            for (int g = 0; g < NG; ++g) {
-                const int c = g * GC + lane % GC;
-                m_new[g] = fmaxf(fmaxf(sh->mx[0][c], sh->mx[1][c]), fmaxf(sh->mx[2][c], sh->mx[3][c]));
-                grew = grew || m_new[g] > ref_c[g] + LT_GROW;
+            for (int c = 0; c < N; c += 4) {
+                const float4 f = *reinterpret_cast<const float4 *>(&sh->ref[q][c]);
+                v[c] = fmaf(__uint_as_float(raw[c]), scale2, -f.x);
+                v[c + 1] = fmaf(__uint_as_float(raw[c + 1]), scale2, -f.y);
+                v[c + 2] = fmaf(__uint_as_float(raw[c + 2]), scale2, -f.z);
+                v[c + 3] = fmaf(__uint_as_float(raw[c + 3]), scale2, -f.w);
+                top = fmaxf(top, fmaxf(fmaxf(v[c], v[c + 1]), fmaxf(v[c + 2], v[c + 3])));
             }
-            if (__any_sync(0xffffffffu, grew)) {  // the same in all four warps: they look at the same numbers
+            if (lt_sync_or(tile == tile0 || (visible && top > LT_GROW))) {
 #pragma unroll
                 for (int g = 0; g < NG; ++g) {
-                    const float m = fmaxf(ref_c[g], m_new[g]);
+                    float w[GC];
+#pragma unroll
+                    for (int c = 0; c < GC; ++c) w[c] = visible ? __uint_as_float(raw[g * GC + c]) * scale2 : -INFINITY;
+                    const float m = lt_columns<GC, true>(w);
+                    if (lane < GC) sh->mx[q][g * GC + lane] = m;
+                }
+                lt_sync_and(true);
+#pragma unroll
+                for (int g = 0; g < NG; ++g) {
+                    const int c = g * GC + lane % GC;
+                    const float m = fmaxf(fmaxf(fmaxf(sh->mx[0][c], sh->mx[1][c]), fmaxf(sh->mx[2][c], sh->mx[3][c])), ref_c[g]);
                     if (lane < GC) {
-                        sh->ref[q][g * GC + lane] = m;
-                        sh->corr[q][g * GC + lane] = ref_c[g] == -INFINITY ? 0.f : exp2f(ref_c[g] - m);
+                        sh->ref[q][c] = m;
+                        sh->corr[q][c] = ref_c[g] == -INFINITY ? 0.f : exp2f(ref_c[g] - m);
                     }
                     ref_c[g] = m;
                 }
                 __syncwarp();
 #pragma unroll
-                for (int c = 0; c < N; ++c) l[c] *= sh->corr[q][c];
+                for (int c = 0; c < N; ++c) {
+                    l[c] *= sh->corr[q][c];
+                    v[c] = fmaf(__uint_as_float(raw[c]), scale2, -sh->ref[q][c]);
+                }
                 if (tile > tile0) {  // the scores' commit covers the earlier products: O^T is at rest
                     for (int p = 0; p < npiece; ++p)
 #pragma unroll
@@ -294,14 +352,18 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
                     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
                 }
             }
-            // probabilities: [head][position] rows of 64 positions, 128-byte swizzle
-            unsigned char *pd = Ps + (size_t)(pt >> 6) * (N * 128) + (pt & 7) * 2;
-            const int chunk = (pt & 63) >> 3;
 #pragma unroll
-            for (int c = 0; c < N; ++c) {
-                const bf16 pb = __float2bfloat16_rn(visible ? exp2f(v[c] - sh->ref[q][c]) : 0.f);
-                l[c] += __bfloat162float(pb);
-                *reinterpret_cast<bf16 *>(pd + c * 128 + ((chunk ^ (c & 7)) << 4)) = pb;
+            for (int j = 0; j < N / 8; ++j) {
+                uint32_t w[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int c = 8 * j + 2 * i;
+                    w[i] = visible ? Act<bf16>::pack(lt_exp2(v[c]), lt_exp2(v[c + 1])) : 0u;
+                    const float2 f = Act<bf16>::to_f2(w[i]);
+                    l[c] += f.x;
+                    l[c + 1] += f.y;
+                }
+                *reinterpret_cast<uint4 *>(Ps + lt_p_off<N>(pt, j)) = make_uint4(w[0], w[1], w[2], w[3]);
             }
             __syncwarp();  // every lane has read this tile's references before the next tile may replace them
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -327,17 +389,18 @@ latent_tc_kernel(const LatentAttnArgs a, const __grid_constant__ CUtensorMap map
                 reinterpret_cast<float2 *>(a.part_ml)[(size_t)(row0 + c0) * a.splits + sp] = make_float2(sh->ref[q][c0], s);
                 if (sp == 0) a.part_n[row0 + c0] = my_splits;
             }
-            for (int p = 0; p < npiece; ++p)
+            for (int p = 0; p < npiece; ++p) {
+                uint32_t o[N];
 #pragma unroll
-                for (int c = 0; c < N; c += 16) {
-                    uint32_t o[16];
-                    tc_ld16(tmem_o + lanes + p * N + c, o);
-                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (p * 128 + pt < R)
+                for (int c = 0; c < N; c += 16) tc_ld16(tmem_o + lanes + p * N + c, o + c);
+                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                if (p * 128 + pt < R) {
+                    float *dst = a.part_o + ((size_t)row0 * a.splits + sp) * R + p * 128 + pt;
 #pragma unroll
-                        for (int i = 0; i < 16; ++i)
-                            if (c + i < rows) a.part_o[((size_t)(row0 + c + i) * a.splits + sp) * R + p * 128 + pt] = __uint_as_float(o[i]);
+                    for (int c = 0; c < N; ++c)
+                        if (c < rows) __stcg(dst + (size_t)c * a.splits * R, __uint_as_float(o[c]));
                 }
+            }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         }
     }
