@@ -43,6 +43,7 @@ struct Tuning {
     int tc_block = 256;            // most tokens one tcgen05 launch takes (64, 128, 256): prefill rounds are cut into such blocks
     int tc_cluster = 1;            // cluster split-K form of the tcgen05 kernel: 0 never, 1 where it measured faster, 2 wherever it applies
     int stack_pdl = 1;             // layered models, small rounds: every launch is a programmatic dependent of its predecessor
+    int stack_fuse = 1;            // layered models, rounds of one or two decoded tokens: norms and residual as GEMV prologues (1: where it measured faster, 2: always)
     int latent_tc = 1;             // latent attention of decode rounds on tcgen05 (0: mma.sync kernel)
     int expand_min = 0;            // latent attention: fewest tokens of a portion that expands keys and values (0: by operation count, -1: never)
     int p2p_scatter_ranks = 8;     // ranks from which the peer all-reduce takes the reduce-scatter + all-gather form

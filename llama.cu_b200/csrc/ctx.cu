@@ -588,6 +588,7 @@ int lcu_set_tuning(lcu_ctx *c, const char *key, long long value) {
     else if (k == "tc_block") { LCU_REQUIRE(value == 64 || value == 128 || value == 256, "set_tuning: tc_block = %lld (64, 128, 256)", value); t.tc_block = (int)value; }
     else if (k == "tc_cluster") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: tc_cluster = %lld (0..2)", value); t.tc_cluster = (int)value; }
     else if (k == "stack_pdl") t.stack_pdl = value != 0;
+    else if (k == "stack_fuse") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_fuse = %lld (0..2)", value); t.stack_fuse = (int)value; }
     else if (k == "latent_tc") t.latent_tc = value != 0;
     else if (k == "expand_min") t.expand_min = (int)value;
     else if (k == "p2p_scatter_ranks") t.p2p_scatter_ranks = (int)value;

@@ -50,8 +50,13 @@ __device__ __forceinline__ void vec8_to_f32(const uint4 &v, float f[8]) {
     f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
 }
 
+__device__ __forceinline__ void gemv_cp16(float *smem_dst, const float *src) {
+    unsigned d = (unsigned)__cvta_generic_to_shared(smem_dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+
 // PRO: 0 = activations staged as they are, 1 = RMSNorm (any token count, f32 or 16-bit norm weights), 2 = RMSNorm of one
-// token from registers
+// token from registers, 3 / 4 = PRO_LATENT / PRO_RESIDUAL
 // STK: the epilogues of layered models instead of the LLaMA ones
 template <class T, bool Q8, int NT, int KI, int RP, int PRO, bool STK>
 __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(const GemvArgs a, int KS, int RS, int n_pairs) {
@@ -137,6 +142,16 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
             nwv[j] = i < nv8 ? __ldg(reinterpret_cast<const uint4 *>(a.norm_w) + i) : make_uint4(0, 0, 0, 0);
         }
     }
+    // prologues of layered models stage their f32 rows behind the partial sums; the shift state is that of an earlier round
+    [[maybe_unused]] float *stage = part + (size_t)2 * 16 * R * NT;
+    if constexpr (PRO == PRO_RESIDUAL) {
+        if (a.pro.shift)
+            for (int t = 0; t < NT && t < a.n_tok; ++t) {
+                const int sg = a.pro.req_slot[t];
+                const float *st = a.pro.state + (size_t)(sg & 1) * a.pro.state_gen_stride + (size_t)(sg >> 1) * a.in;
+                for (int i = threadIdx.x; i < a.in / 4; i += blockDim.x) gemv_cp16(stage + (size_t)(3 * t + 2) * a.in + 4 * i, st + 4 * i);
+            }
+    }
     if (a.pdl_trigger == 0) grid_dep_launch();
     grid_dep_wait();
     if (a.early_prefetch == 0 && n_groups > 0) load_group(0);
@@ -181,6 +196,103 @@ __global__ void __launch_bounds__(512, (NT == 1 && !Q8) ? 2 : 1) gemv_kernel(con
             }
         }
         __syncthreads();
+    } else if constexpr (PRO == PRO_RESIDUAL || PRO == PRO_LATENT) {
+        // every thread handles the 4-column pieces it copied itself, so its own wait is all it needs
+        constexpr int ROWS = PRO == PRO_RESIDUAL ? 3 : 1;
+        const int n4 = a.in / 4;
+        for (int t = 0; t < NT && t < a.n_tok; ++t)
+            for (int i = threadIdx.x; i < n4; i += blockDim.x) {
+                float *d = stage + (size_t)(ROWS * t) * a.in + 4 * i;
+                if constexpr (PRO == PRO_RESIDUAL) {
+                    gemv_cp16(d, a.pro.y_in + (size_t)t * a.in + 4 * i);
+                    gemv_cp16(d + a.in, a.pro.x_in + (size_t)t * a.in + 4 * i);
+                } else {
+                    gemv_cp16(d, a.pro.lat + (size_t)t * a.pro.lat_stride + 4 * i);
+                }
+            }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (x_first && n_groups > 0) load_group(0);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            float ss = 0.f;
+            if (t < a.n_tok)
+                for (int i = threadIdx.x; i < n4; i += blockDim.x) {
+                    const float4 f = *reinterpret_cast<const float4 *>(stage + (size_t)(ROWS * t) * a.in + 4 * i);
+                    ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+                }
+            ss = warp_sum(ss);
+            if (lane == 0) part[t * 16 + warp] = ss;
+        }
+        __syncthreads();
+        float rms[NT];
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            float v = 0.f;
+            for (int w = 0; w < nwarps; ++w) v += part[t * 16 + w];
+            rms[t] = 1.f / sqrtf(v / (float)a.pro.n_true + a.eps);
+        }
+        auto put4 = [&](int t, int i, const float4 &v) {
+            *reinterpret_cast<uint2 *>(xs + (size_t)t * a.in + 4 * i) = make_uint2(Act<T>::pack(v.x, v.y), Act<T>::pack(v.z, v.w));
+        };
+        for (int t = 0; t < NT; ++t) {
+            if (t >= a.n_tok) {
+                for (int i = threadIdx.x; i < n4; i += blockDim.x) put4(t, i, make_float4(0.f, 0.f, 0.f, 0.f));
+                continue;
+            }
+            const float *row = stage + (size_t)(ROWS * t) * a.in;
+            const float r = rms[t];
+            if constexpr (PRO == PRO_LATENT) {
+                for (int i = threadIdx.x; i < n4; i += blockDim.x) {
+                    const float4 f = *reinterpret_cast<const float4 *>(row + 4 * i);
+                    const uint2 u = __ldg(reinterpret_cast<const uint2 *>(a.pro.q_norm) + i);
+                    const float2 g0 = Act<T>::to_f2(u.x), g1 = Act<T>::to_f2(u.y);
+                    put4(t, i, make_float4(f.x * r * g0.x, f.y * r * g0.y, f.z * r * g1.x, f.w * r * g1.y));
+                }
+            } else {
+                const bool shifted = a.pro.shift != nullptr;
+                float *st = nullptr;
+                bool first = false;
+                if (shifted) {
+                    const int sg = a.pro.req_slot[t];
+                    first = a.pro.req_pos[t] == 0;
+                    if (blockIdx.x == 0) st = a.pro.state + (size_t)((sg & 1) ^ 1) * a.pro.state_gen_stride + (size_t)(sg >> 1) * a.in;
+                }
+                for (int i = threadIdx.x; i < n4; i += blockDim.x) {
+                    const float4 y = *reinterpret_cast<const float4 *>(row + 4 * i);
+                    float4 v = *reinterpret_cast<const float4 *>(row + a.in + 4 * i);
+                    const float4 g = a.pro.gain_stride ? *reinterpret_cast<const float4 *>(a.pro.gain + 4 * i)
+                                                       : make_float4(a.pro.gain[0], a.pro.gain[0], a.pro.gain[0], a.pro.gain[0]);
+                    v.x += y.x * r * g.x; v.y += y.y * r * g.y; v.z += y.z * r * g.z; v.w += y.w * r * g.w;
+                    if (blockIdx.x == 0) *reinterpret_cast<float4 *>(a.pro.x_out + (size_t)t * a.in + 4 * i) = v;
+                    if (shifted) {
+                        if (st) *reinterpret_cast<float4 *>(st + 4 * i) = v;
+                        const float4 p = first ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4 *>(row + 2 * a.in + 4 * i);
+                        const uint2 u = __ldg(reinterpret_cast<const uint2 *>(a.pro.shift) + i);
+                        const float2 m0 = Act<T>::to_f2(u.x), m1 = Act<T>::to_f2(u.y);
+                        v.x += (p.x - v.x) * m0.x; v.y += (p.y - v.y) * m0.y; v.z += (p.z - v.z) * m1.x; v.w += (p.w - v.w) * m1.y;
+                    }
+                    put4(t, i, v);
+                }
+            }
+        }
+        __syncthreads();
+        if constexpr (PRO == PRO_LATENT) {
+            // the last CTA normalises the cached latent and appends it (a warp per token)
+            if (blockIdx.x == gridDim.x - 1 && warp < a.n_tok) {
+                const int t = warp;
+                const float *c = a.pro.lat + (size_t)t * a.pro.lat_stride + a.in;
+                float ss = 0.f;
+                for (int i = lane; i < a.pro.r_p; i += 32) ss += c[i] * c[i];
+                const float r = 1.f / sqrtf(warp_sum(ss) / (float)a.pro.kv_rank + a.eps);
+                const uint32_t p = a.pos[t];
+                const int page = a.page_table[(size_t)a.tok_seq[t] * a.pt_stride + (p >> a.pro.page_shift)];
+                T *dst = reinterpret_cast<T *>(a.pro.pool) + (size_t)page * a.pro.page_elems + a.pro.c_off +
+                         (size_t)(p & ((1u << a.pro.page_shift) - 1)) * a.pro.r_p;
+                for (int i = lane; i < a.pro.r_p; i += 32)
+                    dst[i] = Act<T>::from_f(c[i] * r * Act<T>::to_f(reinterpret_cast<const T *>(a.pro.kv_norm)[i]));
+            }
+        }
     } else {
         // ---- stage the activations (optionally RMS-normalised) in shared memory
         const T *xg = reinterpret_cast<const T *>(a.x);
@@ -418,6 +530,7 @@ static int launch_inst(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaS
     auto kernel = gemv_kernel<T, Q8, NT, KI, RP, PRO, STK>;
     // activations + double-buffered per-warp partial sums (also the RMSNorm scratch)
     size_t smem = (size_t)NT * a.in * sizeof(T) + (size_t)2 * 16 * (2 * RP * NT) * sizeof(float);
+    if (PRO == PRO_LATENT || PRO == PRO_RESIDUAL) smem += (size_t)NT * (PRO == PRO_RESIDUAL ? 3 : 1) * a.in * sizeof(float);  // f32 rows
     int block = pl.nwarps * 32;
 
     struct Info { int ctas_per_sm; };
@@ -463,12 +576,18 @@ static int launch_inst(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaS
 template <class T, bool Q8, int NT, bool STK>
 static int launch_nt(const GemvArgs &a, const GemvPlan &pl, int n_pairs, cudaStream_t s, bool pdl, bool dry) {
     // prologue variant: the one-token register form needs 16-bit norm weights and at most two vectors per thread
-    const int pro = a.prologue != PRO_RMSNORM ? 0 : ((NT == 1 && !a.norm_f32 && a.lean_norm && a.in / 8 <= 2 * pl.nwarps * 32) ? 2 : 1);
+    const int pro = a.prologue >= PRO_LATENT ? 3 : a.prologue != PRO_RMSNORM ? 0 : ((NT == 1 && !a.norm_f32 && a.lean_norm && a.in / 8 <= 2 * pl.nwarps * 32) ? 2 : 1);
 #define LCU_GEMV_CASE(KI_, RP_)                                                                                   \
     if (pl.KI == KI_ && pl.RP == RP_) {                                                                           \
         if (pro == 0) return launch_inst<T, Q8, NT, KI_, RP_, 0, STK>(a, pl, n_pairs, s, pdl, dry);               \
-        if constexpr (STK) return LCU_ERR_INVALID;                                                                \
-        else {                                                                                                    \
+        if constexpr (STK) {                                                                                      \
+            if constexpr (NT <= 2) {                                                                              \
+                if (a.prologue == PRO_LATENT) return launch_inst<T, Q8, NT, KI_, RP_, PRO_LATENT, STK>(a, pl, n_pairs, s, pdl, dry);     \
+                if (a.prologue == PRO_RESIDUAL) return launch_inst<T, Q8, NT, KI_, RP_, PRO_RESIDUAL, STK>(a, pl, n_pairs, s, pdl, dry); \
+            }                                                                                                     \
+            set_error("gemv: prologue %d with %d tokens", a.prologue, NT);                                        \
+            return LCU_ERR_INVALID;                                                                               \
+        } else {                                                                                                  \
         if (pro == 1) return launch_inst<T, Q8, NT, KI_, RP_, 1, STK>(a, pl, n_pairs, s, pdl, dry);                    \
         if constexpr (NT == 1) return launch_inst<T, Q8, NT, KI_, RP_, 2, STK>(a, pl, n_pairs, s, pdl, dry);      \
         }                                                                                                         \
@@ -517,7 +636,7 @@ int gemv_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry) {
         LCU_REQUIRE(a.out == a.qd + 2 * a.kvd && a.dh % 2 == 0, "gemv: rope/kv epilogue shape mismatch");
     GemvArgs b = a;
     b.lean_norm = tuning().gemv_lean_norm;
-    if (b.epilogue >= EPI_STORE_F32) {
+    if (b.epilogue >= EPI_STORE_F32 || b.prologue >= PRO_LATENT) {
         LCU_REQUIRE(dt == LCU_BF16 && !b.w_q8, "gemv: epilogue %d takes bf16 activations and weights", b.epilogue);
         return launch_t<__nv_bfloat16, false, true>(b, s, pdl, dry);
     }
@@ -536,6 +655,18 @@ namespace lcu {
 // Sets the shared-memory attribute and caches the occupancy of every kernel variant a
 // context with these shapes can launch, so that nothing of the kind happens inside a
 // stream capture.
+int gemv_warm_stack(int in, int out, int r_p, int epilogue, int prologue) {
+    for (int nt = 1; nt <= 2 && gemv_stack_fits(in, nt, prologue); ++nt) {
+        GemvArgs a{};
+        a.in = in; a.out = out; a.n_tok = nt; a.stride_x = in; a.epilogue = epilogue; a.prologue = prologue; a.pro.r_p = r_p;
+        int rc = gemv_launch(a, LCU_BF16, nullptr, false, true);
+        if (rc) return rc;
+    }
+    return LCU_OK;
+}
+bool gemv_stack_fits(int in, int n_tok, int prologue) {
+    return n_tok <= 2 && (size_t)n_tok * in * (2 + (prologue == PRO_RESIDUAL ? 12 : 4)) + 16384 <= (size_t)227 * 1024;
+}
 int gemv_warm(int in, int out, bool q8, int dt, int epilogue) {
     for (int nt = 1; nt <= gemv_max_tokens(in); nt *= 2) {
         GemvArgs a{};

@@ -6,10 +6,32 @@
 
 namespace lcu {
 
-enum GemvPrologue { PRO_NONE = 0, PRO_RMSNORM = 1 };
+enum GemvPrologue { PRO_NONE = 0, PRO_RMSNORM = 1,
+                    PRO_LATENT = 3,    // layered models: the query latent's norm; one CTA also appends the cached latent
+                    PRO_RESIDUAL = 4 }; // layered models: norm of the previous sublayer's output, residual, token shift
 enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU = 3,
                     EPI_STORE_F32 = 4,  // y is f32
                     EPI_XIELU = 5 };    // y = xielu(row) with the two numbers at act_pq
+
+// Inputs of the prologues of layered models, for rounds of one token per request (token t is request t).  Every CTA computes
+// the rows it multiplies; what later kernels need (new residual, shift state, cached latent) is written by the first CTA.
+struct StackPrologue {
+    const float *x_in, *y_in;  // PRO_RESIDUAL: x = x_in + gain * y_in / rms(y_in), f32 [n_tok, in]
+    float *x_out;
+    const float *gain;
+    int gain_stride;
+    int n_true;                // coordinates the mean of squares runs over (PRO_LATENT: of the query latent)
+    const void *shift;         // bf16 token-shift weights, or nullptr
+    float *state;              // f32 [2][slots][in] of this layer, rows (generation, slot)
+    size_t state_gen_stride;
+    const int32_t *req_pos, *req_slot;
+    const float *lat;          // PRO_LATENT: [n_tok, lat_stride] query latent (in columns) | latent (r_p columns)
+    int lat_stride, kv_rank, r_p;
+    const void *q_norm, *kv_norm;
+    void *pool;
+    size_t page_elems, c_off;
+    int page_shift;
+};
 
 struct GemvArgs {
     // weights [out, in] row-major in the activation dtype, or Q8_0 planes
@@ -52,6 +74,7 @@ struct GemvArgs {
     int lean_norm;       // one token: RMSNorm prologue from registers (norm weights fetched before the wait)
     // tensor parallelism: EPI_STORE / EPI_RESIDUAL outputs go to every rank's all-reduce slot instead of y
     P2pPush push;
+    StackPrologue pro;
 };
 
 #ifdef __CUDACC__
@@ -160,7 +183,9 @@ __device__ void gemv_epilogue(const GemvArgs &a, int pair, int t, float va, floa
 template <class T>
 __device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int t, float va, float vb) {
     const size_t off = (size_t)t * a.stride_y + (size_t)pair * 2;
-    if (a.epilogue == EPI_STORE_F32) {
+    if (a.epilogue == EPI_STORE) {
+        *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(va, vb);
+    } else if (a.epilogue == EPI_STORE_F32) {
         *reinterpret_cast<float2 *>(reinterpret_cast<float *>(a.y) + off) = make_float2(va, vb);
     } else {
         const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
@@ -173,6 +198,9 @@ __device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int 
 int gemv_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry = false);
 // Prepares (attributes, occupancy) every variant used for this shape without launching.
 int gemv_warm(int in, int out, bool q8, int dt, int epilogue = EPI_STORE);
+// The same for the prologues of layered models (one and two tokens).
+bool gemv_stack_fits(int in, int n_tok, int prologue);
+int gemv_warm_stack(int in, int out, int r_p, int epilogue, int prologue);
 // Batched form for up to 64 tokens per launch (gemm_skinny.cu): same arguments and epilogues, but the
 // activations must be prepared (no RMSNorm prologue, no row gather).
 bool gemm_skinny_supported(int in, int w_q8);

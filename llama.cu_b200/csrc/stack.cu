@@ -162,6 +162,9 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
         }
         if (!rc) rc = gemv_warm(S->d_p, L.in_rows(), false, c->dt, EPI_STORE_F32);
         if (!rc) rc = gemv_warm(L.qr_p, L.d.heads * L.dim_p, false, c->dt);
+        if (!rc) rc = gemv_warm_stack(S->d_p, L.in_rows(), 0, EPI_STORE_F32, PRO_RESIDUAL);
+        if (!rc) rc = gemv_warm_stack(L.qr_p, L.d.heads * L.dim_p, L.r_p, EPI_STORE, PRO_LATENT);
+        if (!rc && L.d.ff) rc = gemv_warm_stack(S->d_p, L.ff_p, 0, EPI_XIELU, PRO_RESIDUAL);
         if (!rc) rc = gemv_warm(L.hv_p, S->d_p, false, c->dt, EPI_STORE_F32);
         if (!rc && L.d.ff) rc = gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_XIELU);
         if (!rc && L.d.ff) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
@@ -299,7 +302,8 @@ struct Launcher {
     bool pdl;
 
     // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
-    int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr) {
+    int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr,
+               int prologue = PRO_NONE, const GemvArgs *pro = nullptr) {
         if (c->dt == LCU_F32) {
             LinearF32Args a{};
             a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w;
@@ -323,6 +327,10 @@ struct Launcher {
             a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
             a.stride_y = stride_y;
             // a dependent launch requests its first weights ahead of the wait for its predecessor
+            if (pro) {  // one launch (at most two tokens): the prologue's rows, and the tokens' places in the cache
+                a.pro = pro->pro; a.pos = pro->pos; a.tok_seq = pro->tok_seq; a.page_table = pro->page_table; a.pt_stride = pro->pt_stride;
+                a.eps = pro->eps; a.prologue = prologue;
+            }
             a.pdl_trigger = pdl ? 0 : 2;
             a.early_prefetch = pdl ? 3 : 1;
             int rc = tc ? gemm_tc_launch(a, c->dt, s, pdl) : gemv_launch(a, c->dt, s, pdl);
@@ -357,6 +365,14 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
     mi.state_gen_stride = (size_t)d.n_layers * S.n_slots * S.d_p;
     mi.tok_req = tok_req; mi.req_first = i32(o.req_first); mi.req_pos = i32(o.req_pos); mi.req_slot = i32(o.req_slot);
     mi.h = S.h;
+    // rounds of one or two decoded tokens: norms, residual and token shift run as prologues of the projections that read them,
+    // up to the width where the rows every CTA then re-reads cost more than the launches saved (batch 1, 8 layers: width 2048
+    // 0.423 -> 0.408 ms per step, width 4096 0.812 -> 0.821 ms)
+    bool fused = (tuning().stack_fuse == 2 || (tuning().stack_fuse == 1 && S.d_p <= 2048)) && dt == LCU_BF16 && r.decode_only && gemv_stack_fits(S.d_p, n, PRO_RESIDUAL);
+    for (const StackLayer &Y : S.layers) fused = fused && gemv_stack_fits(Y.qr_p, n, PRO_LATENT);
+    GemvArgs pend{};  // the prologue the next projection of x takes (fused rounds)
+    bool pending = false;
+    pend.pos = pos; pend.tok_seq = tok_req; pend.page_table = page_table; pend.pt_stride = c->pt_stride; pend.eps = d.eps;
     // x (and the shifted input of layer `next`, if there is one) after a sublayer's output y; layer -1: the embedding
     auto residual = [&](const float *gain, int next, bool mixer_input) -> int {
         MixInputArgs a = mi;
@@ -374,8 +390,22 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
                 a.state = S.state + (size_t)next * S.n_slots * S.d_p;
             }
         }
+        if (fused && gain && a.h) {
+            StackPrologue &p = pend.pro;
+            p = StackPrologue{};
+            p.x_in = a.x_in; p.y_in = a.y; p.x_out = a.x_out; p.gain = gain; p.n_true = d.d; p.shift = a.shift; p.state = a.state;
+            p.state_gen_stride = a.state_gen_stride; p.req_pos = a.req_pos; p.req_slot = a.req_slot;
+            pending = true;
+            return LCU_OK;
+        }
         ++*count;
         return op_mix_input(a, dt, s, pdl);
+    };
+    // projection of the residual stream (or its shifted form), through the pending prologue if there is one
+    auto project = [&](const void *w, int out, void *y, int epilogue, const float *act_pq) -> int {
+        const bool p = pending;
+        pending = false;
+        return L.linear(w, S.d_p, out, S.h, n, y, out, epilogue, act_pq, p ? PRO_RESIDUAL : PRO_NONE, p ? &pend : nullptr);
     };
     rc = residual(nullptr, 0, true);
     if (rc) return rc;
@@ -384,17 +414,26 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
         const StackWeights &W = S.w[Y.src];
         const int heads = Y.d.heads, lat_stride = Y.in_rows(), q_stride = heads * Y.dim_p;
         // --- both latents and the head gates in one projection; norms; append to the cache; queries
-        rc = L.linear(W.in, S.d_p, Y.in_rows(), S.h, n, S.lat, lat_stride, EPI_STORE_F32);
+        rc = project(W.in, lat_stride, S.lat, EPI_STORE_F32, nullptr);
         if (rc) return rc;
         LatentNormArgs ln{};
         ln.lat = S.lat; ln.stride = lat_stride; ln.n_tok = n; ln.q_rank = Y.d.q_rank; ln.qr_p = Y.qr_p; ln.kv_rank = Y.d.kv_rank; ln.r_p = Y.r_p;
         ln.q_norm = W.q_norm; ln.kv_norm = W.kv_norm; ln.eps = d.eps; ln.cq = S.cq;
         ln.pool = c->pool; ln.page_elems = c->geom.page_elems; ln.c_off = Y.c_off; ln.page_shift = c->geom.page_shift;
         ln.tok_req = tok_req; ln.pos = pos; ln.page_table = page_table; ln.pt_stride = c->pt_stride;
-        rc = latent_norm_launch(ln, dt, s, pdl);
-        if (rc) return rc;
-        ++*count;
-        rc = L.linear(W.uq, Y.qr_p, q_stride, S.cq, n, S.q, q_stride, EPI_STORE);
+        if (fused) {
+            GemvArgs g = pend;
+            g.pro = StackPrologue{};
+            g.pro.lat = S.lat; g.pro.lat_stride = lat_stride; g.pro.n_true = Y.d.q_rank; g.pro.kv_rank = Y.d.kv_rank; g.pro.r_p = Y.r_p;
+            g.pro.q_norm = W.q_norm; g.pro.kv_norm = W.kv_norm; g.pro.pool = c->pool; g.pro.page_elems = c->geom.page_elems;
+            g.pro.c_off = Y.c_off; g.pro.page_shift = c->geom.page_shift;
+            rc = L.linear(W.uq, Y.qr_p, q_stride, S.cq, n, S.q, q_stride, EPI_STORE, nullptr, PRO_LATENT, &g);
+        } else {
+            rc = latent_norm_launch(ln, dt, s, pdl);
+            if (rc) return rc;
+            ++*count;
+            rc = L.linear(W.uq, Y.qr_p, q_stride, S.cq, n, S.q, q_stride, EPI_STORE);
+        }
         if (rc) return rc;
         const float *gate = Y.d.out_gate ? S.lat + Y.qr_p + Y.r_p : nullptr;
         const unsigned char *uv = reinterpret_cast<const unsigned char *>(W.ukv) + (size_t)heads * Y.dim_p * Y.r_p * 2;
@@ -462,7 +501,7 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
             continue;
         }
         // --- feed-forward
-        rc = L.linear(W.up, S.d_p, Y.ff_p, S.h, n, S.act, Y.ff_p, EPI_XIELU, W.scalars + 2);
+        rc = project(W.up, Y.ff_p, S.act, EPI_XIELU, W.scalars + 2);
         if (!rc) rc = L.linear(W.down, Y.ff_p, S.d_p, S.act, n, S.y, S.d_p, EPI_STORE_F32);
         if (!rc) rc = residual(W.scalars + 1, l + 1, true);
         if (rc) return rc;

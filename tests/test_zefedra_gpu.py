@@ -20,7 +20,7 @@ BF16, F32 = 1, 2
 @pytest.fixture(autouse=True)
 def default_tuning(L):
     yield
-    for k, v in (("expand_min", 0), ("stack_pdl", 1), ("tc_block", 256)):
+    for k, v in (("expand_min", 0), ("stack_pdl", 1), ("stack_fuse", 1), ("latent_tc", 1), ("tc_block", 256)):
         L.set_tuning(k, v)
 
 
@@ -175,6 +175,24 @@ def test_slots_and_pages_carry_nothing_over(L, dt):
     for i, n in enumerate((128, 1, 2, 127, 3, 65, 1)):
         toks = M.random_tokens(raw, n, 60 + i)
         check(r.whole(toks, [[n], [1, 2], [5]][i % 3]), M.reference(raw, w, toks), dt, f"request {i} of {n} tokens")
+    ctx.close()
+
+
+@pytest.mark.parametrize("key", ["latent_tc", "stack_fuse", "stack_pdl", "tc_block"])
+def test_every_form_of_a_decode_round(L, key):
+    """The alternatives behind the tuning keys compute the same: two requests decode together, then one alone."""
+    raw = M.config([M.layer(True, heads=20, dim=32, vdim=16, q_rank=48, kv_rank=128, ff=64), M.layer(heads=3)])
+    w = M.weights(raw, 65)
+    a, b = M.random_tokens(raw, 290, 66), M.random_tokens(raw, 150, 67)
+    want = {"a": M.reference(raw, w, a), "b": M.reference(raw, w, b)}
+    _, ctx = M.load(L, raw, w, BF16)
+    L.set_tuning(key, 64 if key == "tc_block" else 0, ctx)
+    r = M.Runner(ctx)
+    r.step([("a", a[:200]), ("b", b[:120])])
+    for i in range(90):
+        r.step([("a", a[200 + i:201 + i])] + ([("b", b[120 + i:121 + i])] if i < 30 else []))
+    for k in want:
+        check(r.logits(k), want[k], BF16, k)
     ctx.close()
 
 
