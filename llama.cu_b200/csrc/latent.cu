@@ -77,12 +77,13 @@ int latent_norm_launch(const LatentNormArgs &a, int dt, cudaStream_t s, bool pdl
 // Weight rows on M (16 per warp), tokens on N.  The whole K range of both operands is requested up front, the weights ahead of the
 // dependency wait.  Without `x` the activations are the merged attention partials:
 // sum over splits of 2^(m_s - M) o_s (running maxima are kept in powers of two), divided by the merged sum.
-constexpr int HL_THREADS = 128;
+constexpr int HL_THREADS = 256, HL_WARPS = 8;
 constexpr int HL_MAX_SPLITS = 64;
 
 template <int NT>
 __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinearArgs a) {
     constexpr int NF = NT / 8, YLD = 64 + 8;
+    constexpr int NFW = NF == 1 ? 1 : NF / 2;  // 8-token tiles per warp: four warps over the rows, twice over the tokens
     extern __shared__ __align__(16) unsigned char smem[];
     const int ld = a.in + 8;
     bf16 *Ws = reinterpret_cast<bf16 *>(smem);   // [64][in + 8]
@@ -96,7 +97,7 @@ __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinea
     const int ch = a.in / 8;
     // rows are dealt to lane groups of the chunk count's next power of two, so no lane computes a division per chunk
     const int lpr = ch >= 32 ? 32 : (ch > 16 ? 32 : (ch > 8 ? 16 : (ch > 4 ? 8 : (ch > 2 ? 4 : 2)))), rpw = 32 / lpr;
-    const int lr = warp * rpw + lane / lpr, lc = lane % lpr, rstep = 4 * rpw;
+    const int lr = warp * rpw + lane / lpr, lc = lane % lpr, rstep = HL_WARPS * rpw;
     for (int r = lr; r < 64; r += rstep)  // weights do not depend on the previous kernel
         for (int c = lc; c < ch; c += lpr) la_cp_async_16(Ws + (size_t)r * ld + c * 8, w + (r < no ? (size_t)r * a.in + c * 8 : 0), r < no);
     la_commit();
@@ -110,27 +111,26 @@ __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinea
         la_commit();
     } else {
         // a warp per row: lane s holds split s's weight 2^(m_s - M) / sum (two splits per lane)
-        for (int r = warp; r < NT; r += HL_THREADS / 32) {
-            const size_t row = (size_t)(n0 + r) * a.heads + h;
+        for (int r = warp; r < NT; r += HL_WARPS) {
+            const size_t row = (size_t)(n0 + (r < nt ? r : 0)) * a.heads + h;
+            const float2 *ml = reinterpret_cast<const float2 *>(a.part_ml) + row * a.splits;
+            // (max, sum) of every split the grid has, requested together with the number in use
+            float2 e0 = lane < a.splits ? ml[lane] : make_float2(-INFINITY, 0.f);
+            float2 e1 = lane + 32 < a.splits ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
             const int ns = r < nt ? a.part_n[row] : 0;
-            float w0 = 0.f, w1 = 0.f;
-            if (ns) {
-                const float2 *ml = reinterpret_cast<const float2 *>(a.part_ml) + row * a.splits;
-                const float2 e0 = lane < ns ? ml[lane] : make_float2(-INFINITY, 0.f);
-                const float2 e1 = lane + 32 < ns ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
-                const float M = warp_max(fmaxf(e0.x, e1.x));
-                w0 = e0.x == -INFINITY ? 0.f : exp2f(e0.x - M);
-                w1 = e1.x == -INFINITY ? 0.f : exp2f(e1.x - M);
-                const float inv = 1.f / warp_sum(w0 * e0.y + w1 * e1.y);
-                w0 *= inv;
-                w1 *= inv;
-            }
+            if (lane >= ns) e0 = make_float2(-INFINITY, 0.f);
+            if (lane + 32 >= ns) e1 = make_float2(-INFINITY, 0.f);
+            const float M = warp_max(fmaxf(e0.x, e1.x));
+            float w0 = e0.x == -INFINITY ? 0.f : exp2f(e0.x - M), w1 = e1.x == -INFINITY ? 0.f : exp2f(e1.x - M);
+            const float inv = ns ? 1.f / warp_sum(w0 * e0.y + w1 * e1.y) : 0.f;
+            w0 *= inv;
+            w1 *= inv;
             const int c = lane * 4;  // up to four 4-column pieces of the row per lane (a row holds at most 512)
             float4 v[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
             const float *src = a.part_o + row * a.splits * a.in + c;
-#pragma unroll 2
+#pragma unroll 4
             for (int s2 = 0; s2 < ns; ++s2, src += a.in) {
                 const float f = __shfl_sync(0xffffffffu, s2 < 32 ? w0 : w1, s2 & 31);
 #pragma unroll
@@ -148,41 +148,46 @@ __global__ void __launch_bounds__(HL_THREADS) head_linear_kernel(const HeadLinea
     }
     la_wait<0>();
     __syncthreads();
-    float acc[NF][4];
+    const int wm = warp & 3, wn = NF == 1 ? 0 : warp >> 2;
+    if (NF > 1 || warp < 4) {
+        float acc[NFW][4];
 #pragma unroll
-    for (int i = 0; i < NF; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    const bf16 *wrow = Ws + (size_t)(warp * 16 + (lane & 15)) * ld + (lane >> 4) * 8;
+        for (int i = 0; i < NFW; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+        const bf16 *wrow = Ws + (size_t)(wm * 16 + (lane & 15)) * ld + (lane >> 4) * 8;
+        const bf16 *xrow = Xs + (size_t)(wn * NFW * 8) * ld;
 #pragma unroll 4
-    for (int k = 0; k < a.in; k += 16) {
-        uint32_t af[4];
-        la_ldsm4(af, wrow + k);
-        if constexpr (NF == 1) {
-            uint32_t b[2];
-            la_ldsm2(b, Xs + (size_t)(lane & 7) * ld + k + ((lane >> 3) & 1) * 8);
-            mma16816<bf16>(acc[0], af[0], af[1], af[2], af[3], b[0], b[1]);
-        } else {
+        for (int k = 0; k < a.in; k += 16) {
+            uint32_t af[4];
+            la_ldsm4(af, wrow + k);
+            if constexpr (NFW == 1) {
+                uint32_t b[2];
+                la_ldsm2(b, xrow + (size_t)(lane & 7) * ld + k + ((lane >> 3) & 1) * 8);
+                mma16816<bf16>(acc[0], af[0], af[1], af[2], af[3], b[0], b[1]);
+            } else {
 #pragma unroll
-            for (int np = 0; np < NF / 2; ++np) {
-                uint32_t b[4];
-                la_ldsm4(b, Xs + (size_t)(np * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * ld + k + ((lane >> 3) & 1) * 8);
-                mma16816<bf16>(acc[2 * np], af[0], af[1], af[2], af[3], b[0], b[1]);
-                mma16816<bf16>(acc[2 * np + 1], af[0], af[1], af[2], af[3], b[2], b[3]);
+                for (int np = 0; np < NFW / 2; ++np) {
+                    uint32_t b[4];
+                    la_ldsm4(b, xrow + (size_t)(np * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * ld + k + ((lane >> 3) & 1) * 8);
+                    mma16816<bf16>(acc[2 * np], af[0], af[1], af[2], af[3], b[0], b[1]);
+                    mma16816<bf16>(acc[2 * np + 1], af[0], af[1], af[2], af[3], b[2], b[3]);
+                }
             }
         }
+#pragma unroll
+        for (int f = 0; f < NFW; ++f)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int nl = (wn * NFW + f) * 8 + 2 * t4 + c;
+                bf16 *d = Ys + nl * YLD + wm * 16 + gid;
+                float g = 1.f;
+                if (a.gate && nl < nt) {
+                    const int n = n0 + nl;
+                    g = 1.f / (1.f + expf(-a.gate[(size_t)(a.y_rows ? a.y_rows[n] : n) * a.stride_gate + h]));
+                }
+                d[0] = __float2bfloat16_rn(acc[f][c] * g);
+                d[8] = __float2bfloat16_rn(acc[f][c + 2] * g);
+            }
     }
-#pragma unroll
-    for (int f = 0; f < NF; ++f)
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            bf16 *d = Ys + (f * 8 + 2 * t4 + c) * YLD + warp * 16 + gid;
-            float g = 1.f;
-            if (a.gate && f * 8 + 2 * t4 + c < nt) {
-                const int n = n0 + f * 8 + 2 * t4 + c;
-                g = 1.f / (1.f + expf(-a.gate[(size_t)(a.y_rows ? a.y_rows[n] : n) * a.stride_gate + h]));
-            }
-            d[0] = __float2bfloat16_rn(acc[f][c] * g);
-            d[8] = __float2bfloat16_rn(acc[f][c + 2] * g);
-        }
     __syncthreads();
     bf16 *y = reinterpret_cast<bf16 *>(a.y) + (size_t)h * a.head_y + o0;
     for (int i = tid; i < nt * 8; i += HL_THREADS) {
