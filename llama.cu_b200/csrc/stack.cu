@@ -370,7 +370,7 @@ int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
     mi.h = S.h;
     // rounds of one or two decoded tokens: norms, residual and token shift run as prologues of the projections that read them,
     // up to the width where the rows every CTA then re-reads cost more than the launches saved (batch 1, 8 layers: width 2048
-    // 0.423 -> 0.408 ms per step, width 4096 0.812 -> 0.821 ms)
+    // 0.410 -> 0.409 ms per step with 23 launches less, width 4096 0.773 -> 0.793 ms)
     bool fused = (tuning().stack_fuse == 2 || (tuning().stack_fuse == 1 && S.d_p <= 2048)) && dt == LCU_BF16 && r.decode_only && gemv_stack_fits(S.d_p, n, PRO_RESIDUAL);
     for (const StackLayer &Y : S.layers) fused = fused && gemv_stack_fits(Y.qr_p, n, PRO_LATENT);
     L.weights_first = !fused;
