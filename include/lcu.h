@@ -58,7 +58,8 @@ typedef enum {
     LCU_W_OUT_NORM = 7,  /* output_norm         [d]                         */
     LCU_W_LM_HEAD = 8,   /* output.weight       [vocab, d]                  */
     /* Models described layer by layer (lcu_ctx_create_layers); packed shapes from lcu_layer_weight_shape.  All bf16
-     * except LCU_W_SCALARS; EMBD, OUT_NORM (one f32 gain) and LM_HEAD are shared with the kinds above. */
+     * except LCU_W_SCALARS; EMBD, OUT_NORM (f32: one gain, or one per coordinate in pre-norm models) and LM_HEAD are shared
+     * with the kinds above. */
     LCU_W_LAT_IN = 16,   /* rows: query latent | latent | head gates        */
     LCU_W_Q_NORM = 17,   /* norm weight of the query latent                 */
     LCU_W_KV_NORM = 18,  /* norm weight of the latent                       */
@@ -69,7 +70,19 @@ typedef enum {
     LCU_W_UP = 23,       /* feed-forward up                                 */
     LCU_W_FF_DOWN = 24,  /* feed-forward down                               */
     LCU_W_SHIFT = 25,    /* token-shift weights                             */
-    LCU_W_SCALARS = 26   /* f32: mixer norm gain, feed-forward norm gain, activation p, q */
+    LCU_W_SCALARS = 26,  /* f32: mixer norm gain, feed-forward norm gain, activation p, q */
+    /* pre-norm layers, softmax attention and delta-rule mixers; f32 unless it is a matrix */
+    LCU_W_MIX_IN = 27,      /* rows: attention q | k | v, delta q | k | v | output gate | step size | decay */
+    LCU_W_MIX_BIAS = 28,    /* biases of the attention's q | k | v                      */
+    LCU_W_ATT_OUT = 29,     /* attention output projection, [heads][v_dim] columns      */
+    LCU_W_DELTA_OUT = 30,   /* delta-rule output projection, [heads][v_dim] columns     */
+    LCU_W_CONV = 31,        /* short convolutions of the delta rule's q | k | v: [taps][channels] */
+    LCU_W_DELTA_DECAY = 32, /* [2][heads]: logarithm of the decay rate, bias of the step */
+    LCU_W_DELTA_NORM = 33,  /* norm weight of a delta-rule head's output                */
+    LCU_W_BRANCH_NORM = 34, /* [2][d]: gains on the two mixers' outputs                 */
+    LCU_W_NORM1 = 35,       /* gain of the norm ahead of the mixer                      */
+    LCU_W_NORM2 = 36,       /* gain of the norm ahead of the feed-forward               */
+    LCU_W_STEP = 37         /* vector added to the residual stream ahead of the layer   */
 } lcu_weight_kind;
 
 /* Model description: the fields llama.cu/src/model/mod.rs:61-78 reads from GGUF metadata.
@@ -87,22 +100,41 @@ typedef struct {
 } lcu_model_desc;
 
 /* Mixers and activations of layered models */
-enum { LCU_MIX_LATENT = 1 };  /* latent attention: per-head keys and values are linear maps of one cached vector per token */
-enum { LCU_ACT_XIELU = 1 };
+enum {
+    LCU_MIX_LATENT = 1,    /* latent attention: per-head keys and values are linear maps of one cached vector per token */
+    LCU_MIX_ATTENTION = 2, /* softmax attention over cached keys and values, grouped heads, rotary positions            */
+    LCU_MIX_DELTA = 4      /* gated delta rule: one state matrix per head and sequence                                  */
+}; /* ATTENTION | DELTA: both read the same input, their outputs are RMS-normed with a gain each and added */
+enum { LCU_ACT_XIELU = 1, LCU_ACT_RELU2 = 2 };
 
-/* One layer of a model described layer by layer: x += norm(mixer(h)), x += norm(ff(x)), both norms RMS with a single gain
- * on the sublayer's OUTPUT, h = x or (token_shift) x mixed per coordinate with the previous token's x.  (No counterpart in
- * the reference, whose models are LLaMA-shaped.) */
+/* One layer of a model described layer by layer.  Post-norm: x += norm(mixer(h)), x += norm(ff(x)), both norms RMS with a
+ * single gain on the sublayer's OUTPUT, h = x or (token_shift) x mixed per coordinate with the previous token's x.
+ * Pre-norm: x += mixer(norm(x)), x += ff(norm(x)), a gain per coordinate.  The layers of a model are all of one form.
+ * (No counterpart in the reference, whose models are LLaMA-shaped.) */
 typedef struct {
-    int32_t mixer;       /* LCU_MIX_LATENT                                                      */
-    int32_t heads, dim, v_dim; /* query/key and value size per head                             */
-    int32_t q_rank, kv_rank;   /* query latent, cached latent                                   */
-    int32_t out_gate;    /* 1: head h's output is multiplied by sigmoid(W_g h)_h                 */
+    int32_t mixer;       /* LCU_MIX_*                                                           */
+    int32_t heads, dim, v_dim; /* latent or softmax attention: query heads, query/key and value size per head */
+    int32_t q_rank, kv_rank;   /* LATENT: query latent, cached latent                            */
+    int32_t out_gate;    /* LATENT: 1: head h's output is multiplied by sigmoid(W_g h)_h         */
     int32_t token_shift; /* 1: the mixer reads h + (previous h - h) * shift (recurrent state)    */
     int32_t ff;          /* feed-forward width, 0: the layer has none                            */
-    int32_t ff_act;      /* LCU_ACT_XIELU                                                        */
+    int32_t ff_act;      /* LCU_ACT_*                                                            */
     int32_t weights_of;  /* -1, or the layer whose tensors this one uses (own cache and state)   */
     float scale;         /* of the attention scores                                              */
+    int32_t pre_norm;    /* norm placement, see above                                            */
+    int32_t add_embed;   /* PRE-NORM: the embedding row is added to x ahead of this layer        */
+    int32_t add_step;    /* PRE-NORM: LCU_W_STEP of this layer is added to x ahead of it (never shared) */
+    /* ATTENTION */
+    int32_t kv_heads;    /* key/value heads; query head h reads head h / (heads / kv_heads)      */
+    int32_t bias;        /* 1: biases on q, k and v                                              */
+    int32_t qk_norm;     /* 1: q and k are divided by their root mean square after the rotation  */
+    int32_t rot_dims;    /* rotated dimensions of a head (pairs i, i + rot_dims / 2), 0: none    */
+    /* DELTA */
+    int32_t delta_heads, delta_kv_heads, delta_dim, delta_v_dim;
+    int32_t delta_conv;  /* taps of the short convolutions                                       */
+    /* ATTENTION: frequencies base^(-2i / rot_dims); rot_factor > 0: YaRN, frequencies of fewer than rot_slow turns in
+     * rot_original positions divided by the factor, those of more than rot_fast left, a ramp between */
+    double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
 } lcu_layer_desc;
 
 /* == `KVPair` (llama.cu/src/op/random_sample/mod.rs:29-36) == cub::KeyValuePair<int,half> */
@@ -141,8 +173,8 @@ LCU_API int lcu_ctx_create(const lcu_model_desc *desc, int device, int tp_rank, 
 LCU_API int lcu_ctx_destroy(lcu_ctx *ctx);
 /* A context for a model described layer by layer: desc gives n_layers, d, vocab, nctx, eps, act_dtype (LCU_BF16, or LCU_F32:
  * every operation in true 32-bit arithmetic), weight_dtype (LCU_BF16), page_tokens, max_tokens, max_seqs; its other fields are
- * ignored.  Pages hold page_tokens latents of every layer; sequences of models with token shift also take one of max_seqs
- * recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
+ * ignored.  Pages hold page_tokens latents, or keys and values, of every layer; sequences of models with token shift or a delta
+ * rule also take one of max_seqs recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
  * graphs, round builder, sampling).  One GPU.  (No counterpart in the reference.) */
 LCU_API int lcu_ctx_create_layers(const lcu_model_desc *desc, const lcu_layer_desc *layers, int device, lcu_ctx **out);
 /* Packed (zero-padded) shape of one weight of a layered context; layer is ignored for EMBD, OUT_NORM and LM_HEAD.

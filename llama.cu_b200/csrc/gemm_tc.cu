@@ -117,6 +117,10 @@ __device__ __forceinline__ void tc_finish(const GemvArgs &a, int n, int first, f
 #pragma unroll
         for (int i = 0; i < 8; ++i) v[i] = xielu_act(v[i], sp, sq);
     }
+    if (a.epilogue == EPI_RELU2) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = relu2_act(v[i]);
+    }
     uint4 o;
     o.x = Act<T>::pack(v[0], v[1]); o.y = Act<T>::pack(v[2], v[3]); o.z = Act<T>::pack(v[4], v[5]); o.w = Act<T>::pack(v[6], v[7]);
     if (a.push.n && (a.epilogue == EPI_STORE || a.epilogue == EPI_RESIDUAL)) {

@@ -11,7 +11,8 @@ enum GemvPrologue { PRO_NONE = 0, PRO_RMSNORM = 1,
                     PRO_RESIDUAL = 4 }; // layered models: norm of the previous sublayer's output, residual, token shift
 enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU = 3,
                     EPI_STORE_F32 = 4,  // y is f32
-                    EPI_XIELU = 5 };    // y = xielu(row) with the two numbers at act_pq
+                    EPI_XIELU = 5,      // y = xielu(row) with the two numbers at act_pq
+                    EPI_RELU2 = 6 };    // y = max(row, 0)^2
 
 // Inputs of the prologues of layered models, for rounds of one token per request (token t is request t).  Every CTA computes
 // the rows it multiplies; what later kernels need (new residual, shift state, cached latent) is written by the first CTA.
@@ -88,6 +89,8 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 __device__ __forceinline__ float xielu_act(float z, float sp, float sq) {
     return z > 0.f ? fmaf(sp * z, z, 0.5f * z) : fmaf(0.5f + sq, expm1f(z) - z, 0.5f * z);
 }
+
+__device__ __forceinline__ float relu2_act(float z) { return z > 0.f ? z * z : 0.f; }
 
 // Values an epilogue would otherwise fetch from global memory behind the weight stream: the per-token constants of the
 // RoPE / KV-append epilogue (position, cache page, sin and cos rows; head sizes up to 128), staged in shared memory
@@ -187,6 +190,8 @@ __device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int 
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(va, vb);
     } else if (a.epilogue == EPI_STORE_F32) {
         *reinterpret_cast<float2 *>(reinterpret_cast<float *>(a.y) + off) = make_float2(va, vb);
+    } else if (a.epilogue == EPI_RELU2) {
+        *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(relu2_act(va), relu2_act(vb));
     } else {
         const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(xielu_act(va, sp, sq), xielu_act(vb, sp, sq));

@@ -48,6 +48,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Args a) 
             if (o >= a.out) continue;
             float v = acc[i][j];
             if (a.epilogue == EPI_XIELU) v = xielu_act(v, softplus_f(a.act_pq[0]), softplus_f(a.act_pq[1]));
+            else if (a.epilogue == EPI_RELU2) v = relu2_act(v);
             a.y[yr * a.stride_y + (size_t)head * a.head_y + o] = a.gate ? v * g : v;
         }
     }
@@ -55,7 +56,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Args a) 
 
 int linear_f32_launch(const LinearF32Args &a, cudaStream_t s) {
     if (a.n <= 0) return LCU_OK;
-    LCU_REQUIRE(a.epilogue == EPI_STORE_F32 || (a.epilogue == EPI_XIELU && a.act_pq), "linear_f32: epilogue %d", a.epilogue);
+    LCU_REQUIRE(a.epilogue == EPI_STORE_F32 || a.epilogue == EPI_RELU2 || (a.epilogue == EPI_XIELU && a.act_pq), "linear_f32: epilogue %d", a.epilogue);
     dim3 grid((a.out + 63) / 64, (a.n + 63) / 64, a.heads);
     LCU_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "linear_f32: grid out of range");
     LCU_CHECK_CUDA(launch_kernel(linear_f32_kernel, grid, dim3(256), 0, s, false, a));

@@ -1,0 +1,88 @@
+// Mixers of pre-norm layers: softmax attention over cached keys and values (gqa.cu) and the gated delta rule (delta.cu).
+// Both read f32 rows of one fused input projection and write operands of their output projections.  Interface only.
+#pragma once
+#include "common.cuh"
+
+namespace lcu {
+
+constexpr int MIX_MAX_HEAD = 256;  // largest head size of either mixer
+
+// ---- softmax attention, grouped heads, rotary positions
+struct GqaArgs {
+    // rows of the fused projection: q heads | k heads | v heads, every head padded to dim_p / vdim_p
+    const float *lat;
+    int stride, n_tok;
+    int heads, kv_heads, dim, dim_p, v_dim, vdim_p;
+    const float *bias;          // [q | k | v] or nullptr
+    int qk_norm;                // q and k divided by their root mean square after the rotation
+    float eps;
+    int rot_dims;               // pairs (i, i + rot_dims / 2)
+    const float2 *rot;          // [positions][rot_dims / 2] (cos, sin), the frequency scaling's factor included
+    void *q;                    // [n_tok][heads * dim_p]
+    // pages: this layer's keys [kv head][slot][dim_p] at c_off, its values [kv head][slot][vdim_p] behind them
+    void *pool;
+    size_t page_elems, c_off;
+    int page_shift;
+    const int32_t *tok_req, *page_table;
+    const uint32_t *pos;
+    int pt_stride;
+    // attention
+    void *o;                    // [n_tok][stride_o], heads x vdim_p
+    int stride_o;
+    float scale;
+    const int4 *reqs;           // (request of the round, first token, tokens, position of the first token)
+    int n_reqs, max_len;        // longest of them in tokens
+    int n_blocks;               // long form: blocks of 64 (token, head) rows of all requests
+    // short form: contexts cut into splits, merged by the last CTA to arrive
+    int splits;
+    float *part_o, *part_ml;    // [request][kv head x row tile][split][16][vdim_p], [...][16][2]
+    unsigned *tickets;          // [request][kv head x row tile], zero between launches
+    __host__ __device__ size_t v_off() const { return c_off + ((size_t)kv_heads * dim_p << page_shift); }
+    __host__ __device__ int group() const { return heads / kv_heads; }
+};
+// Biases, rotation, norms; queries to q, keys and values to the cache.
+int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl);
+// A portion takes the short form up to this many tokens.
+int gqa_short_tokens(int heads, int kv_heads);
+int gqa_row_tiles(int heads, int kv_heads, int len);   // 16-row tiles of a request's short form, per key/value head
+size_t gqa_part_floats(int ctas, int vdim_p);          // scratch of `ctas` CTAs of the short form (part_o and part_ml)
+int gqa_short_ctas_per_sm(int dim_p, int vdim_p);
+int gqa_short_launch(const GqaArgs &a, cudaStream_t s, bool pdl, bool dry = false);
+int gqa_long_launch(const GqaArgs &a, cudaStream_t s, bool dry = false);
+int gqa_f32_launch(const GqaArgs &a, cudaStream_t s);
+
+// ---- gated delta rule
+struct DeltaArgs {
+    // rows of the fused projection: q heads | k heads (dk_p) | v heads | output gate (dv_p) | step size | decay (heads_p)
+    const float *lat;
+    int stride, n_tok, n_req;
+    int heads, kv_heads, dk, dk_p, dv, dv_p, heads_p, taps;
+    float eps;
+    const float *conv;          // [taps][channels]
+    const float *decay;         // [2][heads_p]: logarithm of the rate, bias
+    const float *norm;          // [dv_p]
+    // state: inputs of the convolutions [generation][slot][taps - 1][channels], matrices [slot][head][dv_p][dk_p]
+    float *conv_state;
+    size_t conv_gen_stride;
+    float *state;
+    const int32_t *tok_req, *req_first, *req_pos, *req_slot;
+    // between the kernels of a round with several tokens per request
+    float *q, *k;               // [n_tok][kv_heads * dk_p], unit vectors, q scaled
+    float *v;                   // [n_tok][heads * dv_p]; the scan overwrites it with its outputs
+    float4 *gate;               // [n_tok][heads]: decay, step size, q . k
+    void *o;                    // [n_tok][stride_o], heads x dv_p
+    int stride_o;
+    __host__ __device__ int channels() const { return 2 * kv_heads * dk_p + heads * dv_p; }
+    __host__ __device__ int g_off() const { return channels(); }
+    __host__ __device__ int b_off() const { return channels() + heads * dv_p; }
+    __host__ __device__ int a_off() const { return b_off() + heads_p; }
+    __host__ __device__ int rows() const { return a_off() + heads_p; }
+};
+// Rounds with several tokens per request: convolutions and gates; the recurrence; norm and output gate.
+int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
+int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
+int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
+// Rounds of one token per request: all of it in one launch, beside the attention's preparation (nullptr: none).
+int delta_decode_launch(const DeltaArgs &a, const GqaArgs *attn, int dt, cudaStream_t s, bool pdl);
+
+}  // namespace lcu

@@ -1,34 +1,13 @@
 // Rounds of models described layer by layer: shapes and storage, the plan of a round's attention, and the launches of every
 // layer.  Context, pages, descriptor staging, graphs and sampling are those of ctx.cu.
-#include "ctx.cuh"
-#include "gemv.cuh"
-#include "stack.cuh"
+#include "stack_round.cuh"
+
+#include <cmath>
 
 namespace lcu {
 
 static size_t align256(size_t v) { return (v + 255) & ~(size_t)255; }
-static size_t act_bytes(const lcu_ctx *c) { return c->dt == LCU_F32 ? 4 : 2; }
 
-// offsets inside the stack section of the round descriptor
-struct StackDesc {
-    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, total;
-};
-constexpr int EXPAND_GROUP = 64;  // query tokens per group of the expanded attention
-static StackDesc stack_desc(int n_tok, int n_req) {
-    StackDesc d;
-    size_t o = 0;
-    auto take = [&](size_t bytes) { size_t r = o; o += (bytes + 15) & ~(size_t)15; return r; };
-    d.req_first = take((size_t)(n_req + 1) * 4);
-    d.req_pos = take((size_t)n_req * 4);
-    d.req_slot = take((size_t)n_req * 4);
-    d.abs_first = take((size_t)(n_req + 1) * 4);
-    d.abs_id = take((size_t)n_req * 4);
-    d.abs_tok = take((size_t)n_tok * 4);
-    d.xreq = take((size_t)n_req * 16);
-    d.xgroups = take((size_t)(n_tok / EXPAND_GROUP + n_req) * 16);
-    d.total = o;
-    return d;
-}
 size_t stack_desc_bytes(int max_tok, int max_req) { return stack_desc(max_tok, max_req).total; }
 
 // Fewest tokens of a portion for which expanding pays: per cached token and head the absorbed form multiplies 2 r_p
@@ -61,11 +40,73 @@ static int attn_splits_for(const lcu_ctx *c, int blocks) {
 
 static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, int i) {
     const lcu_layer_desc &l = layers[i];
-    LCU_REQUIRE(l.mixer == LCU_MIX_LATENT, "layer %d: unknown mixer %d", i, l.mixer);
-    LCU_REQUIRE(l.heads > 0 && l.dim > 0 && l.v_dim > 0 && l.q_rank > 0 && l.kv_rank > 0 && l.ff >= 0, "layer %d: non-positive size", i);
-    LCU_REQUIRE(l.kv_rank <= 512 && l.dim <= 512, "layer %d: latent of %d, head size %d (at most 512)", i, l.kv_rank, l.dim);
-    LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_XIELU, "layer %d: unknown activation %d", i, l.ff_act);
+    LCU_REQUIRE((l.pre_norm != 0) == (layers[0].pre_norm != 0), "layer %d: pre-norm and post-norm layers in one model", i);
+    if (!l.pre_norm) {
+        LCU_REQUIRE(l.mixer == LCU_MIX_LATENT, "layer %d: unknown mixer %d", i, l.mixer);
+        LCU_REQUIRE(l.heads > 0 && l.dim > 0 && l.v_dim > 0 && l.q_rank > 0 && l.kv_rank > 0 && l.ff >= 0, "layer %d: non-positive size", i);
+        LCU_REQUIRE(l.kv_rank <= 512 && l.dim <= 512, "layer %d: latent of %d, head size %d (at most 512)", i, l.kv_rank, l.dim);
+        LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_XIELU, "layer %d: unknown activation %d", i, l.ff_act);
+        LCU_REQUIRE(!l.add_embed && !l.add_step, "layer %d: additions to the residual stream need pre-norm layers", i);
+    } else {
+        const int most = MIX_MAX_HEAD;
+        LCU_REQUIRE(l.mixer > 0 && (l.mixer & ~(LCU_MIX_ATTENTION | LCU_MIX_DELTA)) == 0, "layer %d: unknown mixer %d", i, l.mixer);
+        LCU_REQUIRE(l.ff >= 0 && !l.token_shift, "layer %d: negative size, or a token shift", i);
+        if (l.mixer & LCU_MIX_ATTENTION) {
+            LCU_REQUIRE(l.heads > 0 && l.kv_heads > 0 && l.heads % l.kv_heads == 0, "layer %d: %d query heads, %d key heads", i, l.heads, l.kv_heads);
+            LCU_REQUIRE(l.dim > 0 && l.dim <= most && l.v_dim > 0 && l.v_dim <= most, "layer %d: head sizes %d / %d (1..%d)", i, l.dim, l.v_dim, most);
+            LCU_REQUIRE(l.rot_dims >= 0 && l.rot_dims % 2 == 0 && l.rot_dims <= l.dim && (l.rot_dims == 0 || l.rot_base > 0),
+                        "layer %d: %d rotated dimensions of %d, base %g", i, l.rot_dims, l.dim, l.rot_base);
+            LCU_REQUIRE(l.rot_dims == 0 || l.rot_factor <= 0 || (l.rot_original > 0 && l.rot_fast > 0 && l.rot_slow > 0 && l.rot_base != 1),
+                        "layer %d: frequency scaling by %g needs positive constants", i, l.rot_factor);
+        }
+        if (l.mixer & LCU_MIX_DELTA) {
+            LCU_REQUIRE(l.delta_heads > 0 && l.delta_kv_heads > 0 && l.delta_heads % l.delta_kv_heads == 0, "layer %d: %d value heads, %d key heads", i,
+                        l.delta_heads, l.delta_kv_heads);
+            LCU_REQUIRE(l.delta_dim > 0 && l.delta_dim <= most && l.delta_v_dim > 0 && l.delta_v_dim <= most, "layer %d: head sizes %d / %d (1..%d)", i,
+                        l.delta_dim, l.delta_v_dim, most);
+            LCU_REQUIRE(l.delta_conv >= 1 && l.delta_conv <= 64, "layer %d: convolution of %d taps (1..64)", i, l.delta_conv);
+        }
+        LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_RELU2, "layer %d: unknown activation %d", i, l.ff_act);
+    }
     LCU_REQUIRE(l.weights_of >= -1 && l.weights_of < d.n_layers && l.weights_of != i, "layer %d uses the weights of layer %d", i, l.weights_of);
+    return LCU_OK;
+}
+
+// Fewest split CTAs per SM that keep a decode round's copies in flight: two waves of what fits.
+static int gqa_target_ctas(const StackLayer &L) { return 2 * sm_count() * gqa_short_ctas_per_sm(L.dim_p, L.vdim_p); }
+int gqa_splits_for(const lcu_ctx *c, const StackLayer &L, int reqs, int len) {
+    const int ctas = reqs * L.d.kv_heads * gqa_row_tiles(L.d.heads, L.d.kv_heads, len), units = (c->desc.nctx + 63) / 64;
+    int z = ctas > 0 ? gqa_target_ctas(L) / ctas : 1;
+    if (z > 64) z = 64;
+    if (z > units) z = units;
+    return z < 1 ? 1 : z;
+}
+
+// (cos, sin) of every position and rotated pair, angles in f64; YaRN: frequencies of fewer than `slow` turns in `original`
+// positions are divided by the factor, those of more than `fast` stay, a linear ramp over the pair's index lies between, and
+// both functions are scaled by 0.1 ln(factor) + 1.
+static int make_rot_table(Stack *S, const lcu_layer_desc &l, int nctx, const float2 **out) {
+    const int half = l.rot_dims / 2;
+    std::vector<double> freq(half);
+    double gain = 1.0;
+    for (int i = 0; i < half; ++i) freq[i] = pow(l.rot_base, -2.0 * i / l.rot_dims);
+    if (l.rot_factor > 0) {
+        auto index_of = [&](double turns) { return l.rot_dims * log(l.rot_original / (2.0 * M_PI * turns)) / (2.0 * log(l.rot_base)); };
+        const double lo = fmax(floor(index_of(l.rot_fast)), 0.0), hi = fmin(ceil(index_of(l.rot_slow)), l.rot_dims - 1.0);
+        for (int i = 0; i < half; ++i) {
+            const double ramp = fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0);
+            freq[i] = freq[i] / l.rot_factor * ramp + freq[i] * (1.0 - ramp);
+        }
+        gain = 0.1 * log(l.rot_factor) + 1.0;
+    }
+    std::vector<float2> host((size_t)nctx * half);
+    for (int p = 0; p < nctx; ++p)
+        for (int i = 0; i < half; ++i) host[(size_t)p * half + i] = make_float2((float)(cos(p * freq[i]) * gain), (float)(sin(p * freq[i]) * gain));
+    float2 *dev = nullptr;
+    LCU_CHECK_CUDA(cudaMalloc(reinterpret_cast<void **>(&dev), host.size() * sizeof(float2)));
+    S->rot_tables.push_back(dev);
+    LCU_CHECK_CUDA(cudaMemcpy(dev, host.data(), host.size() * sizeof(float2), cudaMemcpyHostToDevice));
+    *out = dev;
     return LCU_OK;
 }
 
@@ -83,7 +124,10 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->w.resize(d.n_layers);
     size_t off = 0;
     int max_lat = 0, max_qr = 0, max_q = 0, max_hr = 0, max_hv = 64, max_ff = 64, max_kv = 0;
-    bool any_shift = false, can_expand = c->dt != LCU_F32;
+    int max_dk = 0, max_dv = 0, max_dh = 0, max_dhv = 0, max_vp = 0;
+    size_t conv_total = 0, mat_total = 0;  // f32 values of recurrent state per slot
+    S->pre_norm = layers[0].pre_norm != 0;
+    bool any_shift = false, any_delta = false, can_expand = c->dt != LCU_F32 && !S->pre_norm;
     for (int i = 0; i < d.n_layers; ++i) {
         StackLayer &L = S->layers[i];
         L.d = layers[i];
@@ -94,35 +138,75 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
         }
         const lcu_layer_desc &o = layers[L.src];
         LCU_REQUIRE(o.heads == L.d.heads && o.dim == L.d.dim && o.v_dim == L.d.v_dim && o.q_rank == L.d.q_rank && o.kv_rank == L.d.kv_rank &&
-                        o.out_gate == L.d.out_gate && o.ff == L.d.ff && o.token_shift == L.d.token_shift,
+                        o.out_gate == L.d.out_gate && o.ff == L.d.ff && o.token_shift == L.d.token_shift && o.mixer == L.d.mixer &&
+                        o.kv_heads == L.d.kv_heads && o.bias == L.d.bias && o.delta_heads == L.d.delta_heads &&
+                        o.delta_kv_heads == L.d.delta_kv_heads && o.delta_dim == L.d.delta_dim && o.delta_v_dim == L.d.delta_v_dim &&
+                        o.delta_conv == L.d.delta_conv,
                     "layer %d differs from layer %d whose weights it uses", i, L.src);
-        L.dim_p = stack_pad(L.d.dim, 16);
-        L.vdim_p = stack_pad(L.d.v_dim, 16);
-        L.qr_p = stack_pad(L.d.q_rank, 64);
-        L.r_p = stack_pad(L.d.kv_rank, 64);
-        L.g_p = L.d.out_gate ? stack_pad(L.d.heads, 8) : 0;
-        L.ff_p = stack_pad(L.d.ff, 64);
-        L.hv_p = stack_pad(L.d.heads * L.vdim_p, 64);
-        L.c_off = off;
-        off += (size_t)L.r_p * c->geom.page_tokens;
-        any_shift = any_shift || L.d.token_shift;
-        can_expand = can_expand && expanded_attn_supported(L.dim_p, L.vdim_p);
         auto up = [](int &m, int v) { if (v > m) m = v; };
-        up(max_lat, L.in_rows()); up(max_qr, L.qr_p); up(max_q, L.d.heads * L.dim_p); up(max_hr, L.d.heads * L.r_p);
-        up(max_hv, L.hv_p); up(max_ff, L.ff_p); up(max_kv, L.kv_cols()); up(S->max_heads, L.d.heads); up(S->max_r, L.r_p);
+        L.ff_p = stack_pad(L.d.ff, 64);
+        L.c_off = off;
+        up(max_ff, L.ff_p);
+        if (L.latent()) {
+            L.dim_p = stack_pad(L.d.dim, 16);
+            L.vdim_p = stack_pad(L.d.v_dim, 16);
+            L.qr_p = stack_pad(L.d.q_rank, 64);
+            L.r_p = stack_pad(L.d.kv_rank, 64);
+            L.g_p = L.d.out_gate ? stack_pad(L.d.heads, 8) : 0;
+            L.hv_p = stack_pad(L.d.heads * L.vdim_p, 64);
+            off += (size_t)L.r_p * c->geom.page_tokens;
+            any_shift = any_shift || L.d.token_shift;
+            can_expand = can_expand && expanded_attn_supported(L.dim_p, L.vdim_p);
+            up(max_hr, L.d.heads * L.r_p); up(max_kv, L.kv_cols()); up(S->max_heads, L.d.heads); up(S->max_r, L.r_p);
+            up(max_q, L.d.heads * L.dim_p);
+        }
+        if (L.attention()) {
+            L.dim_p = stack_pad(L.d.dim, 16);
+            L.vdim_p = stack_pad(L.d.v_dim, 16);
+            L.hv_p = stack_pad(L.d.heads * L.vdim_p, 64);
+            L.att_rows = (L.d.heads + L.d.kv_heads) * L.dim_p + L.d.kv_heads * L.vdim_p;
+            off += (size_t)L.d.kv_heads * (L.dim_p + L.vdim_p) * c->geom.page_tokens;
+            up(max_q, L.d.heads * L.dim_p); up(max_vp, L.vdim_p);
+            if (gqa_target_ctas(L) > S->gqa_ctas) S->gqa_ctas = gqa_target_ctas(L);
+            for (int j = 0; j < i && !L.rot; ++j) {  // layers with the same rotation share a table
+                const lcu_layer_desc &e = layers[j];
+                if (S->layers[j].rot && e.rot_dims == L.d.rot_dims && e.rot_base == L.d.rot_base && e.rot_factor == L.d.rot_factor &&
+                    e.rot_original == L.d.rot_original && e.rot_fast == L.d.rot_fast && e.rot_slow == L.d.rot_slow)
+                    L.rot = S->layers[j].rot;
+            }
+            if (L.d.rot_dims && !L.rot) {
+                int rc = make_rot_table(S, L.d, d.nctx, &L.rot);
+                if (rc) return rc;
+            }
+        }
+        if (L.delta()) {
+            L.dk_p = stack_pad(L.d.delta_dim, 32);
+            L.dv_p = stack_pad(L.d.delta_v_dim, 16);
+            L.dh_p = stack_pad(L.d.delta_heads, 8);
+            L.dhv_p = stack_pad(L.d.delta_heads * L.dv_p, 64);
+            L.conv_off = conv_total;
+            conv_total += (size_t)(L.d.delta_conv - 1) * L.conv_channels();
+            L.mat_off = mat_total;
+            mat_total += (size_t)L.d.delta_heads * L.dv_p * L.dk_p;
+            any_delta = true;
+            up(max_dk, L.d.delta_kv_heads * L.dk_p); up(max_dv, L.d.delta_heads * L.dv_p); up(max_dh, L.d.delta_heads); up(max_dhv, L.dhv_p);
+        }
+        up(max_lat, L.in_rows()); up(max_qr, L.qr_p); up(max_hv, L.hv_p);
     }
     c->geom.page_elems = off;
-    S->n_slots = any_shift ? c->max_seqs : 0;
+    if (off == 0) c->geom.page_elems = 8;  // nothing is cached per token: pages still count tokens
+    S->n_slots = any_shift || any_delta ? c->max_seqs : 0;
     c->free_slots.clear();
     for (int i = S->n_slots - 1; i >= 0; --i) c->free_slots.push_back(i);
 
     const size_t T = (size_t)c->max_tokens, eb = act_bytes(c);
     S->abs_cap = c->max_tokens;
+    S->conv_gen = conv_total * S->n_slots;
     S->expand_cap = can_expand ? stack_pad(d.nctx > c->max_tokens ? d.nctx : c->max_tokens, 64) : 0;
     // partial rows: a small round is split so that about one CTA per SM runs, a large one is not split
     size_t rows = 0;
     for (const StackLayer &L : S->layers)
-        for (int dec = 0; dec < 2; ++dec)
+        for (int dec = 0; dec < 2 && L.latent(); ++dec)
             for (int n = 1; n <= c->max_tokens; n = n < 64 ? n + 1 : (n == c->max_tokens ? n + 1 : (2 * n < c->max_tokens ? 2 * n : c->max_tokens))) {
                 const int rpb = latent_attn_rows_per_block(L.d.heads, dec != 0, c->dt, c->geom.page_tokens);
                 const int blocks = dec ? n * ((L.d.heads + rpb - 1) / rpb) : n * L.d.heads / rpb + 1;
@@ -134,11 +218,14 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     size_t total = 0;
     auto reserve = [&](size_t bytes) { size_t r = total; total += align256(bytes); return r; };
     const size_t o_x0 = reserve(T * S->d_p * 4), o_x1 = reserve(T * S->d_p * 4), o_y = reserve(T * S->d_p * 4), o_lat = reserve(T * max_lat * 4),
-                 o_state = reserve((size_t)2 * d.n_layers * S->n_slots * S->d_p * 4), o_h = reserve(T * S->d_p * eb), o_cq = reserve(T * max_qr * eb),
+                 o_state = reserve(any_shift ? (size_t)2 * d.n_layers * S->n_slots * S->d_p * 4 : 0), o_h = reserve(T * S->d_p * eb), o_cq = reserve(T * max_qr * eb),
                  o_q = reserve(T * max_q * eb), o_qa = reserve(T * max_hr * eb), o_att = reserve(T * max_hv * eb), o_act = reserve(T * max_ff * eb),
                  o_xc = reserve((size_t)S->expand_cap * S->max_r * eb), o_xkv = reserve((size_t)S->expand_cap * max_kv * eb),
                  o_hout = reserve((T > (size_t)c->max_seqs ? T : c->max_seqs) * S->d_p * eb), o_po = reserve(rows * S->max_r * 4),
-                 o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4);
+                 o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4), o_y2 = reserve(S->pre_norm ? T * S->d_p * 4 : 0),
+                 o_dq = reserve(T * max_dk * 4), o_dk = reserve(T * max_dk * 4), o_dv = reserve(T * max_dv * 4), o_dg = reserve(T * max_dh * 16),
+                 o_att2 = reserve(T * max_dhv * eb), o_conv = reserve(2 * S->conv_gen * 4), o_mat = reserve(mat_total * S->n_slots * 4),
+                 o_gp = reserve(gqa_part_floats(S->gqa_ctas, max_vp) * 4), o_gt = reserve((size_t)S->gqa_ctas * 4);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
     LCU_CHECK_CUDA(cudaMemset(S->arena, 0, total));  // pads of att (columns past the heads) stay zero from here on
     unsigned char *p = reinterpret_cast<unsigned char *>(S->arena);
@@ -148,7 +235,30 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->xc = p + o_xc; S->xkv = p + o_xkv; S->hout = p + o_hout;
     S->part_o = reinterpret_cast<float *>(p + o_po); S->part_ml = reinterpret_cast<float *>(p + o_pml); S->part_n = reinterpret_cast<int *>(p + o_pn);
 
+    S->y2 = reinterpret_cast<float *>(p + o_y2); S->dq = reinterpret_cast<float *>(p + o_dq); S->dk = reinterpret_cast<float *>(p + o_dk);
+    S->dv = reinterpret_cast<float *>(p + o_dv); S->dgate = reinterpret_cast<float4 *>(p + o_dg); S->att2 = p + o_att2;
+    S->conv_state = reinterpret_cast<float *>(p + o_conv); S->mat_state = reinterpret_cast<float *>(p + o_mat);
+    S->gqa_part = reinterpret_cast<float *>(p + o_gp); S->gqa_tickets = reinterpret_cast<unsigned *>(p + o_gt);
+
     // every kernel variant a round can launch
+    if (S->pre_norm) {
+        if (c->dt == LCU_F32) return LCU_OK;
+        int rc = gemm_tc_warm(c->dt);
+        for (const StackLayer &L : S->layers) {
+            GqaArgs g{};
+            g.dim_p = L.dim_p; g.vdim_p = L.vdim_p;
+            if (!rc && L.attention()) rc = gqa_short_launch(g, nullptr, false, true);
+            if (!rc && L.attention()) rc = gqa_long_launch(g, nullptr, true);
+            if (!rc) rc = gemv_warm(S->d_p, L.in_rows(), false, c->dt, EPI_STORE_F32);
+            if (!rc && L.attention()) rc = gemv_warm(L.hv_p, S->d_p, false, c->dt, EPI_STORE_F32);
+            if (!rc && L.delta()) rc = gemv_warm(L.dhv_p, S->d_p, false, c->dt, EPI_STORE_F32);
+            if (!rc && L.d.ff) rc = gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_RELU2);
+            if (!rc && L.d.ff) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
+        }
+        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt);
+        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, EPI_STORE_F32);
+        return rc;
+    }
     int rc = latent_attn_launch(LatentAttnArgs{}, c->dt, nullptr, false, true);
     if (rc || c->dt == LCU_F32) return rc;
     rc = head_linear_launch(HeadLinearArgs{}, nullptr, false, true);
@@ -177,6 +287,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
 void stack_destroy(lcu_ctx *c) {
     if (!c->stack) return;
     if (c->stack->arena) cudaFree(c->stack->arena);
+    for (float2 *t : c->stack->rot_tables) cudaFree(t);
     delete c->stack;
     c->stack = nullptr;
 }
@@ -189,11 +300,32 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
     switch (kind) {
     case LCU_W_EMBD: *rows = c->desc.vocab; *cols = S.d_p; return true;
     case LCU_W_LM_HEAD: *rows = S.vocab_p; *cols = S.d_p; return true;
-    case LCU_W_OUT_NORM: *rows = 1; *cols = 1; *elem_bytes = 4; return true;
+    case LCU_W_OUT_NORM: *rows = 1; *cols = S.pre_norm ? S.d_p : 1; *elem_bytes = 4; return true;
     default: break;
     }
-    if (layer < 0 || layer >= c->desc.n_layers || S.layers[layer].src != layer) return false;
+    if (layer < 0 || layer >= c->desc.n_layers) return false;
     const StackLayer &L = S.layers[layer];
+    auto f32 = [&](int r, int n, bool has) { *rows = r; *cols = n; *elem_bytes = 4; return has; };
+    if (kind == LCU_W_STEP) return f32(1, S.d_p, L.d.add_step != 0);
+    if (L.src != layer) return false;
+    switch (kind) {
+    case LCU_W_UP: *rows = L.ff_p; *cols = S.d_p; return L.d.ff > 0;
+    case LCU_W_FF_DOWN: *rows = S.d_p; *cols = L.ff_p; return L.d.ff > 0;
+    default: break;
+    }
+    if (S.pre_norm) switch (kind) {
+    case LCU_W_MIX_IN: *rows = L.in_rows(); *cols = S.d_p; return true;
+    case LCU_W_MIX_BIAS: return f32(1, L.att_rows, L.attention() && L.d.bias);
+    case LCU_W_ATT_OUT: *rows = S.d_p; *cols = L.hv_p; return L.attention();
+    case LCU_W_DELTA_OUT: *rows = S.d_p; *cols = L.dhv_p; return L.delta();
+    case LCU_W_CONV: return f32(L.d.delta_conv, L.conv_channels(), L.delta());
+    case LCU_W_DELTA_DECAY: return f32(2, L.dh_p, L.delta());
+    case LCU_W_DELTA_NORM: return f32(1, L.dv_p, L.delta());
+    case LCU_W_BRANCH_NORM: return f32(2, S.d_p, L.attention() && L.delta());
+    case LCU_W_NORM1: return f32(1, S.d_p, true);
+    case LCU_W_NORM2: return f32(1, S.d_p, L.d.ff > 0);
+    default: return false;
+    }
     switch (kind) {
     case LCU_W_LAT_IN: *rows = L.in_rows(); *cols = S.d_p; return true;
     case LCU_W_Q_NORM: *rows = 1; *cols = L.qr_p; return true;
@@ -202,8 +334,6 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
     case LCU_W_UKT: *rows = L.d.heads * L.r_p; *cols = L.dim_p; return true;
     case LCU_W_UKV: *rows = L.kv_cols(); *cols = L.r_p; return true;
     case LCU_W_LAT_OUT: *rows = S.d_p; *cols = L.hv_p; return true;
-    case LCU_W_UP: *rows = L.ff_p; *cols = S.d_p; return L.d.ff > 0;
-    case LCU_W_FF_DOWN: *rows = S.d_p; *cols = L.ff_p; return L.d.ff > 0;
     case LCU_W_SHIFT: *rows = 1; *cols = S.d_p; return L.d.token_shift != 0;
     case LCU_W_SCALARS: *rows = 1; *cols = 4; *elem_bytes = 4; return true;
     default: return false;
@@ -212,7 +342,19 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
 
 int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
     StackWeights &w = c->stack->w[layer];
+    const float *f = reinterpret_cast<const float *>(ptr);
     switch (kind) {
+    case LCU_W_MIX_IN: w.in = ptr; break;
+    case LCU_W_MIX_BIAS: w.bias = f; break;
+    case LCU_W_ATT_OUT: w.att_out = ptr; break;
+    case LCU_W_DELTA_OUT: w.delta_out = ptr; break;
+    case LCU_W_CONV: w.conv = f; break;
+    case LCU_W_DELTA_DECAY: w.decay = f; break;
+    case LCU_W_DELTA_NORM: w.delta_norm = f; break;
+    case LCU_W_BRANCH_NORM: w.branch_norm = f; break;
+    case LCU_W_NORM1: w.norm1 = f; break;
+    case LCU_W_NORM2: w.norm2 = f; break;
+    case LCU_W_STEP: w.step = f; break;
     case LCU_W_LAT_IN: w.in = ptr; break;
     case LCU_W_Q_NORM: w.q_norm = ptr; break;
     case LCU_W_KV_NORM: w.kv_norm = ptr; break;
@@ -232,11 +374,18 @@ int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
 bool stack_ready(const lcu_ctx *c) {
     const Stack &S = *c->stack;
     for (size_t i = 0; i < S.layers.size(); ++i) {
-        if (S.layers[i].src != (int)i) continue;
         const StackWeights &w = S.w[i];
-        const lcu_layer_desc &d = S.layers[i].d;
-        if (!w.in || !w.q_norm || !w.kv_norm || !w.uq || !w.ukt || !w.ukv || !w.out || !w.scalars || (d.ff && (!w.up || !w.down)) ||
-            (d.token_shift && !w.shift)) {
+        const StackLayer &L = S.layers[i];
+        const lcu_layer_desc &d = L.d;
+        bool ok = !d.add_step || w.step;
+        if (L.src == (int)i) {
+            ok = ok && w.in && (!d.ff || (w.up && w.down)) && (!d.token_shift || w.shift);
+            if (L.latent()) ok = ok && w.q_norm && w.kv_norm && w.uq && w.ukt && w.ukv && w.out && w.scalars;
+            if (L.attention()) ok = ok && w.att_out && (!d.bias || w.bias);
+            if (L.delta()) ok = ok && w.delta_out && w.conv && w.decay && w.delta_norm;
+            if (S.pre_norm) ok = ok && w.norm1 && (!d.ff || w.norm2) && (!(L.attention() && L.delta()) || w.branch_norm);
+        }
+        if (!ok) {
             set_error("step: weights of layer %zu missing", i);
             return false;
         }
@@ -256,6 +405,10 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
             *slot = reinterpret_cast<int32_t *>(B + D.req_slot), *afirst = reinterpret_cast<int32_t *>(B + D.abs_first),
             *aid = reinterpret_cast<int32_t *>(B + D.abs_id), *atok = reinterpret_cast<int32_t *>(B + D.abs_tok);
     int4 *xreq = reinterpret_cast<int4 *>(B + D.xreq), *xg = reinterpret_cast<int4 *>(B + D.xgroups);
+    int4 *sreq = reinterpret_cast<int4 *>(B + D.sreq), *lreq = reinterpret_cast<int4 *>(B + D.lreq);
+    int short_max = 1 << 30;  // one decision per request and round: the layer with the largest head groups decides
+    for (const StackLayer &L : S.layers)
+        if (L.attention()) { const int v = gqa_short_tokens(L.d.heads, L.d.kv_heads); if (v < short_max) short_max = v; }
     const int expand_min = S.expand_cap ? round_expand_min(S) : 1 << 30;
     int t = 0, nx = 0, ng = 0;
     StackRound::Batch cur{0, 0, 0, 0, 0};
@@ -265,7 +418,15 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
         first[i] = t;
         pos[i] = (int)reqs[i].pos;
         slot[i] = sq.slot * 2 + sq.gen;
-        if (len < expand_min) {
+        if (S.pre_norm) {
+            if (len <= short_max) {
+                sreq[q.n_short++] = make_int4(i, t, len, pos[i]);
+                if (len > q.max_short) q.max_short = len;
+            } else {
+                lreq[q.n_long++] = make_int4(i, t, len, pos[i]);
+                q.long_len.push_back(len);
+            }
+        } else if (len < expand_min) {
             aid[q.n_abs_req] = i;
             afirst[q.n_abs_req++] = q.n_abs_tok;
             for (int j = 0; j < len; ++j) atok[q.n_abs_tok++] = t + j;
@@ -293,62 +454,9 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
 
 bool stack_pdl(const lcu_ctx *c, int n_tok) { return tuning().stack_pdl && c->dt != LCU_F32 && n_tok <= 256; }
 
-namespace {
-
-struct Launcher {
-    lcu_ctx *c;
-    cudaStream_t s;
-    int *count;
-    bool pdl;
-    bool weights_first = false;  // one-token GEMVs of this round request weights before activations
-
-    // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
-    int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr,
-               int prologue = PRO_NONE, const GemvArgs *pro = nullptr) {
-        if (c->dt == LCU_F32) {
-            LinearF32Args a{};
-            a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w;
-            a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
-            a.n = n; a.in = in; a.out = out; a.heads = 1;
-            a.epilogue = epilogue == EPI_STORE ? EPI_STORE_F32 : epilogue;
-            a.act_pq = act_pq;
-            ++*count;
-            return linear_f32_launch(a, s);
-        }
-        const size_t yb = epilogue == EPI_STORE_F32 ? 4 : 2;
-        const bool tc = n > 4;
-        for (int t0 = 0; t0 < n;) {
-            const int most = tc ? (tuning().tc_block < 256 ? tuning().tc_block : GEMM_TC_MAX_TOKENS) : gemv_max_tokens(in);
-            const int nt = n - t0 < most ? n - t0 : most;
-            GemvArgs a{};
-            a.w = w;
-            a.x = reinterpret_cast<const unsigned char *>(x) + (size_t)t0 * in * 2;
-            a.stride_x = in; a.n_tok = nt; a.in = in; a.out = out;
-            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq;
-            a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
-            a.stride_y = stride_y;
-            if (pro) {  // one launch (at most two tokens): the prologue's rows, and the tokens' places in the cache
-                a.pro = pro->pro; a.pos = pro->pos; a.tok_seq = pro->tok_seq; a.page_table = pro->page_table; a.pt_stride = pro->pt_stride;
-                a.eps = pro->eps; a.prologue = prologue;
-            }
-            // Dependent launches.  The GEMV's CTAs fill every register file, so it releases its own dependents at its exit only
-            // (releasing them at entry: 0.79 -> 0.91 ms per 8-layer step of width 4096 at batch 1), and asks for weights ahead of
-            // the wait only where that measured faster (one token, no norm prologue: 0.79 -> 0.77 ms; two tokens 0.92 -> 0.94).
-            a.pdl_trigger = pdl && tc ? 0 : 2;
-            a.early_prefetch = pdl && weights_first && n == 1 ? 3 : 1;
-            int rc = tc ? gemm_tc_launch(a, c->dt, s, pdl) : gemv_launch(a, c->dt, s, pdl);
-            if (rc) return rc;
-            ++*count;
-            t0 += nt;
-        }
-        return LCU_OK;
-    }
-};
-
-}  // namespace
-
 int stack_layers(lcu_ctx *c, const Round &r, cudaStream_t s, int *count) {
     Stack &S = *c->stack;
+    if (S.pre_norm) return pre_norm_layers(c, r, s, count);
     const lcu_model_desc &d = c->desc;
     const int dt = c->dt, n = r.n_tok;
     const size_t eb = act_bytes(c);
@@ -520,7 +628,7 @@ int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, flo
     Stack &S = *c->stack;
     const bool pdl = stack_pdl(c, r.n_tok);
     int rc = op_scalar_norm_rows(S.hout, reinterpret_cast<const float *>(c->x), rows, n_rows, c->desc.d, S.d_p,
-                                 reinterpret_cast<const float *>(c->out_norm), 0, c->desc.eps, c->dt, s, pdl);
+                                 reinterpret_cast<const float *>(c->out_norm), S.pre_norm, c->desc.eps, c->dt, s, pdl);
     if (rc) return rc;
     ++*count;
     Launcher L{c, s, count, pdl};
@@ -528,17 +636,20 @@ int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, flo
     return L.linear(c->lm_head, S.d_p, S.vocab_p, S.hout, n_rows, y, S.vocab_p, out_f32 ? EPI_STORE_F32 : EPI_STORE);
 }
 
-// Algorithmic bytes of a round: the weights the round's forms of attention touch, the head, the cached latents read.
+// Algorithmic bytes of a round: the weights the round's forms of attention touch, the head, cached rows and state.
 double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_out) {
     const Stack &S = *c->stack;
     const double wb = 2.0, eb = (double)act_bytes(c);
     double bytes = n_out ? (double)S.vocab_p * S.d_p * wb : 0.0;
     for (const StackLayer &L : S.layers) {
         const lcu_layer_desc &d = L.d;
-        bytes += wb * ((double)L.in_rows() * S.d_p + (double)d.heads * L.dim_p * L.qr_p + (double)L.kv_cols() * L.r_p + (double)S.d_p * L.hv_p +
-                       2.0 * L.ff_p * S.d_p);
-        for (int i = 0; i < n_req; ++i)
-            for (uint32_t j = 0; j < reqs[i].len; ++j) bytes += (double)(reqs[i].pos + j + 1) * L.r_p * eb;
+        bytes += wb * ((double)L.in_rows() * S.d_p + 2.0 * L.ff_p * S.d_p + (double)S.d_p * (L.hv_p + L.dhv_p));
+        if (L.latent()) bytes += wb * ((double)d.heads * L.dim_p * L.qr_p + (double)L.kv_cols() * L.r_p);
+        const double row = L.latent() ? L.r_p : (L.attention() ? (double)d.kv_heads * (L.dim_p + L.vdim_p) : 0.0);
+        for (int i = 0; i < n_req; ++i) {
+            for (uint32_t j = 0; j < reqs[i].len; ++j) bytes += (double)(reqs[i].pos + j + 1) * row * eb;
+            if (L.delta()) bytes += 8.0 * d.delta_heads * L.dv_p * L.dk_p;  // matrices read and written
+        }
     }
     return bytes;
 }

@@ -1,6 +1,7 @@
 // Models described layer by layer (lcu_ctx_create_layers): per-layer shapes and weights, the part of a round that is
 // theirs, and the kernels their layers are made of.  Interface only; rounds are built in stack.cu, the mixer kernels
-// are in latent.cu, norms / residual / token shift in stack_ops.cu, the 32-bit linear layer in linear_f32.cu.
+// are in latent.cu, gqa.cu and delta.cu, norms / residual / token shift in stack_ops.cu, the 32-bit linear layer in
+// linear_f32.cu.
 //
 // Storage conventions: every dimension a matrix product sums over is padded with zeros to a multiple of 64 (per-head
 // query/key and value sizes to a multiple of 16), so each shape takes the tensor-core kernels; the pads stay zero through
@@ -10,6 +11,7 @@
 #include <vector>
 
 #include "common.cuh"
+#include "mixers.cuh"
 
 struct lcu_ctx;
 
@@ -23,7 +25,17 @@ struct StackLayer {
     size_t c_off;   // element offset of this layer's cached rows inside a page: [page_tokens][r_p]
     // padded sizes
     int dim_p, vdim_p, qr_p, r_p, g_p, ff_p, hv_p;
-    int in_rows() const { return qr_p + r_p + g_p; }    // rows of the fused input projection: query latent | latent | gate
+    // softmax attention and delta rule
+    int att_rows = 0;                     // rows of the fused input projection that are the attention's (the first ones)
+    int dk_p = 0, dv_p = 0, dh_p = 0, dhv_p = 0;
+    size_t conv_off = 0, mat_off = 0;     // f32 offsets of this layer's recurrent state in its arena section
+    const float2 *rot = nullptr;          // [nctx][rot_dims / 2] (cos, sin)
+    bool latent() const { return d.mixer == LCU_MIX_LATENT; }
+    bool attention() const { return (d.mixer & LCU_MIX_ATTENTION) != 0; }
+    bool delta() const { return (d.mixer & LCU_MIX_DELTA) != 0; }
+    int delta_rows() const { return delta() ? 2 * d.delta_kv_heads * dk_p + 2 * d.delta_heads * dv_p + 2 * dh_p : 0; }
+    int conv_channels() const { return 2 * d.delta_kv_heads * dk_p + d.delta_heads * dv_p; }
+    int in_rows() const { return latent() ? qr_p + r_p + g_p : att_rows + delta_rows(); }  // rows of the fused input projection: query latent | latent | gate, or attention | delta rule
     int kv_cols() const { return d.heads * (dim_p + vdim_p); }  // columns of the expanded keys and values
 };
 
@@ -31,6 +43,10 @@ struct StackWeights {
     const void *in = nullptr, *q_norm = nullptr, *kv_norm = nullptr, *uq = nullptr, *ukt = nullptr, *ukv = nullptr,
                *out = nullptr, *up = nullptr, *down = nullptr, *shift = nullptr;
     const float *scalars = nullptr;  // mixer norm gain, feed-forward norm gain, activation p, q
+    // pre-norm layers
+    const void *att_out = nullptr, *delta_out = nullptr;
+    const float *bias = nullptr, *conv = nullptr, *decay = nullptr, *delta_norm = nullptr, *branch_norm = nullptr, *norm1 = nullptr,
+                *norm2 = nullptr, *step = nullptr;
 };
 
 // What the host decides about a round: which requests run their attention in latent space ("absorbed") and which expand
@@ -40,6 +56,9 @@ struct StackRound {
     bool abs_decode = false;  // every absorbed request brings one token
     struct Batch { int n_rows, req0, n_req, group0, n_groups; };
     std::vector<Batch> batches;
+    // softmax attention: requests whose portion takes the short form, and those that take the long one
+    int n_short = 0, max_short = 0, n_long = 0;
+    std::vector<int> long_len;
 };
 
 struct Stack {
@@ -58,6 +77,15 @@ struct Stack {
     int abs_cap = 0;        // absorbed tokens a round may hold
     int expand_cap = 0;     // rows of the expansion buffer (0: never expand)
     int max_heads = 0, max_r = 0;
+    // pre-norm models
+    bool pre_norm = false;
+    float *y2 = nullptr, *dq = nullptr, *dk = nullptr, *dv = nullptr, *conv_state = nullptr, *mat_state = nullptr, *gqa_part = nullptr;
+    float4 *dgate = nullptr;
+    void *att2 = nullptr;
+    unsigned *gqa_tickets = nullptr;
+    size_t conv_gen = 0;    // f32 values of one generation of the convolutions' state
+    int gqa_ctas = 0;       // CTAs of split short-form attention the partial buffer holds
+    std::vector<float2 *> rot_tables;
 };
 
 // ---- stack.cu
@@ -99,6 +127,22 @@ struct MixInputArgs {
     const int32_t *tok_req, *req_first, *req_pos, *req_slot;  // request of a token; first token, position, slot * 2 + generation of a request
 };
 int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl);
+// Pre-norm layers: x_out = x_in + sum of the sublayer's outputs y (each y * y_gain / rms(y) when gains are given) + embedding row
+// + step, then h = gain * x_out / rms(x_out), rounded to the activation dtype; every input and h may be missing.
+struct PreNormArgs {
+    const float *x_in;
+    const float *y[2];
+    const float *y_gain;  // [2][d_p]
+    const void *embd;     // bf16 [vocab, d_p]
+    const uint32_t *tokens;
+    const float *step;
+    float *x_out;
+    void *h;
+    const float *gain;
+    float eps;
+    int n_tok, d, d_p;
+};
+int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl);
 // y = x[rows[i]] * gain / rms(x), rounded
 int op_scalar_norm_rows(void *y, const float *x, const uint32_t *rows, int n, int d, int d_p, const float *gain, int gain_stride, float eps,
                         int dt, cudaStream_t s, bool pdl);

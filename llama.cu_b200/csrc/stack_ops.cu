@@ -97,6 +97,86 @@ int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl) {
     return dt == LCU_F32 ? mix_input_t<float>(a, s, pdl) : mix_input_t<__nv_bfloat16>(a, s, pdl);
 }
 
+// One block per token: the residual step of pre-norm layers.
+template <class T, int MAXV>
+__global__ void pre_norm_kernel(const PreNormArgs a) {
+    grid_dep_launch();
+    const int t = blockIdx.x, n4 = a.d_p / 4;
+    __shared__ float2 part[32], part2[32];
+    const size_t row = (size_t)t * a.d_p;
+    const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;
+    grid_dep_wait();
+    float4 x[MAXV], y0[MAXV], y1[MAXV];
+    float s0 = 0.f, s1 = 0.f;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        x[j] = y0[j] = y1[j] = zero;
+        if (i >= n4) continue;
+        if (a.x_in) x[j] = *reinterpret_cast<const float4 *>(a.x_in + row + 4 * i);
+        if (a.y[0]) y0[j] = *reinterpret_cast<const float4 *>(a.y[0] + row + 4 * i);
+        if (a.y[1]) y1[j] = *reinterpret_cast<const float4 *>(a.y[1] + row + 4 * i);
+        s0 += dot4(y0[j]);
+        s1 += dot4(y1[j]);
+    }
+    if (a.y_gain) {
+        const float2 s = block_sum2(s0, s1, part);
+        s0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
+        s1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        float4 g0 = make_float4(1.f, 1.f, 1.f, 1.f), g1 = g0, v = x[j];
+        if (a.y_gain) {
+            g0 = *reinterpret_cast<const float4 *>(a.y_gain + 4 * i);
+            g1 = *reinterpret_cast<const float4 *>(a.y_gain + a.d_p + 4 * i);
+            g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
+            g1.x *= s1; g1.y *= s1; g1.z *= s1; g1.w *= s1;
+        }
+        v.x += y0[j].x * g0.x + y1[j].x * g1.x; v.y += y0[j].y * g0.y + y1[j].y * g1.y;
+        v.z += y0[j].z * g0.z + y1[j].z * g1.z; v.w += y0[j].w * g0.w + y1[j].w * g1.w;
+        if (a.embd) {
+            const float4 e = ld4_bf16(a.embd, e0 + 4 * i);
+            v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+        }
+        if (a.step) {
+            const float4 e = *reinterpret_cast<const float4 *>(a.step + 4 * i);
+            v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+        }
+        *reinterpret_cast<float4 *>(a.x_out + row + 4 * i) = v;
+        x[j] = v;
+        ss += dot4(v);
+    }
+    if (!a.h) return;
+    const float r = 1.f / sqrtf(block_sum2(ss, 0.f, part2).x / (float)a.d + a.eps);
+#pragma unroll
+    for (int j = 0; j < MAXV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        const float4 g = *reinterpret_cast<const float4 *>(a.gain + 4 * i), v = x[j];
+        st4<T>(reinterpret_cast<T *>(a.h) + row + 4 * i, make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w));
+    }
+}
+
+template <class T>
+static int pre_norm_t(const PreNormArgs &a, cudaStream_t s, bool pdl) {
+    const int n4 = a.d_p / 4;
+    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1>, dim3(a.n_tok), dim3(128), 0, s, pdl, a));
+    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2>, dim3(a.n_tok), dim3(512), 0, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4>, dim3(a.n_tok), dim3(1024), 0, s, pdl, a));
+    return LCU_OK;
+}
+
+int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl) {
+    if (a.n_tok <= 0) return LCU_OK;
+    LCU_REQUIRE(a.d_p % 4 == 0 && a.d_p <= 16384, "pre_norm: width %d (a multiple of 4, at most 16384)", a.d_p);
+    return dt == LCU_F32 ? pre_norm_t<float>(a, s, pdl) : pre_norm_t<__nv_bfloat16>(a, s, pdl);
+}
+
 template <class T>
 __global__ void __launch_bounds__(256) scalar_norm_rows_kernel(T *__restrict__ y, const float *__restrict__ x, const uint32_t *__restrict__ rows,
                                                                int d, int d_p, const float *__restrict__ gain, int gain_stride, float eps) {
