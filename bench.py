@@ -37,6 +37,8 @@ WORKLOADS = {
     "llama70b-tp8shard-f16-b64": ("llama70b_tp8shard", 64, (1024, 1024)),  # one rank's share, for profiling
     "zefedra8b-bf16-b1": ("zefedra8b", 1, (128, 128)),
     "zefedra8b-bf16-b32": ("zefedra8b", 32, (128, 1024)),
+    "galarax8b-bf16-b1": ("galarax8b", 1, (128, 128)),
+    "galarax8b-bf16-b32": ("galarax8b", 32, (128, 1024)),
     "tiny-f16-b1": ("tiny", 1, (16, 16)),
 }
 DEFAULT_WORKLOAD = "llama8b-f16-b1"
@@ -473,9 +475,9 @@ def run_decode(L, env, cfg, batch, prompt_range, steps, warmup, want_e2e=True, w
     return res
 
 
-# --family-bench: sizes at which a layered family runs beside the LLaMA shape of equal width and feed-forward, cut to
-# `layers` layers and a vocabulary of 32000 (name, layered config, LLaMA config, layers)
-FAMILY_SIZES = [("8b", "zefedra8b", "llama8b", 8), ("1b", "zefedra1b", "llama1b", 8)]
+# --family-bench: sizes at which the layered families run beside the LLaMA shape of equal width and feed-forward, cut to
+# `layers` layers and a vocabulary of 32000 (name, configs, layers)
+FAMILY_SIZES = [("8b", ("galarax8b", "zefedra8b", "llama8b"), 8), ("1b", ("galarax1b", "zefedra1b", "llama1b"), 8)]
 FAMILY_PREFILL = (2048, 8192)                            # prompt lengths
 FAMILY_DECODE = ((1, 1024), (32, 1024), (32, 4096), (4, 8192))  # (sequences, context)
 
@@ -495,8 +497,8 @@ def kernel_table(events, steps):
     return {k: [round(n / steps, 2), round(t / n, 2)] for k, (n, t) in sorted(table.items(), key=lambda kv: -kv[1][1])}
 
 
-def family_bench(L, env, only=None, profile_kernels=False):
-    """Prefill and decode throughput of the layered family and of its LLaMA counterpart; one JSON line per measurement.
+def family_bench(L, env, only=None, models=None, profile_kernels=False):
+    """Prefill and decode throughput of the layered families and of their LLaMA counterpart; one JSON line per measurement.
     Prefill: one prompt in one round.  Decode: a captured round, device-side token feedback; weights exceed L2.
     Device time between CUDA events, after warm-up."""
     import numpy as np
@@ -505,10 +507,12 @@ def family_bench(L, env, only=None, profile_kernels=False):
     from llama_cu_b200.model import reduced
     from torch.profiler import ProfilerActivity, profile
     dev = env.dev
-    for size, lname, gname, layers in FAMILY_SIZES:
+    for size, names, layers in FAMILY_SIZES:
         if only and size not in only:
             continue
-        for cname in (lname, gname):
+        for cname in names:
+            if models and not any(cname.startswith(m) for m in models):
+                continue
             cfg = replace(reduced(L.CONFIGS[cname], layers, 32000), act_dtype=L.BF16)
             nctx = 8192 + 128
             tokens = max(max(b * (c + 128) for b, c in FAMILY_DECODE), nctx)
@@ -608,7 +612,8 @@ def main():
     ap.add_argument("--probe-q8", action="store_true", help="with --probe-linear: Q8_0 weights")
     ap.add_argument("--probe-shape", default="gate_up", choices=["gate_up", "down", "qkv", "o"])
     ap.add_argument("--family-bench", nargs="*", default=None, metavar="SIZE", choices=[s[0] for s in FAMILY_SIZES],
-                    help="prefill and decode throughput of the layered family beside the LLaMA shape of equal width, instead of the workload")
+                    help="prefill and decode throughput of the layered families beside the LLaMA shape of equal width, instead of the workload")
+    ap.add_argument("--family-models", nargs="*", default=None, metavar="NAME", help="with --family-bench: only models whose name starts with one of these")
     ap.add_argument("--family-kernels", action="store_true", help="with --family-bench: launches and time of every kernel (CUPTI)")
     args = ap.parse_args()
     if args.probe_linear > 0:
@@ -625,7 +630,7 @@ def main():
         key, value = kv.split("=", 1)
         L.set_tuning(key, int(value))
     if args.family_bench is not None:
-        family_bench(L, env, args.family_bench, args.family_kernels)
+        family_bench(L, env, args.family_bench, args.family_models, args.family_kernels)
         return 0
     cname, batch, prange = WORKLOADS[args.workload]
     cfg = L.CONFIGS[cname]

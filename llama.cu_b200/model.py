@@ -11,7 +11,7 @@ import numpy as np
 
 from . import (BF16, F16, F32, LINEAR_KINDS, Q8_0, W_ATTN_NORM, W_DOWN, W_EMBD, W_FFN_NORM, W_GATE_UP, W_LM_HEAD,
                W_O, W_OUT_NORM, W_QKV, Context, ModelDesc, check, load_library, stream_ptr)
-from . import zefedra
+from . import galarax, zefedra
 from .layered import LayeredConfig
 
 
@@ -74,6 +74,8 @@ CONFIGS = {
 # layered families at the widths of the LLaMA shapes above (no published checkpoint has these sizes)
 CONFIGS["zefedra8b"] = zefedra.uniform("zefedra8b", 32, 4096, 32, 128, 128, 1536, 512, 14336, 128256)
 CONFIGS["zefedra1b"] = zefedra.uniform("zefedra1b", 16, 2048, 16, 128, 128, 768, 256, 8192, 128256)
+CONFIGS["galarax8b"] = galarax.uniform("galarax8b", 32, 4096, 32, 8, 128, 32, 16, 128, 128, 14336, 128256)
+CONFIGS["galarax1b"] = galarax.uniform("galarax1b", 16, 2048, 32, 8, 64, 16, 8, 128, 128, 8192, 128256)
 
 
 def reduced(cfg, n_layers, vocab=None, name=None):
