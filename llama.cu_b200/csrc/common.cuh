@@ -46,6 +46,8 @@ struct Tuning {
     int stack_fuse = 1;            // layered models, rounds of one or two decoded tokens: norms and residual as GEMV prologues (1: where it measured faster, 2: always)
     int latent_tc = 1;             // latent attention of decode rounds on tcgen05 (0: mma.sync kernel)
     int expand_min = 0;            // latent attention: fewest tokens of a portion that expands keys and values (0: by operation count, -1: never)
+    int stack_tc = 1;              // layered models, rounds of three or four tokens: linear layers on tcgen05 (0: never, 1: large ones, 2: all)
+    int delta_cols = 0;            // delta rule: columns per half warp of the scan (2, 4; 0: by the number of warps they leave)
     int p2p_scatter_ranks = 8;     // ranks from which the peer all-reduce takes the reduce-scatter + all-gather form
     long p2p_scatter_min = 131072; // ... for rounds of at least this many bytes
 };

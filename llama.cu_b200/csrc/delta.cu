@@ -3,15 +3,21 @@
 //     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // with q, k, v behind short causal convolutions, q and k unit vectors, and o normed and gated per head.
 //
-// Both products with the state run over the matrix as it was BEFORE the token, so that their reductions share one pass:
-//     u = beta (v - g (S^T k)),  S <- g S + k u^T,  o = g (S^T q) + (q . k) u
-// A column of S (one value dimension) lies in the registers of eight lanes, four columns in a warp; S never leaves the
-// registers inside a portion.  All of it is f32 arithmetic (two values per instruction), whatever the activation dtype.
+// Portions run in blocks of eight tokens.  With S the matrix ahead of a block, D_ij the decay between tokens j and i, and
+// G_i the decay up to token i, the recurrence unrolls to
+//     w_i = v_i - G_i (S^T k_i)
+//     u_i = beta_i (w_i - sum_{j < i} D_ij (k_i . k_j) u_j)       u = T w, T a lower triangle that depends on k, g, beta alone
+//     o_i = G_i (S^T q_i) + sum_{j <= i} D_ij (q_i . k_j) u_j     the sum is (B T) w with B_ij = D_ij (q_i . k_j)
+//     S   <- G_8 S + sum_j k_j (D_8j u_j)^T
+// The preparation solves for T and B T of every block in parallel; the scan then needs one pass of dot products with S, one
+// eight-term sum per token and one pass of updates, with a single reduction across lanes per block.  All decays are products of
+// numbers up to one: nothing is divided by a decay.  Everything is f32 arithmetic (two values per instruction in the scan),
+// whatever the activation dtype, and S stays in registers throughout a portion.
 //
-// Rounds with several tokens per request take three launches (convolutions and gates / the scan / norm and output gate), rounds
-// of one token per request a single one.  The inputs of the convolutions that a later round needs are double-buffered by
-// generation (a request's first token reads one half, its last token writes the other); the matrices are updated in place, every
-// column by the one warp that read it.
+// Rounds with several tokens per request take three launches (convolutions, gates and triangles / the scan / norm and output
+// gate), rounds of one token per request a single one.  The inputs of the convolutions that a later round needs are
+// double-buffered by generation (a request's first token reads one half, its last token writes the other); the matrices are
+// updated in place, every column by the one warp that read it.
 #include "gqa_prep.cuh"
 #include "stack.cuh"
 
@@ -62,6 +68,11 @@ struct ConvIn {
         if (back > seen) return 0.f;
         return state[(size_t)(taps - 1 - (back - in_portion)) * channels + c];
     }
+    __device__ __forceinline__ float4 at4(int back, int c) const {  // four channels
+        if (back <= in_portion) return *reinterpret_cast<const float4 *>(row + (c - (ptrdiff_t)back * stride));
+        if (back > seen) return make_float4(0.f, 0.f, 0.f, 0.f);
+        return *reinterpret_cast<const float4 *>(state + (size_t)(taps - 1 - (back - in_portion)) * channels + c);
+    }
 };
 __device__ __forceinline__ ConvIn conv_in(const DeltaArgs &a, int t, int r) {
     ConvIn c;
@@ -80,158 +91,329 @@ __device__ __forceinline__ float *conv_out(const DeltaArgs &a, int r) {
 // convolution and activation of one channel; `out`: state to leave behind (the request's last token), or nullptr
 __device__ __forceinline__ float conv_silu(const DeltaArgs &a, const ConvIn &in, int c, float *out) {
     float y = 0.f;
-    for (int j = 0; j < a.taps; ++j) {
-        const int back = a.taps - 1 - j;
-        const float x = in.at(back, c);
-        y = fmaf(a.conv[(size_t)j * in.channels + c], x, y);
-        if (out && j > 0) out[(size_t)(j - 1) * in.channels + c] = x;
-    }
+#pragma unroll 4
+    for (int j = 0; j < a.taps; ++j) y = fmaf(in.at(a.taps - 1 - j, c), a.conv[(size_t)j * in.channels + c], y);
+    if (out)  // after all loads: stores in between would hold them up
+#pragma unroll 4
+        for (int j = 1; j < a.taps; ++j) out[(size_t)(j - 1) * in.channels + c] = in.at(a.taps - 1 - j, c);
     return silu_f(y);
 }
 
-// ------------------------------------------------------------------ portions: convolutions and gates
-// One warp per (token, query/key head) or (token, value head).
+// ------------------------------------------------------------------ portions: convolutions, gates, triangles
+// One warp per (block of tokens, query/key head) or (block, value head).  Coefficients of a block and head: rows of T [8][8],
+// rows of B T [8][8], G [8], decay from token j to the block's end [8].
+constexpr int DB = DELTA_BLOCK;
+static_assert(DB == 8, "the lane layouts below are those of blocks of eight tokens");
+
+// Convolution and activation of four channels for the tokens of a block, put(token, values); tokens past `count` give zero.
+// Every input is requested before the first is used.
+__device__ __forceinline__ float4 fma4(const float4 &x, const float4 &w, const float4 &y) {
+    return make_float4(fmaf(x.x, w.x, y.x), fmaf(x.y, w.y, y.y), fmaf(x.z, w.z, y.z), fmaf(x.w, w.w, y.w));
+}
+template <int TAPS, class F>
+__device__ __forceinline__ void conv_block(const DeltaArgs &a, const ConvIn &in, int c, int count, float *out, const F &put) {
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (TAPS > 0) {
+        float4 w[TAPS], x[TAPS - 1 + DB];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float4 *>(a.conv + (size_t)j * in.channels + c));
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) x[j] = in.at4(TAPS - 1 - j, c);
+#pragma unroll
+        for (int i = 0; i < DB; ++i) x[TAPS - 1 + i] = i < count ? *reinterpret_cast<const float4 *>(in.row + c + (size_t)i * in.stride) : zero;
+#pragma unroll
+        for (int i = 0; i < DB; ++i) {
+            float4 y = zero;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) y = fma4(x[i + j], w[j], y);
+            put(i, i < count ? make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w)) : zero);
+            if (out && i + 1 == count)
+#pragma unroll
+                for (int j = 1; j < TAPS; ++j) *reinterpret_cast<float4 *>(out + (size_t)(j - 1) * in.channels + c) = x[i + j];
+        }
+    } else {
+        ConvIn t = in;
+        for (int i = 0; i < DB; ++i) {
+            float4 y = zero;
+            for (int j = 0; j < a.taps && i < count; ++j) {
+                const float4 x = t.at4(a.taps - 1 - j, c);
+                y = fma4(x, *reinterpret_cast<const float4 *>(a.conv + (size_t)j * in.channels + c), y);
+                if (out && i + 1 == count && j > 0) *reinterpret_cast<float4 *>(out + (size_t)(j - 1) * in.channels + c) = x;
+            }
+            put(i, make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w)));
+            t.row += t.stride; ++t.in_portion; ++t.seen;
+        }
+    }
+}
+
+template <int TAPS>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
+    extern __shared__ __align__(16) float sm[];
     grid_dep_launch();
-    const int t = blockIdx.y, lane = threadIdx.x & 31;
-    int item = blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int item = blockIdx.x * 8 + warp;
     if (item >= a.kv_heads + a.heads) return;
-    const int r = a.tok_req[t];
-    const bool last = t + 1 == a.req_first[r + 1];
+    const int4 blk = a.blocks[blockIdx.y];  // request, first token, tokens, slot of the coefficients
+    const int t0 = blk.y, count = blk.z;
+    const bool last = t0 + count == a.req_first[blk.x + 1];
     grid_dep_wait();
-    const ConvIn in = conv_in(a, t, r);
-    float *out = last ? conv_out(a, r) : nullptr;
+    const ConvIn in = conv_in(a, t0, blk.x);
+    float *out = last ? conv_out(a, blk.x) : nullptr;
     if (item >= a.kv_heads) {
         item -= a.kv_heads;
         const int c0 = 2 * a.kv_heads * a.dk_p + item * a.dv_p;
-        float *v = a.v + (size_t)t * a.heads * a.dv_p + (size_t)item * a.dv_p;
-        for (int d = lane; d < a.dv_p; d += 32) v[d] = conv_silu(a, in, c0 + d, out);
+        float *v = a.v + (size_t)t0 * a.heads * a.dv_p + (size_t)item * a.dv_p;
+        for (int d = 4 * lane; d < a.dv_p; d += 128)
+            conv_block<TAPS>(a, in, c0 + d, count, out, [&](int i, const float4 &y) { if (i < count) *reinterpret_cast<float4 *>(v + (size_t)i * a.heads * a.dv_p + d) = y; });
         return;
     }
-    float q[MIX_MAX_HEAD / 32], k[MIX_MAX_HEAD / 32], sq = 0.f, sk = 0.f, qk = 0.f;
-#pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
-        q[j] = k[j] = 0.f;
-        if (d < a.dk_p) {
-            q[j] = conv_silu(a, in, item * a.dk_p + d, out);
-            k[j] = conv_silu(a, in, (a.kv_heads + item) * a.dk_p + d, out);
-        }
-        sq += q[j] * q[j];
-        sk += k[j] * k[j];
-        qk += q[j] * k[j];
+    const int ld = a.dk_p + 4;
+    float *ks = sm + (size_t)warp * (2 * DB * ld + 2 * DB * DB), *qs = ks + DB * ld, *kk = qs + DB * ld, *qk = kk + DB * DB;
+    for (int d = 4 * lane; d < a.dk_p; d += 128) {
+        conv_block<TAPS>(a, in, item * a.dk_p + d, count, out, [&](int i, const float4 &y) { *reinterpret_cast<float4 *>(qs + i * ld + d) = y; });
+        conv_block<TAPS>(a, in, (a.kv_heads + item) * a.dk_p + d, count, out, [&](int i, const float4 &y) { *reinterpret_cast<float4 *>(ks + i * ld + d) = y; });
     }
-    const float rq = 1.f / sqrtf(warp_sum(sq) + 1e-6f) * (1.f / sqrtf((float)a.dk)), rk = 1.f / sqrtf(warp_sum(sk) + 1e-6f);
-    qk = warp_sum(qk) * rq * rk;
-    const size_t base = ((size_t)t * a.kv_heads + item) * a.dk_p;
+    __syncwarp();
+    {  // unit vectors: four lanes sum the squares of a token
+        float sq = 0.f, sk = 0.f;
+        for (int d = 4 * (lane & 3); d < a.dk_p; d += 16) {
+            sq += dot4(*reinterpret_cast<const float4 *>(qs + (lane >> 2) * ld + d));
+            sk += dot4(*reinterpret_cast<const float4 *>(ks + (lane >> 2) * ld + d));
+        }
+        sq += __shfl_xor_sync(0xffffffffu, sq, 1); sk += __shfl_xor_sync(0xffffffffu, sk, 1);
+        sq += __shfl_xor_sync(0xffffffffu, sq, 2); sk += __shfl_xor_sync(0xffffffffu, sk, 2);
+        const float my_rq = 1.f / sqrtf(sq + 1e-6f) * (1.f / sqrtf((float)a.dk)), my_rk = 1.f / sqrtf(sk + 1e-6f);
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
-        if (d < a.dk_p) {
-            a.q[base + d] = q[j] * rq;
-            a.k[base + d] = k[j] * rk;
+        for (int i = 0; i < DB; ++i) {
+            const float rq = __shfl_sync(0xffffffffu, my_rq, 4 * i), rk = __shfl_sync(0xffffffffu, my_rk, 4 * i);
+            for (int d = 4 * lane; d < a.dk_p; d += 128) {
+                float4 x = *reinterpret_cast<float4 *>(qs + i * ld + d), y = *reinterpret_cast<float4 *>(ks + i * ld + d);
+                x.x *= rq; x.y *= rq; x.z *= rq; x.w *= rq;
+                y.x *= rk; y.y *= rk; y.z *= rk; y.w *= rk;
+                *reinterpret_cast<float4 *>(qs + i * ld + d) = x;
+                *reinterpret_cast<float4 *>(ks + i * ld + d) = y;
+                if (i < count) {
+                    const size_t at = ((size_t)(t0 + i) * a.kv_heads + item) * a.dk_p + d;
+                    *reinterpret_cast<float4 *>(a.q + at) = x;
+                    *reinterpret_cast<float4 *>(a.k + at) = y;
+                }
+            }
         }
     }
-    const int reps = a.heads / a.kv_heads;
-    for (int i = lane; i < reps; i += 32) {
-        const int h = item * reps + i;
-        const float g = expf(-expf(a.decay[h]) * softplus_of(in.row[a.a_off() + h] + a.decay[a.heads_p + h]));
-        const float beta = 1.f / (1.f + expf(-in.row[a.b_off() + h]));
-        a.gate[(size_t)t * a.heads + h] = make_float4(g, beta, qk, 0.f);
+    __syncwarp();
+    {  // products of all pairs of tokens: this lane's row i against columns j and j + 1
+        const int i = lane >> 2, j = 2 * (lane & 3);
+        float k0 = 0.f, k1 = 0.f, q0 = 0.f, q1 = 0.f;
+        for (int d = 0; d < a.dk_p; d += 4) {
+            const float4 ki = *reinterpret_cast<const float4 *>(ks + i * ld + d), qi = *reinterpret_cast<const float4 *>(qs + i * ld + d);
+            const float4 x = *reinterpret_cast<const float4 *>(ks + j * ld + d), y = *reinterpret_cast<const float4 *>(ks + (j + 1) * ld + d);
+            k0 = fmaf(ki.x, x.x, k0); k0 = fmaf(ki.y, x.y, k0); k0 = fmaf(ki.z, x.z, k0); k0 = fmaf(ki.w, x.w, k0);
+            k1 = fmaf(ki.x, y.x, k1); k1 = fmaf(ki.y, y.y, k1); k1 = fmaf(ki.z, y.z, k1); k1 = fmaf(ki.w, y.w, k1);
+            q0 = fmaf(qi.x, x.x, q0); q0 = fmaf(qi.y, x.y, q0); q0 = fmaf(qi.z, x.z, q0); q0 = fmaf(qi.w, x.w, q0);
+            q1 = fmaf(qi.x, y.x, q1); q1 = fmaf(qi.y, y.y, q1); q1 = fmaf(qi.z, y.z, q1); q1 = fmaf(qi.w, y.w, q1);
+        }
+        kk[i * DB + j] = k0; kk[i * DB + j + 1] = k1;
+        qk[i * DB + j] = q0; qk[i * DB + j + 1] = q1;
+    }
+    __syncwarp();
+    // four heads at a time, eight lanes each: lane c solves column c of the head's triangles
+    const int reps = a.heads / a.kv_heads, c = lane & 7;
+    for (int r0 = 0; r0 < reps; r0 += 4) {
+        const int rep = r0 + (lane >> 3);
+        const bool ok = rep < reps;
+        const int h = item * reps + (ok ? rep : 0);
+        float my_g = 1.f, my_b = 0.f;  // a token past the end changes nothing
+        if (c < count) {
+            const float *row = in.row + (size_t)c * in.stride;
+            my_g = expf(-expf(a.decay[h]) * softplus_of(row[a.a_off() + h] + a.decay[a.heads_p + h]));
+            my_b = 1.f / (1.f + expf(-row[a.b_off() + h]));
+        }
+        float g[DB], x[DB], m[DB], total = 1.f, upto = 1.f, rest = 1.f;
+#pragma unroll
+        for (int i = 0; i < DB; ++i) {
+            g[i] = __shfl_sync(0xffffffffu, my_g, i, 8);
+            total *= g[i];
+            if (i <= c) upto = total;
+        }
+#pragma unroll
+        for (int i = DB - 1; i > 0; --i)
+            if (i > c) rest *= g[i];
+#pragma unroll
+        for (int i = 0; i < DB; ++i) {
+            const float bi = __shfl_sync(0xffffffffu, my_b, i, 8);
+            float sum = 0.f, p = 1.f, mm = 0.f;
+#pragma unroll
+            for (int j = i - 1; j >= 0; --j) {
+                p *= g[j + 1];
+                sum = fmaf(p * kk[i * DB + j], x[j], sum);
+                mm = fmaf(p * qk[i * DB + j], x[j], mm);
+            }
+            x[i] = (i == c ? my_b : 0.f) - bi * sum;
+            m[i] = fmaf(qk[i * DB + i], x[i], mm);
+        }
+        if (ok) {
+            float *dst = a.coef + ((size_t)blk.w * a.heads + h) * DELTA_COEF;
+#pragma unroll
+            for (int i = 0; i < DB; ++i) {
+                dst[i * DB + c] = x[i];
+                dst[(DB + i) * DB + c] = m[i];
+            }
+            dst[2 * DB * DB + c] = upto;
+            dst[2 * DB * DB + DB + c] = rest;
+        }
     }
 }
 
 // ------------------------------------------------------------------ portions: the scan
-constexpr int DS_TOK = 16;  // tokens per shared-memory tile
-
-__device__ __forceinline__ void ds_cp16(float *smem_dst, const float *src) {
+__device__ __forceinline__ void ds_cp16(float *smem_dst, const float *src, bool valid) {
     unsigned d = (unsigned)__cvta_generic_to_shared(smem_dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+    int sz = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(sz) : "memory");
 }
+constexpr int DS_STAGES = 3;
 
-// grid (column slices, heads, requests); a warp holds four columns, lane = 8 (column of the warp) + part of the key dimension.
-// R key dimensions per lane: 4 consecutive ones of every 32.
-template <int R>
-__global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaArgs a) {
-    constexpr int DK = 8 * R;
+// grid (column slices, heads, requests).  A half warp holds NC columns; lane p of it the key dimensions 2 p, 2 p + 1 of every 32
+// (R in all).  After the reduction lane p holds the products of token p & 7, with its key (p < 8) or its query.
+template <int R, int NC>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
+    constexpr int DK = 16 * R;
     extern __shared__ __align__(16) float sm[];
+    __shared__ __align__(16) float s_w[4][2][DB][NC], s_u[4][2][DB][NC];
     grid_dep_launch();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane & 7;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, grp = lane >> 4, p = lane & 15, tok = p & 7;
+    const bool is_q = p >= 8;
     const int h = blockIdx.y, r = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
-    const int cols = blockDim.x / 8, col0 = blockIdx.x * cols, lc = warp * 4 + (lane >> 3), col = col0 + lc;
-    const bool valid = col < a.dv_p;
-    const int row = 2 * DK + cols + 4;  // q | k | v | gate of a token
-    const int first = a.req_first[r], end = a.req_first[r + 1];
-    float *st = a.state + (((size_t)(a.req_slot[r] >> 1) * a.heads + h) * a.dv_p + (valid ? col : 0)) * DK + part * 4;
+    const int cols = (blockDim.x >> 5) * 2 * NC, col0 = blockIdx.x * cols, lc = (warp * 2 + grp) * NC, col = col0 + lc;
+    const bool valid = col < a.dv_p;  // columns come in whole groups of 16
+    const int stage = 2 * DB * DK + DB * cols + DELTA_COEF;
+    const int first = a.req_first[r], end = a.req_first[r + 1], n_blk = (end - first + DB - 1) / DB;
+    const size_t slot0 = first / DB + r;
+    float *st = a.state + (((size_t)(a.req_slot[r] >> 1) * a.heads + h) * a.dv_p + (valid ? col : 0)) * DK + 2 * p;
     const bool fresh = a.req_pos[r] == 0;
-    f32x2 s[R / 2];
+    f32x2 s[R / 2][NC];
 #pragma unroll
-    for (int j = 0; j < R / 4; ++j) {
-        const float4 v = valid && !fresh ? *reinterpret_cast<const float4 *>(st + 32 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
-        s[2 * j] = pk2(v.x, v.y);
-        s[2 * j + 1] = pk2(v.z, v.w);
-    }
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) {
+            const float2 v = valid && !fresh ? *reinterpret_cast<const float2 *>(st + (size_t)c * DK + 32 * i) : make_float2(0.f, 0.f);
+            s[i][c] = pk2(v.x, v.y);
+        }
     grid_dep_wait();
-    const int vcols = min(cols, a.dv_p - col0);
-    auto load = [&](int t0, int buf) {
-        float *dst = sm + (size_t)buf * DS_TOK * row;
-        const int n = min(DS_TOK, end - t0), per = 2 * (DK / 4) + vcols / 4 + 1;
-        for (int i = tid; i < n * per; i += blockDim.x) {
-            const int j = i / per, c = i - j * per;
-            const size_t t = t0 + j;
-            const float *src;
-            int at;
-            if (c < DK / 4) src = a.q + (t * a.kv_heads + kvh) * DK + 4 * c, at = 4 * c;
-            else if (c < 2 * (DK / 4)) src = a.k + (t * a.kv_heads + kvh) * DK + 4 * c - DK, at = 4 * c;
-            else if (c < 2 * (DK / 4) + vcols / 4) src = a.v + (t * a.heads + h) * a.dv_p + col0 + 4 * c - 2 * DK, at = 4 * c;
-            else src = reinterpret_cast<const float *>(a.gate + t * a.heads + h), at = 2 * DK + cols;
-            ds_cp16(dst + j * row + at, src);
+    const int vch = min(cols, a.dv_p - col0) / 4;  // 16-byte pieces of a value row
+    auto load = [&](int b) {
+        float *dst = sm + (size_t)(b % DS_STAGES) * stage;
+        const int t0 = first + b * DB;
+        for (int i = tid; i < DB * (DK / 4); i += blockDim.x) {
+            const int j = i / (DK / 4), c = 4 * (i % (DK / 4));
+            const bool ok = t0 + j < end;
+            const size_t off = ((size_t)(ok ? t0 + j : first) * a.kv_heads + kvh) * DK + c;
+            ds_cp16(dst + j * DK + c, a.k + off, ok);
+            ds_cp16(dst + (DB + j) * DK + c, a.q + off, ok);
         }
+        for (int i = tid; i < DB * (cols / 4); i += blockDim.x) {
+            const int j = i / (cols / 4), c = i % (cols / 4);
+            const bool ok = t0 + j < end && c < vch;
+            ds_cp16(dst + 2 * DB * DK + j * cols + 4 * c, a.v + ((size_t)(ok ? t0 + j : first) * a.heads + h) * a.dv_p + (ok ? col0 + 4 * c : 0), ok);
+        }
+        for (int i = tid; i < DELTA_COEF / 4; i += blockDim.x)
+            ds_cp16(dst + 2 * DB * DK + DB * cols + 4 * i, a.coef + ((slot0 + b) * a.heads + h) * DELTA_COEF + 4 * i, true);
     };
-    load(first, 0);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    int buf = 0;
-    for (int t0 = first; t0 < end; t0 += DS_TOK, buf ^= 1) {
-        if (t0 + DS_TOK < end) load(t0 + DS_TOK, buf ^ 1);
+#pragma unroll
+    for (int b = 0; b < DS_STAGES - 1; ++b) {
+        if (b < n_blk) load(b);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
-        const float *tile = sm + (size_t)buf * DS_TOK * row;
-        const int n = min(DS_TOK, end - t0);
-        for (int j = 0; j < n; ++j) {
-            const float *p = tile + j * row;
-            const float4 gate = *reinterpret_cast<const float4 *>(p + 2 * DK + cols);
-            const float v = p[2 * DK + (valid ? lc : 0)];
-            f32x2 k[R / 2], k2[2] = {0ull, 0ull}, q2[2] = {0ull, 0ull};
+    }
+    for (int b = 0; b < n_blk; ++b) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(DS_STAGES - 2) : "memory");
+        __syncthreads();  // block b has landed, block b - 1 has been read
+        if (b + DS_STAGES - 1 < n_blk) load(b + DS_STAGES - 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const float *tile = sm + (size_t)(b % DS_STAGES) * stage, *coef = tile + 2 * DB * DK + DB * cols;
+
+        float acc[8][NC];  // after the first exchange: products with the eight keys (p < 8) or queries
+        {
+            f32x2 d[2 * DB][NC];
 #pragma unroll
-            for (int i = 0; i < R / 4; ++i) {
-                const ulonglong2 kv = *reinterpret_cast<const ulonglong2 *>(p + DK + 32 * i + part * 4);
-                const ulonglong2 qv = *reinterpret_cast<const ulonglong2 *>(p + 32 * i + part * 4);
-                k[2 * i] = kv.x;
-                k[2 * i + 1] = kv.y;
-                k2[0] = fma2(s[2 * i], kv.x, k2[0]);
-                k2[1] = fma2(s[2 * i + 1], kv.y, k2[1]);
-                q2[0] = fma2(s[2 * i], qv.x, q2[0]);
-                q2[1] = fma2(s[2 * i + 1], qv.y, q2[1]);
-            }
-            const float2 ka = up2(k2[0]), kb = up2(k2[1]), qa = up2(q2[0]), qb = up2(q2[1]);
-            const float sk = octet_sum((ka.x + ka.y) + (kb.x + kb.y));
-            const float u = gate.y * (v - gate.x * sk);
-            const f32x2 g2 = pk2(gate.x, gate.x), u2 = pk2(u, u);
+            for (int i = 0; i < 2 * DB; ++i)
 #pragma unroll
-            for (int i = 0; i < R / 2; ++i) s[i] = fma2(k[i], u2, mul2(s[i], g2));
-            const float sq = octet_sum((qa.x + qa.y) + (qb.x + qb.y));
-            if (part == 0 && valid) a.v[((size_t)(t0 + j) * a.heads + h) * a.dv_p + col] = gate.x * sq + gate.z * u;
+                for (int c = 0; c < NC; ++c) d[i][c] = 0ull;
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i)
+#pragma unroll
+                for (int j = 0; j < 2 * DB; ++j) {
+                    const f32x2 x = *reinterpret_cast<const f32x2 *>(tile + j * DK + 32 * i + 2 * p);
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) d[j][c] = fma2(s[i][c], x, d[j][c]);
+                }
+#pragma unroll
+            for (int j = 0; j < DB; ++j)
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float2 x = up2(d[j][c]), y = up2(d[DB + j][c]);
+                    const float kd = x.x + x.y, qd = y.x + y.y;
+                    acc[j][c] = (is_q ? qd : kd) + __shfl_xor_sync(0xffffffffu, is_q ? kd : qd, 8);
+                }
         }
-        __syncthreads();
+#pragma unroll
+        for (int m = 4; m > 0; m >>= 1)
+#pragma unroll
+            for (int j = 0; j < m; ++j)
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float lo = acc[j][c], hi = acc[j + m][c];
+                    acc[j][c] = ((p & m) ? hi : lo) + __shfl_xor_sync(0xffffffffu, (p & m) ? lo : hi, m);
+                }
+        const float upto = coef[2 * DB * DB + tok], rest = coef[2 * DB * DB + DB + tok], total = coef[2 * DB * DB + DB - 1];
+        if (!is_q)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) s_w[warp][grp][tok][c] = (valid ? tile[2 * DB * DK + tok * cols + lc + c] : 0.f) - upto * acc[0][c];
+        __syncwarp();
+        float row[DB], y[NC];
+#pragma unroll
+        for (int j = 0; j < DB; j += 4) {
+            const float4 x = *reinterpret_cast<const float4 *>(coef + p * DB + j);
+            row[j] = x.x; row[j + 1] = x.y; row[j + 2] = x.z; row[j + 3] = x.w;
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) y[c] = is_q ? upto * acc[0][c] : 0.f;
+#pragma unroll
+        for (int j = 0; j < DB; ++j)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) y[c] = fmaf(row[j], s_w[warp][grp][j][c], y[c]);
+        const int t = first + b * DB + tok;
+        if (!is_q) {
+#pragma unroll
+            for (int c = 0; c < NC; ++c) s_u[warp][grp][tok][c] = rest * y[c];
+        } else if (valid && t < end) {
+            float *dst = a.v + ((size_t)t * a.heads + h) * a.dv_p + col;
+            if constexpr (NC == 4) *reinterpret_cast<float4 *>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+            else *reinterpret_cast<float2 *>(dst) = make_float2(y[0], y[1]);
+        }
+        __syncwarp();
+        const f32x2 total2 = pk2(total, total);
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) s[i][c] = mul2(s[i][c], total2);
+#pragma unroll
+        for (int j = 0; j < DB; ++j) {
+            f32x2 u[NC];
+#pragma unroll
+            for (int c = 0; c < NC; ++c) { const float x = s_u[warp][grp][j][c]; u[c] = pk2(x, x); }
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i) {
+                const f32x2 x = *reinterpret_cast<const f32x2 *>(tile + j * DK + 32 * i + 2 * p);
+#pragma unroll
+                for (int c = 0; c < NC; ++c) s[i][c] = fma2(x, u[c], s[i][c]);
+            }
+        }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     if (!valid) return;
 #pragma unroll
-    for (int j = 0; j < R / 4; ++j) {
-        const float2 x = up2(s[2 * j]), y = up2(s[2 * j + 1]);
-        *reinterpret_cast<float4 *>(st + 32 * j) = make_float4(x.x, x.y, y.x, y.y);
-    }
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) *reinterpret_cast<float2 *>(st + (size_t)c * DK + 32 * i) = up2(s[i][c]);
 }
 
 // ------------------------------------------------------------------ portions: norm and output gate, a warp per (token, head)
@@ -244,22 +426,27 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs a) {
     const int t = (int)(i / a.heads), h = (int)(i - (long)t * a.heads);
     grid_dep_wait();
     const float *o = a.v + (size_t)i * a.dv_p, *g = a.lat + (size_t)t * a.stride + a.g_off() + h * a.dv_p;
-    float v[MIX_MAX_HEAD / 32], ss = 0.f;
+    float4 v[MIX_MAX_HEAD / 128], z[MIX_MAX_HEAD / 128];
+    float ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
-        v[j] = d < a.dv_p ? o[d] : 0.f;
-        ss += v[j] * v[j];
+    for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
+        const int d = 4 * lane + 128 * j;
+        v[j] = z[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d < a.dv_p) {
+            v[j] = *reinterpret_cast<const float4 *>(o + d);
+            z[j] = *reinterpret_cast<const float4 *>(g + d);
+        }
+        ss += dot4(v[j]);
     }
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)a.dv + a.eps);
     T *dst = reinterpret_cast<T *>(a.o) + (size_t)t * a.stride_o + (size_t)h * a.dv_p;
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
+    for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
+        const int d = 4 * lane + 128 * j;
         if (d >= a.dv_p) continue;
-        const float x = v[j] * r * a.norm[d] * silu_f(g[d]);
-        if constexpr (sizeof(T) == 4) dst[d] = x;
-        else dst[d] = Act<T>::from_f(x);
+        const float4 w = *reinterpret_cast<const float4 *>(a.norm + d);
+        st4<T>(dst + d, make_float4(v[j].x * r * w.x * silu_f(z[j].x), v[j].y * r * w.y * silu_f(z[j].y), v[j].z * r * w.z * silu_f(z[j].z),
+                                    v[j].w * r * w.w * silu_f(z[j].w)));
     }
 }
 
@@ -371,14 +558,22 @@ struct ScanLaunch {
     const DeltaArgs &a;
     cudaStream_t s;
     bool pdl;
-    template <int R> int run() const {
-        // 32 columns per CTA where that still fills the SMs, 16 otherwise
-        const int cols = a.dv_p > 16 && (long)a.n_req * a.heads * ((a.dv_p + 31) / 32) * 4 >= 3 * sm_count() ? 32 : 16;
-        const size_t smem = (size_t)2 * DS_TOK * (16 * R + cols + 4) * 4;
+    template <int R, int NC> int launch(int warps) const {
+        const int cols = warps * 2 * NC;
+        const size_t smem = (size_t)DS_STAGES * (2 * DB * 16 * R + DB * cols + DELTA_COEF) * 4;
         const dim3 grid((a.dv_p + cols - 1) / cols, a.heads, a.n_req);
-        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        LCU_CHECK_CUDA(launch_kernel(delta_scan_kernel<R>, grid, dim3(cols * 8), smem, s, pdl, a));
+        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(delta_scan_kernel<R, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LCU_CHECK_CUDA(launch_kernel(delta_scan_kernel<R, NC>, grid, dim3(warps * 32), smem, s, pdl, a));
         return LCU_OK;
+    }
+    template <int R8> int run() const {
+        constexpr int R = R8 / 2;  // key dimensions per lane of a half warp
+        // columns per half warp: four where that leaves a warp for every scheduler, two otherwise
+        const long groups = (long)a.n_req * a.heads * ((a.dv_p + 15) / 16);
+        if constexpr (R <= 8) {
+            if (tuning().delta_cols == 4 || (tuning().delta_cols == 0 && groups * 2 >= 3l * sm_count())) return launch<R, 4>(a.dv_p > 16 ? 4 : 2);
+        }
+        return launch<R, 2>(4);
     }
 };
 struct DecodeLaunch {
@@ -399,10 +594,21 @@ struct DecodeLaunch {
 }  // namespace
 
 int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
-    if (a.n_tok <= 0) return LCU_OK;
-    LCU_REQUIRE(a.n_tok <= 65535 && a.dk_p <= MIX_MAX_HEAD && a.dv_p <= MIX_MAX_HEAD, "delta rule: %d tokens, head sizes %d / %d", a.n_tok, a.dk_p, a.dv_p);
-    LCU_CHECK_CUDA(launch_kernel(delta_prep_kernel, dim3((a.kv_heads + a.heads + 7) / 8, a.n_tok), dim3(256), 0, s, pdl, a));
-    return LCU_OK;
+    if (a.n_blocks <= 0) return LCU_OK;
+    LCU_REQUIRE(a.n_blocks <= 65535 && a.dk_p <= MIX_MAX_HEAD && a.dv_p <= MIX_MAX_HEAD, "delta rule: %d blocks, head sizes %d / %d", a.n_blocks, a.dk_p, a.dv_p);
+    const dim3 grid((a.kv_heads + a.heads + 7) / 8, a.n_blocks);
+    const size_t smem = (size_t)8 * (2 * DB * (a.dk_p + 4) + 2 * DB * DB) * 4;
+    auto go = [&](auto kernel) -> int {
+        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(256), smem, s, pdl, a));
+        return LCU_OK;
+    };
+    switch (a.taps) {
+    case 2: return go(delta_prep_kernel<2>);
+    case 3: return go(delta_prep_kernel<3>);
+    case 4: return go(delta_prep_kernel<4>);
+    default: return go(delta_prep_kernel<0>);
+    }
 }
 int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
     if (a.n_req <= 0) return LCU_OK;

@@ -1,7 +1,7 @@
 // The step between the fused input projection and softmax attention, one warp per (token, head): bias, rotation, norm; the
 // query to its buffer, key and value to the cache.  Shared by the kernels of gqa.cu and the decode kernel of delta.cu.
 #pragma once
-#include "mixers.cuh"
+#include "stack.cuh"
 
 namespace lcu {
 
@@ -24,32 +24,52 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     }
     const int half = a.rot_dims >> 1;
     const float2 *rot = a.rot + (size_t)p * half;
-    float v[MIX_MAX_HEAD / 32];
+    auto load4 = [&](int d) {
+        float4 x = *reinterpret_cast<const float4 *>(src + d);
+        if (bias) {
+            const float4 y = *reinterpret_cast<const float4 *>(bias + d);
+            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+        }
+        return x;
+    };
+    float4 v[MIX_MAX_HEAD / 128];
     float ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
-        v[j] = 0.f;
+    for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
+        const int d = 4 * lane + 128 * j;
+        v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (d >= size_p) continue;
-        float x = src[d] + (bias ? bias[d] : 0.f);
+        float4 x = load4(d);
         if (!is_v && d < a.rot_dims) {
-            const int e = d < half ? d + half : d - half;
-            const float y = src[e] + (bias ? bias[e] : 0.f);
-            const float2 cs = rot[d < half ? d : e];
-            x = d < half ? x * cs.x - y * cs.y : x * cs.x + y * cs.y;
+            if (half % 4 == 0) {  // four pairs: the partners are four consecutive dimensions too
+                const bool lower = d < half;
+                const int e = lower ? d + half : d - half;
+                const float4 y = load4(e), c0 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e)), c1 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e) + 2);
+                const float sgn = lower ? -1.f : 1.f;
+                x.x = x.x * c0.x + sgn * y.x * c0.y; x.y = x.y * c0.z + sgn * y.y * c0.w;
+                x.z = x.z * c1.x + sgn * y.z * c1.y; x.w = x.w * c1.z + sgn * y.w * c1.w;
+            } else {
+                float *xs = reinterpret_cast<float *>(&x);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const int i = d + k;
+                    if (i >= a.rot_dims) continue;
+                    const int e = i < half ? i + half : i - half;
+                    const float y = src[e] + (bias ? bias[e] : 0.f);
+                    const float2 cs = rot[i < half ? i : e];
+                    xs[k] = i < half ? xs[k] * cs.x - y * cs.y : xs[k] * cs.x + y * cs.y;
+                }
+            }
         }
         v[j] = x;
-        ss += x * x;
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
     }
     float r = 1.f;
     if (!is_v && a.qk_norm) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
-        const int d = lane + 32 * j;
-        if (d < size_p) {
-            if constexpr (sizeof(T) == 4) dst[d] = v[j] * r;
-            else dst[d] = Act<T>::from_f(v[j] * r);
-        }
+    for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
+        const int d = 4 * lane + 128 * j;
+        if (d < size_p) st4<T>(dst + d, make_float4(v[j].x * r, v[j].y * r, v[j].z * r, v[j].w * r));
     }
 }
 

@@ -52,6 +52,8 @@ int gqa_long_launch(const GqaArgs &a, cudaStream_t s, bool dry = false);
 int gqa_f32_launch(const GqaArgs &a, cudaStream_t s);
 
 // ---- gated delta rule
+constexpr int DELTA_BLOCK = 8;                                                   // tokens of a block of the scan
+constexpr int DELTA_COEF = 2 * DELTA_BLOCK * DELTA_BLOCK + 2 * DELTA_BLOCK;      // coefficients of a block and head
 struct DeltaArgs {
     // rows of the fused projection: q heads | k heads (dk_p) | v heads | output gate (dv_p) | step size | decay (heads_p)
     const float *lat;
@@ -69,7 +71,9 @@ struct DeltaArgs {
     // between the kernels of a round with several tokens per request
     float *q, *k;               // [n_tok][kv_heads * dk_p], unit vectors, q scaled
     float *v;                   // [n_tok][heads * dv_p]; the scan overwrites it with its outputs
-    float4 *gate;               // [n_tok][heads]: decay, step size, q . k
+    const int4 *blocks;         // (request, first token, tokens, slot first / 8 + request + number of the block in its request)
+    int n_blocks;
+    float *coef;                // [slot][heads][DELTA_COEF]
     void *o;                    // [n_tok][stride_o], heads x dv_p
     int stride_o;
     __host__ __device__ int channels() const { return 2 * kv_heads * dk_p + heads * dv_p; }
@@ -78,7 +82,7 @@ struct DeltaArgs {
     __host__ __device__ int a_off() const { return b_off() + heads_p; }
     __host__ __device__ int rows() const { return a_off() + heads_p; }
 };
-// Rounds with several tokens per request: convolutions and gates; the recurrence; norm and output gate.
+// Rounds with several tokens per request: convolutions, gates and triangles; the scan; norm and output gate.
 int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
 int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);

@@ -223,7 +223,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                  o_xc = reserve((size_t)S->expand_cap * S->max_r * eb), o_xkv = reserve((size_t)S->expand_cap * max_kv * eb),
                  o_hout = reserve((T > (size_t)c->max_seqs ? T : c->max_seqs) * S->d_p * eb), o_po = reserve(rows * S->max_r * 4),
                  o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4), o_y2 = reserve(S->pre_norm ? T * S->d_p * 4 : 0),
-                 o_dq = reserve(T * max_dk * 4), o_dk = reserve(T * max_dk * 4), o_dv = reserve(T * max_dv * 4), o_dg = reserve(T * max_dh * 16),
+                 o_dq = reserve(T * max_dk * 4), o_dk = reserve(T * max_dk * 4), o_dv = reserve(T * max_dv * 4), o_dg = reserve((T / DELTA_BLOCK + c->max_seqs + 1) * max_dh * DELTA_COEF * 4),
                  o_att2 = reserve(T * max_dhv * eb), o_conv = reserve(2 * S->conv_gen * 4), o_mat = reserve(mat_total * S->n_slots * 4),
                  o_gp = reserve(gqa_part_floats(S->gqa_ctas, max_vp) * 4), o_gt = reserve((size_t)S->gqa_ctas * 4);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
@@ -236,7 +236,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->part_o = reinterpret_cast<float *>(p + o_po); S->part_ml = reinterpret_cast<float *>(p + o_pml); S->part_n = reinterpret_cast<int *>(p + o_pn);
 
     S->y2 = reinterpret_cast<float *>(p + o_y2); S->dq = reinterpret_cast<float *>(p + o_dq); S->dk = reinterpret_cast<float *>(p + o_dk);
-    S->dv = reinterpret_cast<float *>(p + o_dv); S->dgate = reinterpret_cast<float4 *>(p + o_dg); S->att2 = p + o_att2;
+    S->dv = reinterpret_cast<float *>(p + o_dv); S->dcoef = reinterpret_cast<float *>(p + o_dg); S->att2 = p + o_att2;
     S->conv_state = reinterpret_cast<float *>(p + o_conv); S->mat_state = reinterpret_cast<float *>(p + o_mat);
     S->gqa_part = reinterpret_cast<float *>(p + o_gp); S->gqa_tickets = reinterpret_cast<unsigned *>(p + o_gt);
 
@@ -405,7 +405,7 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
             *slot = reinterpret_cast<int32_t *>(B + D.req_slot), *afirst = reinterpret_cast<int32_t *>(B + D.abs_first),
             *aid = reinterpret_cast<int32_t *>(B + D.abs_id), *atok = reinterpret_cast<int32_t *>(B + D.abs_tok);
     int4 *xreq = reinterpret_cast<int4 *>(B + D.xreq), *xg = reinterpret_cast<int4 *>(B + D.xgroups);
-    int4 *sreq = reinterpret_cast<int4 *>(B + D.sreq), *lreq = reinterpret_cast<int4 *>(B + D.lreq);
+    int4 *sreq = reinterpret_cast<int4 *>(B + D.sreq), *lreq = reinterpret_cast<int4 *>(B + D.lreq), *dblk = reinterpret_cast<int4 *>(B + D.dblk);
     int short_max = 1 << 30;  // one decision per request and round: the layer with the largest head groups decides
     for (const StackLayer &L : S.layers)
         if (L.attention()) { const int v = gqa_short_tokens(L.d.heads, L.d.kv_heads); if (v < short_max) short_max = v; }
@@ -426,6 +426,8 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
                 lreq[q.n_long++] = make_int4(i, t, len, pos[i]);
                 q.long_len.push_back(len);
             }
+            for (int j = 0; j < len; j += DELTA_BLOCK)
+                dblk[q.n_delta_blocks++] = make_int4(i, t + j, len - j < DELTA_BLOCK ? len - j : DELTA_BLOCK, t / DELTA_BLOCK + i + j / DELTA_BLOCK);
         } else if (len < expand_min) {
             aid[q.n_abs_req] = i;
             afirst[q.n_abs_req++] = q.n_abs_tok;

@@ -59,6 +59,7 @@ struct StackRound {
     // softmax attention: requests whose portion takes the short form, and those that take the long one
     int n_short = 0, max_short = 0, n_long = 0;
     std::vector<int> long_len;
+    int n_delta_blocks = 0;  // delta rule: blocks of tokens
 };
 
 struct Stack {
@@ -79,8 +80,7 @@ struct Stack {
     int max_heads = 0, max_r = 0;
     // pre-norm models
     bool pre_norm = false;
-    float *y2 = nullptr, *dq = nullptr, *dk = nullptr, *dv = nullptr, *conv_state = nullptr, *mat_state = nullptr, *gqa_part = nullptr;
-    float4 *dgate = nullptr;
+    float *y2 = nullptr, *dq = nullptr, *dk = nullptr, *dv = nullptr, *dcoef = nullptr, *conv_state = nullptr, *mat_state = nullptr, *gqa_part = nullptr;
     void *att2 = nullptr;
     unsigned *gqa_tickets = nullptr;
     size_t conv_gen = 0;    // f32 values of one generation of the convolutions' state

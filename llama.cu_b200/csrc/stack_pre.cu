@@ -90,7 +90,8 @@ struct PreNormRound {
         a.conv_state = S().conv_state + Y.conv_off * S().n_slots; a.conv_gen_stride = S().conv_gen; a.state = S().mat_state + Y.mat_off * S().n_slots;
         a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req);
         a.req_first = i32(o.req_first); a.req_pos = i32(o.req_pos); a.req_slot = i32(o.req_slot);
-        a.q = S().dq; a.k = S().dk; a.v = S().dv; a.gate = S().dgate; a.o = S().att2; a.stride_o = Y.dhv_p;
+        a.q = S().dq; a.k = S().dk; a.v = S().dv; a.coef = S().dcoef;
+        a.blocks = reinterpret_cast<const int4 *>(B + o.dblk); a.n_blocks = r.sr.n_delta_blocks; a.o = S().att2; a.stride_o = Y.dhv_p;
         return a;
     }
 

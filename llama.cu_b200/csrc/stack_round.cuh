@@ -10,7 +10,7 @@ inline size_t act_bytes(const lcu_ctx *c) { return c->dt == LCU_F32 ? 4 : 2; }
 
 // offsets inside the stack section of the round descriptor
 struct StackDesc {
-    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, sreq, lreq, total;
+    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, sreq, lreq, dblk, total;
 };
 constexpr int EXPAND_GROUP = 64;  // query tokens per group of the expanded attention
 inline StackDesc stack_desc(int n_tok, int n_req) {
@@ -27,6 +27,7 @@ inline StackDesc stack_desc(int n_tok, int n_req) {
     d.xgroups = take((size_t)(n_tok / EXPAND_GROUP + n_req) * 16);
     d.sreq = take((size_t)n_req * 16);
     d.lreq = take((size_t)n_req * 16);
+    d.dblk = take((size_t)(n_tok / DELTA_BLOCK + n_req) * 16);
     d.total = o;
     return d;
 }
@@ -52,7 +53,9 @@ struct Launcher {
             return linear_f32_launch(a, s);
         }
         const size_t yb = epilogue == EPI_STORE_F32 ? 4 : 2;
-        const bool tc = n > 4;
+        // three and four tokens: the GEMV streams small matrices faster, the tcgen05 kernels large ones (4 sequences at 8192, per
+        // 8-layer step: width 4096 1.88 -> 1.55 ms, width 2048 0.88 -> 1.04 ms)
+        const bool tc = n > 4 || (n > 2 && (tuning().stack_tc == 2 || (tuning().stack_tc == 1 && (long)in * out >= (32l << 20))));
         for (int t0 = 0; t0 < n;) {
             const int most = tc ? (tuning().tc_block < 256 ? tuning().tc_block : GEMM_TC_MAX_TOKENS) : gemv_max_tokens(in);
             const int nt = n - t0 < most ? n - t0 : most;
