@@ -47,7 +47,7 @@ struct Tuning {
     int latent_tc = 1;             // latent attention of decode rounds on tcgen05 (0: mma.sync kernel)
     int expand_min = 0;            // latent attention: fewest tokens of a portion that expands keys and values (0: by operation count, -1: never)
     int stack_tc = 1;              // layered models, rounds of three or four tokens: linear layers on tcgen05 (0: never, 1: large ones, 2: all)
-    int delta_cols = 0;            // delta rule: columns per half warp of the scan (2, 4; 0: by the number of warps they leave)
+    int delta_tc = 1;              // delta rule: the scan of bf16 contexts on tensor cores (0: f32 pipes)
     int p2p_scatter_ranks = 8;     // ranks from which the peer all-reduce takes the reduce-scatter + all-gather form
     long p2p_scatter_min = 131072; // ... for rounds of at least this many bytes
 };

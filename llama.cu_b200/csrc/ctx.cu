@@ -591,7 +591,7 @@ int lcu_set_tuning(lcu_ctx *c, const char *key, long long value) {
     else if (k == "stack_fuse") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_fuse = %lld (0..2)", value); t.stack_fuse = (int)value; }
     else if (k == "latent_tc") t.latent_tc = value != 0;
     else if (k == "stack_tc") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_tc = %lld (0..2)", value); t.stack_tc = (int)value; }
-    else if (k == "delta_cols") { LCU_REQUIRE(value == 0 || value == 2 || value == 4, "set_tuning: delta_cols = %lld (0, 2, 4)", value); t.delta_cols = (int)value; }
+    else if (k == "delta_tc") t.delta_tc = value != 0;
     else if (k == "expand_min") t.expand_min = (int)value;
     else if (k == "p2p_scatter_ranks") t.p2p_scatter_ranks = (int)value;
     else if (k == "p2p_scatter_min") t.p2p_scatter_min = (long)value;

@@ -11,8 +11,9 @@
 //     S   <- G_8 S + sum_j k_j (D_8j u_j)^T
 // The preparation solves for T and B T of every block in parallel; the scan then needs one pass of dot products with S, one
 // eight-term sum per token and one pass of updates, with a single reduction across lanes per block.  All decays are products of
-// numbers up to one: nothing is divided by a decay.  Everything is f32 arithmetic (two values per instruction in the scan),
-// whatever the activation dtype, and S stays in registers throughout a portion.
+// numbers up to one: nothing is divided by a decay.  S is f32 and stays in registers throughout a portion.  Everything is
+// 32-bit arithmetic whatever the activation dtype; the scan's products run on the f32 pipes in all-32-bit contexts, and as three
+// tf32 products each (21 bits of both factors, f32 sums) on tensor cores otherwise.
 //
 // Rounds with several tokens per request take three launches (convolutions, gates and triangles / the scan / norm and output
 // gate), rounds of one token per request a single one.  The inputs of the convolutions that a later round needs are
@@ -146,12 +147,13 @@ __device__ __forceinline__ void conv_block(const DeltaArgs &a, const ConvIn &in,
     }
 }
 
+constexpr int DP_WARPS = 4;
 template <int TAPS>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(DP_WARPS * 32, 4) delta_prep_kernel(const DeltaArgs a) {
     extern __shared__ __align__(16) float sm[];
     grid_dep_launch();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    int item = blockIdx.x * 8 + warp;
+    int item = blockIdx.x * DP_WARPS + warp;
     if (item >= a.kv_heads + a.heads) return;
     const int4 blk = a.blocks[blockIdx.y];  // request, first token, tokens, slot of the coefficients
     const int t0 = blk.y, count = blk.z;
@@ -416,6 +418,174 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
         for (int i = 0; i < R / 2; ++i) *reinterpret_cast<float2 *>(st + (size_t)c * DK + 32 * i) = up2(s[i][c]);
 }
 
+// ---- the same on tensor cores, for contexts whose activations are bf16
+// Every product of two f32 numbers is made of three tf32 products (x = hi + lo to 21 bits; the product of both low parts is left
+// out), summed in f32.  A group of 16 value columns belongs to DT_PARTS warps, each with its part of the key dimension: KW tiles
+// of eight.  All matrices are kept transposed (value columns are the rows), so that the accumulator of one product IS the first
+// operand of the next: a lane's accumulator pair (row, 2 t), (row, 2 t + 1) goes into the operand's slots t and t + 4, and the
+// other operand is read in the same order.  Dot products of the parts are summed through shared memory, once per block.
+constexpr int DT_PARTS = 4;
+
+__device__ __forceinline__ uint32_t tf32_hi(float x) {
+    uint32_t r;
+    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
+    return r;
+}
+__device__ __forceinline__ void tf32_split(float x, uint32_t &hi, uint32_t &lo) {
+    hi = tf32_hi(x);
+    lo = __float_as_uint(x - __uint_as_float(hi));
+}
+__device__ __forceinline__ void mma1688(float c[4], const uint32_t a[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// accumulator layout -> operand slots, split
+__device__ __forceinline__ void tf32_operand(const float c[4], uint32_t hi[4], uint32_t lo[4]) {
+    tf32_split(c[0], hi[0], lo[0]);
+    tf32_split(c[2], hi[1], lo[1]);
+    tf32_split(c[1], hi[2], lo[2]);
+    tf32_split(c[3], hi[3], lo[3]);
+}
+
+template <int KW>
+__global__ void __launch_bounds__(256) delta_scan_tc_kernel(const DeltaArgs a) {
+    constexpr int DK = 8 * KW * DT_PARTS, LD = DK + 8;  // padded rows: operand reads meet 32 banks
+    extern __shared__ __align__(16) float sm[];
+    __shared__ __align__(16) float s_part[2][DT_PARTS][32][8];
+    grid_dep_launch();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int part = warp % DT_PARTS, cg = warp / DT_PARTS;  // part of the key dimension, group of columns
+    const int h = blockIdx.y, r = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
+    const int cols = (blockDim.x >> 5) / DT_PARTS * 16, ldv = cols + 4, col0 = blockIdx.x * cols, col = col0 + 16 * cg;
+    const bool valid = col < a.dv_p;
+    const int stage = 2 * DB * LD + DB * ldv + DELTA_COEF;
+    const int first = a.req_first[r], end = a.req_first[r + 1], n_blk = (end - first + DB - 1) / DB;
+    const size_t slot0 = first / DB + r;
+    const int d0 = part * KW * 8;  // first key dimension of this warp
+    float *st = a.state + (((size_t)(a.req_slot[r] >> 1) * a.heads + h) * a.dv_p + (valid ? col + g : 0)) * DK + d0 + 2 * t;
+    const bool fresh = a.req_pos[r] == 0;
+    float s[KW][4];
+#pragma unroll
+    for (int k = 0; k < KW; ++k) {
+        const float2 x = valid && !fresh ? *reinterpret_cast<const float2 *>(st + 8 * k) : make_float2(0.f, 0.f);
+        const float2 y = valid && !fresh ? *reinterpret_cast<const float2 *>(st + (size_t)8 * DK + 8 * k) : make_float2(0.f, 0.f);
+        s[k][0] = x.x; s[k][1] = x.y; s[k][2] = y.x; s[k][3] = y.y;
+    }
+    grid_dep_wait();
+    const int vch = min(cols, a.dv_p - col0) / 4;  // 16-byte pieces of a value row
+    auto load = [&](int b) {
+        float *dst = sm + (size_t)(b % DS_STAGES) * stage;
+        const int t0 = first + b * DB;
+        for (int i = tid; i < DB * (DK / 4); i += blockDim.x) {
+            const int j = i / (DK / 4), c = 4 * (i % (DK / 4));
+            const bool ok = t0 + j < end;
+            const size_t off = ((size_t)(ok ? t0 + j : first) * a.kv_heads + kvh) * DK + c;
+            ds_cp16(dst + j * LD + c, a.k + off, ok);
+            ds_cp16(dst + (DB + j) * LD + c, a.q + off, ok);
+        }
+        float *dv = dst + 2 * DB * LD;
+        if (tid < DB * 8) {
+            const int j = tid >> 3, c = tid & 7;
+            const bool ok = t0 + j < end && c < vch;
+            if (4 * c < cols) ds_cp16(dv + j * ldv + 4 * c, a.v + ((size_t)(ok ? t0 + j : first) * a.heads + h) * a.dv_p + (ok ? col0 + 4 * c : 0), ok);
+        } else if (tid - DB * 8 < DELTA_COEF / 4) {
+            const int i = tid - DB * 8;
+            ds_cp16(dv + DB * ldv + 4 * i, a.coef + ((slot0 + b) * a.heads + h) * DELTA_COEF + 4 * i, true);
+        }
+    };
+#pragma unroll
+    for (int b = 0; b < DS_STAGES - 1; ++b) {
+        if (b < n_blk) load(b);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    for (int b = 0; b < n_blk; ++b) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(DS_STAGES - 2) : "memory");
+        __syncthreads();  // block b has landed, block b - 1 has been read
+        if (b + DS_STAGES - 1 < n_blk) load(b + DS_STAGES - 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const float *tile = sm + (size_t)(b % DS_STAGES) * stage, *tv = tile + 2 * DB * LD, *coef = tv + DB * ldv;
+
+        // products of the 16 columns with the eight keys (0) and the eight queries (1), this warp's key dimensions
+        float dot[2][4] = {}, low[2][4] = {};
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+            uint32_t hi[4], lo[4];
+            tf32_operand(s[k], hi, lo);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const float2 x = *reinterpret_cast<const float2 *>(tile + (n * DB + g) * LD + d0 + 8 * k + 2 * t);
+                uint32_t h0, l0, h1, l1;
+                tf32_split(x.x, h0, l0);
+                tf32_split(x.y, h1, l1);
+                mma1688(dot[n], hi, h0, h1);
+                mma1688(low[n], hi, l0, l1);
+                mma1688(low[n], lo, h0, h1);
+            }
+        }
+        float4 *mine = reinterpret_cast<float4 *>(s_part[cg][part][lane]);
+        mine[0] = make_float4(dot[0][0] + low[0][0], dot[0][1] + low[0][1], dot[0][2] + low[0][2], dot[0][3] + low[0][3]);
+        mine[1] = make_float4(dot[1][0] + low[1][0], dot[1][1] + low[1][1], dot[1][2] + low[1][2], dot[1][3] + low[1][3]);
+        const float2 upto = *reinterpret_cast<const float2 *>(coef + 2 * DB * DB + 2 * t), rest = *reinterpret_cast<const float2 *>(coef + 2 * DB * DB + DB + 2 * t);
+        const float total = coef[2 * DB * DB + DB - 1];
+        const float *vp = tv + 2 * t * ldv + 16 * cg + g;
+        float w[4] = {vp[0], vp[ldv], vp[8], vp[ldv + 8]};  // values of columns g, g + 8 at tokens 2 t, 2 t + 1
+        asm volatile("bar.sync %0, %1;" ::"r"(1 + cg), "n"(32 * DT_PARTS) : "memory");
+        float dk[4] = {}, y[4] = {};
+#pragma unroll
+        for (int i = 0; i < DT_PARTS; ++i) {
+            const float4 *src = reinterpret_cast<const float4 *>(s_part[cg][i][lane]);
+            const float4 u = src[0], v = src[1];
+            dk[0] += u.x; dk[1] += u.y; dk[2] += u.z; dk[3] += u.w;
+            y[0] += v.x; y[1] += v.y; y[2] += v.z; y[3] += v.w;
+        }
+        w[0] -= upto.x * dk[0]; w[1] -= upto.y * dk[1]; w[2] -= upto.x * dk[2]; w[3] -= upto.y * dk[3];
+        y[0] *= upto.x; y[1] *= upto.y; y[2] *= upto.x; y[3] *= upto.y;
+        float u[4] = {};
+        {
+            uint32_t hi[4], lo[4], h0, l0, h1, l1;
+            tf32_operand(w, hi, lo);
+            const float2 x = *reinterpret_cast<const float2 *>(coef + g * DB + 2 * t), z = *reinterpret_cast<const float2 *>(coef + (DB + g) * DB + 2 * t);
+            tf32_split(x.x, h0, l0);
+            tf32_split(x.y, h1, l1);
+            mma1688(u, lo, h0, h1);
+            mma1688(u, hi, l0, l1);
+            mma1688(u, hi, h0, h1);
+            tf32_split(z.x, h0, l0);
+            tf32_split(z.y, h1, l1);
+            mma1688(y, lo, h0, h1);
+            mma1688(y, hi, l0, l1);
+            mma1688(y, hi, h0, h1);
+        }
+        {  // every warp of the group has all outputs: each stores a quarter, (column g or g + 8, token 2 t or 2 t + 1)
+            const int tok = first + b * DB + 2 * t + (part & 1), c = col + g + (part >> 1) * 8;
+            const float out = part == 0 ? y[0] : (part == 1 ? y[1] : (part == 2 ? y[2] : y[3]));
+            if (valid && tok < end) a.v[((size_t)tok * a.heads + h) * a.dv_p + c] = out;
+        }
+        u[0] *= rest.x; u[1] *= rest.y; u[2] *= rest.x; u[3] *= rest.y;
+        uint32_t uh[4], ul[4];
+        tf32_operand(u, uh, ul);
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+            const float *kp = tile + 2 * t * LD + d0 + 8 * k + g;
+            uint32_t h0, l0, h1, l1;
+            tf32_split(kp[0], h0, l0);
+            tf32_split(kp[LD], h1, l1);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[k][e] *= total;
+            mma1688(s[k], ul, h0, h1);
+            mma1688(s[k], uh, l0, l1);
+            mma1688(s[k], uh, h0, h1);
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (!valid) return;
+#pragma unroll
+    for (int k = 0; k < KW; ++k) {
+        *reinterpret_cast<float2 *>(st + 8 * k) = make_float2(s[k][0], s[k][1]);
+        *reinterpret_cast<float2 *>(st + (size_t)8 * DK + 8 * k) = make_float2(s[k][2], s[k][3]);
+    }
+}
+
 // ------------------------------------------------------------------ portions: norm and output gate, a warp per (token, head)
 template <class T>
 __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs a) {
@@ -556,24 +726,27 @@ int by_dk(int dk_p, const F &f) {
 
 struct ScanLaunch {
     const DeltaArgs &a;
+    int dt;
     cudaStream_t s;
     bool pdl;
-    template <int R, int NC> int launch(int warps) const {
-        const int cols = warps * 2 * NC;
-        const size_t smem = (size_t)DS_STAGES * (2 * DB * 16 * R + DB * cols + DELTA_COEF) * 4;
+    template <class K> int launch(K kernel, int cols, int threads, int ld, int ldv) const {
+        const size_t smem = (size_t)DS_STAGES * (2 * DB * ld + DB * ldv + DELTA_COEF) * 4;
         const dim3 grid((a.dv_p + cols - 1) / cols, a.heads, a.n_req);
-        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(delta_scan_kernel<R, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        LCU_CHECK_CUDA(launch_kernel(delta_scan_kernel<R, NC>, grid, dim3(warps * 32), smem, s, pdl, a));
+        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(threads), smem, s, pdl, a));
         return LCU_OK;
     }
     template <int R8> int run() const {
-        constexpr int R = R8 / 2;  // key dimensions per lane of a half warp
-        // columns per half warp: four where that leaves a warp for every scheduler, two otherwise
-        const long groups = (long)a.n_req * a.heads * ((a.dv_p + 15) / 16);
-        if constexpr (R <= 8) {
-            if (tuning().delta_cols == 4 || (tuning().delta_cols == 0 && groups * 2 >= 3l * sm_count())) return launch<R, 4>(a.dv_p > 16 ? 4 : 2);
+        constexpr int DK = 8 * R8;
+        if (dt != LCU_F32 && tuning().delta_tc) {
+            // two groups of columns share a CTA's tiles where one group each would not fit the SMs at once
+            const int groups = a.dv_p > 16 && (long)a.n_req * a.heads * (a.dv_p / 16) > sm_count() ? 2 : 1;
+            return launch(delta_scan_tc_kernel<DK / 8 / DT_PARTS>, 16 * groups, 32 * DT_PARTS * groups, DK + 8, 16 * groups + 4);
         }
-        return launch<R, 2>(4);
+        constexpr int NC = DK <= 128 ? 4 : 2;  // columns per half warp
+        int warps = (a.dv_p + 2 * NC - 1) / (2 * NC);
+        if (warps > 4) warps = 4;
+        return launch(delta_scan_kernel<DK / 16, NC>, warps * 2 * NC, warps * 32, DK, warps * 2 * NC);
     }
 };
 struct DecodeLaunch {
@@ -596,11 +769,11 @@ struct DecodeLaunch {
 int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
     if (a.n_blocks <= 0) return LCU_OK;
     LCU_REQUIRE(a.n_blocks <= 65535 && a.dk_p <= MIX_MAX_HEAD && a.dv_p <= MIX_MAX_HEAD, "delta rule: %d blocks, head sizes %d / %d", a.n_blocks, a.dk_p, a.dv_p);
-    const dim3 grid((a.kv_heads + a.heads + 7) / 8, a.n_blocks);
-    const size_t smem = (size_t)8 * (2 * DB * (a.dk_p + 4) + 2 * DB * DB) * 4;
+    const dim3 grid((a.kv_heads + a.heads + DP_WARPS - 1) / DP_WARPS, a.n_blocks);
+    const size_t smem = (size_t)DP_WARPS * (2 * DB * (a.dk_p + 4) + 2 * DB * DB) * 4;
     auto go = [&](auto kernel) -> int {
         if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(256), smem, s, pdl, a));
+        LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(DP_WARPS * 32), smem, s, pdl, a));
         return LCU_OK;
     };
     switch (a.taps) {
@@ -610,10 +783,10 @@ int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
     default: return go(delta_prep_kernel<0>);
     }
 }
-int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
+int delta_scan_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_req <= 0) return LCU_OK;
     LCU_REQUIRE(a.n_req <= 65535 && a.heads <= 65535, "delta rule: grid out of range");
-    return by_dk(a.dk_p, ScanLaunch{a, s, pdl});
+    return by_dk(a.dk_p, ScanLaunch{a, dt, s, pdl});
 }
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_tok <= 0) return LCU_OK;

@@ -84,7 +84,7 @@ struct DeltaArgs {
 };
 // Rounds with several tokens per request: convolutions, gates and triangles; the scan; norm and output gate.
 int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
-int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
+int delta_scan_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
 // Rounds of one token per request: all of it in one launch, beside the attention's preparation (nullptr: none).
 int delta_decode_launch(const DeltaArgs &a, const GqaArgs *attn, int dt, cudaStream_t s, bool pdl);

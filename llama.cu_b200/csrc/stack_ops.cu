@@ -104,8 +104,8 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     const int t = blockIdx.x, n4 = a.d_p / 4;
     __shared__ float2 part[32], part2[32];
     const size_t row = (size_t)t * a.d_p;
-    const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;
     grid_dep_wait();
+    const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;  // fed-back tokens are written by the kernel before the round's first one
     float4 x[MAXV], y0[MAXV], y1[MAXV];
     float s0 = 0.f, s1 = 0.f;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);

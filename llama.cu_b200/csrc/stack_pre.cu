@@ -106,7 +106,7 @@ struct PreNormRound {
         } else {
             if (!rc && Y.attention()) rc = done(gqa_prep_launch(g, dt, s, L.pdl));
             if (!rc && Y.delta()) rc = done(delta_prep_launch(e, s, L.pdl));
-            if (!rc && Y.delta()) rc = done(delta_scan_launch(e, s, L.pdl));
+            if (!rc && Y.delta()) rc = done(delta_scan_launch(e, dt, s, L.pdl));
             if (!rc && Y.delta()) rc = done(delta_out_launch(e, dt, s, L.pdl));
         }
         if (!rc && Y.attention()) rc = attention(g, Y);

@@ -56,6 +56,14 @@ def reference(raw, w, tokens, keep_layers=False):
     return G.forward(raw, w, list(tokens), torch.float64, keep_layers)
 
 
+def tolerance(dt, raw, w, toks, want=None):
+    """What a bf16 run may differ by: three times what rounding the inputs of the matrix products changes in the restatement."""
+    if dt == 2:
+        return TOL[dt]
+    want = reference(raw, w, toks) if want is None else want
+    return max(TOL[dt], 3 * rel_err(G.forward(raw, w, list(toks), torch.float64, operand=torch.bfloat16), want))
+
+
 def silence(w, raw, *what):
     """Weights with mechanisms switched off in every layer: "left" or "right" (gain on that mixer's output), "ff"."""
     w = dict(w)

@@ -8,6 +8,17 @@ import math
 import torch
 
 
+_operand = None  # dtype that inputs of matrix products are rounded to (`forward` sets it); None: not at all
+
+
+def rounded(x):
+    return x if _operand is None else x.to(_operand).to(x.dtype)
+
+
+def linear(x, w):
+    return rounded(x) @ w.T
+
+
 def rms(x, eps):
     """x / sqrt(mean(x^2) + eps) over the last axis."""
     return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
@@ -60,7 +71,7 @@ def rotate(x, rot):
 
 def attention_inputs(h, w, pre, m, eps):
     n = h.shape[0]
-    q, k, v = (h @ w[pre + t].T + w[pre + t + ".b"] for t in "qkv")
+    q, k, v = (linear(h, w[pre + t]) + w[pre + t + ".b"] for t in "qkv")
     q, k, v = q.view(n, m["heads"], m["dim"]), k.view(n, m["kv_heads"], m["dim"]), v.view(n, m["kv_heads"], m["vdim"])
     return rms(rotate(q, m["rot"]), eps), rms(rotate(k, m["rot"]), eps), v
 
@@ -69,14 +80,14 @@ def causal_attention(q, k, v, scale):
     """[tokens, heads, vdim]; query head h reads key head h // (heads / kv_heads)."""
     n, reps = q.shape[0], q.shape[1] // k.shape[1]
     k, v = k.repeat_interleave(reps, 1), v.repeat_interleave(reps, 1)
-    s = torch.einsum("qhd,khd->hqk", q, k) * scale
+    s = torch.einsum("qhd,khd->hqk", rounded(q), rounded(k)) * scale
     s = s.masked_fill(~torch.ones(n, n, dtype=torch.bool).tril(), -math.inf)
-    return torch.einsum("hqk,khd->qhd", torch.softmax(s, -1), v)
+    return torch.einsum("hqk,khd->qhd", rounded(torch.softmax(s, -1)), rounded(v))
 
 
 def left(h, w, pre, m, eps):
     q, k, v = attention_inputs(h, w, pre, m, eps)
-    return causal_attention(q, k, v, m["scale"]).reshape(h.shape[0], -1) @ w[pre + "o"].T
+    return linear(causal_attention(q, k, v, m["scale"]).reshape(h.shape[0], -1), w[pre + "o"])
 
 
 # ---- gated delta rule
@@ -96,11 +107,11 @@ def delta_inputs(h, w, pre, m):
     """q, k [tokens, heads, dim] (repeated for the heads that share them), v [tokens, heads, vdim], decay and step size
     [tokens, heads]."""
     n, reps = h.shape[0], m["heads"] // m["kv_heads"]
-    q, k, v = (silu(causal_conv(h @ w[pre + t].T, w[pre + t + ".conv"])) for t in "qkv")
+    q, k, v = (silu(causal_conv(linear(h, w[pre + t]), w[pre + t + ".conv"])) for t in "qkv")
     q = unit(q.view(n, m["kv_heads"], m["dim"])) * m["dim"] ** -0.5
     k = unit(k.view(n, m["kv_heads"], m["dim"]))
-    decay = torch.exp(-torch.exp(w[pre + "A_log"]) * softplus(h @ w[pre + "a"].T + w[pre + "dt_bias"]))
-    beta = torch.sigmoid(h @ w[pre + "b"].T)
+    decay = torch.exp(-torch.exp(w[pre + "A_log"]) * softplus(linear(h, w[pre + "a"]) + w[pre + "dt_bias"]))
+    beta = torch.sigmoid(linear(h, w[pre + "b"]))
     return q.repeat_interleave(reps, 1), k.repeat_interleave(reps, 1), v.view(n, m["heads"], m["vdim"]), decay, beta
 
 
@@ -118,8 +129,8 @@ def delta_rule(q, k, v, decay, beta):
 
 def right(h, w, pre, m, eps):
     o = delta_rule(*delta_inputs(h, w, pre, m))
-    o = rms(o, eps) * w[pre + "norm"] * silu(h @ w[pre + "g"].T).view(o.shape)
-    return o.reshape(h.shape[0], -1) @ w[pre + "o"].T
+    o = rms(o, eps) * w[pre + "norm"] * silu(linear(h, w[pre + "g"])).view(o.shape)
+    return linear(o.reshape(h.shape[0], -1), w[pre + "o"])
 
 
 def parallel(h, w, pre, m, eps):
@@ -130,7 +141,7 @@ def parallel(h, w, pre, m, eps):
 # ---- model
 
 def feed_forward(h, w, pre):
-    return torch.relu(h @ w[pre + "up"].T).square() @ w[pre + "down"].T
+    return linear(torch.relu(linear(h, w[pre + "up"])).square(), w[pre + "down"])
 
 
 def layer(x, raw, w, i):
@@ -153,8 +164,18 @@ def schedule(raw):
     return runs + [(i, None) for i in range(b, n)]
 
 
-def forward(raw, weights, tokens, dtype=torch.float64, keep_layers=False):
-    """Logits [tokens, vocab]; with keep_layers also the residual stream after every layer run."""
+def forward(raw, weights, tokens, dtype=torch.float64, keep_layers=False, operand=None):
+    """Logits [tokens, vocab]; with keep_layers also the residual stream after every layer run.  operand: the dtype that inputs of
+    matrix products are rounded to -- what rounding alone changes, to set a tolerance by."""
+    global _operand
+    _operand = operand
+    try:
+        return _forward(raw, weights, tokens, dtype, keep_layers)
+    finally:
+        _operand = None
+
+
+def _forward(raw, weights, tokens, dtype, keep_layers):
     w = {k: v.to(dtype) for k, v in weights.items()}
     first = x = w["embed"][torch.tensor(list(tokens))]
     kept = []
@@ -164,5 +185,5 @@ def forward(raw, weights, tokens, dtype=torch.float64, keep_layers=False):
             x = x + w["loop.step"][t]
         x = layer(x, raw, w, i)
         kept.append(x)
-    logits = centred_norm(x, w["final.norm"], raw["norm"]["eps"]) @ w["head"].T
+    logits = linear(centred_norm(x, w["final.norm"], raw["norm"]["eps"]), w["head"])
     return (logits, torch.stack(kept)) if keep_layers else logits

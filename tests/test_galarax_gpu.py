@@ -19,13 +19,13 @@ BF16, F32 = 1, 2
 @pytest.fixture(autouse=True)
 def default_tuning(L):
     yield
-    for k, v in (("stack_pdl", 1), ("stack_fuse", 1), ("stack_tc", 1), ("delta_cols", 0), ("tc_block", 256)):
+    for k, v in (("stack_pdl", 1), ("stack_fuse", 1), ("stack_tc", 1), ("delta_tc", 1), ("tc_block", 256)):
         L.set_tuning(k, v)
 
 
-def check(got, want, dt, what=""):
-    e = M.rel_err(got, want)
-    assert e <= M.TOL[dt], f"{what}: error {e:.3g} > {M.TOL[dt]}"
+def check(got, want, dt, what="", tol=None):
+    e, tol = M.rel_err(got, want), tol or M.TOL[dt]
+    assert e <= tol, f"{what}: error {e:.3g} > {tol:.3g}"
     return e
 
 
@@ -163,9 +163,10 @@ def test_sizes(L, name, dt):
     want = M.reference(raw, w, toks)
     _, ctx = M.load(L, raw, w, dt)
     r = M.Runner(ctx)
-    check(r.whole(toks), want, dt, "whole")
-    check(r.whole(toks, [120] + [1] * 30), want, dt, "decoded")
-    check(r.whole(toks, [2, 64, 3, 17]), want, dt, "portions")
+    tol = M.tolerance(dt, raw, w, toks, want)
+    check(r.whole(toks), want, dt, "whole", tol)
+    check(r.whole(toks, [120] + [1] * 30), want, dt, "decoded", tol)
+    check(r.whole(toks, [2, 64, 3, 17]), want, dt, "portions", tol)
     assert ctx.device_status() == 0 and ctx.pages_free == ctx.pages_total
     ctx.close()
 
@@ -262,7 +263,7 @@ def test_slots_and_pages_carry_nothing_over(L, dt):
     ctx.close()
 
 
-@pytest.mark.parametrize("key,value", [("stack_pdl", 0), ("stack_fuse", 0), ("stack_fuse", 2), ("stack_tc", 0), ("stack_tc", 2), ("tc_block", 64), ("delta_cols", 2), ("delta_cols", 4)])
+@pytest.mark.parametrize("key,value", [("stack_pdl", 0), ("stack_fuse", 0), ("stack_fuse", 2), ("stack_tc", 0), ("stack_tc", 2), ("tc_block", 64), ("delta_tc", 0)])
 def test_every_form_of_a_round(L, key, value):
     """The alternatives behind the tuning keys compute the same: prompts, then one to four requests decode together."""
     raw = M.config([M.layer(heads=20, kv_heads=5, d_dim=64, d_vdim=64), M.layer(ff=0), M.layer()], loop=(0, 2, 2))
@@ -397,10 +398,11 @@ def test_decays_from_none_to_complete(L, dt, decay):
             w[k] = torch.full_like(w[k], decay)
     toks = M.random_tokens(raw, 90, 94)
     want = M.reference(raw, w, toks)
+    tol = M.tolerance(dt, raw, w, toks, want)
     for cuts in (None, [1], [30]):
         got = whole(L, raw, w, toks, dt, cuts)
         assert torch.isfinite(got).all()
-        check(got, want, dt, f"decay {decay}, portions {cuts}")
+        check(got, want, dt, f"decay {decay}, portions {cuts}", tol)
 
 
 def test_repeated_keys_with_full_steps(L):
@@ -432,21 +434,24 @@ def greedy(raw, w, prompt, steps):
 @pytest.mark.parametrize("graph", [True, False])
 @pytest.mark.parametrize("dt", [F32, BF16])
 def test_greedy_generation(L, dt, graph):
-    raw = M.MIXED
+    raw = M.config([M.layer(), M.layer(heads=6, kv_heads=2, dim=36, conv=3, ff=0), M.layer(d_heads=3, d_kv_heads=1)], loop=(1, 3, 2))
     w = M.weights(raw, 101)
     prompts = [M.random_tokens(raw, n, 110 + n) for n in (5, 70, 1, 33)]
     want = [greedy(raw, w, p, 10) for p in prompts]
+    # a bf16 run may take the other of two tokens whose logits rounding can swap
+    near = [4 * M.tolerance(dt, raw, w, p + ids) if dt == BF16 else 0 for p, (ids, _) in zip(prompts, want)]
     _, ctx = M.load(L, raw, w, dt, tokens=1024, max_seqs=8)
     ctx.set_cuda_graph(graph)
 
     def compare(got):
-        for g, (ids, margins) in zip(got, want):
+        for g, (ids, margins), limit in zip(got, want, near):
             for a, b, m in zip(g, ids, margins):
                 if a != b:
-                    assert dt == BF16 and m < 0.1, (g, ids, m)
+                    assert m < limit, (g, ids, m, limit)
                     break
-    compare(L.generate(ctx, [np.array(p, np.uint32) for p in prompts], 10))
-    compare(L.generate_continuous(ctx, [np.array(p, np.uint32) for p in prompts], 10, max_round_tokens=24, prefill_chunk=16))
+    for _ in range(3):  # rounds that follow one another without a pause
+        compare(L.generate(ctx, [np.array(p, np.uint32) for p in prompts], 10))
+        compare(L.generate_continuous(ctx, [np.array(p, np.uint32) for p in prompts], 10, max_round_tokens=24, prefill_chunk=16))
     assert ctx.pages_free == ctx.pages_total and ctx.device_status() == 0
     ctx.close()
 
