@@ -12,8 +12,8 @@
 // The preparation solves for T and B T of every block in parallel; the scan then needs one pass of dot products with S, one
 // eight-term sum per token and one pass of updates, with a single reduction across lanes per block.  All decays are products of
 // numbers up to one: nothing is divided by a decay.  S is f32 and stays in registers throughout a portion.  Everything is
-// 32-bit arithmetic whatever the activation dtype; the scan's products run on the f32 pipes in all-32-bit contexts, and as three
-// tf32 products each (21 bits of both factors, f32 sums) on tensor cores otherwise.
+// 32-bit arithmetic whatever the activation dtype; the scan's products run on the f32 pipes in all-32-bit contexts, and on
+// tensor cores with factors of three bf16 numbers (24 bits, f32 sums) otherwise.
 //
 // Rounds with several tokens per request take three launches (convolutions, gates and triangles / the scan / norm and output
 // gate), rounds of one token per request a single one.  The inputs of the convolutions that a later round needs are
@@ -49,6 +49,24 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
     f32x2 r;
     asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
     return r;
+}
+
+// Two f32 numbers as sums of three bf16 ones (24 bits): planes[0] + planes[1] + planes[2], two numbers per word.
+__device__ __forceinline__ void split3(float x, float y, uint32_t planes[3]) {
+#pragma unroll
+    for (int i = 0; i < 3; ++i) {
+        planes[i] = Act<bf16>::pack(x, y);
+        const float2 v = Act<bf16>::to_f2(planes[i]);
+        x -= v.x;
+        y -= v.y;
+    }
+}
+__device__ __forceinline__ void store_split4(void *row, int dk, int d, const float4 &v) {  // row: [3][dk] bf16
+    uint32_t a[3], b[3];
+    split3(v.x, v.y, a);
+    split3(v.z, v.w, b);
+#pragma unroll
+    for (int i = 0; i < 3; ++i) *reinterpret_cast<uint2 *>(reinterpret_cast<bf16 *>(row) + (size_t)i * dk + d) = make_uint2(a[i], b[i]);
 }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
@@ -195,9 +213,14 @@ __global__ void __launch_bounds__(DP_WARPS * 32, 4) delta_prep_kernel(const Delt
                 *reinterpret_cast<float4 *>(qs + i * ld + d) = x;
                 *reinterpret_cast<float4 *>(ks + i * ld + d) = y;
                 if (i < count) {
-                    const size_t at = ((size_t)(t0 + i) * a.kv_heads + item) * a.dk_p + d;
-                    *reinterpret_cast<float4 *>(a.q + at) = x;
-                    *reinterpret_cast<float4 *>(a.k + at) = y;
+                    const size_t at = ((size_t)(t0 + i) * a.kv_heads + item) * a.dk_p;
+                    if (a.split) {
+                        store_split4(reinterpret_cast<bf16 *>(a.q) + 3 * at, a.dk_p, d, x);
+                        store_split4(reinterpret_cast<bf16 *>(a.k) + 3 * at, a.dk_p, d, y);
+                    } else {
+                        *reinterpret_cast<float4 *>(a.q + at + d) = x;
+                        *reinterpret_cast<float4 *>(a.k + at + d) = y;
+                    }
                 }
             }
         }
@@ -419,38 +442,62 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
 }
 
 // ---- the same on tensor cores, for contexts whose activations are bf16
-// Every product of two f32 numbers is made of three tf32 products (x = hi + lo to 21 bits; the product of both low parts is left
-// out), summed in f32.  A group of 16 value columns belongs to DT_PARTS warps, each with its part of the key dimension: KW tiles
-// of eight.  All matrices are kept transposed (value columns are the rows), so that the accumulator of one product IS the first
-// operand of the next: a lane's accumulator pair (row, 2 t), (row, 2 t + 1) goes into the operand's slots t and t + 4, and the
-// other operand is read in the same order.  Dot products of the parts are summed through shared memory, once per block.
+// Every f32 factor is the sum of three bf16 numbers (24 bits); a product is the six largest of their nine products, summed in
+// f32.  A group of 16 value columns belongs to DT_PARTS warps, each with its part of the key dimension: KW tiles of eight.  All
+// matrices are kept transposed (value columns are the rows), so that the accumulator of one product IS, pair by pair, the first
+// operand of the next.  Keys and queries come split from the preparation.  Dot products of the parts are summed through shared
+// memory, once per block.
 constexpr int DT_PARTS = 4;
 
-__device__ __forceinline__ uint32_t tf32_hi(float x) {
-    uint32_t r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
-    return r;
+__device__ __forceinline__ void dt_mma16(float c[4], const uint32_t a[2], const uint32_t a2[2], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a2[0]), "r"(a2[1]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void tf32_split(float x, uint32_t &hi, uint32_t &lo) {
-    hi = tf32_hi(x);
-    lo = __float_as_uint(x - __uint_as_float(hi));
+__device__ __forceinline__ void dt_mma8(float c[4], const uint32_t a[2], uint32_t b) {
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5}, {%6}, {%0,%1,%2,%3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(b));
 }
-__device__ __forceinline__ void mma1688(float c[4], const uint32_t a[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+// accumulator -> first operand (rows g and g + 8, columns 2 t and 2 t + 1), split: [plane][row half]
+__device__ __forceinline__ void dt_operand(const float c[4], uint32_t a[3][2]) {
+    uint32_t x[3], y[3];
+    split3(c[0], c[1], x);
+    split3(c[2], c[3], y);
+#pragma unroll
+    for (int i = 0; i < 3; ++i) { a[i][0] = x[i]; a[i][1] = y[i]; }
 }
-// accumulator layout -> operand slots, split
-__device__ __forceinline__ void tf32_operand(const float c[4], uint32_t hi[4], uint32_t lo[4]) {
-    tf32_split(c[0], hi[0], lo[0]);
-    tf32_split(c[2], hi[1], lo[1]);
-    tf32_split(c[1], hi[2], lo[2]);
-    tf32_split(c[3], hi[3], lo[3]);
+__device__ __forceinline__ void dt_mma8x6(float c[4], const uint32_t a[3][2], const uint32_t b[3]) {  // smallest products first
+    dt_mma8(c, a[1], b[1]);
+    dt_mma8(c, a[0], b[2]);
+    dt_mma8(c, a[2], b[0]);
+    dt_mma8(c, a[0], b[1]);
+    dt_mma8(c, a[1], b[0]);
+    dt_mma8(c, a[0], b[0]);
+}
+// tiles [0, KW) of 8 x 8 at `row` (this lane's row of a tile), 16 bytes apart
+template <int KW, bool TRANS>
+__device__ __forceinline__ void dt_tiles(uint32_t *dst, const unsigned char *row, int lane) {
+#pragma unroll
+    for (int k = 0; k < KW; k += 4) {
+        const int tile = min(k + (lane >> 3), KW - 1);
+        const unsigned at = (unsigned)__cvta_generic_to_shared(row + tile * 16);
+        uint32_t r[4];
+        if constexpr (TRANS) asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+        else asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (k + i < KW) dst[k + i] = r[i];
+    }
+}
+__device__ __forceinline__ void dt_cp16(unsigned char *smem_dst, const void *src, bool valid) {
+    unsigned d = (unsigned)__cvta_generic_to_shared(smem_dst);
+    int sz = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(sz) : "memory");
 }
 
 template <int KW>
 __global__ void __launch_bounds__(256) delta_scan_tc_kernel(const DeltaArgs a) {
-    constexpr int DK = 8 * KW * DT_PARTS, LD = DK + 8;  // padded rows: operand reads meet 32 banks
-    extern __shared__ __align__(16) float sm[];
+    constexpr int DK = 8 * KW * DT_PARTS, RB = 6 * DK + 16;  // bytes of a token's row of planes, padded against bank conflicts
+    extern __shared__ __align__(16) unsigned char smb[];
     __shared__ __align__(16) float s_part[2][DT_PARTS][32][8];
     grid_dep_launch();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
@@ -458,7 +505,7 @@ __global__ void __launch_bounds__(256) delta_scan_tc_kernel(const DeltaArgs a) {
     const int h = blockIdx.y, r = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
     const int cols = (blockDim.x >> 5) / DT_PARTS * 16, ldv = cols + 4, col0 = blockIdx.x * cols, col = col0 + 16 * cg;
     const bool valid = col < a.dv_p;
-    const int stage = 2 * DB * LD + DB * ldv + DELTA_COEF;
+    const int stage = 2 * DB * RB + (DB * ldv + DELTA_COEF) * 4;
     const int first = a.req_first[r], end = a.req_first[r + 1], n_blk = (end - first + DB - 1) / DB;
     const size_t slot0 = first / DB + r;
     const int d0 = part * KW * 8;  // first key dimension of this warp
@@ -473,24 +520,26 @@ __global__ void __launch_bounds__(256) delta_scan_tc_kernel(const DeltaArgs a) {
     }
     grid_dep_wait();
     const int vch = min(cols, a.dv_p - col0) / 4;  // 16-byte pieces of a value row
+    const bf16 *kg = reinterpret_cast<const bf16 *>(a.k), *qg = reinterpret_cast<const bf16 *>(a.q);
     auto load = [&](int b) {
-        float *dst = sm + (size_t)(b % DS_STAGES) * stage;
+        unsigned char *dst = smb + (size_t)(b % DS_STAGES) * stage;
         const int t0 = first + b * DB;
-        for (int i = tid; i < DB * (DK / 4); i += blockDim.x) {
-            const int j = i / (DK / 4), c = 4 * (i % (DK / 4));
+        constexpr int CH = 3 * DK / 8;  // 16-byte pieces of a row of planes
+        for (int i = tid; i < DB * CH; i += blockDim.x) {
+            const int j = i / CH, c = i - j * CH;
             const bool ok = t0 + j < end;
-            const size_t off = ((size_t)(ok ? t0 + j : first) * a.kv_heads + kvh) * DK + c;
-            ds_cp16(dst + j * LD + c, a.k + off, ok);
-            ds_cp16(dst + (DB + j) * LD + c, a.q + off, ok);
+            const size_t off = ((size_t)(ok ? t0 + j : first) * a.kv_heads + kvh) * 3 * DK + 8 * c;
+            dt_cp16(dst + j * RB + 16 * c, kg + off, ok);
+            dt_cp16(dst + (DB + j) * RB + 16 * c, qg + off, ok);
         }
-        float *dv = dst + 2 * DB * LD;
+        unsigned char *dv = dst + 2 * DB * RB;
         if (tid < DB * 8) {
             const int j = tid >> 3, c = tid & 7;
             const bool ok = t0 + j < end && c < vch;
-            if (4 * c < cols) ds_cp16(dv + j * ldv + 4 * c, a.v + ((size_t)(ok ? t0 + j : first) * a.heads + h) * a.dv_p + (ok ? col0 + 4 * c : 0), ok);
+            if (4 * c < cols) dt_cp16(dv + (j * ldv + 4 * c) * 4, a.v + ((size_t)(ok ? t0 + j : first) * a.heads + h) * a.dv_p + (ok ? col0 + 4 * c : 0), ok);
         } else if (tid - DB * 8 < DELTA_COEF / 4) {
             const int i = tid - DB * 8;
-            ds_cp16(dv + DB * ldv + 4 * i, a.coef + ((slot0 + b) * a.heads + h) * DELTA_COEF + 4 * i, true);
+            dt_cp16(dv + (DB * ldv + 4 * i) * 4, a.coef + ((slot0 + b) * a.heads + h) * DELTA_COEF + 4 * i, true);
         }
     };
 #pragma unroll
@@ -503,78 +552,82 @@ __global__ void __launch_bounds__(256) delta_scan_tc_kernel(const DeltaArgs a) {
         __syncthreads();  // block b has landed, block b - 1 has been read
         if (b + DS_STAGES - 1 < n_blk) load(b + DS_STAGES - 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        const float *tile = sm + (size_t)(b % DS_STAGES) * stage, *tv = tile + 2 * DB * LD, *coef = tv + DB * ldv;
+        const unsigned char *tile = smb + (size_t)(b % DS_STAGES) * stage;
+        const float *tv = reinterpret_cast<const float *>(tile + 2 * DB * RB), *coef = tv + DB * ldv;
 
         // products of the 16 columns with the eight keys (0) and the eight queries (1), this warp's key dimensions
-        float dot[2][4] = {}, low[2][4] = {};
+        uint32_t x[2][3][KW];
 #pragma unroll
-        for (int k = 0; k < KW; ++k) {
-            uint32_t hi[4], lo[4];
-            tf32_operand(s[k], hi, lo);
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int i = 0; i < 3; ++i) dt_tiles<KW, false>(x[n][i], tile + (n * DB + (lane & 7)) * RB + (i * DK + d0) * 2, lane);
+        float dot[2][4] = {}, low[2][4] = {}, mid[2][4] = {};
+#pragma unroll
+        for (int k = 0; k < KW; k += 2) {
+            uint32_t s0[3][2], s1[3][2];
+            dt_operand(s[k], s0);
+            if (k + 1 < KW) dt_operand(s[k + 1 < KW ? k + 1 : k], s1);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                const float2 x = *reinterpret_cast<const float2 *>(tile + (n * DB + g) * LD + d0 + 8 * k + 2 * t);
-                uint32_t h0, l0, h1, l1;
-                tf32_split(x.x, h0, l0);
-                tf32_split(x.y, h1, l1);
-                mma1688(dot[n], hi, h0, h1);
-                mma1688(low[n], hi, l0, l1);
-                mma1688(low[n], lo, h0, h1);
+                auto mul = [&](float c[4], int i, int j) {
+                    if (k + 1 < KW) dt_mma16(c, s0[i], s1[i], x[n][j][k], x[n][j][k + 1 < KW ? k + 1 : k]);
+                    else dt_mma8(c, s0[i], x[n][j][k]);
+                };
+                mul(low[n], 1, 1);
+                mul(mid[n], 0, 1);
+                mul(dot[n], 0, 0);
+                mul(low[n], 0, 2);
+                mul(mid[n], 1, 0);
+                mul(low[n], 2, 0);
             }
         }
         float4 *mine = reinterpret_cast<float4 *>(s_part[cg][part][lane]);
-        mine[0] = make_float4(dot[0][0] + low[0][0], dot[0][1] + low[0][1], dot[0][2] + low[0][2], dot[0][3] + low[0][3]);
-        mine[1] = make_float4(dot[1][0] + low[1][0], dot[1][1] + low[1][1], dot[1][2] + low[1][2], dot[1][3] + low[1][3]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+            mine[n] = make_float4(dot[n][0] + (mid[n][0] + low[n][0]), dot[n][1] + (mid[n][1] + low[n][1]), dot[n][2] + (mid[n][2] + low[n][2]),
+                                  dot[n][3] + (mid[n][3] + low[n][3]));
         const float2 upto = *reinterpret_cast<const float2 *>(coef + 2 * DB * DB + 2 * t), rest = *reinterpret_cast<const float2 *>(coef + 2 * DB * DB + DB + 2 * t);
         const float total = coef[2 * DB * DB + DB - 1];
         const float *vp = tv + 2 * t * ldv + 16 * cg + g;
         float w[4] = {vp[0], vp[ldv], vp[8], vp[ldv + 8]};  // values of columns g, g + 8 at tokens 2 t, 2 t + 1
+        uint32_t tri[2][3];                                 // rows g of T and of B T at tokens 2 t, 2 t + 1
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const float2 z = *reinterpret_cast<const float2 *>(coef + (n * DB + g) * DB + 2 * t);
+            split3(z.x, z.y, tri[n]);
+        }
         asm volatile("bar.sync %0, %1;" ::"r"(1 + cg), "n"(32 * DT_PARTS) : "memory");
         float dk[4] = {}, y[4] = {};
 #pragma unroll
         for (int i = 0; i < DT_PARTS; ++i) {
             const float4 *src = reinterpret_cast<const float4 *>(s_part[cg][i][lane]);
-            const float4 u = src[0], v = src[1];
-            dk[0] += u.x; dk[1] += u.y; dk[2] += u.z; dk[3] += u.w;
-            y[0] += v.x; y[1] += v.y; y[2] += v.z; y[3] += v.w;
+            const float4 e = src[0], f = src[1];
+            dk[0] += e.x; dk[1] += e.y; dk[2] += e.z; dk[3] += e.w;
+            y[0] += f.x; y[1] += f.y; y[2] += f.z; y[3] += f.w;
         }
         w[0] -= upto.x * dk[0]; w[1] -= upto.y * dk[1]; w[2] -= upto.x * dk[2]; w[3] -= upto.y * dk[3];
         y[0] *= upto.x; y[1] *= upto.y; y[2] *= upto.x; y[3] *= upto.y;
         float u[4] = {};
-        {
-            uint32_t hi[4], lo[4], h0, l0, h1, l1;
-            tf32_operand(w, hi, lo);
-            const float2 x = *reinterpret_cast<const float2 *>(coef + g * DB + 2 * t), z = *reinterpret_cast<const float2 *>(coef + (DB + g) * DB + 2 * t);
-            tf32_split(x.x, h0, l0);
-            tf32_split(x.y, h1, l1);
-            mma1688(u, lo, h0, h1);
-            mma1688(u, hi, l0, l1);
-            mma1688(u, hi, h0, h1);
-            tf32_split(z.x, h0, l0);
-            tf32_split(z.y, h1, l1);
-            mma1688(y, lo, h0, h1);
-            mma1688(y, hi, l0, l1);
-            mma1688(y, hi, h0, h1);
-        }
+        uint32_t op[3][2];
+        dt_operand(w, op);
+        dt_mma8x6(u, op, tri[0]);
+        dt_mma8x6(y, op, tri[1]);
         {  // every warp of the group has all outputs: each stores a quarter, (column g or g + 8, token 2 t or 2 t + 1)
             const int tok = first + b * DB + 2 * t + (part & 1), c = col + g + (part >> 1) * 8;
             const float out = part == 0 ? y[0] : (part == 1 ? y[1] : (part == 2 ? y[2] : y[3]));
             if (valid && tok < end) a.v[((size_t)tok * a.heads + h) * a.dv_p + c] = out;
         }
         u[0] *= rest.x; u[1] *= rest.y; u[2] *= rest.x; u[3] *= rest.y;
-        uint32_t uh[4], ul[4];
-        tf32_operand(u, uh, ul);
+        dt_operand(u, op);
+        uint32_t kt[3][KW];
+#pragma unroll
+        for (int i = 0; i < 3; ++i) dt_tiles<KW, true>(kt[i], tile + (lane & 7) * RB + (i * DK + d0) * 2, lane);
 #pragma unroll
         for (int k = 0; k < KW; ++k) {
-            const float *kp = tile + 2 * t * LD + d0 + 8 * k + g;
-            uint32_t h0, l0, h1, l1;
-            tf32_split(kp[0], h0, l0);
-            tf32_split(kp[LD], h1, l1);
 #pragma unroll
             for (int e = 0; e < 4; ++e) s[k][e] *= total;
-            mma1688(s[k], ul, h0, h1);
-            mma1688(s[k], uh, l0, l1);
-            mma1688(s[k], uh, h0, h1);
+            const uint32_t kb[3] = {kt[0][k], kt[1][k], kt[2][k]};
+            dt_mma8x6(s[k], op, kb);
         }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -726,27 +779,26 @@ int by_dk(int dk_p, const F &f) {
 
 struct ScanLaunch {
     const DeltaArgs &a;
-    int dt;
     cudaStream_t s;
     bool pdl;
-    template <class K> int launch(K kernel, int cols, int threads, int ld, int ldv) const {
-        const size_t smem = (size_t)DS_STAGES * (2 * DB * ld + DB * ldv + DELTA_COEF) * 4;
+    template <class K> int launch(K kernel, int cols, int threads, size_t row_bytes, int ldv) const {
+        const size_t smem = (size_t)DS_STAGES * (2 * DB * row_bytes + (DB * ldv + DELTA_COEF) * 4);
         const dim3 grid((a.dv_p + cols - 1) / cols, a.heads, a.n_req);
-        if (smem > 48 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 32 * 1024) LCU_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));  // beside up to 8 KB of static memory
         LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(threads), smem, s, pdl, a));
         return LCU_OK;
     }
     template <int R8> int run() const {
         constexpr int DK = 8 * R8;
-        if (dt != LCU_F32 && tuning().delta_tc) {
+        if (a.split) {
             // two groups of columns share a CTA's tiles where one group each would not fit the SMs at once
             const int groups = a.dv_p > 16 && (long)a.n_req * a.heads * (a.dv_p / 16) > sm_count() ? 2 : 1;
-            return launch(delta_scan_tc_kernel<DK / 8 / DT_PARTS>, 16 * groups, 32 * DT_PARTS * groups, DK + 8, 16 * groups + 4);
+            return launch(delta_scan_tc_kernel<DK / 8 / DT_PARTS>, 16 * groups, 32 * DT_PARTS * groups, 6 * DK + 16, 16 * groups + 4);
         }
         constexpr int NC = DK <= 128 ? 4 : 2;  // columns per half warp
         int warps = (a.dv_p + 2 * NC - 1) / (2 * NC);
         if (warps > 4) warps = 4;
-        return launch(delta_scan_kernel<DK / 16, NC>, warps * 2 * NC, warps * 32, DK, warps * 2 * NC);
+        return launch(delta_scan_kernel<DK / 16, NC>, warps * 2 * NC, warps * 32, 4 * DK, warps * 2 * NC);
     }
 };
 struct DecodeLaunch {
@@ -783,10 +835,10 @@ int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
     default: return go(delta_prep_kernel<0>);
     }
 }
-int delta_scan_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl) {
+int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl) {
     if (a.n_req <= 0) return LCU_OK;
     LCU_REQUIRE(a.n_req <= 65535 && a.heads <= 65535, "delta rule: grid out of range");
-    return by_dk(a.dk_p, ScanLaunch{a, dt, s, pdl});
+    return by_dk(a.dk_p, ScanLaunch{a, s, pdl});
 }
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_tok <= 0) return LCU_OK;

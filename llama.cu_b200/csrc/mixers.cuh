@@ -69,6 +69,7 @@ struct DeltaArgs {
     float *state;
     const int32_t *tok_req, *req_first, *req_pos, *req_slot;
     // between the kernels of a round with several tokens per request
+    int split;                  // the scan runs on tensor cores: q and k as three bf16 planes [n_tok][kv_heads][3][dk_p]
     float *q, *k;               // [n_tok][kv_heads * dk_p], unit vectors, q scaled
     float *v;                   // [n_tok][heads * dv_p]; the scan overwrites it with its outputs
     const int4 *blocks;         // (request, first token, tokens, slot first / 8 + request + number of the block in its request)
@@ -84,7 +85,7 @@ struct DeltaArgs {
 };
 // Rounds with several tokens per request: convolutions, gates and triangles; the scan; norm and output gate.
 int delta_prep_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
-int delta_scan_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
+int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
 // Rounds of one token per request: all of it in one launch, beside the attention's preparation (nullptr: none).
 int delta_decode_launch(const DeltaArgs &a, const GqaArgs *attn, int dt, cudaStream_t s, bool pdl);

@@ -223,7 +223,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                  o_xc = reserve((size_t)S->expand_cap * S->max_r * eb), o_xkv = reserve((size_t)S->expand_cap * max_kv * eb),
                  o_hout = reserve((T > (size_t)c->max_seqs ? T : c->max_seqs) * S->d_p * eb), o_po = reserve(rows * S->max_r * 4),
                  o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4), o_y2 = reserve(S->pre_norm ? T * S->d_p * 4 : 0),
-                 o_dq = reserve(T * max_dk * 4), o_dk = reserve(T * max_dk * 4), o_dv = reserve(T * max_dv * 4), o_dg = reserve((T / DELTA_BLOCK + c->max_seqs + 1) * max_dh * DELTA_COEF * 4),
+                 o_dq = reserve(T * max_dk * 6), o_dk = reserve(T * max_dk * 6), o_dv = reserve(T * max_dv * 4), o_dg = reserve((T / DELTA_BLOCK + c->max_seqs + 1) * max_dh * DELTA_COEF * 4),
                  o_att2 = reserve(T * max_dhv * eb), o_conv = reserve(2 * S->conv_gen * 4), o_mat = reserve(mat_total * S->n_slots * 4),
                  o_gp = reserve(gqa_part_floats(S->gqa_ctas, max_vp) * 4), o_gt = reserve((size_t)S->gqa_ctas * 4);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));

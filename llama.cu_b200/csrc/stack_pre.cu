@@ -90,6 +90,7 @@ struct PreNormRound {
         a.conv_state = S().conv_state + Y.conv_off * S().n_slots; a.conv_gen_stride = S().conv_gen; a.state = S().mat_state + Y.mat_off * S().n_slots;
         a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req);
         a.req_first = i32(o.req_first); a.req_pos = i32(o.req_pos); a.req_slot = i32(o.req_slot);
+        a.split = c->dt != LCU_F32 && tuning().delta_tc;
         a.q = S().dq; a.k = S().dk; a.v = S().dv; a.coef = S().dcoef;
         a.blocks = reinterpret_cast<const int4 *>(B + o.dblk); a.n_blocks = r.sr.n_delta_blocks; a.o = S().att2; a.stride_o = Y.dhv_p;
         return a;
@@ -106,7 +107,7 @@ struct PreNormRound {
         } else {
             if (!rc && Y.attention()) rc = done(gqa_prep_launch(g, dt, s, L.pdl));
             if (!rc && Y.delta()) rc = done(delta_prep_launch(e, s, L.pdl));
-            if (!rc && Y.delta()) rc = done(delta_scan_launch(e, dt, s, L.pdl));
+            if (!rc && Y.delta()) rc = done(delta_scan_launch(e, s, L.pdl));
             if (!rc && Y.delta()) rc = done(delta_out_launch(e, dt, s, L.pdl));
         }
         if (!rc && Y.attention()) rc = attention(g, Y);
