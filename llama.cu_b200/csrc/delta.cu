@@ -1,6 +1,6 @@
 // Gated delta rule.  Per head a matrix S (f32, one per sequence) is decayed, corrected towards the new value along the new key
-// and read along the query:
-//     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// and read along the query: at token i
+//     u_i = beta_i (v_i - g_i S_{i-1}^T k_i),   S_i = g_i S_{i-1} + k_i u_i^T,   o_i = S_i^T q_i
 // with q, k, v behind short causal convolutions, q and k unit vectors, and o normed and gated per head.
 //
 // Portions run in blocks of eight tokens.  With S the matrix ahead of a block, D_ij the decay between tokens j and i, and
