@@ -71,18 +71,28 @@ typedef enum {
     LCU_W_FF_DOWN = 24,  /* feed-forward down                               */
     LCU_W_SHIFT = 25,    /* token-shift weights                             */
     LCU_W_SCALARS = 26,  /* f32: mixer norm gain, feed-forward norm gain, activation p, q */
-    /* pre-norm layers, softmax attention and delta-rule mixers; f32 unless it is a matrix */
-    LCU_W_MIX_IN = 27,      /* rows: attention q | k | v, delta q | k | v | output gate | step size | decay */
+    /* pre-norm layers, softmax attention and recurrent mixers; f32 unless it is a matrix */
+    LCU_W_MIX_IN = 27,      /* rows: attention q | k | v | head gates; recurrent q | k | v | output gate, then step size | decay
+                             * (DELTA), step size (SSD) or the first map of the decays (GLA)  */
     LCU_W_MIX_BIAS = 28,    /* biases of the attention's q | k | v                      */
     LCU_W_ATT_OUT = 29,     /* attention output projection, [heads][v_dim] columns      */
-    LCU_W_DELTA_OUT = 30,   /* delta-rule output projection, [heads][v_dim] columns     */
-    LCU_W_CONV = 31,        /* short convolutions of the delta rule's q | k | v: [taps][channels] */
-    LCU_W_DELTA_DECAY = 32, /* [2][heads]: logarithm of the decay rate, bias of the step */
-    LCU_W_DELTA_NORM = 33,  /* norm weight of a delta-rule head's output                */
+    LCU_W_DELTA_OUT = 30,   /* recurrent mixer's output projection, [heads][v_dim] columns */
+    LCU_W_CONV = 31,        /* short convolutions of q | k | v (DELTA, SSD): [taps][channels] */
+    LCU_W_DELTA_DECAY = 32, /* [2][heads]: logarithm of the decay rate, bias of the step; SSD: [3], weight of v in the output */
+    LCU_W_DELTA_NORM = 33,  /* norm weight of a head's output; SSD: of all heads' outputs */
     LCU_W_BRANCH_NORM = 34, /* [2][d]: gains on the two mixers' outputs                 */
     LCU_W_NORM1 = 35,       /* gain of the norm ahead of the mixer                      */
     LCU_W_NORM2 = 36,       /* gain of the norm ahead of the feed-forward               */
-    LCU_W_STEP = 37         /* vector added to the residual stream ahead of the layer   */
+    LCU_W_STEP = 37,        /* vector added to the residual stream ahead of the layer   */
+    LCU_W_POST1 = 38,       /* gain of the norm on the mixer's output (post_norm)       */
+    LCU_W_POST2 = 39,       /* gain of the norm on the feed-forward's output            */
+    LCU_W_QK_GAIN = 40,     /* weights of the query / key norms: q | k, one head each (qk_norm 2) or all heads (3) */
+    LCU_W_CONV_BIAS = 41,   /* biases of the short convolutions                         */
+    LCU_W_GATE_MAP = 42,    /* GLA: [rank + 1][heads x key size], second map of the decays transposed, then its bias */
+    LCU_W_ROUTER = 43,      /* experts: matrix of the router                            */
+    LCU_W_SHARED_UP = 44,   /* shared expert; gated feed-forwards hold gate and up rows in turn */
+    LCU_W_SHARED_DOWN = 45,
+    LCU_W_PAIR_EMBD = 46    /* embedding of token pairs, [buckets + 1, d]               */
 } lcu_weight_kind;
 
 /* Model description: the fields llama.cu/src/model/mod.rs:61-78 reads from GGUF metadata.
@@ -103,9 +113,13 @@ typedef struct {
 enum {
     LCU_MIX_LATENT = 1,    /* latent attention: per-head keys and values are linear maps of one cached vector per token */
     LCU_MIX_ATTENTION = 2, /* softmax attention over cached keys and values, grouped heads, rotary positions            */
-    LCU_MIX_DELTA = 4      /* gated delta rule: one state matrix per head and sequence                                  */
-}; /* ATTENTION | DELTA: both read the same input, their outputs are RMS-normed with a gain each and added */
-enum { LCU_ACT_XIELU = 1, LCU_ACT_RELU2 = 2 };
+    LCU_MIX_DELTA = 4,     /* gated delta rule: one state matrix per head and sequence                                  */
+    LCU_MIX_SSD = 8,       /* state space duality: state matrices with one decay per head, keys and queries per group   */
+    LCU_MIX_GLA = 16       /* gated linear attention: state matrices with one decay per head and key channel            */
+}; /* ATTENTION | a recurrent one: both read the same input, their outputs are added: RMS-normed with a gain each, or (post_norm)
+    * with a factor each */
+enum { LCU_ACT_XIELU = 1, LCU_ACT_RELU2 = 2,
+       LCU_ACT_GLU = 3 }; /* g = min(W_gate x, limit), u = clamp(W_up x, +-limit): g sigmoid(alpha g) (u + shift) */
 
 /* One layer of a model described layer by layer.  Post-norm: x += norm(mixer(h)), x += norm(ff(x)), both norms RMS with a
  * single gain on the sublayer's OUTPUT, h = x or (token_shift) x mixed per coordinate with the previous token's x.
@@ -115,7 +129,7 @@ typedef struct {
     int32_t mixer;       /* LCU_MIX_*                                                           */
     int32_t heads, dim, v_dim; /* latent or softmax attention: query heads, query/key and value size per head */
     int32_t q_rank, kv_rank;   /* LATENT: query latent, cached latent                            */
-    int32_t out_gate;    /* LATENT: 1: head h's output is multiplied by sigmoid(W_g h)_h         */
+    int32_t out_gate;    /* LATENT, ATTENTION: 1: head h's output is multiplied by sigmoid(W_g h)_h */
     int32_t token_shift; /* 1: the mixer reads h + (previous h - h) * shift (recurrent state)    */
     int32_t ff;          /* feed-forward width, 0: the layer has none                            */
     int32_t ff_act;      /* LCU_ACT_*                                                            */
@@ -127,7 +141,8 @@ typedef struct {
     /* ATTENTION */
     int32_t kv_heads;    /* key/value heads; query head h reads head h / (heads / kv_heads)      */
     int32_t bias;        /* 1: biases on q, k and v                                              */
-    int32_t qk_norm;     /* 1: q and k are divided by their root mean square after the rotation  */
+    int32_t qk_norm;     /* 1: q and k are divided by their root mean square after the rotation; 2, 3: RMS norm with weights ahead
+                          * of the rotation, per head (2) or over all heads of a token (3)       */
     int32_t rot_dims;    /* rotated dimensions of a head (pairs i, i + rot_dims / 2), 0: none    */
     /* DELTA */
     int32_t delta_heads, delta_kv_heads, delta_dim, delta_v_dim;
@@ -135,6 +150,28 @@ typedef struct {
     /* ATTENTION: frequencies base^(-2i / rot_dims); rot_factor > 0: YaRN, frequencies of fewer than rot_slow turns in
      * rot_original positions divided by the factor, those of more than rot_fast left, a ramp between */
     double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
+    /* PRE-NORM */
+    int32_t post_norm;   /* 1: the sublayers' outputs are RMS-normed too, x += norm(mixer(norm(x))), a gain per coordinate */
+    /* ATTENTION (out_gate as above) */
+    int32_t rot_adjacent;/* 1: pairs (2 i, 2 i + 1)                                              */
+    int32_t window;      /* > 0: position i sees j with i - j < window                           */
+    int32_t sink;        /* 1: the softmax counts one more key of score 0 and without value      */
+    int32_t kv_from;     /* 0: own keys and values; j + 1: those of layer j (a layer before, same key heads, head sizes and rotation) */
+    /* SSD and GLA share the delta_ fields (heads; heads of q and k; key size; value size; taps of SSD) */
+    int32_t norm_parts;  /* SSD: equal parts of the gated output that are normed                 */
+    int32_t gate_rank;   /* GLA: inner size of the decays' map                                   */
+    /* feed-forward of experts (LCU_ACT_GLU): `ff` is an expert's width; a token's weights, sigmoids of its `top` largest router
+     * logits, scale the experts' inputs */
+    int32_t experts, top;
+    int32_t shared_ff;   /* width of an expert that every token uses, 0: none                    */
+    float out_scale, out_scale2; /* post_norm, two mixers: factors on the attention's and the recurrent mixer's output */
+    float gate_tau;      /* GLA: decay = sigmoid(z)^(1 / tau)                                    */
+    float glu_limit, shared_limit, glu_alpha, glu_shift; /* LCU_ACT_GLU                          */
+    /* read from the first layer: the embedding ahead of it */
+    float embed_scale;    /* factor on the embedding rows; 0 = 1                                 */
+    int32_t pair_buckets; /* > 0: row (previous token * pair_prev + token * pair_cur) mod pair_buckets of LCU_W_PAIR_EMBD is added
+                           * to a token's embedding, row pair_buckets to that of a sequence's first token */
+    int32_t pair_prev, pair_cur; /* in [0, pair_buckets)                                         */
 } lcu_layer_desc;
 
 /* == `KVPair` (llama.cu/src/op/random_sample/mod.rs:29-36) == cub::KeyValuePair<int,half> */

@@ -18,9 +18,10 @@ LIB_PATH = os.path.join(_HERE, "liblcu.so")
 F16, BF16, F32, Q8_0, U32 = 0, 1, 2, 3, 4
 W_EMBD, W_ATTN_NORM, W_QKV, W_O, W_FFN_NORM, W_GATE_UP, W_DOWN, W_OUT_NORM, W_LM_HEAD = range(9)
 (W_LAT_IN, W_Q_NORM, W_KV_NORM, W_UQ, W_UKT, W_UKV, W_LAT_OUT, W_UP, W_FF_DOWN, W_SHIFT, W_SCALARS, W_MIX_IN, W_MIX_BIAS,
- W_ATT_OUT, W_DELTA_OUT, W_CONV, W_DELTA_DECAY, W_DELTA_NORM, W_BRANCH_NORM, W_NORM1, W_NORM2, W_STEP) = range(16, 38)
-MIX_LATENT, MIX_ATTENTION, MIX_DELTA = 1, 2, 4
-ACT_XIELU, ACT_RELU2 = 1, 2
+ W_ATT_OUT, W_DELTA_OUT, W_CONV, W_DELTA_DECAY, W_DELTA_NORM, W_BRANCH_NORM, W_NORM1, W_NORM2, W_STEP, W_POST1, W_POST2, W_QK_GAIN,
+ W_CONV_BIAS, W_GATE_MAP, W_ROUTER, W_SHARED_UP, W_SHARED_DOWN, W_PAIR_EMBD) = range(16, 47)
+MIX_LATENT, MIX_ATTENTION, MIX_DELTA, MIX_SSD, MIX_GLA = 1, 2, 4, 8, 16
+ACT_XIELU, ACT_RELU2, ACT_GLU = 1, 2, 3
 LINEAR_KINDS = (W_QKV, W_O, W_GATE_UP, W_DOWN)
 NO_OUTPUT = 2**64 - 1  # LCU_ENGINE_NO_OUTPUT: a prefill chunk that samples nothing
 OK, ERR_INVALID, ERR_CUDA, ERR_OVERFLOW, ERR_NO_PAGES, ERR_STATE, ERR_COMM, ERR_TIMEOUT = 0, -1, -2, -3, -4, -5, -6, -7
@@ -44,7 +45,11 @@ class LayerDesc(C.Structure):
                                          "ff_act", "weights_of")] + [("scale", C.c_float)] + [
         (n, C.c_int32) for n in ("pre_norm", "add_embed", "add_step", "kv_heads", "bias", "qk_norm", "rot_dims", "delta_heads",
                                  "delta_kv_heads", "delta_dim", "delta_v_dim", "delta_conv")] + [
-        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + [
+        (n, C.c_int32) for n in ("post_norm", "rot_adjacent", "window", "sink", "kv_from", "norm_parts", "gate_rank", "experts", "top",
+                                 "shared_ff")] + [
+        (n, C.c_float) for n in ("out_scale", "out_scale2", "gate_tau", "glu_limit", "shared_limit", "glu_alpha", "glu_shift", "embed_scale")] + [
+        (n, C.c_int32) for n in ("pair_buckets", "pair_prev", "pair_cur")]
 
 
 class KVPair(C.Structure):

@@ -14,7 +14,7 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(CSRC, "_obj")
 LIB = os.path.join(HERE, "liblcu.so")
 SOURCES = ["ctx.cu", "api.cu", "ops.cu", "gemv.cu", "attention.cu", "sample.cu", "comm.cu", "gemm_skinny.cu", "gemm_tc.cu", "p2p.cu", "engine.cpp", "gguf.cpp",
-           "stack.cu", "stack_pre.cu", "stack_ops.cu", "latent.cu", "latent_tc.cu", "gqa.cu", "delta.cu", "linear_f32.cu"]
+           "stack.cu", "stack_pre.cu", "stack_ops.cu", "latent.cu", "latent_tc.cu", "gqa.cu", "delta.cu", "scan.cu", "moe.cu", "linear_f32.cu"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden", "--expt-relaxed-constexpr",

@@ -121,6 +121,13 @@ __device__ __forceinline__ void tc_finish(const GemvArgs &a, int n, int first, f
 #pragma unroll
         for (int i = 0; i < 8; ++i) v[i] = relu2_act(v[i]);
     }
+    if (a.epilogue == EPI_GLU) {
+        const float sc = a.row_scale ? a.row_scale[n] : 1.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] = glu_act(sc * v[2 * i], sc * v[2 * i + 1], a.glu);
+        *reinterpret_cast<uint2 *>(reinterpret_cast<T *>(a.y) + (size_t)n * a.stride_y + first / 2) = make_uint2(Act<T>::pack(v[0], v[1]), Act<T>::pack(v[2], v[3]));
+        return;
+    }
     uint4 o;
     o.x = Act<T>::pack(v[0], v[1]); o.y = Act<T>::pack(v[2], v[3]); o.z = Act<T>::pack(v[4], v[5]); o.w = Act<T>::pack(v[6], v[7]);
     if (a.push.n && (a.epilogue == EPI_STORE || a.epilogue == EPI_RESIDUAL)) {
@@ -483,7 +490,13 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
     const bool swiglu = a.epilogue == EPI_SWIGLU;
     const int ks = (int)tc_cluster_rank();
     const int rb = (int)blockIdx.x / KS;
-    const int tb = (int)blockIdx.y * N;  // first token of this CTA's block
+    int tb = (int)blockIdx.y * N, n_end = a.n_tok, wrow = 0;  // first token of this CTA's block, end of the tokens, first weight row
+    if (a.tiles) {  // grouped: the table is the predecessor's; every CTA of a cluster has the same tile
+        grid_dep_wait();
+        const int4 tile = a.tiles[blockIdx.y];
+        if (tile.z == 0) return;
+        tb = tile.y; n_end = tile.y + tile.z; wrow = tile.x * a.out;
+    }
     const int kb0 = (int)((long)ks * nkb / KS), kb1 = (int)((long)(ks + 1) * nkb / KS);
     const int n_units = kb1 - kb0;
     const int tm_cols = N < 32 ? 32 : N;
@@ -516,8 +529,8 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
             const int kx = (kb0 + j) * TC_BK;
             if (weights) {
                 tc_mbar_expect_tx(bar, (uint32_t)stage_bytes);
-                tc_tma_2d(dst, &map_w, kx, swiglu ? rb * 64 : rb * TC_BM, bar);
-                tc_tma_2d(dst + TC_A_BYTES / 2, &map_w, kx, swiglu ? a.di + rb * 64 : rb * TC_BM + 64, bar);
+                tc_tma_2d(dst, &map_w, kx, wrow + (swiglu ? rb * 64 : rb * TC_BM), bar);
+                tc_tma_2d(dst + TC_A_BYTES / 2, &map_w, kx, wrow + (swiglu ? a.di + rb * 64 : rb * TC_BM + 64), bar);
             }
             if (acts) tc_tma_2d(dst + TC_A_BYTES, &map_x, kx, tb, bar);
         };
@@ -582,7 +595,7 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
         __syncthreads();
         tc_cluster_sync();  // every CTA of the row block has staged its partial tile
 
-        if (warp >= 2 && tb + t0 < a.n_tok) {
+        if (warp >= 2 && tb + t0 < n_end) {
             // ---------------- this CTA's share of the items: chunk c of 8 rows (8 pairs for SwiGLU) with c % KS == ks
             const int et = tid - 64;
             const int chunks = swiglu ? 8 : 16;
@@ -592,13 +605,13 @@ gemm_tck_kernel(const GemvArgs a, const __grid_constant__ CUtensorMap map_w, con
             for (int idx = et; idx < mine * NS; idx += 128, ++cnt) {
                 const int c = ks + (idx % mine) * KS, n = tb + t0 + idx / mine;
                 const int first = swiglu ? rb * 64 + 8 * c : rb * TC_BM + 8 * c;
-                if (n < a.n_tok && first + 8 <= (swiglu ? a.di : a.out)) tc_prefetch<T>(a, n, first, pre[cnt]);
+                if (n < n_end && first + 8 <= (swiglu ? a.di : a.out)) tc_prefetch<T>(a, n, first, pre[cnt]);
             }
             cnt = 0;
             for (int idx = et; idx < mine * NS; idx += 128, ++cnt) {
                 const int c = ks + (idx % mine) * KS, nl = idx / mine, n = tb + t0 + nl;
                 const int first = swiglu ? rb * 64 + 8 * c : rb * TC_BM + 8 * c;
-                if (!(n < a.n_tok && first + 8 <= (swiglu ? a.di : a.out))) continue;
+                if (!(n < n_end && first + 8 <= (swiglu ? a.di : a.out))) continue;
                 float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
                 const uint32_t sv = tc_smem(stg + (size_t)nl * TCK_LD + 8 * c);
                 for (int p = 0; p < KS; ++p) {
@@ -675,7 +688,7 @@ static size_t tc_smem_bytes(int N, int stages) {
 template <class T>
 static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry) {
     auto kernel = gemm_tc_kernel<T>;
-    const int N = a.n_tok <= 16 ? 16 : (a.n_tok <= 32 ? 32 : (a.n_tok <= 64 ? 64 : (a.n_tok <= 128 ? 128 : 256)));
+    const int N = a.tiles ? a.tile_rows : a.n_tok <= 16 ? 16 : (a.n_tok <= 32 ? 32 : (a.n_tok <= 64 ? 64 : (a.n_tok <= 128 ? 128 : 256)));
     int stages = 8;
     while (stages > 2 && tc_smem_bytes(N, stages) > (size_t)227 * 1024) --stages;
     const size_t smem = tc_smem_bytes(N, stages);
@@ -711,7 +724,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
     const int vec = vec_ok ? 1 : 0;
     LCU_REQUIRE(vec || a.epilogue < EPI_STORE_F32, "gemm_tc: epilogue %d needs rows of a multiple of 8 outputs", a.epilogue);
     // ---- weight rows on M (any output shape; row blocks of 128)
-    rc = tc_make_map(&mw, a.w, dt, (uint64_t)a.out, (uint64_t)a.in, (uint64_t)a.in, 64);
+    rc = tc_make_map(&mw, a.w, dt, (uint64_t)a.out * (a.tiles ? a.groups : 1), (uint64_t)a.in, (uint64_t)a.in, 64);
     if (rc) return rc;
     // the activation map has exactly n_tok rows: the rest of the N-row box is out of bounds and zero-filled
     rc = tc_make_map(&mx, a.x, dt, (uint64_t)a.n_tok, (uint64_t)a.in, (uint64_t)a.stride_x, (uint32_t)N);
@@ -723,7 +736,7 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
         // blocks the balanced stream-K split wins: 4.75 against 4.95 ms), 2: wherever it applies, 0: never
         const int cluster_mode = tuning().tc_cluster;
         const int n_rb_c = (n_pairs + 63) / 64, nkb_c = a.in / TC_BK;
-        const int n_tb = (a.n_tok + N - 1) / N;  // token blocks: more than one only for rounds of more than 256 tokens
+        const int n_tb = a.tiles ? a.n_tiles : (a.n_tok + N - 1) / N;  // token blocks: more than one for rounds of more than 256 tokens, and tiles
         int KS = sms / (n_rb_c * n_tb);
         if (KS > 8) KS = 8;
         if (KS < 1) KS = 1;
@@ -732,8 +745,9 @@ static int tc_launch_t(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool
         // 1: where it measured faster than the stream-K split: 64-token blocks, and matrices whose row blocks leave room
         // for clusters of four and more (8B batch 32, per launch: O 20.9 -> 18.3 us, down 35.4 -> 32.9 us; the 48-row-block
         // QKV matrix with clusters of three 26.8 -> 34.5 us, so it stays on stream-K)
-        const bool cluster_on = N > 64 || cluster_mode == 2 || (cluster_mode == 1 && (N == 64 || n_rb_c * 4 <= sms));
-        if (vec && cluster_on && (KS >= 2 || N > 64)) {
+        if (a.tiles) KS = 1;
+        const bool cluster_on = a.tiles || N > 64 || cluster_mode == 2 || (cluster_mode == 1 && (N == 64 || n_rb_c * 4 <= sms));
+        if (vec && cluster_on && (KS >= 2 || N > 64 || a.tiles)) {
             const int stage_bytes = TC_A_BYTES + N * 128;
             const int NS = N > 64 ? 64 : N;
             const size_t fixed = 1024 + (size_t)NS * TCK_LD * 4 + sizeof(TcShared) + 64;
@@ -804,6 +818,8 @@ int gemm_tc_launch(const GemvArgs &a, int dt, cudaStream_t s, bool pdl, bool dry
     LCU_REQUIRE(a.prologue == PRO_NONE && !a.x_rows, "gemm_tc: takes prepared activations only");
     LCU_REQUIRE(a.stride_x % 8 == 0, "gemm_tc: x row stride %d must be a multiple of 8 elements", a.stride_x);
     LCU_REQUIRE(dry || (((uintptr_t)a.x | (uintptr_t)a.w) % 16) == 0, "gemm_tc: operands must be 16-byte aligned");
+    LCU_REQUIRE(!a.tiles || (a.out % 8 == 0 && (a.tile_rows == 64 || a.tile_rows == 128 || a.tile_rows == 256) && a.n_tiles <= 65535),
+                "gemm_tc: groups of %d rows in %d tiles of %d", a.out, a.n_tiles, a.tile_rows);
     if (a.epilogue == EPI_SWIGLU) LCU_REQUIRE(a.out == 2 * a.di, "gemm_tc: swiglu needs out == 2*di");
     if (dt == LCU_F16) return tc_launch_t<__half>(a, dt, s, pdl, dry);
     if (dt == LCU_BF16) return tc_launch_t<__nv_bfloat16>(a, dt, s, pdl, dry);

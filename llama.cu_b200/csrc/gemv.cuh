@@ -12,7 +12,11 @@ enum GemvPrologue { PRO_NONE = 0, PRO_RMSNORM = 1,
 enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU = 3,
                     EPI_STORE_F32 = 4,  // y is f32
                     EPI_XIELU = 5,      // y = xielu(row) with the two numbers at act_pq
-                    EPI_RELU2 = 6 };    // y = max(row, 0)^2
+                    EPI_RELU2 = 6,      // y = max(row, 0)^2
+                    EPI_GLU = 7 };      // rows are gate and up in turn: y[n, out / 2] of glu
+
+// Gated activation: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(alpha g) (u + shift).
+struct GluArgs { float limit, alpha, shift; };
 
 // Inputs of the prologues of layered models, for rounds of one token per request (token t is request t).  Every CTA computes
 // the rows it multiplies; what later kernels need (new residual, shift state, cached latent) is written by the first CTA.
@@ -67,6 +71,11 @@ struct GemvArgs {
     const int32_t *page_table;  // [slots, pt_stride]
     int pt_stride;
     const float *act_pq;  // EPI_XIELU: p, q
+    GluArgs glu;          // EPI_GLU
+    // grouped products (gemm_tc.cu): row t.y .. t.y + t.z of x and y meet matrix t.x of `groups` ones of `out` rows; a factor per row
+    const int4 *tiles;
+    int n_tiles, tile_rows, groups;
+    const float *row_scale;  // EPI_GLU, or nullptr
     // EPI_SWIGLU: rows [0,di) gate, [di,2di) up; y gets [n_tok, di]
     int di;
     // tuning: 0 = trigger dependents at kernel start, 1 = after the main loop, 2 = never (implicit at exit)
@@ -91,6 +100,10 @@ __device__ __forceinline__ float xielu_act(float z, float sp, float sq) {
 }
 
 __device__ __forceinline__ float relu2_act(float z) { return z > 0.f ? z * z : 0.f; }
+__device__ __forceinline__ float glu_act(float gate, float up, const GluArgs &a) {
+    const float g = fminf(gate, a.limit), u = fminf(fmaxf(up, -a.limit), a.limit);
+    return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
+}
 
 // Values an epilogue would otherwise fetch from global memory behind the weight stream: the per-token constants of the
 // RoPE / KV-append epilogue (position, cache page, sin and cos rows; head sizes up to 128), staged in shared memory
@@ -192,6 +205,8 @@ __device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int 
         *reinterpret_cast<float2 *>(reinterpret_cast<float *>(a.y) + off) = make_float2(va, vb);
     } else if (a.epilogue == EPI_RELU2) {
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(relu2_act(va), relu2_act(vb));
+    } else if (a.epilogue == EPI_GLU) {
+        reinterpret_cast<T *>(a.y)[(size_t)t * a.stride_y + pair] = Act<T>::from_f(glu_act(va, vb, a.glu));
     } else {
         const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(xielu_act(va, sp, sq), xielu_act(vb, sp, sq));

@@ -5,6 +5,7 @@
 //               of a tensor-core tile; every warp walks its own blocks of 16 cached rows with a copy ring and running softmax of
 //               its own (no barrier in the loop); contexts are cut into splits, the last CTA of a row tile to arrive merges;
 //   long form   64 (token, head) rows per CTA share tiles of 64 cached rows.
+// Options: a sliding window (tiles that no row sees are skipped), a sink in the softmax's denominator, a gate per head.
 //
 // Arithmetic: scores, softmax and its running state in f32; probabilities are rounded to bf16 only as operands of the second
 // product, the row sum is taken over the rounded values; all sums accumulate in f32.  All-32-bit contexts use f32 FMA throughout.
@@ -43,10 +44,25 @@ __device__ __forceinline__ float quad_sum(float v) {
 template <class T>
 __global__ void __launch_bounds__(256) gqa_prep_kernel(const GqaArgs a) {
     grid_dep_launch();
-    const int item = blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int per = (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x;
     grid_dep_wait();
-    if (item < gqa_prep_items(a)) gqa_prep_item<T>(a, blockIdx.y, item, threadIdx.x & 31);
+    gqa_prep_block<T>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
 }
+
+// Denominator and factor that end a row of softmax (scores in powers of two): maximum M, sum L over it.  A key of score 0 may
+// count in the denominator; the head's gate multiplies the output.
+__device__ __forceinline__ float softmax_end(const GqaArgs &a, float M, float L, int tok, int head) {
+    float f = 1.f;
+    if (a.sink) {
+        const float top = fmaxf(M, 0.f);
+        f = exp2f(M - top);
+        L = fmaf(L, f, exp2f(-top));
+    }
+    if (a.gate) f /= 1.f + expf(-a.gate[(size_t)tok * a.stride + head]);
+    return f / L;
+}
+// first position that position p sees
+__device__ __forceinline__ int first_seen(const GqaArgs &a, int p) { return a.window > 0 && p >= a.window ? p - a.window + 1 : 0; }
 
 // ------------------------------------------------------------------ short form
 constexpr int GS_WARPS = 4, GS_KEYS = 16, GS_STAGES = 3;
@@ -70,11 +86,11 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
     const int kvh = blockIdx.x % a.kv_heads, row0 = blockIdx.x / a.kv_heads * 16;
     const int4 rq = a.reqs[blockIdx.y];  // request, first token, tokens, position
     const int rows = rq.z * g, sp = blockIdx.z;
-    const int ctx = rq.w + rq.z, units = (ctx + GS_UNIT - 1) / GS_UNIT;
+    const int ctx = rq.w + rq.z, unit0 = first_seen(a, rq.w) / GS_UNIT, units = (ctx + GS_UNIT - 1) / GS_UNIT - unit0;
     const int ups = (units + a.splits - 1) / a.splits, n_split = (units + ups - 1) / ups;
     grid_dep_launch();
     if (row0 >= rows || sp >= n_split) return;
-    const int u0 = sp * ups, u1 = min(units, u0 + ups);
+    const int u0 = unit0 + sp * ups, u1 = min(unit0 + units, u0 + ups);
     const bf16 *pool = reinterpret_cast<const bf16 *>(a.pool);
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)rq.x * a.pt_stride;
@@ -112,6 +128,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
     const bool v0 = r0 < rows, v1 = r1 < rows;
     const int tk0 = v0 ? r0 / g : 0, tk1 = v1 ? r1 / g : 0;
     const int lim0 = v0 ? rq.w + tk0 : -1, lim1 = v1 ? rq.w + tk1 : -1;
+    const int lo0 = first_seen(a, lim0), lo1 = first_seen(a, lim1);
     uint32_t qa[KS][4];
     {
         const bf16 *q = reinterpret_cast<const bf16 *>(a.q);
@@ -151,10 +168,10 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
             const int p = u * GS_UNIT + warp * GS_KEYS + nt * 8 + 2 * t4;
-            sc[nt][0] = p <= lim0 ? sc[nt][0] * scale2 : -INFINITY;
-            sc[nt][1] = p + 1 <= lim0 ? sc[nt][1] * scale2 : -INFINITY;
-            sc[nt][2] = p <= lim1 ? sc[nt][2] * scale2 : -INFINITY;
-            sc[nt][3] = p + 1 <= lim1 ? sc[nt][3] * scale2 : -INFINITY;
+            sc[nt][0] = p <= lim0 && p >= lo0 ? sc[nt][0] * scale2 : -INFINITY;
+            sc[nt][1] = p + 1 <= lim0 && p + 1 >= lo0 ? sc[nt][1] * scale2 : -INFINITY;
+            sc[nt][2] = p <= lim1 && p >= lo1 ? sc[nt][2] * scale2 : -INFINITY;
+            sc[nt][3] = p + 1 <= lim1 && p + 1 >= lo1 ? sc[nt][3] * scale2 : -INFINITY;
             t0 = fmaxf(t0, fmaxf(sc[nt][0], sc[nt][1]));
             t1 = fmaxf(t1, fmaxf(sc[nt][2], sc[nt][3]));
         }
@@ -226,8 +243,8 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
             for (int e = 0; e < 8; ++e) x[e] += src[e] * f;
         }
         if (n_split == 1) {
-            const float inv = 1.f / L;
             const int row = row0 + r;
+            const float inv = softmax_end(a, M, L, rq.y + row / g, kvh * g + row % g);
             uint4 u;
             u.x = Act<bf16>::pack(x[0] * inv, x[1] * inv); u.y = Act<bf16>::pack(x[2] * inv, x[3] * inv);
             u.z = Act<bf16>::pack(x[4] * inv, x[5] * inv); u.w = Act<bf16>::pack(x[6] * inv, x[7] * inv);
@@ -259,8 +276,8 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
             x[0] += lo.x * f; x[1] += lo.y * f; x[2] += lo.z * f; x[3] += lo.w * f;
             x[4] += hi.x * f; x[5] += hi.y * f; x[6] += hi.z * f; x[7] += hi.w * f;
         }
-        const float inv = 1.f / L;
         const int row = row0 + r;
+        const float inv = softmax_end(a, M, L, rq.y + row / g, kvh * g + row % g);
         uint4 u;
         u.x = Act<bf16>::pack(x[0] * inv, x[1] * inv); u.y = Act<bf16>::pack(x[2] * inv, x[3] * inv);
         u.z = Act<bf16>::pack(x[4] * inv, x[5] * inv); u.w = Act<bf16>::pack(x[6] * inv, x[7] * inv);
@@ -303,7 +320,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
     const int4 rq = a.reqs[ri];
     const int rows = rq.z * g, row0 = blk * 64;
     const int last_tok = min(rq.z - 1, (row0 + 63) / g);
-    const int ctx = rq.w + last_tok + 1, n_tiles = (ctx + GL_TILE - 1) / GL_TILE;
+    const int ctx = rq.w + last_tok + 1, n_tiles = (ctx + GL_TILE - 1) / GL_TILE, tile0 = first_seen(a, rq.w + row0 / g) / GL_TILE;
     const bf16 *pool = reinterpret_cast<const bf16 *>(a.pool);
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)rq.x * a.pt_stride;
@@ -333,6 +350,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
     const bool v0 = r0 < rows, v1 = r1 < rows;
     const int tk0 = v0 ? r0 / g : 0, tk1 = v1 ? r1 / g : 0;
     const int lim0 = v0 ? rq.w + tk0 : -1, lim1 = v1 ? rq.w + tk1 : -1;
+    const int lo0 = first_seen(a, lim0), lo1 = first_seen(a, lim1);
     const int h0 = kvh * g + (v0 ? r0 % g : 0), h1 = kvh * g + (v1 ? r1 % g : 0);
     uint32_t qa[KS][4];
     {
@@ -347,7 +365,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
             qa[ks][3] = in && v1 ? *reinterpret_cast<const uint32_t *>(q1 + ks * 16 + 8) : 0u;
         }
     }
-    load_tile(0, 0);
+    load_tile(tile0, 0);
     ga_commit();
     const float scale2 = a.scale * 1.4426950408889634f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
@@ -355,8 +373,8 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
 #pragma unroll
     for (int i = 0; i < NTO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
 
-    for (int tile = 0; tile < n_tiles; ++tile) {
-        const int buf = tile & 1;
+    for (int tile = tile0; tile < n_tiles; ++tile) {
+        const int buf = (tile - tile0) & 1;
         if (tile + 1 < n_tiles) load_tile(tile + 1, buf ^ 1);
         ga_commit();
         ga_wait<1>();
@@ -378,7 +396,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
             }
         }
         float t0 = -INFINITY, t1 = -INFINITY;
-        if (tile * GL_TILE + GL_TILE - 1 <= min(lim0, lim1)) {  // every position visible
+        if (tile * GL_TILE + GL_TILE - 1 <= min(lim0, lim1) && tile * GL_TILE >= max(lo0, lo1)) {  // every position visible
 #pragma unroll
             for (int nt = 0; nt < NTS; ++nt) {
 #pragma unroll
@@ -390,10 +408,10 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
 #pragma unroll
             for (int nt = 0; nt < NTS; ++nt) {
                 const int p = tile * GL_TILE + nt * 8 + 2 * t4;
-                sc[nt][0] = p <= lim0 ? sc[nt][0] * scale2 : -INFINITY;
-                sc[nt][1] = p + 1 <= lim0 ? sc[nt][1] * scale2 : -INFINITY;
-                sc[nt][2] = p <= lim1 ? sc[nt][2] * scale2 : -INFINITY;
-                sc[nt][3] = p + 1 <= lim1 ? sc[nt][3] * scale2 : -INFINITY;
+                sc[nt][0] = p <= lim0 && p >= lo0 ? sc[nt][0] * scale2 : -INFINITY;
+                sc[nt][1] = p + 1 <= lim0 && p + 1 >= lo0 ? sc[nt][1] * scale2 : -INFINITY;
+                sc[nt][2] = p <= lim1 && p >= lo1 ? sc[nt][2] * scale2 : -INFINITY;
+                sc[nt][3] = p + 1 <= lim1 && p + 1 >= lo1 ? sc[nt][3] * scale2 : -INFINITY;
                 t0 = fmaxf(t0, fmaxf(sc[nt][0], sc[nt][1]));
                 t1 = fmaxf(t1, fmaxf(sc[nt][2], sc[nt][3]));
             }
@@ -442,7 +460,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
 #pragma unroll
     for (int hf = 0; hf < 2; ++hf) {
         if (!(hf ? v1 : v0)) continue;
-        const float inv = 1.f / (hf ? l1 : l0);
+        const float inv = softmax_end(a, hf ? m1 : m0, hf ? l1 : l0, rq.y + (hf ? tk1 : tk0), hf ? h1 : h0);
         bf16 *dst = out + (size_t)(rq.y + (hf ? tk1 : tk0)) * a.stride_o + (size_t)(hf ? h1 : h0) * a.vdim_p + 2 * t4;
 #pragma unroll
         for (int i = 0; i < NTO; ++i)
@@ -465,7 +483,7 @@ __global__ void __launch_bounds__(256) gqa_f32_kernel(const GqaArgs a) {
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)a.tok_req[t] * a.pt_stride;
     float m = -INFINITY, l = 0.f, acc[MIX_MAX_HEAD / 32] = {};
-    for (int k0 = 0; k0 < ctx; k0 += 32) {
+    for (int k0 = first_seen(a, ctx - 1); k0 < ctx; k0 += 32) {
         const int key = k0 + lane;
         const bool ok = key < ctx;
         const int slot = key & ((1 << a.page_shift) - 1);
@@ -496,10 +514,11 @@ __global__ void __launch_bounds__(256) gqa_f32_kernel(const GqaArgs a) {
                 if (lane + 32 * j < a.vdim_p) acc[j] = fmaf(pi, vr[lane + 32 * j], acc[j]);
         }
     }
+    const float inv = softmax_end(a, m * 1.4426950408889634f, l, t, h);
     float *out = reinterpret_cast<float *>(a.o) + (size_t)t * a.stride_o + (size_t)h * a.vdim_p;
 #pragma unroll
     for (int j = 0; j < MIX_MAX_HEAD / 32; ++j)
-        if (lane + 32 * j < a.vdim_p) out[lane + 32 * j] = acc[j] / l;
+        if (lane + 32 * j < a.vdim_p) out[lane + 32 * j] = acc[j] * inv;
 }
 
 template <class K>
@@ -550,7 +569,8 @@ struct ShortCtas {
 int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_tok <= 0) return LCU_OK;
     LCU_REQUIRE(a.n_tok <= 65535, "attention: %d tokens in a round", a.n_tok);
-    const dim3 grid((a.heads + 2 * a.kv_heads + 7) / 8, a.n_tok);
+    // a norm over all heads is summed once per block: one block per token where there are many
+    const dim3 grid(a.qk_norm == 3 && a.n_tok > 64 ? 1 : (gqa_prep_items(a) + 7) / 8, a.n_tok);
     if (dt == LCU_F32) LCU_CHECK_CUDA(launch_kernel(gqa_prep_kernel<float>, grid, dim3(256), 0, s, pdl, a));
     else LCU_CHECK_CUDA(launch_kernel(gqa_prep_kernel<bf16>, grid, dim3(256), 0, s, pdl, a));
     return LCU_OK;

@@ -1,14 +1,15 @@
-// The step between the fused input projection and softmax attention, one warp per (token, head): bias, rotation, norm; the
-// query to its buffer, key and value to the cache.  Shared by the kernels of gqa.cu and the decode kernel of delta.cu.
+// The step between the fused input projection and softmax attention, one warp per (token, head): bias, norm, rotation; the
+// query to its buffer, key and value to the cache.  Shared by the kernels of gqa.cu and the decode kernels of the recurrent mixers.
 #pragma once
 #include "stack.cuh"
 
 namespace lcu {
 
-__device__ __forceinline__ int gqa_prep_items(const GqaArgs &a) { return a.heads + 2 * a.kv_heads; }
+__host__ __device__ __forceinline__ int gqa_prep_items(const GqaArgs &a) { return a.heads + (a.own_kv ? 2 * a.kv_heads : 0); }
 
+// row_norm: what qk_norm 3 divides all of q and all of k by (as factors)
 template <class T>
-__device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item, int lane) {
+__device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item, int lane, const float2 &row_norm) {
     const bool is_v = item >= a.heads + a.kv_heads, is_q = item < a.heads;
     const int size_p = is_v ? a.vdim_p : a.dim_p;
     const int head = is_q ? item : (is_v ? item - a.heads - a.kv_heads : item - a.heads);
@@ -24,11 +25,30 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     }
     const int half = a.rot_dims >> 1;
     const float2 *rot = a.rot + (size_t)p * half;
-    auto load4 = [&](int d) {
+    const float *gain = nullptr;
+    float pre = 1.f;  // factor of a norm ahead of the rotation
+    auto raw4 = [&](int d) {
         float4 x = *reinterpret_cast<const float4 *>(src + d);
         if (bias) {
             const float4 y = *reinterpret_cast<const float4 *>(bias + d);
             x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+        }
+        return x;
+    };
+    if (!is_v && a.qk_norm == 2) {
+        float ss = 0.f;
+        for (int d = 4 * lane; d < size_p; d += 128) ss += dot4(raw4(d));
+        pre = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+        gain = a.qk_gain + (is_q ? 0 : a.dim_p);
+    } else if (!is_v && a.qk_norm == 3) {
+        pre = is_q ? row_norm.x : row_norm.y;
+        gain = a.qk_gain + off;
+    }
+    auto load4 = [&](int d) {
+        float4 x = raw4(d);
+        if (gain) {
+            const float4 g = *reinterpret_cast<const float4 *>(gain + d);
+            x.x *= pre * g.x; x.y *= pre * g.y; x.z *= pre * g.z; x.w *= pre * g.w;
         }
         return x;
     };
@@ -41,7 +61,10 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         if (d >= size_p) continue;
         float4 x = load4(d);
         if (!is_v && d < a.rot_dims) {
-            if (half % 4 == 0) {  // four pairs: the partners are four consecutive dimensions too
+            if (a.rot_adjacent) {  // two pairs
+                const float2 c0 = rot[d >> 1], c1 = d + 2 < a.rot_dims ? rot[(d >> 1) + 1] : make_float2(1.f, 0.f);
+                x = make_float4(x.x * c0.x - x.y * c0.y, x.y * c0.x + x.x * c0.y, x.z * c1.x - x.w * c1.y, x.w * c1.x + x.z * c1.y);
+            } else if (half % 4 == 0) {  // four pairs: the partners are four consecutive dimensions too
                 const bool lower = d < half;
                 const int e = lower ? d + half : d - half;
                 const float4 y = load4(e), c0 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e)), c1 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e) + 2);
@@ -55,7 +78,7 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
                     const int i = d + k;
                     if (i >= a.rot_dims) continue;
                     const int e = i < half ? i + half : i - half;
-                    const float y = src[e] + (bias ? bias[e] : 0.f);
+                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (gain ? pre * gain[e] : 1.f);
                     const float2 cs = rot[i < half ? i : e];
                     xs[k] = i < half ? xs[k] * cs.x - y * cs.y : xs[k] * cs.x + y * cs.y;
                 }
@@ -65,12 +88,37 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
     }
     float r = 1.f;
-    if (!is_v && a.qk_norm) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    if (!is_v && a.qk_norm == 1) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
 #pragma unroll
     for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
         const int d = 4 * lane + 128 * j;
         if (d < size_p) st4<T>(dst + d, make_float4(v[j].x * r, v[j].y * r, v[j].z * r, v[j].w * r));
     }
+}
+
+// Items [item0, item1) of token t by one block; every thread of the block calls it.
+template <class T>
+__device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item0, int item1) {
+    float2 norm = make_float2(1.f, 1.f);
+    if (a.qk_norm == 3) {
+        __shared__ float2 part[32];
+        const int nq = a.heads * a.dim_p, n = nq + (a.own_kv ? a.kv_heads * a.dim_p : 0);
+        const float *src = a.lat + (size_t)t * a.stride;
+        float2 ss = make_float2(0.f, 0.f);
+        for (int d = 4 * threadIdx.x; d < n; d += 4 * blockDim.x) {
+            float4 x = *reinterpret_cast<const float4 *>(src + d);
+            if (a.bias) {
+                const float4 y = *reinterpret_cast<const float4 *>(a.bias + d);
+                x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+            }
+            (d < nq ? ss.x : ss.y) += dot4(x);
+        }
+        ss = block_sum2(ss.x, ss.y, part);
+        norm.x = 1.f / sqrtf(ss.x / (float)(a.heads * a.dim) + a.eps);
+        norm.y = 1.f / sqrtf(ss.y / (float)(a.kv_heads * a.dim) + a.eps);
+    }
+    item1 = min(item1, gqa_prep_items(a));
+    for (int item = item0 + (int)(threadIdx.x >> 5); item < item1; item += (int)(blockDim.x >> 5)) gqa_prep_item<T>(a, t, item, threadIdx.x & 31, norm);
 }
 
 }  // namespace lcu

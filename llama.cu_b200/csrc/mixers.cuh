@@ -1,5 +1,5 @@
-// Mixers of pre-norm layers: softmax attention over cached keys and values (gqa.cu) and the gated delta rule (delta.cu).
-// Both read f32 rows of one fused input projection and write operands of their output projections.  Interface only.
+// Mixers of pre-norm layers: softmax attention over cached keys and values (gqa.cu), the gated delta rule (delta.cu), state space
+// duality and gated linear attention (scan.cu).  All read f32 rows of one fused input projection and write operands of their output projections.  Interface only.
 #pragma once
 #include "common.cuh"
 
@@ -9,14 +9,17 @@ constexpr int MIX_MAX_HEAD = 256;  // largest head size of either mixer
 
 // ---- softmax attention, grouped heads, rotary positions
 struct GqaArgs {
-    // rows of the fused projection: q heads | k heads | v heads, every head padded to dim_p / vdim_p
+    // rows of the fused projection: q heads | k heads | v heads, every head padded to dim_p / vdim_p (q heads alone when the layer
+    // reads another one's cache)
     const float *lat;
     int stride, n_tok;
     int heads, kv_heads, dim, dim_p, v_dim, vdim_p;
     const float *bias;          // [q | k | v] or nullptr
-    int qk_norm;                // q and k divided by their root mean square after the rotation
+    int own_kv;                 // 0: the cache at c_off is another layer's
+    int qk_norm;                // RMS norm of q and k: 1 per head after the rotation, 2 / 3 ahead of it, per head / over all heads
+    const float *qk_gain;       // qk_norm 2: [q dim_p | k dim_p], 3: [q heads | k heads]
     float eps;
-    int rot_dims;               // pairs (i, i + rot_dims / 2)
+    int rot_dims, rot_adjacent; // pairs (i, i + rot_dims / 2), or (2 i, 2 i + 1)
     const float2 *rot;          // [positions][rot_dims / 2] (cos, sin), the frequency scaling's factor included
     void *q;                    // [n_tok][heads * dim_p]
     // pages: this layer's keys [kv head][slot][dim_p] at c_off, its values [kv head][slot][vdim_p] behind them
@@ -30,6 +33,9 @@ struct GqaArgs {
     void *o;                    // [n_tok][stride_o], heads x vdim_p
     int stride_o;
     float scale;
+    int window;                 // > 0: a position sees the `window` last ones up to itself
+    int sink;                   // one more key of score 0 without value
+    const float *gate;          // output gates before the sigmoid: gate[token * stride + head], or nullptr
     const int4 *reqs;           // (request of the round, first token, tokens, position of the first token)
     int n_reqs, max_len;        // longest of them in tokens
     int n_blocks;               // long form: blocks of 64 (token, head) rows of all requests
@@ -61,6 +67,7 @@ struct DeltaArgs {
     int heads, kv_heads, dk, dk_p, dv, dv_p, heads_p, taps;
     float eps;
     const float *conv;          // [taps][channels]
+    const float *conv_bias;     // [channels] or nullptr
     const float *decay;         // [2][heads_p]: logarithm of the rate, bias
     const float *norm;          // [dv_p]
     // state: inputs of the convolutions [generation][slot][taps - 1][channels], matrices [slot][head][dv_p][dk_p]
@@ -89,5 +96,32 @@ int delta_scan_launch(const DeltaArgs &a, cudaStream_t s, bool pdl);
 int delta_out_launch(const DeltaArgs &a, int dt, cudaStream_t s, bool pdl);
 // Rounds of one token per request: all of it in one launch, beside the attention's preparation (nullptr: none).
 int delta_decode_launch(const DeltaArgs &a, const GqaArgs *attn, int dt, cudaStream_t s, bool pdl);
+
+// ---- linear recurrences: S <- decay S + k v^T, o = S^T q
+// SSD: one decay per head, keys and queries of a group of heads behind short convolutions, values scaled by a step size; the
+// output takes D v up, is gated, then normed in parts of the whole width.  GLA: one decay per head and key channel, no
+// convolutions, output normed per head, then gated.  The rows of the fused projection are those of DeltaArgs with, behind the
+// output gate, SSD: step size (heads_p), GLA: the first map of the decays (rank_p).
+constexpr int SCAN_BLOCK = 16;                                      // tokens of a block of the scan
+constexpr int SCAN_COEF = SCAN_BLOCK * SCAN_BLOCK + 2 * SCAN_BLOCK; // coefficients of a block and head
+struct ScanArgs : DeltaArgs {   // decay: SSD [3][heads_p], weight of v behind the bias; norm: SSD [heads][dv_p]
+    int per_channel;            // GLA
+    const float *gate_map;      // GLA: [rank + 1][heads * dk_p]
+    int rank, rank_p;
+    float inv_tau, q_scale;
+    int parts;                  // SSD: parts of the output norm
+    const float *vin;           // values the scan reads: [n_tok][vin_stride], heads x dv_p
+    int vin_stride;
+    float *tail;                // GLA: decay over a block [slot][heads][dk_p]
+    __host__ __device__ int rec_rows() const { return b_off() + (per_channel ? rank_p : heads_p); }
+};
+// Portions in bf16 contexts: operands and coefficients of blocks; the scan.  Then scan_out.
+int scan_prep_launch(const ScanArgs &a, cudaStream_t s, bool pdl);
+int scan_launch(const ScanArgs &a, cudaStream_t s, bool pdl);
+// Token by token, everything up to the output's norm (GLA: with it): rounds of one token per request, beside the attention's
+// preparation, and portions of all-32-bit contexts (attn nullptr).
+int scan_step_launch(const ScanArgs &a, const GqaArgs *attn, int dt, cudaStream_t s, bool pdl);
+// SSD: gate and norm
+int scan_out_launch(const ScanArgs &a, int dt, cudaStream_t s, bool pdl);
 
 }  // namespace lcu

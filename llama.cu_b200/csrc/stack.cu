@@ -1,5 +1,6 @@
 // Rounds of models described layer by layer: shapes and storage, the plan of a round's attention, and the launches of every
 // layer.  Context, pages, descriptor staging, graphs and sampling are those of ctx.cu.
+#include "moe.cuh"
 #include "stack_round.cuh"
 
 #include <cmath>
@@ -48,9 +49,10 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
         LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_XIELU, "layer %d: unknown activation %d", i, l.ff_act);
         LCU_REQUIRE(!l.add_embed && !l.add_step, "layer %d: additions to the residual stream need pre-norm layers", i);
     } else {
-        const int most = MIX_MAX_HEAD;
-        LCU_REQUIRE(l.mixer > 0 && (l.mixer & ~(LCU_MIX_ATTENTION | LCU_MIX_DELTA)) == 0, "layer %d: unknown mixer %d", i, l.mixer);
-        LCU_REQUIRE(l.ff >= 0 && !l.token_shift, "layer %d: negative size, or a token shift", i);
+        const int most = MIX_MAX_HEAD, rec = l.mixer & (LCU_MIX_DELTA | LCU_MIX_SSD | LCU_MIX_GLA);
+        LCU_REQUIRE(l.mixer > 0 && (l.mixer & ~(LCU_MIX_ATTENTION | LCU_MIX_DELTA | LCU_MIX_SSD | LCU_MIX_GLA)) == 0 && (rec & (rec - 1)) == 0,
+                    "layer %d: unknown mixer %d", i, l.mixer);
+        LCU_REQUIRE(l.ff >= 0 && l.shared_ff >= 0 && l.experts >= 0 && !l.token_shift, "layer %d: negative size, or a token shift", i);
         if (l.mixer & LCU_MIX_ATTENTION) {
             LCU_REQUIRE(l.heads > 0 && l.kv_heads > 0 && l.heads % l.kv_heads == 0, "layer %d: %d query heads, %d key heads", i, l.heads, l.kv_heads);
             LCU_REQUIRE(l.dim > 0 && l.dim <= most && l.v_dim > 0 && l.v_dim <= most, "layer %d: head sizes %d / %d (1..%d)", i, l.dim, l.v_dim, most);
@@ -58,16 +60,38 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
                         "layer %d: %d rotated dimensions of %d, base %g", i, l.rot_dims, l.dim, l.rot_base);
             LCU_REQUIRE(l.rot_dims == 0 || l.rot_factor <= 0 || (l.rot_original > 0 && l.rot_fast > 0 && l.rot_slow > 0 && l.rot_base != 1),
                         "layer %d: frequency scaling by %g needs positive constants", i, l.rot_factor);
+            LCU_REQUIRE(l.qk_norm >= 0 && l.qk_norm <= 3 && l.window >= 0, "layer %d: norm %d of queries and keys, window of %d", i, l.qk_norm, l.window);
+            LCU_REQUIRE(l.kv_from >= 0 && l.kv_from <= i, "layer %d: keys and values of layer %d", i, l.kv_from - 1);
+            if (l.kv_from) {
+                const lcu_layer_desc &o = layers[l.kv_from - 1];
+                LCU_REQUIRE((o.mixer & LCU_MIX_ATTENTION) && !o.kv_from && o.kv_heads == l.kv_heads && o.dim == l.dim && o.v_dim == l.v_dim,
+                            "layer %d: the keys and values of layer %d do not fit", i, l.kv_from - 1);
+            }
         }
-        if (l.mixer & LCU_MIX_DELTA) {
+        if (rec) {
             LCU_REQUIRE(l.delta_heads > 0 && l.delta_kv_heads > 0 && l.delta_heads % l.delta_kv_heads == 0, "layer %d: %d value heads, %d key heads", i,
                         l.delta_heads, l.delta_kv_heads);
             LCU_REQUIRE(l.delta_dim > 0 && l.delta_dim <= most && l.delta_v_dim > 0 && l.delta_v_dim <= most, "layer %d: head sizes %d / %d (1..%d)", i,
                         l.delta_dim, l.delta_v_dim, most);
-            LCU_REQUIRE(l.delta_conv >= 1 && l.delta_conv <= 64, "layer %d: convolution of %d taps (1..64)", i, l.delta_conv);
+            LCU_REQUIRE(rec == LCU_MIX_GLA || (l.delta_conv >= 1 && l.delta_conv <= 64), "layer %d: convolution of %d taps (1..64)", i, l.delta_conv);
+            LCU_REQUIRE(rec != LCU_MIX_SSD || (l.norm_parts > 0 && l.delta_heads * l.delta_v_dim % l.norm_parts == 0), "layer %d: norm of %d values in %d parts", i,
+                        l.delta_heads * l.delta_v_dim, l.norm_parts);
+            LCU_REQUIRE(rec != LCU_MIX_GLA || (l.gate_rank > 0 && l.gate_rank <= 1024 && l.gate_tau > 0 && l.delta_kv_heads == l.delta_heads),
+                        "layer %d: decays of rank %d, tau %g, %d key heads for %d", i, l.gate_rank, l.gate_tau, l.delta_kv_heads, l.delta_heads);
         }
-        LCU_REQUIRE(l.ff == 0 || l.ff_act == LCU_ACT_RELU2, "layer %d: unknown activation %d", i, l.ff_act);
+        LCU_REQUIRE((l.mixer & LCU_MIX_ATTENTION) == 0 || rec == 0 || (rec == LCU_MIX_DELTA) == (l.post_norm == 0),
+                    "layer %d: side by side, outputs of a delta rule are normed one by one, those of other mixers added ahead of a norm", i);
+        const bool ff = l.ff > 0 || l.shared_ff > 0;
+        LCU_REQUIRE(!ff || l.ff_act == LCU_ACT_RELU2 || l.ff_act == LCU_ACT_GLU, "layer %d: unknown activation %d", i, l.ff_act);
+        LCU_REQUIRE(l.experts == 0 ? l.shared_ff == 0 : (l.ff_act == LCU_ACT_GLU && l.ff > 0 && l.top > 0 && l.top <= l.experts && l.post_norm),
+                    "layer %d: %d experts, %d per token, widths %d and %d", i, l.experts, l.top, l.ff, l.shared_ff);
+        LCU_REQUIRE(l.experts <= 4096 && l.experts * 12 + MOE_SMALL_ROUND * l.top * 8 <= 48 * 1024, "layer %d: %d experts, %d per token", i, l.experts, l.top);
+        LCU_REQUIRE(!ff || l.ff_act != LCU_ACT_GLU || (l.glu_limit > 0 && (l.shared_ff == 0 || l.shared_limit > 0)), "layer %d: limit %g of a gated activation", i, l.glu_limit);
+        LCU_REQUIRE((l.post_norm != 0) == (layers[0].post_norm != 0), "layer %d: norms on outputs in some layers only", i);
     }
+    if (i == 0)
+        LCU_REQUIRE(l.pair_buckets >= 0 && l.pair_prev >= 0 && l.pair_cur >= 0 && (l.pair_buckets == 0 || (l.pre_norm && l.pair_prev < l.pair_buckets && l.pair_cur < l.pair_buckets)),
+                    "embedding of token pairs: %d buckets, factors %d and %d", l.pair_buckets, l.pair_prev, l.pair_cur);
     LCU_REQUIRE(l.weights_of >= -1 && l.weights_of < d.n_layers && l.weights_of != i, "layer %d uses the weights of layer %d", i, l.weights_of);
     return LCU_OK;
 }
@@ -75,7 +99,8 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
 // Fewest split CTAs per SM that keep a decode round's copies in flight: two waves of what fits.
 static int gqa_target_ctas(const StackLayer &L) { return 2 * sm_count() * gqa_short_ctas_per_sm(L.dim_p, L.vdim_p); }
 int gqa_splits_for(const lcu_ctx *c, const StackLayer &L, int reqs, int len) {
-    const int ctas = reqs * L.d.kv_heads * gqa_row_tiles(L.d.heads, L.d.kv_heads, len), units = (c->desc.nctx + 63) / 64;
+    const int ctas = reqs * L.d.kv_heads * gqa_row_tiles(L.d.heads, L.d.kv_heads, len);
+    const int seen = L.d.window > 0 && L.d.window + len < c->desc.nctx ? L.d.window + len + 63 : c->desc.nctx, units = (seen + 63) / 64;
     int z = ctas > 0 ? gqa_target_ctas(L) / ctas : 1;
     if (z > 64) z = 64;
     if (z > units) z = units;
@@ -124,10 +149,10 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->w.resize(d.n_layers);
     size_t off = 0;
     int max_lat = 0, max_qr = 0, max_q = 0, max_hr = 0, max_hv = 64, max_ff = 64, max_kv = 0;
-    int max_dk = 0, max_dv = 0, max_dh = 0, max_dhv = 0, max_vp = 0;
+    int max_dk = 0, max_dv = 0, max_coef = 0, max_tail = 0, max_dhv = 0, max_vp = 0, max_top = 0, max_ep = 0, max_eff = 0;
     size_t conv_total = 0, mat_total = 0;  // f32 values of recurrent state per slot
     S->pre_norm = layers[0].pre_norm != 0;
-    bool any_shift = false, any_delta = false, can_expand = c->dt != LCU_F32 && !S->pre_norm;
+    bool any_shift = false, any_rec = layers[0].pair_buckets > 0, can_expand = c->dt != LCU_F32 && !S->pre_norm;
     for (int i = 0; i < d.n_layers; ++i) {
         StackLayer &L = S->layers[i];
         L.d = layers[i];
@@ -141,7 +166,8 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                         o.out_gate == L.d.out_gate && o.ff == L.d.ff && o.token_shift == L.d.token_shift && o.mixer == L.d.mixer &&
                         o.kv_heads == L.d.kv_heads && o.bias == L.d.bias && o.delta_heads == L.d.delta_heads &&
                         o.delta_kv_heads == L.d.delta_kv_heads && o.delta_dim == L.d.delta_dim && o.delta_v_dim == L.d.delta_v_dim &&
-                        o.delta_conv == L.d.delta_conv,
+                        o.delta_conv == L.d.delta_conv && o.qk_norm == L.d.qk_norm && o.kv_from == L.d.kv_from && o.norm_parts == L.d.norm_parts &&
+                        o.gate_rank == L.d.gate_rank && o.experts == L.d.experts && o.shared_ff == L.d.shared_ff && o.ff_act == L.d.ff_act,
                     "layer %d differs from layer %d whose weights it uses", i, L.src);
         auto up = [](int &m, int v) { if (v > m) m = v; };
         L.ff_p = stack_pad(L.d.ff, 64);
@@ -164,8 +190,11 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
             L.dim_p = stack_pad(L.d.dim, 16);
             L.vdim_p = stack_pad(L.d.v_dim, 16);
             L.hv_p = stack_pad(L.d.heads * L.vdim_p, 64);
-            L.att_rows = (L.d.heads + L.d.kv_heads) * L.dim_p + L.d.kv_heads * L.vdim_p;
-            off += (size_t)L.d.kv_heads * (L.dim_p + L.vdim_p) * c->geom.page_tokens;
+            L.att_rows = L.d.heads * L.dim_p + (L.own_kv() ? L.d.kv_heads * (L.dim_p + L.vdim_p) : 0);
+            L.g_p = L.d.out_gate ? stack_pad(L.d.heads, 8) : 0;
+            L.kv_src = L.own_kv() ? i : L.d.kv_from - 1;
+            if (L.own_kv()) off += (size_t)L.d.kv_heads * (L.dim_p + L.vdim_p) * c->geom.page_tokens;
+            else L.c_off = S->layers[L.kv_src].c_off;
             up(max_q, L.d.heads * L.dim_p); up(max_vp, L.vdim_p);
             if (gqa_target_ctas(L) > S->gqa_ctas) S->gqa_ctas = gqa_target_ctas(L);
             for (int j = 0; j < i && !L.rot; ++j) {  // layers with the same rotation share a table
@@ -179,27 +208,38 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                 if (rc) return rc;
             }
         }
-        if (L.delta()) {
+        if (L.recurrent()) {
             L.dk_p = stack_pad(L.d.delta_dim, 32);
             L.dv_p = stack_pad(L.d.delta_v_dim, 16);
             L.dh_p = stack_pad(L.d.delta_heads, 8);
             L.dhv_p = stack_pad(L.d.delta_heads * L.dv_p, 64);
             L.conv_off = conv_total;
-            conv_total += (size_t)(L.d.delta_conv - 1) * L.conv_channels();
+            if (L.conv_channels()) conv_total += (size_t)(L.d.delta_conv - 1) * L.conv_channels();
+            if (L.gla()) L.rank_p = stack_pad(L.d.gate_rank, 8);
             L.mat_off = mat_total;
             mat_total += (size_t)L.d.delta_heads * L.dv_p * L.dk_p;
-            any_delta = true;
-            up(max_dk, L.d.delta_kv_heads * L.dk_p); up(max_dv, L.d.delta_heads * L.dv_p); up(max_dh, L.d.delta_heads); up(max_dhv, L.dhv_p);
+            any_rec = true;
+            const int coef = L.delta() ? DELTA_COEF * SCAN_BLOCK / DELTA_BLOCK : SCAN_COEF;
+            up(max_coef, L.d.delta_heads * coef);
+            if (L.gla()) up(max_tail, L.d.delta_heads * L.dk_p);
+            up(max_dk, L.d.delta_kv_heads * L.dk_p); up(max_dv, L.d.delta_heads * L.dv_p); up(max_dhv, L.dhv_p);
+        }
+        if (L.d.shared_ff) { L.sff_p = stack_pad(L.d.shared_ff, 64); up(max_ff, L.sff_p); }
+        if (L.d.experts) {
+            L.e_p = stack_pad(L.d.experts, 8);
+            up(max_ep, L.e_p); up(max_top, L.d.top); up(max_eff, L.ff_p); up(S->max_experts, L.d.experts);
         }
         up(max_lat, L.in_rows()); up(max_qr, L.qr_p); up(max_hv, L.hv_p);
     }
     c->geom.page_elems = off;
     if (off == 0) c->geom.page_elems = 8;  // nothing is cached per token: pages still count tokens
-    S->n_slots = any_shift || any_delta ? c->max_seqs : 0;
+    S->n_slots = any_shift || any_rec ? c->max_seqs : 0;
     c->free_slots.clear();
     for (int i = S->n_slots - 1; i >= 0; --i) c->free_slots.push_back(i);
 
     const size_t T = (size_t)c->max_tokens, eb = act_bytes(c);
+    S->max_rows = c->max_tokens * max_top;
+    S->n_tiles = max_top ? moe_max_tiles(S->max_rows, S->max_experts, 64) : 0;
     S->abs_cap = c->max_tokens;
     S->conv_gen = conv_total * S->n_slots;
     S->expand_cap = can_expand ? stack_pad(d.nctx > c->max_tokens ? d.nctx : c->max_tokens, 64) : 0;
@@ -223,9 +263,11 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                  o_xc = reserve((size_t)S->expand_cap * S->max_r * eb), o_xkv = reserve((size_t)S->expand_cap * max_kv * eb),
                  o_hout = reserve((T > (size_t)c->max_seqs ? T : c->max_seqs) * S->d_p * eb), o_po = reserve(rows * S->max_r * 4),
                  o_pml = reserve(rows * 2 * 4), o_pn = reserve(T * S->max_heads * 4), o_y2 = reserve(S->pre_norm ? T * S->d_p * 4 : 0),
-                 o_dq = reserve(T * max_dk * 6), o_dk = reserve(T * max_dk * 6), o_dv = reserve(T * max_dv * 4), o_dg = reserve((T / DELTA_BLOCK + c->max_seqs + 1) * max_dh * DELTA_COEF * 4),
+                 o_dq = reserve(T * max_dk * 6), o_dk = reserve(T * max_dk * 6), o_dv = reserve(T * max_dv * 4), o_dg = reserve((T / SCAN_BLOCK + c->max_seqs + 1) * (size_t)max_coef * 4), o_dt = reserve((T / SCAN_BLOCK + c->max_seqs + 1) * (size_t)max_tail * 4),
                  o_att2 = reserve(T * max_dhv * eb), o_conv = reserve(2 * S->conv_gen * 4), o_mat = reserve(mat_total * S->n_slots * 4),
                  o_gp = reserve(gqa_part_floats(S->gqa_ctas, max_vp) * 4), o_gt = reserve((size_t)S->gqa_ctas * 4);
+    const size_t R = S->max_rows, o_lt = reserve((size_t)2 * S->n_slots * 4), o_ro = reserve(T * max_ep * 4), o_ye = reserve(R * S->d_p * 4), o_mi = reserve(R * 16), o_mw = reserve(R * 8),
+                 o_mc = reserve((size_t)S->max_experts * 4), o_mt = reserve((size_t)S->n_tiles * 16), o_xg = reserve(R * S->d_p * eb), o_ae = reserve(R * max_eff * eb);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
     LCU_CHECK_CUDA(cudaMemset(S->arena, 0, total));  // pads of att (columns past the heads) stay zero from here on
     unsigned char *p = reinterpret_cast<unsigned char *>(S->arena);
@@ -240,6 +282,11 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->conv_state = reinterpret_cast<float *>(p + o_conv); S->mat_state = reinterpret_cast<float *>(p + o_mat);
     S->gqa_part = reinterpret_cast<float *>(p + o_gp); S->gqa_tickets = reinterpret_cast<unsigned *>(p + o_gt);
 
+    S->dtail = reinterpret_cast<float *>(p + o_dt); S->last_token = reinterpret_cast<uint32_t *>(p + o_lt);
+    S->router = reinterpret_cast<float *>(p + o_ro); S->ye = reinterpret_cast<float *>(p + o_ye); S->moe_ints = reinterpret_cast<int *>(p + o_mi);
+    S->moe_w = reinterpret_cast<float *>(p + o_mw); S->moe_slot_w = S->moe_w + R; S->moe_count = reinterpret_cast<unsigned *>(p + o_mc);
+    S->moe_tiles = reinterpret_cast<int4 *>(p + o_mt); S->xg = p + o_xg; S->act_e = p + o_ae;
+
     // every kernel variant a round can launch
     if (S->pre_norm) {
         if (c->dt == LCU_F32) return LCU_OK;
@@ -251,9 +298,10 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
             if (!rc && L.attention()) rc = gqa_long_launch(g, nullptr, true);
             if (!rc) rc = gemv_warm(S->d_p, L.in_rows(), false, c->dt, EPI_STORE_F32);
             if (!rc && L.attention()) rc = gemv_warm(L.hv_p, S->d_p, false, c->dt, EPI_STORE_F32);
-            if (!rc && L.delta()) rc = gemv_warm(L.dhv_p, S->d_p, false, c->dt, EPI_STORE_F32);
-            if (!rc && L.d.ff) rc = gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_RELU2);
-            if (!rc && L.d.ff) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
+            if (!rc && L.recurrent()) rc = gemv_warm(L.dhv_p, S->d_p, false, c->dt, EPI_STORE_F32);
+            if (!rc && L.d.experts) rc = gemv_warm(S->d_p, L.e_p, false, c->dt, EPI_STORE_F32);
+            else if (!rc && L.d.ff) rc = L.glu() ? gemv_warm(S->d_p, 2 * L.ff_p, false, c->dt, EPI_GLU) : gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_RELU2);
+            if (!rc && L.d.ff && !L.d.experts) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
         }
         if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt);
         if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, EPI_STORE_F32);
@@ -301,6 +349,7 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
     case LCU_W_EMBD: *rows = c->desc.vocab; *cols = S.d_p; return true;
     case LCU_W_LM_HEAD: *rows = S.vocab_p; *cols = S.d_p; return true;
     case LCU_W_OUT_NORM: *rows = 1; *cols = S.pre_norm ? S.d_p : 1; *elem_bytes = 4; return true;
+    case LCU_W_PAIR_EMBD: *rows = S.layers[0].d.pair_buckets + 1; *cols = S.d_p; return S.layers[0].d.pair_buckets > 0;
     default: break;
     }
     if (layer < 0 || layer >= c->desc.n_layers) return false;
@@ -309,21 +358,29 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
     if (kind == LCU_W_STEP) return f32(1, S.d_p, L.d.add_step != 0);
     if (L.src != layer) return false;
     switch (kind) {
-    case LCU_W_UP: *rows = L.ff_p; *cols = S.d_p; return L.d.ff > 0;
-    case LCU_W_FF_DOWN: *rows = S.d_p; *cols = L.ff_p; return L.d.ff > 0;
+    case LCU_W_UP: *rows = (L.d.experts ? L.d.experts : 1) * (L.glu() ? 2 : 1) * L.ff_p; *cols = S.d_p; return L.d.ff > 0;
+    case LCU_W_FF_DOWN: *rows = (L.d.experts ? L.d.experts : 1) * S.d_p; *cols = L.ff_p; return L.d.ff > 0;
     default: break;
     }
     if (S.pre_norm) switch (kind) {
     case LCU_W_MIX_IN: *rows = L.in_rows(); *cols = S.d_p; return true;
     case LCU_W_MIX_BIAS: return f32(1, L.att_rows, L.attention() && L.d.bias);
     case LCU_W_ATT_OUT: *rows = S.d_p; *cols = L.hv_p; return L.attention();
-    case LCU_W_DELTA_OUT: *rows = S.d_p; *cols = L.dhv_p; return L.delta();
-    case LCU_W_CONV: return f32(L.d.delta_conv, L.conv_channels(), L.delta());
-    case LCU_W_DELTA_DECAY: return f32(2, L.dh_p, L.delta());
-    case LCU_W_DELTA_NORM: return f32(1, L.dv_p, L.delta());
+    case LCU_W_DELTA_OUT: *rows = S.d_p; *cols = L.dhv_p; return L.recurrent();
+    case LCU_W_QK_GAIN: return L.d.qk_norm == 2 ? f32(1, 2 * L.dim_p, L.attention()) : f32(1, (L.d.heads + (L.own_kv() ? L.d.kv_heads : 0)) * L.dim_p, L.attention() && L.d.qk_norm == 3);
+    case LCU_W_CONV: return f32(L.d.delta_conv, L.conv_channels(), L.conv_channels() > 0);
+    case LCU_W_CONV_BIAS: return f32(1, L.conv_channels(), L.ssd());
+    case LCU_W_DELTA_DECAY: return f32(L.ssd() ? 3 : 2, L.dh_p, L.delta() || L.ssd());
+    case LCU_W_GATE_MAP: return f32(L.d.gate_rank + 1, L.d.delta_heads * L.dk_p, L.gla());
+    case LCU_W_DELTA_NORM: return f32(1, L.ssd() ? L.d.delta_heads * L.dv_p : L.dv_p, L.recurrent());
     case LCU_W_BRANCH_NORM: return f32(2, S.d_p, L.attention() && L.delta());
     case LCU_W_NORM1: return f32(1, S.d_p, true);
-    case LCU_W_NORM2: return f32(1, S.d_p, L.d.ff > 0);
+    case LCU_W_NORM2: return f32(1, S.d_p, L.has_ff());
+    case LCU_W_POST1: return f32(1, S.d_p, L.d.post_norm != 0);
+    case LCU_W_POST2: return f32(1, S.d_p, L.d.post_norm && L.has_ff());
+    case LCU_W_ROUTER: *rows = L.e_p; *cols = S.d_p; return L.d.experts > 0;
+    case LCU_W_SHARED_UP: *rows = 2 * L.sff_p; *cols = S.d_p; return L.d.shared_ff > 0;
+    case LCU_W_SHARED_DOWN: *rows = S.d_p; *cols = L.sff_p; return L.d.shared_ff > 0;
     default: return false;
     }
     switch (kind) {
@@ -341,6 +398,10 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
 }
 
 int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
+    if (kind == LCU_W_PAIR_EMBD) {
+        c->stack->pair_embd = ptr;
+        return LCU_OK;
+    }
     StackWeights &w = c->stack->w[layer];
     const float *f = reinterpret_cast<const float *>(ptr);
     switch (kind) {
@@ -355,6 +416,14 @@ int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
     case LCU_W_NORM1: w.norm1 = f; break;
     case LCU_W_NORM2: w.norm2 = f; break;
     case LCU_W_STEP: w.step = f; break;
+    case LCU_W_POST1: w.post1 = f; break;
+    case LCU_W_POST2: w.post2 = f; break;
+    case LCU_W_QK_GAIN: w.qk_gain = f; break;
+    case LCU_W_CONV_BIAS: w.conv_bias = f; break;
+    case LCU_W_GATE_MAP: w.gate_map = f; break;
+    case LCU_W_ROUTER: w.router = ptr; break;
+    case LCU_W_SHARED_UP: w.shared_up = ptr; break;
+    case LCU_W_SHARED_DOWN: w.shared_down = ptr; break;
     case LCU_W_LAT_IN: w.in = ptr; break;
     case LCU_W_Q_NORM: w.q_norm = ptr; break;
     case LCU_W_KV_NORM: w.kv_norm = ptr; break;
@@ -373,6 +442,10 @@ int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
 
 bool stack_ready(const lcu_ctx *c) {
     const Stack &S = *c->stack;
+    if (S.layers[0].d.pair_buckets && !S.pair_embd) {
+        set_error("step: the embedding of token pairs is missing");
+        return false;
+    }
     for (size_t i = 0; i < S.layers.size(); ++i) {
         const StackWeights &w = S.w[i];
         const StackLayer &L = S.layers[i];
@@ -381,9 +454,11 @@ bool stack_ready(const lcu_ctx *c) {
         if (L.src == (int)i) {
             ok = ok && w.in && (!d.ff || (w.up && w.down)) && (!d.token_shift || w.shift);
             if (L.latent()) ok = ok && w.q_norm && w.kv_norm && w.uq && w.ukt && w.ukv && w.out && w.scalars;
-            if (L.attention()) ok = ok && w.att_out && (!d.bias || w.bias);
-            if (L.delta()) ok = ok && w.delta_out && w.conv && w.decay && w.delta_norm;
-            if (S.pre_norm) ok = ok && w.norm1 && (!d.ff || w.norm2) && (!(L.attention() && L.delta()) || w.branch_norm);
+            if (L.attention()) ok = ok && w.att_out && (!d.bias || w.bias) && (d.qk_norm < 2 || w.qk_gain);
+            if (L.recurrent()) ok = ok && w.delta_out && w.delta_norm && (L.gla() ? w.gate_map != nullptr : w.conv && w.decay) && (!L.ssd() || w.conv_bias);
+            if (S.pre_norm) ok = ok && w.norm1 && (!L.has_ff() || w.norm2) && (!(L.attention() && L.delta()) || w.branch_norm);
+            if (d.post_norm) ok = ok && w.post1 && (!L.has_ff() || w.post2);
+            ok = ok && (!d.experts || w.router) && (!d.shared_ff || (w.shared_up && w.shared_down));
         }
         if (!ok) {
             set_error("step: weights of layer %zu missing", i);
@@ -405,7 +480,7 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
             *slot = reinterpret_cast<int32_t *>(B + D.req_slot), *afirst = reinterpret_cast<int32_t *>(B + D.abs_first),
             *aid = reinterpret_cast<int32_t *>(B + D.abs_id), *atok = reinterpret_cast<int32_t *>(B + D.abs_tok);
     int4 *xreq = reinterpret_cast<int4 *>(B + D.xreq), *xg = reinterpret_cast<int4 *>(B + D.xgroups);
-    int4 *sreq = reinterpret_cast<int4 *>(B + D.sreq), *lreq = reinterpret_cast<int4 *>(B + D.lreq), *dblk = reinterpret_cast<int4 *>(B + D.dblk);
+    int4 *sreq = reinterpret_cast<int4 *>(B + D.sreq), *lreq = reinterpret_cast<int4 *>(B + D.lreq), *dblk = reinterpret_cast<int4 *>(B + D.dblk), *sblk = reinterpret_cast<int4 *>(B + D.sblk);
     int short_max = 1 << 30;  // one decision per request and round: the layer with the largest head groups decides
     for (const StackLayer &L : S.layers)
         if (L.attention()) { const int v = gqa_short_tokens(L.d.heads, L.d.kv_heads); if (v < short_max) short_max = v; }
@@ -428,6 +503,8 @@ int stack_stage(lcu_ctx *c, Round &r, const lcu_req *reqs, unsigned char *H) {
             }
             for (int j = 0; j < len; j += DELTA_BLOCK)
                 dblk[q.n_delta_blocks++] = make_int4(i, t + j, len - j < DELTA_BLOCK ? len - j : DELTA_BLOCK, t / DELTA_BLOCK + i + j / DELTA_BLOCK);
+            for (int j = 0; j < len; j += SCAN_BLOCK)
+                sblk[q.n_scan_blocks++] = make_int4(i, t + j, len - j < SCAN_BLOCK ? len - j : SCAN_BLOCK, t / SCAN_BLOCK + i + j / SCAN_BLOCK);
         } else if (len < expand_min) {
             aid[q.n_abs_req] = i;
             afirst[q.n_abs_req++] = q.n_abs_tok;
@@ -645,12 +722,21 @@ double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_
     double bytes = n_out ? (double)S.vocab_p * S.d_p * wb : 0.0;
     for (const StackLayer &L : S.layers) {
         const lcu_layer_desc &d = L.d;
-        bytes += wb * ((double)L.in_rows() * S.d_p + 2.0 * L.ff_p * S.d_p + (double)S.d_p * (L.hv_p + L.dhv_p));
+        double ff = (L.glu() ? 3.0 : 2.0) * L.ff_p * S.d_p;
+        if (d.experts) {  // the experts that this many tokens use when they choose evenly
+            double tokens = 0.0;
+            for (int i = 0; i < n_req; ++i) tokens += reqs[i].len;
+            ff *= d.experts * (1.0 - pow(1.0 - (double)d.top / d.experts, tokens));
+        }
+        bytes += wb * ((double)L.in_rows() * S.d_p + ff + 3.0 * L.sff_p * S.d_p + (double)L.e_p * S.d_p + (double)S.d_p * (L.hv_p + L.dhv_p));
         if (L.latent()) bytes += wb * ((double)d.heads * L.dim_p * L.qr_p + (double)L.kv_cols() * L.r_p);
         const double row = L.latent() ? L.r_p : (L.attention() ? (double)d.kv_heads * (L.dim_p + L.vdim_p) : 0.0);
         for (int i = 0; i < n_req; ++i) {
-            for (uint32_t j = 0; j < reqs[i].len; ++j) bytes += (double)(reqs[i].pos + j + 1) * row * eb;
-            if (L.delta()) bytes += 8.0 * d.delta_heads * L.dv_p * L.dk_p;  // matrices read and written
+            for (uint32_t j = 0; j < reqs[i].len; ++j) {
+                const uint32_t seen = reqs[i].pos + j + 1;
+                bytes += (double)(d.window > 0 && seen > (uint32_t)d.window ? (uint32_t)d.window : seen) * row * eb;
+            }
+            if (L.recurrent()) bytes += 8.0 * d.delta_heads * L.dv_p * L.dk_p;  // matrices read and written
         }
     }
     return bytes;

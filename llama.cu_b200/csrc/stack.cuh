@@ -11,6 +11,7 @@
 #include <vector>
 
 #include "common.cuh"
+#include "gemv.cuh"
 #include "mixers.cuh"
 
 struct lcu_ctx;
@@ -25,17 +26,26 @@ struct StackLayer {
     size_t c_off;   // element offset of this layer's cached rows inside a page: [page_tokens][r_p]
     // padded sizes
     int dim_p, vdim_p, qr_p, r_p, g_p, ff_p, hv_p;
-    // softmax attention and delta rule
-    int att_rows = 0;                     // rows of the fused input projection that are the attention's (the first ones)
-    int dk_p = 0, dv_p = 0, dh_p = 0, dhv_p = 0;
+    // softmax attention and recurrent mixers
+    int att_rows = 0;                     // rows of the fused input projection that are the attention's q, k, v (the first ones; g_p head gates behind them)
+    int kv_src = 0;                       // layer whose cache this one reads
+    int dk_p = 0, dv_p = 0, dh_p = 0, dhv_p = 0, rank_p = 0;
+    int e_p = 0, sff_p = 0;               // experts, width of the shared one
     size_t conv_off = 0, mat_off = 0;     // f32 offsets of this layer's recurrent state in its arena section
     const float2 *rot = nullptr;          // [nctx][rot_dims / 2] (cos, sin)
     bool latent() const { return d.mixer == LCU_MIX_LATENT; }
     bool attention() const { return (d.mixer & LCU_MIX_ATTENTION) != 0; }
     bool delta() const { return (d.mixer & LCU_MIX_DELTA) != 0; }
-    int delta_rows() const { return delta() ? 2 * d.delta_kv_heads * dk_p + 2 * d.delta_heads * dv_p + 2 * dh_p : 0; }
-    int conv_channels() const { return 2 * d.delta_kv_heads * dk_p + d.delta_heads * dv_p; }
-    int in_rows() const { return latent() ? qr_p + r_p + g_p : att_rows + delta_rows(); }  // rows of the fused input projection: query latent | latent | gate, or attention | delta rule
+    bool ssd() const { return (d.mixer & LCU_MIX_SSD) != 0; }
+    bool gla() const { return (d.mixer & LCU_MIX_GLA) != 0; }
+    bool recurrent() const { return delta() || ssd() || gla(); }
+    bool own_kv() const { return d.kv_from == 0; }
+    bool glu() const { return d.ff_act == LCU_ACT_GLU; }
+    bool has_ff() const { return d.ff > 0 || d.shared_ff > 0; }
+    int qkv_rows() const { return 2 * d.delta_kv_heads * dk_p + d.delta_heads * dv_p; }  // of a recurrent mixer
+    int rec_rows() const { return recurrent() ? qkv_rows() + d.delta_heads * dv_p + (gla() ? rank_p : ssd() ? dh_p : 2 * dh_p) : 0; }
+    int conv_channels() const { return gla() ? 0 : qkv_rows(); }
+    int in_rows() const { return latent() ? qr_p + r_p + g_p : att_rows + g_p + rec_rows(); }  // rows of the fused input projection: query latent | latent | gate, or attention | recurrent mixer
     int kv_cols() const { return d.heads * (dim_p + vdim_p); }  // columns of the expanded keys and values
 };
 
@@ -46,7 +56,8 @@ struct StackWeights {
     // pre-norm layers
     const void *att_out = nullptr, *delta_out = nullptr;
     const float *bias = nullptr, *conv = nullptr, *decay = nullptr, *delta_norm = nullptr, *branch_norm = nullptr, *norm1 = nullptr,
-                *norm2 = nullptr, *step = nullptr;
+                *norm2 = nullptr, *step = nullptr, *post1 = nullptr, *post2 = nullptr, *qk_gain = nullptr, *conv_bias = nullptr, *gate_map = nullptr;
+    const void *router = nullptr, *shared_up = nullptr, *shared_down = nullptr;
 };
 
 // What the host decides about a round: which requests run their attention in latent space ("absorbed") and which expand
@@ -59,7 +70,7 @@ struct StackRound {
     // softmax attention: requests whose portion takes the short form, and those that take the long one
     int n_short = 0, max_short = 0, n_long = 0;
     std::vector<int> long_len;
-    int n_delta_blocks = 0;  // delta rule: blocks of tokens
+    int n_delta_blocks = 0, n_scan_blocks = 0;  // recurrent mixers: blocks of tokens
 };
 
 struct Stack {
@@ -86,6 +97,16 @@ struct Stack {
     size_t conv_gen = 0;    // f32 values of one generation of the convolutions' state
     int gqa_ctas = 0;       // CTAs of split short-form attention the partial buffer holds
     std::vector<float2 *> rot_tables;
+    const void *pair_embd = nullptr;
+    uint32_t *last_token = nullptr;  // [generation 2][slots]
+    float *dtail = nullptr;          // linear recurrences: decays over blocks
+    // experts: routing, lists, activations in slot order, products
+    float *router = nullptr, *ye = nullptr, *moe_w = nullptr, *moe_slot_w = nullptr;
+    int *moe_ints = nullptr;         // expert, place, slot_of, slot_tok: [max_tokens * top] each
+    unsigned *moe_count = nullptr;
+    int4 *moe_tiles = nullptr;
+    void *xg = nullptr, *act_e = nullptr;
+    int max_rows = 0, max_experts = 0, n_tiles = 0;  // capacities
 };
 
 // ---- stack.cu
@@ -93,7 +114,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers);
 void stack_destroy(lcu_ctx *c);
 size_t stack_page_elems(const Stack &s, int page_tokens);
 bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *cols, int *elem_bytes);
-int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr);
+int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr);  // layer < 0: a weight of the model
 bool stack_ready(const lcu_ctx *c);
 size_t stack_desc_bytes(int max_tok, int max_req);
 struct Round;
@@ -127,20 +148,36 @@ struct MixInputArgs {
     const int32_t *tok_req, *req_first, *req_pos, *req_slot;  // request of a token; first token, position, slot * 2 + generation of a request
 };
 int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl);
-// Pre-norm layers: x_out = x_in + sum of the sublayer's outputs y (each y * y_gain / rms(y) when gains are given) + embedding row
-// + step, then h = gain * x_out / rms(x_out), rounded to the activation dtype; every input and h may be missing.
+// Pre-norm layers: x_out = x_in + the sublayer's output + embedding + step, then h = gain * x_out / rms(x_out), rounded to the
+// activation dtype; every input and h may be missing.  The sublayer's output is one of
+//     sum of y (each y * y_gain / rms(y) when gains are given)
+//     post_gain * s / rms(s), s = sum of y_scale * y and of the token's rows of ye
 struct PreNormArgs {
     const float *x_in;
     const float *y[2];
     const float *y_gain;  // [2][d_p]
-    const void *embd;     // bf16 [vocab, d_p]
+    const float *post_gain;
+    float y_scale[2];
+    const float *ye;      // outputs of experts [slot][d_p], `top` slots per token
+    const int *slot_of;
+    int top;
+    const void *embd;     // bf16 [vocab, d_p], times embd_scale
+    float embd_scale;
     const uint32_t *tokens;
+    // embedding of token pairs: bf16 [buckets + 1, d_p]; a sequence's last token is kept per (generation, slot)
+    const void *pair_embd;
+    int pair_buckets, pair_prev, pair_cur;
+    uint32_t *last_token;
+    size_t last_gen_stride;
+    const int32_t *tok_req, *req_first, *req_pos, *req_slot;
     const float *step;
     float *x_out;
     void *h;
     const float *gain;
     float eps;
     int n_tok, d, d_p;
+    unsigned *zero;       // counters that the kernels behind expect to be zero
+    int n_zero;
 };
 int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl);
 // y = x[rows[i]] * gain / rms(x), rounded
@@ -159,10 +196,14 @@ struct LinearF32Args {
     int stride_y, head_y;
     const int32_t *y_rows;      // optional row scatter
     int n, in, out, heads;
-    int epilogue;               // EPI_STORE_F32, EPI_XIELU
+    int epilogue;               // EPI_STORE_F32, EPI_XIELU, EPI_RELU2, EPI_GLU
     const float *act_pq;
     const float *gate;          // optional: multiplied by sigmoid(gate[y row * stride_gate + head])
     int stride_gate;
+    GluArgs glu;                // EPI_GLU
+    const int4 *tiles;          // grouped: (matrix, first row, rows up to 64), `heads` 1, no gather; see GemvArgs
+    int n_tiles;
+    const float *row_scale;
 };
 int linear_f32_launch(const LinearF32Args &a, cudaStream_t s);
 

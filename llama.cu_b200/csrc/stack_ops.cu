@@ -97,6 +97,16 @@ int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl) {
     return dt == LCU_F32 ? mix_input_t<float>(a, s, pdl) : mix_input_t<__nv_bfloat16>(a, s, pdl);
 }
 
+// Row of the pair table for token t: the previous token is in this round, or the last one of the sequence's state.
+__device__ __forceinline__ size_t pair_row(const PreNormArgs &a, int t) {
+    const int r = a.tok_req[t], sg = a.req_slot[r];
+    const bool at_start = t == a.req_first[r];
+    if (threadIdx.x == 0 && t + 1 == a.req_first[r + 1]) a.last_token[(size_t)((sg & 1) ^ 1) * a.last_gen_stride + (sg >> 1)] = a.tokens[t];
+    if (at_start && a.req_pos[r] == 0) return (size_t)a.pair_buckets;
+    const unsigned long long prev = at_start ? a.last_token[(size_t)(sg & 1) * a.last_gen_stride + (sg >> 1)] : a.tokens[t - 1];
+    return (size_t)((prev * (unsigned)a.pair_prev + (unsigned long long)a.tokens[t] * (unsigned)a.pair_cur) % (unsigned)a.pair_buckets);
+}
+
 // One block per token: the residual step of pre-norm layers.
 template <class T, int MAXV>
 __global__ void pre_norm_kernel(const PreNormArgs a) {
@@ -106,6 +116,9 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     const size_t row = (size_t)t * a.d_p;
     grid_dep_wait();
     const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;  // fed-back tokens are written by the kernel before the round's first one
+    const size_t e1 = a.pair_embd ? pair_row(a, t) * a.d_p : 0;
+    if (t == 0)
+        for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
     float4 x[MAXV], y0[MAXV], y1[MAXV];
     float s0 = 0.f, s1 = 0.f;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -117,10 +130,20 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
         if (a.x_in) x[j] = *reinterpret_cast<const float4 *>(a.x_in + row + 4 * i);
         if (a.y[0]) y0[j] = *reinterpret_cast<const float4 *>(a.y[0] + row + 4 * i);
         if (a.y[1]) y1[j] = *reinterpret_cast<const float4 *>(a.y[1] + row + 4 * i);
+        if (a.post_gain) {  // one sum
+            float4 &u = y0[j], &v = y1[j];
+            u = make_float4(u.x * a.y_scale[0] + v.x * a.y_scale[1], u.y * a.y_scale[0] + v.y * a.y_scale[1], u.z * a.y_scale[0] + v.z * a.y_scale[1],
+                            u.w * a.y_scale[0] + v.w * a.y_scale[1]);
+            v = zero;
+            for (int k = 0; k < a.top; ++k) {
+                const float4 e = *reinterpret_cast<const float4 *>(a.ye + (size_t)a.slot_of[t * a.top + k] * a.d_p + 4 * i);
+                u.x += e.x; u.y += e.y; u.z += e.z; u.w += e.w;
+            }
+        }
         s0 += dot4(y0[j]);
         s1 += dot4(y1[j]);
     }
-    if (a.y_gain) {
+    if (a.y_gain || a.post_gain) {
         const float2 s = block_sum2(s0, s1, part);
         s0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
         s1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
@@ -136,11 +159,18 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
             g1 = *reinterpret_cast<const float4 *>(a.y_gain + a.d_p + 4 * i);
             g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
             g1.x *= s1; g1.y *= s1; g1.z *= s1; g1.w *= s1;
+        } else if (a.post_gain) {
+            g0 = *reinterpret_cast<const float4 *>(a.post_gain + 4 * i);
+            g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
         }
         v.x += y0[j].x * g0.x + y1[j].x * g1.x; v.y += y0[j].y * g0.y + y1[j].y * g1.y;
         v.z += y0[j].z * g0.z + y1[j].z * g1.z; v.w += y0[j].w * g0.w + y1[j].w * g1.w;
         if (a.embd) {
             const float4 e = ld4_bf16(a.embd, e0 + 4 * i);
+            v.x += e.x * a.embd_scale; v.y += e.y * a.embd_scale; v.z += e.z * a.embd_scale; v.w += e.w * a.embd_scale;
+        }
+        if (a.pair_embd) {
+            const float4 e = ld4_bf16(a.pair_embd, e1 + 4 * i);
             v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
         }
         if (a.step) {

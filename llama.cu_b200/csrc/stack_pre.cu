@@ -1,7 +1,11 @@
-// Layers of pre-norm models: x += mixer(norm(x)), x += ff(norm(x)).  A mixer is softmax attention, a gated delta rule, or both
-// side by side on the same input, their outputs normed and added.  One projection serves both; rounds, pages, state slots, head
-// and sampling are those of every layered model.
+// Layers of pre-norm models: x += mixer(norm(x)), x += ff(norm(x)), or with norms on the outputs too.  A mixer is softmax
+// attention, a recurrent mixer (delta rule, state space duality, gated linear attention), or one of each side by side on the same
+// input, their outputs added.  One projection serves both; the feed-forward is one for all tokens or one of experts.  Rounds,
+// pages, state slots, head and sampling are those of every layered model.
+#include "moe.cuh"
 #include "stack_round.cuh"
+
+#include <cmath>
 
 namespace lcu {
 
@@ -29,32 +33,53 @@ struct PreNormRound {
         return rc;
     }
 
-    // x after a sublayer's outputs (none: the embedding), what comes ahead of layer `next`, and h, normed with `gain`
-    int residual(const float *y0, const float *y1, const float *y_gain, bool embed, const float *step, const float *gain) {
+    // what a sublayer left behind (see PreNormArgs); no output at all: the embedding
+    struct Outputs {
+        const float *y0 = nullptr, *y1 = nullptr, *y_gain = nullptr, *post_gain = nullptr;
+        float scale0 = 1.f, scale1 = 1.f;
+        int top = 0;  // rows of experts per token
+    };
+    // x after a sublayer's outputs, what comes ahead of the next one, and h, normed with `gain`
+    int residual(const Outputs &u, bool embed, const float *step, const float *gain, int n_zero = 0) {
         PreNormArgs a{};
         const lcu_model_desc &d = c->desc;
+        const bool start = !u.y0 && !u.top;
         a.n_tok = r.n_tok; a.d = d.d; a.d_p = S().d_p; a.eps = d.eps;
-        if (y0) {
+        if (!start) {
             a.x_in = S().x[cur];
             cur ^= 1;
         }
-        a.y[0] = y0; a.y[1] = y1; a.y_gain = y_gain;
-        if (embed) { a.embd = c->embd; a.tokens = reinterpret_cast<const uint32_t *>(D + r.L.tokens); }
+        a.y[0] = u.y0; a.y[1] = u.y1; a.y_gain = u.y_gain; a.post_gain = u.post_gain; a.y_scale[0] = u.scale0; a.y_scale[1] = u.scale1;
+        if (u.top) { a.top = u.top; a.ye = S().ye; a.slot_of = moe_int(2); }
+        if (embed || start) {
+            const lcu_layer_desc &l = S().layers[0].d;
+            a.embd = c->embd; a.tokens = reinterpret_cast<const uint32_t *>(D + r.L.tokens);
+            a.embd_scale = l.embed_scale ? l.embed_scale : 1.f;
+            if (l.pair_buckets) {
+                a.pair_embd = S().pair_embd; a.pair_buckets = l.pair_buckets; a.pair_prev = l.pair_prev; a.pair_cur = l.pair_cur;
+                a.last_token = S().last_token; a.last_gen_stride = S().n_slots;
+                a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req);
+                a.req_first = i32(o.req_first); a.req_pos = i32(o.req_pos); a.req_slot = i32(o.req_slot);
+            }
+        }
         a.step = step; a.x_out = S().x[cur]; a.gain = gain; a.h = gain ? S().h : nullptr;
+        a.zero = S().moe_count; a.n_zero = n_zero;
         return done(op_pre_norm(a, c->dt, s, L.pdl));
     }
     // ... ahead of layer `next` (past the last one: the head reads x itself)
-    int residual_into(int next, const float *y0, const float *y1, const float *y_gain) {
-        if (next >= c->desc.n_layers) return residual(y0, y1, y_gain, false, nullptr, nullptr);
+    int residual_into(int next, const Outputs &u) {
+        if (next >= c->desc.n_layers) return residual(u, false, nullptr, nullptr);
         const StackLayer &Y = S().layers[next];
-        return residual(y0, y1, y_gain, !y0 || Y.d.add_embed, Y.d.add_step ? S().w[next].step : nullptr, S().w[Y.src].norm1);
+        return residual(u, Y.d.add_embed, Y.d.add_step ? S().w[next].step : nullptr, S().w[Y.src].norm1);
     }
 
     GqaArgs gqa(const StackLayer &Y, const StackWeights &W) const {
         GqaArgs a{};
         a.lat = S().lat; a.stride = Y.in_rows(); a.n_tok = r.n_tok;
         a.heads = Y.d.heads; a.kv_heads = Y.d.kv_heads; a.dim = Y.d.dim; a.dim_p = Y.dim_p; a.v_dim = Y.d.v_dim; a.vdim_p = Y.vdim_p;
-        a.bias = W.bias; a.qk_norm = Y.d.qk_norm; a.eps = c->desc.eps; a.rot_dims = Y.d.rot_dims; a.rot = Y.rot; a.q = S().q;
+        a.bias = W.bias; a.own_kv = Y.own_kv(); a.qk_norm = Y.d.qk_norm; a.qk_gain = W.qk_gain; a.eps = c->desc.eps;
+        a.rot_dims = Y.d.rot_dims; a.rot_adjacent = Y.d.rot_adjacent; a.rot = Y.rot; a.q = S().q;
+        a.window = Y.d.window; a.sink = Y.d.sink; a.gate = Y.d.out_gate ? S().lat + Y.att_rows : nullptr;
         a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift;
         a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req); a.page_table = reinterpret_cast<const int32_t *>(D + r.L.page_table);
         a.pos = reinterpret_cast<const uint32_t *>(D + r.L.pos); a.pt_stride = c->pt_stride;
@@ -82,57 +107,153 @@ struct PreNormRound {
         return rc;
     }
 
-    DeltaArgs delta(const StackLayer &Y, const StackWeights &W) const {
-        DeltaArgs a{};
-        a.lat = S().lat + Y.att_rows; a.stride = Y.in_rows(); a.n_tok = r.n_tok; a.n_req = r.n_req;
+    void recurrent(DeltaArgs &a, const StackLayer &Y, const StackWeights &W) const {
+        a.lat = S().lat + Y.att_rows + Y.g_p; a.stride = Y.in_rows(); a.n_tok = r.n_tok; a.n_req = r.n_req;
         a.heads = Y.d.delta_heads; a.kv_heads = Y.d.delta_kv_heads; a.dk = Y.d.delta_dim; a.dk_p = Y.dk_p; a.dv = Y.d.delta_v_dim; a.dv_p = Y.dv_p;
-        a.heads_p = Y.dh_p; a.taps = Y.d.delta_conv; a.eps = c->desc.eps; a.conv = W.conv; a.decay = W.decay; a.norm = W.delta_norm;
+        a.heads_p = Y.dh_p; a.taps = Y.d.delta_conv; a.eps = c->desc.eps; a.conv = W.conv; a.conv_bias = W.conv_bias; a.decay = W.decay; a.norm = W.delta_norm;
         a.conv_state = S().conv_state + Y.conv_off * S().n_slots; a.conv_gen_stride = S().conv_gen; a.state = S().mat_state + Y.mat_off * S().n_slots;
         a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req);
         a.req_first = i32(o.req_first); a.req_pos = i32(o.req_pos); a.req_slot = i32(o.req_slot);
         a.split = c->dt != LCU_F32 && tuning().delta_tc;
         a.q = S().dq; a.k = S().dk; a.v = S().dv; a.coef = S().dcoef;
         a.blocks = reinterpret_cast<const int4 *>(B + o.dblk); a.n_blocks = r.sr.n_delta_blocks; a.o = S().att2; a.stride_o = Y.dhv_p;
+    }
+    ScanArgs scan(const StackLayer &Y, const StackWeights &W) const {
+        ScanArgs a{};
+        recurrent(a, Y, W);
+        a.blocks = reinterpret_cast<const int4 *>(B + o.sblk); a.n_blocks = r.sr.n_scan_blocks;
+        a.per_channel = Y.gla(); a.gate_map = W.gate_map; a.rank = Y.d.gate_rank; a.rank_p = Y.rank_p;
+        if (Y.gla()) {
+            a.inv_tau = 1.f / Y.d.gate_tau;
+            a.q_scale = 1.f / sqrtf((float)Y.d.delta_dim);
+            a.vin = a.lat + 2 * a.heads * a.dk_p; a.vin_stride = a.stride;
+        } else {
+            a.vin = a.v; a.vin_stride = a.heads * a.dv_p;
+        }
+        a.parts = Y.d.norm_parts; a.tail = S().dtail;
         return a;
+    }
+
+    // the recurrent mixer and, ahead of the attention itself, its preparation
+    int recurrent_and_prep(const StackLayer &Y, const StackWeights &W, const GqaArgs &g) {
+        const int dt = c->dt;
+        const GqaArgs *attn = Y.attention() ? &g : nullptr;
+        int rc = LCU_OK;
+        if (Y.delta()) {
+            DeltaArgs e{};
+            recurrent(e, Y, W);
+            if (r.decode_only) return done(delta_decode_launch(e, attn, dt, s, L.pdl));
+            if (attn) rc = done(gqa_prep_launch(g, dt, s, L.pdl));
+            if (!rc) rc = done(delta_prep_launch(e, s, L.pdl));
+            if (!rc) rc = done(delta_scan_launch(e, s, L.pdl));
+            return rc ? rc : done(delta_out_launch(e, dt, s, L.pdl));
+        }
+        if (!Y.recurrent() || !r.decode_only) rc = attn ? done(gqa_prep_launch(g, dt, s, L.pdl)) : LCU_OK;
+        if (rc || !Y.recurrent()) return rc;
+        const ScanArgs e = scan(Y, W);
+        if (r.decode_only) rc = done(scan_step_launch(e, attn, dt, s, L.pdl));
+        else if (dt == LCU_F32) rc = done(scan_step_launch(e, nullptr, dt, s, L.pdl));
+        else {
+            rc = done(scan_prep_launch(e, s, L.pdl));
+            if (!rc) rc = done(scan_launch(e, s, L.pdl));
+            if (!rc && Y.gla()) rc = done(delta_out_launch(e, dt, s, L.pdl));
+        }
+        return rc || !Y.ssd() ? rc : done(scan_out_launch(e, dt, s, L.pdl));
     }
 
     // h -> outputs of the layer's mixers in y and y2
     int mixers(const StackLayer &Y, const StackWeights &W) {
-        const int n = r.n_tok, dt = c->dt;
+        const int n = r.n_tok;
         int rc = L.linear(W.in, S().d_p, Y.in_rows(), S().h, n, S().lat, Y.in_rows(), EPI_STORE_F32);
         const GqaArgs g = gqa(Y, W);
-        const DeltaArgs e = delta(Y, W);
-        if (Y.delta() && r.decode_only) {
-            if (!rc) rc = done(delta_decode_launch(e, Y.attention() ? &g : nullptr, dt, s, L.pdl));
-        } else {
-            if (!rc && Y.attention()) rc = done(gqa_prep_launch(g, dt, s, L.pdl));
-            if (!rc && Y.delta()) rc = done(delta_prep_launch(e, s, L.pdl));
-            if (!rc && Y.delta()) rc = done(delta_scan_launch(e, s, L.pdl));
-            if (!rc && Y.delta()) rc = done(delta_out_launch(e, dt, s, L.pdl));
-        }
+        if (!rc) rc = recurrent_and_prep(Y, W, g);
         if (!rc && Y.attention()) rc = attention(g, Y);
         if (!rc && Y.attention()) rc = L.linear(W.att_out, Y.hv_p, S().d_p, S().att, n, S().y, S().d_p, EPI_STORE_F32);
-        if (!rc && Y.delta()) rc = L.linear(W.delta_out, Y.dhv_p, S().d_p, S().att2, n, Y.attention() ? S().y2 : S().y, S().d_p, EPI_STORE_F32);
+        if (!rc && Y.recurrent()) rc = L.linear(W.delta_out, Y.dhv_p, S().d_p, S().att2, n, Y.attention() ? S().y2 : S().y, S().d_p, EPI_STORE_F32);
         return rc;
+    }
+
+    // ---- feed-forward: h -> y (and rows of experts in ye)
+    int *moe_int(int i) const { return S().moe_ints + (size_t)i * S().max_rows; }
+    GluArgs glu(const StackLayer &Y, float limit) const { return GluArgs{limit, Y.d.glu_alpha, Y.d.glu_shift}; }
+    int dense_glu(const void *up, const void *down, int ff_p, const GluArgs &u) {
+        int rc = L.linear(up, S().d_p, 2 * ff_p, S().h, r.n_tok, S().act, ff_p, EPI_GLU, nullptr, PRO_NONE, nullptr, u);
+        return rc ? rc : L.linear(down, ff_p, S().d_p, S().act, r.n_tok, S().y, S().d_p, EPI_STORE_F32);
+    }
+    bool small_experts() const { return c->dt != LCU_F32 && r.n_tok <= MOE_SMALL_ROUND; }
+    int experts(const StackLayer &Y, const StackWeights &W) {
+        const int n = r.n_tok, d_p = S().d_p, rows = n * Y.d.top;
+        const GluArgs u = glu(Y, Y.d.glu_limit), us = glu(Y, Y.d.shared_limit);
+        int rc = L.linear(W.router, d_p, Y.e_p, S().h, n, S().router, Y.e_p, EPI_STORE_F32);
+        MoeRoute m{};
+        m.logits = S().router; m.n_tok = n; m.experts = Y.d.experts; m.experts_p = Y.e_p; m.top = Y.d.top;
+        m.expert = moe_int(0); m.place = moe_int(1); m.slot_of = moe_int(2); m.slot_tok = moe_int(3);
+        m.weight = S().moe_w; m.slot_w = S().moe_slot_w; m.count = S().moe_count; m.tiles = S().moe_tiles;
+        m.h = S().h; m.xg = S().xg; m.d_p = d_p;
+        if (small_experts()) {
+            m.max_tiles = rows < Y.d.experts ? rows : Y.d.experts; m.tile_rows = n;
+            if (!rc) rc = done(moe_plan_launch(m, s, L.pdl));
+            MoeProduct p{};
+            p.tiles = m.tiles; p.max_tiles = m.max_tiles; p.n_tok = n; p.shared = Y.d.shared_ff > 0; p.slot_w = m.slot_w; p.slot_tok = m.slot_tok;
+            p.up = 1; p.w = W.up; p.ws = W.shared_up; p.out = 2 * Y.ff_p; p.in = d_p; p.outs = 2 * Y.sff_p; p.ins = d_p;
+            p.x = p.xs = S().h; p.y = S().act_e; p.ys = S().act; p.glu = u; p.glus = us;
+            if (!rc) rc = done(moe_product_launch(p, s, L.pdl));
+            p.up = 0; p.w = W.down; p.ws = W.shared_down; p.out = p.outs = d_p; p.in = Y.ff_p; p.ins = Y.sff_p;
+            p.x = S().act_e; p.xs = S().act; p.y = S().ye; p.ys = S().y;
+            return rc ? rc : done(moe_product_launch(p, s, L.pdl));
+        }
+        // tiles as wide as an expert's share of the round
+        const int share = rows / Y.d.experts;
+        m.tile_rows = c->dt == LCU_F32 || share <= 64 ? 64 : (share <= 128 ? 128 : 256);
+        m.max_tiles = moe_max_tiles(rows, Y.d.experts, m.tile_rows);
+        if (!rc) rc = done(moe_route_launch(m, s, L.pdl));
+        if (!rc) rc = done(moe_gather_launch(m, c->dt, s, L.pdl));
+        auto grouped = [&](const void *w, int in, int out, const void *x, void *y, int stride_y, int epilogue) -> int {
+            if (c->dt == LCU_F32) {
+                LinearF32Args a{};
+                a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w; a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
+                a.n = rows; a.in = in; a.out = out; a.heads = 1; a.epilogue = epilogue; a.glu = u;
+                a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.row_scale = m.slot_w;
+                return done(linear_f32_launch(a, s));
+            }
+            GemvArgs a{};
+            a.w = w; a.x = x; a.stride_x = in; a.n_tok = rows; a.in = in; a.out = out; a.epilogue = epilogue; a.y = y; a.stride_y = stride_y; a.glu = u;
+            a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.tile_rows = m.tile_rows; a.groups = Y.d.experts; a.row_scale = m.slot_w;
+            return done(gemm_tc_launch(a, c->dt, s, L.pdl));
+        };
+        if (!rc) rc = grouped(W.up, d_p, 2 * Y.ff_p, S().xg, S().act_e, Y.ff_p, EPI_GLU);
+        if (!rc) rc = grouped(W.down, Y.ff_p, d_p, S().act_e, S().ye, d_p, EPI_STORE_F32);
+        if (!rc && Y.d.shared_ff) rc = dense_glu(W.shared_up, W.shared_down, Y.sff_p, us);
+        return rc;
+    }
+    int feed_forward(const StackLayer &Y, const StackWeights &W) {
+        if (Y.d.experts) return experts(Y, W);
+        if (Y.glu()) return dense_glu(W.up, W.down, Y.ff_p, glu(Y, Y.d.glu_limit));
+        int rc = L.linear(W.up, S().d_p, Y.ff_p, S().h, r.n_tok, S().act, Y.ff_p, EPI_RELU2);
+        return rc ? rc : L.linear(W.down, Y.ff_p, S().d_p, S().act, r.n_tok, S().y, S().d_p, EPI_STORE_F32);
     }
 
     int run() {
         gemm_tc_set_scratch(c->sk_ws, c->sk_ws_bytes, c->sk_tickets, 4096, c->dev_status);
-        int rc = residual_into(0, nullptr, nullptr, nullptr);
+        int rc = residual_into(0, Outputs{});
         for (int l = 0; l < c->desc.n_layers && !rc; ++l) {
             const StackLayer &Y = S().layers[l];
             const StackWeights &W = S().w[Y.src];
-            const bool both = Y.attention() && Y.delta();
+            const bool both = Y.attention() && Y.recurrent();
             rc = mixers(Y, W);
             if (rc) break;
-            if (!Y.d.ff) {
-                rc = residual_into(l + 1, S().y, both ? S().y2 : nullptr, both ? W.branch_norm : nullptr);
+            Outputs u;
+            u.y0 = S().y; u.y1 = both ? S().y2 : nullptr; u.y_gain = both ? W.branch_norm : nullptr; u.post_gain = W.post1;
+            if (both && Y.d.post_norm) { u.scale0 = Y.d.out_scale; u.scale1 = Y.d.out_scale2; }
+            if (!Y.has_ff()) {
+                rc = residual_into(l + 1, u);
                 continue;
             }
-            rc = residual(S().y, both ? S().y2 : nullptr, both ? W.branch_norm : nullptr, false, nullptr, W.norm2);
-            if (!rc) rc = L.linear(W.up, S().d_p, Y.ff_p, S().h, r.n_tok, S().act, Y.ff_p, EPI_RELU2);
-            if (!rc) rc = L.linear(W.down, Y.ff_p, S().d_p, S().act, r.n_tok, S().y, S().d_p, EPI_STORE_F32);
-            if (!rc) rc = residual_into(l + 1, S().y, nullptr, nullptr);
+            rc = residual(u, false, nullptr, W.norm2, Y.d.experts && !small_experts() ? Y.d.experts : 0);
+            if (!rc) rc = feed_forward(Y, W);
+            u = Outputs{};
+            u.y0 = Y.d.experts && !Y.d.shared_ff ? nullptr : S().y; u.top = Y.d.experts ? Y.d.top : 0; u.post_gain = W.post2;
+            if (!rc) rc = residual_into(l + 1, u);
         }
         c->x = S().x[cur];
         return rc;

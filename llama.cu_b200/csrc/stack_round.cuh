@@ -10,7 +10,7 @@ inline size_t act_bytes(const lcu_ctx *c) { return c->dt == LCU_F32 ? 4 : 2; }
 
 // offsets inside the stack section of the round descriptor
 struct StackDesc {
-    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, sreq, lreq, dblk, total;
+    size_t req_first, req_pos, req_slot, abs_first, abs_id, abs_tok, xreq, xgroups, sreq, lreq, dblk, sblk, total;
 };
 constexpr int EXPAND_GROUP = 64;  // query tokens per group of the expanded attention
 inline StackDesc stack_desc(int n_tok, int n_req) {
@@ -28,6 +28,7 @@ inline StackDesc stack_desc(int n_tok, int n_req) {
     d.sreq = take((size_t)n_req * 16);
     d.lreq = take((size_t)n_req * 16);
     d.dblk = take((size_t)(n_tok / DELTA_BLOCK + n_req) * 16);
+    d.sblk = take((size_t)(n_tok / SCAN_BLOCK + n_req) * 16);
     d.total = o;
     return d;
 }
@@ -41,14 +42,14 @@ struct Launcher {
 
     // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
     int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr,
-               int prologue = PRO_NONE, const GemvArgs *pro = nullptr) {
+               int prologue = PRO_NONE, const GemvArgs *pro = nullptr, const GluArgs &glu = GluArgs{}) {
         if (c->dt == LCU_F32) {
             LinearF32Args a{};
             a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w;
             a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
             a.n = n; a.in = in; a.out = out; a.heads = 1;
             a.epilogue = epilogue == EPI_STORE ? EPI_STORE_F32 : epilogue;
-            a.act_pq = act_pq;
+            a.act_pq = act_pq; a.glu = glu;
             ++*count;
             return linear_f32_launch(a, s);
         }
@@ -63,7 +64,7 @@ struct Launcher {
             a.w = w;
             a.x = reinterpret_cast<const unsigned char *>(x) + (size_t)t0 * in * 2;
             a.stride_x = in; a.n_tok = nt; a.in = in; a.out = out;
-            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq;
+            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq; a.glu = glu;
             a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
             a.stride_y = stride_y;
             if (pro) {  // one launch (at most two tokens): the prologue's rows, and the tokens' places in the cache

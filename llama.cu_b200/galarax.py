@@ -40,7 +40,7 @@ def unroll(layers, loop):
     return tuple(out + list(layers[b:]))
 
 
-def read_config(raw):
+def read_config(raw, shapes=None):
     """LayeredConfig from the parsed config.json."""
     layers = unroll([read_layer(i, e) for i, e in enumerate(raw["layers"])], raw.get("loop"))
     return LayeredConfig("galarax", raw["width"], raw["vocab"], layers, raw["norm"]["eps"], arch="Galarax")

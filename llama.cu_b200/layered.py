@@ -11,9 +11,10 @@ from dataclasses import dataclass
 
 import numpy as np
 
-from . import (ACT_RELU2, ACT_XIELU, BF16, F32, MIX_ATTENTION, MIX_DELTA, MIX_LATENT, W_ATT_OUT, W_BRANCH_NORM, W_CONV, W_DELTA_DECAY,
-               W_DELTA_NORM, W_DELTA_OUT, W_EMBD, W_FF_DOWN, W_KV_NORM, W_LAT_IN, W_LAT_OUT, W_LM_HEAD, W_MIX_BIAS, W_MIX_IN, W_NORM1,
-               W_NORM2, W_OUT_NORM, W_Q_NORM, W_SCALARS, W_SHIFT, W_STEP, W_UKT, W_UKV, W_UP, W_UQ, LayerDesc, ModelDesc)
+from . import (ACT_GLU, ACT_RELU2, ACT_XIELU, BF16, F32, MIX_ATTENTION, MIX_DELTA, MIX_GLA, MIX_LATENT, MIX_SSD, W_ATT_OUT, W_BRANCH_NORM,
+               W_CONV, W_CONV_BIAS, W_DELTA_DECAY, W_DELTA_NORM, W_DELTA_OUT, W_EMBD, W_FF_DOWN, W_GATE_MAP, W_KV_NORM, W_LAT_IN, W_LAT_OUT,
+               W_LM_HEAD, W_MIX_BIAS, W_MIX_IN, W_NORM1, W_NORM2, W_OUT_NORM, W_PAIR_EMBD, W_POST1, W_POST2, W_Q_NORM, W_QK_GAIN, W_ROUTER,
+               W_SCALARS, W_SHARED_DOWN, W_SHARED_UP, W_SHIFT, W_STEP, W_UKT, W_UKV, W_UP, W_UQ, LayerDesc, ModelDesc)
 
 
 def pad_to(v, m):
@@ -55,11 +56,13 @@ class Rotary:
     original: float = 0.0
     fast: float = 0.0
     slow: float = 0.0
+    adjacent: bool = False  # pairs (2i, 2i + 1) instead of (i, i + dims / 2)
 
 
 @dataclass(frozen=True)
 class AttentionMixer:
-    """Softmax attention with grouped heads, rotary positions, optionally biases and normalised queries and keys."""
+    """Softmax attention with grouped heads, optionally rotary positions, biases, normalised queries and keys (qk_norm: see
+    lcu_layer_desc), a sliding window, a sink in the softmax, a gate per head, another layer's keys and values."""
     heads: int
     kv_heads: int
     dim: int
@@ -67,23 +70,33 @@ class AttentionMixer:
     scale: float
     rot: Rotary
     bias: bool = True
-    qk_norm: bool = True
+    qk_norm: int = 1
+    window: int = 0
+    sink: bool = False
+    out_gate: bool = False
+    kv_from: int = -1  # the layer whose keys and values are used, -1: its own
 
     def describe(self, o):
         o.mixer |= MIX_ATTENTION
         o.heads, o.kv_heads, o.dim, o.v_dim, o.scale = self.heads, self.kv_heads, self.dim, self.v_dim, self.scale
         o.bias, o.qk_norm, r = int(self.bias), int(self.qk_norm), self.rot
+        o.window, o.sink, o.out_gate, o.kv_from = self.window, int(self.sink), int(self.out_gate), self.kv_from + 1
         if r is not None:
             o.rot_dims, o.rot_base, o.rot_factor, o.rot_original, o.rot_fast, o.rot_slow = r.dims, r.base, r.factor, r.original, r.fast, r.slow
+            o.rot_adjacent = int(r.adjacent)
+
+    @property
+    def own_kv_heads(self):
+        return self.kv_heads if self.kv_from < 0 else 0
 
     def cached_per_token(self):
-        return self.kv_heads * (pad_to(self.dim, 16) + pad_to(self.v_dim, 16))
+        return self.own_kv_heads * (pad_to(self.dim, 16) + pad_to(self.v_dim, 16))
 
     def state_bytes(self):
         return 0
 
     def weights(self, d):
-        return d * (self.heads + self.kv_heads) * (self.dim + self.v_dim)
+        return d * ((self.heads + self.own_kv_heads) * (self.dim + self.v_dim) + (self.heads if self.out_gate else 0))
 
 
 @dataclass(frozen=True)
@@ -109,15 +122,78 @@ class DeltaMixer:
         return d * (2 * self.kv_heads * self.dim + 3 * self.heads * self.v_dim + 2 * self.heads)
 
 
+def describe_recurrent(m, o, kv_heads):
+    o.delta_heads, o.delta_kv_heads, o.delta_dim, o.delta_v_dim = m.heads, kv_heads, m.dim, m.v_dim
+
+
+def recurrent_state_bytes(m):
+    return 4 * m.heads * pad_to(m.v_dim, 16) * pad_to(m.dim, 32)
+
+
+@dataclass(frozen=True)
+class SsdMixer:
+    """State space duality: one decay per head, keys and queries (`dim` numbers) per group of heads, short convolutions with biases,
+    the gated output normed in equal parts."""
+    heads: int
+    groups: int
+    dim: int
+    v_dim: int
+    conv: int
+    norm_parts: int
+
+    def describe(self, o):
+        o.mixer |= MIX_SSD
+        describe_recurrent(self, o, self.groups)
+        o.delta_conv, o.norm_parts = self.conv, self.norm_parts
+
+    def cached_per_token(self):
+        return 0
+
+    def state_bytes(self):
+        return recurrent_state_bytes(self)
+
+    def weights(self, d):
+        return d * (2 * self.groups * self.dim + 3 * self.heads * self.v_dim + self.heads)
+
+
+@dataclass(frozen=True)
+class GlaMixer:
+    """Gated linear attention: one decay per head and key channel, sigmoid(z)^(1 / tau) with z of low rank, the output normed and gated
+    per head."""
+    heads: int
+    dim: int
+    v_dim: int
+    tau: float
+    rank: int
+
+    def describe(self, o):
+        o.mixer |= MIX_GLA
+        describe_recurrent(self, o, self.heads)
+        o.gate_tau, o.gate_rank = self.tau, self.rank
+
+    def cached_per_token(self):
+        return 0
+
+    def state_bytes(self):
+        return recurrent_state_bytes(self)
+
+    def weights(self, d):
+        return d * (2 * self.heads * self.dim + 3 * self.heads * self.v_dim + self.rank)
+
+
 @dataclass(frozen=True)
 class ParallelMixer:
-    """Two mixers on the same input, their outputs normed over the width and averaged."""
+    """Softmax attention and a recurrent mixer on the same input, their outputs added: normed over the width with a gain each (scales
+    None), or with a factor each."""
     left: AttentionMixer
-    right: DeltaMixer
+    right: object
+    scales: tuple = None
 
     def describe(self, o):
         self.left.describe(o)
         self.right.describe(o)
+        if self.scales:
+            o.out_scale, o.out_scale2 = self.scales
 
     def cached_per_token(self):
         return self.left.cached_per_token() + self.right.cached_per_token()
@@ -130,10 +206,41 @@ class ParallelMixer:
 
 
 @dataclass(frozen=True)
+class GluFf:
+    """Gated feed-forward: g = min(W_gate x, limit), u = clamp(W_up x, +-limit), W_down (g sigmoid(alpha g) (u + shift)).  With
+    `experts` > 0 every token uses `top` of that many, their inputs scaled by the sigmoids of their router logits, and the shared
+    one (width `shared`, 0: none)."""
+    ff: int
+    limit: float
+    alpha: float = 1.0
+    shift: float = 0.0
+    experts: int = 0
+    top: int = 0
+    shared: int = 0
+    shared_limit: float = 0.0
+
+    def describe(self, o):
+        o.ff, o.ff_act, o.experts, o.top, o.shared_ff = self.ff, ACT_GLU, self.experts, self.top, self.shared
+        o.glu_limit, o.shared_limit, o.glu_alpha, o.glu_shift = self.limit, self.shared_limit, self.alpha, self.shift
+
+    def weights(self, d):
+        """Weights one token meets."""
+        return d * (3 * (self.ff * (self.top or 1) + self.shared) + self.experts)
+
+
+@dataclass(frozen=True)
+class PairEmbedding:
+    """Row (previous token * prev + token * cur) mod buckets is added to a token's embedding, row `buckets` to the first one's."""
+    buckets: int
+    prev: int
+    cur: int
+
+
+@dataclass(frozen=True)
 class LayerConfig:
     """One layer as it runs; a layer that runs several times is listed several times (`weights_of`)."""
     mixer: object
-    ff: int = 0  # 0: no feed-forward
+    ff: object = 0  # width, 0: no feed-forward; or a GluFf
     token_shift: bool = True
     weights_of: int = -1
     act: int = ACT_XIELU
@@ -141,6 +248,10 @@ class LayerConfig:
     add_embed: bool = False  # the embedding output is added to the residual stream ahead of the layer
     step: int = -1           # row of the table of vectors added ahead of the layer, -1: none
     file_layer: int = -1     # the layer's number in the model file, -1: its place in the list
+    post_norm: bool = False  # pre-norm layers: norms on the sublayers' outputs too
+
+    def ff_weights(self, d):
+        return self.ff.weights(d) if isinstance(self.ff, GluFf) else 2 * self.ff * d
 
 
 @dataclass(frozen=True)
@@ -153,6 +264,8 @@ class LayeredConfig:
     act_dtype: int = BF16  # or F32: everything in 32-bit arithmetic
     nctx: int = 2048
     arch: str = "Zefedra"  # key of `architectures()`
+    embed_scale: float = 1.0
+    pairs: PairEmbedding = None
 
     @property
     def family(self):
@@ -177,8 +290,16 @@ class LayeredConfig:
         out = (LayerDesc * self.n_layers)()
         for o, l in zip(out, self.layers):
             l.mixer.describe(o)
-            o.token_shift, o.ff, o.ff_act, o.weights_of = int(l.token_shift), l.ff, l.act, l.weights_of
-            o.pre_norm, o.add_embed, o.add_step = int(l.pre_norm), int(l.add_embed), int(l.step >= 0)
+            o.token_shift, o.weights_of = int(l.token_shift), l.weights_of
+            if isinstance(l.ff, GluFf):
+                l.ff.describe(o)
+            else:
+                o.ff, o.ff_act = l.ff, l.act
+            o.pre_norm, o.post_norm, o.add_embed, o.add_step = int(l.pre_norm), int(l.post_norm), int(l.add_embed), int(l.step >= 0)
+        out[0].embed_scale = self.embed_scale
+        if self.pairs:
+            b = self.pairs.buckets
+            out[0].pair_buckets, out[0].pair_prev, out[0].pair_cur = b, self.pairs.prev % b, self.pairs.cur % b
         return out
 
     def kv_bytes_per_token(self, tp=1):
@@ -190,7 +311,7 @@ class LayeredConfig:
         return sum(l.mixer.state_bytes() for l in self.layers)
 
     def weight_bytes_per_step(self, tp=1):
-        return self.vocab * self.d * 2.0 + sum(2.0 * (l.mixer.weights(self.d) + 2 * l.ff * self.d) for l in self.layers)
+        return self.vocab * self.d * 2.0 + sum(2.0 * (l.mixer.weights(self.d) + l.ff_weights(self.d)) for l in self.layers)
 
 
 def _pad(t, *shape):
@@ -230,21 +351,27 @@ def _out_columns(o, d, heads, size, to):
     return _pad(_pad(o.reshape(d, heads, size), d, heads, to).reshape(d, heads * to), wp, pad_to(heads * to, 64))
 
 
-def attention_rows(m, d, q, k, v):
-    """Rows of the fused input projection of an AttentionMixer."""
+def attention_rows(m, d, q, k=None, v=None, g=None):
+    """Rows of the fused input projection of an AttentionMixer (k and v: unless they are another layer's)."""
     wp, dp, vp = pad_to(d, 64), pad_to(m.dim, 16), pad_to(m.v_dim, 16)
-    return [_pad(_pad_heads(w, n, a, b), n * b, wp) for w, n, a, b in
-            ((q, m.heads, m.dim, dp), (k, m.kv_heads, m.dim, dp), (v, m.kv_heads, m.v_dim, vp))]
+    rows = [_pad(_pad_heads(w, n, a, b), n * b, wp) for w, n, a, b in
+            ((q, m.heads, m.dim, dp), (k, m.kv_heads, m.dim, dp), (v, m.kv_heads, m.v_dim, vp)) if w is not None]
+    return rows + ([_pad(g, pad_to(m.heads, 8), wp)] if m.out_gate else [])
 
 
-def pack_attention(m, d, o, bias=None):
-    """[(kind, tensor)] of an AttentionMixer besides its input projection; bias: (q, k, v)."""
+def pack_attention(m, d, o, bias=None, gains=None):
+    """[(kind, tensor)] of an AttentionMixer besides its input projection; bias: (q, k, v), or (q,) without own keys; gains: the
+    weights of the norms of q and k, one head's or all heads' ((q,) without own keys)."""
     import torch
     dp, vp = pad_to(m.dim, 16), pad_to(m.v_dim, 16)
     out = [(W_ATT_OUT, _out_columns(o, d, m.heads, m.v_dim, vp))]
     if m.bias:
         out.append((W_MIX_BIAS, torch.cat([_pad_heads(b.float(), n, x, y) for b, n, x, y in
                                            zip(bias, (m.heads, m.kv_heads, m.kv_heads), (m.dim, m.dim, m.v_dim), (dp, dp, vp))])))
+    if m.qk_norm == 2:
+        out.append((W_QK_GAIN, torch.cat([_pad(g.float(), dp) for g in gains])))
+    if m.qk_norm == 3:
+        out.append((W_QK_GAIN, torch.cat([_pad_heads(g.float(), n, m.dim, dp) for g, n in zip(gains, (m.heads, m.kv_heads))])))
     return out
 
 
@@ -264,6 +391,73 @@ def pack_delta(m, d, conv_q, conv_k, conv_v, a_log, dt_bias, norm, o):
                       ((conv_q, m.kv_heads, m.dim, dp), (conv_k, m.kv_heads, m.dim, dp), (conv_v, m.heads, m.v_dim, vp))])
     return [(W_CONV, conv.T.contiguous()), (W_DELTA_DECAY, torch.stack([_pad(a_log.float(), hp), _pad(dt_bias.float(), hp)])),
             (W_DELTA_NORM, _pad(norm.float(), vp)), (W_DELTA_OUT, _out_columns(o, d, m.heads, m.v_dim, vp))]
+
+
+def ssd_rows(m, d, w):
+    """Rows of the fused input projection of an SsdMixer; w: rows z | x | B | C | dt."""
+    import torch
+    wp, dp, vp, hp, inner, gn = pad_to(d, 64), pad_to(m.dim, 32), pad_to(m.v_dim, 16), pad_to(m.heads, 8), m.heads * m.v_dim, m.groups * m.dim
+    z, x, b, c, dt = torch.split(w, [inner, inner, gn, gn, m.heads])
+    return [_pad(_pad_heads(t, n, p, q), n * q, wp) for t, n, p, q in
+            ((c, m.groups, m.dim, dp), (b, m.groups, m.dim, dp), (x, m.heads, m.v_dim, vp), (z, m.heads, m.v_dim, vp))] + [_pad(dt, hp, wp)]
+
+
+def pack_ssd(m, d, conv, conv_bias, a_log, dt_bias, skip, norm, o):
+    """[(kind, tensor)] of an SsdMixer besides its input projection; conv [x | B | C, taps]."""
+    import torch
+    dp, vp, hp, inner, gn = pad_to(m.dim, 32), pad_to(m.v_dim, 16), pad_to(m.heads, 8), m.heads * m.v_dim, m.groups * m.dim
+
+    def channels(t):
+        x, b, c = torch.split(t.float(), [inner, gn, gn])
+        return torch.cat([_pad_heads(c, m.groups, m.dim, dp), _pad_heads(b, m.groups, m.dim, dp), _pad_heads(x, m.heads, m.v_dim, vp)])
+    return [(W_CONV, channels(conv).T.contiguous()), (W_CONV_BIAS, channels(conv_bias)),
+            (W_DELTA_DECAY, torch.stack([_pad(t.float(), hp) for t in (a_log, dt_bias, skip)])),
+            (W_DELTA_NORM, _pad_heads(norm.float(), m.heads, m.v_dim, vp)), (W_DELTA_OUT, _out_columns(o, d, m.heads, m.v_dim, vp))]
+
+
+def gla_rows(m, d, q, k, v, g, a1):
+    """Rows of the fused input projection of a GlaMixer."""
+    wp, dp, vp = pad_to(d, 64), pad_to(m.dim, 32), pad_to(m.v_dim, 16)
+    return [_pad(_pad_heads(w, m.heads, x, y), m.heads * y, wp) for w, x, y in ((q, m.dim, dp), (k, m.dim, dp), (v, m.v_dim, vp), (g, m.v_dim, vp))] + [
+            _pad(a1, pad_to(m.rank, 8), wp)]
+
+
+def pack_gla(m, d, a2, a2_bias, norm, o):
+    """[(kind, tensor)] of a GlaMixer besides its input projection."""
+    import torch
+    dp, vp = pad_to(m.dim, 32), pad_to(m.v_dim, 16)
+    gate = torch.cat([_pad_heads(a2.float(), m.heads, m.dim, dp).T, _pad_heads(a2_bias.float(), m.heads, m.dim, dp)[None]])
+    return [(W_GATE_MAP, gate.contiguous()), (W_DELTA_NORM, _pad(norm.float(), vp)), (W_DELTA_OUT, _out_columns(o, d, m.heads, m.v_dim, vp))]
+
+
+def glu_rows(gate, up, d, ff):
+    """Gate and up rows in turn."""
+    import torch
+    fp, wp = pad_to(ff, 64), pad_to(d, 64)
+    return torch.stack([_pad(gate, fp, wp), _pad(up, fp, wp)], 1).reshape(2 * fp, wp)
+
+
+def pack_experts(f, d, router, experts, shared=None):
+    """[(kind, tensor)] of a GluFf of experts; experts: an iterable of (gate, up, down), shared: one of them or None."""
+    import torch
+    wp, fp = pad_to(d, 64), pad_to(f.ff, 64)
+    ups, downs = torch.empty(f.experts, 2 * fp, wp, dtype=router.dtype, device=router.device), torch.empty(f.experts, wp, fp, dtype=router.dtype, device=router.device)
+    for i, (gate, up, down) in enumerate(experts):
+        ups[i], downs[i] = glu_rows(gate, up, d, f.ff), _pad(down, wp, fp)
+    out = [(W_ROUTER, _pad(router, pad_to(f.experts, 8), wp)), (W_UP, ups), (W_FF_DOWN, downs)]
+    if f.shared:
+        out += [(W_SHARED_UP, glu_rows(*shared[:2], d, f.shared)), (W_SHARED_DOWN, _pad(shared[2], wp, pad_to(f.shared, 64)))]
+    return out
+
+
+def pack_glu(f, d, gate, up, down):
+    """[(kind, tensor)] of a GluFf without experts."""
+    return [(W_UP, glu_rows(gate, up, d, f.ff)), (W_FF_DOWN, _pad(down, pad_to(d, 64), pad_to(f.ff, 64)))]
+
+
+def pack_norms(d, norm1, post1, norm2=None, post2=None):
+    """[(kind, tensor)] of the gains (f32) of a layer with norms ahead of its sublayers and on their outputs."""
+    return [(k, _pad(g.float(), pad_to(d, 64))) for k, g in ((W_NORM1, norm1), (W_POST1, post1), (W_NORM2, norm2), (W_POST2, post2)) if g is not None]
 
 
 def pack_common(d, embed, final_gain, head):
@@ -325,6 +519,9 @@ def read_safetensors(path):
 class Tensors(dict):
     """The tensors of a model file; reads are checked against the configuration."""
 
+    def shapes(self):
+        return {k: tuple(v.shape) for k, v in self.items()}
+
     def take(self, name, *shape):
         if name not in self:
             raise ValueError(f"tensor {name} is missing")
@@ -336,9 +533,10 @@ class Tensors(dict):
 
 
 def architectures():
-    """config.json's "architecture" -> module with read_config(dict) and pack(cfg, Tensors)."""
-    from . import galarax, zefedra
-    return {"Galarax": galarax, "Zefedra": zefedra}
+    """config.json's "architecture" -> module with read_config(dict, shapes) and pack(cfg, Tensors); shapes: {name: shape} of the
+    model file, for sizes that the configuration does not name."""
+    from . import galarax, mupuvik, zefedra
+    return {"Galarax": galarax, "Mupuvik": mupuvik, "Zefedra": zefedra}
 
 
 def load_pretrained(path, act_dtype=BF16, device=0, nctx=None, kv_tokens=None, page_tokens=0, max_tokens=0, max_seqs=0):
@@ -352,10 +550,11 @@ def load_pretrained(path, act_dtype=BF16, device=0, nctx=None, kv_tokens=None, p
     known = architectures()
     if arch not in known:
         raise ValueError(f"{path}: architecture {arch!r} is not one of {sorted(known)}")
-    cfg = replace(known[arch].read_config(raw), act_dtype=act_dtype)
+    tensors = Tensors(read_safetensors(os.path.join(path, "model.safetensors")))
+    cfg = replace(known[arch].read_config(raw, tensors.shapes()), act_dtype=act_dtype)
     if nctx:
         cfg = replace(cfg, nctx=nctx)
-    weights = known[arch].pack(cfg, Tensors(read_safetensors(os.path.join(path, "model.safetensors"))))
+    weights = known[arch].pack(cfg, tensors)
     tokens = kv_tokens or cfg.nctx
     pt = page_tokens or 64
     ctx = load_model(cfg, weights, device=device, kv_bytes=(tokens + pt - 1) // pt * pt * cfg.kv_bytes_per_token(), page_tokens=page_tokens,

@@ -11,7 +11,7 @@ import numpy as np
 
 from . import (BF16, F16, F32, LINEAR_KINDS, Q8_0, W_ATTN_NORM, W_DOWN, W_EMBD, W_FFN_NORM, W_GATE_UP, W_LM_HEAD,
                W_O, W_OUT_NORM, W_QKV, Context, ModelDesc, check, load_library, stream_ptr)
-from . import galarax, zefedra
+from . import galarax, mupuvik, zefedra
 from .layered import LayeredConfig
 
 

@@ -6,7 +6,7 @@ from .layered import LatentMixer, LayerConfig, LayeredConfig, pack_block, pack_c
 MIXERS = {"latent_attention": False, "latent_attention_2": True}  # -> per-head output gate
 
 
-def read_config(raw):
+def read_config(raw, shapes=None):
     """LayeredConfig from the parsed config.json."""
     layers = []
     for i, e in enumerate(raw["layers"]):
