@@ -39,6 +39,8 @@ WORKLOADS = {
     "zefedra8b-bf16-b32": ("zefedra8b", 32, (128, 1024)),
     "galarax8b-bf16-b1": ("galarax8b", 1, (128, 128)),
     "galarax8b-bf16-b32": ("galarax8b", 32, (128, 1024)),
+    "mupuvik8b-bf16-b1": ("mupuvik8b", 1, (128, 128)),
+    "mupuvik8b-bf16-b32": ("mupuvik8b", 32, (128, 1024)),
     "tiny-f16-b1": ("tiny", 1, (16, 16)),
 }
 DEFAULT_WORKLOAD = "llama8b-f16-b1"
@@ -477,7 +479,8 @@ def run_decode(L, env, cfg, batch, prompt_range, steps, warmup, want_e2e=True, w
 
 # --family-bench: sizes at which the layered families run beside the LLaMA shape of equal width and feed-forward, cut to
 # `layers` layers and a vocabulary of 32000 (name, configs, layers)
-FAMILY_SIZES = [("8b", ("galarax8b", "zefedra8b", "llama8b"), 8), ("1b", ("galarax1b", "zefedra1b", "llama1b"), 8)]
+FAMILY_SIZES = [("8b", ("mupuvik8b", "galarax8b", "zefedra8b", "llama8b"), 8),
+                ("1b", ("mupuvik1b", "galarax1b", "zefedra1b", "llama1b"), 8)]
 FAMILY_PREFILL = (2048, 8192)                            # prompt lengths
 FAMILY_DECODE = ((1, 1024), (32, 1024), (32, 4096), (4, 8192))  # (sequences, context)
 
@@ -562,8 +565,14 @@ def family_bench(L, env, only=None, models=None, profile_kernels=False):
                     ctx.step([(s, pos[0], 1) for s in seqs], np.full(batch, 7, np.uint32), out, stream=stream)
                     pos[0] += 1
 
+                    # fed-back tokens of a model with random weights are alike, and so would be the experts they choose
+                    experts = any(getattr(l.ff, "experts", 0) for l in getattr(cfg, "layers", ()))
+
                     def one():
-                        ctx.step([(s, pos[0], 1) for s in seqs], np.zeros(batch, np.uint32), out, fast_map=fm, stream=stream)
+                        if experts:
+                            ctx.step([(s, pos[0], 1) for s in seqs], rng.integers(3, cfg.vocab, batch).astype(np.uint32), out, stream=stream)
+                        else:
+                            ctx.step([(s, pos[0], 1) for s in seqs], np.zeros(batch, np.uint32), out, fast_map=fm, stream=stream)
                         pos[0] += 1
                     ms, clocks, table = timed(one, 32, 8)
                     gbs = ctx.last_step_bytes / ms / 1e6

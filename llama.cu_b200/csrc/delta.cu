@@ -529,7 +529,7 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(const DeltaArgs a, co
     if (blockIdx.x >= a.heads) {
         grid_dep_wait();
         const int item0 = ((int)blockIdx.x - a.heads) * 8;
-        if (has_attn) gqa_prep_block<T>(attn, t, item0, item0 + 8);
+        if (has_attn) gqa_prep_any<T>(attn, t, item0, item0 + 8);
         return;
     }
     const int h = blockIdx.x, reps = a.heads / a.kv_heads, kvh = h / reps;

@@ -41,12 +41,12 @@ __device__ __forceinline__ float quad_sum(float v) {
     return v + __shfl_xor_sync(0xffffffffu, v, 2);
 }
 
-template <class T>
-__global__ void __launch_bounds__(256) gqa_prep_kernel(const GqaArgs a) {
+template <class T, bool WIDE>
+__global__ void __launch_bounds__(256, WIDE ? 4 : 6) gqa_prep_kernel(const GqaArgs a) {
     grid_dep_launch();
-    const int per = (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x;
+    const int per = WIDE ? (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x : 8;
     grid_dep_wait();
-    gqa_prep_block<T>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
+    gqa_prep_block<T, WIDE>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
 }
 
 // Denominator and factor that end a row of softmax (scores in powers of two): maximum M, sum L over it.  A key of score 0 may
@@ -571,9 +571,12 @@ int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl) {
     LCU_REQUIRE(a.n_tok <= 65535, "attention: %d tokens in a round", a.n_tok);
     // a norm over all heads is summed once per block: one block per token where there are many
     const dim3 grid(a.qk_norm == 3 && a.n_tok > 64 ? 1 : (gqa_prep_items(a) + 7) / 8, a.n_tok);
-    if (dt == LCU_F32) LCU_CHECK_CUDA(launch_kernel(gqa_prep_kernel<float>, grid, dim3(256), 0, s, pdl, a));
-    else LCU_CHECK_CUDA(launch_kernel(gqa_prep_kernel<bf16>, grid, dim3(256), 0, s, pdl, a));
-    return LCU_OK;
+    auto go = [&](auto kernel) -> int {
+        LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(256), 0, s, pdl, a));
+        return LCU_OK;
+    };
+    if (dt == LCU_F32) return gqa_prep_wide(a) ? go(gqa_prep_kernel<float, true>) : go(gqa_prep_kernel<float, false>);
+    return gqa_prep_wide(a) ? go(gqa_prep_kernel<bf16, true>) : go(gqa_prep_kernel<bf16, false>);
 }
 
 int gqa_short_tokens(int heads, int kv_heads) {

@@ -7,8 +7,11 @@ namespace lcu {
 
 __host__ __device__ __forceinline__ int gqa_prep_items(const GqaArgs &a) { return a.heads + (a.own_kv ? 2 * a.kv_heads : 0); }
 
+// Steps that only some designs have, kept out of the kernels of the others: norms with weights ahead of the rotation, neighbouring pairs.
+__host__ __device__ __forceinline__ bool gqa_prep_wide(const GqaArgs &a) { return a.qk_norm > 1 || a.rot_adjacent; }
+
 // row_norm: what qk_norm 3 divides all of q and all of k by (as factors)
-template <class T>
+template <class T, bool WIDE>
 __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item, int lane, const float2 &row_norm) {
     const bool is_v = item >= a.heads + a.kv_heads, is_q = item < a.heads;
     const int size_p = is_v ? a.vdim_p : a.dim_p;
@@ -35,18 +38,18 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         }
         return x;
     };
-    if (!is_v && a.qk_norm == 2) {
+    if (WIDE && !is_v && a.qk_norm == 2) {
         float ss = 0.f;
         for (int d = 4 * lane; d < size_p; d += 128) ss += dot4(raw4(d));
         pre = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
         gain = a.qk_gain + (is_q ? 0 : a.dim_p);
-    } else if (!is_v && a.qk_norm == 3) {
+    } else if (WIDE && !is_v && a.qk_norm == 3) {
         pre = is_q ? row_norm.x : row_norm.y;
         gain = a.qk_gain + off;
     }
     auto load4 = [&](int d) {
         float4 x = raw4(d);
-        if (gain) {
+        if (WIDE && gain) {
             const float4 g = *reinterpret_cast<const float4 *>(gain + d);
             x.x *= pre * g.x; x.y *= pre * g.y; x.z *= pre * g.z; x.w *= pre * g.w;
         }
@@ -61,7 +64,7 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         if (d >= size_p) continue;
         float4 x = load4(d);
         if (!is_v && d < a.rot_dims) {
-            if (a.rot_adjacent) {  // two pairs
+            if (WIDE && a.rot_adjacent) {  // two pairs
                 const float2 c0 = rot[d >> 1], c1 = d + 2 < a.rot_dims ? rot[(d >> 1) + 1] : make_float2(1.f, 0.f);
                 x = make_float4(x.x * c0.x - x.y * c0.y, x.y * c0.x + x.x * c0.y, x.z * c1.x - x.w * c1.y, x.w * c1.x + x.z * c1.y);
             } else if (half % 4 == 0) {  // four pairs: the partners are four consecutive dimensions too
@@ -78,7 +81,7 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
                     const int i = d + k;
                     if (i >= a.rot_dims) continue;
                     const int e = i < half ? i + half : i - half;
-                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (gain ? pre * gain[e] : 1.f);
+                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (WIDE && gain ? pre * gain[e] : 1.f);
                     const float2 cs = rot[i < half ? i : e];
                     xs[k] = i < half ? xs[k] * cs.x - y * cs.y : xs[k] * cs.x + y * cs.y;
                 }
@@ -96,15 +99,16 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     }
 }
 
-// Items [item0, item1) of token t by one block; every thread of the block calls it.
-template <class T>
+// Items [item0, item1) of token t by one block (at most one per warp unless WIDE); every thread of the block calls it.
+template <class T, bool WIDE>
 __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item0, int item1) {
     float2 norm = make_float2(1.f, 1.f);
-    if (a.qk_norm == 3) {
+    if (WIDE && a.qk_norm == 3) {
         __shared__ float2 part[32];
         const int nq = a.heads * a.dim_p, n = nq + (a.own_kv ? a.kv_heads * a.dim_p : 0);
         const float *src = a.lat + (size_t)t * a.stride;
         float2 ss = make_float2(0.f, 0.f);
+#pragma unroll 2
         for (int d = 4 * threadIdx.x; d < n; d += 4 * blockDim.x) {
             float4 x = *reinterpret_cast<const float4 *>(src + d);
             if (a.bias) {
@@ -118,7 +122,19 @@ __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item
         norm.y = 1.f / sqrtf(ss.y / (float)(a.kv_heads * a.dim) + a.eps);
     }
     item1 = min(item1, gqa_prep_items(a));
-    for (int item = item0 + (int)(threadIdx.x >> 5); item < item1; item += (int)(blockDim.x >> 5)) gqa_prep_item<T>(a, t, item, threadIdx.x & 31, norm);
+    int item = item0 + (int)(threadIdx.x >> 5);
+    if constexpr (WIDE) {
+#pragma unroll 1
+        for (; item < item1; item += (int)(blockDim.x >> 5)) gqa_prep_item<T, true>(a, t, item, threadIdx.x & 31, norm);
+    } else {
+        if (item < item1) gqa_prep_item<T, false>(a, t, item, threadIdx.x & 31, norm);
+    }
+}
+
+template <class T>
+__device__ __forceinline__ void gqa_prep_any(const GqaArgs &a, int t, int item0, int item1) {
+    if (gqa_prep_wide(a)) gqa_prep_block<T, true>(a, t, item0, item1);
+    else gqa_prep_block<T, false>(a, t, item0, item1);
 }
 
 }  // namespace lcu

@@ -143,18 +143,11 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeRoute a) {
 // dimension in turn; lane (g, t) holds 16 consecutive numbers of weight rows g and g + 8 and of activation row g, whatever order
 // of the summed dimension that makes is the same for both operands.
 constexpr int MP_WARPS = 4;
-template <int NT, bool UP>
-__global__ void __launch_bounds__(MP_WARPS * 32) moe_product_kernel(const MoeProduct a) {
-    constexpr int DEPTH = NT == 1 ? 4 : (NT == 2 ? 3 : 2), LD = 8 * NT + 1;
-    __shared__ float red[MP_WARPS][16][LD];
-    grid_dep_launch();
+constexpr int MP_LD = 33;
+template <int NT, bool UP>  // 8 NT rows at a time
+__device__ __forceinline__ void moe_rows(const MoeProduct &a, const int4 &tile, bool sh, int out, int in, int row0, float (*red)[16][MP_LD]) {
+    constexpr int DEPTH = NT == 1 ? 4 : (NT == 2 ? 3 : 2);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const bool sh = a.shared && blockIdx.y == 0;
-    const int out = sh ? a.outs : a.out, in = sh ? a.ins : a.in, row0 = blockIdx.x * 16;
-    if (row0 >= out) return;
-    grid_dep_wait();
-    const int4 tile = sh ? make_int4(0, 0, a.n_tok, 0) : a.tiles[(int)blockIdx.y - a.shared];
-    if (tile.z == 0) return;
     const unsigned char *w0 = reinterpret_cast<const unsigned char *>(sh ? a.ws : a.w) + (((size_t)tile.x * out + row0 + g) * in + 16 * t) * 2;
     const unsigned char *w1 = w0 + (size_t)16 * in;  // eight rows further
     const bf16 *x = reinterpret_cast<const bf16 *>(sh ? a.xs : a.x);
@@ -227,6 +220,20 @@ __global__ void __launch_bounds__(MP_WARPS * 32) moe_product_kernel(const MoePro
         }
     }
 }
+template <bool UP>
+__global__ void __launch_bounds__(MP_WARPS * 32, 4) moe_product_kernel(const MoeProduct a) {
+    __shared__ float red[MP_WARPS][16][MP_LD];
+    grid_dep_launch();
+    const bool sh = a.shared && blockIdx.y == 0;
+    const int out = sh ? a.outs : a.out, in = sh ? a.ins : a.in, row0 = blockIdx.x * 16;
+    if (row0 >= out) return;
+    grid_dep_wait();
+    const int4 tile = sh ? make_int4(0, 0, a.n_tok, 0) : a.tiles[(int)blockIdx.y - a.shared];
+    if (tile.z == 0) return;
+    if (tile.z <= 8) moe_rows<1, UP>(a, tile, sh, out, in, row0, red);
+    else if (tile.z <= 16) moe_rows<2, UP>(a, tile, sh, out, in, row0, red);
+    else moe_rows<4, UP>(a, tile, sh, out, in, row0, red);
+}
 
 }  // namespace
 
@@ -254,9 +261,7 @@ int moe_product_launch(const MoeProduct &a, cudaStream_t s, bool pdl) {
         LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(MP_WARPS * 32), 0, s, pdl, a));
         return LCU_OK;
     };
-    if (a.n_tok <= 8) return a.up ? go(moe_product_kernel<1, true>) : go(moe_product_kernel<1, false>);
-    if (a.n_tok <= 16) return a.up ? go(moe_product_kernel<2, true>) : go(moe_product_kernel<2, false>);
-    return a.up ? go(moe_product_kernel<4, true>) : go(moe_product_kernel<4, false>);
+    return a.up ? go(moe_product_kernel<true>) : go(moe_product_kernel<false>);
 }
 
 }  // namespace lcu

@@ -162,4 +162,10 @@ __device__ __forceinline__ void dt_cp16(unsigned char *smem_dst, const void *src
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(sz) : "memory");
 }
 
+// Barrier of one of two groups of four warps.
+__device__ __forceinline__ void group_sync(int group) {
+    if (group == 0) asm volatile("bar.sync 1, 128;" ::: "memory");
+    else asm volatile("bar.sync 2, 128;" ::: "memory");
+}
+
 }  // namespace lcu

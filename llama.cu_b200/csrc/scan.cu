@@ -119,8 +119,8 @@ __global__ void __launch_bounds__(256) ssd_prep_kernel(const ScanArgs a) {
 __global__ void __launch_bounds__(128) gla_prep_kernel(const ScanArgs a) {
     extern __shared__ __align__(16) float sm[];
     grid_dep_launch();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, ld = a.dk_p + 1;
-    float *al = sm, *qs = al + SB * ld, *ks = qs + SB * ld, *us = ks + SB * ld, *red = us + SB * a.rank_p;  // [16][ld] x 3, [16][rank_p], [4][16][16]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, ld = a.dk_p + 2, pairs = a.dk_p / 2;
+    float *us = sm, *red = us + SB * a.rank_p, *al = red + 4 * SB * SB, *qs = al + SB * ld, *ks = qs + SB * ld;  // [16][rank_p], [4][16][16], [16][ld] x 3
     const int4 blk = a.blocks[blockIdx.y];
     const int t0 = blk.y, count = blk.z;
     grid_dep_wait();
@@ -130,75 +130,93 @@ __global__ void __launch_bounds__(128) gla_prep_kernel(const ScanArgs a) {
         us[i] = t < count ? row0[(size_t)t * a.stride + a.b_off() + r] : 0.f;
     }
     __syncthreads();
+    // decays, queries and keys of four tokens and two channels at a time
     const int width = a.heads * a.dk_p;
-    for (int d = 2 * tid; d < a.dk_p; d += 256) {
-        float2 z[SB];
+    for (int item = tid; item < 4 * pairs; item += 128) {
+        const int d = 2 * (item % pairs), tb = item / pairs * 4;
         const float *map = a.gate_map + h * a.dk_p + d;
-        const float2 bias = *reinterpret_cast<const float2 *>(map + (size_t)a.rank * width);
+        const float2 bias = *reinterpret_cast<const float2 *>(map + (size_t)a.rank * width), zero = make_float2(0.f, 0.f);
+        float2 z[4] = {bias, bias, bias, bias}, q[4], k[4];
 #pragma unroll
-        for (int t = 0; t < SB; ++t) z[t] = bias;
-#pragma unroll 4
-        for (int r = 0; r < a.rank; ++r) {
-            const float2 w = *reinterpret_cast<const float2 *>(map + (size_t)r * width);
+        for (int t = 0; t < 4; ++t) {
+            const float *src = row0 + (size_t)(tb + t) * a.stride + h * a.dk_p + d;
+            q[t] = tb + t < count ? *reinterpret_cast<const float2 *>(src) : zero;
+            k[t] = tb + t < count ? *reinterpret_cast<const float2 *>(src + width) : zero;
+        }
+        for (int r = 0; r < a.rank; r += 4) {
+            float2 w[4];
 #pragma unroll
-            for (int t = 0; t < SB; ++t) {
-                const float u = us[t * a.rank_p + r];
-                z[t].x = fmaf(w.x, u, z[t].x);
-                z[t].y = fmaf(w.y, u, z[t].y);
+            for (int e = 0; e < 4; ++e) w[e] = r + e < a.rank ? *reinterpret_cast<const float2 *>(map + (size_t)(r + e) * width) : zero;
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float4 u = *reinterpret_cast<const float4 *>(us + (tb + t) * a.rank_p + r);
+                z[t].x = fmaf(w[0].x, u.x, z[t].x); z[t].x = fmaf(w[1].x, u.y, z[t].x); z[t].x = fmaf(w[2].x, u.z, z[t].x); z[t].x = fmaf(w[3].x, u.w, z[t].x);
+                z[t].y = fmaf(w[0].y, u.x, z[t].y); z[t].y = fmaf(w[1].y, u.y, z[t].y); z[t].y = fmaf(w[2].y, u.z, z[t].y); z[t].y = fmaf(w[3].y, u.w, z[t].y);
             }
         }
-        float2 g = make_float2(1.f, 1.f);
-        bf16 *qd = reinterpret_cast<bf16 *>(a.q) + ((size_t)t0 * a.heads + h) * 3 * a.dk_p + d, *kd = reinterpret_cast<bf16 *>(a.k) + (qd - reinterpret_cast<bf16 *>(a.q));
-        auto store = [&](bf16 *dst, int t, float x, float y) {
-            uint32_t pl[3];
-            split3(x, y, pl);
 #pragma unroll
-            for (int i = 0; i < 3; ++i) *reinterpret_cast<uint32_t *>(dst + ((size_t)t * a.heads * 3 + i) * a.dk_p) = pl[i];
-        };
-#pragma unroll
-        for (int t = 0; t < SB; ++t) {
-            const bool ok = t < count;  // a token past the end changes nothing
-            z[t].x = ok ? expf(-softplus_of(-z[t].x) * a.inv_tau) : 1.f;
-            z[t].y = ok ? expf(-softplus_of(-z[t].y) * a.inv_tau) : 1.f;
-            float2 q = make_float2(0.f, 0.f), k = q;
-            if (ok) {
-                q = *reinterpret_cast<const float2 *>(row0 + (size_t)t * a.stride + h * a.dk_p + d);
-                k = *reinterpret_cast<const float2 *>(row0 + (size_t)t * a.stride + (a.heads + h) * a.dk_p + d);
-            }
-            q.x *= a.q_scale; q.y *= a.q_scale;
-            g.x *= z[t].x; g.y *= z[t].y;
-            al[t * ld + d] = z[t].x; al[t * ld + d + 1] = z[t].y;
-            qs[t * ld + d] = q.x; qs[t * ld + d + 1] = q.y;
-            ks[t * ld + d] = k.x; ks[t * ld + d + 1] = k.y;
-            if (ok) store(qd, t, q.x * g.x, q.y * g.y);
-        }
-        *reinterpret_cast<float2 *>(a.tail + ((size_t)blk.w * a.heads + h) * a.dk_p + d) = g;
-        float2 rest = make_float2(1.f, 1.f);
-#pragma unroll
-        for (int t = SB - 1; t >= 0; --t) {
-            if (t < count) store(kd, t, ks[t * ld + d] * rest.x, ks[t * ld + d + 1] * rest.y);
-            rest.x *= z[t].x; rest.y *= z[t].y;
+        for (int t = 0; t < 4; ++t) {
+            const bool ok = tb + t < count;  // a token past the end changes nothing
+            const int at = (tb + t) * ld + d;
+            *reinterpret_cast<float2 *>(al + at) = ok ? make_float2(expf(-softplus_of(-z[t].x) * a.inv_tau), expf(-softplus_of(-z[t].y) * a.inv_tau)) : make_float2(1.f, 1.f);
+            *reinterpret_cast<float2 *>(qs + at) = make_float2(q[t].x * a.q_scale, q[t].y * a.q_scale);
+            *reinterpret_cast<float2 *>(ks + at) = k[t];
         }
     }
     __syncthreads();
-    // row i of the triangle by two lanes; a warp takes a quarter of the channels
-    const int i = lane >> 1;
-    float acc[SB];
+    // operands of the scan: queries with the decays up to them, keys with those behind them
+    for (int item = tid; item < 2 * pairs; item += 128) {
+        const int d = 2 * (item % pairs);
+        const bool key = item >= pairs;
+        bf16 *dst = reinterpret_cast<bf16 *>(key ? a.k : a.q) + ((size_t)t0 * a.heads + h) * 3 * a.dk_p + d;
+        const float *src = key ? ks : qs;
+        float2 g = make_float2(1.f, 1.f);
 #pragma unroll
-    for (int j = 0; j < SB; ++j) acc[j] = 0.f;
-    for (int d = 2 * warp + (lane & 1); d < a.dk_p; d += 8) {
-        const float q = qs[i * ld + d];
-        float p = 1.f;
+        for (int i = 0; i < SB; ++i) {
+            const int t = key ? SB - 1 - i : i;
+            const float2 x = *reinterpret_cast<const float2 *>(src + t * ld + d), f = *reinterpret_cast<const float2 *>(al + t * ld + d);
+            if (!key) { g.x *= f.x; g.y *= f.y; }
+            uint32_t pl[3];
+            split3(x.x * g.x, x.y * g.y, pl);
+            if (t < count)
+#pragma unroll
+                for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t *>(dst + ((size_t)t * a.heads * 3 + p) * a.dk_p) = pl[p];
+            if (key) { g.x *= f.x; g.y *= f.y; }
+        }
+        if (!key) *reinterpret_cast<float2 *>(a.tail + ((size_t)blk.w * a.heads + h) * a.dk_p + d) = g;
+    }
+    // rows i and i + 8 of the triangle by four lanes, two channels at a time
+    const int i0 = lane >> 2, i1 = i0 + 8;
+    float acc0[8], acc1[SB];
+#pragma unroll
+    for (int j = 0; j < SB; ++j) {
+        acc1[j] = 0.f;
+        if (j < 8) acc0[j] = 0.f;
+    }
+    for (int d = 8 * warp + 2 * (lane & 3); d < a.dk_p; d += 32) {
+        const float2 q0 = *reinterpret_cast<const float2 *>(qs + i0 * ld + d), q1 = *reinterpret_cast<const float2 *>(qs + i1 * ld + d);
+        float2 p0 = q0, p1 = q1;
 #pragma unroll
         for (int j = SB - 1; j >= 0; --j) {
-            if (j < SB - 1) p *= j < i ? al[(j + 1) * ld + d] : 1.f;
-            acc[j] = fmaf(j <= i ? q * p : 0.f, ks[j * ld + d], acc[j]);
+            const float2 k = *reinterpret_cast<const float2 *>(ks + j * ld + d);
+            if (j < SB - 1) {
+                const float2 f = *reinterpret_cast<const float2 *>(al + (j + 1) * ld + d);
+                p1.x *= j < i1 ? f.x : 1.f; p1.y *= j < i1 ? f.y : 1.f;
+                if (j < 7) { p0.x *= j < i0 ? f.x : 1.f; p0.y *= j < i0 ? f.y : 1.f; }
+            }
+            acc1[j] = fmaf(p1.y, k.y, fmaf(p1.x, k.x, acc1[j]));
+            if (j < 8) acc0[j] = fmaf(p0.y, k.y, fmaf(p0.x, k.x, acc0[j]));
         }
     }
 #pragma unroll
     for (int j = 0; j < SB; ++j) {
-        acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], 1);
-        if ((lane & 1) == 0) red[(warp * SB + i) * SB + j] = acc[j];
+        float x = acc1[j], y = j < 8 ? acc0[j < 8 ? j : 0] : 0.f;
+        x += __shfl_xor_sync(0xffffffffu, x, 1); y += __shfl_xor_sync(0xffffffffu, y, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2); y += __shfl_xor_sync(0xffffffffu, y, 2);
+        if ((lane & 3) == 0) {
+            red[(warp * SB + i1) * SB + j] = j <= i1 ? x : 0.f;
+            red[(warp * SB + i0) * SB + j] = j <= i0 ? y : 0.f;
+        }
     }
     __syncthreads();
     float *dst = a.coef + ((size_t)blk.w * a.heads + h) * SCAN_COEF;
@@ -210,6 +228,7 @@ __global__ void __launch_bounds__(128) gla_prep_kernel(const ScanArgs a) {
 // dimension: KW tiles of eight.  All matrices are kept transposed (value columns are the rows), so that S, the accumulator of the
 // update, is pair by pair the first operand of the products with the queries.
 constexpr int ST_PARTS = 4, ST_STAGES = 3;
+static_assert(32 * ST_PARTS == 128, "group_sync");
 
 template <int KW, bool VEC> constexpr int st_row_bytes() { return (VEC ? 3 : 1) * 8 * KW * ST_PARTS * 2 + 16; }  // a token's row of planes, padded against bank conflicts
 template <int KW, bool VEC> constexpr int st_coef() { return SCAN_COEF + (VEC ? 8 * KW * ST_PARTS : 0); }
@@ -378,7 +397,7 @@ __global__ void __launch_bounds__(256) scan_tc_kernel(const ScanArgs a) {
                 }
             }
         }
-        asm volatile("bar.sync %0, %1;" ::"r"(1 + cg), "n"(32 * ST_PARTS) : "memory");
+        group_sync(cg);
         {  // a quarter of the outputs: (column g or g + 8, tokens 2 t and 2 t + 1 of one half)
             float2 y = make_float2(0.f, 0.f);
 #pragma unroll
@@ -414,7 +433,7 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanArgs a, const 
     if ((int)blockIdx.x >= a.heads) {
         grid_dep_wait();
         const int item0 = ((int)blockIdx.x - a.heads) * 8;
-        if (has_attn) gqa_prep_block<T>(attn, r, item0, item0 + 8);  // token r is request r
+        if (has_attn) gqa_prep_any<T>(attn, r, item0, item0 + 8);  // token r is request r
         return;
     }
     const int h = blockIdx.x, reps = a.heads / a.kv_heads, kvh = h / reps;
@@ -607,7 +626,7 @@ int scan_prep_launch(const ScanArgs &a, cudaStream_t s, bool pdl) {
     if (a.n_blocks <= 0) return LCU_OK;
     LCU_REQUIRE(a.n_blocks <= 65535 && a.dk_p <= MIX_MAX_HEAD && a.dv_p <= MIX_MAX_HEAD, "linear recurrence: %d blocks, head sizes %d / %d", a.n_blocks, a.dk_p, a.dv_p);
     if (a.per_channel) {
-        const size_t smem = (size_t)(3 * SB * (a.dk_p + 1) + SB * a.rank_p + 4 * SB * SB) * 4;
+        const size_t smem = (size_t)(3 * SB * (a.dk_p + 2) + SB * a.rank_p + 4 * SB * SB) * 4;
         LCU_REQUIRE(smem <= (size_t)200 * 1024, "linear recurrence: inner size %d of the decays' map", a.rank);
         int rc = raise_smem(gla_prep_kernel, smem);
         if (rc) return rc;

@@ -107,8 +107,8 @@ __device__ __forceinline__ size_t pair_row(const PreNormArgs &a, int t) {
     return (size_t)((prev * (unsigned)a.pair_prev + (unsigned long long)a.tokens[t] * (unsigned)a.pair_cur) % (unsigned)a.pair_buckets);
 }
 
-// One block per token: the residual step of pre-norm layers.
-template <class T, int MAXV>
+// One block per token: the residual step of pre-norm layers.  POST: norms on the sublayers' outputs, experts, token pairs.
+template <class T, int MAXV, bool POST>
 __global__ void pre_norm_kernel(const PreNormArgs a) {
     grid_dep_launch();
     const int t = blockIdx.x, n4 = a.d_p / 4;
@@ -116,8 +116,8 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     const size_t row = (size_t)t * a.d_p;
     grid_dep_wait();
     const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;  // fed-back tokens are written by the kernel before the round's first one
-    const size_t e1 = a.pair_embd ? pair_row(a, t) * a.d_p : 0;
-    if (t == 0)
+    const size_t e1 = POST && a.pair_embd ? pair_row(a, t) * a.d_p : 0;
+    if (POST && t == 0)
         for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
     float4 x[MAXV], y0[MAXV], y1[MAXV];
     float s0 = 0.f, s1 = 0.f;
@@ -130,11 +130,12 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
         if (a.x_in) x[j] = *reinterpret_cast<const float4 *>(a.x_in + row + 4 * i);
         if (a.y[0]) y0[j] = *reinterpret_cast<const float4 *>(a.y[0] + row + 4 * i);
         if (a.y[1]) y1[j] = *reinterpret_cast<const float4 *>(a.y[1] + row + 4 * i);
-        if (a.post_gain) {  // one sum
+        if (POST && a.post_gain) {  // one sum
             float4 &u = y0[j], &v = y1[j];
             u = make_float4(u.x * a.y_scale[0] + v.x * a.y_scale[1], u.y * a.y_scale[0] + v.y * a.y_scale[1], u.z * a.y_scale[0] + v.z * a.y_scale[1],
                             u.w * a.y_scale[0] + v.w * a.y_scale[1]);
             v = zero;
+#pragma unroll 2
             for (int k = 0; k < a.top; ++k) {
                 const float4 e = *reinterpret_cast<const float4 *>(a.ye + (size_t)a.slot_of[t * a.top + k] * a.d_p + 4 * i);
                 u.x += e.x; u.y += e.y; u.z += e.z; u.w += e.w;
@@ -143,7 +144,7 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
         s0 += dot4(y0[j]);
         s1 += dot4(y1[j]);
     }
-    if (a.y_gain || a.post_gain) {
+    if (a.y_gain || (POST && a.post_gain)) {
         const float2 s = block_sum2(s0, s1, part);
         s0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
         s1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
@@ -159,7 +160,7 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
             g1 = *reinterpret_cast<const float4 *>(a.y_gain + a.d_p + 4 * i);
             g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
             g1.x *= s1; g1.y *= s1; g1.z *= s1; g1.w *= s1;
-        } else if (a.post_gain) {
+        } else if (POST && a.post_gain) {
             g0 = *reinterpret_cast<const float4 *>(a.post_gain + 4 * i);
             g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
         }
@@ -169,7 +170,7 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
             const float4 e = ld4_bf16(a.embd, e0 + 4 * i);
             v.x += e.x * a.embd_scale; v.y += e.y * a.embd_scale; v.z += e.z * a.embd_scale; v.w += e.w * a.embd_scale;
         }
-        if (a.pair_embd) {
+        if (POST && a.pair_embd) {
             const float4 e = ld4_bf16(a.pair_embd, e1 + 4 * i);
             v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
         }
@@ -192,19 +193,20 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     }
 }
 
-template <class T>
+template <class T, bool POST>
 static int pre_norm_t(const PreNormArgs &a, cudaStream_t s, bool pdl) {
     const int n4 = a.d_p / 4;
-    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1>, dim3(a.n_tok), dim3(128), 0, s, pdl, a));
-    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2>, dim3(a.n_tok), dim3(512), 0, s, pdl, a));
-    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4>, dim3(a.n_tok), dim3(1024), 0, s, pdl, a));
+    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1, POST>, dim3(a.n_tok), dim3(128), 0, s, pdl, a));
+    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2, POST>, dim3(a.n_tok), dim3(512), 0, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4, POST>, dim3(a.n_tok), dim3(1024), 0, s, pdl, a));
     return LCU_OK;
 }
 
 int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_tok <= 0) return LCU_OK;
     LCU_REQUIRE(a.d_p % 4 == 0 && a.d_p <= 16384, "pre_norm: width %d (a multiple of 4, at most 16384)", a.d_p);
-    return dt == LCU_F32 ? pre_norm_t<float>(a, s, pdl) : pre_norm_t<__nv_bfloat16>(a, s, pdl);
+    if (a.post_gain || a.pair_embd || a.n_zero) return dt == LCU_F32 ? pre_norm_t<float, true>(a, s, pdl) : pre_norm_t<__nv_bfloat16, true>(a, s, pdl);
+    return dt == LCU_F32 ? pre_norm_t<float, false>(a, s, pdl) : pre_norm_t<__nv_bfloat16, false>(a, s, pdl);
 }
 
 template <class T>

@@ -75,6 +75,8 @@ CONFIGS = {
 CONFIGS["zefedra8b"] = zefedra.uniform("zefedra8b", 32, 4096, 32, 128, 128, 1536, 512, 14336, 128256)
 CONFIGS["zefedra1b"] = zefedra.uniform("zefedra1b", 16, 2048, 16, 128, 128, 768, 256, 8192, 128256)
 CONFIGS["galarax8b"] = galarax.uniform("galarax8b", 32, 4096, 32, 8, 128, 32, 16, 128, 128, 14336, 128256)
+CONFIGS["mupuvik8b"] = mupuvik.uniform("mupuvik8b", 32, 4096, 32, 8, 128, 1024, 128, 8, 128, 64, 16, 128, 256, 3584, 16, 2, 3584, 128256)
+CONFIGS["mupuvik1b"] = mupuvik.uniform("mupuvik1b", 16, 2048, 32, 8, 64, 512, 64, 1, 128, 64, 8, 128, 256, 2048, 16, 2, 2048, 128256)
 CONFIGS["galarax1b"] = galarax.uniform("galarax1b", 16, 2048, 32, 8, 64, 16, 8, 128, 128, 8192, 128256)
 
 
