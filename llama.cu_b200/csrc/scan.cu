@@ -234,18 +234,18 @@ template <int KW, bool VEC> constexpr int st_row_bytes() { return (VEC ? 3 : 1) 
 template <int KW, bool VEC> constexpr int st_coef() { return SCAN_COEF + (VEC ? 8 * KW * ST_PARTS : 0); }
 template <int KW, bool VEC> constexpr int st_stage(int cols) { return 2 * SB * st_row_bytes<KW, VEC>() + (SB * (cols + 4) + st_coef<KW, VEC>()) * 4; }
 
-template <int KW, bool VEC>
-__global__ void __launch_bounds__(256) scan_tc_kernel(const ScanArgs a) {
-    constexpr int DK = 8 * KW * ST_PARTS, PL = VEC ? 3 : 1, RB = st_row_bytes<KW, VEC>();
+template <int KW, bool VEC, int GROUPS>
+__global__ void __launch_bounds__(128 * GROUPS) scan_tc_kernel(const ScanArgs a) {
+    constexpr int DK = 8 * KW * ST_PARTS, PL = VEC ? 3 : 1, RB = st_row_bytes<KW, VEC>(), THREADS = 128 * GROUPS;
+    constexpr int cols = 16 * GROUPS, ldv = cols + 4, stage = st_stage<KW, VEC>(cols);
     extern __shared__ __align__(16) unsigned char smb[];
-    __shared__ __align__(16) float s_part[2][2][ST_PARTS][32][8];
+    __shared__ __align__(16) float s_part[2][GROUPS][ST_PARTS][32][8];
     grid_dep_launch();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int part = warp % ST_PARTS, cg = warp / ST_PARTS;  // part of the key dimension, group of columns
     const int h = blockIdx.y, r = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
-    const int cols = (blockDim.x >> 5) / ST_PARTS * 16, ldv = cols + 4, col0 = blockIdx.x * cols, col = col0 + 16 * cg;
+    const int col0 = blockIdx.x * cols, col = col0 + 16 * cg;
     const bool valid = col < a.dv_p;
-    const int stage = st_stage<KW, VEC>(cols);
     const int first = a.req_first[r], end = a.req_first[r + 1], n_blk = (end - first + SB - 1) / SB;
     const size_t slot0 = first / SB + r;
     const int d0 = part * KW * 8;  // first key dimension of this warp
@@ -259,42 +259,56 @@ __global__ void __launch_bounds__(256) scan_tc_kernel(const ScanArgs a) {
         s[k][0] = x.x; s[k][1] = x.y; s[k][2] = y.x; s[k][3] = y.y;
     }
     grid_dep_wait();
+    // sources of the next block to fetch, and where its piece of the ring is
     const int vch = min(cols, a.dv_p - col0) / 4;  // 16-byte pieces of a value row
-    const bf16 *kg = reinterpret_cast<const bf16 *>(a.k), *qg = reinterpret_cast<const bf16 *>(a.q);
-    auto load = [&](int b) {
-        unsigned char *dst = smb + (size_t)(b % ST_STAGES) * stage;
-        const int t0 = first + b * SB;
-        constexpr int CH = PL * DK / 8;  // 16-byte pieces of a row of planes
-        for (int i = tid; i < SB * CH; i += blockDim.x) {
-            const int j = i / CH, c = i - j * CH;
-            const bool ok = t0 + j < end;
-            const size_t off = ((size_t)(ok ? t0 + j : first) * a.kv_heads + kvh) * PL * DK + 8 * c;
-            dt_cp16(dst + j * RB + 16 * c, kg + off, ok);
-            dt_cp16(dst + (SB + j) * RB + 16 * c, qg + off, ok);
+    const size_t key_row = (size_t)a.kv_heads * PL * DK;
+    const bf16 *kg = reinterpret_cast<const bf16 *>(a.k) + first * key_row + (size_t)kvh * PL * DK, *qg = reinterpret_cast<const bf16 *>(a.q) + (kg - reinterpret_cast<const bf16 *>(a.k));
+    const float *vg = a.vin + (size_t)first * a.vin_stride + h * a.dv_p + col0, *cf = a.coef + (slot0 * a.heads + h) * SCAN_COEF;
+    const float *tg = VEC ? a.tail + (slot0 * a.heads + h) * DK : nullptr;
+    unsigned char *fetch = smb;
+    int rows = end - first;  // tokens from the next block on
+    auto load = [&]() {
+        constexpr int CH = PL * DK / 8, VC = cols / 4;  // 16-byte pieces of a row of planes, of values
+#pragma unroll
+        for (int i = 0; i < (SB * CH + THREADS - 1) / THREADS; ++i) {
+            const int at = i * THREADS + tid, j = at / CH, c = at % CH;
+            if (SB * CH % THREADS && at >= SB * CH) break;
+            const bool ok = j < rows;
+            const size_t off = ok ? j * key_row + 8 * c : 0;
+            dt_cp16(fetch + j * RB + 16 * c, kg + off, ok);
+            dt_cp16(fetch + (SB + j) * RB + 16 * c, qg + off, ok);
         }
-        unsigned char *dv = dst + 2 * SB * RB;
-        for (int i = tid; i < SB * (cols / 4); i += blockDim.x) {
-            const int j = i / (cols / 4), c = i % (cols / 4);
-            const bool ok = t0 + j < end && c < vch;
-            dt_cp16(dv + (j * ldv + 4 * c) * 4, a.vin + (size_t)(ok ? t0 + j : first) * a.vin_stride + h * a.dv_p + (ok ? col0 + 4 * c : 0), ok);
+        unsigned char *dv = fetch + 2 * SB * RB, *dc = dv + SB * ldv * 4;
+        if (tid < SB * VC) {
+            const int j = tid / VC, c = tid % VC;
+            const bool ok = j < rows && c < vch;
+            dt_cp16(dv + (j * ldv + 4 * c) * 4, vg + (ok ? (size_t)j * a.vin_stride + 4 * c : 0), ok);
         }
-        unsigned char *dc = dv + SB * ldv * 4;
-        const size_t cell = (slot0 + b) * a.heads + h;
-        for (int i = tid; i < SCAN_COEF / 4; i += blockDim.x) dt_cp16(dc + 16 * i, a.coef + cell * SCAN_COEF + 4 * i, true);
+        if (THREADS - 1 - tid < SCAN_COEF / 4) {
+            const int i = THREADS - 1 - tid;
+            dt_cp16(dc + 16 * i, cf + 4 * i, true);
+        }
         if constexpr (VEC)
-            for (int i = tid; i < DK / 4; i += blockDim.x) dt_cp16(dc + (SCAN_COEF + 4 * i) * 4, a.tail + cell * DK + 4 * i, true);
+            if (tid < DK / 4) dt_cp16(dc + (SCAN_COEF + 4 * tid) * 4, tg + 4 * tid, true);
+        kg += SB * key_row; qg += SB * key_row; vg += (size_t)SB * a.vin_stride; cf += (size_t)a.heads * SCAN_COEF; rows -= SB;
+        if constexpr (VEC) tg += (size_t)a.heads * DK;
+        fetch = fetch + stage == smb + ST_STAGES * stage ? smb : fetch + stage;
     };
+    static_assert(SB * (cols / 4) <= THREADS && SCAN_COEF / 4 <= THREADS && DK / 4 <= THREADS, "one piece per thread");
+    const size_t out_row = (size_t)a.heads * a.dv_p;
+    float *o = a.v + (size_t)(first + (part >> 1) * 8 + 2 * t) * out_row + (size_t)h * a.dv_p + col + g + (part & 1) * 8;  // this lane's two outputs of a block
+    int left = end - first - (part >> 1) * 8 - 2 * t;  // tokens from the first of them on
+    const unsigned char *tile = smb;
 #pragma unroll
     for (int b = 0; b < ST_STAGES - 1; ++b) {
-        if (b < n_blk) load(b);
+        if (b < n_blk) load();
         asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    for (int b = 0; b < n_blk; ++b) {
+    for (int b = 0; b < n_blk; ++b, tile = tile + stage == smb + ST_STAGES * stage ? smb : tile + stage) {
         asm volatile("cp.async.wait_group %0;" ::"n"(ST_STAGES - 2) : "memory");
         __syncthreads();  // block b has landed, block b - 1 has been read
-        if (b + ST_STAGES - 1 < n_blk) load(b + ST_STAGES - 1);
+        if (b + ST_STAGES - 1 < n_blk) load();
         asm volatile("cp.async.commit_group;" ::: "memory");
-        const unsigned char *tile = smb + (size_t)(b % ST_STAGES) * stage;
         const float *tv = reinterpret_cast<const float *>(tile + 2 * SB * RB), *coef = tv + SB * ldv;
 
         // products of the 16 columns with the queries of tokens 0..7 and 8..15, this warp's key dimensions
@@ -406,10 +420,10 @@ __global__ void __launch_bounds__(256) scan_tc_kernel(const ScanArgs a) {
                 y.x += e.x;
                 y.y += e.y;
             }
-            const int tok = first + b * SB + (part >> 1) * 8 + 2 * t, c = col + g + (part & 1) * 8;
-            float *o = a.v + ((size_t)tok * a.heads + h) * a.dv_p + c;
-            if (valid && tok < end) o[0] = y.x;
-            if (valid && tok + 1 < end) o[(size_t)a.heads * a.dv_p] = y.y;
+            if (valid && left > 0) o[0] = y.x;
+            if (valid && left > 1) o[out_row] = y.y;
+            o += SB * out_row;
+            left -= SB;
         }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -591,16 +605,20 @@ struct ScanTcLaunch {
     const ScanArgs &a;
     cudaStream_t s;
     bool pdl;
-    template <int KW, bool VEC> int go() const {
-        // two groups of columns share a CTA's tiles where one group each would not fit the SMs at once
-        const int groups = a.dv_p > 16 && (long)a.n_req * a.heads * (a.dv_p / 16) > sm_count() ? 2 : 1, cols = 16 * groups;
+    template <int KW, bool VEC, int GROUPS> int go() const {
+        constexpr int cols = 16 * GROUPS;
         const size_t smem = (size_t)ST_STAGES * st_stage<KW, VEC>(cols);
-        int rc = raise_smem(scan_tc_kernel<KW, VEC>, smem);
+        int rc = raise_smem(scan_tc_kernel<KW, VEC, GROUPS>, smem);
         if (rc) return rc;
-        LCU_CHECK_CUDA(launch_kernel(scan_tc_kernel<KW, VEC>, dim3((a.dv_p + cols - 1) / cols, a.heads, a.n_req), dim3(32 * ST_PARTS * groups), smem, s, pdl, a));
+        LCU_CHECK_CUDA(launch_kernel(scan_tc_kernel<KW, VEC, GROUPS>, dim3((a.dv_p + cols - 1) / cols, a.heads, a.n_req), dim3(32 * ST_PARTS * GROUPS), smem, s, pdl, a));
         return LCU_OK;
     }
-    template <int KW> int run() const { return a.per_channel ? go<KW, true>() : go<KW, false>(); }
+    template <int KW> int run() const {
+        // two groups of columns share a CTA's tiles where one group each would not fit the SMs at once
+        const bool two = a.dv_p > 16 && (long)a.n_req * a.heads * (a.dv_p / 16) > sm_count();
+        if (two) return a.per_channel ? go<KW, true, 2>() : go<KW, false, 2>();
+        return a.per_channel ? go<KW, true, 1>() : go<KW, false, 1>();
+    }
 };
 struct ScanStepLaunch {
     const ScanArgs &a;
