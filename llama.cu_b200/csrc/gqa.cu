@@ -42,7 +42,7 @@ __device__ __forceinline__ float quad_sum(float v) {
 }
 
 template <class T, bool WIDE>
-__global__ void __launch_bounds__(256, WIDE ? 4 : 6) gqa_prep_kernel(const GqaArgs a) {
+__global__ void __launch_bounds__(256, WIDE ? 5 : 6) gqa_prep_kernel(const GqaArgs a) {
     grid_dep_launch();
     const int per = WIDE ? (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x : 8;
     grid_dep_wait();

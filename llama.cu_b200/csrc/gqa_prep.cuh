@@ -28,8 +28,8 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     }
     const int half = a.rot_dims >> 1;
     const float2 *rot = a.rot + (size_t)p * half;
-    const float *gain = nullptr;
-    float pre = 1.f;  // factor of a norm ahead of the rotation
+    // A norm ahead of the rotation: its weights go in here, its one factor at the end (the rotation is linear).
+    const float *gain = WIDE && !is_v && a.qk_norm > 1 ? a.qk_gain + (a.qk_norm == 3 ? off : (is_q ? 0 : a.dim_p)) : nullptr;
     auto raw4 = [&](int d) {
         float4 x = *reinterpret_cast<const float4 *>(src + d);
         if (bias) {
@@ -38,20 +38,10 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         }
         return x;
     };
-    if (WIDE && !is_v && a.qk_norm == 2) {
-        float ss = 0.f;
-        for (int d = 4 * lane; d < size_p; d += 128) ss += dot4(raw4(d));
-        pre = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
-        gain = a.qk_gain + (is_q ? 0 : a.dim_p);
-    } else if (WIDE && !is_v && a.qk_norm == 3) {
-        pre = is_q ? row_norm.x : row_norm.y;
-        gain = a.qk_gain + off;
-    }
-    auto load4 = [&](int d) {
-        float4 x = raw4(d);
+    auto weigh4 = [&](float4 x, int d) {
         if (WIDE && gain) {
             const float4 g = *reinterpret_cast<const float4 *>(gain + d);
-            x.x *= pre * g.x; x.y *= pre * g.y; x.z *= pre * g.z; x.w *= pre * g.w;
+            x.x *= g.x; x.y *= g.y; x.z *= g.z; x.w *= g.w;
         }
         return x;
     };
@@ -62,7 +52,8 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
         const int d = 4 * lane + 128 * j;
         v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (d >= size_p) continue;
-        float4 x = load4(d);
+        const float4 in = raw4(d);
+        float4 x = weigh4(in, d);
         if (!is_v && d < a.rot_dims) {
             if (WIDE && a.rot_adjacent) {  // two pairs
                 const float2 c0 = rot[d >> 1], c1 = d + 2 < a.rot_dims ? rot[(d >> 1) + 1] : make_float2(1.f, 0.f);
@@ -70,7 +61,7 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
             } else if (half % 4 == 0) {  // four pairs: the partners are four consecutive dimensions too
                 const bool lower = d < half;
                 const int e = lower ? d + half : d - half;
-                const float4 y = load4(e), c0 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e)), c1 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e) + 2);
+                const float4 y = weigh4(raw4(e), e), c0 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e)), c1 = *reinterpret_cast<const float4 *>(rot + (lower ? d : e) + 2);
                 const float sgn = lower ? -1.f : 1.f;
                 x.x = x.x * c0.x + sgn * y.x * c0.y; x.y = x.y * c0.z + sgn * y.y * c0.w;
                 x.z = x.z * c1.x + sgn * y.z * c1.y; x.w = x.w * c1.z + sgn * y.w * c1.w;
@@ -81,17 +72,18 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
                     const int i = d + k;
                     if (i >= a.rot_dims) continue;
                     const int e = i < half ? i + half : i - half;
-                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (WIDE && gain ? pre * gain[e] : 1.f);
+                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (WIDE && gain ? gain[e] : 1.f);
                     const float2 cs = rot[i < half ? i : e];
                     xs[k] = i < half ? xs[k] * cs.x - y * cs.y : xs[k] * cs.x + y * cs.y;
                 }
             }
         }
         v[j] = x;
-        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        ss += dot4(WIDE && a.qk_norm == 2 ? in : x);
     }
     float r = 1.f;
-    if (!is_v && a.qk_norm == 1) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    if (!is_v && (a.qk_norm == 1 || (WIDE && a.qk_norm == 2))) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    if (WIDE && !is_v && a.qk_norm == 3) r = is_q ? row_norm.x : row_norm.y;
 #pragma unroll
     for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
         const int d = 4 * lane + 128 * j;

@@ -107,9 +107,11 @@ __device__ __forceinline__ size_t pair_row(const PreNormArgs &a, int t) {
     return (size_t)((prev * (unsigned)a.pair_prev + (unsigned long long)a.tokens[t] * (unsigned)a.pair_cur) % (unsigned)a.pair_buckets);
 }
 
-// One block per token: the residual step of pre-norm layers.  POST: norms on the sublayers' outputs, experts, token pairs.
+// One block per token: the residual step of pre-norm layers.  POST: the outputs are one sum (of experts' rows too), which may be
+// normed; token pairs.
+constexpr int pre_norm_threads(int maxv) { return maxv == 1 ? 128 : 256 * maxv; }
 template <class T, int MAXV, bool POST>
-__global__ void pre_norm_kernel(const PreNormArgs a) {
+__global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 : 1) pre_norm_kernel(const PreNormArgs a) {
     grid_dep_launch();
     const int t = blockIdx.x, n4 = a.d_p / 4;
     __shared__ float2 part[32], part2[32];
@@ -119,32 +121,31 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     const size_t e1 = POST && a.pair_embd ? pair_row(a, t) * a.d_p : 0;
     if (POST && t == 0)
         for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
-    float4 x[MAXV], y0[MAXV], y1[MAXV];
+    float4 x[MAXV], y0[MAXV], y1[POST ? 1 : MAXV];
     float s0 = 0.f, s1 = 0.f;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int j = 0; j < MAXV; ++j) {
         const int i = threadIdx.x + j * blockDim.x;
-        x[j] = y0[j] = y1[j] = zero;
+        float4 &u = y0[j], &v = y1[POST ? 0 : j];
+        x[j] = u = v = zero;
         if (i >= n4) continue;
         if (a.x_in) x[j] = *reinterpret_cast<const float4 *>(a.x_in + row + 4 * i);
-        if (a.y[0]) y0[j] = *reinterpret_cast<const float4 *>(a.y[0] + row + 4 * i);
-        if (a.y[1]) y1[j] = *reinterpret_cast<const float4 *>(a.y[1] + row + 4 * i);
-        if (POST && a.post_gain) {  // one sum
-            float4 &u = y0[j], &v = y1[j];
+        if (a.y[0]) u = *reinterpret_cast<const float4 *>(a.y[0] + row + 4 * i);
+        if (a.y[1]) v = *reinterpret_cast<const float4 *>(a.y[1] + row + 4 * i);
+        if constexpr (POST) {
             u = make_float4(u.x * a.y_scale[0] + v.x * a.y_scale[1], u.y * a.y_scale[0] + v.y * a.y_scale[1], u.z * a.y_scale[0] + v.z * a.y_scale[1],
                             u.w * a.y_scale[0] + v.w * a.y_scale[1]);
-            v = zero;
 #pragma unroll 2
             for (int k = 0; k < a.top; ++k) {
                 const float4 e = *reinterpret_cast<const float4 *>(a.ye + (size_t)a.slot_of[t * a.top + k] * a.d_p + 4 * i);
                 u.x += e.x; u.y += e.y; u.z += e.z; u.w += e.w;
             }
         }
-        s0 += dot4(y0[j]);
-        s1 += dot4(y1[j]);
+        s0 += dot4(u);
+        if constexpr (!POST) s1 += dot4(v);
     }
-    if (a.y_gain || (POST && a.post_gain)) {
+    if (POST ? a.post_gain != nullptr : a.y_gain != nullptr) {
         const float2 s = block_sum2(s0, s1, part);
         s0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
         s1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
@@ -154,18 +155,23 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
     for (int j = 0; j < MAXV; ++j) {
         const int i = threadIdx.x + j * blockDim.x;
         if (i >= n4) continue;
-        float4 g0 = make_float4(1.f, 1.f, 1.f, 1.f), g1 = g0, v = x[j];
-        if (a.y_gain) {
-            g0 = *reinterpret_cast<const float4 *>(a.y_gain + 4 * i);
-            g1 = *reinterpret_cast<const float4 *>(a.y_gain + a.d_p + 4 * i);
-            g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
-            g1.x *= s1; g1.y *= s1; g1.z *= s1; g1.w *= s1;
-        } else if (POST && a.post_gain) {
-            g0 = *reinterpret_cast<const float4 *>(a.post_gain + 4 * i);
-            g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
+        float4 v = x[j];
+        const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+        if constexpr (POST) {
+            const float4 g = a.post_gain ? *reinterpret_cast<const float4 *>(a.post_gain + 4 * i) : one;
+            const float r = a.post_gain ? s0 : 1.f;
+            v.x += y0[j].x * r * g.x; v.y += y0[j].y * r * g.y; v.z += y0[j].z * r * g.z; v.w += y0[j].w * r * g.w;
+        } else {
+            float4 g0 = one, g1 = one;
+            if (a.y_gain) {
+                g0 = *reinterpret_cast<const float4 *>(a.y_gain + 4 * i);
+                g1 = *reinterpret_cast<const float4 *>(a.y_gain + a.d_p + 4 * i);
+                g0.x *= s0; g0.y *= s0; g0.z *= s0; g0.w *= s0;
+                g1.x *= s1; g1.y *= s1; g1.z *= s1; g1.w *= s1;
+            }
+            v.x += y0[j].x * g0.x + y1[j].x * g1.x; v.y += y0[j].y * g0.y + y1[j].y * g1.y;
+            v.z += y0[j].z * g0.z + y1[j].z * g1.z; v.w += y0[j].w * g0.w + y1[j].w * g1.w;
         }
-        v.x += y0[j].x * g0.x + y1[j].x * g1.x; v.y += y0[j].y * g0.y + y1[j].y * g1.y;
-        v.z += y0[j].z * g0.z + y1[j].z * g1.z; v.w += y0[j].w * g0.w + y1[j].w * g1.w;
         if (a.embd) {
             const float4 e = ld4_bf16(a.embd, e0 + 4 * i);
             v.x += e.x * a.embd_scale; v.y += e.y * a.embd_scale; v.z += e.z * a.embd_scale; v.w += e.w * a.embd_scale;
@@ -196,16 +202,18 @@ __global__ void pre_norm_kernel(const PreNormArgs a) {
 template <class T, bool POST>
 static int pre_norm_t(const PreNormArgs &a, cudaStream_t s, bool pdl) {
     const int n4 = a.d_p / 4;
-    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1, POST>, dim3(a.n_tok), dim3(128), 0, s, pdl, a));
-    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2, POST>, dim3(a.n_tok), dim3(512), 0, s, pdl, a));
-    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4, POST>, dim3(a.n_tok), dim3(1024), 0, s, pdl, a));
+    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1, POST>, dim3(a.n_tok), dim3(pre_norm_threads(1)), 0, s, pdl, a));
+    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2, POST>, dim3(a.n_tok), dim3(pre_norm_threads(2)), 0, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4, POST>, dim3(a.n_tok), dim3(pre_norm_threads(4)), 0, s, pdl, a));
     return LCU_OK;
 }
 
 int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl) {
     if (a.n_tok <= 0) return LCU_OK;
     LCU_REQUIRE(a.d_p % 4 == 0 && a.d_p <= 16384, "pre_norm: width %d (a multiple of 4, at most 16384)", a.d_p);
-    if (a.post_gain || a.pair_embd || a.n_zero) return dt == LCU_F32 ? pre_norm_t<float, true>(a, s, pdl) : pre_norm_t<__nv_bfloat16, true>(a, s, pdl);
+    const bool post = a.post_gain || a.pair_embd || a.n_zero || a.top;
+    LCU_REQUIRE(!post || !a.y_gain, "pre_norm: outputs normed one by one and as a sum");
+    if (post) return dt == LCU_F32 ? pre_norm_t<float, true>(a, s, pdl) : pre_norm_t<__nv_bfloat16, true>(a, s, pdl);
     return dt == LCU_F32 ? pre_norm_t<float, false>(a, s, pdl) : pre_norm_t<__nv_bfloat16, false>(a, s, pdl);
 }
 
