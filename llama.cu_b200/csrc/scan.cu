@@ -538,7 +538,7 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanArgs a, const 
 // grid (parts, tokens).  V numbers at a time: 4 where neither a head nor a part ends inside four.
 constexpr int SO_STASH = 8192;  // gated numbers of a part kept in shared memory (longer parts are computed twice)
 template <class T, int V>
-__global__ void __launch_bounds__(256) ssd_out_kernel(const ScanArgs a) {
+__global__ void __launch_bounds__(1024) ssd_out_kernel(const ScanArgs a) {
     extern __shared__ __align__(16) float stash[];
     __shared__ float2 sums[32];
     grid_dep_launch();
@@ -553,7 +553,7 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(const ScanArgs a) {
         return make_float4(u.x * silu_f(w.x), u.y * silu_f(w.y), u.z * silu_f(w.z), u.w * silu_f(w.w));
     };
     float ss = 0.f;
-    for (int i = V * threadIdx.x; i < len; i += V * 256) {
+    for (int i = V * threadIdx.x; i < len; i += V * blockDim.x) {
         const int at = place(i);
         if constexpr (V == 4) {
             const float4 x = gated4(at);
@@ -566,7 +566,7 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(const ScanArgs a) {
         }
     }
     const float n = 1.f / sqrtf(block_sum2(ss, 0.f, sums).x / (float)len + a.eps);
-    for (int i = V * threadIdx.x; i < len; i += V * 256) {
+    for (int i = V * threadIdx.x; i < len; i += V * blockDim.x) {
         const int at = place(i);
         if constexpr (V == 4) {
             const float4 x = keep ? *reinterpret_cast<const float4 *>(stash + i) : gated4(at), w = *reinterpret_cast<const float4 *>(a.norm + at);
@@ -682,9 +682,12 @@ int scan_out_launch(const ScanArgs &a, int dt, cudaStream_t s, bool pdl) {
     const int len = a.heads * a.dv / a.parts;
     const bool four = a.dv % 4 == 0 && len % 4 == 0;
     const size_t smem = len <= SO_STASH ? (size_t)len * 4 : 0;
-    const dim3 grid(a.parts, a.n_tok);
-    if (dt == LCU_F32) LCU_CHECK_CUDA(launch_kernel(four ? ssd_out_kernel<float, 4> : ssd_out_kernel<float, 1>, grid, dim3(256), smem, s, pdl, a));
-    else LCU_CHECK_CUDA(launch_kernel(four ? ssd_out_kernel<bf16, 4> : ssd_out_kernel<bf16, 1>, grid, dim3(256), smem, s, pdl, a));
+    // eight numbers per thread where that takes little time, small blocks where there are many
+    const int want = (len / 8 + 31) / 32 * 32, most = (long)a.parts * a.n_tok > 8 * sm_count() ? (len > 2048 ? 256 : 128) : 1024;
+    const int threads = want < 128 ? 128 : want > most ? most : want;
+    const dim3 grid(a.parts, a.n_tok), block(threads);
+    if (dt == LCU_F32) LCU_CHECK_CUDA(launch_kernel(four ? ssd_out_kernel<float, 4> : ssd_out_kernel<float, 1>, grid, block, smem, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(four ? ssd_out_kernel<bf16, 4> : ssd_out_kernel<bf16, 1>, grid, block, smem, s, pdl, a));
     return LCU_OK;
 }
 
