@@ -210,8 +210,8 @@ LCU_API int lcu_ctx_create(const lcu_model_desc *desc, int device, int tp_rank, 
 LCU_API int lcu_ctx_destroy(lcu_ctx *ctx);
 /* A context for a model described layer by layer: desc gives n_layers, d, vocab, nctx, eps, act_dtype (LCU_BF16, or LCU_F32:
  * every operation in true 32-bit arithmetic), weight_dtype (LCU_BF16), page_tokens, max_tokens, max_seqs; its other fields are
- * ignored.  Pages hold page_tokens latents, or keys and values, of every layer; sequences of models with token shift or a delta
- * rule also take one of max_seqs recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
+ * ignored.  Pages hold page_tokens latents, or keys and values, of every layer; sequences of models with token shift, a
+ * recurrent mixer or an embedding of token pairs also take one of max_seqs recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
  * graphs, round builder, sampling).  One GPU.  (No counterpart in the reference.) */
 LCU_API int lcu_ctx_create_layers(const lcu_model_desc *desc, const lcu_layer_desc *layers, int device, lcu_ctx **out);
 /* Packed (zero-padded) shape of one weight of a layered context; layer is ignored for EMBD, OUT_NORM and LM_HEAD.
