@@ -92,7 +92,14 @@ typedef enum {
     LCU_W_ROUTER = 43,      /* experts: matrix of the router                            */
     LCU_W_SHARED_UP = 44,   /* shared expert; gated feed-forwards hold gate and up rows in turn */
     LCU_W_SHARED_DOWN = 45,
-    LCU_W_PAIR_EMBD = 46    /* embedding of token pairs, [buckets + 1, d]               */
+    LCU_W_PAIR_EMBD = 46,   /* embedding of token pairs, [buckets + 1, d]               */
+    LCU_W_ATT_CONV = 47,    /* short convolutions of the attention's q | k | v: [taps][channels] */
+    LCU_W_SINK = 48,        /* [heads]: scores of the softmax's sinks (sink 2)          */
+    LCU_W_HEAD_TEMP = 49,   /* [heads]: factors on the scores                           */
+    LCU_W_UP_BIAS = 50,     /* biases of the feed-forward (ff_bias)                     */
+    LCU_W_DOWN_BIAS = 51,
+    LCU_W_ACT = 52,         /* four numbers of LCU_ACT_POLYNORM                         */
+    LCU_W_CORRECTION = 53   /* experts: added to the scores that choose (route_softmax), identity experts included */
 } lcu_weight_kind;
 
 /* Model description: the fields llama.cu/src/model/mod.rs:61-78 reads from GGUF metadata.
@@ -119,7 +126,8 @@ enum {
 }; /* ATTENTION | a recurrent one: both read the same input, their outputs are added: RMS-normed with a gain each, or (post_norm)
     * with a factor each */
 enum { LCU_ACT_XIELU = 1, LCU_ACT_RELU2 = 2,
-       LCU_ACT_GLU = 3 }; /* g = min(W_gate x, limit), u = clamp(W_up x, +-limit): g sigmoid(alpha g) (u + shift) */
+       LCU_ACT_GLU = 3,       /* g = min(W_gate x, limit), u = clamp(W_up x, +-limit): g sigmoid(alpha g) (u + shift) */
+       LCU_ACT_POLYNORM = 4 };/* a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e, every rms over the token's whole vector */
 
 /* One layer of a model described layer by layer.  Post-norm: x += norm(mixer(h)), x += norm(ff(x)), both norms RMS with a
  * single gain on the sublayer's OUTPUT, h = x or (token_shift) x mixed per coordinate with the previous token's x.
@@ -155,7 +163,7 @@ typedef struct {
     /* ATTENTION (out_gate as above) */
     int32_t rot_adjacent;/* 1: pairs (2 i, 2 i + 1)                                              */
     int32_t window;      /* > 0: position i sees j with i - j < window                           */
-    int32_t sink;        /* 1: the softmax counts one more key of score 0 and without value      */
+    int32_t sink;        /* 1: the softmax counts one more key of score 0 and without value, 2: of score LCU_W_SINK[head] */
     int32_t kv_from;     /* 0: own keys and values; j + 1: those of layer j (a layer before, same key heads, head sizes and rotation) */
     /* SSD and GLA share the delta_ fields (heads; heads of q and k; key size; value size; taps of SSD) */
     int32_t norm_parts;  /* SSD: equal parts of the gated output that are normed                 */
@@ -172,6 +180,23 @@ typedef struct {
     int32_t pair_buckets; /* > 0: row (previous token * pair_prev + token * pair_cur) mod pair_buckets of LCU_W_PAIR_EMBD is added
                            * to a token's embedding, row pair_buckets to that of a sequence's first token */
     int32_t pair_prev, pair_cur; /* in [0, pair_buckets)                                         */
+    /* PRE-NORM */
+    int32_t parallel_ff; /* 1: x += mixer(norm1(x)) + ff(norm2(x)), both norms of the same x     */
+    /* ATTENTION */
+    int32_t conv;        /* > 0: taps of a causal convolution over time on every channel of q, k and v, right after the projection;
+                          * the last taps - 1 projected values are state of a sequence           */
+    int32_t head_temp;   /* 1: scores are multiplied by LCU_W_HEAD_TEMP[head] too                */
+    int32_t keep_first;  /* with a window: the first tokens of a sequence stay visible behind it */
+    int32_t rot_values;  /* 1: values are rotated by their positions (all pairs (2 i, 2 i + 1) of v_dim, frequencies
+                          * rot_base^(-2 i / v_dim)) and cached so, each head's output is rotated back by its token's position */
+    /* feed-forward */
+    int32_t ff_bias;     /* LCU_ACT_POLYNORM: 1: biases on both matrices                         */
+    int32_t route_softmax; /* experts: 0: sigmoids of the logits on the inputs; 1: the softmax over all logits: the largest
+                          * scores + LCU_W_CORRECTION choose, the chosen scores divided by their sum weigh the OUTPUTS */
+    int32_t identity;    /* route_softmax: so many more experts behind the others whose output is their input */
+    /* read from the first layer: logits = cap tanh(scale head x / cap) */
+    float logit_scale;   /* 0 = 1                                                                */
+    float logit_cap;     /* 0: none                                                              */
 } lcu_layer_desc;
 
 /* == `KVPair` (llama.cu/src/op/random_sample/mod.rs:29-36) == cub::KeyValuePair<int,half> */
@@ -211,7 +236,7 @@ LCU_API int lcu_ctx_destroy(lcu_ctx *ctx);
 /* A context for a model described layer by layer: desc gives n_layers, d, vocab, nctx, eps, act_dtype (LCU_BF16, or LCU_F32:
  * every operation in true 32-bit arithmetic), weight_dtype (LCU_BF16), page_tokens, max_tokens, max_seqs; its other fields are
  * ignored.  Pages hold page_tokens latents, or keys and values, of every layer; sequences of models with token shift, a
- * recurrent mixer or an embedding of token pairs also take one of max_seqs recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
+ * recurrent mixer, convolutions or an embedding of token pairs also take one of max_seqs recurrent-state slots from their first round until lcu_seq_free.  Everything below works on it unchanged (pages, rounds,
  * graphs, round builder, sampling).  One GPU.  (No counterpart in the reference.) */
 LCU_API int lcu_ctx_create_layers(const lcu_model_desc *desc, const lcu_layer_desc *layers, int device, lcu_ctx **out);
 /* Packed (zero-padded) shape of one weight of a layered context; layer is ignored for EMBD, OUT_NORM and LM_HEAD.

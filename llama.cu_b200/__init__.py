@@ -19,9 +19,10 @@ F16, BF16, F32, Q8_0, U32 = 0, 1, 2, 3, 4
 W_EMBD, W_ATTN_NORM, W_QKV, W_O, W_FFN_NORM, W_GATE_UP, W_DOWN, W_OUT_NORM, W_LM_HEAD = range(9)
 (W_LAT_IN, W_Q_NORM, W_KV_NORM, W_UQ, W_UKT, W_UKV, W_LAT_OUT, W_UP, W_FF_DOWN, W_SHIFT, W_SCALARS, W_MIX_IN, W_MIX_BIAS,
  W_ATT_OUT, W_DELTA_OUT, W_CONV, W_DELTA_DECAY, W_DELTA_NORM, W_BRANCH_NORM, W_NORM1, W_NORM2, W_STEP, W_POST1, W_POST2, W_QK_GAIN,
- W_CONV_BIAS, W_GATE_MAP, W_ROUTER, W_SHARED_UP, W_SHARED_DOWN, W_PAIR_EMBD) = range(16, 47)
+ W_CONV_BIAS, W_GATE_MAP, W_ROUTER, W_SHARED_UP, W_SHARED_DOWN, W_PAIR_EMBD, W_ATT_CONV, W_SINK, W_HEAD_TEMP, W_UP_BIAS, W_DOWN_BIAS, W_ACT,
+ W_CORRECTION) = range(16, 54)
 MIX_LATENT, MIX_ATTENTION, MIX_DELTA, MIX_SSD, MIX_GLA = 1, 2, 4, 8, 16
-ACT_XIELU, ACT_RELU2, ACT_GLU = 1, 2, 3
+ACT_XIELU, ACT_RELU2, ACT_GLU, ACT_POLYNORM = 1, 2, 3, 4
 LINEAR_KINDS = (W_QKV, W_O, W_GATE_UP, W_DOWN)
 NO_OUTPUT = 2**64 - 1  # LCU_ENGINE_NO_OUTPUT: a prefill chunk that samples nothing
 OK, ERR_INVALID, ERR_CUDA, ERR_OVERFLOW, ERR_NO_PAGES, ERR_STATE, ERR_COMM, ERR_TIMEOUT = 0, -1, -2, -3, -4, -5, -6, -7
@@ -49,7 +50,8 @@ class LayerDesc(C.Structure):
         (n, C.c_int32) for n in ("post_norm", "rot_adjacent", "window", "sink", "kv_from", "norm_parts", "gate_rank", "experts", "top",
                                  "shared_ff")] + [
         (n, C.c_float) for n in ("out_scale", "out_scale2", "gate_tau", "glu_limit", "shared_limit", "glu_alpha", "glu_shift", "embed_scale")] + [
-        (n, C.c_int32) for n in ("pair_buckets", "pair_prev", "pair_cur")]
+        (n, C.c_int32) for n in ("pair_buckets", "pair_prev", "pair_cur", "parallel_ff", "conv", "head_temp", "keep_first", "rot_values",
+                                 "ff_bias", "route_softmax", "identity")] + [(n, C.c_float) for n in ("logit_scale", "logit_cap")]
 
 
 class KVPair(C.Structure):

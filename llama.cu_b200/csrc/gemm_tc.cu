@@ -106,7 +106,10 @@ __device__ __forceinline__ void tc_finish(const GemvArgs &a, int n, int first, f
             dst = reinterpret_cast<T *>(a.kv_pool) + a.geom.block_off(pre.page, a.layer, sect - 1, head) + (size_t)slot * a.dh + e;
         }
     }
-    if (a.epilogue == EPI_STORE_F32) {
+    if (a.epilogue >= EPI_CAP)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = cap_logit(v[i], a.cap);
+    if (a.epilogue == EPI_STORE_F32 || a.epilogue == EPI_CAP_F32) {
         float4 *f = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.y) + (size_t)n * a.stride_y + first);
         f[0] = make_float4(v[0], v[1], v[2], v[3]);
         f[1] = make_float4(v[4], v[5], v[6], v[7]);

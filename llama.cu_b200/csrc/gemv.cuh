@@ -13,10 +13,14 @@ enum GemvEpilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_ROPE_KV = 2, EPI_SWIGLU
                     EPI_STORE_F32 = 4,  // y is f32
                     EPI_XIELU = 5,      // y = xielu(row) with the two numbers at act_pq
                     EPI_RELU2 = 6,      // y = max(row, 0)^2
-                    EPI_GLU = 7 };      // rows are gate and up in turn: y[n, out / 2] of glu
+                    EPI_GLU = 7,        // rows are gate and up in turn: y[n, out / 2] of glu
+                    EPI_CAP = 8,        // y = cap of head
+                    EPI_CAP_F32 = 9 };  // the same as f32
 
 // Gated activation: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(alpha g) (u + shift).
 struct GluArgs { float limit, alpha, shift; };
+// Logits: cap tanh(scale v / cap), cap 0: scale v.
+struct CapArgs { float scale, cap; };
 
 // Inputs of the prologues of layered models, for rounds of one token per request (token t is request t).  Every CTA computes
 // the rows it multiplies; what later kernels need (new residual, shift state, cached latent) is written by the first CTA.
@@ -72,6 +76,7 @@ struct GemvArgs {
     int pt_stride;
     const float *act_pq;  // EPI_XIELU: p, q
     GluArgs glu;          // EPI_GLU
+    CapArgs cap;          // EPI_CAP, EPI_CAP_F32
     // grouped products (gemm_tc.cu): row t.y .. t.y + t.z of x and y meet matrix t.x of `groups` ones of `out` rows; a factor per row
     const int4 *tiles;
     int n_tiles, tile_rows, groups;
@@ -104,6 +109,7 @@ __device__ __forceinline__ float glu_act(float gate, float up, const GluArgs &a)
     const float g = fminf(gate, a.limit), u = fminf(fmaxf(up, -a.limit), a.limit);
     return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
 }
+__device__ __forceinline__ float cap_logit(float v, const CapArgs &a) { return a.cap > 0.f ? a.cap * tanhf(v * a.scale / a.cap) : v * a.scale; }
 
 // Values an epilogue would otherwise fetch from global memory behind the weight stream: the per-token constants of the
 // RoPE / KV-append epilogue (position, cache page, sin and cos rows; head sizes up to 128), staged in shared memory
@@ -207,6 +213,10 @@ __device__ __forceinline__ void stack_epilogue(const GemvArgs &a, int pair, int 
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(relu2_act(va), relu2_act(vb));
     } else if (a.epilogue == EPI_GLU) {
         reinterpret_cast<T *>(a.y)[(size_t)t * a.stride_y + pair] = Act<T>::from_f(glu_act(va, vb, a.glu));
+    } else if (a.epilogue == EPI_CAP) {
+        *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(cap_logit(va, a.cap), cap_logit(vb, a.cap));
+    } else if (a.epilogue == EPI_CAP_F32) {
+        *reinterpret_cast<float2 *>(reinterpret_cast<float *>(a.y) + off) = make_float2(cap_logit(va, a.cap), cap_logit(vb, a.cap));
     } else {
         const float sp = softplus_f(__ldg(a.act_pq)), sq = softplus_f(__ldg(a.act_pq + 1));
         *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(a.y) + off) = Act<T>::pack(xielu_act(va, sp, sq), xielu_act(vb, sp, sq));

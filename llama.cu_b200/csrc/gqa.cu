@@ -5,7 +5,8 @@
 //               of a tensor-core tile; every warp walks its own blocks of 16 cached rows with a copy ring and running softmax of
 //               its own (no barrier in the loop); contexts are cut into splits, the last CTA of a row tile to arrive merges;
 //   long form   64 (token, head) rows per CTA share tiles of 64 cached rows.
-// Options: a sliding window (tiles that no row sees are skipped), a sink in the softmax's denominator, a gate per head.
+// Options: a sliding window, with or without the first tokens of a sequence (tiles that no row sees are skipped), a sink in the
+// softmax's denominator, a gate per head, outputs rotated back where the cached values are rotated.
 //
 // Arithmetic: scores, softmax and its running state in f32; probabilities are rounded to bf16 only as operands of the second
 // product, the row sum is taken over the rounded values; all sums accumulate in f32.  All-32-bit contexts use f32 FMA throughout.
@@ -41,28 +42,59 @@ __device__ __forceinline__ float quad_sum(float v) {
     return v + __shfl_xor_sync(0xffffffffu, v, 2);
 }
 
-template <class T, bool WIDE>
-__global__ void __launch_bounds__(256, WIDE ? 5 : 6) gqa_prep_kernel(const GqaArgs a) {
+template <class T, int FORM>
+__global__ void __launch_bounds__(256, FORM == GQA_PREP ? 6 : (FORM == GQA_PREP_CONV ? 4 : 5)) gqa_prep_kernel(const GqaArgs a) {
     grid_dep_launch();
-    const int per = WIDE ? (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x : 8;
+    const int per = FORM >= GQA_PREP_WIDE ? (gqa_prep_items(a) + (int)gridDim.x - 1) / (int)gridDim.x : 8;
     grid_dep_wait();
-    gqa_prep_block<T, WIDE>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
+    gqa_prep_block<T, FORM>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
 }
 
-// Denominator and factor that end a row of softmax (scores in powers of two): maximum M, sum L over it.  A key of score 0 may
-// count in the denominator; the head's gate multiplies the output.
+// Denominator and factor that end a row of softmax (scores in powers of two): maximum M, sum L over it.  A key without
+// value may count in the denominator; the head's gate multiplies the output.
 __device__ __forceinline__ float softmax_end(const GqaArgs &a, float M, float L, int tok, int head) {
     float f = 1.f;
     if (a.sink) {
-        const float top = fmaxf(M, 0.f);
+        const float z = a.sink_score ? a.sink_score[head] * 1.4426950408889634f : 0.f, top = fmaxf(M, z);
         f = exp2f(M - top);
-        L = fmaf(L, f, exp2f(-top));
+        L = fmaf(L, f, exp2f(z - top));
     }
     if (a.gate) f /= 1.f + expf(-a.gate[(size_t)tok * a.stride + head]);
     return f / L;
 }
 // first position that position p sees
 __device__ __forceinline__ int first_seen(const GqaArgs &a, int p) { return a.window > 0 && p >= a.window ? p - a.window + 1 : 0; }
+// Tiles of `size` positions, from the one at position `lo` up to `ctx`, those of the kept first tokens ahead of them: number of
+// both, and a tile's number in the sequence.
+struct SeenTiles {
+    int kept, jump, n;
+    __device__ __forceinline__ SeenTiles(const GqaArgs &a, int lo, int ctx, int size) {
+        const int tile0 = lo / size;
+        kept = min((a.keep + size - 1) / size, tile0);
+        jump = tile0 - kept;
+        n = (ctx + size - 1) / size - jump;
+    }
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : i + jump; }
+};
+// Positions [keep, keep + gap) are those up to p's first seen one that p does not see.
+__device__ __forceinline__ int gap_of(const GqaArgs &a, int p) { return max(first_seen(a, p) - a.keep, 0); }
+__device__ __forceinline__ bool seen(int pos, int lim, int keep, int gap) { return pos <= lim && (unsigned)(pos - keep) >= (unsigned)gap; }
+// Columns d and d + 1 of an output, rotated back by position p.
+__device__ __forceinline__ float2 turn_back(const GqaArgs &a, int p, int d, float x, float y) {
+    if (d >= a.v_dim) return make_float2(x, y);
+    const float2 c = a.vrot[(size_t)p * (a.v_dim >> 1) + (d >> 1)];
+    return make_float2(x * c.x + y * c.y, y * c.x - x * c.y);
+}
+// Eight columns from d on of a row's output, rounded; p: position of its token.
+__device__ __forceinline__ uint4 end_of_row(const GqaArgs &a, const float x[8], float f, int p, int d) {
+    float2 v[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[i] = make_float2(x[2 * i] * f, x[2 * i + 1] * f);
+        if (a.vrot) v[i] = turn_back(a, p, d + 2 * i, v[i].x, v[i].y);
+    }
+    return make_uint4(Act<bf16>::pack(v[0].x, v[0].y), Act<bf16>::pack(v[1].x, v[1].y), Act<bf16>::pack(v[2].x, v[2].y), Act<bf16>::pack(v[3].x, v[3].y));
+}
 
 // ------------------------------------------------------------------ short form
 constexpr int GS_WARPS = 4, GS_KEYS = 16, GS_STAGES = 3;
@@ -86,11 +118,12 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
     const int kvh = blockIdx.x % a.kv_heads, row0 = blockIdx.x / a.kv_heads * 16;
     const int4 rq = a.reqs[blockIdx.y];  // request, first token, tokens, position
     const int rows = rq.z * g, sp = blockIdx.z;
-    const int ctx = rq.w + rq.z, unit0 = first_seen(a, rq.w) / GS_UNIT, units = (ctx + GS_UNIT - 1) / GS_UNIT - unit0;
-    const int ups = (units + a.splits - 1) / a.splits, n_split = (units + ups - 1) / ups;
+    const int ctx = rq.w + rq.z;
+    const SeenTiles tiles(a, first_seen(a, rq.w), ctx, GS_UNIT);
+    const int ups = (tiles.n + a.splits - 1) / a.splits, n_split = (tiles.n + ups - 1) / ups;
     grid_dep_launch();
     if (row0 >= rows || sp >= n_split) return;
-    const int u0 = unit0 + sp * ups, u1 = min(unit0 + units, u0 + ups);
+    const int u0 = sp * ups, u1 = min(tiles.n, u0 + ups);
     const bf16 *pool = reinterpret_cast<const bf16 *>(a.pool);
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)rq.x * a.pt_stride;
@@ -99,7 +132,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
 
     auto load = [&](int u, int stage) {
         bf16 *kd = ring + stage * STAGE, *vd = kd + GS_KEYS * KROW;
-        const int key0 = u * GS_UNIT + warp * GS_KEYS;
+        const int key0 = tiles.at(u) * GS_UNIT + warp * GS_KEYS;
         constexpr int KL = DQ / 8, VL = DV / 8;  // lanes per row (columns past the head's size stay idle)
 #pragma unroll
         for (int i = 0; i < GS_KEYS * KL / 32; ++i) {
@@ -128,7 +161,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
     const bool v0 = r0 < rows, v1 = r1 < rows;
     const int tk0 = v0 ? r0 / g : 0, tk1 = v1 ? r1 / g : 0;
     const int lim0 = v0 ? rq.w + tk0 : -1, lim1 = v1 ? rq.w + tk1 : -1;
-    const int lo0 = first_seen(a, lim0), lo1 = first_seen(a, lim1);
+    const int gap0 = gap_of(a, lim0), gap1 = gap_of(a, lim1);
     uint32_t qa[KS][4];
     {
         const bf16 *q = reinterpret_cast<const bf16 *>(a.q);
@@ -167,11 +200,11 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
         float t0 = -INFINITY, t1 = -INFINITY;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-            const int p = u * GS_UNIT + warp * GS_KEYS + nt * 8 + 2 * t4;
-            sc[nt][0] = p <= lim0 && p >= lo0 ? sc[nt][0] * scale2 : -INFINITY;
-            sc[nt][1] = p + 1 <= lim0 && p + 1 >= lo0 ? sc[nt][1] * scale2 : -INFINITY;
-            sc[nt][2] = p <= lim1 && p >= lo1 ? sc[nt][2] * scale2 : -INFINITY;
-            sc[nt][3] = p + 1 <= lim1 && p + 1 >= lo1 ? sc[nt][3] * scale2 : -INFINITY;
+            const int p = tiles.at(u) * GS_UNIT + warp * GS_KEYS + nt * 8 + 2 * t4;
+            sc[nt][0] = seen(p, lim0, a.keep, gap0) ? sc[nt][0] * scale2 : -INFINITY;
+            sc[nt][1] = seen(p + 1, lim0, a.keep, gap0) ? sc[nt][1] * scale2 : -INFINITY;
+            sc[nt][2] = seen(p, lim1, a.keep, gap1) ? sc[nt][2] * scale2 : -INFINITY;
+            sc[nt][3] = seen(p + 1, lim1, a.keep, gap1) ? sc[nt][3] * scale2 : -INFINITY;
             t0 = fmaxf(t0, fmaxf(sc[nt][0], sc[nt][1]));
             t1 = fmaxf(t1, fmaxf(sc[nt][2], sc[nt][3]));
         }
@@ -245,10 +278,8 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
         if (n_split == 1) {
             const int row = row0 + r;
             const float inv = softmax_end(a, M, L, rq.y + row / g, kvh * g + row % g);
-            uint4 u;
-            u.x = Act<bf16>::pack(x[0] * inv, x[1] * inv); u.y = Act<bf16>::pack(x[2] * inv, x[3] * inv);
-            u.z = Act<bf16>::pack(x[4] * inv, x[5] * inv); u.w = Act<bf16>::pack(x[6] * inv, x[7] * inv);
-            *reinterpret_cast<uint4 *>(out + (size_t)(rq.y + row / g) * a.stride_o + (size_t)(kvh * g + row % g) * a.vdim_p + c) = u;
+            *reinterpret_cast<uint4 *>(out + (size_t)(rq.y + row / g) * a.stride_o + (size_t)(kvh * g + row % g) * a.vdim_p + c) =
+                end_of_row(a, x, inv, rq.w + row / g, c);
         } else {
             float *dst = a.part_o + ((cell * a.splits + sp) * 16 + r) * a.vdim_p + c;
             *reinterpret_cast<float4 *>(dst) = make_float4(x[0], x[1], x[2], x[3]);
@@ -278,10 +309,8 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gqa_short_kernel(const GqaArgs 
         }
         const int row = row0 + r;
         const float inv = softmax_end(a, M, L, rq.y + row / g, kvh * g + row % g);
-        uint4 u;
-        u.x = Act<bf16>::pack(x[0] * inv, x[1] * inv); u.y = Act<bf16>::pack(x[2] * inv, x[3] * inv);
-        u.z = Act<bf16>::pack(x[4] * inv, x[5] * inv); u.w = Act<bf16>::pack(x[6] * inv, x[7] * inv);
-        *reinterpret_cast<uint4 *>(out + (size_t)(rq.y + row / g) * a.stride_o + (size_t)(kvh * g + row % g) * a.vdim_p + c) = u;
+        *reinterpret_cast<uint4 *>(out + (size_t)(rq.y + row / g) * a.stride_o + (size_t)(kvh * g + row % g) * a.vdim_p + c) =
+            end_of_row(a, x, inv, rq.w + row / g, c);
     }
     if (tid == 0) a.tickets[cell] = 0;  // ready for the next launch
 }
@@ -320,7 +349,8 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
     const int4 rq = a.reqs[ri];
     const int rows = rq.z * g, row0 = blk * 64;
     const int last_tok = min(rq.z - 1, (row0 + 63) / g);
-    const int ctx = rq.w + last_tok + 1, n_tiles = (ctx + GL_TILE - 1) / GL_TILE, tile0 = first_seen(a, rq.w + row0 / g) / GL_TILE;
+    const int ctx = rq.w + last_tok + 1;
+    const SeenTiles tiles(a, first_seen(a, rq.w + row0 / g), ctx, GL_TILE);
     const bf16 *pool = reinterpret_cast<const bf16 *>(a.pool);
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)rq.x * a.pt_stride;
@@ -350,7 +380,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
     const bool v0 = r0 < rows, v1 = r1 < rows;
     const int tk0 = v0 ? r0 / g : 0, tk1 = v1 ? r1 / g : 0;
     const int lim0 = v0 ? rq.w + tk0 : -1, lim1 = v1 ? rq.w + tk1 : -1;
-    const int lo0 = first_seen(a, lim0), lo1 = first_seen(a, lim1);
+    const int gap0 = gap_of(a, lim0), gap1 = gap_of(a, lim1);
     const int h0 = kvh * g + (v0 ? r0 % g : 0), h1 = kvh * g + (v1 ? r1 % g : 0);
     uint32_t qa[KS][4];
     {
@@ -365,7 +395,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
             qa[ks][3] = in && v1 ? *reinterpret_cast<const uint32_t *>(q1 + ks * 16 + 8) : 0u;
         }
     }
-    load_tile(tile0, 0);
+    load_tile(tiles.at(0), 0);
     ga_commit();
     const float scale2 = a.scale * 1.4426950408889634f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
@@ -373,9 +403,9 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
 #pragma unroll
     for (int i = 0; i < NTO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
 
-    for (int tile = tile0; tile < n_tiles; ++tile) {
-        const int buf = (tile - tile0) & 1;
-        if (tile + 1 < n_tiles) load_tile(tile + 1, buf ^ 1);
+    for (int i = 0; i < tiles.n; ++i) {
+        const int buf = i & 1, tile = tiles.at(i);
+        if (i + 1 < tiles.n) load_tile(tiles.at(i + 1), buf ^ 1);
         ga_commit();
         ga_wait<1>();
         __syncthreads();
@@ -396,7 +426,7 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
             }
         }
         float t0 = -INFINITY, t1 = -INFINITY;
-        if (tile * GL_TILE + GL_TILE - 1 <= min(lim0, lim1) && tile * GL_TILE >= max(lo0, lo1)) {  // every position visible
+        if (tile * GL_TILE + GL_TILE - 1 <= min(lim0, lim1) && (tile * GL_TILE >= a.keep + max(gap0, gap1) || tile * GL_TILE + GL_TILE <= a.keep)) {  // every position visible
 #pragma unroll
             for (int nt = 0; nt < NTS; ++nt) {
 #pragma unroll
@@ -408,10 +438,10 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
 #pragma unroll
             for (int nt = 0; nt < NTS; ++nt) {
                 const int p = tile * GL_TILE + nt * 8 + 2 * t4;
-                sc[nt][0] = p <= lim0 && p >= lo0 ? sc[nt][0] * scale2 : -INFINITY;
-                sc[nt][1] = p + 1 <= lim0 && p + 1 >= lo0 ? sc[nt][1] * scale2 : -INFINITY;
-                sc[nt][2] = p <= lim1 && p >= lo1 ? sc[nt][2] * scale2 : -INFINITY;
-                sc[nt][3] = p + 1 <= lim1 && p + 1 >= lo1 ? sc[nt][3] * scale2 : -INFINITY;
+                sc[nt][0] = seen(p, lim0, a.keep, gap0) ? sc[nt][0] * scale2 : -INFINITY;
+                sc[nt][1] = seen(p + 1, lim0, a.keep, gap0) ? sc[nt][1] * scale2 : -INFINITY;
+                sc[nt][2] = seen(p, lim1, a.keep, gap1) ? sc[nt][2] * scale2 : -INFINITY;
+                sc[nt][3] = seen(p + 1, lim1, a.keep, gap1) ? sc[nt][3] * scale2 : -INFINITY;
                 t0 = fmaxf(t0, fmaxf(sc[nt][0], sc[nt][1]));
                 t1 = fmaxf(t1, fmaxf(sc[nt][2], sc[nt][3]));
             }
@@ -463,8 +493,12 @@ __global__ void __launch_bounds__(128) gqa_long_kernel(const GqaArgs a) {
         const float inv = softmax_end(a, hf ? m1 : m0, hf ? l1 : l0, rq.y + (hf ? tk1 : tk0), hf ? h1 : h0);
         bf16 *dst = out + (size_t)(rq.y + (hf ? tk1 : tk0)) * a.stride_o + (size_t)(hf ? h1 : h0) * a.vdim_p + 2 * t4;
 #pragma unroll
-        for (int i = 0; i < NTO; ++i)
-            if (i * 8 < a.vdim_p) *reinterpret_cast<uint32_t *>(dst + 8 * i) = Act<bf16>::pack(o[i][2 * hf] * inv, o[i][2 * hf + 1] * inv);
+        for (int i = 0; i < NTO; ++i) {
+            if (i * 8 >= a.vdim_p) continue;
+            float2 v = make_float2(o[i][2 * hf] * inv, o[i][2 * hf + 1] * inv);
+            if (a.vrot) v = turn_back(a, hf ? lim1 : lim0, 8 * i + 2 * t4, v.x, v.y);
+            *reinterpret_cast<uint32_t *>(dst + 8 * i) = Act<bf16>::pack(v.x, v.y);
+        }
     }
 }
 
@@ -483,9 +517,10 @@ __global__ void __launch_bounds__(256) gqa_f32_kernel(const GqaArgs a) {
     const size_t koff = a.c_off + ((size_t)kvh << a.page_shift) * a.dim_p, voff = a.v_off() + ((size_t)kvh << a.page_shift) * a.vdim_p;
     const int32_t *pages = a.page_table + (size_t)a.tok_req[t] * a.pt_stride;
     float m = -INFINITY, l = 0.f, acc[MIX_MAX_HEAD / 32] = {};
-    for (int k0 = first_seen(a, ctx - 1); k0 < ctx; k0 += 32) {
-        const int key = k0 + lane;
-        const bool ok = key < ctx;
+    const int lo = first_seen(a, ctx - 1), kept = min(a.keep, lo);
+    for (int k0 = kept > 0 ? 0 : lo; k0 < ctx; k0 = k0 < lo && k0 + 32 >= kept ? lo : k0 + 32) {
+        const int key = k0 + lane, end = k0 < lo ? kept : ctx;
+        const bool ok = key < end;
         const int slot = key & ((1 << a.page_shift) - 1);
         const size_t base = ok ? (size_t)pages[key >> a.page_shift] * a.page_elems : 0;
         float s = -INFINITY;
@@ -506,7 +541,7 @@ __global__ void __launch_bounds__(256) gqa_f32_kernel(const GqaArgs a) {
 #pragma unroll
         for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) acc[j] *= c;
         const size_t vrow = base + voff + (size_t)slot * a.vdim_p;
-        for (int i = 0; i < 32 && k0 + i < ctx; ++i) {
+        for (int i = 0; i < 32 && k0 + i < end; ++i) {
             const float pi = __shfl_sync(0xffffffffu, p, i);
             const float *vr = pool + __shfl_sync(0xffffffffu, (unsigned long long)vrow, i);
 #pragma unroll
@@ -517,8 +552,15 @@ __global__ void __launch_bounds__(256) gqa_f32_kernel(const GqaArgs a) {
     const float inv = softmax_end(a, m * 1.4426950408889634f, l, t, h);
     float *out = reinterpret_cast<float *>(a.o) + (size_t)t * a.stride_o + (size_t)h * a.vdim_p;
 #pragma unroll
-    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j)
-        if (lane + 32 * j < a.vdim_p) out[lane + 32 * j] = acc[j] * inv;
+    for (int j = 0; j < MIX_MAX_HEAD / 32; ++j) {
+        float v = acc[j] * inv;
+        if (a.vrot) {  // the other one of a pair is in the neighbouring lane
+            const float w = __shfl_xor_sync(0xffffffffu, v, 1);
+            const float2 x = turn_back(a, ctx - 1, (lane & ~1) + 32 * j, lane & 1 ? w : v, lane & 1 ? v : w);
+            v = lane & 1 ? x.y : x.x;
+        }
+        if (lane + 32 * j < a.vdim_p) out[lane + 32 * j] = v;
+    }
 }
 
 template <class K>
@@ -575,8 +617,11 @@ int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl) {
         LCU_CHECK_CUDA(launch_kernel(kernel, grid, dim3(256), 0, s, pdl, a));
         return LCU_OK;
     };
-    if (dt == LCU_F32) return gqa_prep_wide(a) ? go(gqa_prep_kernel<float, true>) : go(gqa_prep_kernel<float, false>);
-    return gqa_prep_wide(a) ? go(gqa_prep_kernel<bf16, true>) : go(gqa_prep_kernel<bf16, false>);
+    const bool f32 = dt == LCU_F32;
+    if (a.conv) return f32 ? go(gqa_prep_kernel<float, GQA_PREP_CONV>) : go(gqa_prep_kernel<bf16, GQA_PREP_CONV>);
+    if (gqa_prep_more(a)) return f32 ? go(gqa_prep_kernel<float, GQA_PREP_TURN>) : go(gqa_prep_kernel<bf16, GQA_PREP_TURN>);
+    if (gqa_prep_wide(a)) return f32 ? go(gqa_prep_kernel<float, GQA_PREP_WIDE>) : go(gqa_prep_kernel<bf16, GQA_PREP_WIDE>);
+    return f32 ? go(gqa_prep_kernel<float, GQA_PREP>) : go(gqa_prep_kernel<bf16, GQA_PREP>);
 }
 
 int gqa_short_tokens(int heads, int kv_heads) {

@@ -1,6 +1,7 @@
-// The step between the fused input projection and softmax attention, one warp per (token, head): bias, norm, rotation; the
-// query to its buffer, key and value to the cache.  Shared by the kernels of gqa.cu and the decode kernels of the recurrent mixers.
+// The step between the fused input projection and softmax attention, one warp per (token, head): bias or convolution over time,
+// norm, rotation; the query to its buffer, key and value to the cache.  Shared by the kernels of gqa.cu and the decode kernels of the recurrent mixers.
 #pragma once
+#include "conv.cuh"
 #include "stack.cuh"
 
 namespace lcu {
@@ -9,10 +10,14 @@ __host__ __device__ __forceinline__ int gqa_prep_items(const GqaArgs &a) { retur
 
 // Steps that only some designs have, kept out of the kernels of the others: norms with weights ahead of the rotation, neighbouring pairs.
 __host__ __device__ __forceinline__ bool gqa_prep_wide(const GqaArgs &a) { return a.qk_norm > 1 || a.rot_adjacent; }
+// ... and only layers without a recurrent mixer: rotated values, factors per head; convolutions.
+enum GqaPrepForm { GQA_PREP = 0, GQA_PREP_WIDE = 1, GQA_PREP_TURN = 2, GQA_PREP_CONV = 3 };
+__host__ __device__ __forceinline__ bool gqa_prep_more(const GqaArgs &a) { return a.vrot || a.head_temp || a.conv; }
 
 // row_norm: what qk_norm 3 divides all of q and all of k by (as factors)
-template <class T, bool WIDE>
+template <class T, int FORM>
 __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item, int lane, const float2 &row_norm) {
+    constexpr bool WIDE = FORM >= GQA_PREP_WIDE, TURN = FORM >= GQA_PREP_TURN, CONV = FORM == GQA_PREP_CONV;
     const bool is_v = item >= a.heads + a.kv_heads, is_q = item < a.heads;
     const int size_p = is_v ? a.vdim_p : a.dim_p;
     const int head = is_q ? item : (is_v ? item - a.heads - a.kv_heads : item - a.heads);
@@ -30,13 +35,42 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     const float2 *rot = a.rot + (size_t)p * half;
     // A norm ahead of the rotation: its weights go in here, its one factor at the end (the rotation is linear).
     const float *gain = WIDE && !is_v && a.qk_norm > 1 ? a.qk_gain + (a.qk_norm == 3 ? off : (is_q ? 0 : a.dim_p)) : nullptr;
+    [[maybe_unused]] ConvIn in_time;
+    [[maybe_unused]] float *state_out = nullptr;
+    if constexpr (CONV) {
+        const int r = a.tok_req[t], sg = a.req_slot[r];
+        const size_t row = (size_t)(sg >> 1) * (a.taps - 1) * a.channels();
+        in_time.row = a.lat + (size_t)t * a.stride;
+        in_time.stride = a.stride; in_time.channels = a.channels(); in_time.taps = a.taps;
+        in_time.in_portion = t - a.req_first[r];
+        in_time.seen = (int)p;
+        in_time.state = a.conv_state + (size_t)(sg & 1) * a.conv_gen_stride + row;
+        if (t + 1 == a.req_first[r + 1]) state_out = a.conv_state + (size_t)((sg & 1) ^ 1) * a.conv_gen_stride + row;
+    }
     auto raw4 = [&](int d) {
+        if constexpr (CONV) {
+            float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int j = 0; j < a.taps; ++j) {
+                const float4 x = in_time.at4(a.taps - 1 - j, off + d), w = *reinterpret_cast<const float4 *>(a.conv + (size_t)j * in_time.channels + off + d);
+                y.x = fmaf(x.x, w.x, y.x); y.y = fmaf(x.y, w.y, y.y); y.z = fmaf(x.z, w.z, y.z); y.w = fmaf(x.w, w.w, y.w);
+            }
+            return y;
+        }
         float4 x = *reinterpret_cast<const float4 *>(src + d);
         if (bias) {
             const float4 y = *reinterpret_cast<const float4 *>(bias + d);
             x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
         }
         return x;
+    };
+    auto raw1 = [&](int d) {
+        if constexpr (CONV) {
+            float y = 0.f;
+            for (int j = 0; j < a.taps; ++j) y = fmaf(in_time.at(a.taps - 1 - j, off + d), a.conv[(size_t)j * in_time.channels + off + d], y);
+            return y;
+        }
+        return src[d] + (bias ? bias[d] : 0.f);
     };
     auto weigh4 = [&](float4 x, int d) {
         if (WIDE && gain) {
@@ -72,11 +106,16 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
                     const int i = d + k;
                     if (i >= a.rot_dims) continue;
                     const int e = i < half ? i + half : i - half;
-                    const float y = (src[e] + (bias ? bias[e] : 0.f)) * (WIDE && gain ? gain[e] : 1.f);
+                    const float y = raw1(e) * (WIDE && gain ? gain[e] : 1.f);
                     const float2 cs = rot[i < half ? i : e];
                     xs[k] = i < half ? xs[k] * cs.x - y * cs.y : xs[k] * cs.x + y * cs.y;
                 }
             }
+        }
+        if (TURN && is_v && a.vrot && d < a.v_dim) {  // two pairs
+            const float2 *vr = a.vrot + (size_t)p * (a.v_dim >> 1) + (d >> 1);
+            const float2 c0 = vr[0], c1 = d + 2 < a.v_dim ? vr[1] : make_float2(1.f, 0.f);
+            x = make_float4(x.x * c0.x - x.y * c0.y, x.y * c0.x + x.x * c0.y, x.z * c1.x - x.w * c1.y, x.w * c1.x + x.z * c1.y);
         }
         v[j] = x;
         ss += dot4(WIDE && a.qk_norm == 2 ? in : x);
@@ -84,16 +123,22 @@ __device__ __forceinline__ void gqa_prep_item(const GqaArgs &a, int t, int item,
     float r = 1.f;
     if (!is_v && (a.qk_norm == 1 || (WIDE && a.qk_norm == 2))) r = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
     if (WIDE && !is_v && a.qk_norm == 3) r = is_q ? row_norm.x : row_norm.y;
+    if (TURN && is_q && a.head_temp) r *= a.head_temp[head];
 #pragma unroll
     for (int j = 0; j < MIX_MAX_HEAD / 128; ++j) {
         const int d = 4 * lane + 128 * j;
         if (d < size_p) st4<T>(dst + d, make_float4(v[j].x * r, v[j].y * r, v[j].z * r, v[j].w * r));
+        if constexpr (CONV) {
+            if (state_out && d < size_p)
+                for (int i = 1; i < a.taps; ++i) *reinterpret_cast<float4 *>(state_out + (size_t)(i - 1) * in_time.channels + off + d) = in_time.at4(a.taps - 1 - i, off + d);
+        }
     }
 }
 
 // Items [item0, item1) of token t by one block (at most one per warp unless WIDE); every thread of the block calls it.
-template <class T, bool WIDE>
+template <class T, int FORM>
 __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item0, int item1) {
+    constexpr bool WIDE = FORM >= GQA_PREP_WIDE;
     float2 norm = make_float2(1.f, 1.f);
     if (WIDE && a.qk_norm == 3) {
         __shared__ float2 part[32];
@@ -117,16 +162,16 @@ __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item
     int item = item0 + (int)(threadIdx.x >> 5);
     if constexpr (WIDE) {
 #pragma unroll 1
-        for (; item < item1; item += (int)(blockDim.x >> 5)) gqa_prep_item<T, true>(a, t, item, threadIdx.x & 31, norm);
+        for (; item < item1; item += (int)(blockDim.x >> 5)) gqa_prep_item<T, FORM>(a, t, item, threadIdx.x & 31, norm);
     } else {
-        if (item < item1) gqa_prep_item<T, false>(a, t, item, threadIdx.x & 31, norm);
+        if (item < item1) gqa_prep_item<T, FORM>(a, t, item, threadIdx.x & 31, norm);
     }
 }
 
 template <class T>
 __device__ __forceinline__ void gqa_prep_any(const GqaArgs &a, int t, int item0, int item1) {
-    if (gqa_prep_wide(a)) gqa_prep_block<T, true>(a, t, item0, item1);
-    else gqa_prep_block<T, false>(a, t, item0, item1);
+    if (gqa_prep_wide(a)) gqa_prep_block<T, GQA_PREP_WIDE>(a, t, item0, item1);
+    else gqa_prep_block<T, GQA_PREP>(a, t, item0, item1);
 }
 
 }  // namespace lcu

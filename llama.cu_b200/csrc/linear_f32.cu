@@ -64,6 +64,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Args a) 
             float v = acc[i][j];
             if (a.epilogue == EPI_XIELU) v = xielu_act(v, softplus_f(a.act_pq[0]), softplus_f(a.act_pq[1]));
             else if (a.epilogue == EPI_RELU2) v = relu2_act(v);
+            else if (a.epilogue == EPI_CAP_F32) v = cap_logit(v, a.cap);
             a.y[yr * a.stride_y + (a.tiles ? 0 : (size_t)head * a.head_y) + o] = a.gate ? v * g : v;
         }
     }
@@ -71,7 +72,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Args a) 
 
 int linear_f32_launch(const LinearF32Args &a, cudaStream_t s) {
     if (a.n <= 0) return LCU_OK;
-    LCU_REQUIRE(a.epilogue == EPI_STORE_F32 || a.epilogue == EPI_RELU2 || a.epilogue == EPI_GLU || (a.epilogue == EPI_XIELU && a.act_pq), "linear_f32: epilogue %d", a.epilogue);
+    LCU_REQUIRE(a.epilogue == EPI_STORE_F32 || a.epilogue == EPI_RELU2 || a.epilogue == EPI_GLU || a.epilogue == EPI_CAP_F32 || (a.epilogue == EPI_XIELU && a.act_pq), "linear_f32: epilogue %d", a.epilogue);
     dim3 grid((a.out + 63) / 64, a.tiles ? a.n_tiles : (a.n + 63) / 64, a.heads);
     LCU_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "linear_f32: grid out of range");
     LCU_CHECK_CUDA(launch_kernel(linear_f32_kernel, grid, dim3(256), 0, s, false, a));

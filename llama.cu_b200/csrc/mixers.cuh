@@ -21,6 +21,15 @@ struct GqaArgs {
     float eps;
     int rot_dims, rot_adjacent; // pairs (i, i + rot_dims / 2), or (2 i, 2 i + 1)
     const float2 *rot;          // [positions][rot_dims / 2] (cos, sin), the frequency scaling's factor included
+    const float2 *vrot;         // [positions][v_dim / 2]: values are rotated by their positions, outputs back by theirs; or nullptr
+    const float *head_temp;     // [heads] factors on the queries, or nullptr
+    // convolutions over time on the rows of the projection: [taps][channels]; inputs before the portion in the state
+    // [generation][slot][taps - 1][channels]
+    const float *conv;
+    int taps;
+    float *conv_state;
+    size_t conv_gen_stride;
+    const int32_t *req_first, *req_pos, *req_slot;
     void *q;                    // [n_tok][heads * dim_p]
     // pages: this layer's keys [kv head][slot][dim_p] at c_off, its values [kv head][slot][vdim_p] behind them
     void *pool;
@@ -34,7 +43,9 @@ struct GqaArgs {
     int stride_o;
     float scale;
     int window;                 // > 0: a position sees the `window` last ones up to itself
-    int sink;                   // one more key of score 0 without value
+    int keep;                   // with a window: the first tokens of the sequence stay visible
+    int sink;                   // one more key without value, of score 0 or sink_score[head]
+    const float *sink_score;
     const float *gate;          // output gates before the sigmoid: gate[token * stride + head], or nullptr
     const int4 *reqs;           // (request of the round, first token, tokens, position of the first token)
     int n_reqs, max_len;        // longest of them in tokens
@@ -45,6 +56,7 @@ struct GqaArgs {
     unsigned *tickets;          // [request][kv head x row tile], zero between launches
     __host__ __device__ size_t v_off() const { return c_off + ((size_t)kv_heads * dim_p << page_shift); }
     __host__ __device__ int group() const { return heads / kv_heads; }
+    __host__ __device__ int channels() const { return heads * dim_p + (own_kv ? kv_heads * (dim_p + vdim_p) : 0); }
 };
 // Biases, rotation, norms; queries to q, keys and values to the cache.
 int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl);

@@ -1,5 +1,5 @@
-// Feed-forwards of experts.  A token's router logits choose `top` experts; the sigmoids of the chosen logits scale the experts'
-// inputs, which the products' linearity lets the epilogue do: W (s x) = s (W x).
+// Feed-forwards of experts.  A token's router logits choose `top` experts.  Weights on the inputs: the products' linearity lets the
+// epilogue apply them, W (s x) = s (W x).  Weights on the outputs, and experts that return their input: the step that adds them up.
 #include "moe.cuh"
 #include "stack.cuh"
 
@@ -9,16 +9,16 @@ namespace {
 
 typedef __nv_bfloat16 bf16;
 
-// The k-th largest logits of a token, one warp: calls put(k, expert, logit) on every lane.  Equal logits: the lower index first.
-template <class F>
-__device__ __forceinline__ void top_experts(const float *z, int n, int top, int lane, const F &put) {
+// The k-th largest scores z(expert) of a token, one warp: calls put(k, expert, score) on every lane.  Equal ones: the lower index first.
+template <class Z, class F>
+__device__ __forceinline__ void top_experts(const Z &z, int n, int top, int lane, const F &put) {
     float last = INFINITY;
     int last_e = -1;
     for (int k = 0; k < top; ++k) {
         float v = -INFINITY;
         int e = n;
         for (int i = lane; i < n; i += 32) {
-            const float x = z[i];
+            const float x = z(i);
             if ((x < last || (x == last && i > last_e)) && (x > v || e == n)) { v = x; e = i; }
         }
 #pragma unroll
@@ -27,13 +27,46 @@ __device__ __forceinline__ void top_experts(const float *z, int n, int top, int 
             const int i = __shfl_xor_sync(0xffffffffu, e, o);
             if (i < n && (e == n || x > v || (x == v && i < e))) { v = x; e = i; }
         }
-        if (e >= n) { e = min(k, n - 1); v = z[e]; }  // logits that are not numbers
+        if (e >= n) { e = min(k, n - 1); v = z(e); }  // scores that are not numbers
         put(k, e, v);
         last = v;
         last_e = e;
     }
 }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Experts and weights of token t, one warp; put(k, expert) on lane 0.
+template <class F>
+__device__ __forceinline__ void route_token(const MoeRoute &a, int t, int lane, const F &put) {
+    const float *z = a.logits + (size_t)t * a.experts_p;
+    float *weight = a.weight + (size_t)t * a.top;
+    const int n = a.experts + a.identity;
+    if (!a.softmax) {
+        top_experts([&](int e) { return z[e]; }, n, a.top, lane, [&](int k, int e, float v) {
+            if (lane == 0) {
+                put(k, e);
+                weight[k] = sigmoid_f(v);
+            }
+        });
+        return;
+    }
+    float m = -INFINITY, sum = 0.f, chosen = 0.f;
+    for (int e = lane; e < n; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    for (int e = lane; e < n; e += 32) sum += expf(z[e] - m);
+    sum = warp_sum(sum);
+    auto score = [&](int e) { return expf(z[e] - m) / sum; };
+    top_experts([&](int e) { return score(e) + a.correction[e]; }, n, a.top, lane, [&](int k, int e, float) {
+        const float s = score(e);
+        chosen += s;
+        if (lane == 0) {
+            put(k, e);
+            weight[k] = s;
+        }
+    });
+    __syncwarp();
+    for (int k = lane; k < a.top; k += 32) weight[k] /= chosen + 1e-20f;
+}
 
 // Exclusive sums of count[0..n) into first, and of (count + per - 1) / per into tile0; one warp; returns the sums of all.
 __device__ __forceinline__ int2 warp_offsets(const unsigned *count, int n, int per, int lane, int *first, int *tile0) {
@@ -65,12 +98,9 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const MoeRoute a) {
     __syncthreads();
     grid_dep_wait();
     for (int t = tid >> 5; t < a.n_tok; t += blockDim.x >> 5)
-        top_experts(a.logits + (size_t)t * a.experts_p, a.experts, a.top, lane, [&](int k, int e, float z) {
-            if (lane == 0) {
-                expert[t * a.top + k] = e;
-                place[t * a.top + k] = (int)atomicAdd(&count[e], 1u);
-                a.weight[t * a.top + k] = sigmoid_f(z);
-            }
+        route_token(a, t, lane, [&](int k, int e) {
+            expert[t * a.top + k] = e;
+            if (e < a.experts) place[t * a.top + k] = (int)atomicAdd(&count[e], 1u);
         });
     __syncthreads();
     if (tid < 32) {
@@ -79,8 +109,9 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const MoeRoute a) {
     }
     __syncthreads();
     for (int i = tid; i < rows; i += blockDim.x) {
-        const int slot = first[expert[i]] + place[i];
+        const int slot = expert[i] < a.experts ? first[expert[i]] + place[i] : -1;
         a.slot_of[i] = slot;
+        if (slot < 0) continue;
         a.slot_tok[slot] = i / a.top;
         a.slot_w[slot] = a.weight[i];
     }
@@ -95,12 +126,9 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const MoeRoute a) {
     const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= a.n_tok) return;
     grid_dep_wait();
-    top_experts(a.logits + (size_t)t * a.experts_p, a.experts, a.top, lane, [&](int k, int e, float z) {
-        if (lane == 0) {
-            a.expert[t * a.top + k] = e;
-            a.place[t * a.top + k] = (int)atomicAdd(&a.count[e], 1u);
-            a.weight[t * a.top + k] = sigmoid_f(z);
-        }
+    route_token(a, t, lane, [&](int k, int e) {
+        a.expert[t * a.top + k] = e;
+        if (e < a.experts) a.place[t * a.top + k] = (int)atomicAdd(&a.count[e], 1u);
     });
 }
 
@@ -121,11 +149,12 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeRoute a) {
     const uint4 *src = reinterpret_cast<const uint4 *>(reinterpret_cast<const T *>(a.h) + (size_t)t * a.d_p);
     constexpr int V = 16 / sizeof(T);
     for (int k = 0; k < a.top; ++k) {
-        const int i = t * a.top + k, slot = first[a.expert[i]] + a.place[i];
+        const int i = t * a.top + k, slot = a.expert[i] < a.experts ? first[a.expert[i]] + a.place[i] : -1;
+        if (tid == 0) a.slot_of[i] = slot;
+        if (slot < 0) continue;
         uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<T *>(a.xg) + (size_t)slot * a.d_p);
         for (int c = tid; c < a.d_p / V; c += 256) dst[c] = src[c];
         if (tid == 0) {
-            a.slot_of[i] = slot;
             a.slot_tok[slot] = t;
             a.slot_w[slot] = a.weight[i];
         }

@@ -12,6 +12,11 @@ constexpr int MOE_SMALL_ROUND = 64;  // tokens up to which a round takes the sma
 struct MoeRoute {
     const float *logits;  // [n_tok][experts_p]
     int n_tok, experts, experts_p, top;
+    // softmax: scores are the softmax of all logits, those + correction choose, the chosen ones divided by their sum are the weights;
+    // otherwise the largest logits choose and their sigmoids are the weights
+    int softmax;
+    const float *correction;
+    int identity;         // experts behind the others that have no matrices: slot_of is -1
     // per (token, rank): expert, its place among the expert's rows, slot; per slot: token, weight
     int *expert, *place, *slot_of, *slot_tok;
     float *weight, *slot_w;  // per (token, rank) and per slot

@@ -1,6 +1,7 @@
 // What the kernels of the recurrent mixers share: short convolutions with their state, f32 numbers as sums of bf16 ones, and the
 // legacy tensor-core products of 8 x 8 tiles.
 #pragma once
+#include "conv.cuh"
 #include "gqa_prep.cuh"
 #include "stack.cuh"
 
@@ -34,22 +35,6 @@ __device__ __forceinline__ float octet_sum(float v) {
     return v + __shfl_xor_sync(0xffffffffu, v, 4);
 }
 
-// A request's view of the convolutions' inputs: rows of this round, before them the state, before the sequence zeros.
-struct ConvIn {
-    const float *row;        // this token's row of the projection
-    const float *state;      // [taps - 1][channels] of the generation to read, newest last
-    int stride, channels, taps, in_portion, seen;  // tokens of the portion before this one, of the sequence before this one
-    __device__ __forceinline__ float at(int back, int c) const {
-        if (back <= in_portion) return row[c - (ptrdiff_t)back * stride];
-        if (back > seen) return 0.f;
-        return state[(size_t)(taps - 1 - (back - in_portion)) * channels + c];
-    }
-    __device__ __forceinline__ float4 at4(int back, int c) const {  // four channels
-        if (back <= in_portion) return *reinterpret_cast<const float4 *>(row + (c - (ptrdiff_t)back * stride));
-        if (back > seen) return make_float4(0.f, 0.f, 0.f, 0.f);
-        return *reinterpret_cast<const float4 *>(state + (size_t)(taps - 1 - (back - in_portion)) * channels + c);
-    }
-};
 __device__ __forceinline__ ConvIn conv_in(const DeltaArgs &a, int t, int r) {
     ConvIn c;
     const int sg = a.req_slot[r];

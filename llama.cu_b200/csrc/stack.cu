@@ -64,9 +64,17 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
             LCU_REQUIRE(l.kv_from >= 0 && l.kv_from <= i, "layer %d: keys and values of layer %d", i, l.kv_from - 1);
             if (l.kv_from) {
                 const lcu_layer_desc &o = layers[l.kv_from - 1];
-                LCU_REQUIRE((o.mixer & LCU_MIX_ATTENTION) && !o.kv_from && o.kv_heads == l.kv_heads && o.dim == l.dim && o.v_dim == l.v_dim,
+                LCU_REQUIRE((o.mixer & LCU_MIX_ATTENTION) && !o.kv_from && o.kv_heads == l.kv_heads && o.dim == l.dim && o.v_dim == l.v_dim &&
+                                o.rot_values == l.rot_values && (!l.rot_values || o.rot_base == l.rot_base),
                             "layer %d: the keys and values of layer %d do not fit", i, l.kv_from - 1);
             }
+            LCU_REQUIRE(l.sink >= 0 && l.sink <= 2 && l.keep_first >= 0 && (l.keep_first == 0 || l.window > 0), "layer %d: sink %d, %d first tokens behind a window of %d",
+                        i, l.sink, l.keep_first, l.window);
+            LCU_REQUIRE(l.conv >= 0 && l.conv <= 64 && (l.conv == 0 || (!l.bias && l.qk_norm != 3)),
+                        "layer %d: convolution of %d taps (0..64), beside biases or a norm over all heads", i, l.conv);
+            LCU_REQUIRE(!l.rot_values || (l.v_dim % 2 == 0 && l.rot_base > 0 && l.rot_factor <= 0 && (l.rot_dims == 0 || l.rot_adjacent)),
+                        "layer %d: rotated values of size %d take neighbouring pairs", i, l.v_dim);
+            LCU_REQUIRE(!rec || !(l.conv || l.rot_values || l.head_temp), "layer %d: convolutions, rotated values or factors per head beside a recurrent mixer", i);
         }
         if (rec) {
             LCU_REQUIRE(l.delta_heads > 0 && l.delta_kv_heads > 0 && l.delta_heads % l.delta_kv_heads == 0, "layer %d: %d value heads, %d key heads", i,
@@ -82,16 +90,21 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
         LCU_REQUIRE((l.mixer & LCU_MIX_ATTENTION) == 0 || rec == 0 || (rec == LCU_MIX_DELTA) == (l.post_norm == 0),
                     "layer %d: side by side, outputs of a delta rule are normed one by one, those of other mixers added ahead of a norm", i);
         const bool ff = l.ff > 0 || l.shared_ff > 0;
-        LCU_REQUIRE(!ff || l.ff_act == LCU_ACT_RELU2 || l.ff_act == LCU_ACT_GLU, "layer %d: unknown activation %d", i, l.ff_act);
-        LCU_REQUIRE(l.experts == 0 ? l.shared_ff == 0 : (l.ff_act == LCU_ACT_GLU && l.ff > 0 && l.top > 0 && l.top <= l.experts && l.post_norm),
+        LCU_REQUIRE(!ff || l.ff_act == LCU_ACT_RELU2 || l.ff_act == LCU_ACT_GLU || l.ff_act == LCU_ACT_POLYNORM, "layer %d: unknown activation %d", i, l.ff_act);
+        LCU_REQUIRE(!l.ff_bias || (l.ff > 0 && l.ff_act == LCU_ACT_POLYNORM), "layer %d: biases of activation %d", i, l.ff_act);
+        LCU_REQUIRE(l.experts == 0 ? l.shared_ff == 0 && l.identity == 0 : (l.ff_act == LCU_ACT_GLU && l.ff > 0 && l.identity >= 0 && l.top > 0 && l.top <= l.experts + l.identity),
                     "layer %d: %d experts, %d per token, widths %d and %d", i, l.experts, l.top, l.ff, l.shared_ff);
-        LCU_REQUIRE(l.experts <= 4096 && l.experts * 12 + MOE_SMALL_ROUND * l.top * 8 <= 48 * 1024, "layer %d: %d experts, %d per token", i, l.experts, l.top);
+        LCU_REQUIRE(l.experts <= 4096 && l.identity <= 4096 && l.experts * 12 + MOE_SMALL_ROUND * l.top * 8 <= 48 * 1024, "layer %d: %d experts, %d per token", i, l.experts, l.top);
+        LCU_REQUIRE((l.route_softmax && l.experts && !l.post_norm) || (!l.route_softmax && !l.identity), "layer %d: weights on the outputs of experts take a softmax and no norm on them", i);
+        LCU_REQUIRE(!l.parallel_ff || (!l.post_norm && !((l.mixer & LCU_MIX_ATTENTION) && rec) && !l.shared_ff && layers[0].pair_buckets == 0),
+                    "layer %d: a feed-forward beside two mixers, a shared expert, norms on outputs or an embedding of pairs", i);
         LCU_REQUIRE(!ff || l.ff_act != LCU_ACT_GLU || (l.glu_limit > 0 && (l.shared_ff == 0 || l.shared_limit > 0)), "layer %d: limit %g of a gated activation", i, l.glu_limit);
         LCU_REQUIRE((l.post_norm != 0) == (layers[0].post_norm != 0), "layer %d: norms on outputs in some layers only", i);
     }
     if (i == 0)
         LCU_REQUIRE(l.pair_buckets >= 0 && l.pair_prev >= 0 && l.pair_cur >= 0 && (l.pair_buckets == 0 || (l.pre_norm && l.pair_prev < l.pair_buckets && l.pair_cur < l.pair_buckets)),
                     "embedding of token pairs: %d buckets, factors %d and %d", l.pair_buckets, l.pair_prev, l.pair_cur);
+    if (i == 0) LCU_REQUIRE(l.logit_cap >= 0, "logits capped at %g", l.logit_cap);
     LCU_REQUIRE(l.weights_of >= -1 && l.weights_of < d.n_layers && l.weights_of != i, "layer %d uses the weights of layer %d", i, l.weights_of);
     return LCU_OK;
 }
@@ -100,7 +113,7 @@ static int check_layer(const lcu_model_desc &d, const lcu_layer_desc *layers, in
 static int gqa_target_ctas(const StackLayer &L) { return 2 * sm_count() * gqa_short_ctas_per_sm(L.dim_p, L.vdim_p); }
 int gqa_splits_for(const lcu_ctx *c, const StackLayer &L, int reqs, int len) {
     const int ctas = reqs * L.d.kv_heads * gqa_row_tiles(L.d.heads, L.d.kv_heads, len);
-    const int seen = L.d.window > 0 && L.d.window + len < c->desc.nctx ? L.d.window + len + 63 : c->desc.nctx, units = (seen + 63) / 64;
+    const int some = L.d.window + L.d.keep_first + len, seen = L.d.window > 0 && some < c->desc.nctx ? some + 63 : c->desc.nctx, units = (seen + 63) / 64;
     int z = ctas > 0 ? gqa_target_ctas(L) / ctas : 1;
     if (z > 64) z = 64;
     if (z > units) z = units;
@@ -110,26 +123,32 @@ int gqa_splits_for(const lcu_ctx *c, const StackLayer &L, int reqs, int len) {
 // (cos, sin) of every position and rotated pair, angles in f64; YaRN: frequencies of fewer than `slow` turns in `original`
 // positions are divided by the factor, those of more than `fast` stay, a linear ramp over the pair's index lies between, and
 // both functions are scaled by 0.1 ln(factor) + 1.
-static int make_rot_table(Stack *S, const lcu_layer_desc &l, int nctx, const float2 **out) {
-    const int half = l.rot_dims / 2;
+static int make_rot_table(Stack *S, Stack::RotTable t, int nctx, const float2 **out) {
+    for (const Stack::RotTable &o : S->rot_tables)
+        if (o.dims == t.dims && o.base == t.base && o.factor == t.factor && o.original == t.original && o.fast == t.fast && o.slow == t.slow) {
+            *out = o.dev;
+            return LCU_OK;
+        }
+    const int half = t.dims / 2;
     std::vector<double> freq(half);
     double gain = 1.0;
-    for (int i = 0; i < half; ++i) freq[i] = pow(l.rot_base, -2.0 * i / l.rot_dims);
-    if (l.rot_factor > 0) {
-        auto index_of = [&](double turns) { return l.rot_dims * log(l.rot_original / (2.0 * M_PI * turns)) / (2.0 * log(l.rot_base)); };
-        const double lo = fmax(floor(index_of(l.rot_fast)), 0.0), hi = fmin(ceil(index_of(l.rot_slow)), l.rot_dims - 1.0);
+    for (int i = 0; i < half; ++i) freq[i] = pow(t.base, -2.0 * i / t.dims);
+    if (t.factor > 0) {
+        auto index_of = [&](double turns) { return t.dims * log(t.original / (2.0 * M_PI * turns)) / (2.0 * log(t.base)); };
+        const double lo = fmax(floor(index_of(t.fast)), 0.0), hi = fmin(ceil(index_of(t.slow)), t.dims - 1.0);
         for (int i = 0; i < half; ++i) {
             const double ramp = fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0);
-            freq[i] = freq[i] / l.rot_factor * ramp + freq[i] * (1.0 - ramp);
+            freq[i] = freq[i] / t.factor * ramp + freq[i] * (1.0 - ramp);
         }
-        gain = 0.1 * log(l.rot_factor) + 1.0;
+        gain = 0.1 * log(t.factor) + 1.0;
     }
     std::vector<float2> host((size_t)nctx * half);
     for (int p = 0; p < nctx; ++p)
         for (int i = 0; i < half; ++i) host[(size_t)p * half + i] = make_float2((float)(cos(p * freq[i]) * gain), (float)(sin(p * freq[i]) * gain));
     float2 *dev = nullptr;
     LCU_CHECK_CUDA(cudaMalloc(reinterpret_cast<void **>(&dev), host.size() * sizeof(float2)));
-    S->rot_tables.push_back(dev);
+    t.dev = dev;
+    S->rot_tables.push_back(t);
     LCU_CHECK_CUDA(cudaMemcpy(dev, host.data(), host.size() * sizeof(float2), cudaMemcpyHostToDevice));
     *out = dev;
     return LCU_OK;
@@ -149,10 +168,10 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->w.resize(d.n_layers);
     size_t off = 0;
     int max_lat = 0, max_qr = 0, max_q = 0, max_hr = 0, max_hv = 64, max_ff = 64, max_kv = 0;
-    int max_dk = 0, max_dv = 0, max_coef = 0, max_tail = 0, max_dhv = 0, max_vp = 0, max_top = 0, max_ep = 0, max_eff = 0;
+    int max_dk = 0, max_dv = 0, max_coef = 0, max_tail = 0, max_dhv = 0, max_vp = 0, max_top = 0, max_ep = 0, max_eff = 0, max_z = 0;
     size_t conv_total = 0, mat_total = 0;  // f32 values of recurrent state per slot
     S->pre_norm = layers[0].pre_norm != 0;
-    bool any_shift = false, any_rec = layers[0].pair_buckets > 0, can_expand = c->dt != LCU_F32 && !S->pre_norm;
+    bool any_shift = false, any_parallel = false, any_rec = layers[0].pair_buckets > 0, can_expand = c->dt != LCU_F32 && !S->pre_norm;
     for (int i = 0; i < d.n_layers; ++i) {
         StackLayer &L = S->layers[i];
         L.d = layers[i];
@@ -167,7 +186,9 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                         o.kv_heads == L.d.kv_heads && o.bias == L.d.bias && o.delta_heads == L.d.delta_heads &&
                         o.delta_kv_heads == L.d.delta_kv_heads && o.delta_dim == L.d.delta_dim && o.delta_v_dim == L.d.delta_v_dim &&
                         o.delta_conv == L.d.delta_conv && o.qk_norm == L.d.qk_norm && o.kv_from == L.d.kv_from && o.norm_parts == L.d.norm_parts &&
-                        o.gate_rank == L.d.gate_rank && o.experts == L.d.experts && o.shared_ff == L.d.shared_ff && o.ff_act == L.d.ff_act,
+                        o.gate_rank == L.d.gate_rank && o.experts == L.d.experts && o.shared_ff == L.d.shared_ff && o.ff_act == L.d.ff_act &&
+                        o.conv == L.d.conv && o.sink == L.d.sink && o.head_temp == L.d.head_temp && o.ff_bias == L.d.ff_bias &&
+                        o.route_softmax == L.d.route_softmax && o.identity == L.d.identity,
                     "layer %d differs from layer %d whose weights it uses", i, L.src);
         auto up = [](int &m, int v) { if (v > m) m = v; };
         L.ff_p = stack_pad(L.d.ff, 64);
@@ -197,17 +218,19 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
             else L.c_off = S->layers[L.kv_src].c_off;
             up(max_q, L.d.heads * L.dim_p); up(max_vp, L.vdim_p);
             if (gqa_target_ctas(L) > S->gqa_ctas) S->gqa_ctas = gqa_target_ctas(L);
-            for (int j = 0; j < i && !L.rot; ++j) {  // layers with the same rotation share a table
-                const lcu_layer_desc &e = layers[j];
-                if (S->layers[j].rot && e.rot_dims == L.d.rot_dims && e.rot_base == L.d.rot_base && e.rot_factor == L.d.rot_factor &&
-                    e.rot_original == L.d.rot_original && e.rot_fast == L.d.rot_fast && e.rot_slow == L.d.rot_slow)
-                    L.rot = S->layers[j].rot;
-            }
-            if (L.d.rot_dims && !L.rot) {
-                int rc = make_rot_table(S, L.d, d.nctx, &L.rot);
-                if (rc) return rc;
+            int rc = LCU_OK;
+            if (L.d.rot_dims)
+                rc = make_rot_table(S, {L.d.rot_dims, L.d.rot_base, L.d.rot_factor, L.d.rot_original, L.d.rot_fast, L.d.rot_slow, nullptr}, d.nctx, &L.rot);
+            if (!rc && L.d.rot_values) rc = make_rot_table(S, {L.d.v_dim, L.d.rot_base, 0.0, 0.0, 0.0, 0.0, nullptr}, d.nctx, &L.vrot);
+            if (rc) return rc;
+            if (L.d.conv > 1) {
+                L.conv_off = conv_total;
+                conv_total += (size_t)(L.d.conv - 1) * L.att_rows;
+                any_rec = true;
             }
         }
+        any_parallel = any_parallel || L.parallel();
+        if (L.poly()) up(max_z, L.ff_p);
         if (L.recurrent()) {
             L.dk_p = stack_pad(L.d.delta_dim, 32);
             L.dv_p = stack_pad(L.d.delta_v_dim, 16);
@@ -226,7 +249,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
         }
         if (L.d.shared_ff) { L.sff_p = stack_pad(L.d.shared_ff, 64); up(max_ff, L.sff_p); }
         if (L.d.experts) {
-            L.e_p = stack_pad(L.d.experts, 8);
+            L.e_p = stack_pad(L.d.experts + L.d.identity, 8);
             up(max_ep, L.e_p); up(max_top, L.d.top); up(max_eff, L.ff_p); up(S->max_experts, L.d.experts);
         }
         up(max_lat, L.in_rows()); up(max_qr, L.qr_p); up(max_hv, L.hv_p);
@@ -268,6 +291,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
                  o_gp = reserve(gqa_part_floats(S->gqa_ctas, max_vp) * 4), o_gt = reserve((size_t)S->gqa_ctas * 4);
     const size_t R = S->max_rows, o_lt = reserve((size_t)2 * S->n_slots * 4), o_ro = reserve(T * max_ep * 4), o_ye = reserve(R * S->d_p * 4), o_mi = reserve(R * 16), o_mw = reserve(R * 8),
                  o_mc = reserve((size_t)S->max_experts * 4), o_mt = reserve((size_t)S->n_tiles * 16), o_xg = reserve(R * S->d_p * eb), o_ae = reserve(R * max_eff * eb);
+    const size_t o_h2 = reserve(any_parallel ? T * S->d_p * eb : 0), o_z = reserve(T * max_z * 4);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
     LCU_CHECK_CUDA(cudaMemset(S->arena, 0, total));  // pads of att (columns past the heads) stay zero from here on
     unsigned char *p = reinterpret_cast<unsigned char *>(S->arena);
@@ -287,6 +311,8 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->moe_w = reinterpret_cast<float *>(p + o_mw); S->moe_slot_w = S->moe_w + R; S->moe_count = reinterpret_cast<unsigned *>(p + o_mc);
     S->moe_tiles = reinterpret_cast<int4 *>(p + o_mt); S->xg = p + o_xg; S->act_e = p + o_ae;
 
+    S->h2 = p + o_h2; S->z = reinterpret_cast<float *>(p + o_z);
+
     // every kernel variant a round can launch
     if (S->pre_norm) {
         if (c->dt == LCU_F32) return LCU_OK;
@@ -300,11 +326,11 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
             if (!rc && L.attention()) rc = gemv_warm(L.hv_p, S->d_p, false, c->dt, EPI_STORE_F32);
             if (!rc && L.recurrent()) rc = gemv_warm(L.dhv_p, S->d_p, false, c->dt, EPI_STORE_F32);
             if (!rc && L.d.experts) rc = gemv_warm(S->d_p, L.e_p, false, c->dt, EPI_STORE_F32);
-            else if (!rc && L.d.ff) rc = L.glu() ? gemv_warm(S->d_p, 2 * L.ff_p, false, c->dt, EPI_GLU) : gemv_warm(S->d_p, L.ff_p, false, c->dt, EPI_RELU2);
+            else if (!rc && L.d.ff) rc = L.glu() ? gemv_warm(S->d_p, 2 * L.ff_p, false, c->dt, EPI_GLU) : gemv_warm(S->d_p, L.ff_p, false, c->dt, L.poly() ? EPI_STORE_F32 : EPI_RELU2);
             if (!rc && L.d.ff && !L.d.experts) rc = gemv_warm(L.ff_p, S->d_p, false, c->dt, EPI_STORE_F32);
         }
-        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt);
-        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, EPI_STORE_F32);
+        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, S->caps() ? EPI_CAP : EPI_STORE);
+        if (!rc) rc = gemv_warm(S->d_p, S->vocab_p, false, c->dt, S->caps() ? EPI_CAP_F32 : EPI_STORE_F32);
         return rc;
     }
     int rc = latent_attn_launch(LatentAttnArgs{}, c->dt, nullptr, false, true);
@@ -335,7 +361,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
 void stack_destroy(lcu_ctx *c) {
     if (!c->stack) return;
     if (c->stack->arena) cudaFree(c->stack->arena);
-    for (float2 *t : c->stack->rot_tables) cudaFree(t);
+    for (const Stack::RotTable &t : c->stack->rot_tables) cudaFree(t.dev);
     delete c->stack;
     c->stack = nullptr;
 }
@@ -379,6 +405,13 @@ bool stack_weight_shape(const lcu_ctx *c, int layer, int kind, int *rows, int *c
     case LCU_W_POST1: return f32(1, S.d_p, L.d.post_norm != 0);
     case LCU_W_POST2: return f32(1, S.d_p, L.d.post_norm && L.has_ff());
     case LCU_W_ROUTER: *rows = L.e_p; *cols = S.d_p; return L.d.experts > 0;
+    case LCU_W_CORRECTION: return f32(1, L.e_p, L.d.route_softmax != 0);
+    case LCU_W_ATT_CONV: return f32(L.d.conv, L.att_rows, L.attention() && L.d.conv > 0);
+    case LCU_W_SINK: return f32(1, L.d.heads, L.attention() && L.d.sink == 2);
+    case LCU_W_HEAD_TEMP: return f32(1, L.d.heads, L.attention() && L.d.head_temp);
+    case LCU_W_UP_BIAS: return f32(1, L.ff_p, L.d.ff_bias != 0);
+    case LCU_W_DOWN_BIAS: return f32(1, S.d_p, L.d.ff_bias != 0);
+    case LCU_W_ACT: return f32(1, 4, L.d.ff > 0 && L.poly());
     case LCU_W_SHARED_UP: *rows = 2 * L.sff_p; *cols = S.d_p; return L.d.shared_ff > 0;
     case LCU_W_SHARED_DOWN: *rows = S.d_p; *cols = L.sff_p; return L.d.shared_ff > 0;
     default: return false;
@@ -422,6 +455,13 @@ int stack_set_weight(lcu_ctx *c, int layer, int kind, const void *ptr) {
     case LCU_W_CONV_BIAS: w.conv_bias = f; break;
     case LCU_W_GATE_MAP: w.gate_map = f; break;
     case LCU_W_ROUTER: w.router = ptr; break;
+    case LCU_W_CORRECTION: w.correction = f; break;
+    case LCU_W_ATT_CONV: w.att_conv = f; break;
+    case LCU_W_SINK: w.sink = f; break;
+    case LCU_W_HEAD_TEMP: w.head_temp = f; break;
+    case LCU_W_UP_BIAS: w.up_bias = f; break;
+    case LCU_W_DOWN_BIAS: w.down_bias = f; break;
+    case LCU_W_ACT: w.act = f; break;
     case LCU_W_SHARED_UP: w.shared_up = ptr; break;
     case LCU_W_SHARED_DOWN: w.shared_down = ptr; break;
     case LCU_W_LAT_IN: w.in = ptr; break;
@@ -454,7 +494,8 @@ bool stack_ready(const lcu_ctx *c) {
         if (L.src == (int)i) {
             ok = ok && w.in && (!d.ff || (w.up && w.down)) && (!d.token_shift || w.shift);
             if (L.latent()) ok = ok && w.q_norm && w.kv_norm && w.uq && w.ukt && w.ukv && w.out && w.scalars;
-            if (L.attention()) ok = ok && w.att_out && (!d.bias || w.bias) && (d.qk_norm < 2 || w.qk_gain);
+            if (L.attention()) ok = ok && w.att_out && (!d.bias || w.bias) && (d.qk_norm < 2 || w.qk_gain) && (!d.conv || w.att_conv) && (d.sink != 2 || w.sink) && (!d.head_temp || w.head_temp);
+            ok = ok && (!d.ff_bias || (w.up_bias && w.down_bias)) && (!d.ff || !L.poly() || w.act) && (!d.route_softmax || w.correction);
             if (L.recurrent()) ok = ok && w.delta_out && w.delta_norm && (L.gla() ? w.gate_map != nullptr : w.conv && w.decay) && (!L.ssd() || w.conv_bias);
             if (S.pre_norm) ok = ok && w.norm1 && (!L.has_ff() || w.norm2) && (!(L.attention() && L.delta()) || w.branch_norm);
             if (d.post_norm) ok = ok && w.post1 && (!L.has_ff() || w.post2);
@@ -712,7 +753,10 @@ int stack_head(lcu_ctx *c, const Round &r, const uint32_t *rows, int n_rows, flo
     ++*count;
     Launcher L{c, s, count, pdl};
     void *y = out_f32 ? reinterpret_cast<void *>(out_f32) : c->logits;
-    return L.linear(c->lm_head, S.d_p, S.vocab_p, S.hout, n_rows, y, S.vocab_p, out_f32 ? EPI_STORE_F32 : EPI_STORE);
+    const lcu_layer_desc &d = S.layers[0].d;
+    L.cap = CapArgs{d.logit_scale ? d.logit_scale : 1.f, d.logit_cap};
+    const int f32 = S.caps() ? EPI_CAP_F32 : EPI_STORE_F32, act = S.caps() ? EPI_CAP : EPI_STORE;
+    return L.linear(c->lm_head, S.d_p, S.vocab_p, S.hout, n_rows, y, S.vocab_p, out_f32 ? f32 : act);
 }
 
 // Algorithmic bytes of a round: the weights the round's forms of attention touch, the head, cached rows and state.
@@ -726,7 +770,7 @@ double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_
         if (d.experts) {  // the experts that this many tokens use when they choose evenly
             double tokens = 0.0;
             for (int i = 0; i < n_req; ++i) tokens += reqs[i].len;
-            ff *= d.experts * (1.0 - pow(1.0 - (double)d.top / d.experts, tokens));
+            ff *= d.experts * (1.0 - pow(1.0 - (double)d.top / (d.experts + d.identity), tokens));
         }
         bytes += wb * ((double)L.in_rows() * S.d_p + ff + 3.0 * L.sff_p * S.d_p + (double)L.e_p * S.d_p + (double)S.d_p * (L.hv_p + L.dhv_p));
         if (L.latent()) bytes += wb * ((double)d.heads * L.dim_p * L.qr_p + (double)L.kv_cols() * L.r_p);
@@ -734,7 +778,8 @@ double stack_step_bytes(const lcu_ctx *c, const lcu_req *reqs, int n_req, int n_
         for (int i = 0; i < n_req; ++i) {
             for (uint32_t j = 0; j < reqs[i].len; ++j) {
                 const uint32_t seen = reqs[i].pos + j + 1;
-                bytes += (double)(d.window > 0 && seen > (uint32_t)d.window ? (uint32_t)d.window : seen) * row * eb;
+                const uint32_t most = (uint32_t)(d.window + d.keep_first);
+                bytes += (double)(d.window > 0 && seen > most ? most : seen) * row * eb;
             }
             if (L.recurrent()) bytes += 8.0 * d.delta_heads * L.dv_p * L.dk_p;  // matrices read and written
         }

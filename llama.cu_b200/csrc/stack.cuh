@@ -31,8 +31,8 @@ struct StackLayer {
     int kv_src = 0;                       // layer whose cache this one reads
     int dk_p = 0, dv_p = 0, dh_p = 0, dhv_p = 0, rank_p = 0;
     int e_p = 0, sff_p = 0;               // experts, width of the shared one
-    size_t conv_off = 0, mat_off = 0;     // f32 offsets of this layer's recurrent state in its arena section
-    const float2 *rot = nullptr;          // [nctx][rot_dims / 2] (cos, sin)
+    size_t conv_off = 0, mat_off = 0;     // f32 offsets of this layer's recurrent state in its arena section (inputs of the mixer's convolutions, matrices)
+    const float2 *rot = nullptr, *vrot = nullptr;  // [nctx][rot_dims / 2] (cos, sin); of values [nctx][v_dim / 2]
     bool latent() const { return d.mixer == LCU_MIX_LATENT; }
     bool attention() const { return (d.mixer & LCU_MIX_ATTENTION) != 0; }
     bool delta() const { return (d.mixer & LCU_MIX_DELTA) != 0; }
@@ -41,6 +41,8 @@ struct StackLayer {
     bool recurrent() const { return delta() || ssd() || gla(); }
     bool own_kv() const { return d.kv_from == 0; }
     bool glu() const { return d.ff_act == LCU_ACT_GLU; }
+    bool poly() const { return d.ff_act == LCU_ACT_POLYNORM; }
+    bool parallel() const { return d.parallel_ff && has_ff(); }
     bool has_ff() const { return d.ff > 0 || d.shared_ff > 0; }
     int qkv_rows() const { return 2 * d.delta_kv_heads * dk_p + d.delta_heads * dv_p; }  // of a recurrent mixer
     int rec_rows() const { return recurrent() ? qkv_rows() + d.delta_heads * dv_p + (gla() ? rank_p : ssd() ? dh_p : 2 * dh_p) : 0; }
@@ -58,6 +60,7 @@ struct StackWeights {
     const float *bias = nullptr, *conv = nullptr, *decay = nullptr, *delta_norm = nullptr, *branch_norm = nullptr, *norm1 = nullptr,
                 *norm2 = nullptr, *step = nullptr, *post1 = nullptr, *post2 = nullptr, *qk_gain = nullptr, *conv_bias = nullptr, *gate_map = nullptr;
     const void *router = nullptr, *shared_up = nullptr, *shared_down = nullptr;
+    const float *att_conv = nullptr, *sink = nullptr, *head_temp = nullptr, *up_bias = nullptr, *down_bias = nullptr, *act = nullptr, *correction = nullptr;
 };
 
 // What the host decides about a round: which requests run their attention in latent space ("absorbed") and which expand
@@ -96,7 +99,10 @@ struct Stack {
     unsigned *gqa_tickets = nullptr;
     size_t conv_gen = 0;    // f32 values of one generation of the convolutions' state
     int gqa_ctas = 0;       // CTAs of split short-form attention the partial buffer holds
-    std::vector<float2 *> rot_tables;
+    struct RotTable { int dims; double base, factor, original, fast, slow; float2 *dev; };
+    std::vector<RotTable> rot_tables;  // layers with the same rotation share one
+    void *h2 = nullptr;                // input of a feed-forward beside a mixer
+    float *z = nullptr;                // f32 rows of the up projection (LCU_ACT_POLYNORM)
     const void *pair_embd = nullptr;
     uint32_t *last_token = nullptr;  // [generation 2][slots]
     float *dtail = nullptr;          // linear recurrences: decays over blocks
@@ -107,6 +113,7 @@ struct Stack {
     int4 *moe_tiles = nullptr;
     void *xg = nullptr, *act_e = nullptr;
     int max_rows = 0, max_experts = 0, n_tiles = 0;  // capacities
+    bool caps() const { return layers[0].d.logit_cap > 0.f || (layers[0].d.logit_scale != 0.f && layers[0].d.logit_scale != 1.f); }
 };
 
 // ---- stack.cu
@@ -152,6 +159,8 @@ int op_mix_input(const MixInputArgs &a, int dt, cudaStream_t s, bool pdl);
 // activation dtype; every input and h may be missing.  The sublayer's output is one of
 //     sum of y (each y * y_gain / rms(y) when gains are given)
 //     post_gain * s / rms(s), s = sum of y_scale * y and of the token's rows of ye
+//     sum of y, y_bias and ye_w * the token's rows of ye (slot -1: of ff_in)
+// h2 = gain2 * x_out / rms(x_out) for a feed-forward beside the mixer.
 struct PreNormArgs {
     const float *x_in;
     const float *y[2];
@@ -159,6 +168,9 @@ struct PreNormArgs {
     const float *post_gain;
     float y_scale[2];
     const float *ye;      // outputs of experts [slot][d_p], `top` slots per token
+    const float *ye_w;    // [n_tok][top] or nullptr
+    const void *ff_in;    // [n_tok][d_p], activation dtype
+    const float *y_bias;  // [d_p] or nullptr
     const int *slot_of;
     int top;
     const void *embd;     // bf16 [vocab, d_p], times embd_scale
@@ -172,14 +184,24 @@ struct PreNormArgs {
     const int32_t *tok_req, *req_first, *req_pos, *req_slot;
     const float *step;
     float *x_out;
-    void *h;
-    const float *gain;
+    void *h, *h2;
+    const float *gain, *gain2;
     float eps;
     int n_tok, d, d_p;
     unsigned *zero;       // counters that the kernels behind expect to be zero
     int n_zero;
 };
 int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl);
+// Activation of LCU_ACT_POLYNORM on z + bias, rounded; columns past ff are zero.
+struct PolyNormArgs {
+    const float *z;       // [n_tok][ff_p]
+    const float *bias;    // [ff_p] or nullptr
+    const float *act;     // a, b, c, e
+    void *y;              // [n_tok][ff_p]
+    int n_tok, ff, ff_p;
+    float eps;
+};
+int op_poly_norm(const PolyNormArgs &a, int dt, cudaStream_t s, bool pdl);
 // y = x[rows[i]] * gain / rms(x), rounded
 int op_scalar_norm_rows(void *y, const float *x, const uint32_t *rows, int n, int d, int d_p, const float *gain, int gain_stride, float eps,
                         int dt, cudaStream_t s, bool pdl);
@@ -196,11 +218,12 @@ struct LinearF32Args {
     int stride_y, head_y;
     const int32_t *y_rows;      // optional row scatter
     int n, in, out, heads;
-    int epilogue;               // EPI_STORE_F32, EPI_XIELU, EPI_RELU2, EPI_GLU
+    int epilogue;               // EPI_STORE_F32, EPI_XIELU, EPI_RELU2, EPI_GLU, EPI_CAP_F32
     const float *act_pq;
     const float *gate;          // optional: multiplied by sigmoid(gate[y row * stride_gate + head])
     int stride_gate;
     GluArgs glu;                // EPI_GLU
+    CapArgs cap;                // EPI_CAP_F32
     const int4 *tiles;          // grouped: (matrix, first row, rows up to 64), `heads` 1, no gather; see GemvArgs
     int n_tiles;
     const float *row_scale;
@@ -294,6 +317,13 @@ template <> __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16 *p,
 }
 __device__ __forceinline__ float4 ld4_bf16(const void *base, size_t i) {
     const uint2 u = __ldg(reinterpret_cast<const uint2 *>(reinterpret_cast<const __nv_bfloat16 *>(base) + i));
+    const float2 a = Act<__nv_bfloat16>::to_f2(u.x), b = Act<__nv_bfloat16>::to_f2(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+template <class T> __device__ __forceinline__ float4 ld4(const T *p);
+template <> __device__ __forceinline__ float4 ld4<float>(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+template <> __device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
     const float2 a = Act<__nv_bfloat16>::to_f2(u.x), b = Act<__nv_bfloat16>::to_f2(u.y);
     return make_float4(a.x, a.y, b.x, b.y);
 }

@@ -107,18 +107,19 @@ __device__ __forceinline__ size_t pair_row(const PreNormArgs &a, int t) {
     return (size_t)((prev * (unsigned)a.pair_prev + (unsigned long long)a.tokens[t] * (unsigned)a.pair_cur) % (unsigned)a.pair_buckets);
 }
 
-// One block per token: the residual step of pre-norm layers.  POST: the outputs are one sum (of experts' rows too), which may be
-// normed; token pairs.
+// One block per token: the residual step of pre-norm layers.  FORM 1 and 2: the outputs are one sum, of experts' rows too.  1: the
+// sum may be normed; token pairs.  2: weights on experts' rows, experts that return their input, a bias, a second norm.
 constexpr int pre_norm_threads(int maxv) { return maxv == 1 ? 128 : 256 * maxv; }
-template <class T, int MAXV, bool POST>
-__global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 : 1) pre_norm_kernel(const PreNormArgs a) {
+template <class T, int MAXV, int FORM>
+__global__ void __launch_bounds__(pre_norm_threads(MAXV), FORM && MAXV == 2 ? 3 : 1) pre_norm_kernel(const PreNormArgs a) {
+    constexpr bool POST = FORM > 0, PAIR = FORM == 2;
     grid_dep_launch();
     const int t = blockIdx.x, n4 = a.d_p / 4;
     __shared__ float2 part[32], part2[32];
     const size_t row = (size_t)t * a.d_p;
     grid_dep_wait();
     const size_t e0 = a.embd ? (size_t)a.tokens[t] * a.d_p : 0;  // fed-back tokens are written by the kernel before the round's first one
-    const size_t e1 = POST && a.pair_embd ? pair_row(a, t) * a.d_p : 0;
+    const size_t e1 = FORM == 1 && a.pair_embd ? pair_row(a, t) * a.d_p : 0;
     if (POST && t == 0)
         for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
     float4 x[MAXV], y0[MAXV], y1[POST ? 1 : MAXV];
@@ -138,14 +139,21 @@ __global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 
                             u.w * a.y_scale[0] + v.w * a.y_scale[1]);
 #pragma unroll 2
             for (int k = 0; k < a.top; ++k) {
-                const float4 e = *reinterpret_cast<const float4 *>(a.ye + (size_t)a.slot_of[t * a.top + k] * a.d_p + 4 * i);
+                const int slot = a.slot_of[t * a.top + k];
+                const float4 e = !PAIR || slot >= 0 ? *reinterpret_cast<const float4 *>(a.ye + (size_t)slot * a.d_p + 4 * i)
+                                                    : ld4<T>(reinterpret_cast<const T *>(a.ff_in) + row + 4 * i);
+                const float w = PAIR && a.ye_w ? a.ye_w[t * a.top + k] : 1.f;
+                u.x += e.x * w; u.y += e.y * w; u.z += e.z * w; u.w += e.w * w;
+            }
+            if (PAIR && a.y_bias) {
+                const float4 e = *reinterpret_cast<const float4 *>(a.y_bias + 4 * i);
                 u.x += e.x; u.y += e.y; u.z += e.z; u.w += e.w;
             }
         }
         s0 += dot4(u);
         if constexpr (!POST) s1 += dot4(v);
     }
-    if (POST ? a.post_gain != nullptr : a.y_gain != nullptr) {
+    if (FORM == 2 ? false : FORM == 1 ? a.post_gain != nullptr : a.y_gain != nullptr) {
         const float2 s = block_sum2(s0, s1, part);
         s0 = 1.f / sqrtf(s.x / (float)a.d + a.eps);
         s1 = 1.f / sqrtf(s.y / (float)a.d + a.eps);
@@ -157,7 +165,9 @@ __global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 
         if (i >= n4) continue;
         float4 v = x[j];
         const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
-        if constexpr (POST) {
+        if constexpr (PAIR) {
+            v.x += y0[j].x; v.y += y0[j].y; v.z += y0[j].z; v.w += y0[j].w;
+        } else if constexpr (POST) {
             const float4 g = a.post_gain ? *reinterpret_cast<const float4 *>(a.post_gain + 4 * i) : one;
             const float r = a.post_gain ? s0 : 1.f;
             v.x += y0[j].x * r * g.x; v.y += y0[j].y * r * g.y; v.z += y0[j].z * r * g.z; v.w += y0[j].w * r * g.w;
@@ -176,7 +186,7 @@ __global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 
             const float4 e = ld4_bf16(a.embd, e0 + 4 * i);
             v.x += e.x * a.embd_scale; v.y += e.y * a.embd_scale; v.z += e.z * a.embd_scale; v.w += e.w * a.embd_scale;
         }
-        if (POST && a.pair_embd) {
+        if (FORM == 1 && a.pair_embd) {
             const float4 e = ld4_bf16(a.pair_embd, e1 + 4 * i);
             v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
         }
@@ -196,15 +206,19 @@ __global__ void __launch_bounds__(pre_norm_threads(MAXV), POST && MAXV == 2 ? 3 
         if (i >= n4) continue;
         const float4 g = *reinterpret_cast<const float4 *>(a.gain + 4 * i), v = x[j];
         st4<T>(reinterpret_cast<T *>(a.h) + row + 4 * i, make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w));
+        if (PAIR && a.h2) {
+            const float4 q = *reinterpret_cast<const float4 *>(a.gain2 + 4 * i);
+            st4<T>(reinterpret_cast<T *>(a.h2) + row + 4 * i, make_float4(v.x * r * q.x, v.y * r * q.y, v.z * r * q.z, v.w * r * q.w));
+        }
     }
 }
 
-template <class T, bool POST>
+template <class T, int FORM>
 static int pre_norm_t(const PreNormArgs &a, cudaStream_t s, bool pdl) {
     const int n4 = a.d_p / 4;
-    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1, POST>, dim3(a.n_tok), dim3(pre_norm_threads(1)), 0, s, pdl, a));
-    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2, POST>, dim3(a.n_tok), dim3(pre_norm_threads(2)), 0, s, pdl, a));
-    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4, POST>, dim3(a.n_tok), dim3(pre_norm_threads(4)), 0, s, pdl, a));
+    if (n4 <= 128) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 1, FORM>, dim3(a.n_tok), dim3(pre_norm_threads(1)), 0, s, pdl, a));
+    else if (n4 <= 1024) LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 2, FORM>, dim3(a.n_tok), dim3(pre_norm_threads(2)), 0, s, pdl, a));
+    else LCU_CHECK_CUDA(launch_kernel(pre_norm_kernel<T, 4, FORM>, dim3(a.n_tok), dim3(pre_norm_threads(4)), 0, s, pdl, a));
     return LCU_OK;
 }
 
@@ -213,8 +227,84 @@ int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl) {
     LCU_REQUIRE(a.d_p % 4 == 0 && a.d_p <= 16384, "pre_norm: width %d (a multiple of 4, at most 16384)", a.d_p);
     const bool post = a.post_gain || a.pair_embd || a.n_zero || a.top;
     LCU_REQUIRE(!post || !a.y_gain, "pre_norm: outputs normed one by one and as a sum");
-    if (post) return dt == LCU_F32 ? pre_norm_t<float, true>(a, s, pdl) : pre_norm_t<__nv_bfloat16, true>(a, s, pdl);
-    return dt == LCU_F32 ? pre_norm_t<float, false>(a, s, pdl) : pre_norm_t<__nv_bfloat16, false>(a, s, pdl);
+    if (a.h2 || a.ye_w || a.y_bias) {
+        LCU_REQUIRE(!a.post_gain && !a.pair_embd && !a.y_gain && (!a.h2 || a.h), "pre_norm: two norms ahead of sublayers, and norms on outputs or token pairs");
+        return dt == LCU_F32 ? pre_norm_t<float, 2>(a, s, pdl) : pre_norm_t<__nv_bfloat16, 2>(a, s, pdl);
+    }
+    if (post) return dt == LCU_F32 ? pre_norm_t<float, 1>(a, s, pdl) : pre_norm_t<__nv_bfloat16, 1>(a, s, pdl);
+    return dt == LCU_F32 ? pre_norm_t<float, 0>(a, s, pdl) : pre_norm_t<__nv_bfloat16, 0>(a, s, pdl);
+}
+
+// One block per token: a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e, z = row + bias.  MAXV float4 values of the row per
+// thread stay in registers between the passes; 0: any width, the row is read twice.
+template <class T, int MAXV>
+__global__ void __launch_bounds__(MAXV == 1 ? 128 : (MAXV == 2 ? 512 : 1024)) poly_norm_kernel(const PolyNormArgs a) {
+    grid_dep_launch();
+    __shared__ float2 part[32], part2[32];
+    const int t = blockIdx.x, n4 = a.ff_p / 4;
+    const float *z = a.z + (size_t)t * a.ff_p;
+    const float k1 = a.act[0], k2 = a.act[1], k3 = a.act[2], k0 = a.act[3];
+    grid_dep_wait();
+    auto load = [&](int i) {
+        float4 v = *reinterpret_cast<const float4 *>(z + 4 * i);
+        if (a.bias) {
+            const float4 b = *reinterpret_cast<const float4 *>(a.bias + 4 * i);
+            v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+        }
+        return v;
+    };
+    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    auto count = [&](const float4 &v) {  // padding is zero
+        const float4 q = make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w);
+        s1 += q.x + q.y + q.z + q.w;
+        s2 += dot4(q);
+        s3 += q.x * q.x * q.x + q.y * q.y * q.y + q.z * q.z * q.z + q.w * q.w * q.w;
+    };
+    float4 x[MAXV ? MAXV : 1];
+    if constexpr (MAXV > 0) {
+#pragma unroll
+        for (int j = 0; j < MAXV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            x[j] = i < n4 ? load(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            count(x[j]);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n4; i += blockDim.x) count(load(i));
+    }
+    const float2 s = block_sum2(s1, s2, part);
+    s3 = block_sum2(s3, 0.f, part2).x;
+    const float n = (float)a.ff, r1 = k1 / sqrtf(s.x / n + a.eps), r2 = k2 / sqrtf(s.y / n + a.eps), r3 = k3 / sqrtf(s3 / n + a.eps);
+    auto act = [&](float v, int i) { return i < a.ff ? fmaf(v, fmaf(v, fmaf(v, r3, r2), r1), k0) : 0.f; };
+    auto put = [&](const float4 &v, int i) {
+        st4<T>(reinterpret_cast<T *>(a.y) + (size_t)t * a.ff_p + 4 * i, make_float4(act(v.x, 4 * i), act(v.y, 4 * i + 1), act(v.z, 4 * i + 2), act(v.w, 4 * i + 3)));
+    };
+    if constexpr (MAXV > 0) {
+#pragma unroll
+        for (int j = 0; j < MAXV; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < n4) put(x[j], i);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n4; i += blockDim.x) put(load(i), i);
+    }
+}
+
+int op_poly_norm(const PolyNormArgs &a, int dt, cudaStream_t s, bool pdl) {
+    if (a.n_tok <= 0) return LCU_OK;
+    LCU_REQUIRE(a.ff_p % 4 == 0 && a.ff > 0 && a.ff <= a.ff_p, "poly_norm: width %d padded to %d", a.ff, a.ff_p);
+    const int n4 = a.ff_p / 4;
+    auto go = [&](auto kernel, int threads) -> int {
+        LCU_CHECK_CUDA(launch_kernel(kernel, dim3(a.n_tok), dim3(threads), 0, s, pdl, a));
+        return LCU_OK;
+    };
+    auto by_width = [&](auto t) -> int {
+        using T = decltype(t);
+        if (n4 <= 128) return go(poly_norm_kernel<T, 1>, 128);
+        if (n4 <= 1024) return go(poly_norm_kernel<T, 2>, 512);
+        if (n4 <= 4096) return go(poly_norm_kernel<T, 4>, 1024);
+        return go(poly_norm_kernel<T, 0>, 1024);
+    };
+    return dt == LCU_F32 ? by_width(float{}) : by_width(__nv_bfloat16{});
 }
 
 template <class T>

@@ -1,4 +1,5 @@
-// Layers of pre-norm models: x += mixer(norm(x)), x += ff(norm(x)), or with norms on the outputs too.  A mixer is softmax
+// Layers of pre-norm models: x += mixer(norm(x)), x += ff(norm(x)), or with norms on the outputs too, or both at once on one x with
+// a norm each.  A mixer is softmax
 // attention, a recurrent mixer (delta rule, state space duality, gated linear attention), or one of each side by side on the same
 // input, their outputs added.  One projection serves both; the feed-forward is one for all tokens or one of experts.  Rounds,
 // pages, state slots, head and sampling are those of every layered model.
@@ -38,9 +39,11 @@ struct PreNormRound {
         const float *y0 = nullptr, *y1 = nullptr, *y_gain = nullptr, *post_gain = nullptr;
         float scale0 = 1.f, scale1 = 1.f;
         int top = 0;  // rows of experts per token
+        const float *weights = nullptr, *bias = nullptr;  // on experts' rows; of the feed-forward's last matrix
+        const void *ff_in = nullptr;                      // what experts without matrices return
     };
-    // x after a sublayer's outputs, what comes ahead of the next one, and h, normed with `gain`
-    int residual(const Outputs &u, bool embed, const float *step, const float *gain, int n_zero = 0) {
+    // x after a sublayer's outputs, what comes ahead of the next one, and h, normed with `gain` (and h2 with `gain2`)
+    int residual(const Outputs &u, bool embed, const float *step, const float *gain, int n_zero = 0, const float *gain2 = nullptr) {
         PreNormArgs a{};
         const lcu_model_desc &d = c->desc;
         const bool start = !u.y0 && !u.top;
@@ -50,7 +53,8 @@ struct PreNormRound {
             cur ^= 1;
         }
         a.y[0] = u.y0; a.y[1] = u.y1; a.y_gain = u.y_gain; a.post_gain = u.post_gain; a.y_scale[0] = u.scale0; a.y_scale[1] = u.scale1;
-        if (u.top) { a.top = u.top; a.ye = S().ye; a.slot_of = moe_int(2); }
+        if (u.top) { a.top = u.top; a.ye = S().ye; a.slot_of = moe_int(2); a.ye_w = u.weights; a.ff_in = u.ff_in; }
+        a.y_bias = u.bias; a.gain2 = gain2; a.h2 = gain2 ? S().h2 : nullptr;
         if (embed || start) {
             const lcu_layer_desc &l = S().layers[0].d;
             a.embd = c->embd; a.tokens = reinterpret_cast<const uint32_t *>(D + r.L.tokens);
@@ -70,7 +74,8 @@ struct PreNormRound {
     int residual_into(int next, const Outputs &u) {
         if (next >= c->desc.n_layers) return residual(u, false, nullptr, nullptr);
         const StackLayer &Y = S().layers[next];
-        return residual(u, Y.d.add_embed, Y.d.add_step ? S().w[next].step : nullptr, S().w[Y.src].norm1);
+        const StackWeights &W = S().w[Y.src];
+        return residual(u, Y.d.add_embed, Y.d.add_step ? S().w[next].step : nullptr, W.norm1, Y.parallel() ? counters(Y) : 0, Y.parallel() ? W.norm2 : nullptr);
     }
 
     GqaArgs gqa(const StackLayer &Y, const StackWeights &W) const {
@@ -79,6 +84,11 @@ struct PreNormRound {
         a.heads = Y.d.heads; a.kv_heads = Y.d.kv_heads; a.dim = Y.d.dim; a.dim_p = Y.dim_p; a.v_dim = Y.d.v_dim; a.vdim_p = Y.vdim_p;
         a.bias = W.bias; a.own_kv = Y.own_kv(); a.qk_norm = Y.d.qk_norm; a.qk_gain = W.qk_gain; a.eps = c->desc.eps;
         a.rot_dims = Y.d.rot_dims; a.rot_adjacent = Y.d.rot_adjacent; a.rot = Y.rot; a.q = S().q;
+        a.vrot = Y.vrot; a.head_temp = W.head_temp; a.keep = Y.d.window ? Y.d.keep_first : 0; a.sink_score = W.sink;
+        if (Y.d.conv) {
+            a.conv = W.att_conv; a.taps = Y.d.conv; a.conv_state = S().conv_state + Y.conv_off * S().n_slots; a.conv_gen_stride = S().conv_gen;
+            a.req_first = i32(o.req_first); a.req_pos = i32(o.req_pos); a.req_slot = i32(o.req_slot);
+        }
         a.window = Y.d.window; a.sink = Y.d.sink; a.gate = Y.d.out_gate ? S().lat + Y.att_rows : nullptr;
         a.pool = c->pool; a.page_elems = c->geom.page_elems; a.c_off = Y.c_off; a.page_shift = c->geom.page_shift;
         a.tok_req = reinterpret_cast<const int32_t *>(D + r.L.tok_req); a.page_table = reinterpret_cast<const int32_t *>(D + r.L.page_table);
@@ -173,37 +183,41 @@ struct PreNormRound {
         return rc;
     }
 
-    // ---- feed-forward: h -> y (and rows of experts in ye)
+    // ---- feed-forward: h -> y (or rows of experts in ye)
     int *moe_int(int i) const { return S().moe_ints + (size_t)i * S().max_rows; }
     GluArgs glu(const StackLayer &Y, float limit) const { return GluArgs{limit, Y.d.glu_alpha, Y.d.glu_shift}; }
-    int dense_glu(const void *up, const void *down, int ff_p, const GluArgs &u) {
-        int rc = L.linear(up, S().d_p, 2 * ff_p, S().h, r.n_tok, S().act, ff_p, EPI_GLU, nullptr, PRO_NONE, nullptr, u);
-        return rc ? rc : L.linear(down, ff_p, S().d_p, S().act, r.n_tok, S().y, S().d_p, EPI_STORE_F32);
+    int dense_glu(const void *up, const void *down, int ff_p, const GluArgs &u, const void *h, float *y) {
+        int rc = L.linear(up, S().d_p, 2 * ff_p, h, r.n_tok, S().act, ff_p, EPI_GLU, nullptr, PRO_NONE, nullptr, u);
+        return rc ? rc : L.linear(down, ff_p, S().d_p, S().act, r.n_tok, y, S().d_p, EPI_STORE_F32);
     }
     bool small_experts() const { return c->dt != LCU_F32 && r.n_tok <= MOE_SMALL_ROUND; }
-    int experts(const StackLayer &Y, const StackWeights &W) {
+    // counters that a round's routing expects to be zero
+    int counters(const StackLayer &Y) const { return Y.d.experts && !small_experts() ? Y.d.experts : 0; }
+    int experts(const StackLayer &Y, const StackWeights &W, const void *h, float *y) {
         const int n = r.n_tok, d_p = S().d_p, rows = n * Y.d.top;
         const GluArgs u = glu(Y, Y.d.glu_limit), us = glu(Y, Y.d.shared_limit);
-        int rc = L.linear(W.router, d_p, Y.e_p, S().h, n, S().router, Y.e_p, EPI_STORE_F32);
+        int rc = L.linear(W.router, d_p, Y.e_p, h, n, S().router, Y.e_p, EPI_STORE_F32);
         MoeRoute m{};
         m.logits = S().router; m.n_tok = n; m.experts = Y.d.experts; m.experts_p = Y.e_p; m.top = Y.d.top;
+        m.softmax = Y.d.route_softmax; m.correction = W.correction; m.identity = Y.d.identity;
         m.expert = moe_int(0); m.place = moe_int(1); m.slot_of = moe_int(2); m.slot_tok = moe_int(3);
         m.weight = S().moe_w; m.slot_w = S().moe_slot_w; m.count = S().moe_count; m.tiles = S().moe_tiles;
-        m.h = S().h; m.xg = S().xg; m.d_p = d_p;
+        m.h = h; m.xg = S().xg; m.d_p = d_p;
+        const float *in_scale = Y.d.route_softmax ? nullptr : m.slot_w;  // weights on the inputs
         if (small_experts()) {
             m.max_tiles = rows < Y.d.experts ? rows : Y.d.experts; m.tile_rows = n;
             if (!rc) rc = done(moe_plan_launch(m, s, L.pdl));
             MoeProduct p{};
-            p.tiles = m.tiles; p.max_tiles = m.max_tiles; p.n_tok = n; p.shared = Y.d.shared_ff > 0; p.slot_w = m.slot_w; p.slot_tok = m.slot_tok;
+            p.tiles = m.tiles; p.max_tiles = m.max_tiles; p.n_tok = n; p.shared = Y.d.shared_ff > 0; p.slot_w = in_scale; p.slot_tok = m.slot_tok;
             p.up = 1; p.w = W.up; p.ws = W.shared_up; p.out = 2 * Y.ff_p; p.in = d_p; p.outs = 2 * Y.sff_p; p.ins = d_p;
-            p.x = p.xs = S().h; p.y = S().act_e; p.ys = S().act; p.glu = u; p.glus = us;
+            p.x = p.xs = h; p.y = S().act_e; p.ys = S().act; p.glu = u; p.glus = us;
             if (!rc) rc = done(moe_product_launch(p, s, L.pdl));
             p.up = 0; p.w = W.down; p.ws = W.shared_down; p.out = p.outs = d_p; p.in = Y.ff_p; p.ins = Y.sff_p;
-            p.x = S().act_e; p.xs = S().act; p.y = S().ye; p.ys = S().y;
+            p.x = S().act_e; p.xs = S().act; p.y = S().ye; p.ys = y;
             return rc ? rc : done(moe_product_launch(p, s, L.pdl));
         }
         // tiles as wide as an expert's share of the round
-        const int share = rows / Y.d.experts;
+        const int share = rows / (Y.d.experts + Y.d.identity);
         m.tile_rows = c->dt == LCU_F32 || share <= 64 ? 64 : (share <= 128 ? 128 : 256);
         m.max_tiles = moe_max_tiles(rows, Y.d.experts, m.tile_rows);
         if (!rc) rc = done(moe_route_launch(m, s, L.pdl));
@@ -213,24 +227,38 @@ struct PreNormRound {
                 LinearF32Args a{};
                 a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w; a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
                 a.n = rows; a.in = in; a.out = out; a.heads = 1; a.epilogue = epilogue; a.glu = u;
-                a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.row_scale = m.slot_w;
+                a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.row_scale = in_scale;
                 return done(linear_f32_launch(a, s));
             }
             GemvArgs a{};
             a.w = w; a.x = x; a.stride_x = in; a.n_tok = rows; a.in = in; a.out = out; a.epilogue = epilogue; a.y = y; a.stride_y = stride_y; a.glu = u;
-            a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.tile_rows = m.tile_rows; a.groups = Y.d.experts; a.row_scale = m.slot_w;
+            a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.tile_rows = m.tile_rows; a.groups = Y.d.experts; a.row_scale = in_scale;
             return done(gemm_tc_launch(a, c->dt, s, L.pdl));
         };
         if (!rc) rc = grouped(W.up, d_p, 2 * Y.ff_p, S().xg, S().act_e, Y.ff_p, EPI_GLU);
         if (!rc) rc = grouped(W.down, Y.ff_p, d_p, S().act_e, S().ye, d_p, EPI_STORE_F32);
-        if (!rc && Y.d.shared_ff) rc = dense_glu(W.shared_up, W.shared_down, Y.sff_p, us);
+        if (!rc && Y.d.shared_ff) rc = dense_glu(W.shared_up, W.shared_down, Y.sff_p, us, h, y);
         return rc;
     }
-    int feed_forward(const StackLayer &Y, const StackWeights &W) {
-        if (Y.d.experts) return experts(Y, W);
-        if (Y.glu()) return dense_glu(W.up, W.down, Y.ff_p, glu(Y, Y.d.glu_limit));
-        int rc = L.linear(W.up, S().d_p, Y.ff_p, S().h, r.n_tok, S().act, Y.ff_p, EPI_RELU2);
-        return rc ? rc : L.linear(W.down, Y.ff_p, S().d_p, S().act, r.n_tok, S().y, S().d_p, EPI_STORE_F32);
+    int feed_forward(const StackLayer &Y, const StackWeights &W, const void *h, float *y) {
+        if (Y.d.experts) return experts(Y, W, h, y);
+        if (Y.glu()) return dense_glu(W.up, W.down, Y.ff_p, glu(Y, Y.d.glu_limit), h, y);
+        int rc;
+        if (Y.poly()) {
+            rc = L.linear(W.up, S().d_p, Y.ff_p, h, r.n_tok, S().z, Y.ff_p, EPI_STORE_F32);
+            const PolyNormArgs a{S().z, W.up_bias, W.act, S().act, r.n_tok, Y.d.ff, Y.ff_p, c->desc.eps};
+            if (!rc) rc = done(op_poly_norm(a, c->dt, s, L.pdl));
+        } else {
+            rc = L.linear(W.up, S().d_p, Y.ff_p, h, r.n_tok, S().act, Y.ff_p, EPI_RELU2);
+        }
+        return rc ? rc : L.linear(W.down, Y.ff_p, S().d_p, S().act, r.n_tok, y, S().d_p, EPI_STORE_F32);
+    }
+    // outputs of a feed-forward, dense ones in y
+    void add_ff(Outputs &u, const StackLayer &Y, const StackWeights &W, const void *h) const {
+        u.bias = W.down_bias;
+        if (!Y.d.experts) return;
+        u.top = Y.d.top;
+        if (Y.d.route_softmax) { u.weights = S().moe_w; u.ff_in = h; }
     }
 
     int run() {
@@ -240,19 +268,25 @@ struct PreNormRound {
             const StackLayer &Y = S().layers[l];
             const StackWeights &W = S().w[Y.src];
             const bool both = Y.attention() && Y.recurrent();
-            rc = mixers(Y, W);
+            if (Y.parallel()) rc = feed_forward(Y, W, S().h2, S().y2);
+            if (!rc) rc = mixers(Y, W);
             if (rc) break;
             Outputs u;
             u.y0 = S().y; u.y1 = both ? S().y2 : nullptr; u.y_gain = both ? W.branch_norm : nullptr; u.post_gain = W.post1;
             if (both && Y.d.post_norm) { u.scale0 = Y.d.out_scale; u.scale1 = Y.d.out_scale2; }
-            if (!Y.has_ff()) {
+            if (Y.parallel()) {
+                if (!Y.d.experts) u.y1 = S().y2;
+                add_ff(u, Y, W, S().h2);
+            }
+            if (!Y.has_ff() || Y.parallel()) {
                 rc = residual_into(l + 1, u);
                 continue;
             }
-            rc = residual(u, false, nullptr, W.norm2, Y.d.experts && !small_experts() ? Y.d.experts : 0);
-            if (!rc) rc = feed_forward(Y, W);
+            rc = residual(u, false, nullptr, W.norm2, counters(Y));
+            if (!rc) rc = feed_forward(Y, W, S().h, S().y);
             u = Outputs{};
-            u.y0 = Y.d.experts && !Y.d.shared_ff ? nullptr : S().y; u.top = Y.d.experts ? Y.d.top : 0; u.post_gain = W.post2;
+            u.y0 = Y.d.experts && !Y.d.shared_ff ? nullptr : S().y; u.post_gain = W.post2;
+            add_ff(u, Y, W, S().h);
             if (!rc) rc = residual_into(l + 1, u);
         }
         c->x = S().x[cur];

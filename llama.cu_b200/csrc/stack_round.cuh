@@ -39,6 +39,7 @@ struct Launcher {
     int *count;
     bool pdl;
     bool weights_first = false;  // one-token GEMVs of this round request weights before activations
+    CapArgs cap{};               // of EPI_CAP and EPI_CAP_F32
 
     // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
     int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr,
@@ -48,12 +49,12 @@ struct Launcher {
             a.x = reinterpret_cast<const float *>(x); a.stride_x = in; a.w = w;
             a.y = reinterpret_cast<float *>(y); a.stride_y = stride_y;
             a.n = n; a.in = in; a.out = out; a.heads = 1;
-            a.epilogue = epilogue == EPI_STORE ? EPI_STORE_F32 : epilogue;
-            a.act_pq = act_pq; a.glu = glu;
+            a.epilogue = epilogue == EPI_STORE ? EPI_STORE_F32 : epilogue == EPI_CAP ? EPI_CAP_F32 : epilogue;
+            a.act_pq = act_pq; a.glu = glu; a.cap = cap;
             ++*count;
             return linear_f32_launch(a, s);
         }
-        const size_t yb = epilogue == EPI_STORE_F32 ? 4 : 2;
+        const size_t yb = epilogue == EPI_STORE_F32 || epilogue == EPI_CAP_F32 ? 4 : 2;
         // three and four tokens: the GEMV streams small matrices faster, the tcgen05 kernels large ones (4 sequences at 8192, per
         // 8-layer step: width 4096 1.88 -> 1.55 ms, width 2048 0.88 -> 1.04 ms)
         const bool tc = n > 4 || (n > 2 && (tuning().stack_tc == 2 || (tuning().stack_tc == 1 && (long)in * out >= (32l << 20))));
@@ -64,7 +65,7 @@ struct Launcher {
             a.w = w;
             a.x = reinterpret_cast<const unsigned char *>(x) + (size_t)t0 * in * 2;
             a.stride_x = in; a.n_tok = nt; a.in = in; a.out = out;
-            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq; a.glu = glu;
+            a.prologue = PRO_NONE; a.epilogue = epilogue; a.act_pq = act_pq; a.glu = glu; a.cap = cap;
             a.y = reinterpret_cast<unsigned char *>(y) + (size_t)t0 * stride_y * yb;
             a.stride_y = stride_y;
             if (pro) {  // one launch (at most two tokens): the prologue's rows, and the tokens' places in the cache

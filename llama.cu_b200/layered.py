@@ -11,10 +11,11 @@ from dataclasses import dataclass
 
 import numpy as np
 
-from . import (ACT_GLU, ACT_RELU2, ACT_XIELU, BF16, F32, MIX_ATTENTION, MIX_DELTA, MIX_GLA, MIX_LATENT, MIX_SSD, W_ATT_OUT, W_BRANCH_NORM,
-               W_CONV, W_CONV_BIAS, W_DELTA_DECAY, W_DELTA_NORM, W_DELTA_OUT, W_EMBD, W_FF_DOWN, W_GATE_MAP, W_KV_NORM, W_LAT_IN, W_LAT_OUT,
-               W_LM_HEAD, W_MIX_BIAS, W_MIX_IN, W_NORM1, W_NORM2, W_OUT_NORM, W_PAIR_EMBD, W_POST1, W_POST2, W_Q_NORM, W_QK_GAIN, W_ROUTER,
-               W_SCALARS, W_SHARED_DOWN, W_SHARED_UP, W_SHIFT, W_STEP, W_UKT, W_UKV, W_UP, W_UQ, LayerDesc, ModelDesc)
+from . import (ACT_GLU, ACT_POLYNORM, ACT_RELU2, ACT_XIELU, BF16, F32, MIX_ATTENTION, MIX_DELTA, MIX_GLA, MIX_LATENT, MIX_SSD, W_ACT, W_ATT_CONV,
+               W_ATT_OUT, W_BRANCH_NORM, W_CONV, W_CONV_BIAS, W_CORRECTION, W_DELTA_DECAY, W_DELTA_NORM, W_DELTA_OUT, W_DOWN_BIAS, W_EMBD,
+               W_FF_DOWN, W_GATE_MAP, W_HEAD_TEMP, W_KV_NORM, W_LAT_IN, W_LAT_OUT, W_LM_HEAD, W_MIX_BIAS, W_MIX_IN, W_NORM1, W_NORM2, W_OUT_NORM,
+               W_PAIR_EMBD, W_POST1, W_POST2, W_Q_NORM, W_QK_GAIN, W_ROUTER, W_SCALARS, W_SHARED_DOWN, W_SHARED_UP, W_SHIFT, W_SINK, W_STEP, W_UKT,
+               W_UKV, W_UP, W_UP_BIAS, W_UQ, LayerDesc, ModelDesc)
 
 
 def pad_to(v, m):
@@ -62,7 +63,9 @@ class Rotary:
 @dataclass(frozen=True)
 class AttentionMixer:
     """Softmax attention with grouped heads, optionally rotary positions, biases, normalised queries and keys (qk_norm: see
-    lcu_layer_desc), a sliding window, a sink in the softmax, a gate per head, another layer's keys and values."""
+    lcu_layer_desc), a sliding window that may keep the first tokens, a sink in the softmax (1: of score 0, 2: of a learned score per
+    head), a gate per head, another layer's keys and values, convolutions over time behind the projections (`conv` taps), a factor
+    on the scores per head, values rotated by their positions."""
     heads: int
     kv_heads: int
     dim: int
@@ -72,9 +75,13 @@ class AttentionMixer:
     bias: bool = True
     qk_norm: int = 1
     window: int = 0
-    sink: bool = False
+    sink: int = 0
     out_gate: bool = False
     kv_from: int = -1  # the layer whose keys and values are used, -1: its own
+    keep_first: int = 0
+    conv: int = 0
+    head_temp: bool = False
+    rot_values: bool = False
 
     def describe(self, o):
         o.mixer |= MIX_ATTENTION
@@ -84,6 +91,7 @@ class AttentionMixer:
         if r is not None:
             o.rot_dims, o.rot_base, o.rot_factor, o.rot_original, o.rot_fast, o.rot_slow = r.dims, r.base, r.factor, r.original, r.fast, r.slow
             o.rot_adjacent = int(r.adjacent)
+        o.keep_first, o.conv, o.head_temp, o.rot_values = self.keep_first, self.conv, int(self.head_temp), int(self.rot_values)
 
     @property
     def own_kv_heads(self):
@@ -93,7 +101,7 @@ class AttentionMixer:
         return self.own_kv_heads * (pad_to(self.dim, 16) + pad_to(self.v_dim, 16))
 
     def state_bytes(self):
-        return 0
+        return 0  # the convolutions' inputs are a few rows
 
     def weights(self, d):
         return d * ((self.heads + self.own_kv_heads) * (self.dim + self.v_dim) + (self.heads if self.out_gate else 0))
@@ -209,7 +217,8 @@ class ParallelMixer:
 class GluFf:
     """Gated feed-forward: g = min(W_gate x, limit), u = clamp(W_up x, +-limit), W_down (g sigmoid(alpha g) (u + shift)).  With
     `experts` > 0 every token uses `top` of that many, their inputs scaled by the sigmoids of their router logits, and the shared
-    one (width `shared`, 0: none)."""
+    one (width `shared`, 0: none).  softmax: scores are a softmax over all experts and `identity` more that return their input;
+    corrected scores choose, the chosen scores divided by their sum weigh the outputs."""
     ff: int
     limit: float
     alpha: float = 1.0
@@ -218,14 +227,30 @@ class GluFf:
     top: int = 0
     shared: int = 0
     shared_limit: float = 0.0
+    softmax: bool = False
+    identity: int = 0
 
     def describe(self, o):
         o.ff, o.ff_act, o.experts, o.top, o.shared_ff = self.ff, ACT_GLU, self.experts, self.top, self.shared
         o.glu_limit, o.shared_limit, o.glu_alpha, o.glu_shift = self.limit, self.shared_limit, self.alpha, self.shift
+        o.route_softmax, o.identity = int(self.softmax), self.identity
 
     def weights(self, d):
         """Weights one token meets."""
-        return d * (3 * (self.ff * (self.top or 1) + self.shared) + self.experts)
+        used = self.top * self.experts / (self.experts + self.identity) if self.experts else 1
+        return d * (3 * (self.ff * used + self.shared) + self.experts + self.identity)
+
+
+@dataclass(frozen=True)
+class PolyNormFf:
+    """W_down (a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e) with z = W_up x, both with biases."""
+    ff: int
+
+    def describe(self, o):
+        o.ff, o.ff_act, o.ff_bias = self.ff, ACT_POLYNORM, 1
+
+    def weights(self, d):
+        return 2 * self.ff * d
 
 
 @dataclass(frozen=True)
@@ -240,7 +265,7 @@ class PairEmbedding:
 class LayerConfig:
     """One layer as it runs; a layer that runs several times is listed several times (`weights_of`)."""
     mixer: object
-    ff: object = 0  # width, 0: no feed-forward; or a GluFf
+    ff: object = 0  # width, 0: no feed-forward; or a GluFf or PolyNormFf
     token_shift: bool = True
     weights_of: int = -1
     act: int = ACT_XIELU
@@ -249,9 +274,10 @@ class LayerConfig:
     step: int = -1           # row of the table of vectors added ahead of the layer, -1: none
     file_layer: int = -1     # the layer's number in the model file, -1: its place in the list
     post_norm: bool = False  # pre-norm layers: norms on the sublayers' outputs too
+    parallel_ff: bool = False  # pre-norm layers: mixer and feed-forward read the same x, each through a norm of its own
 
     def ff_weights(self, d):
-        return self.ff.weights(d) if isinstance(self.ff, GluFf) else 2 * self.ff * d
+        return 2 * self.ff * d if isinstance(self.ff, int) else self.ff.weights(d)
 
 
 @dataclass(frozen=True)
@@ -266,6 +292,8 @@ class LayeredConfig:
     arch: str = "Zefedra"  # key of `architectures()`
     embed_scale: float = 1.0
     pairs: PairEmbedding = None
+    logit_scale: float = 1.0
+    logit_cap: float = 0.0  # logits = cap tanh(scale head x / cap), 0: not capped
 
     @property
     def family(self):
@@ -291,12 +319,13 @@ class LayeredConfig:
         for o, l in zip(out, self.layers):
             l.mixer.describe(o)
             o.token_shift, o.weights_of = int(l.token_shift), l.weights_of
-            if isinstance(l.ff, GluFf):
-                l.ff.describe(o)
-            else:
+            if isinstance(l.ff, int):
                 o.ff, o.ff_act = l.ff, l.act
+            else:
+                l.ff.describe(o)
+            o.parallel_ff = int(l.parallel_ff)
             o.pre_norm, o.post_norm, o.add_embed, o.add_step = int(l.pre_norm), int(l.post_norm), int(l.add_embed), int(l.step >= 0)
-        out[0].embed_scale = self.embed_scale
+        out[0].embed_scale, out[0].logit_scale, out[0].logit_cap = self.embed_scale, self.logit_scale, self.logit_cap
         if self.pairs:
             b = self.pairs.buckets
             out[0].pair_buckets, out[0].pair_prev, out[0].pair_cur = b, self.pairs.prev % b, self.pairs.cur % b
@@ -359,9 +388,9 @@ def attention_rows(m, d, q, k=None, v=None, g=None):
     return rows + ([_pad(g, pad_to(m.heads, 8), wp)] if m.out_gate else [])
 
 
-def pack_attention(m, d, o, bias=None, gains=None):
-    """[(kind, tensor)] of an AttentionMixer besides its input projection; bias: (q, k, v), or (q,) without own keys; gains: the
-    weights of the norms of q and k, one head's or all heads' ((q,) without own keys)."""
+def pack_attention(m, d, o, bias=None, gains=None, conv=None, sink=None, temp=None):
+    """[(kind, tensor)] of an AttentionMixer besides its input projection; bias, conv: of (q, k, v), or (q,) without own keys; gains:
+    the weights of the norms of q and k, one head's or all heads' ((q,) without own keys); sink, temp: a number per head."""
     import torch
     dp, vp = pad_to(m.dim, 16), pad_to(m.v_dim, 16)
     out = [(W_ATT_OUT, _out_columns(o, d, m.heads, m.v_dim, vp))]
@@ -372,7 +401,11 @@ def pack_attention(m, d, o, bias=None, gains=None):
         out.append((W_QK_GAIN, torch.cat([_pad(g.float(), dp) for g in gains])))
     if m.qk_norm == 3:
         out.append((W_QK_GAIN, torch.cat([_pad_heads(g.float(), n, m.dim, dp) for g, n in zip(gains, (m.heads, m.kv_heads))])))
-    return out
+    if m.conv:
+        taps = torch.cat([_pad_heads(c.float(), n, x, y) for c, n, x, y in
+                          zip(conv, (m.heads, m.kv_heads, m.kv_heads), (m.dim, m.dim, m.v_dim), (dp, dp, vp))])
+        out.append((W_ATT_CONV, taps.T.contiguous()))
+    return out + [(k, t.float().contiguous()) for k, t in ((W_SINK, sink), (W_HEAD_TEMP, temp)) if t is not None]
 
 
 def delta_rows(m, d, q, k, v, g, b, a):
@@ -437,14 +470,17 @@ def glu_rows(gate, up, d, ff):
     return torch.stack([_pad(gate, fp, wp), _pad(up, fp, wp)], 1).reshape(2 * fp, wp)
 
 
-def pack_experts(f, d, router, experts, shared=None):
+def pack_experts(f, d, router, experts, shared=None, correction=None):
     """[(kind, tensor)] of a GluFf of experts; experts: an iterable of (gate, up, down), shared: one of them or None."""
     import torch
     wp, fp = pad_to(d, 64), pad_to(f.ff, 64)
     ups, downs = torch.empty(f.experts, 2 * fp, wp, dtype=router.dtype, device=router.device), torch.empty(f.experts, wp, fp, dtype=router.dtype, device=router.device)
     for i, (gate, up, down) in enumerate(experts):
         ups[i], downs[i] = glu_rows(gate, up, d, f.ff), _pad(down, wp, fp)
-    out = [(W_ROUTER, _pad(router, pad_to(f.experts, 8), wp)), (W_UP, ups), (W_FF_DOWN, downs)]
+    n = pad_to(f.experts + f.identity, 8)
+    out = [(W_ROUTER, _pad(router, n, wp)), (W_UP, ups), (W_FF_DOWN, downs)]
+    if f.softmax:
+        out.append((W_CORRECTION, _pad(correction.float(), n)))
     if f.shared:
         out += [(W_SHARED_UP, glu_rows(*shared[:2], d, f.shared)), (W_SHARED_DOWN, _pad(shared[2], wp, pad_to(f.shared, 64)))]
     return out
@@ -455,7 +491,14 @@ def pack_glu(f, d, gate, up, down):
     return [(W_UP, glu_rows(gate, up, d, f.ff)), (W_FF_DOWN, _pad(down, pad_to(d, 64), pad_to(f.ff, 64)))]
 
 
-def pack_norms(d, norm1, post1, norm2=None, post2=None):
+def pack_poly(f, d, up, up_bias, down, down_bias, act):
+    """[(kind, tensor)] of a PolyNormFf."""
+    fp, wp = pad_to(f.ff, 64), pad_to(d, 64)
+    return [(W_UP, _pad(up, fp, wp)), (W_FF_DOWN, _pad(down, wp, fp)), (W_UP_BIAS, _pad(up_bias.float(), fp)), (W_DOWN_BIAS, _pad(down_bias.float(), wp)),
+            (W_ACT, act.float().contiguous())]
+
+
+def pack_norms(d, norm1, post1=None, norm2=None, post2=None):
     """[(kind, tensor)] of the gains (f32) of a layer with norms ahead of its sublayers and on their outputs."""
     return [(k, _pad(g.float(), pad_to(d, 64))) for k, g in ((W_NORM1, norm1), (W_POST1, post1), (W_NORM2, norm2), (W_POST2, post2)) if g is not None]
 
@@ -535,8 +578,8 @@ class Tensors(dict):
 def architectures():
     """config.json's "architecture" -> module with read_config(dict, shapes) and pack(cfg, Tensors); shapes: {name: shape} of the
     model file, for sizes that the configuration does not name."""
-    from . import galarax, mupuvik, zefedra
-    return {"Galarax": galarax, "Mupuvik": mupuvik, "Zefedra": zefedra}
+    from . import galarax, gunulorn, mupuvik, zefedra
+    return {"Galarax": galarax, "Gunulorn": gunulorn, "Mupuvik": mupuvik, "Zefedra": zefedra}
 
 
 def load_pretrained(path, act_dtype=BF16, device=0, nctx=None, kv_tokens=None, page_tokens=0, max_tokens=0, max_seqs=0):
