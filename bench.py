@@ -41,6 +41,8 @@ WORKLOADS = {
     "galarax8b-bf16-b32": ("galarax8b", 32, (128, 1024)),
     "mupuvik8b-bf16-b1": ("mupuvik8b", 1, (128, 128)),
     "mupuvik8b-bf16-b32": ("mupuvik8b", 32, (128, 1024)),
+    "gunulorn8b-bf16-b1": ("gunulorn8b", 1, (128, 128)),
+    "gunulorn8b-bf16-b32": ("gunulorn8b", 32, (128, 1024)),
     "tiny-f16-b1": ("tiny", 1, (16, 16)),
 }
 DEFAULT_WORKLOAD = "llama8b-f16-b1"
@@ -479,8 +481,8 @@ def run_decode(L, env, cfg, batch, prompt_range, steps, warmup, want_e2e=True, w
 
 # --family-bench: sizes at which the layered families run beside the LLaMA shape of equal width and feed-forward, cut to
 # `layers` layers and a vocabulary of 32000 (name, configs, layers)
-FAMILY_SIZES = [("8b", ("mupuvik8b", "galarax8b", "zefedra8b", "llama8b"), 8),
-                ("1b", ("mupuvik1b", "galarax1b", "zefedra1b", "llama1b"), 8)]
+FAMILY_SIZES = [("8b", ("gunulorn8b", "mupuvik8b", "galarax8b", "zefedra8b", "llama8b"), 8),
+                ("1b", ("gunulorn1b", "mupuvik1b", "galarax1b", "zefedra1b", "llama1b"), 8)]
 FAMILY_PREFILL = (2048, 8192)                            # prompt lengths
 FAMILY_DECODE = ((1, 1024), (32, 1024), (32, 4096), (4, 8192))  # (sequences, context)
 

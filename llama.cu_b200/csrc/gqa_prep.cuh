@@ -168,6 +168,83 @@ __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item
     }
 }
 
+// Large rounds of layers with these steps alone: rotation of neighbouring pairs, rotated values, factors per head, convolutions of
+// at most four taps.  A warp takes one head of RUN tokens in a row and holds the rows its convolution needs; every row is requested
+// before the first is used.  TAPS 0: none.
+constexpr int GQA_RUN = 4;
+__host__ __device__ __forceinline__ bool gqa_prep_runs(const GqaArgs &a) {
+    return !a.bias && !a.qk_norm && (a.rot_dims == 0 || a.rot_adjacent) && (!a.conv || a.taps <= 4);
+}
+template <class T, int TAPS>
+__device__ __forceinline__ void gqa_prep_run(const GqaArgs &a, int t0, int item, int lane) {
+    constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;
+    const bool is_v = item >= a.heads + a.kv_heads, is_q = item < a.heads;
+    const int size_p = is_v ? a.vdim_p : a.dim_p;
+    const int head = is_q ? item : (is_v ? item - a.heads - a.kv_heads : item - a.heads);
+    const int off = is_q ? head * a.dim_p : (is_v ? (a.heads + a.kv_heads) * a.dim_p + head * a.vdim_p : (a.heads + head) * a.dim_p);
+    const float2 *rot = is_v ? a.vrot : a.rot;
+    const int turned = is_v ? (a.vrot ? a.v_dim : 0) : a.rot_dims;
+    const float temp = is_q && a.head_temp ? a.head_temp[head] : 1.f;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int d = 4 * lane; d < size_p; d += 128) {
+        float4 x[BACK + GQA_RUN], w[TAPS ? TAPS : 1];
+#pragma unroll
+        for (int i = 0; i < BACK + GQA_RUN; ++i) {
+            const int t = t0 + i - BACK;
+            x[i] = t >= 0 && t < a.n_tok ? *reinterpret_cast<const float4 *>(a.lat + (size_t)t * a.stride + off + d) : zero;
+        }
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const float4 *>(a.conv + (size_t)j * a.channels() + off + d);
+#pragma unroll
+        for (int i = 0; i < GQA_RUN; ++i) {
+            const int t = t0 + i;
+            if (t >= a.n_tok) break;
+            const int p = (int)a.pos[t], r = a.tok_req[t];
+            float4 y = x[BACK + i];
+            if constexpr (TAPS > 0) {
+                const int before = t - a.req_first[r];  // tokens of the portion before this one
+                float4 u[TAPS];                         // inputs of the taps
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) u[j] = x[i + j];
+                const bool last = TAPS > 1 && t + 1 == a.req_first[r + 1];
+                if (TAPS > 1 && (before < BACK || last)) {
+                    const int sg = a.req_slot[r];
+                    const size_t row = (size_t)(sg >> 1) * BACK * a.channels() + off + d;
+                    const float *in = a.conv_state + (size_t)(sg & 1) * a.conv_gen_stride + row;
+                    float *out = a.conv_state + (size_t)((sg & 1) ^ 1) * a.conv_gen_stride + row;
+#pragma unroll
+                    for (int j = 0; j < BACK; ++j) {
+                        const int back = BACK - j;
+                        if (back > before) u[j] = back > p ? zero : *reinterpret_cast<const float4 *>(in + (size_t)(before + j) * a.channels());
+                    }
+                    if (last)
+#pragma unroll
+                        for (int j = 0; j < BACK; ++j) *reinterpret_cast<float4 *>(out + (size_t)j * a.channels()) = u[j + 1];
+                }
+                y = zero;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    y.x = fmaf(u[j].x, w[j].x, y.x); y.y = fmaf(u[j].y, w[j].y, y.y);
+                    y.z = fmaf(u[j].z, w[j].z, y.z); y.w = fmaf(u[j].w, w[j].w, y.w);
+                }
+            }
+            if (d < turned) {  // two pairs
+                const float2 *cs = rot + (size_t)p * (turned >> 1) + (d >> 1);
+                const float2 c0 = cs[0], c1 = d + 2 < turned ? cs[1] : make_float2(1.f, 0.f);
+                y = make_float4(y.x * c0.x - y.y * c0.y, y.y * c0.x + y.x * c0.y, y.z * c1.x - y.w * c1.y, y.w * c1.x + y.z * c1.y);
+            }
+            T *dst;
+            if (is_q) dst = reinterpret_cast<T *>(a.q) + ((size_t)t * a.heads + head) * a.dim_p;
+            else {
+                const int page = a.page_table[(size_t)r * a.pt_stride + (p >> a.page_shift)];
+                const size_t row = ((size_t)head << a.page_shift) + (p & ((1 << a.page_shift) - 1));
+                dst = reinterpret_cast<T *>(a.pool) + (size_t)page * a.page_elems + (is_v ? a.v_off() : a.c_off) + row * size_p;
+            }
+            st4<T>(dst + d, make_float4(y.x * temp, y.y * temp, y.z * temp, y.w * temp));
+        }
+    }
+}
+
 template <class T>
 __device__ __forceinline__ void gqa_prep_any(const GqaArgs &a, int t, int item0, int item1) {
     if (gqa_prep_wide(a)) gqa_prep_block<T, GQA_PREP_WIDE>(a, t, item0, item1);

@@ -9,17 +9,26 @@ namespace {
 
 typedef __nv_bfloat16 bf16;
 
-// The k-th largest scores z(expert) of a token, one warp: calls put(k, expert, score) on every lane.  Equal ones: the lower index first.
-template <class Z, class F>
+// The k-th largest scores z(expert) of a token, one warp: calls put(k, expert, score) on every lane.  Equal ones: the lower index
+// first.  Scores of up to 32 PER experts are asked for once.
+template <int PER, class Z, class F>
 __device__ __forceinline__ void top_experts(const Z &z, int n, int top, int lane, const F &put) {
-    float last = INFINITY;
+    float last = INFINITY, own[PER ? PER : 1];
     int last_e = -1;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) own[j] = lane + 32 * j < n ? z(lane + 32 * j) : 0.f;
     for (int k = 0; k < top; ++k) {
         float v = -INFINITY;
         int e = n;
-        for (int i = lane; i < n; i += 32) {
-            const float x = z(i);
+        auto look = [&](int i, float x) {
             if ((x < last || (x == last && i > last_e)) && (x > v || e == n)) { v = x; e = i; }
+        };
+        if constexpr (PER > 0) {
+#pragma unroll
+            for (int j = 0; j < PER; ++j)
+                if (lane + 32 * j < n) look(lane + 32 * j, own[j]);
+        } else {
+            for (int i = lane; i < n; i += 32) look(i, z(i));
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -35,14 +44,14 @@ __device__ __forceinline__ void top_experts(const Z &z, int n, int top, int lane
 }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 
-// Experts and weights of token t, one warp; put(k, expert) on lane 0.
-template <class F>
-__device__ __forceinline__ void route_token(const MoeRoute &a, int t, int lane, const F &put) {
+// Experts and weights of token t, one warp; put(k, expert) on lane 0.  PER: as above, 0: any number of experts.
+template <int PER, class F>
+__device__ __forceinline__ void route_token_n(const MoeRoute &a, int t, int lane, const F &put) {
     const float *z = a.logits + (size_t)t * a.experts_p;
     float *weight = a.weight + (size_t)t * a.top;
     const int n = a.experts + a.identity;
     if (!a.softmax) {
-        top_experts([&](int e) { return z[e]; }, n, a.top, lane, [&](int k, int e, float v) {
+        top_experts<PER>([&](int e) { return z[e]; }, n, a.top, lane, [&](int k, int e, float v) {
             if (lane == 0) {
                 put(k, e);
                 weight[k] = sigmoid_f(v);
@@ -50,14 +59,34 @@ __device__ __forceinline__ void route_token(const MoeRoute &a, int t, int lane, 
         });
         return;
     }
-    float m = -INFINITY, sum = 0.f, chosen = 0.f;
-    for (int e = lane; e < n; e += 32) m = fmaxf(m, z[e]);
+    float m = -INFINITY, sum = 0.f, chosen = 0.f, own[PER ? PER : 1];
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        own[j] = lane + 32 * j < n ? z[lane + 32 * j] : -INFINITY;
+        m = fmaxf(m, own[j]);
+    }
+    if constexpr (PER == 0)
+        for (int e = lane; e < n; e += 32) m = fmaxf(m, z[e]);
     m = warp_max(m);
-    for (int e = lane; e < n; e += 32) sum += expf(z[e] - m);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        own[j] = expf(own[j] - m);
+        sum += own[j];
+    }
+    if constexpr (PER == 0)
+        for (int e = lane; e < n; e += 32) sum += expf(z[e] - m);
     sum = warp_sum(sum);
-    auto score = [&](int e) { return expf(z[e] - m) / sum; };
-    top_experts([&](int e) { return score(e) + a.correction[e]; }, n, a.top, lane, [&](int k, int e, float) {
-        const float s = score(e);
+    auto score = [&](int e) {  // of this lane's expert e
+        if constexpr (PER > 0) {
+            float s = own[0];
+#pragma unroll
+            for (int j = 1; j < PER; ++j) s = e >= 32 * j ? own[j] : s;
+            return s / sum;
+        }
+        return expf(z[e] - m) / sum;
+    };
+    top_experts<PER>([&](int e) { return score(e) + a.correction[e]; }, n, a.top, lane, [&](int k, int e, float) {
+        const float s = PER > 0 ? __shfl_sync(0xffffffffu, score((e & ~31) + lane), e & 31) : score(e);
         chosen += s;
         if (lane == 0) {
             put(k, e);
@@ -66,6 +95,13 @@ __device__ __forceinline__ void route_token(const MoeRoute &a, int t, int lane, 
     });
     __syncwarp();
     for (int k = lane; k < a.top; k += 32) weight[k] /= chosen + 1e-20f;
+}
+template <class F>
+__device__ __forceinline__ void route_token(const MoeRoute &a, int t, int lane, const F &put) {
+    const int n = a.experts + a.identity;
+    if (n <= 32) route_token_n<1>(a, t, lane, put);
+    else if (n <= 128) route_token_n<4>(a, t, lane, put);
+    else route_token_n<0>(a, t, lane, put);
 }
 
 // Exclusive sums of count[0..n) into first, and of (count + per - 1) / per into tile0; one warp; returns the sums of all.

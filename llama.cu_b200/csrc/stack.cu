@@ -292,6 +292,7 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     const size_t R = S->max_rows, o_lt = reserve((size_t)2 * S->n_slots * 4), o_ro = reserve(T * max_ep * 4), o_ye = reserve(R * S->d_p * 4), o_mi = reserve(R * 16), o_mw = reserve(R * 8),
                  o_mc = reserve((size_t)S->max_experts * 4), o_mt = reserve((size_t)S->n_tiles * 16), o_xg = reserve(R * S->d_p * eb), o_ae = reserve(R * max_eff * eb);
     const size_t o_h2 = reserve(any_parallel ? T * S->d_p * eb : 0), o_z = reserve(T * max_z * 4);
+    const size_t o_sw = reserve(any_parallel ? c->sk_ws_bytes : 0), o_st = reserve(any_parallel ? 4096 * sizeof(unsigned) : 0);
     LCU_CHECK_CUDA(cudaMalloc(&S->arena, total));
     LCU_CHECK_CUDA(cudaMemset(S->arena, 0, total));  // pads of att (columns past the heads) stay zero from here on
     unsigned char *p = reinterpret_cast<unsigned char *>(S->arena);
@@ -312,6 +313,12 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->moe_tiles = reinterpret_cast<int4 *>(p + o_mt); S->xg = p + o_xg; S->act_e = p + o_ae;
 
     S->h2 = p + o_h2; S->z = reinterpret_cast<float *>(p + o_z);
+    S->side_ws = p + o_sw; S->side_tickets = reinterpret_cast<unsigned *>(p + o_st);
+    if (any_parallel) {
+        LCU_CHECK_CUDA(cudaStreamCreateWithFlags(&S->side, cudaStreamNonBlocking));
+        LCU_CHECK_CUDA(cudaEventCreateWithFlags(&S->fork, cudaEventDisableTiming));
+        LCU_CHECK_CUDA(cudaEventCreateWithFlags(&S->join, cudaEventDisableTiming));
+    }
 
     // every kernel variant a round can launch
     if (S->pre_norm) {
@@ -361,6 +368,9 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
 void stack_destroy(lcu_ctx *c) {
     if (!c->stack) return;
     if (c->stack->arena) cudaFree(c->stack->arena);
+    if (c->stack->side) cudaStreamDestroy(c->stack->side);
+    if (c->stack->fork) cudaEventDestroy(c->stack->fork);
+    if (c->stack->join) cudaEventDestroy(c->stack->join);
     for (const Stack::RotTable &t : c->stack->rot_tables) cudaFree(t.dev);
     delete c->stack;
     c->stack = nullptr;

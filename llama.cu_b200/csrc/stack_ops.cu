@@ -238,7 +238,7 @@ int op_pre_norm(const PreNormArgs &a, int dt, cudaStream_t s, bool pdl) {
 // One block per token: a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e, z = row + bias.  MAXV float4 values of the row per
 // thread stay in registers between the passes; 0: any width, the row is read twice.
 template <class T, int MAXV>
-__global__ void __launch_bounds__(MAXV == 1 ? 128 : (MAXV == 2 ? 512 : 1024)) poly_norm_kernel(const PolyNormArgs a) {
+__global__ void __launch_bounds__(MAXV == 1 ? 128 : 512, MAXV == 1 ? 8 : (MAXV == 8 ? 2 : 3)) poly_norm_kernel(const PolyNormArgs a) {
     grid_dep_launch();
     __shared__ float2 part[32], part2[32];
     const int t = blockIdx.x, n4 = a.ff_p / 4;
@@ -301,8 +301,9 @@ int op_poly_norm(const PolyNormArgs &a, int dt, cudaStream_t s, bool pdl) {
         using T = decltype(t);
         if (n4 <= 128) return go(poly_norm_kernel<T, 1>, 128);
         if (n4 <= 1024) return go(poly_norm_kernel<T, 2>, 512);
-        if (n4 <= 4096) return go(poly_norm_kernel<T, 4>, 1024);
-        return go(poly_norm_kernel<T, 0>, 1024);
+        if (n4 <= 2048) return go(poly_norm_kernel<T, 4>, 512);
+        if (n4 <= 4096) return go(poly_norm_kernel<T, 8>, 512);
+        return go(poly_norm_kernel<T, 0>, 512);
     };
     return dt == LCU_F32 ? by_width(float{}) : by_width(__nv_bfloat16{});
 }

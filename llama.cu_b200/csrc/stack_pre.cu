@@ -68,7 +68,7 @@ struct PreNormRound {
         }
         a.step = step; a.x_out = S().x[cur]; a.gain = gain; a.h = gain ? S().h : nullptr;
         a.zero = S().moe_count; a.n_zero = n_zero;
-        return done(op_pre_norm(a, c->dt, s, L.pdl));
+        return done(op_pre_norm(a, c->dt, s, L.dependent()));
     }
     // ... ahead of layer `next` (past the last one: the head reads x itself)
     int residual_into(int next, const Outputs &u) {
@@ -107,7 +107,7 @@ struct PreNormRound {
             LCU_REQUIRE(a.splits == 1 || cells * a.splits <= S().gqa_ctas, "step: %d attention partials do not fit", cells * a.splits);
             a.tickets = S().gqa_tickets;
             a.part_ml = S().gqa_part; a.part_o = S().gqa_part + (size_t)cells * a.splits * 32;
-            rc = done(gqa_short_launch(a, s, L.pdl));
+            rc = done(gqa_short_launch(a, s, L.dependent()));
         }
         if (!rc && q.n_long) {
             a.reqs = reinterpret_cast<const int4 *>(B + o.lreq); a.n_reqs = q.n_long; a.n_blocks = 0;
@@ -152,23 +152,23 @@ struct PreNormRound {
         if (Y.delta()) {
             DeltaArgs e{};
             recurrent(e, Y, W);
-            if (r.decode_only) return done(delta_decode_launch(e, attn, dt, s, L.pdl));
-            if (attn) rc = done(gqa_prep_launch(g, dt, s, L.pdl));
-            if (!rc) rc = done(delta_prep_launch(e, s, L.pdl));
-            if (!rc) rc = done(delta_scan_launch(e, s, L.pdl));
-            return rc ? rc : done(delta_out_launch(e, dt, s, L.pdl));
+            if (r.decode_only) return done(delta_decode_launch(e, attn, dt, s, L.dependent()));
+            if (attn) rc = done(gqa_prep_launch(g, dt, s, L.dependent()));
+            if (!rc) rc = done(delta_prep_launch(e, s, L.dependent()));
+            if (!rc) rc = done(delta_scan_launch(e, s, L.dependent()));
+            return rc ? rc : done(delta_out_launch(e, dt, s, L.dependent()));
         }
-        if (!Y.recurrent() || !r.decode_only) rc = attn ? done(gqa_prep_launch(g, dt, s, L.pdl)) : LCU_OK;
+        if (!Y.recurrent() || !r.decode_only) rc = attn ? done(gqa_prep_launch(g, dt, s, L.dependent())) : LCU_OK;
         if (rc || !Y.recurrent()) return rc;
         const ScanArgs e = scan(Y, W);
-        if (r.decode_only) rc = done(scan_step_launch(e, attn, dt, s, L.pdl));
-        else if (dt == LCU_F32) rc = done(scan_step_launch(e, nullptr, dt, s, L.pdl));
+        if (r.decode_only) rc = done(scan_step_launch(e, attn, dt, s, L.dependent()));
+        else if (dt == LCU_F32) rc = done(scan_step_launch(e, nullptr, dt, s, L.dependent()));
         else {
-            rc = done(scan_prep_launch(e, s, L.pdl));
-            if (!rc) rc = done(scan_launch(e, s, L.pdl));
-            if (!rc && Y.gla()) rc = done(delta_out_launch(e, dt, s, L.pdl));
+            rc = done(scan_prep_launch(e, s, L.dependent()));
+            if (!rc) rc = done(scan_launch(e, s, L.dependent()));
+            if (!rc && Y.gla()) rc = done(delta_out_launch(e, dt, s, L.dependent()));
         }
-        return rc || !Y.ssd() ? rc : done(scan_out_launch(e, dt, s, L.pdl));
+        return rc || !Y.ssd() ? rc : done(scan_out_launch(e, dt, s, L.dependent()));
     }
 
     // h -> outputs of the layer's mixers in y and y2
@@ -206,22 +206,22 @@ struct PreNormRound {
         const float *in_scale = Y.d.route_softmax ? nullptr : m.slot_w;  // weights on the inputs
         if (small_experts()) {
             m.max_tiles = rows < Y.d.experts ? rows : Y.d.experts; m.tile_rows = n;
-            if (!rc) rc = done(moe_plan_launch(m, s, L.pdl));
+            if (!rc) rc = done(moe_plan_launch(m, s, L.dependent()));
             MoeProduct p{};
             p.tiles = m.tiles; p.max_tiles = m.max_tiles; p.n_tok = n; p.shared = Y.d.shared_ff > 0; p.slot_w = in_scale; p.slot_tok = m.slot_tok;
             p.up = 1; p.w = W.up; p.ws = W.shared_up; p.out = 2 * Y.ff_p; p.in = d_p; p.outs = 2 * Y.sff_p; p.ins = d_p;
             p.x = p.xs = h; p.y = S().act_e; p.ys = S().act; p.glu = u; p.glus = us;
-            if (!rc) rc = done(moe_product_launch(p, s, L.pdl));
+            if (!rc) rc = done(moe_product_launch(p, s, L.dependent()));
             p.up = 0; p.w = W.down; p.ws = W.shared_down; p.out = p.outs = d_p; p.in = Y.ff_p; p.ins = Y.sff_p;
             p.x = S().act_e; p.xs = S().act; p.y = S().ye; p.ys = y;
-            return rc ? rc : done(moe_product_launch(p, s, L.pdl));
+            return rc ? rc : done(moe_product_launch(p, s, L.dependent()));
         }
         // tiles as wide as an expert's share of the round
         const int share = rows / (Y.d.experts + Y.d.identity);
         m.tile_rows = c->dt == LCU_F32 || share <= 64 ? 64 : (share <= 128 ? 128 : 256);
         m.max_tiles = moe_max_tiles(rows, Y.d.experts, m.tile_rows);
-        if (!rc) rc = done(moe_route_launch(m, s, L.pdl));
-        if (!rc) rc = done(moe_gather_launch(m, c->dt, s, L.pdl));
+        if (!rc) rc = done(moe_route_launch(m, s, L.dependent()));
+        if (!rc) rc = done(moe_gather_launch(m, c->dt, s, L.dependent()));
         auto grouped = [&](const void *w, int in, int out, const void *x, void *y, int stride_y, int epilogue) -> int {
             if (c->dt == LCU_F32) {
                 LinearF32Args a{};
@@ -233,7 +233,7 @@ struct PreNormRound {
             GemvArgs a{};
             a.w = w; a.x = x; a.stride_x = in; a.n_tok = rows; a.in = in; a.out = out; a.epilogue = epilogue; a.y = y; a.stride_y = stride_y; a.glu = u;
             a.tiles = m.tiles; a.n_tiles = m.max_tiles; a.tile_rows = m.tile_rows; a.groups = Y.d.experts; a.row_scale = in_scale;
-            return done(gemm_tc_launch(a, c->dt, s, L.pdl));
+            return done(gemm_tc_launch(a, c->dt, s, L.dependent()));
         };
         if (!rc) rc = grouped(W.up, d_p, 2 * Y.ff_p, S().xg, S().act_e, Y.ff_p, EPI_GLU);
         if (!rc) rc = grouped(W.down, Y.ff_p, d_p, S().act_e, S().ye, d_p, EPI_STORE_F32);
@@ -247,7 +247,7 @@ struct PreNormRound {
         if (Y.poly()) {
             rc = L.linear(W.up, S().d_p, Y.ff_p, h, r.n_tok, S().z, Y.ff_p, EPI_STORE_F32);
             const PolyNormArgs a{S().z, W.up_bias, W.act, S().act, r.n_tok, Y.d.ff, Y.ff_p, c->desc.eps};
-            if (!rc) rc = done(op_poly_norm(a, c->dt, s, L.pdl));
+            if (!rc) rc = done(op_poly_norm(a, c->dt, s, L.dependent()));
         } else {
             rc = L.linear(W.up, S().d_p, Y.ff_p, h, r.n_tok, S().act, Y.ff_p, EPI_RELU2);
         }
@@ -261,15 +261,45 @@ struct PreNormRound {
         if (Y.d.route_softmax) { u.weights = S().moe_w; u.ff_in = h; }
     }
 
+    // The feed-forward of a layer whose mixer reads the same x: on its own stream, so that the mixer's short steps run while weights
+    // stream, or ahead of the mixer.
+    bool forks() const { return S().side && tuning().stack_fork; }
+    void stream_scratch(bool side) const {
+        gemm_tc_set_scratch(side ? S().side_ws : c->sk_ws, c->sk_ws_bytes, side ? S().side_tickets : c->sk_tickets, 4096, c->dev_status);
+    }
+    int beside(const StackLayer &Y, const StackWeights &W) {
+        if (!forks()) return feed_forward(Y, W, S().h2, S().y2);
+        const cudaStream_t main = s;
+        LCU_CHECK_CUDA(cudaEventRecord(S().fork, main));
+        LCU_CHECK_CUDA(cudaStreamWaitEvent(S().side, S().fork, 0));
+        s = L.s = S().side;
+        L.joined = true;
+        stream_scratch(true);
+        const int rc = feed_forward(Y, W, S().h2, S().y2);
+        s = L.s = main;
+        L.joined = false;
+        stream_scratch(false);
+        LCU_CHECK_CUDA(cudaEventRecord(S().join, S().side));
+        return rc;
+    }
+    int joined(int rc) {
+        if (forks()) {
+            LCU_CHECK_CUDA(cudaStreamWaitEvent(s, S().join, 0));
+            L.joined = true;
+        }
+        return rc;
+    }
+
     int run() {
-        gemm_tc_set_scratch(c->sk_ws, c->sk_ws_bytes, c->sk_tickets, 4096, c->dev_status);
+        stream_scratch(false);
         int rc = residual_into(0, Outputs{});
         for (int l = 0; l < c->desc.n_layers && !rc; ++l) {
             const StackLayer &Y = S().layers[l];
             const StackWeights &W = S().w[Y.src];
             const bool both = Y.attention() && Y.recurrent();
-            if (Y.parallel()) rc = feed_forward(Y, W, S().h2, S().y2);
+            if (Y.parallel()) rc = beside(Y, W);
             if (!rc) rc = mixers(Y, W);
+            if (Y.parallel()) rc = joined(rc);
             if (rc) break;
             Outputs u;
             u.y0 = S().y; u.y1 = both ? S().y2 : nullptr; u.y_gain = both ? W.branch_norm : nullptr; u.post_gain = W.post1;

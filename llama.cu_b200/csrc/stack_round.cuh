@@ -40,6 +40,13 @@ struct Launcher {
     bool pdl;
     bool weights_first = false;  // one-token GEMVs of this round request weights before activations
     CapArgs cap{};               // of EPI_CAP and EPI_CAP_F32
+    bool joined = false;         // the next launch follows an event of another stream: no programmatic dependent
+
+    bool dependent() {
+        const bool r = pdl && !joined;
+        joined = false;
+        return r;
+    }
 
     // y[n, out] = x[n, in] W^T; x and bf16 y in the activation dtype, EPI_STORE_F32 into f32 rows
     int linear(const void *w, int in, int out, const void *x, int n, void *y, int stride_y, int epilogue, const float *act_pq = nullptr,
@@ -61,6 +68,7 @@ struct Launcher {
         for (int t0 = 0; t0 < n;) {
             const int most = tc ? (tuning().tc_block < 256 ? tuning().tc_block : GEMM_TC_MAX_TOKENS) : gemv_max_tokens(in);
             const int nt = n - t0 < most ? n - t0 : most;
+            const bool pdl = dependent();
             GemvArgs a{};
             a.w = w;
             a.x = reinterpret_cast<const unsigned char *>(x) + (size_t)t0 * in * 2;

@@ -11,7 +11,7 @@ import numpy as np
 
 from . import (BF16, F16, F32, LINEAR_KINDS, Q8_0, W_ATTN_NORM, W_DOWN, W_EMBD, W_FFN_NORM, W_GATE_UP, W_LM_HEAD,
                W_O, W_OUT_NORM, W_QKV, Context, ModelDesc, check, load_library, stream_ptr)
-from . import galarax, mupuvik, zefedra
+from . import galarax, gunulorn, mupuvik, zefedra
 from .layered import LayeredConfig
 
 
@@ -77,6 +77,8 @@ CONFIGS["zefedra1b"] = zefedra.uniform("zefedra1b", 16, 2048, 16, 128, 128, 768,
 CONFIGS["galarax8b"] = galarax.uniform("galarax8b", 32, 4096, 32, 8, 128, 32, 16, 128, 128, 14336, 128256)
 CONFIGS["mupuvik8b"] = mupuvik.uniform("mupuvik8b", 32, 4096, 32, 8, 128, 1024, 128, 8, 128, 64, 16, 128, 256, 3584, 16, 2, 3584, 128256)
 CONFIGS["mupuvik1b"] = mupuvik.uniform("mupuvik1b", 16, 2048, 32, 8, 64, 512, 64, 1, 128, 64, 8, 128, 256, 2048, 16, 2, 2048, 128256)
+CONFIGS["gunulorn8b"] = gunulorn.uniform("gunulorn8b", 32, 4096, 32, 8, 128, 1024, 64, 14336, 3584, 16, 3, 4, 128256)
+CONFIGS["gunulorn1b"] = gunulorn.uniform("gunulorn1b", 16, 2048, 32, 8, 64, 512, 64, 8192, 2048, 16, 3, 4, 128256)
 CONFIGS["galarax1b"] = galarax.uniform("galarax1b", 16, 2048, 32, 8, 64, 16, 8, 128, 128, 8192, 128256)
 
 
