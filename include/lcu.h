@@ -333,7 +333,7 @@ LCU_API int lcu_set_wait_limit_us(lcu_ctx *ctx, long long us);
  * "rms_pdl" (0: the stand-alone RMSNorm of batched rounds is a plain launch), "expand_min" (latent attention: fewest tokens of
  * a portion that expands keys and values; 0 = from the operation counts, -1 = never), "latent_tc" (0: mma.sync kernel in decode
  * rounds), "stack_fuse" (0..2: norm prologues in one- and two-token rounds of layered models never, where faster, always), "stack_pdl" (0: plain launches in small rounds of layered models),
- * "stack_fork" (0..2: feed-forwards beside a mixer on a stream of their own never, where faster, always), "delta_tc" (0: the delta rule's scan of bf16 contexts on the f32 pipes), "stack_tc" (0..2: linear layers
+ * "stack_fork" (0: mixers beside a feed-forward run behind it, not on a stream of their own), "delta_tc" (0: the delta rule's scan of bf16 contexts on the f32 pipes), "stack_tc" (0..2: linear layers
  * of three- and four-token rounds of layered models on tcgen05 never, large ones, all).
  * `ctx` (may be NULL) drops its captured rounds.  A measurement aid without counterpart in the reference. */
 LCU_API int lcu_set_tuning(lcu_ctx *ctx, const char *key, long long value);

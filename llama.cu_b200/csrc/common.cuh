@@ -44,7 +44,7 @@ struct Tuning {
     int tc_cluster = 1;            // cluster split-K form of the tcgen05 kernel: 0 never, 1 where it measured faster, 2 wherever it applies
     int stack_pdl = 1;             // layered models, small rounds: every launch is a programmatic dependent of its predecessor
     int stack_fuse = 1;            // layered models, rounds of one or two decoded tokens: norms and residual as GEMV prologues (1: where it measured faster, 2: always)
-    int stack_fork = 1;            // feed-forwards beside a mixer on a stream of their own: 0 never, 1 where it measured faster, 2 always
+    int stack_fork = 1;            // mixers beside a feed-forward run on a stream of their own
     int latent_tc = 1;             // latent attention of decode rounds on tcgen05 (0: mma.sync kernel)
     int expand_min = 0;            // latent attention: fewest tokens of a portion that expands keys and values (0: by operation count, -1: never)
     int stack_tc = 1;              // layered models, rounds of three or four tokens: linear layers on tcgen05 (0: never, 1: large ones, 2: all)

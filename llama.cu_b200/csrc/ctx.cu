@@ -589,7 +589,7 @@ int lcu_set_tuning(lcu_ctx *c, const char *key, long long value) {
     else if (k == "tc_cluster") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: tc_cluster = %lld (0..2)", value); t.tc_cluster = (int)value; }
     else if (k == "stack_pdl") t.stack_pdl = value != 0;
     else if (k == "stack_fuse") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_fuse = %lld (0..2)", value); t.stack_fuse = (int)value; }
-    else if (k == "stack_fork") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_fork = %lld (0..2)", value); t.stack_fork = (int)value; }
+    else if (k == "stack_fork") t.stack_fork = value != 0;
     else if (k == "latent_tc") t.latent_tc = value != 0;
     else if (k == "stack_tc") { LCU_REQUIRE(value >= 0 && value <= 2, "set_tuning: stack_tc = %lld (0..2)", value); t.stack_tc = (int)value; }
     else if (k == "delta_tc") t.delta_tc = value != 0;

@@ -50,12 +50,12 @@ __global__ void __launch_bounds__(256, FORM == GQA_PREP ? 6 : (FORM == GQA_PREP_
     gqa_prep_block<T, FORM>(a, blockIdx.y, blockIdx.x * per, blockIdx.x * per + per);
 }
 
-template <class T, int TAPS>
-__global__ void __launch_bounds__(256, TAPS > 2 ? 2 : (TAPS ? 3 : 4)) gqa_prep_run_kernel(const GqaArgs a) {
+template <class T, int TAPS, int RUN>
+__global__ void __launch_bounds__(256, RUN == 1 ? 4 : (TAPS > 2 ? 2 : (TAPS ? 3 : 4))) gqa_prep_run_kernel(const GqaArgs a) {
     grid_dep_launch();
     const int item = blockIdx.x * 8 + (threadIdx.x >> 5);
     grid_dep_wait();
-    if (item < gqa_prep_items(a)) gqa_prep_run<T, TAPS>(a, blockIdx.y * GQA_RUN, item, threadIdx.x & 31);
+    if (item < gqa_prep_items(a)) gqa_prep_run<T, TAPS, RUN>(a, blockIdx.y * RUN, item, threadIdx.x & 31);
 }
 
 // Denominator and factor that end a row of softmax (scores in powers of two): maximum M, sum L over it.  A key without
@@ -626,19 +626,21 @@ int gqa_prep_launch(const GqaArgs &a, int dt, cudaStream_t s, bool pdl) {
         return LCU_OK;
     };
     const bool f32 = dt == LCU_F32;
-    if (gqa_prep_more(a) && a.n_tok >= 64 && gqa_prep_runs(a)) {
-        auto run = [&](auto kernel) -> int {
-            LCU_CHECK_CUDA(launch_kernel(kernel, dim3((gqa_prep_items(a) + 7) / 8, (a.n_tok + GQA_RUN - 1) / GQA_RUN), dim3(256), 0, s, pdl, a));
+    if (gqa_prep_more(a) && gqa_prep_runs(a)) {
+        const bool runs = a.n_tok >= 64;
+        auto run = [&](auto one, auto four) -> int {
+            const int n = runs ? 4 : 1;
+            LCU_CHECK_CUDA(launch_kernel(runs ? four : one, dim3((gqa_prep_items(a) + 7) / 8, (a.n_tok + n - 1) / n), dim3(256), 0, s, pdl, a));
             return LCU_OK;
         };
         auto by_taps = [&](auto t) -> int {
             using T = decltype(t);
             switch (a.conv ? a.taps : 0) {
-            case 0: return run(gqa_prep_run_kernel<T, 0>);
-            case 1: return run(gqa_prep_run_kernel<T, 1>);
-            case 2: return run(gqa_prep_run_kernel<T, 2>);
-            case 3: return run(gqa_prep_run_kernel<T, 3>);
-            default: return run(gqa_prep_run_kernel<T, 4>);
+            case 0: return run(gqa_prep_run_kernel<T, 0, 1>, gqa_prep_run_kernel<T, 0, 4>);
+            case 1: return run(gqa_prep_run_kernel<T, 1, 1>, gqa_prep_run_kernel<T, 1, 4>);
+            case 2: return run(gqa_prep_run_kernel<T, 2, 1>, gqa_prep_run_kernel<T, 2, 4>);
+            case 3: return run(gqa_prep_run_kernel<T, 3, 1>, gqa_prep_run_kernel<T, 3, 4>);
+            default: return run(gqa_prep_run_kernel<T, 4, 1>, gqa_prep_run_kernel<T, 4, 4>);
             }
         };
         return f32 ? by_taps(float{}) : by_taps(bf16{});

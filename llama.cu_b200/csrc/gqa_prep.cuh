@@ -168,14 +168,13 @@ __device__ __forceinline__ void gqa_prep_block(const GqaArgs &a, int t, int item
     }
 }
 
-// Large rounds of layers with these steps alone: rotation of neighbouring pairs, rotated values, factors per head, convolutions of
+// Layers with these steps alone: rotation of neighbouring pairs, rotated values, factors per head, convolutions of
 // at most four taps.  A warp takes one head of RUN tokens in a row and holds the rows its convolution needs; every row is requested
-// before the first is used.  TAPS 0: none.
-constexpr int GQA_RUN = 4;
+// before the first is used.  TAPS 0: no convolution.
 __host__ __device__ __forceinline__ bool gqa_prep_runs(const GqaArgs &a) {
     return !a.bias && !a.qk_norm && (a.rot_dims == 0 || a.rot_adjacent) && (!a.conv || a.taps <= 4);
 }
-template <class T, int TAPS>
+template <class T, int TAPS, int RUN>
 __device__ __forceinline__ void gqa_prep_run(const GqaArgs &a, int t0, int item, int lane) {
     constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;
     const bool is_v = item >= a.heads + a.kv_heads, is_q = item < a.heads;
@@ -187,16 +186,16 @@ __device__ __forceinline__ void gqa_prep_run(const GqaArgs &a, int t0, int item,
     const float temp = is_q && a.head_temp ? a.head_temp[head] : 1.f;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int d = 4 * lane; d < size_p; d += 128) {
-        float4 x[BACK + GQA_RUN], w[TAPS ? TAPS : 1];
+        float4 x[BACK + RUN], w[TAPS ? TAPS : 1];
 #pragma unroll
-        for (int i = 0; i < BACK + GQA_RUN; ++i) {
+        for (int i = 0; i < BACK + RUN; ++i) {
             const int t = t0 + i - BACK;
             x[i] = t >= 0 && t < a.n_tok ? *reinterpret_cast<const float4 *>(a.lat + (size_t)t * a.stride + off + d) : zero;
         }
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const float4 *>(a.conv + (size_t)j * a.channels() + off + d);
 #pragma unroll
-        for (int i = 0; i < GQA_RUN; ++i) {
+        for (int i = 0; i < RUN; ++i) {
             const int t = t0 + i;
             if (t >= a.n_tok) break;
             const int p = (int)a.pos[t], r = a.tok_req[t];

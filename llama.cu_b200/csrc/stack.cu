@@ -315,7 +315,9 @@ int stack_create(lcu_ctx *c, const lcu_layer_desc *layers) {
     S->h2 = p + o_h2; S->z = reinterpret_cast<float *>(p + o_z);
     S->side_ws = p + o_sw; S->side_tickets = reinterpret_cast<unsigned *>(p + o_st);
     if (any_parallel) {
-        LCU_CHECK_CUDA(cudaStreamCreateWithFlags(&S->side, cudaStreamNonBlocking));
+        int least = 0, greatest = 0;
+        LCU_CHECK_CUDA(cudaDeviceGetStreamPriorityRange(&least, &greatest));
+        LCU_CHECK_CUDA(cudaStreamCreateWithPriority(&S->side, cudaStreamNonBlocking, greatest));
         LCU_CHECK_CUDA(cudaEventCreateWithFlags(&S->fork, cudaEventDisableTiming));
         LCU_CHECK_CUDA(cudaEventCreateWithFlags(&S->join, cudaEventDisableTiming));
     }

@@ -103,7 +103,7 @@ struct Stack {
     std::vector<RotTable> rot_tables;  // layers with the same rotation share one
     void *h2 = nullptr;                // input of a feed-forward beside a mixer
     float *z = nullptr;                // f32 rows of the up projection (LCU_ACT_POLYNORM)
-    // feed-forwards beside a mixer: a stream of their own between two events, with scratch for its linear layers
+    // mixers beside a feed-forward: a stream of their own between two events, with scratch for its linear layers
     cudaStream_t side = nullptr;
     cudaEvent_t fork = nullptr, join = nullptr;
     void *side_ws = nullptr;

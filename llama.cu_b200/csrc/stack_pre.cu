@@ -261,34 +261,33 @@ struct PreNormRound {
         if (Y.d.route_softmax) { u.weights = S().moe_w; u.ff_in = h; }
     }
 
-    // The feed-forward of a layer whose mixer reads the same x: on its own stream, so that the mixer's short steps run while weights
-    // stream, or ahead of the mixer.
-    bool forks() const { return S().side && tuning().stack_fork; }
     void stream_scratch(bool side) const {
         gemm_tc_set_scratch(side ? S().side_ws : c->sk_ws, c->sk_ws_bytes, side ? S().side_tickets : c->sk_tickets, 4096, c->dev_status);
     }
-    int beside(const StackLayer &Y, const StackWeights &W) {
-        if (!forks()) return feed_forward(Y, W, S().h2, S().y2);
+    // Mixer and feed-forward of one x: one after the other, or the mixer on a stream of its own, of higher priority, so that its short
+    // steps run while the feed-forward's weights stream.
+    int both(const StackLayer &Y, const StackWeights &W) {
+        if (!forks()) {
+            const int rc = feed_forward(Y, W, S().h2, S().y2);
+            return rc ? rc : mixers(Y, W);
+        }
         const cudaStream_t main = s;
         LCU_CHECK_CUDA(cudaEventRecord(S().fork, main));
         LCU_CHECK_CUDA(cudaStreamWaitEvent(S().side, S().fork, 0));
         s = L.s = S().side;
         L.joined = true;
         stream_scratch(true);
-        const int rc = feed_forward(Y, W, S().h2, S().y2);
+        int rc = mixers(Y, W);
         s = L.s = main;
         L.joined = false;
         stream_scratch(false);
         LCU_CHECK_CUDA(cudaEventRecord(S().join, S().side));
+        if (!rc) rc = feed_forward(Y, W, S().h2, S().y2);
+        LCU_CHECK_CUDA(cudaStreamWaitEvent(main, S().join, 0));
+        L.joined = true;
         return rc;
     }
-    int joined(int rc) {
-        if (forks()) {
-            LCU_CHECK_CUDA(cudaStreamWaitEvent(s, S().join, 0));
-            L.joined = true;
-        }
-        return rc;
-    }
+    bool forks() const { return S().side && tuning().stack_fork; }
 
     int run() {
         stream_scratch(false);
@@ -296,14 +295,12 @@ struct PreNormRound {
         for (int l = 0; l < c->desc.n_layers && !rc; ++l) {
             const StackLayer &Y = S().layers[l];
             const StackWeights &W = S().w[Y.src];
-            const bool both = Y.attention() && Y.recurrent();
-            if (Y.parallel()) rc = beside(Y, W);
-            if (!rc) rc = mixers(Y, W);
-            if (Y.parallel()) rc = joined(rc);
+            const bool pair = Y.attention() && Y.recurrent();
+            rc = Y.parallel() ? both(Y, W) : mixers(Y, W);
             if (rc) break;
             Outputs u;
-            u.y0 = S().y; u.y1 = both ? S().y2 : nullptr; u.y_gain = both ? W.branch_norm : nullptr; u.post_gain = W.post1;
-            if (both && Y.d.post_norm) { u.scale0 = Y.d.out_scale; u.scale1 = Y.d.out_scale2; }
+            u.y0 = S().y; u.y1 = pair ? S().y2 : nullptr; u.y_gain = pair ? W.branch_norm : nullptr; u.post_gain = W.post1;
+            if (pair && Y.d.post_norm) { u.scale0 = Y.d.out_scale; u.scale1 = Y.d.out_scale2; }
             if (Y.parallel()) {
                 if (!Y.d.experts) u.y1 = S().y2;
                 add_ff(u, Y, W, S().h2);

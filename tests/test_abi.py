@@ -98,7 +98,7 @@ def test_tuning_keys_are_validated(L):
     """lcu_set_tuning accepts the documented keys (restoring their defaults here) and refuses anything else; it needs
     neither a context nor a GPU."""
     defaults = {"pdl_edges": -1, "gemv_ctas_per_sm": 2, "q8_rows": 4, "gemv_lean_norm": 1, "rms_pdl": 1, "tc": 1,
-                "tc_block": 256, "tc_cluster": 1, "expand_min": 0, "stack_pdl": 1, "stack_fuse": 1, "latent_tc": 1, "delta_tc": 1, "stack_tc": 1, "p2p_scatter_ranks": 8, "p2p_scatter_min": 131072}
+                "tc_block": 256, "tc_cluster": 1, "expand_min": 0, "stack_pdl": 1, "stack_fuse": 1, "stack_fork": 1, "latent_tc": 1, "delta_tc": 1, "stack_tc": 1, "p2p_scatter_ranks": 8, "p2p_scatter_min": 131072}
     for key, value in defaults.items():
         L.set_tuning(key, value)
     with pytest.raises(L.LcuError):

@@ -20,7 +20,7 @@ LAYERS = {"conv": M.conv(), "window": M.window(), "dense": M.window(mlp=M.dense(
 @pytest.fixture(autouse=True)
 def default_tuning(L):
     yield
-    for k, v in (("stack_pdl", 1), ("stack_tc", 1), ("tc_block", 256), ("tc_cluster", 1)):
+    for k, v in (("stack_pdl", 1), ("stack_fork", 1), ("stack_tc", 1), ("tc_block", 256), ("tc_cluster", 1)):
         L.set_tuning(k, v)
 
 
@@ -349,7 +349,7 @@ def test_slots_and_pages_carry_nothing_over(L, mixed, dt):
     ctx.close()
 
 
-@pytest.mark.parametrize("key,value", [("stack_pdl", 0), ("stack_tc", 0), ("stack_tc", 2), ("tc_block", 64), ("tc_cluster", 0), ("tc_cluster", 2)])
+@pytest.mark.parametrize("key,value", [("stack_pdl", 0), ("stack_fork", 0), ("stack_tc", 0), ("stack_tc", 2), ("tc_block", 64), ("tc_cluster", 0), ("tc_cluster", 2)])
 def test_every_form_of_a_round(L, key, value):
     """The alternatives behind the tuning keys compute the same: prompts, then one to four requests decode together."""
     raw = M.config([M.window(50, 20, heads=20, kv_heads=5, mlp=M.dense(200)), M.conv(heads=20, kv_heads=5), M.window(100, 5), M.conv(heads=20, kv_heads=5, kv_from=1, mlp=None)])
